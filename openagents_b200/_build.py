@@ -27,6 +27,17 @@ NVCC_FLAGS += ["-D" + d for d in os.environ.get("B200_NVCC_DEFINES", "").replace
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fopenmp", "-Wall", "-Wno-unused-function", "-ffp-contract=off"]
 
 
+# Kernels whose results are specified in IEEE 32-bit arithmetic (accurate division, roots, exponentials): no fast math.
+PRECISE = ("kernels/hybrid_ops.cu", "kernels/linear_attn.cu")
+
+# Parts of the libraries that stand on their own, for a process that serves one model family from a tree without built files.
+SUBSETS = {
+    "hybrid": {"host": ("kv/kv_alloc.cpp",),
+               "cuda": ("kernels/attn_decode.cu", "kernels/attn_prefill_tc05.cu", "kernels/decode_ops.cu", "kernels/gemm_tc05.cu",
+                        "kernels/hybrid_ops.cu", "kernels/linear_attn.cu", "kernels/matvec.cu")},
+}
+
+
 def _sources(sub: str, exts: tuple[str, ...]) -> list[Path]:
     root = CSRC / sub
     return sorted(p for p in root.rglob("*") if p.suffix in exts)
@@ -65,6 +76,16 @@ def _digest(paths: list[Path], flags: list[str]) -> str:
     return h.hexdigest()
 
 
+def _flags_for(src: Path, flags: list[str]) -> list[str]:
+    if str(src.relative_to(CSRC)) in PRECISE:
+        return [f for f in flags if f != "--use_fast_math"]
+    return flags
+
+
+def _subset(srcs: list[Path], kind: str, subset: str | None) -> list[Path]:
+    return srcs if subset is None else [s for s in srcs if str(s.relative_to(CSRC)) in SUBSETS[subset][kind]]
+
+
 def _run(cmd: list[str]) -> None:
     r = subprocess.run(cmd, capture_output=True, text=True)
     if r.returncode != 0:
@@ -82,14 +103,15 @@ def _compile_objects(srcs: list[Path], compiler: list[str], flags: list[str], ta
     for s in srcs:
         obj = objdir / (tag + "_" + "_".join(s.relative_to(CSRC).with_suffix("").parts) + ".o")
         stamp = obj.with_suffix(".stamp")
-        want = _digest([s] + hdrs, compiler + flags)
+        own = _flags_for(s, flags)
+        want = _digest([s] + hdrs, compiler + own)
         objs.append(obj)
         if obj.exists() and stamp.exists() and stamp.read_text() == want:
             continue
-        jobs.append((s, obj, stamp, want))
+        jobs.append((s, obj, stamp, want, own))
     def one(job):
-        s, obj, stamp, want = job
-        _run(compiler + flags + ["-I", str(CSRC), "-c", str(s), "-o", str(obj)])
+        s, obj, stamp, want, own = job
+        _run(compiler + own + ["-I", str(CSRC), "-c", str(s), "-o", str(obj)])
         stamp.write_text(want)
     if jobs:
         with cf.ThreadPoolExecutor(max_workers=min(len(jobs), os.cpu_count() or 4)) as ex:
@@ -106,31 +128,31 @@ def _link(objs: list[Path], out: Path, linker: list[str], extra: list[str]) -> N
     stamp.write_text(want)
 
 
-def host_lib_path() -> Path:
-    return LIB / "libb200_host.so"
+def host_lib_path(subset: str | None = None) -> Path:
+    return LIB / ("libb200_host.so" if subset is None else f"libb200_host_{subset}.so")
 
 
-def cuda_lib_path() -> Path:
-    return LIB / "libb200_cuda.so"
+def cuda_lib_path(subset: str | None = None) -> Path:
+    return LIB / ("libb200_cuda.so" if subset is None else f"libb200_cuda_{subset}.so")
 
 
 def node_cli_path() -> Path:
     return LIB / "b200-node"
 
 
-def build_host() -> Path:
-    objs = _compile_objects(host_sources(), ["g++"], CXX_FLAGS, "host")
-    _link(objs, host_lib_path(), ["g++", "-shared", "-fopenmp"], [])
-    return host_lib_path()
+def build_host(subset: str | None = None) -> Path:
+    objs = _compile_objects(_subset(host_sources(), "host", subset), ["g++"], CXX_FLAGS, "host")
+    _link(objs, host_lib_path(subset), ["g++", "-shared", "-fopenmp"], [])
+    return host_lib_path(subset)
 
 
-def build_cuda() -> Path:
+def build_cuda(subset: str | None = None) -> Path:
     nvcc = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
     if not Path(nvcc).exists():
         raise RuntimeError("nvcc not found; the CUDA library cannot be built")
-    objs = _compile_objects(cuda_sources(), [nvcc], NVCC_ARCH + NVCC_FLAGS, "cuda")
-    _link(objs, cuda_lib_path(), [nvcc, "-shared"] + NVCC_ARCH, ["-lcudart_static", "-ldl", "-lrt", "-lpthread"])
-    return cuda_lib_path()
+    objs = _compile_objects(_subset(cuda_sources(), "cuda", subset), [nvcc], NVCC_ARCH + NVCC_FLAGS, "cuda")
+    _link(objs, cuda_lib_path(subset), [nvcc, "-shared"] + NVCC_ARCH, ["-lcudart_static", "-ldl", "-lrt", "-lpthread"])
+    return cuda_lib_path(subset)
 
 
 def build_node() -> Path | None:
@@ -156,21 +178,21 @@ def build_all(verbose: bool = False) -> dict[str, str]:
     return out
 
 
-def is_stale(kind: str) -> bool:
+def is_stale(kind: str, subset: str | None = None) -> bool:
     """True when the library of that kind is missing or older than its sources."""
     try:
         if kind == "host":
-            srcs, comp, flags, out = host_sources(), ["g++"], CXX_FLAGS, host_lib_path()
+            srcs, comp, flags, out = _subset(host_sources(), "host", subset), ["g++"], CXX_FLAGS, host_lib_path(subset)
         else:
             nvcc = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
-            srcs, comp, flags, out = cuda_sources(), [nvcc], NVCC_ARCH + NVCC_FLAGS, cuda_lib_path()
+            srcs, comp, flags, out = _subset(cuda_sources(), "cuda", subset), [nvcc], NVCC_ARCH + NVCC_FLAGS, cuda_lib_path(subset)
         if not out.exists():
             return True
         hdrs = _headers()
         for s in srcs:
             obj = LIB / "obj" / (kind + "_" + "_".join(s.relative_to(CSRC).with_suffix("").parts) + ".o")
             stamp = obj.with_suffix(".stamp")
-            if not stamp.exists() or stamp.read_text() != _digest([s] + hdrs, comp + flags):
+            if not stamp.exists() or stamp.read_text() != _digest([s] + hdrs, comp + _flags_for(s, flags)):
                 return True
         return False
     except Exception:

@@ -52,7 +52,8 @@ int make_tmap_2d(CUtensorMap* map, const void* base, int elem_bytes, uint64_t ro
 
 // ACT_SWIGLU_PAIR: B rows are interleaved (gate_0, up_0, gate_1, ...); the epilogue writes
 // silu(gate) * up as bf16, N / 2 values per row of out_bf16 (row stride ldc), nothing else.
-enum { ACT_NONE = 0, ACT_GELU = 1, ACT_SWIGLU_PAIR = 2 };
+// ACT_RELU2: the square of relu.
+enum { ACT_NONE = 0, ACT_GELU = 1, ACT_SWIGLU_PAIR = 2, ACT_RELU2 = 3 };
 
 struct GemmEpi {
   float* out_f32;            // either or both outputs
@@ -212,6 +213,7 @@ __device__ __forceinline__ void epilogue_col(const GemmEpi& e, int n, int t0, in
       continue;
     }
     if (e.act == ACT_GELU) x = gelu_tanh(x);
+    else if (e.act == ACT_RELU2) x = x > 0.f ? x * x : 0.f;
     if (e.resid_f32) x += e.resid_f32[idx];
     if (e.resid_bf16) x += __bfloat162float(e.resid_bf16[idx]);
     if (e.out_f32) e.out_f32[idx] = e.accumulate ? e.out_f32[idx] + x : x;
@@ -285,6 +287,9 @@ __device__ __forceinline__ void epilogue_row(const GemmEpi& e, int m, int n0, in
     if (e.act == ACT_GELU) {
 #pragma unroll
       for (int j = 0; j < 32; j++) v[j] = gelu_tanh(v[j]);
+    } else if (e.act == ACT_RELU2) {
+#pragma unroll
+      for (int j = 0; j < 32; j++) v[j] = v[j] > 0.f ? v[j] * v[j] : 0.f;
     }
     if (e.resid_f32) {
 #pragma unroll
@@ -334,6 +339,7 @@ __device__ __forceinline__ void epilogue_row(const GemmEpi& e, int m, int n0, in
       float x = v[j];
       if (e.bias) x += e.bias[n0 + j];
       if (e.act == ACT_GELU) x = gelu_tanh(x);
+      else if (e.act == ACT_RELU2) x = x > 0.f ? x * x : 0.f;
       if (e.resid_f32) x += e.resid_f32[base + j];
       if (e.resid_bf16) x += __bfloat162float(e.resid_bf16[base + j]);
       if (e.out_f32) e.out_f32[base + j] = e.accumulate ? e.out_f32[base + j] + x : x;

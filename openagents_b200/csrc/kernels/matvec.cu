@@ -13,7 +13,7 @@
 using namespace b200;
 
 enum { WT_Q4KR = 0, WT_Q6KR = 1, WT_Q8R = 2, WT_BF16 = 3 };
-enum { EPI_STORE = 0, EPI_RESID = 1, EPI_SWIGLU_Q8 = 2, EPI_SWIGLU_F32 = 3, EPI_ALLREDUCE = 4, EPI_ROPE_KV = 5 };
+enum { EPI_STORE = 0, EPI_RESID = 1, EPI_SWIGLU_Q8 = 2, EPI_SWIGLU_F32 = 3, EPI_ALLREDUCE = 4, EPI_ROPE_KV = 5, EPI_RELU2 = 6 };
 
 struct MatvecArgs {
   const uint8_t* w;     // main plane
@@ -226,6 +226,8 @@ __device__ __forceinline__ void matvec_epilogue(const MatvecArgs& a, const float
       float v2 = res[32 * B + lane * B + b] + (a.bias ? a.bias[2 * n + 1] : 0.f);
       a.y[(size_t)b * a.ldy + a.N + n] = v2;
     }
+  } else if (a.epi == EPI_RELU2) {
+    if (live) a.y[(size_t)b * a.ldy + n] = v > 0.f ? v * v : 0.f;
   } else if (a.epi == EPI_RESID) {
     if (live) a.y[(size_t)b * a.ldy + n] = a.resid[(size_t)b * a.ldy + n] + v;
   } else if (a.epi == EPI_ALLREDUCE) {

@@ -19,6 +19,7 @@ namespace {
 struct Seq {
   std::vector<int32_t> pages;
   int64_t n_tokens = 0;
+  int32_t slot = -1;            // recurrent-state slot (pools of models with recurrent layers)
   std::vector<uint64_t> chain;  // hash of each full page's prefix chain, parallel to pages
 };
 
@@ -39,6 +40,10 @@ struct Pool {
   std::vector<uint8_t> is_retained;
   bool retain = true;                  // off: a page nobody holds leaves the index at once (prefix hits among live sequences only)
   std::unordered_map<int64_t, Seq> seqs;
+  // Models with recurrent layers keep one fixed-size state per sequence: a slot is taken when a sequence begins and given back
+  // when it ends.  0 slots = the model has no recurrent state.
+  int32_t n_slots = 0;
+  std::vector<int32_t> free_slots;
   uint64_t hits = 0, lookups = 0;
 };
 
@@ -145,10 +150,18 @@ uint64_t b200_kv_prefix_lookups(void* h) { return ((Pool*)h)->lookups; }
 // Start a sequence.  If `tokens` is given, full pages whose prefix chain is already cached are
 // shared; returns the number of tokens covered by shared pages (a multiple of the page size, and
 // always less than n_tokens so at least one token is left to compute), or -1 if the id is in use.
+// Pools with state slots: the sequence takes one (-2 if none is free; nothing has changed then) and shares no pages,
+// because the state after the shared tokens is not kept.
 int64_t b200_kv_seq_begin(void* h, int64_t seq_id, const int32_t* tokens, int64_t n_tokens) {
   Pool* p = (Pool*)h;
   if (p->seqs.count(seq_id)) return -1;
+  if (p->n_slots > 0 && p->free_slots.empty()) return -2;
   Seq& s = p->seqs[seq_id];
+  if (p->n_slots > 0) {
+    s.slot = p->free_slots.back();
+    p->free_slots.pop_back();
+    return 0;
+  }
   if (!tokens) return 0;
   uint64_t chain = 0;
   int64_t full = (n_tokens - 1) / p->page_size;  // leave the last token uncached
@@ -189,7 +202,7 @@ int32_t b200_kv_seq_extend(void* h, int64_t seq_id, int64_t n_new) {
 void b200_kv_seq_publish(void* h, int64_t seq_id, const int32_t* tokens, int64_t n_tokens) {
   Pool* p = (Pool*)h;
   auto it = p->seqs.find(seq_id);
-  if (it == p->seqs.end()) return;
+  if (it == p->seqs.end() || p->n_slots > 0) return;
   Seq& s = it->second;
   if (n_tokens > s.n_tokens) n_tokens = s.n_tokens;
   int64_t full = n_tokens / p->page_size;
@@ -320,7 +333,29 @@ void b200_kv_seq_end(void* h, int64_t seq_id) {
   auto it = p->seqs.find(seq_id);
   if (it == p->seqs.end()) return;
   for (int32_t pg : it->second.pages) release_page(p, pg);
+  if (it->second.slot >= 0) p->free_slots.push_back(it->second.slot);
   p->seqs.erase(it);
+}
+
+// Give the pool `n` recurrent-state slots (before the first sequence begins).  Returns 0, or -1 when sequences exist.
+int32_t b200_kv_set_slots(void* h, int32_t n) {
+  Pool* p = (Pool*)h;
+  if (!p->seqs.empty() || n < 0) return -1;
+  p->n_slots = n;
+  p->free_slots.clear();
+  for (int32_t i = n - 1; i >= 0; i--) p->free_slots.push_back(i);
+  return 0;
+}
+int32_t b200_kv_free_slots(void* h) { return (int32_t)((Pool*)h)->free_slots.size(); }
+// State slots of B sequences into `out`; -1 for an unknown sequence (returned, nothing else written past it).
+int32_t b200_kv_seq_slots(void* h, const int64_t* seq_ids, int32_t B, int32_t* out) {
+  Pool* p = (Pool*)h;
+  for (int32_t b = 0; b < B; b++) {
+    auto it = p->seqs.find(seq_ids[b]);
+    if (it == p->seqs.end()) return -1;
+    out[b] = it->second.slot;
+  }
+  return 0;
 }
 
 }  // extern "C"

@@ -6,12 +6,56 @@ The presets are the shapes the benchmark configurations name; the server detects
 """
 from __future__ import annotations
 
+import json
 from dataclasses import asdict, dataclass, replace
 
 
 @dataclass(frozen=True)
+class MixerSpec:
+    """What mixes tokens in one layer of a hybrid stack.  ``kind`` "attention": softmax attention over the paged cache;
+    "gla": gated linear attention with a decay per key channel and a state slot per sequence."""
+    kind: str
+    heads: int
+    dim: int                       # per-head query / key size
+    vdim: int                      # per-head value size
+    # attention
+    kv_heads: int = 0
+    scale: float = 1.0             # multiplies q . k
+    rope_base: float = 10000.0
+    rope_dims: int = 0             # leading dimensions of a head that rotate
+    rope_style: str = "pairs"
+    qk_norm: bool = False          # q and k divided by their root mean square per head, after the rotation
+    head_gate: bool = False        # one sigmoid gate per head on the output
+    kv_from: int | None = None     # this layer reads the keys and values of an earlier one
+    # gla
+    tau: float = 1.0               # decay = sigmoid(z)^(1/tau)
+    rank: int = 16                 # rank of the decay's projection
+
+    def __post_init__(self):
+        if self.kind not in ("attention", "gla"):
+            raise ValueError(f"unknown mixer {self.kind!r}")
+        if min(self.heads, self.dim, self.vdim) < 1:
+            raise ValueError("a mixer's heads and sizes must be positive")
+        if self.kind == "attention":
+            if self.kv_heads < 1 or self.heads % self.kv_heads:
+                raise ValueError("the key/value heads must divide the query heads")
+            if not 0 <= self.rope_dims <= self.dim or self.rope_dims % 2:
+                raise ValueError("the rotated dimensions must be even and within the head")
+        elif self.tau == 0:
+            raise ValueError("tau must not be zero")
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    """One layer of a hybrid stack: a mixer and, unless ``ffn`` is 0, a feed-forward of that width; a norm before and behind each."""
+    mixer: MixerSpec
+    ffn: int = 0
+    act: str = "relu2"             # the square of relu
+
+
+@dataclass(frozen=True)
 class ModelConfig:
-    arch: str = "llama"            # llama | gpt2 | gpt-oss
+    arch: str = "llama"            # llama | gpt2 | gpt-oss | folirax
     n_layers: int = 2
     d_model: int = 256
     n_heads: int = 4
@@ -31,6 +75,10 @@ class ModelConfig:
     swa_every: int = 2             # layer i uses the window when sliding_window > 0 and i % swa_every == 0
     attn_sinks: bool = False
     qkv_bias: bool = False
+    # hybrid stacks: the layers one by one (the flat head and width fields above then hold the largest of each)
+    layers: tuple[LayerSpec, ...] = ()
+    logit_scale: float = 1.0
+    logit_softcap: float = 0.0     # 0 = none
     name: str = "tiny-llama"
 
     @property
@@ -44,8 +92,22 @@ class ModelConfig:
     def layer_uses_window(self, i: int) -> bool:
         return self.sliding_window > 0 and i % self.swa_every == 0
 
+    @property
+    def has_state(self) -> bool:
+        """Whether some layer carries a recurrent state from token to token."""
+        return any(l.mixer.kind == "gla" for l in self.layers)
+
     def n_params(self) -> int:
         d, f, v = self.d_model, self.ffn, self.vocab
+        if self.layers:
+            from .weights import tensor_specs
+            n = 0
+            for s in tensor_specs(self):
+                k = 1
+                for e in s.shape:
+                    k *= e
+                n += k
+            return n
         if self.arch == "gpt2":
             per = 4 * d * d + 2 * d * f + 9 * d + f
             return self.n_layers * per + v * d + self.context * d + 2 * d
@@ -56,6 +118,9 @@ class ModelConfig:
 
     def to_gguf_metadata(self) -> dict:
         a = self.arch
+        if self.layers:
+            return {"general.architecture": a, "general.name": self.name, f"{a}.context_length": self.context,
+                    "b200.model_json": json.dumps(hybrid_to_json(self))}
         md = {
             "general.architecture": a,
             "general.name": self.name,
@@ -85,6 +150,10 @@ class ModelConfig:
     @staticmethod
     def from_gguf_metadata(md: dict) -> "ModelConfig":
         a = md.get("general.architecture")
+        own = md.get("b200.model_json")
+        if own:
+            return config_from_json(json.loads(own if isinstance(own, str) else bytes(own).decode()), name=md.get("general.name", a),
+                                    context=int(md.get(f"{a}.context_length", HYBRID_CONTEXT)))
         if a not in ("llama", "gpt2", "gpt-oss"):
             raise ValueError(f"unsupported architecture {a!r}")
         g = lambda k, dflt=None: md.get(f"{a}.{k}", dflt)
@@ -112,6 +181,94 @@ class ModelConfig:
         return asdict(self)
 
 
+# ------------------------------------------------------------------ configurations given as JSON
+HYBRID_CONTEXT = 1 << 20           # such a file names no limit; the engine's cache sets it
+
+
+def _need(d: dict, key: str, kind, where: str):
+    v = d.get(key) if isinstance(d, dict) else None
+    if kind is float:
+        ok = isinstance(v, (int, float)) and not isinstance(v, bool)
+    else:
+        ok = isinstance(v, kind) and not isinstance(v, bool)
+    if not ok:
+        raise ValueError(f"config: {where}{key} must be {'a number' if kind is float else kind.__name__}")
+    return float(v) if kind is float else v
+
+
+def _folirax(c: dict, ranks: dict[int, int], name: str, context: int) -> ModelConfig:
+    """Folirax: attention (rotated, then unit-RMS queries and keys, a sigmoid gate per head, keys and values optionally those of an
+    earlier layer) and gated linear attention in any order, a norm on both sides of every sublayer, squared-relu
+    feed-forwards, scaled and soft-capped logits."""
+    layers = []
+    for i, e in enumerate(_need(c, "layers", list, "")):
+        w = f"layers[{i}]."
+        mx, kind = _need(e, "mixer", dict, w), _need(e, "type", str, w)
+        w2 = w + "mixer."
+        common = dict(heads=_need(mx, "heads", int, w2), dim=_need(mx, "dim", int, w2), vdim=_need(mx, "vdim", int, w2))
+        if kind == "gla":
+            m = MixerSpec("gla", **common, tau=_need(mx, "tau", float, w2), rank=ranks.get(i, MixerSpec.rank))
+        elif kind == "attention":
+            rot, src = _need(mx, "rot", dict, w2), mx.get("kv_from")
+            m = MixerSpec("attention", **common, kv_heads=_need(mx, "kv_heads", int, w2), scale=_need(mx, "scale", float, w2),
+                          rope_base=_need(rot, "base", float, w2 + "rot."), rope_dims=_need(rot, "dims", int, w2 + "rot."),
+                          qk_norm=True, head_gate=True, kv_from=None if src is None else _need(mx, "kv_from", int, w2))
+            if src is not None:
+                if not 0 <= src < i or layers[src].mixer.kind != "attention" or layers[src].mixer.kv_from is not None:
+                    raise ValueError(f"config: {w2}kv_from must name an earlier attention layer with keys and values of its own")
+                o = layers[src].mixer
+                if (o.kv_heads, o.dim, o.vdim) != (m.kv_heads, m.dim, m.vdim):
+                    raise ValueError(f"config: {w2}kv_from names a layer with other key/value sizes")
+        else:
+            raise ValueError(f"config: {w}type {kind!r} is not a mixer of this design")
+        mlp = e.get("mlp")
+        if mlp is not None and _need(mlp, "kind", str, w + "mlp.") != "dense":
+            raise ValueError(f"config: {w}mlp.kind {mlp['kind']!r} is not known")
+        layers.append(LayerSpec(m, 0 if mlp is None else _need(mlp, "ff", int, w + "mlp.")))
+    if not layers:
+        raise ValueError("config: layers is empty")
+    mx = [l.mixer for l in layers]
+    cap = c.get("logit_softcap")
+    return ModelConfig(arch="folirax", n_layers=len(layers), d_model=_need(c, "width", int, ""), vocab=_need(c, "vocab", int, ""),
+                       n_heads=max(m.heads for m in mx), n_kv_heads=max(1, *(m.kv_heads for m in mx)), head_dim=max(m.dim for m in mx),
+                       ffn=max(l.ffn for l in layers), context=context, norm_eps=_need(_need(c, "norm", dict, ""), "eps", float, "norm."),
+                       layers=tuple(layers), logit_scale=_need(c, "logit_scale", float, ""),
+                       logit_softcap=0.0 if cap is None else _need(c, "logit_softcap", float, ""), name=name)
+
+
+def hybrid_to_json(cfg: ModelConfig) -> dict:
+    """The inverse of ``config_from_json``."""
+    layers = []
+    for l in cfg.layers:
+        m = l.mixer
+        mx = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim}
+        if m.kind == "gla":
+            mx.update(tau=m.tau)
+        else:
+            mx.update(kv_heads=m.kv_heads, scale=m.scale, rot={"base": m.rope_base, "dims": m.rope_dims})
+            if m.kv_from is not None:
+                mx["kv_from"] = m.kv_from
+        layers.append({"type": m.kind, "mixer": mx, "mlp": {"kind": "dense", "ff": l.ffn} if l.ffn else None})
+    return {"architecture": "Folirax", "layers": layers, "width": cfg.d_model, "vocab": cfg.vocab, "norm": {"eps": cfg.norm_eps},
+            "logit_scale": cfg.logit_scale, "logit_softcap": cfg.logit_softcap,
+            "ranks": {str(i): l.mixer.rank for i, l in enumerate(cfg.layers) if l.mixer.kind == "gla"}}
+
+
+JSON_ARCHITECTURES = {"Folirax": _folirax}
+
+
+def config_from_json(c: dict, ranks: dict[int, int] | None = None, name: str | None = None, context: int = HYBRID_CONTEXT) -> ModelConfig:
+    """A model configuration from a checkpoint folder's config.json.  ``ranks``: sizes the file leaves to the tensors' shapes (rank
+    of the decay projection by layer)."""
+    arch = _need(c, "architecture", str, "")
+    reader = JSON_ARCHITECTURES.get(arch)
+    if reader is None:
+        raise ValueError(f"unsupported architecture {arch!r}")
+    if ranks is None:
+        ranks = {int(k): int(v) for k, v in c.get("ranks", {}).items()}
+    return reader(c, ranks, name or arch.lower(), context)
+
+
 TINY_LLAMA = ModelConfig()
 LLAMA3_8B = ModelConfig(arch="llama", n_layers=32, d_model=4096, n_heads=32, n_kv_heads=8, head_dim=128,
                         ffn=14336, vocab=128256, context=8192, rope_theta=500000.0, name="llama-3-8b-shape")
@@ -125,4 +282,26 @@ GPT_OSS_20B = ModelConfig(arch="gpt-oss", n_layers=24, d_model=2880, n_heads=64,
                           n_experts=32, top_k=4, sliding_window=128, swa_every=2, attn_sinks=True,
                           name="gpt-oss-20b-shape")
 
-PRESETS = {c.name: c for c in (TINY_LLAMA, LLAMA3_8B, LLAMA3_70B, GPT2_SMALL, GPT_OSS_20B)}
+
+
+def folirax_stack(width: int, ffn: int, vocab: int, groups: int, heads: int, kv_heads: int, head_dim: int, gla_heads: int, gla_dim: int,
+                  gla_vdim: int, name: str, ratio: int = 2) -> ModelConfig:
+    """A regular stack: ``groups`` times (``ratio`` recurrent layers, then an attention layer with keys and values of its own and one
+    that shares them)."""
+    gla = LayerSpec(MixerSpec("gla", gla_heads, gla_dim, gla_vdim, tau=16.0), ffn)
+    own = MixerSpec("attention", heads, head_dim, head_dim, kv_heads=kv_heads, scale=head_dim ** -0.5, rope_dims=head_dim // 2, qk_norm=True,
+                    head_gate=True)
+    layers: list[LayerSpec] = []
+    for _ in range(groups):
+        layers += [gla] * ratio
+        layers += [LayerSpec(own, ffn), LayerSpec(replace(own, kv_from=len(layers)), ffn)]
+    return ModelConfig(arch="folirax", n_layers=len(layers), d_model=width, n_heads=max(heads, gla_heads), n_kv_heads=kv_heads,
+                       head_dim=max(head_dim, gla_dim), ffn=ffn, vocab=vocab, context=HYBRID_CONTEXT, norm_eps=1e-6, layers=tuple(layers),
+                       logit_scale=0.5, logit_softcap=30.0, name=name)
+
+
+# layers of the size of the 8B preset's (width, heads, feed-forward), and a smaller stack
+FOLIRAX_8B = folirax_stack(4096, 14336, 128256, 8, 32, 8, 128, 16, 128, 256, "folirax-8b-shape")
+FOLIRAX_1B = folirax_stack(2048, 8192, 32000, 4, 16, 4, 128, 8, 128, 256, "folirax-1b-shape")
+
+PRESETS = {c.name: c for c in (TINY_LLAMA, LLAMA3_8B, LLAMA3_70B, GPT2_SMALL, GPT_OSS_20B, FOLIRAX_8B, FOLIRAX_1B)}

@@ -23,6 +23,8 @@ class TensorSpec:
 
 def tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
     d, f, V = cfg.d_model, cfg.ffn, cfg.vocab
+    if cfg.layers:
+        return hybrid_tensor_specs(cfg)
     s: list[TensorSpec] = [TensorSpec("token_embd.weight", (V, d), "embed")]
     if cfg.arch == "gpt2":
         s.append(TensorSpec("position_embd.weight", (cfg.context, d), "pos"))
@@ -63,6 +65,31 @@ def tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
     if not cfg.tied_embeddings:
         s.append(TensorSpec("output.weight", (V, d), "output"))
     return s
+
+
+def hybrid_tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
+    """Hybrid stacks go by their checkpoints' own tensor names.  Norms stored around zero are of kind "bias" (initialised to 0)."""
+    d = cfg.d_model
+    s = [TensorSpec("embed", (cfg.vocab, d), "embed")]
+    for i, l in enumerate(cfg.layers):
+        p, m = f"l{i}.", l.mixer
+        s += [TensorSpec(p + n, (d,), "bias") for n in (("norm1", "norm1b", "norm2", "norm2b") if l.ffn else ("norm1", "norm1b"))]
+        p += "mix."
+        s.append(TensorSpec(p + "q", (m.heads * m.dim, d), "matrix"))
+        if m.kind == "gla":
+            s += [TensorSpec(p + "k", (m.heads * m.dim, d), "matrix"), TensorSpec(p + "v", (m.heads * m.vdim, d), "matrix"),
+                  TensorSpec(p + "g", (m.heads * m.vdim, d), "matrix"), TensorSpec(p + "norm", (m.vdim,), "norm"),
+                  TensorSpec(p + "a1", (m.rank, d), "matrix"), TensorSpec(p + "a2", (m.heads * m.dim, m.rank), "matrix"),
+                  TensorSpec(p + "a2.b", (m.heads * m.dim,), "bias")]
+        else:
+            if m.kv_from is None:
+                s += [TensorSpec(p + "k", (m.kv_heads * m.dim, d), "matrix"), TensorSpec(p + "v", (m.kv_heads * m.vdim, d), "matrix")]
+            if m.head_gate:
+                s.append(TensorSpec(p + "g", (m.heads, d), "matrix"))
+        s.append(TensorSpec(p + "o", (d, m.heads * m.vdim), "matrix"))
+        if l.ffn:
+            s += [TensorSpec(f"l{i}.mlp.up", (l.ffn, d), "matrix"), TensorSpec(f"l{i}.mlp.down", (d, l.ffn), "matrix")]
+    return s + [TensorSpec("final.norm", (d,), "bias"), TensorSpec("head", (cfg.vocab, d), "output")]
 
 
 @dataclass(frozen=True)

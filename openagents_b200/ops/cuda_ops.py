@@ -7,17 +7,17 @@ from __future__ import annotations
 
 import ctypes
 import os
-from ctypes import c_float, c_int, c_long, c_size_t, c_void_p
+from ctypes import c_double, c_float, c_int, c_long, c_size_t, c_void_p
 
 import torch
 
 from .. import _native
 
 WT_Q4KR, WT_Q6KR, WT_Q8R, WT_BF16, WT_MXFP4R = 0, 1, 2, 3, 4
-EPI_STORE, EPI_RESID, EPI_SWIGLU_Q8, EPI_SWIGLU_F32, EPI_ALLREDUCE = 0, 1, 2, 3, 4
+EPI_STORE, EPI_RESID, EPI_SWIGLU_Q8, EPI_SWIGLU_F32, EPI_ALLREDUCE, EPI_RELU2 = 0, 1, 2, 3, 4, 6
 SYM_NONE, SYM_ALLREDUCE, SYM_RSCATTER, SYM_RSCATTER_ROWS = 0, 1, 2, 3
 EMB_F32, EMB_BF16, EMB_Q8R, EMB_Q6KR = 0, 1, 2, 3
-ACT_NONE, ACT_GELU, ACT_SWIGLU_PAIR = 0, 1, 2
+ACT_NONE, ACT_GELU, ACT_SWIGLU_PAIR, ACT_RELU2 = 0, 1, 2, 3
 
 _P = c_void_p
 _SIGS = {
@@ -56,6 +56,13 @@ _SIGS = {
     "b200_modp_matvec": [_P, _P, _P, c_int, c_int, ctypes.c_uint, _P],
     "b200_modp_matmul": [_P, _P, _P, c_int, c_int, c_int, ctypes.c_uint, _P],
     "b200_count_mismatch": [_P, _P, c_size_t, _P, _P],
+    "b200_norm_residual": [_P, c_int, _P, _P, c_int, c_int, _P, c_float, _P, _P, c_int, c_int, _P, c_long, _P, c_long, _P],
+    "b200_qkv_finish": [_P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, c_double, c_int, c_int, c_int, c_int, c_int, c_int,
+                        c_int, c_int, c_int, c_float, c_float, c_int, _P, _P, _P, _P, c_int, _P],
+    "b200_attn_exact": [_P, _P, _P, c_int, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, c_int, _P],
+    "b200_gemm_f32": [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P],
+    "b200_logits_finish": [_P, c_size_t, c_float, c_float, _P],
+    "b200_gla_recurrent": [_P] + [c_int] * 7 + [_P] * 8 + [c_int] * 5 + [c_float] * 3 + [_P, _P, c_int, _P],
 }
 
 _lib = None
@@ -66,6 +73,8 @@ def lib():
     if _lib is None:
         L = _native.cuda()
         for name, args in _SIGS.items():
+            if _native.cuda_subset and not hasattr(L, name):       # a partial library: kernels of other families are not in it
+                continue
             fn = getattr(L, name)
             fn.argtypes = args
             fn.restype = c_int
@@ -317,3 +326,53 @@ def count_mismatch(a, b) -> torch.Tensor:
     out = torch.zeros(1, dtype=torch.int32, device=a.device)
     _check(lib().b200_count_mismatch(_p(a), _p(b), a.numel(), _p(out), _st()), "count_mismatch")
     return out
+
+
+# ---------------------------------------------------------------- hybrid stacks (attention and recurrent layers, norms on both sides)
+def norm_residual(x, eps, y=None, gy=None, gh=None, hb=None, hf=None, y_clear=False, zero=None, zero2=None):
+    """``x += y / rms(y) * gy`` (with ``y``), then ``h = x / rms(x) * gh`` (with ``gh``) into ``hb`` (bf16) and/or ``hf`` (fp32), whose
+    columns beyond x's width are written as zeros.  ``y_clear`` leaves y's rows zeroed; ``zero`` / ``zero2``: contiguous fp32
+    tensors cleared on the side."""
+    T, D = x.shape
+    h = hb if hb is not None else hf
+    _check(lib().b200_norm_residual(_p(y), 0 if y is None else y.stride(0), _p(gy), _p(x), T, D, _p(gh), eps, _p(hb), _p(hf),
+                                    0 if h is None else h.stride(0), int(y_clear), _p(zero), 0 if zero is None else zero.numel(),
+                                    _p(zero2), 0 if zero2 is None else zero2.numel(), _st()), "norm_residual")
+
+
+def qkv_finish(proj, q_off, k_off, v_off, pos, slot, table, base, H, G, dim, vdim, DK, DV, rot, style, qk_norm, eps, q_scale, page_size,
+               q32=None, q16=None, kc=None, vc=None):
+    """Rotation, unit-RMS norm and scale of the queries and keys of a fused projection row, and the paged-cache write of keys and
+    values (``k_off`` < 0: the layer has none); see ``hybrid_ops.cu``."""
+    f32 = int(kc is not None and kc.dtype == torch.float32)
+    _check(lib().b200_qkv_finish(_p(proj), proj.stride(0), proj.shape[0], q_off, k_off, v_off, _p(pos), _p(slot), _p(table),
+                                 0 if table is None else table.shape[0], base, H, G, dim, vdim, DK, DV, rot, style, int(qk_norm), eps,
+                                 q_scale, page_size, _p(q32), _p(q16), _p(kc), _p(vc), f32, _st()), "qkv_finish")
+
+
+def attn_exact(q32, kc, vc, page_table, q_start, q_len, ctx_len, n_seqs, max_q, H, G, DK, DV, gate=None, out_f32=None, out_bf16=None):
+    """Causal attention in 32-bit arithmetic for any head sizes; ``gate``: fp32 [T, >= H] view whose sigmoid scales each head."""
+    o = out_f32 if out_f32 is not None else out_bf16
+    _check(lib().b200_attn_exact(_p(q32), _p(kc), _p(vc), int(kc.dtype == torch.float32), _p(page_table), page_table.shape[1], _p(q_start),
+                                 _p(q_len), _p(ctx_len), n_seqs, max_q, H, G, DK, DV, _p(gate), 0 if gate is None else gate.stride(0),
+                                 _p(out_f32), _p(out_bf16), o.stride(0), _st()), "attn_exact")
+
+
+def gemm_f32(A, W, out, act=0):
+    """``out = act(A @ W^T)`` in true 32-bit: A fp32 [M, K], W bf16 [N, K]; ``act`` 1: the square of relu."""
+    M, (N, K) = A.shape[0], W.shape
+    _check(lib().b200_gemm_f32(_p(A), A.stride(0), _p(W), W.stride(0), _p(out), out.stride(0), M, N, K, act, _st()), "gemm_f32")
+
+
+def logits_finish(logits, scale, cap):
+    _check(lib().b200_logits_finish(_p(logits), logits.numel(), scale, cap, _st()), "logits_finish")
+
+
+def gla_recurrent(proj, offs, rank, a2, b2, w, state, q_start, q_len, ctx_len, slots, n_seqs, H, dim, vdim, VP, tau, q_scale, eps,
+                  out_f32=None, out_bf16=None):
+    """Gated linear attention token by token over every sequence's new tokens (see ``linear_attn.cu``).  ``offs``: columns of q, k, v,
+    the output gate and the low-rank decay input in ``proj``; ``state`` fp32 [slots, H, dim, VP]."""
+    o = out_f32 if out_f32 is not None else out_bf16
+    _check(lib().b200_gla_recurrent(_p(proj), proj.stride(0), *offs, rank, _p(a2), _p(b2), _p(w), _p(state), _p(q_start), _p(q_len),
+                                    _p(ctx_len), _p(slots), n_seqs, H, dim, vdim, VP, tau, q_scale, eps, _p(out_f32), _p(out_bf16),
+                                    o.stride(0), _st()), "gla_recurrent")

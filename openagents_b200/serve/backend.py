@@ -159,8 +159,8 @@ class CpuBackend(Backend):
 
 
 class CudaBackend(Backend):
-    """The sm_100a engine (dense ``LlamaEngine``, tensor-parallel when given a communicator, or the expert-parallel
-    ``MoEEngine`` for models with experts).  Sampling happens on the device: greedy rows take the engine's fused
+    """A sm_100a engine (the registry's pick: dense ``LlamaEngine``, tensor-parallel when given a communicator, the
+    expert-parallel ``MoEEngine`` for models with experts, ``HybridEngine`` for stacks with recurrent layers).  Sampling happens on the device: greedy rows take the engine's fused
     arg-max (merged across vocabulary shards under tensor parallelism), the others the top-k / top-p kernel; a step
     copies back four bytes per sequence."""
     name = "cuda"
@@ -172,18 +172,18 @@ class CudaBackend(Backend):
     @classmethod
     def from_gguf(cls, path: str, device="cuda:0", max_num_seqs: int = 64, max_ctx: int = 4096, max_tokens: int = 4096,
                   tp_rank: int = 0, tp_world: int = 1, comm=None, ep_rank: int = 0, ep_world: int = 1):
-        from ..models.qweight import GGUFSource
-        src = GGUFSource(path, device)
-        if src.cfg.n_experts:
-            from ..models.moe_engine import MoEEngine
-            eng = MoEEngine(src.cfg, src, device=device, max_batch=max_num_seqs, max_ctx=max_ctx, max_tokens=max_tokens,
-                            ep_rank=ep_rank, ep_world=ep_world, comm=comm)
-        else:
-            from ..models.engine import LlamaEngine
-            eng = LlamaEngine(src.cfg, src, device=device, max_batch=max_num_seqs, max_ctx=max_ctx, max_tokens=max_tokens,
-                              tp_rank=tp_rank, tp_world=tp_world, comm=comm)
-        b = cls(eng)
-        b.tokenizer_metadata = {k: v for k, v in src.file.metadata.items() if k.startswith("tokenizer.")}
+        return cls.open(path, device, max_num_seqs, max_ctx, max_tokens, tp_rank=tp_rank, tp_world=tp_world, comm=comm, ep_rank=ep_rank,
+                        ep_world=ep_world)
+
+    @classmethod
+    def open(cls, path: str, device="cuda:0", max_num_seqs: int = 64, max_ctx: int = 4096, max_tokens: int = 4096,
+             dtype: str = "bfloat16", **options):
+        """A GGUF file or a checkpoint folder on the engine its architecture names; ``dtype`` "float32" computes in true 32-bit
+        (families that have it), ``options`` go to ``models.registry.build_engine``."""
+        from ..models.registry import build_engine, open_source, tokenizer_metadata
+        src = open_source(path, device)
+        b = cls(build_engine(src, device, max_num_seqs, max_ctx, max_tokens, dtype=dtype, **options))
+        b.tokenizer_metadata = tokenizer_metadata(path)
         return b
 
     def begin(self, seq_id, prompt):
@@ -196,6 +196,17 @@ class CudaBackend(Backend):
 
     def forward(self, seq_ids, new_tokens):
         logits, _ = self._run(seq_ids, new_tokens)
+        return self._full_rows(logits).float().cpu()
+
+    def forward_at(self, seq_ids, new_tokens, positions):
+        """One step of the batch; logits [n, V] (float, CPU) at ``positions[b]`` among sequence b's new tokens, in that order.  Takes the
+        path generation takes: a batch of single tokens is a (graph-replayed) decode step."""
+        if all(len(t) == 1 for t in new_tokens):
+            logits, _ = self.engine.decode(seq_ids, [t[0] for t in new_tokens])
+            rows = [b for b, want in enumerate(positions) for _ in want]
+            logits = logits[torch.tensor(rows, dtype=torch.long, device=logits.device)]
+        else:
+            logits, _ = self.engine.forward_tokens(seq_ids, new_tokens, greedy=False, positions=positions)
         return self._full_rows(logits).float().cpu()
 
     def _full_rows(self, logits):
@@ -240,7 +251,10 @@ class CudaBackend(Backend):
     def end(self, seq_id):
         self.engine.end(seq_id)
 
-    supports_verify = True
+    @property
+    def supports_verify(self):
+        """A rejected draft is cut off again, which a recurrent state cannot be."""
+        return not getattr(self.engine, "state_slots", 0)
 
     def verify(self, seq_id, tokens):
         _, ids = self.engine.forward_tokens([seq_id], [list(tokens)], all_positions=True)
@@ -276,7 +290,8 @@ class CudaBackend(Backend):
     def kv_stats(self):
         p = self.engine.pool
         hits, lookups = p.prefix_stats
-        return {"pages_total": p.n_pages, "pages_free": p.free_pages, "pages_retained": p.retained_pages, "page_size": p.page_size,
+        state = {"state_slots_total": p.state_slots, "state_slots_free": p.free_slots} if p.state_slots else {}
+        return {**state, "pages_total": p.n_pages, "pages_free": p.free_pages, "pages_retained": p.retained_pages, "page_size": p.page_size,
                 "prefix_hits": hits, "prefix_lookups": lookups}
 
     def topology(self):
@@ -291,11 +306,12 @@ class CudaBackend(Backend):
 
 
 def open_backend(path: str, backend: str = "cuda", device="cuda:0", **engine_args) -> Backend:
-    """The backend for a GGUF file by its architecture: the paged engine (or the fp32 oracle) for the llama and gpt-oss
-    families, the recompute backends for GPT-2-shape checkpoints."""
-    from ..gguf import GGUFFile
-    with GGUFFile(path) as f:
-        arch = f.metadata.get("general.architecture")
+    """The backend for a model (GGUF file or checkpoint folder) by its architecture: the paged engines (or the fp32 oracle) for the
+    llama and gpt-oss families, the paged hybrid engine for folirax, the recompute backends for GPT-2-shape checkpoints."""
+    from ..models.registry import peek_architecture
+    arch = peek_architecture(path)
+    if arch == "folirax" and backend == "cpu":
+        raise ValueError("folirax models are served by the cuda backend only")
     if arch == "gpt2":
         from .gpt2_backend import Gpt2CpuBackend, Gpt2CudaBackend
         if backend == "cpu":
@@ -305,4 +321,4 @@ def open_backend(path: str, backend: str = "cuda", device="cuda:0", **engine_arg
         return Gpt2CudaBackend.from_gguf(path, device=device, rows=min(8, engine_args.get("max_num_seqs", 8)))
     if backend == "cpu":
         return CpuBackend.from_gguf(path)
-    return CudaBackend.from_gguf(path, device=device, **engine_args)
+    return CudaBackend.open(path, device=device, **engine_args)

@@ -737,11 +737,11 @@ def make_handler(state: ServerState):
 
 
 def load_tokenizer(path: str, vocab_size: int):
-    """Tokenizer and chat template of a GGUF file.  The template is used only when its digest is on the allowlist of
+    """Tokenizer and chat template of a model (a checkpoint folder has neither: raw bytes, the built-in template).  The template is used only when its digest is on the allowlist of
     ``control.node_bridge`` (a template is code that runs on every request); otherwise the built-in template applies."""
     from ..control.node_bridge import template_admitted
-    from ..gguf import GGUFFile
-    meta = {k: v for k, v in GGUFFile(path).metadata.items() if k.startswith("tokenizer.")}
+    from ..models.registry import tokenizer_metadata
+    meta = tokenizer_metadata(path)
     tok = tokenizer_from_metadata(meta, vocab_size)
     tpl = meta.get("tokenizer.chat_template")
     return tok, (tpl if isinstance(tpl, str) and template_admitted(tpl) else None)
@@ -750,9 +750,10 @@ def load_tokenizer(path: str, vocab_size: int):
 def build_state(model_paths: list[str], backend: str = "cuda", max_num_seqs: int = 64, kv_page_size: int = 16,
                 max_ctx: int = 4096, reasoning_budget: int = 0, mesh_coordination: str = "disabled",
                 device="cuda:0", tp_rank: int = 0, tp_world: int = 1, ep_rank: int = 0, ep_world: int = 1, comm=None,
-                control_group=None, speculation=None) -> ServerState:
+                control_group=None, speculation=None, dtype: str = "bfloat16") -> ServerState:
     """``tp_world`` / ``ep_world`` > 1: this process is rank 0 of a tensor- or expert-parallel group whose other ranks
     run ``serve.distributed.follower_loop``; every engine call is first announced to them over ``control_group``."""
+    from ..models.registry import weights_file
     from ..receipts.manifests import artifact_digest
     from .backend import open_backend
     if backend not in ("cpu", "cuda"):
@@ -762,13 +763,13 @@ def build_state(model_paths: list[str], backend: str = "cuda", max_num_seqs: int
     models = []
     for p in model_paths:
         b = open_backend(p, backend, device, max_num_seqs=max_num_seqs, max_ctx=max_ctx, tp_rank=tp_rank,
-                         tp_world=tp_world, comm=comm, ep_rank=ep_rank, ep_world=ep_world)
+                         tp_world=tp_world, comm=comm, ep_rank=ep_rank, ep_world=ep_world, dtype=dtype)
         if max(tp_world, ep_world) > 1:
             from .distributed import LeaderBackend
             b = LeaderBackend(b, control_group)
-        mid = p.rsplit("/", 1)[-1].removesuffix(".gguf")
+        mid = p.rstrip("/").rsplit("/", 1)[-1].removesuffix(".gguf")
         tok, tpl = load_tokenizer(p, b.cfg.vocab)
-        models.append(ServedModel(mid, b, artifact_digest(p), tokenizer=tok, max_num_seqs=max_num_seqs, chat_template=tpl,
+        models.append(ServedModel(mid, b, artifact_digest(weights_file(p)), tokenizer=tok, max_num_seqs=max_num_seqs, chat_template=tpl,
                                   speculation=speculation))
     return ServerState(models, reasoning_budget, mesh_coordination)
 
@@ -810,6 +811,8 @@ def parse_args(argv=None):
     ap.add_argument("--kv-page-size", type=int, default=_flag_env("kv-page-size", 16))
     ap.add_argument("--max-num-seqs", type=int, default=_flag_env("max-num-seqs", 64))
     ap.add_argument("--max-ctx", type=int, default=_flag_env("max-ctx", 4096))
+    ap.add_argument("--dtype", default=_flag_env("dtype", "bfloat16"), choices=["bfloat16", "float32"],
+                    help="compute precision (float32: true 32-bit throughout, for the model families that have it)")
     ap.add_argument("--speculation", default=_flag_env("speculation", "none"), choices=["none", "n_gram"],
                     help="low-batch speculative decoding: n-gram drafts verified in one forward (greedy requests only)")
     ap.add_argument("--speculation-max-batch", type=int, default=_flag_env("speculation-max-batch", 4))
@@ -830,7 +833,7 @@ def run_server(a, **parallel):
         from .generation import SpeculationConfig
         spec = SpeculationConfig(max_batch=a.speculation_max_batch)
     state = build_state(a.model, a.backend, a.max_num_seqs, a.kv_page_size, a.max_ctx, a.reasoning_budget, a.mesh_coordination,
-                        speculation=spec, **parallel)
+                        speculation=spec, dtype=getattr(a, "dtype", "bfloat16"), **parallel)
     state.allow_shutdown = bool(getattr(a, "allow_shutdown", False))
     state.api_key = getattr(a, "api_key", None) or None
     httpd = serve(state, a.host, a.port)
