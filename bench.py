@@ -102,11 +102,18 @@ def main():
     ap.add_argument("--layers", type=int, default=0, help="override the layer count (debugging only; marks the run invalid)")
     ap.add_argument("--extras", default="train,moe", help="side benchmarks reported under extra: comma list of train, moe, or none")
     ap.add_argument("--no-baseline", action="store_true", help="skip the PyTorch baseline arm (vs_baseline stays null)")
+    ap.add_argument("--workload", default="decode", choices=["decode", "hybrid"], help="hybrid: prefill and decode of the hybrid engine at "
+                    "--model's layer sizes beside the Llama engine at equal size, and its kernels one by one (bench_hybrid.py)")
     ap.add_argument("--tp", type=int, default=0, help="ranks per tensor-parallel replica (0: all ranks up to 4; 8 GPUs then run "
                     "two replicas of 4, each serving half of the batch)")
     args = ap.parse_args()
     if args.impl == "reference":
         reference_arm()
+        return
+    if args.workload == "hybrid":
+        import bench_hybrid
+        args.model = args.model if args.model.startswith("folirax") else "folirax-8b-shape"
+        print(json.dumps(bench_hybrid.run(args)))
         return
     if args.impl not in ("b200", "baseline"):
         raise SystemExit("--impl is one of b200, baseline, reference")

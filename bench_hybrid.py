@@ -1,0 +1,201 @@
+"""Prefill and decode throughput of the hybrid (Folirax) engine at a real model's layer sizes, beside the Llama engine at equal size.
+
+    python bench.py --workload hybrid [--model folirax-8b-shape] [--steps K] [--warmup W]
+
+Both engines hold bf16 random weights of the same width, feed-forward, head layout, depth and vocabulary, run the same prompts
+and batches, and are timed with CUDA events: a 2048-token prompt, four of them in one call, and decode steps (replayed graphs
+with the autoregression on the device) at several batch sizes on a 2048-token context.  ``kernels`` times every kernel of the
+hybrid layers alone, L2 flushed before each launch, against its roofline (the slower of its bytes at the measured copy
+bandwidth and its FLOPs at the measured bf16 rate), with the like kernel of the Llama layer where there is one.
+"""
+from __future__ import annotations
+
+import gc
+import json
+import os
+
+import torch
+
+PROMPT = 2048
+BATCHES = (1, 8, 64)
+
+
+def peaks() -> tuple[float, float, str]:
+    try:
+        p = json.load(open(os.path.join(os.path.dirname(os.path.abspath(__file__)), "MEASURED_PEAKS.json")))
+        return p["hbm_gbs"] * 1e9, p["bf16_tflops"] * 1e12, "measured"
+    except Exception:      # noqa: BLE001
+        return 6.65e12, 1.59e15, "fallback"
+
+
+def like_llama(cfg):
+    """The Llama shape with the hybrid's width, depth, feed-forward, attention heads and vocabulary."""
+    from openagents_b200.models.config import ModelConfig
+    m = next(l.mixer for l in cfg.layers if l.mixer.kind == "attention")
+    return ModelConfig(arch="llama", n_layers=cfg.n_layers, d_model=cfg.d_model, n_heads=m.heads, n_kv_heads=m.kv_heads, head_dim=m.dim,
+                       ffn=cfg.ffn, vocab=cfg.vocab, context=8192, rope_theta=500000.0, name="llama-" + cfg.name)
+
+
+def time_engine(cfg, dev, steps: int, warmup: int) -> dict:
+    from openagents_b200.models.qweight import RandomSource
+    from openagents_b200.models.registry import build_engine
+    from openagents_b200.models.weights import PLAN_BF16
+    B = max(BATCHES)
+    eng = build_engine(RandomSource(cfg, PLAN_BF16, 0, dev), dev, B, PROMPT + 2 * (steps + warmup) * len(BATCHES) + 64, 4 * PROMPT)
+    g = torch.Generator().manual_seed(1)
+    prompts = torch.randint(0, cfg.vocab, (B, PROMPT), generator=g).tolist()
+
+    def timed(fn):
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        a.record()
+        fn()
+        b.record()
+        torch.cuda.synchronize()
+        return a.elapsed_time(b)
+
+    def prefill(ids):
+        for i in ids:
+            eng.begin(i)
+        ms = timed(lambda: eng.forward_tokens(ids, [prompts[i] for i in ids]))
+        first = eng.out_ids[: len(ids)].tolist()
+        return ms, first
+    out = {"params": cfg.n_params(), "weight_bytes": eng.weight_bytes()}
+    for ids in ([0], [0, 1, 2, 3]):
+        ms = []
+        for _ in range(4):
+            ms.append(prefill(ids)[0])
+            for i in ids:
+                eng.end(i)
+        out[f"prefill_{len(ids)}x{PROMPT}_ms"] = round(min(ms[1:]), 3)
+        out[f"prefill_{len(ids)}x{PROMPT}_tok_s"] = round(len(ids) * PROMPT / min(ms[1:]) * 1e3)
+    last = []
+    for b0 in range(0, B, 4):
+        last += prefill(list(range(b0, min(B, b0 + 4))))[1]
+    for b in BATCHES:
+        ids = list(range(b))
+        last[:b] = eng.decode_steps(ids, last[:b], warmup)[warmup - 1].tolist()
+        mark = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        h = eng.decode_steps(ids, last[:b], steps, on_replay=lambda i: mark[0].record() if i == 0 else None)
+        mark[1].record()
+        torch.cuda.synchronize()
+        last[:b] = h[steps - 1].tolist()
+        ms = mark[0].elapsed_time(mark[1]) / steps
+        out[f"decode_bs{b}_ms"], out[f"decode_bs{b}_tok_s"] = round(ms, 4), round(b / ms * 1e3, 1)
+        out[f"decode_bs{b}_launches"] = eng.launches_per_decode
+    eng.check_status()
+    del eng
+    gc.collect()
+    torch.cuda.empty_cache()
+    return out
+
+
+def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
+    """Every kernel of one hybrid layer pair at 2048 prompt tokens and at a 64-sequence decode step, and its Llama counterpart."""
+    from openagents_b200.ops import cuda_ops as ops
+    hbm, flops, _ = peaks()
+    at = next(l.mixer for l in cfg.layers if l.mixer.kind == "attention")
+    gl = next(l.mixer for l in cfg.layers if l.mixer.kind == "gla")
+    d, F, T, B, ctx = cfg.d_model, cfg.ffn, PROMPT, 64, PROMPT
+    H, G, D = at.heads, at.kv_heads, at.dim
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    rnd = lambda *s: torch.randn(*s, device=dev)                       # noqa: E731
+    bf = lambda *s: torch.randn(*s, device=dev).bfloat16()             # noqa: E731
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)     # noqa: E731
+    rows: list[dict] = []
+
+    def bench(name, fn, nbytes, fl=0.0, like=None):
+        ms = []
+        for i in range(reps + 3):
+            flush.zero_()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            if i >= 3:
+                ms.append(a.elapsed_time(b))
+        ms.sort()
+        us, roof = ms[len(ms) // 2] * 1e3, max(nbytes / hbm, fl / flops) * 1e6
+        rows.append({"kernel": name, "us": round(us, 1), "roofline_us": round(roof, 1), "of_roofline": round(roof / us, 3), "like": like})
+
+    # ---- norms and residual
+    for n in (T, B):
+        x, y, hb, gn = rnd(n, d), rnd(n, d), bf(n, d), rnd(d)
+        bench(f"norm_residual [{n}]", lambda: ops.norm_residual(x, 1e-6, y=y, gy=gn, gh=gn, hb=hb), n * d * 14, like=f"rmsnorm [{n}]")
+        bench(f"rmsnorm [{n}]", lambda: ops.rmsnorm(x, gn, 1e-6, hb=hb), n * d * 6)
+    # ---- attention: projection finish, prompt, decode
+    pages = (ctx + 15) // 16
+    for n, seqs in ((T, 1), (B, B)):
+        N = (H + 2 * G) * D + (H + 7) // 8 * 8
+        row, pos, slot = rnd(n, N), i32([ctx - 1] * n if seqs > 1 else list(range(n))), i32(list(range(n)))
+        q16, q32 = bf(n, H * D).half(), rnd(n, H * D)
+        kc, vc = rnd(seqs * pages + 1, G, 16, D).half(), rnd(seqs * pages + 1, G, 16, D).half()
+        tab, tabf = ops.rope_table(ctx, at.rope_dims, at.rope_base, dev), ops.rope_table(ctx, D, at.rope_base, dev)
+        nb = n * ((H + 2 * G) * D * 4 + H * D * (2 if n == T else 4) + 2 * G * D * 2)
+        q = dict(q16=q16) if n == T else dict(q32=q32)
+        bench(f"qkv_finish [{n}]", lambda: ops.qkv_finish(row, 0, H * D, (H + G) * D, pos, slot, tab, at.rope_base, H, G, D, D, D, D,
+                                                         at.rope_dims, 0, True, 1e-6, at.scale, 16, kc=kc, vc=vc, **q), nb, like=f"rope_kv [{n}]")
+        row2 = row[:, : (H + 2 * G) * D].contiguous()
+        bench(f"rope_kv [{n}]", lambda: ops.rope_kv(row2, pos, slot, None if n == T else q32, q16 if n == T else None, kc, vc, H, G, D, 16, at.rope_base,
+                                                    0, at.scale, table=tabf), nb)
+        table, gate = i32(list(range(seqs * pages))).view(seqs, pages), row[:, (H + 2 * G) * D:]
+        lens = i32([ctx] * seqs)
+        if n == T:
+            o, z = bf(T, H * D), i32([0])
+            fl = 4.0 * T * T / 2 * H * D
+            for nm, gt, lk in (("attn_prefill_tc05 gated", gate, "attn_prefill_tc05"), ("attn_prefill_tc05", None, None)):
+                bench(f"{nm} [{T}]", lambda: ops.attn_prefill_tc05(q16, kc, vc, table, z, lens, lens, 1, T, H, G, out_bf16=o, status=st, dk=D, dv=D, gate=gt),
+                      T * (H + G) * D * 4, fl, like=lk and f"{lk} [{T}]")
+        else:
+            o, S = bf(B, H * D), 4
+            sc, cnt = rnd(ops.attn_decode_scratch_floats(B, H, G, D, S)), torch.zeros(B * H, dtype=torch.int32, device=dev)
+            for nm, gt, lk in (("attn_decode gated", gate, "attn_decode"), ("attn_decode", None, None)):
+                bench(f"{nm} [{B} x {ctx}]", lambda: ops.attn_decode(q32, kc, vc, table, lens, B, H, G, D, S=S, gate=gt, out_bf16=o, scratch=sc, counters=cnt,
+                                                                     status=st), B * ctx * G * D * 4, like=lk and f"{lk} [{B} x {ctx}]")
+    # ---- gated linear attention
+    Hg, dk, dv, r = gl.heads, gl.dim, gl.vdim, gl.rank
+    qk, vv = Hg * dk, Hg * dv
+    ld = (2 * qk + 2 * vv + r + 7) // 8 * 8
+    offs = (0, qk, 2 * qk, 2 * qk + vv, 2 * qk + 2 * vv)
+    a2, b2, w = rnd(r, qk), rnd(qk), rnd(dv)
+    state = torch.zeros(B, Hg, dk, dv, device=dev)
+    for seqs in (1, 4):
+        n = seqs * T
+        row, out = rnd(n, ld), bf(n, vv)
+        ws = torch.empty(ops.gla_chunk_bytes(n, seqs, Hg, dk, dv, r), dtype=torch.uint8, device=dev)
+        qs, ql, sl = i32([T * b for b in range(seqs)]), i32([T] * seqs), i32(list(range(seqs)))
+        fl = n * Hg * (4.0 * dk * dv + 64 * (dk + dv))
+        bench(f"gla_chunked [{seqs} x {T}] (3 launches)", lambda: ops.gla_chunked(row, offs, r, a2, b2, w, state, qs, ql, ql, sl, seqs, Hg, dk, dv, dv, 16.0, dk ** -0.5,
+                                                                                   1e-6, T, ws, out_bf16=out), n * (ld * 4 + vv * 2), fl, like=f"attn_prefill_tc05 [{T}]")
+    for n in (1, B):
+        row, out, sl, one = rnd(n, ld), bf(n, vv), i32(list(range(n))), i32([1] * n)
+        bench(f"gla_recurrent [{n}]", lambda: ops.gla_recurrent(row, offs, r, a2, b2, w, state, sl, one, i32([ctx] * n), sl, n, Hg, dk, dv, dv, 16.0, dk ** -0.5, 1e-6,
+                                                                out_bf16=out), n * (8 * Hg * dk * dv + ld * 4), like=f"attn_decode [{B} x {ctx}]")
+    # ---- products
+    for n in (T, B):
+        a, up, gu = bf(n, d), bf(F, d), bf(2 * F, d)
+        o1, o2 = bf(n, F), bf(n, F)
+        bench(f"gemm relu2 up [{n} x {F} x {d}]", lambda: ops.gemm_bf16(a, up, n, F, d, out_bf16=o1, act=ops.ACT_RELU2, status=st), (F * d + n * (d + F)) * 2, 2.0 * n * F * d,
+              like=f"gemm swiglu gate/up [{n} x {2 * F} x {d}]")
+        bench(f"gemm swiglu gate/up [{n} x {2 * F} x {d}]", lambda: ops.gemm_bf16(a, gu, n, 2 * F, d, out_bf16=o2, ldc=F, act=ops.ACT_SWIGLU_PAIR, status=st),
+              (2 * F * d + n * (d + F)) * 2, 4.0 * n * F * d)
+        for nm, N in (("gemm gla projection", ld), ("gemm qkv projection", (H + 2 * G) * D)):
+            wt, o3 = bf(N, d), torch.zeros(n, N, device=dev)
+            bench(f"{nm} [{n} x {N} x {d}]", lambda: ops.gemm_bf16(a, wt, n, N, d, out_f32=o3, accumulate=n <= 64, status=st), N * d * 2 + n * (d * 2 + N * 4), 2.0 * n * N * d)
+    lg = rnd(B, cfg.vocab)
+    bench(f"logits_finish [{B} x {cfg.vocab}]", lambda: ops.logits_finish(lg, 0.5, 30.0), 8 * B * cfg.vocab)
+    return rows
+
+
+def run(args) -> dict:
+    from openagents_b200.models.config import PRESETS
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    cfg = PRESETS[args.model]
+    ours, llama = time_engine(cfg, dev, args.steps, max(3, args.warmup)), time_engine(like_llama(cfg), dev, args.steps, max(3, args.warmup))
+    return {"workload": "hybrid", "model": cfg.name, "dtype": "bf16", "data": "synthetic", "prompt": PROMPT, "peaks": peaks()[2], "hybrid": ours,
+            "llama_equal_size": llama, "kernels": time_kernels(cfg, dev)}

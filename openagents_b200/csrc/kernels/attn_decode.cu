@@ -8,6 +8,9 @@
 // the query heads of the group as the (padded) M dimension.  Splits are merged by whichever CTA
 // finishes last (a counter, no waiting).
 //
+// Query / key heads and value heads have sizes of their own (DK, DV: multiples of 64; other sizes are padded in the cache), and
+// an optional gate per head multiplies the output by a sigmoid.
+//
 // The softmax follows the reference formulation (max-subtract, exp, normalise:
 // apps/openagents.com/workers/api/src/cs336-a1-real-gradient-workload.ts:478-518).
 #include "tc05.cuh"
@@ -15,20 +18,23 @@
 using namespace b200;
 
 struct AttnDecArgs {
-  const float* q;          // [B][Hq*HD], rotated and pre-scaled by 1/sqrt(HD)
-  const __half* kc;        // [pages][Hkv][16][HD]
-  const __half* vc;
+  const float* q;          // [B][Hq*DK], rotated and pre-scaled
+  const __half* kc;        // [pages][Hkv][16][DK]
+  const __half* vc;        // [pages][Hkv][16][DV]
   const int* page_table;   // [B][max_pages]
   const int* seq_lens;     // [B] keys to attend (includes the current token)
   const float* sinks;      // [Hq] or null
   int max_pages, Hq, Hkv, window, S;
   int kv_rep, Hkv_cache;   // virtual KV heads per cache head (splits wide groups), heads in the cache
-  float* out_f32;          // [B][Hq*HD] or null
-  __nv_bfloat16* out_bf16; // [B][Hq*HD] or null
+  int G;                   // query heads per (virtual) KV head
+  const float* gate;       // [B][ldg] or null: head h's output is multiplied by sigmoid(gate[b][h])
+  int ldg;
+  float* out_f32;          // [B][Hq*DV] or null
+  __nv_bfloat16* out_bf16; // [B][Hq*DV] or null
   int8_t* oq;              // quantized output for a following mat-vec, or null
   float* od;
   float* os16;
-  float* part_acc;         // [B*Hkv*S*G][HD]
+  float* part_acc;         // [B*Hkv*S*G][DV]
   float* part_ml;          // [B*Hkv*S*G][2]
   int* counters;           // [B*Hkv], zero before first use; left zero on exit
   int* status;             // set non-zero if a copy never arrived (may be null)
@@ -38,16 +44,16 @@ __device__ __forceinline__ float exp_scale(float m, float M) {
   return m == -INFINITY ? 0.f : __expf(m - M);
 }
 
-template <int HD, int G>
-__device__ __forceinline__ void write_out(const AttnDecArgs& a, int b, int kh, int g, int e, float o) {
-  const int col = (kh * G + g) * HD + e;
-  const size_t row = (size_t)b * a.Hq * HD;
+template <int DV>
+__device__ __forceinline__ void write_out(const AttnDecArgs& a, int b, int h, int e, float o) {
+  const int col = h * DV + e;
+  const size_t row = (size_t)b * a.Hq * DV;
   if (a.out_f32) a.out_f32[row + col] = o;
   if (a.out_bf16) a.out_bf16[row + col] = __float2bfloat16(o);
   if (a.oq) {
     const int lane = threadIdx.x & 31;
     const int blk = col >> 5;
-    const size_t nblk = (size_t)a.Hq * HD / 32;
+    const size_t nblk = (size_t)a.Hq * DV / 32;
     quantize_block32(o, lane, a.oq + row + (size_t)blk * 32, a.od + (size_t)b * nblk + blk,
                      a.os16 + ((size_t)b * nblk + blk) * 2);
   }
@@ -79,19 +85,21 @@ constexpr int kStages = 8;   // pages in flight per CTA (two per warp)
 // the G query heads padded to a 16-row tile, and re-issues the TMA load for its next page itself,
 // so no CTA-wide synchronisation happens inside the loop.  K/V tiles land in shared memory with the
 // 128-byte swizzle, which makes every ldmatrix conflict-free.
-template <int HD, int G>
+// GT = rows reserved for query heads; EXACT: the group has exactly GT of them, else a.G <= GT.
+template <int DK, int DV, int GT, bool EXACT>
 __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant__ CUtensorMap tmK,
                                                            const __grid_constant__ CUtensorMap tmV,
                                                            const AttnDecArgs a) {
-  constexpr int NBOX = HD / 64;        // 64-column (128-byte) boxes per tile
-  constexpr int BOX = 16 * 128;        // bytes of one box: 16 tokens x 128 bytes
-  constexpr int TILE = NBOX * BOX;     // bytes of one (page, head) K or V tile
+  constexpr int KBOX = DK / 64, VBOX = DV / 64;   // 64-column (128-byte) boxes per tile
+  constexpr int BOX = 16 * 128;                   // bytes of one box: 16 tokens x 128 bytes
+  constexpr int KTILE = KBOX * BOX, SLOT = (KBOX + VBOX) * BOX;     // bytes of a (page, head) K tile, of K and V together
+  const int G = EXACT ? GT : a.G;
   extern __shared__ uint8_t dyn_raw[];
   uint8_t* ring = (uint8_t*)(((uintptr_t)dyn_raw + 1023) & ~(uintptr_t)1023);   // kStages x (K, V)
-  uint64_t* bars = (uint64_t*)(ring + kStages * 2 * TILE);
+  uint64_t* bars = (uint64_t*)(ring + kStages * SLOT);
   int* s_pid = (int*)(bars + kStages);
-  __shared__ float s_acc[4][G][HD];
-  __shared__ float s_ml[4][G][2];
+  __shared__ float s_acc[4][GT][DV];
+  __shared__ float s_ml[4][GT][2];
   __shared__ int s_last;
   __shared__ int s_abort;
 
@@ -125,33 +133,32 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
     const int s = i % kStages;
     const uint32_t bar = tc::smem_u32(bars + s);
     const int row = (s_pid[i] * a.Hkv_cache + kh_cache) * 16;
-    tc::mbar_expect_tx(bar, 2 * TILE);
+    tc::mbar_expect_tx(bar, SLOT);
 #pragma unroll
-    for (int c = 0; c < NBOX; c++) {
-      tc::tma_load_2d(tc::smem_u32(ring + (size_t)s * 2 * TILE + c * BOX), &tmK, bar, c * 64, row);
-      tc::tma_load_2d(tc::smem_u32(ring + (size_t)s * 2 * TILE + TILE + c * BOX), &tmV, bar, c * 64, row);
-    }
+    for (int c = 0; c < KBOX; c++) tc::tma_load_2d(tc::smem_u32(ring + (size_t)s * SLOT + c * BOX), &tmK, bar, c * 64, row);
+#pragma unroll
+    for (int c = 0; c < VBOX; c++) tc::tma_load_2d(tc::smem_u32(ring + (size_t)s * SLOT + KTILE + c * BOX), &tmV, bar, c * 64, row);
   };
   if (lane == 0) {
     if (warp < np) issue(warp);
     if (warp + 4 < np) issue(warp + 4);
   }
 
-  // Q as the A operand: rows = query heads (zero beyond G), fp16, HD/16 k-steps.
-  uint32_t qf[HD / 16][4];
+  // Q as the A operand: rows = query heads (zero beyond G), fp16, DK/16 k-steps.
+  uint32_t qf[DK / 16][4];
   {
-    const float* q0 = a.q + (size_t)b * a.Hq * HD + (size_t)(kh * G) * HD;
+    const float* q0 = a.q + (size_t)b * a.Hq * DK + (size_t)(kh * G) * DK;
 #pragma unroll
-    for (int kk = 0; kk < HD / 16; kk++) {
+    for (int kk = 0; kk < DK / 16; kk++) {
       const int c0 = kk * 16 + t4 * 2;
       float2 v00 = make_float2(0.f, 0.f), v01 = v00, v10 = v00, v11 = v00;
       if (g4 < G) {
-        v00 = *(const float2*)(q0 + g4 * HD + c0);
-        v01 = *(const float2*)(q0 + g4 * HD + c0 + 8);
+        v00 = *(const float2*)(q0 + g4 * DK + c0);
+        v01 = *(const float2*)(q0 + g4 * DK + c0 + 8);
       }
       if (g4 + 8 < G) {
-        v10 = *(const float2*)(q0 + (g4 + 8) * HD + c0);
-        v11 = *(const float2*)(q0 + (g4 + 8) * HD + c0 + 8);
+        v10 = *(const float2*)(q0 + (g4 + 8) * DK + c0);
+        v11 = *(const float2*)(q0 + (g4 + 8) * DK + c0 + 8);
       }
       qf[kk][0] = pack_h2(v00.x, v00.y);
       qf[kk][1] = pack_h2(v10.x, v10.y);
@@ -159,9 +166,9 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
       qf[kk][3] = pack_h2(v11.x, v11.y);
     }
   }
-  float o[HD / 8][4];
+  float o[DV / 8][4];
 #pragma unroll
-  for (int j = 0; j < HD / 8; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  for (int j = 0; j < DV / 8; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;   // rows g4 and g4 + 8
 
   for (int i = warp; i < np; i += 4) {
@@ -169,12 +176,12 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
     bool ok = tc::mbar_wait(tc::smem_u32(bars + s), (uint32_t)((i / kStages) & 1), &s_abort);
     ok = __all_sync(0xffffffffu, ok);
     if (!ok) break;
-    const uint8_t* kt = ring + (size_t)s * 2 * TILE;
-    const uint8_t* vt = kt + TILE;
+    const uint8_t* kt = ring + (size_t)s * SLOT;
+    const uint8_t* vt = kt + KTILE;
     // ---- S = Q K^T : 16 heads x 16 tokens
     float sc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
-    for (int kk = 0; kk < HD / 16; kk++) {
+    for (int kk = 0; kk < DK / 16; kk++) {
       const int r = (lane >> 4) * 8 + (lane & 7);            // token row
       const int c = 2 * kk + ((lane >> 3) & 1);              // 16-byte chunk of the full row
       const uint8_t* p = kt + (c >> 3) * BOX + r * 128 + (((c & 7) ^ (r & 7)) << 4);
@@ -217,12 +224,12 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
     m0 = mn0;
     m1 = mn1;
 #pragma unroll
-    for (int j = 0; j < HD / 8; j++) {
+    for (int j = 0; j < DV / 8; j++) {
       o[j][0] *= c0; o[j][1] *= c0; o[j][2] *= c1; o[j][3] *= c1;
     }
     // ---- O += P V
 #pragma unroll
-    for (int jd = 0; jd < HD / 8; jd += 2) {
+    for (int jd = 0; jd < DV / 8; jd += 2) {
       const int r = (lane & 7) + ((lane >> 3) & 1) * 8;      // token row
       const int c = jd + (lane >> 4);
       const uint8_t* p = vt + (c >> 3) * BOX + r * 128 + (((c & 7) ^ (r & 7)) << 4);
@@ -242,9 +249,9 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
   // this warp's partial (m, l, O) for each real head -> shared
-  if (g4 < G) {
+  if (g4 < GT && g4 < G) {
 #pragma unroll
-    for (int j = 0; j < HD / 8; j++) {
+    for (int j = 0; j < DV / 8; j++) {
       s_acc[warp][g4][j * 8 + t4 * 2] = o[j][0];
       s_acc[warp][g4][j * 8 + t4 * 2 + 1] = o[j][1];
     }
@@ -253,9 +260,9 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
       s_ml[warp][g4][1] = l0;
     }
   }
-  if (g4 + 8 < G) {
+  if (g4 + 8 < GT && g4 + 8 < G) {
 #pragma unroll
-    for (int j = 0; j < HD / 8; j++) {
+    for (int j = 0; j < DV / 8; j++) {
       s_acc[warp][g4 + 8][j * 8 + t4 * 2] = o[j][2];
       s_acc[warp][g4 + 8][j * 8 + t4 * 2 + 1] = o[j][3];
     }
@@ -269,9 +276,10 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
   // merge the four warps: thread e owns output dim e
   const int e = tid;
   const size_t pbase = (((size_t)b * a.Hkv + kh) * a.S + split) * G;
-  float fm[G], fl[G], fa[G];
+  float fm[GT], fl[GT], fa[GT];
 #pragma unroll
-  for (int g = 0; g < G; g++) {
+  for (int g = 0; g < GT; g++) {
+    if (g >= G) continue;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; w++) M = fmaxf(M, s_ml[w][g][0]);
@@ -280,15 +288,16 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
     for (int w = 0; w < 4; w++) {
       const float c = exp_scale(s_ml[w][g][0], M);
       L += s_ml[w][g][1] * c;
-      if (e < HD) A += s_acc[w][g][e] * c;
+      if (e < DV) A += s_acc[w][g][e] * c;
     }
     fm[g] = M; fl[g] = L; fa[g] = A;
   }
 
   if (a.S > 1) {
 #pragma unroll
-    for (int g = 0; g < G; g++) {
-      if (e < HD) a.part_acc[(pbase + g) * HD + e] = fa[g];
+    for (int g = 0; g < GT; g++) {
+      if (g >= G) continue;
+      if (e < DV) a.part_acc[(pbase + g) * DV + e] = fa[g];
       if (e == 0) {
         a.part_ml[(pbase + g) * 2] = fm[g];
         a.part_ml[(pbase + g) * 2 + 1] = fl[g];
@@ -306,7 +315,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
     __threadfence();
     const size_t p0 = ((size_t)b * a.Hkv + kh) * a.S * G;
 #pragma unroll
-    for (int g = 0; g < G; g++) {
+    for (int g = 0; g < GT; g++) {
+      if (g >= G) continue;
       float M = -INFINITY;
       for (int s = 0; s < a.S; s++) M = fmaxf(M, __ldcg(a.part_ml + (p0 + (size_t)s * G + g) * 2));
       float L = 0.f, A = 0.f;
@@ -314,15 +324,16 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
         const size_t idx = p0 + (size_t)s * G + g;
         const float c = exp_scale(__ldcg(a.part_ml + idx * 2), M);
         L += __ldcg(a.part_ml + idx * 2 + 1) * c;
-        if (e < HD) A += __ldcg(a.part_acc + idx * HD + e) * c;
+        if (e < DV) A += __ldcg(a.part_acc + idx * DV + e) * c;
       }
       fm[g] = M; fl[g] = L; fa[g] = A;
     }
   }
 
-  if (warp * 32 < HD) {  // warps that own real output dims (all four when HD = 128)
+  if (warp * 32 < DV) {  // warps that own real output dims (all four when DV = 128)
 #pragma unroll
-    for (int g = 0; g < G; g++) {
+    for (int g = 0; g < GT; g++) {
+      if (g >= G) continue;
       float M = fm[g], L = fl[g], A = fa[g];
       if (a.sinks) {
         const float sk = a.sinks[kh * G + g];
@@ -331,70 +342,88 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
         L = L * c + __expf(sk - M2);
         A *= c;
       }
-      const float o = L > 0.f ? A / L : 0.f;
-      write_out<HD, G>(a, b, kh, g, e, o);
+      float o = L > 0.f ? A / L : 0.f;
+      if (a.gate) o *= 1.f / (1.f + __expf(-a.gate[(size_t)b * a.ldg + kh * G + g]));
+      write_out<DV>(a, b, kh * G + g, e, o);
     }
   }
 }
 
-template <int HD, int G>
+template <int DK, int DV, int GT, bool EXACT>
 static int launch(const AttnDecArgs& a, int B, int n_pages, cudaStream_t st) {
   dim3 grid(a.S, a.Hkv, B);
   const int pages_per_cta = (a.max_pages + a.S - 1) / a.S + 1;
-  const size_t smem = 1024 + (size_t)kStages * 2 * 16 * HD * 2 + kStages * 8 + (size_t)pages_per_cta * 4;
-  if (smem > 200 * 1024) return B200_ERR_BAD_ARG;
+  const size_t smem = 1024 + (size_t)kStages * 16 * (DK + DV) * 2 + kStages * 8 + (size_t)pages_per_cta * 4;
+  if (smem > 180 * 1024) return B200_ERR_BAD_ARG;
+  auto kern = attn_decode_kernel<DK, DV, GT, EXACT>;
   static size_t configured = 0;
   if (smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<HD, G>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = smem;
   }
-  // The cache as a 2-D tensor: one row per (page, head, token), HD columns.
+  // The caches as 2-D tensors: one row per (page, head, token).
   CUtensorMap tk, tv;
   const uint64_t rows = (uint64_t)n_pages * a.Hkv_cache * 16;
-  int rc = make_tmap_2d(&tk, a.kc, 2, rows, HD, (uint64_t)HD * 2, 16, 64, true);
+  int rc = make_tmap_2d(&tk, a.kc, 2, rows, DK, (uint64_t)DK * 2, 16, 64, true);
   if (rc) return rc;
-  rc = make_tmap_2d(&tv, a.vc, 2, rows, HD, (uint64_t)HD * 2, 16, 64, true);
+  rc = make_tmap_2d(&tv, a.vc, 2, rows, DV, (uint64_t)DV * 2, 16, 64, true);
   if (rc) return rc;
-  return launch_pdl(attn_decode_kernel<HD, G>, grid, dim3(128), smem, st, tk, tv, a);
+  return launch_pdl(kern, grid, dim3(128), smem, st, tk, tv, a);
 }
 
-// Floats of scratch the split-merge needs: part_acc then part_ml, plus B*Hkv ints of counters.
+template <int HD>
+static int launch_exact(const AttnDecArgs& a, int B, int n_pages, cudaStream_t st) {
+  switch (a.G) {
+    case 1: return launch<HD, HD, 1, true>(a, B, n_pages, st);
+    case 2: return launch<HD, HD, 2, true>(a, B, n_pages, st);
+    case 4: return launch<HD, HD, 4, true>(a, B, n_pages, st);
+    case 8: return launch<HD, HD, 8, true>(a, B, n_pages, st);
+    case 16: return launch<HD, HD, 16, true>(a, B, n_pages, st);
+  }
+  return a.G < 8 ? launch<HD, HD, 8, false>(a, B, n_pages, st) : launch<HD, HD, 16, false>(a, B, n_pages, st);
+}
+template <int DK, int DV>
+static int launch_any(const AttnDecArgs& a, int B, int n_pages, cudaStream_t st) {
+  if (a.G == 1) return launch<DK, DV, 1, true>(a, B, n_pages, st);
+  return a.G <= 4 ? launch<DK, DV, 4, false>(a, B, n_pages, st) : launch<DK, DV, 16, false>(a, B, n_pages, st);
+}
+
+// Floats of scratch the split-merge needs: part_acc then part_ml (hd = value head size), plus one int of counters per
+// sequence and query head at most.
 B200_API size_t b200_attn_decode_scratch_floats(int B, int Hq, int Hkv, int hd, int S) {
   return (size_t)B * Hq * S * (hd + 2);
 }
 
+// hd: query / key head size, dv: value head size (64..256 and 64..128, multiples of 64).  counters: B * Hq ints, zero before first use.
 B200_API int b200_attn_decode(const float* q, const void* kc, const void* vc, const int* page_table,
                               int max_pages, int n_pages, const int* seq_lens, const float* sinks, int B,
-                              int Hq, int Hkv, int hd, int window, int S, float* out_f32, void* out_bf16,
-                              void* oq, float* od, float* os16, float* scratch, int* counters, int* status,
+                              int Hq, int Hkv, int hd, int dv, int window, int S, const float* gate, int ldg, float* out_f32,
+                              void* out_bf16, void* oq, float* od, float* os16, float* scratch, int* counters, int* status,
                               cudaStream_t st) {
-  if (Hq % Hkv || S < 1) return B200_ERR_BAD_ARG;
-  const int G = Hq / Hkv;
-  if (G > 16) return B200_ERR_BAD_ARG;
+  if (Hkv < 1 || Hq % Hkv || S < 1) return B200_ERR_BAD_ARG;
+  int G = Hq / Hkv, rep = 1;
+  while (G % rep || G / rep > 16) rep++;            // a group wider than the 16-row tile is served as several
   AttnDecArgs a;
   a.q = q; a.kc = (const __half*)kc; a.vc = (const __half*)vc; a.page_table = page_table;
-  a.seq_lens = seq_lens; a.sinks = sinks; a.max_pages = max_pages; a.Hq = Hq; a.Hkv = Hkv;
-  a.window = window; a.S = S; a.kv_rep = 1; a.Hkv_cache = Hkv; a.out_f32 = out_f32; a.out_bf16 = (__nv_bfloat16*)out_bf16;
+  a.seq_lens = seq_lens; a.sinks = sinks; a.max_pages = max_pages; a.Hq = Hq; a.Hkv = Hkv * rep;
+  a.window = window; a.S = S; a.kv_rep = rep; a.Hkv_cache = Hkv; a.G = G / rep; a.gate = gate; a.ldg = ldg;
+  a.out_f32 = out_f32; a.out_bf16 = (__nv_bfloat16*)out_bf16;
   a.oq = (int8_t*)oq; a.od = od; a.os16 = os16;
   a.part_acc = scratch;
-  a.part_ml = scratch ? scratch + (size_t)B * Hq * S * hd : nullptr;
+  a.part_ml = scratch ? scratch + (size_t)B * Hq * S * dv : nullptr;
   a.counters = counters;
   a.status = status;
   if (S > 1 && (!scratch || !counters)) return B200_ERR_BAD_ARG;
-  if (hd == 128) {
-    if (G == 1) return launch<128, 1>(a, B, n_pages, st);
-    if (G == 2) return launch<128, 2>(a, B, n_pages, st);
-    if (G == 4) return launch<128, 4>(a, B, n_pages, st);
-    if (G == 8) return launch<128, 8>(a, B, n_pages, st);
-    if (G == 16) return launch<128, 16>(a, B, n_pages, st);
-  } else if (hd == 64) {
-    if (G == 1) return launch<64, 1>(a, B, n_pages, st);
-    if (G == 2) return launch<64, 2>(a, B, n_pages, st);
-    if (G == 4) return launch<64, 4>(a, B, n_pages, st);
-    if (G == 8) return launch<64, 8>(a, B, n_pages, st);
-    if (G == 16) return launch<64, 16>(a, B, n_pages, st);
+  if (hd == dv && hd == 128) return launch_exact<128>(a, B, n_pages, st);
+  if (hd == dv && hd == 64) return launch_exact<64>(a, B, n_pages, st);
+  switch (hd * 1000 + dv) {
+    case 64128: return launch_any<64, 128>(a, B, n_pages, st);
+    case 128064: return launch_any<128, 64>(a, B, n_pages, st);
+    case 192064: return launch_any<192, 64>(a, B, n_pages, st);
+    case 192128: return launch_any<192, 128>(a, B, n_pages, st);
+    case 256064: return launch_any<256, 64>(a, B, n_pages, st);
+    case 256128: return launch_any<256, 128>(a, B, n_pages, st);
   }
   return B200_ERR_BAD_ARG;
 }

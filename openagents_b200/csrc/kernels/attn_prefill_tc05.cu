@@ -1,4 +1,7 @@
-// Causal grouped-query flash attention for prefill on the 5th-generation tensor cores (head dim 128).
+// Causal grouped-query flash attention for prefill on the 5th-generation tensor cores.
+//
+// Head sizes are template parameters (queries / keys DK = 64..256, values DV = 64 or 128, multiples of 64; other sizes are padded
+// in the cache); the figures below are those of DK = DV = 128.  An optional gate per head multiplies the output by a sigmoid.
 //
 // One CTA = 128 query rows of one head.  Roles: warps 0 and 10 are the TMA producers (a ring of K / V
 // blocks of 64 keys gathered page by page from the paged fp16 cache), warps 1 and 11 issue the two
@@ -28,9 +31,9 @@ using namespace b200::tc;
 
 namespace {
 
-constexpr int QB = 128, KB = 128, HD = 128, KV_STAGES = 3;
-constexpr int K_BYTES = KB * HD * 2;            // 16 KB: two halves of [64 keys][64 dims]
-constexpr uint32_t TMEM_COLS = 512;             // S: 2 x 128 (P is written over the S columns it came from), O: 128, Q: 64
+constexpr int QB = 128, KB = 128;
+constexpr int BOX_BYTES = KB * 128;             // one 64-dim column block of a K or V tile: [128 keys][128 bytes]
+constexpr uint32_t TMEM_COLS = 512;             // S: 2 x 128 (P is written over the S columns it came from), O: DV, Q: DK / 2
 constexpr float kRescaleStep = 8.f;             // log2 units
 constexpr float kLog2e = 1.4426950408889634f;
 
@@ -40,9 +43,11 @@ struct PrefillArgs {
   const int* q_len;        // [n_seqs]
   const int* ctx_len;      // [n_seqs]
   const float* sinks;      // [Hq] or null
-  __nv_bfloat16* out;      // [T_total][Hq * HD]
+  __nv_bfloat16* out;      // [T_total][Hq * DV]
   int* status;
-  const __half* q;         // [T_total][Hq * HD], rotated and scaled
+  const __half* q;         // [T_total][Hq * DK], rotated and scaled
+  const float* gate;       // [T_total][ldg] or null: head h's output is multiplied by sigmoid(gate[t][h])
+  int ldg;
   int max_pages, Hq, Hkv, window, T_total;
 };
 
@@ -92,13 +97,19 @@ __device__ __forceinline__ void umma_ts(uint32_t tmem_d, uint32_t tmem_a, uint64
 }
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
-__global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(                                                                    const __grid_constant__ CUtensorMap tmK,
-                                                                    const __grid_constant__ CUtensorMap tmV,
-                                                                    const PrefillArgs a) {
+template <int DK, int DV>
+constexpr int kv_stages() { return 196608 / (KB * (DK + DV) * 2) < 4 ? 196608 / (KB * (DK + DV) * 2) : 4; }
+
+template <int DK, int DV>
+__global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap tmK,
+                                                                   const __grid_constant__ CUtensorMap tmV,
+                                                                   const PrefillArgs a) {
+  constexpr int K_BYTES = KB * DK * 2, V_BYTES = KB * DV * 2, STAGE_BYTES = K_BYTES + V_BYTES, KV_STAGES = kv_stages<DK, DV>();
+  static_assert(256 + DV + DK / 2 <= (int)TMEM_COLS && KV_STAGES >= 2, "head sizes");
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   uint8_t* sKV = smem;                                    // KV_STAGES x (K, V)
-  uint64_t* bars = (uint64_t*)(sKV + KV_STAGES * 2 * K_BYTES);
+  uint64_t* bars = (uint64_t*)(sKV + KV_STAGES * STAGE_BYTES);
   uint64_t* q_full = bars;                                // [1]
   uint64_t* kv_full = bars + 1;                           // [KV_STAGES]
   uint64_t* kv_empty = kv_full + KV_STAGES;               // [KV_STAGES]
@@ -155,7 +166,7 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(             
   const int jb0 = k_lo / KB, jb1 = live ? (k_hi + KB - 1) / KB : jb0;   // key blocks [jb0, jb1)
   const int nb = jb1 - jb0;
   const uint32_t S_T = tmem_base, O_T = tmem_base + 256;   // S buffers at +0, +128; O at +256
-  const uint32_t Q_T = tmem_base + 384;                    // Q (fp16 pairs, 64 columns)
+  const uint32_t Q_T = O_T + DV;                           // Q (fp16 pairs, DK / 2 columns)
   // P_j (fp16 pairs) overwrites S_j: the warp that owns keys [64 h, 64 h + 64) of a block writes columns [64 h, 64 h + 32)
 
   // Four single-thread roles, each in a warp of its own, because what a thread can issue is the bound here:
@@ -173,16 +184,16 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(             
         const uint32_t bar = smem_u32(kv_full + s);
         // the barrier holds one pending arrival until this arrive.expect_tx, so V bytes that land first cannot
         // complete the phase early
-        if (is_k) mbar_expect_tx(bar, 2 * K_BYTES);
-        uint8_t* dst = sKV + (size_t)s * 2 * K_BYTES + (is_k ? 0 : K_BYTES);
+        if (is_k) mbar_expect_tx(bar, STAGE_BYTES);
+        uint8_t* dst = sKV + (size_t)s * STAGE_BYTES + (is_k ? 0 : K_BYTES);
+        const int boxes = (is_k ? DK : DV) / 64;
         const CUtensorMap* tm = is_k ? &tmK : &tmV;
 #pragma unroll
         for (int p = 0; p < KB / 16; p++) {
           const int pi = (jb0 + j) * (KB / 16) + p;
           const int page = (pi * 16 < ctx) ? pt[pi] : 0;          // pages past the context are masked anyway
           const int row = (page * a.Hkv + kh) * 16;
-#pragma unroll
-          for (int hf = 0; hf < 2; hf++) tma_load_2d(smem_u32(dst + hf * (K_BYTES / 2) + p * 2048), tm, bar, hf * 64, row);
+          for (int hf = 0; hf < boxes; hf++) tma_load_2d(smem_u32(dst + hf * BOX_BYTES + p * 2048), tm, bar, hf * 64, row);
         }
       }
     }
@@ -196,26 +207,26 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(             
         if (!mbar_wait(smem_u32(s_empty + b), ((j >> 1) & 1) ^ 1, abort_flag)) break;
         if (j >= 2 && !mbar_wait(smem_u32(pv_done + b), ((j - 2) >> 1) & 1, abort_flag)) break;   // P_{j-2} sits in S buffer b
         tc_fence_after();
-        const uint32_t ka = smem_u32(sKV + (size_t)s * 2 * K_BYTES);
+        const uint32_t ka = smem_u32(sKV + (size_t)s * STAGE_BYTES);
 #pragma unroll
-        for (int kk = 0; kk < HD / 16; kk++)
-          umma_ts(S_T + b * KB, Q_T + 8 * kk, smem_desc_sw128(ka + (kk >> 2) * (K_BYTES / 2)) + 2 * (kk & 3), idesc_s,
+        for (int kk = 0; kk < DK / 16; kk++)
+          umma_ts(S_T + b * KB, Q_T + 8 * kk, smem_desc_sw128(ka + (kk >> 2) * BOX_BYTES) + 2 * (kk & 3), idesc_s,
                   kk != 0 ? 1u : 0u);
         umma_commit(smem_u32(s_full + b));
       }
     }
   } else if (warp == 11) {
     if (lane == 0 && nb > 0) {
-      constexpr uint32_t idesc_o = idesc_f16(QB, HD, true);
+      constexpr uint32_t idesc_o = idesc_f16(QB, DV, true);
       for (int j = 0; j < nb; j++) {
         const int s = j % KV_STAGES, b = j & 1;
         if (!mbar_wait(smem_u32(kv_full + s), (j / KV_STAGES) & 1, abort_flag)) break;       // V_j has landed
         if (!mbar_wait(smem_u32(p_full + b), (j >> 1) & 1, abort_flag)) break;                // P_j written, O rows rescaled if needed
         tc_fence_after();
-        const uint32_t va = smem_u32(sKV + (size_t)s * 2 * K_BYTES + K_BYTES);
+        const uint32_t va = smem_u32(sKV + (size_t)s * STAGE_BYTES + K_BYTES);
 #pragma unroll
         for (int kk = 0; kk < KB / 16; kk++)
-          umma_ts(O_T, S_T + b * KB + (kk >> 2) * 64 + 8 * (kk & 3), smem_desc_sw128_mn(va + kk * 2048, K_BYTES / 2), idesc_o,
+          umma_ts(O_T, S_T + b * KB + (kk >> 2) * 64 + 8 * (kk & 3), smem_desc_sw128_mn(va + kk * 2048, BOX_BYTES), idesc_o,
                   (j != 0 || kk != 0) ? 1u : 0u);
         // a commit covers this thread's MMAs only; S_j is known to be done because the softmax of block j needed it
         umma_commit(smem_u32(pv_done + b));
@@ -228,16 +239,16 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(             
     const int row = q * 32 + lane;               // query row of this thread (shared with the partner warp's same lane)
     const int qpos = pos0 + row;
     const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
-    constexpr int HK = KB / 2, HO = HD / 2;
+    constexpr int HK = KB / 2, HO = DV / 2;
     float m_used = -INFINITY, l = 0.f;     // exponent offset of this row (log2 units) and this warp's part of the row sum
     bool ok = true;
     // post this warp's half and wait (bounded, like every wait here) for the partner's; use number `u` of buffer `bb`
     if (hsel == 0) {
       // This row of Q (fp16, already rotated and scaled) goes to tensor memory once: column j = dims 2j, 2j + 1.
       const bool in = qs + q0 + row < a.T_total;
-      const uint4* qrow = (const uint4*)(a.q + ((size_t)(qs + q0 + (in ? row : 0)) * a.Hq + h) * HD);
+      const uint4* qrow = (const uint4*)(a.q + ((size_t)(qs + q0 + (in ? row : 0)) * a.Hq + h) * DK);
 #pragma unroll
-      for (int c = 0; c < 2; c++) {
+      for (int c = 0; c < DK / 64; c++) {
         uint32_t r[32];
 #pragma unroll
         for (int i = 0; i < 8; i++) {
@@ -358,9 +369,10 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(             
       l += xl[(hsel ^ 1) * 128 + row];
       tc_fence_after();
       if (a.sinks) l += (m_used == -INFINITY) ? 1.f : ex2_approx(a.sinks[h] * kLog2e - m_used);
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
       const bool wr = ok && row < qlen - q0;
-      __nv_bfloat16* dst = a.out + (size_t)(qs + q0 + row) * a.Hq * HD + (size_t)h * HD + hsel * HO;
+      if (a.gate && wr) inv *= 1.f / (1.f + __expf(-a.gate[(size_t)(qs + q0 + row) * a.ldg + h]));
+      __nv_bfloat16* dst = a.out + (size_t)(qs + q0 + row) * a.Hq * DV + (size_t)h * DV + hsel * HO;
 #pragma unroll
       for (int c = 0; c < HO / 32; c++) {
         uint32_t r[32];
@@ -386,33 +398,49 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(             
   if (threadIdx.x == 0 && *abort_flag && a.status) atomicExch(a.status, (int)B200_ERR_TIMEOUT_MMA);
 }
 
-}  // namespace
-
-// q fp16 [T_total][Hq * 128] (rotated, pre-scaled by 1/sqrt(128)); kc / vc fp16 [n_pages][Hkv][16][128];
-// out bf16 [T_total][Hq * 128].  Sequences as in b200_attn_prefill; max_q = longest chunk.
-B200_API int b200_attn_prefill_tc05(const void* q, const void* kc, const void* vc, const int* page_table, int max_pages,
-                                    int n_pages, const int* q_start, const int* q_len, const int* ctx_len, int n_seqs,
-                                    int max_q, int T_total, int Hq, int Hkv, int window, const float* sinks, void* out,
-                                    int* status, cudaStream_t st) {
-  if (Hq % Hkv || n_seqs < 1 || max_q < 1 || !page_table) return B200_ERR_BAD_ARG;
+template <int DK, int DV>
+int launch_prefill(const void* kc, const void* vc, int n_pages, const PrefillArgs& a, int n_seqs, int max_q, cudaStream_t st) {
   CUtensorMap tk, tv;
-  int rc;
-  const uint64_t rows = (uint64_t)n_pages * Hkv * 16;
-  rc = make_tmap_2d(&tk, kc, 2, rows, HD, (uint64_t)HD * 2, 16, 64, true);
+  const uint64_t rows = (uint64_t)n_pages * a.Hkv * 16;
+  int rc = make_tmap_2d(&tk, kc, 2, rows, DK, (uint64_t)DK * 2, 16, 64, true);
   if (rc) return rc;
-  rc = make_tmap_2d(&tv, vc, 2, rows, HD, (uint64_t)HD * 2, 16, 64, true);
+  rc = make_tmap_2d(&tv, vc, 2, rows, DV, (uint64_t)DV * 2, 16, 64, true);
   if (rc) return rc;
-  PrefillArgs a;
-  a.q = (const __half*)q; a.T_total = T_total;
-  a.page_table = page_table; a.q_start = q_start; a.q_len = q_len; a.ctx_len = ctx_len; a.sinks = sinks;
-  a.out = (__nv_bfloat16*)out; a.status = status; a.max_pages = max_pages; a.Hq = Hq; a.Hkv = Hkv; a.window = window;
-  constexpr size_t smem = 1024 + KV_STAGES * 2 * K_BYTES + 32 * 8 + 2 * 2 * 128 * 4;
+  constexpr size_t smem = 1024 + (size_t)kv_stages<DK, DV>() * KB * (DK + DV) * 2 + 32 * 8 + 2 * 2 * 128 * 4;
+  static_assert(smem <= 232448, "shared memory per CTA");
+  auto kern = attn_prefill_tc05_kernel<DK, DV>;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc05_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  dim3 grid((max_q + QB - 1) / QB, Hq, n_seqs);
-  return launch_pdl(attn_prefill_tc05_kernel, grid, dim3(384), smem, st, tk, tv, a);
+  dim3 grid((max_q + QB - 1) / QB, a.Hq, n_seqs);
+  return launch_pdl(kern, grid, dim3(384), smem, st, tk, tv, a);
+}
+
+}  // namespace
+
+// q fp16 [T_total][Hq * dk] (rotated, pre-scaled); kc fp16 [n_pages][Hkv][16][dk], vc [n_pages][Hkv][16][dv];
+// out bf16 [T_total][Hq * dv].  Sequences as in b200_attn_prefill; max_q = longest chunk.
+B200_API int b200_attn_prefill_tc05(const void* q, const void* kc, const void* vc, const int* page_table, int max_pages,
+                                    int n_pages, const int* q_start, const int* q_len, const int* ctx_len, int n_seqs,
+                                    int max_q, int T_total, int Hq, int Hkv, int dk, int dv, int window, const float* sinks,
+                                    const float* gate, int ldg, void* out, int* status, cudaStream_t st) {
+  if (Hkv < 1 || Hq % Hkv || n_seqs < 1 || max_q < 1 || !page_table) return B200_ERR_BAD_ARG;
+  PrefillArgs a;
+  a.q = (const __half*)q; a.T_total = T_total; a.gate = gate; a.ldg = ldg;
+  a.page_table = page_table; a.q_start = q_start; a.q_len = q_len; a.ctx_len = ctx_len; a.sinks = sinks;
+  a.out = (__nv_bfloat16*)out; a.status = status; a.max_pages = max_pages; a.Hq = Hq; a.Hkv = Hkv; a.window = window;
+  switch (dk * 1000 + dv) {
+    case 64064: return launch_prefill<64, 64>(kc, vc, n_pages, a, n_seqs, max_q, st);
+    case 64128: return launch_prefill<64, 128>(kc, vc, n_pages, a, n_seqs, max_q, st);
+    case 128064: return launch_prefill<128, 64>(kc, vc, n_pages, a, n_seqs, max_q, st);
+    case 128128: return launch_prefill<128, 128>(kc, vc, n_pages, a, n_seqs, max_q, st);
+    case 192064: return launch_prefill<192, 64>(kc, vc, n_pages, a, n_seqs, max_q, st);
+    case 192128: return launch_prefill<192, 128>(kc, vc, n_pages, a, n_seqs, max_q, st);
+    case 256064: return launch_prefill<256, 64>(kc, vc, n_pages, a, n_seqs, max_q, st);
+    case 256128: return launch_prefill<256, 128>(kc, vc, n_pages, a, n_seqs, max_q, st);
+  }
+  return B200_ERR_BAD_ARG;
 }

@@ -81,7 +81,6 @@ class LlamaEngine(PagedEngine):
         self.prefill_tc05 = os.environ.get("B200_PREFILL_TC05", "1") == "1"     # tcgen05 prefill attention (head size 128)
         self.seq_shard = os.environ.get("B200_TP_SEQ_SHARD", "1") == "1"        # sequence-sharded tensor-parallel prefill
         self.fuse_rope = os.environ.get("B200_FUSE_ROPE", "1") == "1"          # small-batch path: rotary + cache write in the QKV mat-vec
-        self.attn_target_ctas = int(os.environ.get("B200_ATTN_CTAS", 0))   # split-K attention: CTAs to aim for (0: built-in rule)
 
     # ------------------------------------------------------------------ weights
     def _shard_rows(self, r: RawTensor, per_head_rows: int | None = None) -> RawTensor:
@@ -178,9 +177,8 @@ class LlamaEngine(PagedEngine):
         self.fd = ws("fd", (nb, kmax // 32 + 1), f32t)
         self.fs = ws("fs", (nb, kmax // 16 + 2), f32t)
         self._alloc_batch()
-        self.max_splits = 64
         self.attn_scratch = ws("attn_scratch", (ops.attn_decode_scratch_floats(self.max_batch, self.Hq, self.Hkv, self.hd, self.max_splits),), f32t)
-        self.attn_counters = ws("attn_counters", (self.max_batch * self.Hkv,), i32, zero=True)
+        self.attn_counters = ws("attn_counters", (self.max_batch * self.Hq,), i32, zero=True)
         self.argmax_scratch = ops.argmax_scratch(self.max_batch, dev)
         self.rope_tab = ops.rope_table(self.max_pages * PAGE, self.hd, self.cfg.rope_theta, dev)
         wmax = max(max(l.wqkv.N * l.wqkv.K, l.wo.N * l.wo.K, *((l.wgu.N * l.wgu.K, l.wdown.N * l.wdown.K) if l.wgu is not None else ()))
@@ -258,18 +256,7 @@ class LlamaEngine(PagedEngine):
 
     # ------------------------------------------------------------------ building blocks
     def _splits(self, B: int, ctx_pages: int) -> int:
-        """Split-K factor of decode attention.  Measured on the 8B shape: a CTA should keep at least ~24
-        pages (the merge of the partial results and each CTA's set-up are a fixed cost), small batches
-        want just enough CTAs to cover the SMs once, and large batches run best at ~2000 CTAs (several
-        waves even out the tail)."""
-        if self.attn_target_ctas:                      # explicit override (benchmark sweeps)
-            want = max(1, (self.attn_target_ctas + B * self.Hkv - 1) // (B * self.Hkv))
-        else:
-            rows = B * self.Hkv
-            fill = (148 + rows - 1) // rows
-            big = (2048 + rows - 1) // rows if rows >= 148 else 0
-            want = min(max(1, ctx_pages // 24), max(fill, big))
-        return max(1, min(self.max_splits, want, ctx_pages))
+        return self._attn_splits(B, self.Hkv, ctx_pages)
 
     @property
     def _sig(self):

@@ -51,6 +51,7 @@ class _Block:
     out: _Lin
     DK: int = 0                  # attention: padded head sizes of queries / keys and values;  gla: DV is the padded value size
     DV: int = 0
+    tc: bool = False             # attention: the tensor-core kernels take these head sizes
     kv: int = -1                 # index of the key / value cache this layer reads
     table: torch.Tensor | None = None
     a2: torch.Tensor | None = None
@@ -115,11 +116,11 @@ class HybridEngine(PagedEngine):
             b = _Block(spec, self._vector(src, p + "norm1", True), self._vector(src, p + "norm1b", True), proj, None)
             if m.kind == "gla":
                 b.DV = _up(m.vdim, 8)
-                b.a2 = src.get(p + "mix.a2").to_float().to(self.device).contiguous()
+                b.a2 = src.get(p + "mix.a2").to_float().to(self.device).t().contiguous()
                 b.b2, b.o_norm = self._vector(src, p + "mix.a2.b"), self._vector(src, p + "mix.norm")
                 b.state = torch.zeros((self.state_slots, m.heads, m.dim, b.DV), dtype=torch.float32, device=self.device)
             else:
-                b.DK, b.DV = self._head_pad(m)
+                b.DK, b.DV, b.tc = self._head_pad(m)
                 if m.kv_from is None:
                     b.kv, n_kv = n_kv, n_kv + 1
                 else:
@@ -138,11 +139,13 @@ class HybridEngine(PagedEngine):
         self.head = self._lin(self._matrix(src, "head"))
         torch.cuda.synchronize(self.device)
 
-    def _head_pad(self, m: MixerSpec) -> tuple[int, int]:
-        """Padded head sizes in the cache."""
-        if self.exact:
-            return _up(m.dim, 8), _up(m.vdim, 8)
-        return _up(m.dim, 64), _up(m.vdim, 64)
+    def _head_pad(self, m: MixerSpec) -> tuple[int, int, bool]:
+        """Padded head sizes in the cache, and whether the tensor-core attention kernels take them (else, and always in the 32-bit
+        mode, the any-size kernel runs)."""
+        dk, dv = _up(m.dim, 64), _up(m.vdim, 64)
+        if self.exact or dk > 256 or dv > 128:
+            return _up(m.dim, 8), _up(m.vdim, 8), False
+        return dk, dv, True
 
     def weight_bytes(self) -> int:
         n = self.head.w.numel()
@@ -168,11 +171,19 @@ class HybridEngine(PagedEngine):
         n_ffn = max((b.up.N for b in self.blocks if b.up is not None), default=8)
         attn = [b for b in self.blocks if b.spec.mixer.kind == "attention"]
         n_q = max((b.spec.mixer.heads * b.DK for b in attn), default=8)
+        n_q32 = max((b.spec.mixer.heads * b.DK for b in attn if not b.tc), default=0)      # rows of a prompt in fp32
         self.x = ws("x", (T, self.d), f32)
         self.y = ws("y", (T, d), f32, zero=True)
         self.proj = ws("proj", (T * n_proj,), f32, zero=True)
-        self.q32 = ws("q32", ((T if self._q32_prefill() else self.max_batch) * n_q,), f32)
-        self.q16 = ws("q16", (8 if self.exact else T * n_q,), torch.float16)
+        self.q32 = ws("q32", (max(T * n_q32, self.max_batch * n_q),), f32)
+        self.q16 = ws("q16", (T * n_q if any(b.tc for b in attn) else 8,), torch.float16)
+        tc = [(b.spec.mixer, b.DV) for b in attn if b.tc]
+        self.attn_scratch = ws("attn_scratch", (max((ops.attn_decode_scratch_floats(self.max_batch, m.heads, m.kv_heads, dv, self.max_splits)
+                                                     for m, dv in tc), default=4),), f32)
+        self.attn_counters = ws("attn_counters", (self.max_batch * max((m.heads for m, _ in tc), default=1),), torch.int32, zero=True)
+        gla = [b for b in self.blocks if b.spec.mixer.kind == "gla"]
+        self.gla_ws = ws("gla_ws", (max((ops.gla_chunk_bytes(T, self.max_batch, m.heads, m.dim, dv, m.rank)
+                                         for m, dv in ((b.spec.mixer, b.DV) for b in gla)), default=0) if not self.exact else 0,), torch.uint8)
         small = self.max_batch if not self.exact else T            # rows of the fp32 activations
         self.hf = ws("hf", (small * d,), f32)
         self.mf = ws("mf", (small * n_mix,), f32)
@@ -189,9 +200,6 @@ class HybridEngine(PagedEngine):
         k_max = max(d, n_mix, n_ffn)
         # the bf16 mat-vec keeps its fp32 activations in shared memory
         self.matvec_rows = max((n for n in (1, 2, 4, 8) if n * (k_max * 4 + 256) <= 200 * 1024), default=0)
-
-    def _q32_prefill(self) -> bool:
-        return True
 
     # ------------------------------------------------------------------ building blocks
     def _mm(self, a: torch.Tensor, L: _Lin, out: torch.Tensor, act: int = 0, add: bool = False):
@@ -215,12 +223,23 @@ class HybridEngine(PagedEngine):
         v_off = k_off + m.kv_heads * m.dim
         g_off = v_off + m.kv_heads * m.vdim if own else m.heads * m.dim
         kc, vc = self.kc[b.kv], self.vc[b.kv]
-        q32 = self.q32[: T * m.heads * b.DK]
+        tc_prompt = b.tc and not decode
+        q = (self.q16 if tc_prompt else self.q32)[: T * m.heads * b.DK].view(T, -1)
         ops.qkv_finish(proj, 0, k_off, v_off, self.pos, self.slot, b.table, m.rope_base, m.heads, m.kv_heads, m.dim, m.vdim, b.DK, b.DV,
-                       m.rope_dims, 0 if m.rope_style == "pairs" else 1, m.qk_norm, cfg.norm_eps, m.scale, PAGE, q32=q32, kc=kc, vc=vc)
+                       m.rope_dims, 0 if m.rope_style == "pairs" else 1, m.qk_norm, cfg.norm_eps, m.scale, PAGE, q32=None if tc_prompt else q,
+                       q16=q if tc_prompt else None, kc=kc, vc=vc)
         gate = proj[:, g_off:] if m.head_gate else None
+        if tc_prompt:
+            ops.attn_prefill_tc05(q, kc, vc, self.page_table, self.q_start, self.q_len, self.seq_lens, n_seqs, max_q, m.heads, m.kv_heads,
+                                  out_bf16=o16, status=self.status, dk=b.DK, dv=b.DV, gate=gate)
+            return 2
+        if b.tc:
+            ops.attn_decode(q, kc, vc, self.page_table, self.seq_lens, n_seqs, m.heads, m.kv_heads, b.DK, dv=b.DV,
+                            S=self._attn_splits(n_seqs, m.kv_heads, pages), gate=gate, out_f32=o32, out_bf16=o16,
+                            scratch=self.attn_scratch, counters=self.attn_counters, status=self.status)
+            return 2
         qs, ql = (self.iota, self.ones) if decode else (self.q_start, self.q_len)
-        ops.attn_exact(q32, kc, vc, self.page_table, qs, ql, self.seq_lens, n_seqs, max_q, m.heads, m.kv_heads, b.DK, b.DV, gate=gate,
+        ops.attn_exact(q, kc, vc, self.page_table, qs, ql, self.seq_lens, n_seqs, max_q, m.heads, m.kv_heads, b.DK, b.DV, gate=gate,
                        out_f32=o32, out_bf16=o16)
         return 2
 
@@ -229,9 +248,13 @@ class HybridEngine(PagedEngine):
         qk, vv = m.heads * m.dim, m.heads * m.vdim
         offs = (0, qk, 2 * qk, 2 * qk + vv, 2 * qk + 2 * vv)
         qs, ql = (self.iota, self.ones) if decode else (self.q_start, self.q_len)
-        ops.gla_recurrent(proj, offs, m.rank, b.a2, b.b2, b.o_norm, b.state, qs, ql, self.seq_lens, self.state_slot, n_seqs, m.heads, m.dim,
-                          m.vdim, b.DV, m.tau, m.dim ** -0.5, self.cfg.norm_eps, out_f32=o32, out_bf16=o16)
-        return 1
+        args = (proj, offs, m.rank, b.a2, b.b2, b.o_norm, b.state, qs, ql, self.seq_lens, self.state_slot, n_seqs, m.heads, m.dim, m.vdim, b.DV,
+                m.tau, m.dim ** -0.5, self.cfg.norm_eps)
+        if decode or self.exact or not ops.gla_chunk_bytes(T, n_seqs, m.heads, m.dim, b.DV, m.rank):
+            ops.gla_recurrent(*args, out_f32=o32, out_bf16=o16)
+            return 1
+        ops.gla_chunked(*args, max_q, self.gla_ws, out_f32=o32, out_bf16=o16)
+        return 3
 
     def _run_layers(self, T: int, decode: bool, n_seqs: int, max_q: int, pages: int) -> int:
         eps, x, y = self.cfg.norm_eps, self.x[:T], self.y[:T]

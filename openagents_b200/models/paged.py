@@ -179,6 +179,8 @@ class PagedEngine:
         self.status = torch.zeros(1, dtype=torch.int32, device=self.device)
         self._graphs: dict[int, tuple] = {}
         self.launches_per_decode = 0
+        self.max_splits = 64
+        self.attn_target_ctas = int(os.environ.get("B200_ATTN_CTAS", 0))   # split-K decode attention: CTAs to aim for (0: built-in rule)
         self.h2d_bytes = 0                              # host-to-device bytes copied by decode() so far
 
     def _alloc_batch(self):
@@ -231,6 +233,20 @@ class PagedEngine:
             if not bool((raw[G + nbytes:] == self._GUARD_FILL).all()):
                 bad.append(name + ":after")
         return bad
+
+    def _attn_splits(self, B: int, kv_heads: int, ctx_pages: int) -> int:
+        """Split-K factor of decode attention.  Measured on the 8B shape: a CTA should keep at least ~24
+        pages (the merge of the partial results and each CTA's set-up are a fixed cost), small batches
+        want just enough CTAs to cover the SMs once, and large batches run best at ~2000 CTAs (several
+        waves even out the tail)."""
+        if self.attn_target_ctas:                      # explicit override (benchmark sweeps)
+            want = max(1, (self.attn_target_ctas + B * kv_heads - 1) // (B * kv_heads))
+        else:
+            rows = B * kv_heads
+            fill = (148 + rows - 1) // rows
+            big = (2048 + rows - 1) // rows if rows >= 148 else 0
+            want = min(max(1, ctx_pages // 24), max(fill, big))
+        return max(1, min(self.max_splits, want, ctx_pages))
 
     # ------------------------------------------------------------------ host-side batch assembly
     def _stage_batch(self, seq_ids, new_tokens: list[list[int]]):

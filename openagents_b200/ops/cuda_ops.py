@@ -36,10 +36,11 @@ _SIGS = {
     "b200_matvec": [c_int, _P, _P, c_int, c_int, c_int, _P, _P, _P, _P, c_int, _P, _P, _P, c_int, _P, _P, _P, _P,
                     c_size_t, c_int, _P],
     "b200_argmax_merge": [_P, _P, c_int, _P, c_size_t, c_int, _P],
-    "b200_attn_decode": [_P, _P, _P, _P, c_int, c_int, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P,
-                         _P, _P, _P, _P, _P],
+    "b200_attn_decode": [_P, _P, _P, _P, c_int, c_int, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, _P,
+                         _P, _P, _P, _P, _P, _P],
     "b200_attn_prefill": [_P, _P, _P, _P, c_int, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P],
-    "b200_attn_prefill_tc05": [_P, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P],
+    "b200_attn_prefill_tc05": [_P, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P,
+                               c_int, _P, _P, _P],
     "b200_gemm_bf16": [_P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int,
                        _P, c_int, _P, c_size_t, c_int, c_int, c_int, c_int, c_int, _P],
     "b200_moe_gemm": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, _P, _P, _P, c_size_t, _P, _P],
@@ -62,6 +63,7 @@ _SIGS = {
     "b200_attn_exact": [_P, _P, _P, c_int, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, c_int, _P],
     "b200_gemm_f32": [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P],
     "b200_logits_finish": [_P, c_size_t, c_float, c_float, _P],
+    "b200_gla_chunked": [_P] + [c_int] * 7 + [_P] * 8 + [c_int] * 5 + [c_float] * 3 + [_P, _P, c_int, c_int, c_int, _P, c_size_t, _P],
     "b200_gla_recurrent": [_P] + [c_int] * 7 + [_P] * 8 + [c_int] * 5 + [c_float] * 3 + [_P, _P, c_int, _P],
 }
 
@@ -80,6 +82,8 @@ def lib():
             fn.restype = c_int
         L.b200_attn_decode_scratch_floats.argtypes = [c_int, c_int, c_int, c_int, c_int]
         L.b200_attn_decode_scratch_floats.restype = c_size_t
+        L.b200_gla_chunk_bytes.argtypes = [c_int] * 6
+        L.b200_gla_chunk_bytes.restype = c_size_t
         _lib = L
         if os.environ.get("B200_PDL", "1") == "0":      # debugging aid: fully serialised launches
             L.b200_set_pdl(0)
@@ -212,9 +216,12 @@ def attn_decode_scratch_floats(B, Hq, Hkv, hd, S):
 
 
 def attn_decode(q, kc, vc, page_table, seq_lens, B, Hq, Hkv, hd, window=0, S=1, sinks=None, out_f32=None, out_bf16=None,
-                oq=None, od=None, os16=None, scratch=None, counters=None, status=None):
+                oq=None, od=None, os16=None, scratch=None, counters=None, status=None, dv=None, gate=None):
+    """``hd`` / ``dv``: query-key and value head sizes (``dv`` defaults to ``hd``); ``gate``: fp32 [B, >= Hq] view whose sigmoid scales
+    each head's output."""
     _check(lib().b200_attn_decode(_p(q), _p(kc), _p(vc), _p(page_table), page_table.shape[1], kc.shape[0], _p(seq_lens), _p(sinks),
-                                  B, Hq, Hkv, hd, window, S, _p(out_f32), _p(out_bf16), _p(oq), _p(od), _p(os16),
+                                  B, Hq, Hkv, hd, hd if dv is None else dv, window, S, _p(gate), 0 if gate is None else gate.stride(0),
+                                  _p(out_f32), _p(out_bf16), _p(oq), _p(od), _p(os16),
                                   _p(scratch), _p(counters), _p(status), _st()), "attn_decode")
 
 
@@ -226,11 +233,12 @@ def attn_prefill(q, kc, vc, page_table, max_pages, q_start, q_len, ctx_len, n_se
 
 
 def attn_prefill_tc05(q16, kc, vc, page_table, q_start, q_len, ctx_len, n_seqs, max_q_len, Hq, Hkv, window=0, sinks=None,
-                      out_bf16=None, status=None):
-    """Prefill attention on tcgen05 (head dim 128, fp16 q / cache, bf16 out); see ``attn_prefill_tc05.cu``."""
+                      out_bf16=None, status=None, dk=128, dv=128, gate=None):
+    """Prefill attention on tcgen05 (fp16 q / cache, bf16 out; ``dk`` 64..256 and ``dv`` 64 or 128, multiples of 64); ``gate``: fp32
+    [T, >= Hq] view whose sigmoid scales each head's output.  See ``attn_prefill_tc05.cu``."""
     _check(lib().b200_attn_prefill_tc05(_p(q16), _p(kc), _p(vc), _p(page_table), page_table.shape[1], kc.shape[0], _p(q_start),
-                                        _p(q_len), _p(ctx_len), n_seqs, max_q_len, q16.shape[0], Hq, Hkv, window, _p(sinks),
-                                        _p(out_bf16), _p(status), _st()), "attn_prefill_tc05")
+                                        _p(q_len), _p(ctx_len), n_seqs, max_q_len, q16.shape[0], Hq, Hkv, dk, dv, window, _p(sinks),
+                                        _p(gate), 0 if gate is None else gate.stride(0), _p(out_bf16), _p(status), _st()), "attn_prefill_tc05")
 
 
 def gemm_bf16(A, B, M, N, K, lda=None, ldb=None, out_f32=None, out_bf16=None, ldc=None, bias=None, resid_f32=None,
@@ -371,8 +379,22 @@ def logits_finish(logits, scale, cap):
 def gla_recurrent(proj, offs, rank, a2, b2, w, state, q_start, q_len, ctx_len, slots, n_seqs, H, dim, vdim, VP, tau, q_scale, eps,
                   out_f32=None, out_bf16=None):
     """Gated linear attention token by token over every sequence's new tokens (see ``linear_attn.cu``).  ``offs``: columns of q, k, v,
-    the output gate and the low-rank decay input in ``proj``; ``state`` fp32 [slots, H, dim, VP]."""
+    the output gate and the low-rank decay input in ``proj``; ``a2`` fp32 [rank, H * dim]; ``state`` fp32 [slots, H, dim, VP]."""
     o = out_f32 if out_f32 is not None else out_bf16
     _check(lib().b200_gla_recurrent(_p(proj), proj.stride(0), *offs, rank, _p(a2), _p(b2), _p(w), _p(state), _p(q_start), _p(q_len),
                                     _p(ctx_len), _p(slots), n_seqs, H, dim, vdim, VP, tau, q_scale, eps, _p(out_f32), _p(out_bf16),
                                     o.stride(0), _st()), "gla_recurrent")
+
+
+def gla_chunk_bytes(T, n_seqs, H, dim, VP, rank):
+    """Workspace of :func:`gla_chunked`; 0 for sizes it does not take."""
+    return lib().b200_gla_chunk_bytes(T, n_seqs, H, dim, VP, rank)
+
+
+def gla_chunked(proj, offs, rank, a2, b2, w, state, q_start, q_len, ctx_len, slots, n_seqs, H, dim, vdim, VP, tau, q_scale, eps, max_q, ws,
+                out_f32=None, out_bf16=None):
+    """:func:`gla_recurrent` for prompts, in 64-token chunks on the tensor cores; ``ws``: uint8 workspace."""
+    o = out_f32 if out_f32 is not None else out_bf16
+    _check(lib().b200_gla_chunked(_p(proj), proj.stride(0), *offs, rank, _p(a2), _p(b2), _p(w), _p(state), _p(q_start), _p(q_len),
+                                  _p(ctx_len), _p(slots), n_seqs, H, dim, vdim, VP, tau, q_scale, eps, _p(out_f32), _p(out_bf16),
+                                  o.stride(0), proj.shape[0], max_q, _p(ws), ws.numel(), _st()), "gla_chunked")
