@@ -99,7 +99,7 @@ def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
     gl = next(l.mixer for l in cfg.layers if l.mixer.kind == "gla")
     d, F, T, B, ctx = cfg.d_model, cfg.ffn, PROMPT, 64, PROMPT
     H, G, D = at.heads, at.kv_heads, at.dim
-    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    flush = torch.empty(1 << 30, dtype=torch.uint8, device=dev)
     st = torch.zeros(1, dtype=torch.int32, device=dev)
     rnd = lambda *s: torch.randn(*s, device=dev)                       # noqa: E731
     bf = lambda *s: torch.randn(*s, device=dev).bfloat16()             # noqa: E731
@@ -109,10 +109,10 @@ def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
     def bench(name, fn, nbytes, fl=0.0, like=None):
         ms = []
         for i in range(reps + 3):
+            torch.cuda.synchronize()
             flush.zero_()
             a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            torch.cuda.synchronize()
-            a.record()
+            a.record()                             # queued behind the flush: the launch itself is not in the time
             fn()
             b.record()
             torch.cuda.synchronize()
@@ -169,7 +169,7 @@ def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
         ws = torch.empty(ops.gla_chunk_bytes(n, seqs, Hg, dk, dv, r), dtype=torch.uint8, device=dev)
         qs, ql, sl = i32([T * b for b in range(seqs)]), i32([T] * seqs), i32(list(range(seqs)))
         fl = n * Hg * (4.0 * dk * dv + 64 * (dk + dv))
-        bench(f"gla_chunked [{seqs} x {T}] (3 launches)", lambda: ops.gla_chunked(row, offs, r, a2, b2, w, state, qs, ql, ql, sl, seqs, Hg, dk, dv, dv, 16.0, dk ** -0.5,
+        bench(f"gla_chunked [{seqs} x {T}] (3 kernels)", lambda: ops.gla_chunked(row, offs, r, a2, b2, w, state, qs, ql, ql, sl, seqs, Hg, dk, dv, dv, 16.0, dk ** -0.5,
                                                                                    1e-6, T, ws, out_bf16=out), n * (ld * 4 + vv * 2), fl, like=f"attn_prefill_tc05 [{T}]")
     for n in (1, B):
         row, out, sl, one = rnd(n, ld), bf(n, vv), i32(list(range(n))), i32([1] * n)

@@ -78,6 +78,69 @@ __global__ void __launch_bounds__(1024) norm_residual_kernel(float* __restrict__
     if (hf) hf[(size_t)t * ldh + i] = o;
   }
 }
+// The same for rows of whole float4s that fit the registers of the block (every real model's width): 16-byte accesses, and blocks
+// small enough for several rows per SM.
+template <int R>
+__global__ void __launch_bounds__(256) norm_residual_vec_kernel(float4* __restrict__ y, int ldy4, const float4* __restrict__ gy,
+                                                                float4* __restrict__ x, int D4, const float4* __restrict__ gh,
+                                                                float eps, __nv_bfloat16* __restrict__ hb,
+                                                                float4* __restrict__ hf, int ldh4, int y_clear,
+                                                                float4* __restrict__ zero_a, int na4, float4* __restrict__ zero_b,
+                                                                int nb4) {
+  __shared__ float red[32];
+  const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+  float4* xr = x + (size_t)t * D4;
+  float4* yr = y + (size_t)t * ldy4;
+  const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 v[R], w[R];
+  pdl_trigger();
+  pdl_wait();
+#pragma unroll
+  for (int k = 0; k < R; k++) {
+    const int i = tid + k * nt;
+    v[k] = i < D4 ? xr[i] : z;
+    w[k] = (y && i < D4) ? yr[i] : z;
+  }
+  for (int i = blockIdx.x * nt + tid; i < na4; i += gridDim.x * nt) zero_a[i] = z;
+  for (int i = blockIdx.x * nt + tid; i < nb4; i += gridDim.x * nt) zero_b[i] = z;
+  const float inv_d = 1.f / (float)(4 * D4);
+  if (y) {
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < R; k++) ss += w[k].x * w[k].x + w[k].y * w[k].y + w[k].z * w[k].z + w[k].w * w[k].w;
+    const float r = 1.f / sqrtf(block_sum(ss, red) * inv_d + eps);
+#pragma unroll
+    for (int k = 0; k < R; k++) {
+      const int i = tid + k * nt;
+      if (i >= D4) continue;
+      const float4 g = gy[i];
+      v[k].x += w[k].x * r * g.x;
+      v[k].y += w[k].y * r * g.y;
+      v[k].z += w[k].z * r * g.z;
+      v[k].w += w[k].w * r * g.w;
+      xr[i] = v[k];
+      if (y_clear) yr[i] = z;
+    }
+  }
+  if (!gh) return;
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < R; k++) ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+  const float r = 1.f / sqrtf(block_sum(ss, red) * inv_d + eps);
+#pragma unroll
+  for (int k = 0; k < R; k++) {
+    const int i = tid + k * nt;
+    if (i >= ldh4) continue;           // ldh4 > D4: padding columns are zeros
+    const float4 g = i < D4 ? gh[i] : z;
+    const float4 o = make_float4(v[k].x * r * g.x, v[k].y * r * g.y, v[k].z * r * g.z, v[k].w * r * g.w);
+    if (hb) {
+      const __nv_bfloat162 p0 = __floats2bfloat162_rn(o.x, o.y), p1 = __floats2bfloat162_rn(o.z, o.w);
+      *(uint2*)(hb + ((size_t)t * ldh4 + i) * 4) = make_uint2(*(const uint32_t*)&p0, *(const uint32_t*)&p1);
+    }
+    if (hf) hf[(size_t)t * ldh4 + i] = o;
+  }
+}
+
 // x fp32 [T][D]; y fp32 [T][ldy] or null; gains fp32 [D]; hb / hf [T][ldh].  zero_*_n: floats, multiples of 4.
 B200_API int b200_norm_residual(float* y, int ldy, const float* gy, float* x, int T, int D, const float* gh, float eps, void* hb,
                                 float* hf, int ldh, int y_clear, float* zero_a, long zero_a_n, float* zero_b, long zero_b_n,
@@ -85,6 +148,14 @@ B200_API int b200_norm_residual(float* y, int ldy, const float* gy, float* x, in
   if (T < 1 || D < 1 || !x || (y && (!gy || ldy < D)) || (gh && (ldh < D || (!hb && !hf)))) return B200_ERR_BAD_ARG;
   if ((zero_a && (zero_a_n % 4 || (uintptr_t)zero_a % 16)) || (zero_b && (zero_b_n % 4 || (uintptr_t)zero_b % 16)))
     return B200_ERR_BAD_ARG;
+  const uintptr_t align = (uintptr_t)x | (uintptr_t)y | (uintptr_t)gy | (uintptr_t)gh | (uintptr_t)hb | (uintptr_t)hf;
+  if (align % 16 == 0 && ((D | ldy | ldh) & 3) == 0 && max(D, ldh) <= 256 * 4 * 8 && (!y || ldy == D || !y_clear)) {
+    const int n4 = max(D, ldh) / 4, nt = n4 > 512 ? 256 : n4 > 128 ? 128 : 64, R = (n4 + nt - 1) / nt;
+    auto kern = R <= 1 ? norm_residual_vec_kernel<1> : R <= 2 ? norm_residual_vec_kernel<2> : R <= 4 ? norm_residual_vec_kernel<4> : norm_residual_vec_kernel<8>;
+    return launch_pdl(kern, dim3(T), dim3(nt), 0, st, (float4*)y, ldy / 4, (const float4*)gy, (float4*)x, D / 4, (const float4*)gh, eps,
+                      (__nv_bfloat16*)hb, (float4*)hf, ldh / 4, y_clear, (float4*)zero_a, zero_a ? (int)(zero_a_n / 4) : 0, (float4*)zero_b,
+                      zero_b ? (int)(zero_b_n / 4) : 0);
+  }
   const int threads = D >= 4096 ? 1024 : D >= 2048 ? 512 : D >= 512 ? 256 : 128;
   return launch_pdl(norm_residual_kernel, dim3(T), dim3(threads), 0, st, y, ldy, gy, x, D, gh, eps, (__nv_bfloat16*)hb, hf, ldh,
                     y_clear, (float4*)zero_a, zero_a ? (int)(zero_a_n / 4) : 0, (float4*)zero_b, zero_b ? (int)(zero_b_n / 4) : 0);

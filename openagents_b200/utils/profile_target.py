@@ -12,7 +12,8 @@ row-parallel GEMM with its fused all-reduce epilogue; ``gemm_ag2048`` / ``gemm_r
 pair (norm + all-gather push -> GEMM, GEMM -> reduce-scatter); ``zero_adamw``: the sharded optimizer step;
 ``attn_train_fwd`` / ``attn_train_bwd``: training attention at GPT-2-small's shape (16 x 1024 tokens, 12 heads of 64);
 ``gemm_mn``: the weight-gradient GEMM (both operands read token-major); ``norm_slots``: the RMSNorm that is the tensor-parallel
-all-reduce, 64 rows of 4096 on a one-rank heap.
+all-reduce, 64 rows of 4096 on a one-rank heap; ``gla_chunked`` / ``gla_decode``: gated linear attention of an 8B-size hybrid layer, a
+2048-token prompt / a decode step of 64 sequences.
 """
 from __future__ import annotations
 
@@ -207,6 +208,21 @@ def main():
             norm2.zero_()
             tops.zero_reduce_norm(heap.table, goff, 0, n_par, gsh, norm2)
             tops.zero_adamw_gather(heap.table, poff, 0, n_par, gsh, master, m, v, norm2, 6e-4, 0.9, 0.95, 1e-8, 0.1, 0.1, 0.05, 1.0, n_par)
+    elif case in ("gla_chunked", "gla_decode"):
+        # one recurrent layer of the 8B-size hybrid stack: 16 heads, keys of 128, values of 256
+        H, dk, dv, r = 16, 128, 256, 16
+        B, T = (1, 2048) if case == "gla_chunked" else (64, 64)
+        qk, vv = H * dk, H * dv
+        offs, ld = (0, qk, 2 * qk, 2 * qk + vv, 2 * qk + 2 * vv), 2 * qk + 2 * vv + r
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=DEV)
+        row, out = torch.randn(T, ld, device=DEV), torch.empty((T, vv), dtype=torch.bfloat16, device=DEV)
+        a2, b2, w = torch.randn(r, qk, device=DEV) / 4, torch.randn(qk, device=DEV), torch.ones(dv, device=DEV)
+        state = torch.zeros(B, H, dk, dv, device=DEV)
+        per = T // B
+        args = (row, offs, r, a2, b2, w, state, i32([per * b for b in range(B)]), i32([per] * B), i32([per + 1] * B), i32(list(range(B))), B, H, dk, dv, dv, 16.0,
+                dk ** -0.5, 1e-6)
+        ws = torch.empty(ops.gla_chunk_bytes(T, B, H, dk, dv, r), dtype=torch.uint8, device=DEV)
+        fn = (lambda: ops.gla_chunked(*args, per, ws, out_bf16=out)) if case == "gla_chunked" else (lambda: ops.gla_recurrent(*args, out_bf16=out))
     else:
         raise SystemExit(f"unknown case {case}")
     fn()                                  # warm-up outside the profiled range

@@ -25,7 +25,7 @@ def i32(*v):
 def test_norm_on_both_sides_of_a_sublayer():
     from openagents_b200.ops import cuda_ops as ops
     g = torch.Generator().manual_seed(0)
-    for T, D, ld in ((3, 72, 72), (5, 100, 104), (2, 4100, 4104), (1, 9000, 9000)):
+    for T, D, ld in ((3, 72, 72), (5, 100, 104), (4, 93, 96), (2, 2048, 2048), (3, 4096, 4096), (2, 4100, 4104), (1, 9000, 9000)):
         x, y = torch.randn(T, D, generator=g), torch.randn(T, ld, generator=g) * 3
         gy, gh = 1 + 0.3 * torch.randn(D, generator=g), 1 + 0.3 * torch.randn(D, generator=g)
         want_x = x.double() + R.centred_norm(y[:, :D].double(), gy.double() - 1, 1e-3)
