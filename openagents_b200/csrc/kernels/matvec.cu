@@ -355,69 +355,86 @@ __global__ void __launch_bounds__(256) matvec_q_kernel(const MatvecArgs a) {
   if (a.epi == EPI_ALLREDUCE) sym_kernel_end_barrier(a.sym, 0, gridDim.x, a.wait_ready != 0);
 }
 
-// bf16 weights [N][K] against fp32 activations.
-template <int B, bool DUAL>
+// bf16 weights [N][K] against fp32 activations.  A warp owns RW rows and walks K once for all of them: every row's loads of a column
+// block are in flight together, and the activations are read from shared memory once per block.
+template <int B, bool DUAL, int RW>
 __global__ void __launch_bounds__(256) matvec_bf16_kernel(const MatvecArgs a) {
   extern __shared__ __align__(16) uint8_t smem[];
+  constexpr int R = 8 * RW, NM = DUAL ? 2 : 1, UN = RW * NM >= 4 ? 1 : 4 / RW;
+  static_assert(!DUAL || RW == 4, "the SwiGLU epilogue quantizes 32-row blocks");
   float* xs = (float*)smem;            // [B][K]
   float* res = xs + (size_t)B * a.K;   // [2][32][B]
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
+  const __nv_bfloat16* W = (const __nv_bfloat16*)a.w;
+  {  // this CTA's weight rows into L2 while the kernel before this one still runs
+    const int r0 = blockIdx.x * R, nr = min(R, a.N - r0);
+    if (nr > 0 && a.prefetch) {
+      const size_t total = (size_t)nr * NM * a.K * 2;      // rows are multiples of 16 bytes
+      constexpr uint32_t CH = 16384;
+      const int nch = (int)((total + CH - 1) / CH);
+      const uint8_t* base = (const uint8_t*)(W + (size_t)r0 * NM * a.K);
+      for (int c = tid; c < nch; c += 256) prefetch_l2(base + (size_t)c * CH, (uint32_t)min((size_t)CH, total - (size_t)c * CH));
+    }
+  }
   pdl_trigger();
   pdl_wait();
-  for (int i = tid; i < B * a.K; i += 256) {
-    const int b = i / a.K;
-    xs[i] = b < a.nb ? a.xf[i] : 0.f;
+  {
+    const int live = a.nb * a.K / 4, all = B * a.K / 4;    // K is a multiple of 8
+#pragma unroll 4
+    for (int i = tid; i < live; i += 256) ((float4*)xs)[i] = ((const float4*)a.xf)[i];
+    for (int i = live + tid; i < all; i += 256) ((float4*)xs)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
   }
   __syncthreads();
-  const __nv_bfloat16* W = (const __nv_bfloat16*)a.w;
-#pragma unroll 1
-  for (int i = 0; i < 4; i++) {
-    const int r = w + 8 * i;
-    const int n = blockIdx.x * 32 + r;
-    float acc0[B], acc1[B];
+  float acc[NM][RW][B];
+  const __nv_bfloat16* wr[NM][RW];
 #pragma unroll
-    for (int b = 0; b < B; b++) acc0[b] = acc1[b] = 0.f;
-    if (n < a.N) {
-      const __nv_bfloat16* wr0 = W + (size_t)(DUAL ? 2 * n : n) * a.K;     // dual: rows interleaved (gate_n, up_n)
-      const __nv_bfloat16* wr1 = W + (size_t)(2 * n + 1) * a.K;
-#pragma unroll 2
-      for (int k = lane * 8; k < a.K; k += 256) {
-        const uint4 q0 = ldg_stream(wr0 + k);
-        uint4 q1 = make_uint4(0, 0, 0, 0);
-        if (DUAL) q1 = ldg_stream(wr1 + k);
-        const __nv_bfloat162* p0 = (const __nv_bfloat162*)&q0;
-        const __nv_bfloat162* p1 = (const __nv_bfloat162*)&q1;
+  for (int i = 0; i < RW; i++) {
+    const int n = min(blockIdx.x * R + w + 8 * i, a.N - 1);            // a row past the end is computed from the last one and not stored
 #pragma unroll
-        for (int b = 0; b < B; b++) {
-          const float4 xa = *(const float4*)(xs + (size_t)b * a.K + k);
-          const float4 xb = *(const float4*)(xs + (size_t)b * a.K + k + 4);
-          float2 f;
-          f = __bfloat1622float2(p0[0]); acc0[b] += f.x * xa.x + f.y * xa.y;
-          f = __bfloat1622float2(p0[1]); acc0[b] += f.x * xa.z + f.y * xa.w;
-          f = __bfloat1622float2(p0[2]); acc0[b] += f.x * xb.x + f.y * xb.y;
-          f = __bfloat1622float2(p0[3]); acc0[b] += f.x * xb.z + f.y * xb.w;
-          if (DUAL) {
-            f = __bfloat1622float2(p1[0]); acc1[b] += f.x * xa.x + f.y * xa.y;
-            f = __bfloat1622float2(p1[1]); acc1[b] += f.x * xa.z + f.y * xa.w;
-            f = __bfloat1622float2(p1[2]); acc1[b] += f.x * xb.x + f.y * xb.y;
-            f = __bfloat1622float2(p1[3]); acc1[b] += f.x * xb.z + f.y * xb.w;
-          }
-        }
-      }
+    for (int m = 0; m < NM; m++) {
+      wr[m][i] = W + (size_t)(DUAL ? 2 * n + m : n) * a.K;             // dual: rows interleaved (gate_n, up_n)
+#pragma unroll
+      for (int b = 0; b < B; b++) acc[m][i][b] = 0.f;
     }
+  }
+#pragma unroll UN
+  for (int k = lane * 8; k < a.K; k += 256) {
+    uint4 q[NM][RW];
+#pragma unroll
+    for (int m = 0; m < NM; m++)
+#pragma unroll
+      for (int i = 0; i < RW; i++) q[m][i] = ldg_stream(wr[m][i] + k);
 #pragma unroll
     for (int b = 0; b < B; b++) {
-      float v0 = warp_sum(acc0[b]);
-      if (lane == 0) res[r * B + b] = v0;
-      if (DUAL) {
-        float v1 = warp_sum(acc1[b]);
-        if (lane == 0) res[32 * B + r * B + b] = v1;
-      }
+      const float4 xa = *(const float4*)(xs + (size_t)b * a.K + k);
+      const float4 xb = *(const float4*)(xs + (size_t)b * a.K + k + 4);
+#pragma unroll
+      for (int m = 0; m < NM; m++)
+#pragma unroll
+        for (int i = 0; i < RW; i++) {
+          const __nv_bfloat162* p = (const __nv_bfloat162*)&q[m][i];
+          float2 f;
+          f = __bfloat1622float2(p[0]); acc[m][i][b] += f.x * xa.x + f.y * xa.y;
+          f = __bfloat1622float2(p[1]); acc[m][i][b] += f.x * xa.z + f.y * xa.w;
+          f = __bfloat1622float2(p[2]); acc[m][i][b] += f.x * xb.x + f.y * xb.y;
+          f = __bfloat1622float2(p[3]); acc[m][i][b] += f.x * xb.z + f.y * xb.w;
+        }
     }
   }
+#pragma unroll
+  for (int i = 0; i < RW; i++)
+#pragma unroll
+    for (int b = 0; b < B; b++) {
+      const float v0 = warp_sum(acc[0][i][b]);
+      if (lane == 0) res[(w + 8 * i) * B + b] = v0;
+      if (DUAL) {
+        const float v1 = warp_sum(acc[NM - 1][i][b]);
+        if (lane == 0) res[32 * B + (w + 8 * i) * B + b] = v1;
+      }
+    }
   if (a.epi == EPI_ALLREDUCE && a.wait_ready && threadIdx.x == 0) sym_wait_ready(a.sym);
   __syncthreads();
-  matvec_epilogue<B>(a, res, DUAL);
+  matvec_epilogue<B, R>(a, res, DUAL);
   if (a.epi == EPI_ALLREDUCE) sym_kernel_end_barrier(a.sym, 0, gridDim.x, a.wait_ready != 0);
 }
 
@@ -442,15 +459,23 @@ static int launch_q(const MatvecArgs& a, cudaStream_t st) {
   }
   return launch_q_rw<WT, B, DUAL, 4>(a, st);
 }
-template <int B, bool DUAL>
-static int launch_bf16(const MatvecArgs& a, cudaStream_t st) {
+template <int B, bool DUAL, int RW>
+static int launch_bf16_rw(const MatvecArgs& a, cudaStream_t st) {
   const size_t smem = (size_t)B * a.K * 4 + 2 * 32 * B * sizeof(float);
-  auto kern = matvec_bf16_kernel<B, DUAL>;
+  auto kern = matvec_bf16_kernel<B, DUAL, RW>;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  return launch_pdl(kern, dim3((a.N + 31) / 32), dim3(256), smem, st, a);
+  return launch_pdl(kern, dim3((a.N + 8 * RW - 1) / (8 * RW)), dim3(256), smem, st, a);
+}
+template <int B, bool DUAL>
+static int launch_bf16(const MatvecArgs& a, cudaStream_t st) {
+  if constexpr (!DUAL) {      // fewer rows per CTA where whole ones would leave SMs idle
+    if ((a.N + 31) / 32 < 3 * 148)      // (long rows: two, so that the activations are staged half as often)
+      return a.K >= 8192 ? launch_bf16_rw<B, DUAL, 2>(a, st) : launch_bf16_rw<B, DUAL, 1>(a, st);
+  }
+  return launch_bf16_rw<B, DUAL, 4>(a, st);
 }
 
 template <int B, bool DUAL>
@@ -493,7 +518,7 @@ B200_API int b200_matvec(int wt, const void* w, const void* w2, int N, int K, in
                          const float* resid, float* y, int ldy, void* oq, float* od, float* os16,
                          const SymTable* sym, size_t sym_off, int wait_ready, cudaStream_t st) {
   if (nb < 1 || nb > 8 || epi == EPI_ROPE_KV) return B200_ERR_BAD_ARG;
-  if (wt == WT_BF16 ? (K % 8 != 0) : (K % 256 != 0 && !(wt == WT_Q8R && K % 32 == 0))) return B200_ERR_BAD_ARG;
+  if (wt == WT_BF16 ? (K % 8 != 0 || (uintptr_t)xf % 16) : (K % 256 != 0 && !(wt == WT_Q8R && K % 32 == 0))) return B200_ERR_BAD_ARG;
   if (epi == EPI_SWIGLU_Q8 && N % 32) return B200_ERR_BAD_ARG;
   MatvecArgs a = {};
   a.w = (const uint8_t*)w; a.w2 = (const __half*)w2; a.N = N; a.K = K; a.nb = nb;

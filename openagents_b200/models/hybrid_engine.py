@@ -79,8 +79,9 @@ class HybridEngine(PagedEngine):
         slots = 0 if not cfg.has_state else (state_slots if state_slots is not None else max_batch)
         self._init_paged(device, max_batch, max_ctx, n_pages, max_tokens, canaries, state_slots=slots)
         self.dp = _up(self.d, 8)
-        # decode batches up to this size take the mat-vec kernels
-        self.small_path_tokens = min(MATVEC_MAX_TOKENS, int(os.environ.get("B200_SMALL_PATH_TOKENS", 4)))
+        # Decode batches up to this size take the mat-vec kernels.  Measured (ms per step, one token, mat-vec / GEMM): width 2048
+        # 1.04 / 1.30, width 4096 4.41 / 4.19; the GEMM costs the same at eight tokens, the mat-vec grows with each.
+        self.small_path_tokens = min(MATVEC_MAX_TOKENS, int(os.environ.get("B200_SMALL_PATH_TOKENS", 1)))
         self._load(src)
         self._alloc()
 

@@ -464,7 +464,7 @@ def test_decode_batches_of_every_path(tmp_path):
     """Decode batches for the mat-vec path, the one-tile GEMM and beyond it (bf16), each sequence against itself alone."""
     cfg = CONFIGS["odd"]
     W = R.random_weights(cfg, seed=9)
-    for B in (2, 7, 40, 70):
+    for B in (1, 2, 7, 40, 70):
         be = open_model(tmp_path / str(B), cfg, W, "bfloat16", max_num_seqs=B, max_ctx=64, max_tokens=B * 12)
         toks = [tokens(cfg, 3 + b % 9, 50 + b) for b in range(B)]
         more = [tokens(cfg, 3, 500 + b) for b in range(B)]
