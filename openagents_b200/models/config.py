@@ -209,7 +209,8 @@ def _folirax(c: dict, ranks: dict[int, int], name: str, context: int) -> ModelCo
         if kind == "gla":
             m = MixerSpec("gla", **common, tau=_need(mx, "tau", float, w2), rank=ranks.get(i, MixerSpec.rank))
         elif kind == "attention":
-            rot, src = _need(mx, "rot", dict, w2), mx.get("kv_from")
+            src = mx.get("kv_from")
+            rot = {"base": 1.0, "dims": 0} if "rot" in mx and mx["rot"] is None else _need(mx, "rot", dict, w2)      # null: no rotation
             m = MixerSpec("attention", **common, kv_heads=_need(mx, "kv_heads", int, w2), scale=_need(mx, "scale", float, w2),
                           rope_base=_need(rot, "base", float, w2 + "rot."), rope_dims=_need(rot, "dims", int, w2 + "rot."),
                           qk_norm=True, head_gate=True, kv_from=None if src is None else _need(mx, "kv_from", int, w2))
@@ -232,7 +233,7 @@ def _folirax(c: dict, ranks: dict[int, int], name: str, context: int) -> ModelCo
     return ModelConfig(arch="folirax", n_layers=len(layers), d_model=_need(c, "width", int, ""), vocab=_need(c, "vocab", int, ""),
                        n_heads=max(m.heads for m in mx), n_kv_heads=max(1, *(m.kv_heads for m in mx)), head_dim=max(m.dim for m in mx),
                        ffn=max(l.ffn for l in layers), context=context, norm_eps=_need(_need(c, "norm", dict, ""), "eps", float, "norm."),
-                       layers=tuple(layers), logit_scale=_need(c, "logit_scale", float, ""),
+                       layers=tuple(layers), logit_scale=1.0 if c.get("logit_scale") is None else _need(c, "logit_scale", float, ""),
                        logit_softcap=0.0 if cap is None else _need(c, "logit_softcap", float, ""), name=name)
 
 

@@ -76,7 +76,8 @@ class HybridEngine(PagedEngine):
             raise ValueError(f"{type(self).__name__} serves {self.ARCHS} models, not {cfg.arch!r}")
         self.cfg, self.d = cfg, cfg.d_model
         self.exact = dtype == "float32"
-        slots = 0 if not cfg.has_state else (state_slots if state_slots is not None else max_batch)
+        # one state slot per sequence that is open: the running ones, and some for idle sessions and scoring
+        slots = 0 if not cfg.has_state else (state_slots if state_slots is not None else max_batch + max(4, max_batch // 4))
         self._init_paged(device, max_batch, max_ctx, n_pages, max_tokens, canaries, state_slots=slots)
         self.dp = _up(self.d, 8)
         # Decode batches up to this size take the mat-vec kernels.  Measured (ms per step, one token, mat-vec / GEMM): width 2048

@@ -62,9 +62,9 @@ def engine_class(cfg: ModelConfig):
 
 
 def build_engine(src, device, max_batch: int, max_ctx: int, max_tokens: int = 4096, n_pages: int | None = None, dtype: str = "bfloat16",
-                 tp_rank: int = 0, tp_world: int = 1, ep_rank: int = 0, ep_world: int = 1, comm=None, **options):
+                 tp_rank: int = 0, tp_world: int = 1, ep_rank: int = 0, ep_world: int = 1, comm=None, state_slots: int | None = None, **options):
     """The engine for ``src.cfg``.  ``dtype``: "float32" computes everything in true 32-bit, for the families that have it;
-    ``options`` are the family's own."""
+    ``state_slots``: sequences that may be open at a time, for the families with a recurrent state; ``options`` are the family's own."""
     cfg, cls = src.cfg, engine_class(src.cfg)
     if dtype not in COMPUTE_DTYPES:
         raise ValueError(f"dtype is one of {COMPUTE_DTYPES}")
@@ -72,7 +72,7 @@ def build_engine(src, device, max_batch: int, max_ctx: int, max_tokens: int = 40
     if cfg.layers:
         if max(tp_world, ep_world) > 1:
             raise ValueError(f"{cfg.arch} models are served on one GPU")
-        return cls(cfg, src, dtype=dtype, **common)
+        return cls(cfg, src, dtype=dtype, state_slots=state_slots, **common)
     if dtype != "bfloat16":
         raise ValueError(f"{cfg.arch} models have no 32-bit mode")
     if cfg.n_experts:

@@ -429,7 +429,7 @@ def make_handler(state: ServerState):
                 return self._json(200, {"object": "list", "data": [
                     {"id": m.id, "object": "model", "created": m.created, "owned_by": ENGINE_NAME,
                      "artifact_digest": m.artifact_digest, "architecture": m.backend.cfg.arch,
-                     "chat_template_digest": CHAT_TEMPLATE_DIGEST, "context_length": m.backend.cfg.context}
+                     "chat_template_digest": CHAT_TEMPLATE_DIGEST, "context_length": m.backend.max_context if m.backend.cfg.layers else m.backend.cfg.context}
                     for m in state.models.values()]})
             if path == "/psionic/management/status":
                 return self._json(200, state.status())

@@ -81,7 +81,8 @@ def main(argv=None) -> int:
     from ..models.paged import PAGE
     from .backend import CudaBackend
     pages = max(1, (a.max_tokens + PAGE - 1) // PAGE)
-    backend = CudaBackend.open(a.model, max_num_seqs=MAX_LIVE, max_ctx=pages * PAGE, max_tokens=pages * PAGE, dtype=a.dtype, n_pages=pages)
+    backend = CudaBackend.open(a.model, max_num_seqs=MAX_LIVE, max_ctx=pages * PAGE, max_tokens=pages * PAGE, dtype=a.dtype, n_pages=pages,
+                               state_slots=MAX_LIVE)
     runner = TraceRunner(backend, a.out)
     for line in sys.stdin:
         if line.strip():

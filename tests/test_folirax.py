@@ -27,12 +27,17 @@ def test_configuration_is_read_layer_by_layer():
     assert [l.ffn for l in c.layers] == [36, 100, 0] and (c.logit_scale, c.logit_softcap) == (0.7, 20.0)
     assert c.has_state and not config_from_json(dict(CFG, layers=[CFG["layers"][1]])).has_state
     assert config_from_json(hybrid_to_json(c)) == c
+    plain = json.loads(json.dumps(dict(CFG, logit_scale=None, logit_softcap=None)))
+    plain["layers"][1]["mixer"]["rot"] = None
+    plain["layers"][2]["mixer"]["rot"] = None
+    p = config_from_json(plain)
+    assert (p.logit_scale, p.logit_softcap, p.layers[1].mixer.rope_dims) == (1.0, 0.0, 0)
     assert ModelConfig.from_gguf_metadata(c.to_gguf_metadata()) == c
 
 
 @pytest.mark.parametrize("path,value", [
-    (("architecture",), "Other"), (("layers",), []), (("layers",), None), (("width",), "72"), (("norm",), {}), (("logit_scale",), None),
-    (("layers", 0, "type"), "conv"), (("layers", 0, "mixer", "tau"), 0), (("layers", 1, "mixer", "rot"), None), (("layers", 1, "mixer", "rot", "dims"), 48),
+    (("architecture",), "Other"), (("layers",), []), (("layers",), None), (("width",), "72"), (("norm",), {}), (("logit_scale",), "1"),
+    (("layers", 0, "type"), "conv"), (("layers", 0, "mixer", "tau"), 0), (("layers", 1, "mixer", "rot"), 16), (("layers", 1, "mixer", "rot", "dims"), 48),
     (("layers", 1, "mixer", "rot", "dims"), 7), (("layers", 1, "mixer", "kv_heads"), 4), (("layers", 1, "mixer", "dim"), True), (("layers", 1, "mlp", "kind"), "moe"),
     (("layers", 2, "mixer", "kv_from"), 0), (("layers", 2, "mixer", "kv_from"), 2), (("layers", 2, "mixer", "kv_from"), -1), (("layers", 2, "mixer", "vdim"), 16)])
 def test_a_bad_configuration_is_refused(path, value):

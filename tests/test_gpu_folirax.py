@@ -311,6 +311,7 @@ CONFIGS = {
 
 def open_model(tmp_path, cfg, W, dtype="float32", max_num_seqs=4, max_ctx=512, max_tokens=512, **kw):
     from openagents_b200.serve.backend import CudaBackend
+    kw.setdefault("state_slots", max_num_seqs)
     return CudaBackend.open(R.save_model(str(tmp_path / "m"), cfg, W), max_num_seqs=max_num_seqs, max_ctx=max_ctx, max_tokens=max_tokens,
                             dtype=dtype, **kw)
 
@@ -584,3 +585,42 @@ def test_trace_runner(tmp_path):
         fa, fb = R.forward(cfg, W, ta, R.Sequence()), R.forward(cfg, W, tb, R.Sequence())
         got = torch.from_numpy(np.concatenate([np.fromfile(out / f"{i}.f32", dtype="<f4") for i in (0, 2)])).view(4, -1)
         close(got, torch.stack([fa[0], fa[29], fa[39], fb[20]]), dtype)
+
+
+def test_http_server_on_a_checkpoint_folder(tmp_path):
+    """The server as `b200-serve -m FOLDER --dtype float32` builds it: completions, sessions beyond the state slots (idle ones give
+    theirs up), log-probabilities, and the answer of the plain implementation."""
+    import json
+    import threading
+    import urllib.request
+
+    from openagents_b200.serve.server import build_state, parse_args, serve
+    cfg = dict(CONFIGS["recurrent"], vocab=300)
+    W = R.random_weights(cfg, seed=16)
+    a = parse_args(["-m", R.save_model(str(tmp_path / "tiny-folirax"), cfg, W), "--dtype", "float32", "--max-num-seqs", "2", "--max-ctx", "512",
+                    "--speculation", "n_gram"])
+    state = build_state(a.model, a.backend, a.max_num_seqs, a.kv_page_size, a.max_ctx, dtype=a.dtype)
+    httpd = serve(state, "127.0.0.1", 0)
+    threading.Thread(target=httpd.serve_forever, daemon=True).start()
+    base = f"http://127.0.0.1:{httpd.server_address[1]}"
+
+    def post(path, obj):
+        req = urllib.request.Request(base + path, json.dumps(obj).encode(), {"Content-Type": "application/json"})
+        with urllib.request.urlopen(req, timeout=60) as r:
+            return json.loads(r.read())
+    try:
+        rows = json.loads(urllib.request.urlopen(base + "/v1/models", timeout=30).read())["data"]
+        assert [m["id"] for m in rows] == ["tiny-folirax"]
+        out = post("/v1/completions", {"model": "tiny-folirax", "prompt": "hello there", "max_tokens": 8, "temperature": 0})
+        ids, _ = R.generate(cfg, W, list(b"hello there"), 8)
+        stop = ids.index(256) if 256 in ids else len(ids)
+        assert out["choices"][0]["text"] == bytes(i for i in ids[:stop] if i < 256).decode("utf-8", "replace")
+        slots = state.models["tiny-folirax"].backend.kv_stats()["state_slots_total"]
+        for _ in range(slots + 3):
+            sid = post("/v1/sessions", {"model": "tiny-folirax"})["id"]
+            assert "output_text" in post(f"/v1/sessions/{sid}/responses", {"prompt": "again", "max_tokens": 3})
+        assert state.sessions_evicted > 0
+    finally:
+        httpd.shutdown()
+        for m in state.models.values():
+            m.close()
