@@ -129,9 +129,9 @@ def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
         bench(f"rmsnorm [{n}]", lambda: ops.rmsnorm(x, gn, 1e-6, hb=hb), n * d * 6)
     # ---- attention: projection finish, prompt, decode
     pages = (ctx + 15) // 16
-    for n, seqs in ((T, 1), (B, B)):
+    for n, seqs in ((T, 1), (B, B), (1, 1)):
         N = (H + 2 * G) * D + (H + 7) // 8 * 8
-        row, pos, slot = rnd(n, N), i32([ctx - 1] * n if seqs > 1 else list(range(n))), i32(list(range(n)))
+        row, pos, slot = rnd(n, N), i32([ctx - 1] * n if n != T else list(range(n))), i32(list(range(n)))
         q16, q32 = bf(n, H * D).half(), rnd(n, H * D)
         kc, vc = rnd(seqs * pages + 1, G, 16, D).half(), rnd(seqs * pages + 1, G, 16, D).half()
         tab, tabf = ops.rope_table(ctx, at.rope_dims, at.rope_base, dev), ops.rope_table(ctx, D, at.rope_base, dev)
@@ -151,11 +151,11 @@ def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
                 bench(f"{nm} [{T}]", lambda: ops.attn_prefill_tc05(q16, kc, vc, table, z, lens, lens, 1, T, H, G, out_bf16=o, status=st, dk=D, dv=D, gate=gt),
                       T * (H + G) * D * 4, fl, like=lk and f"{lk} [{T}]")
         else:
-            o, S = bf(B, H * D), 4
-            sc, cnt = rnd(ops.attn_decode_scratch_floats(B, H, G, D, S)), torch.zeros(B * H, dtype=torch.int32, device=dev)
+            o, S = bf(n, H * D), 4
+            sc, cnt = rnd(ops.attn_decode_scratch_floats(n, H, G, D, S)), torch.zeros(n * H, dtype=torch.int32, device=dev)
             for nm, gt, lk in (("attn_decode gated", gate, "attn_decode"), ("attn_decode", None, None)):
-                bench(f"{nm} [{B} x {ctx}]", lambda: ops.attn_decode(q32, kc, vc, table, lens, B, H, G, D, S=S, gate=gt, out_bf16=o, scratch=sc, counters=cnt,
-                                                                     status=st), B * ctx * G * D * 4, like=lk and f"{lk} [{B} x {ctx}]")
+                bench(f"{nm} [{n} x {ctx}]", lambda: ops.attn_decode(q32, kc, vc, table, lens, n, H, G, D, S=S, gate=gt, out_bf16=o, scratch=sc, counters=cnt,
+                                                                     status=st), n * ctx * G * D * 4, like=lk and f"{lk} [{n} x {ctx}]")
     # ---- gated linear attention
     Hg, dk, dv, r = gl.heads, gl.dim, gl.vdim, gl.rank
     qk, vv = Hg * dk, Hg * dv
@@ -172,9 +172,9 @@ def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
         bench(f"gla_chunked [{seqs} x {T}] (3 kernels)", lambda: ops.gla_chunked(row, offs, r, a2, b2, w, state, qs, ql, ql, sl, seqs, Hg, dk, dv, dv, 16.0, dk ** -0.5,
                                                                                    1e-6, T, ws, out_bf16=out), n * (ld * 4 + vv * 2), fl, like=f"attn_prefill_tc05 [{T}]")
     for n in (1, B):
-        row, out, sl, one = rnd(n, ld), bf(n, vv), i32(list(range(n))), i32([1] * n)
-        bench(f"gla_recurrent [{n}]", lambda: ops.gla_recurrent(row, offs, r, a2, b2, w, state, sl, one, i32([ctx] * n), sl, n, Hg, dk, dv, dv, 16.0, dk ** -0.5, 1e-6,
-                                                                out_bf16=out), n * (8 * Hg * dk * dv + ld * 4), like=f"attn_decode [{B} x {ctx}]")
+        row, out, sl, one, held = rnd(n, ld), bf(n, vv), i32(list(range(n))), i32([1] * n), i32([ctx] * n)
+        bench(f"gla_recurrent [{n}]", lambda: ops.gla_recurrent(row, offs, r, a2, b2, w, state, sl, one, held, sl, n, Hg, dk, dv, dv, 16.0, dk ** -0.5, 1e-6,
+                                                                out_bf16=out), n * (8 * Hg * dk * dv + ld * 4), like=f"attn_decode [{n} x {ctx}]")
     # ---- products
     for n in (T, B):
         a, up, gu = bf(n, d), bf(F, d), bf(2 * F, d)

@@ -53,8 +53,17 @@ __global__ void __launch_bounds__(256) gla_recurrent_kernel(const GlaArgs a) {
   __shared__ float red[32];
   __shared__ float s_part[2];              // this CTA's sum of squares, by token parity
   pdl_trigger();
-  pdl_wait();
   const int h = blockIdx.x / CL, b = blockIdx.y, tid = threadIdx.x;
+  // One channel per thread (heads of up to 256) and up to 16 ranks: the decay's weights are read while the projection still runs.
+  const bool held = a.dim <= 256 && a.rank <= 16;
+  float wz[16], bz = 0.f;
+  if (held && tid < a.dim) {
+    bz = a.b2[h * a.dim + tid];
+#pragma unroll
+    for (int r = 0; r < 16; r++) wz[r] = r < a.rank ? a.a2[(size_t)r * a.H * a.dim + h * a.dim + tid] : 0.f;
+  }
+  const float wo = (tid < W && e0 + tid < a.vdim) ? a.w[e0 + tid] : 0.f;
+  pdl_wait();
   const int n = a.q_len[b], t0 = a.q_start[b], slot = a.slot[b];
   bool fresh = a.ctx_len[b] - n == 0 || slot < 0;
   const int groups = 256 / nv, grp = tid / nv, col = tid % nv;
@@ -71,7 +80,21 @@ __global__ void __launch_bounds__(256) gla_recurrent_kernel(const GlaArgs a) {
     float4 cur[kGlaRows], nxt[kGlaRows];
     fetch(cur, grp);                       // in flight while the decays are computed
     const float* row = a.in + (size_t)(t0 + i) * a.ld;
-    for (int d = tid; d < a.dim; d += 256) {
+    const float gate = (tid < W && e0 + tid < a.vdim) ? row[a.g_off + h * a.vdim + e0 + tid] : 0.f;      // used at the end
+    if (held && tid < a.dim) {
+      const int c = h * a.dim + tid;
+      const float q = row[a.q_off + c], k = row[a.k_off + c];
+      float x[16];
+#pragma unroll
+      for (int r = 0; r < 16; r++) x[r] = r < a.rank ? row[a.a_off + r] : 0.f;
+      float z = bz;
+#pragma unroll
+      for (int r = 0; r < 16; r++) z = fmaf(wz[r], x[r], z);
+      s_q[tid] = q * a.q_scale;
+      s_k[tid] = k;
+      s_al[tid] = expf(log_decay(z, a.inv_tau));
+    }
+    for (int d = held ? a.dim : tid; d < a.dim; d += 256) {
       const int c = h * a.dim + d;
       float z = a.b2[c];
 #pragma unroll 8
@@ -127,8 +150,8 @@ __global__ void __launch_bounds__(256) gla_recurrent_kernel(const GlaArgs a) {
     for (int e = tid; e < W; e += 256) {
       float o = 0.f;
       if (e0 + e < a.vdim) {
-        const float g = row[a.g_off + h * a.vdim + e0 + e];
-        o = s_o[e] * r * a.w[e0 + e] * (g / (1.f + expf(-g)));
+        const float g = e < 256 ? gate : row[a.g_off + h * a.vdim + e0 + e];
+        o = s_o[e] * r * (e < 256 ? wo : a.w[e0 + e]) * (g / (1.f + expf(-g)));
       }
       const size_t at = (size_t)(t0 + i) * a.ldo + (size_t)h * a.VP + e0 + e;
       if (a.out_f32) a.out_f32[at] = o;

@@ -45,7 +45,7 @@ def test_rotation_then_unit_norm_then_cache(style):
     """Partial rotation, unit-RMS queries and keys, the padded cache rows, and a layer without keys of its own."""
     from openagents_b200.ops import cuda_ops as ops
     g = torch.Generator().manual_seed(1)
-    for H, G, dim, vdim, DK, DV, rot in ((6, 2, 40, 24, 64, 64, 16), (4, 4, 96, 48, 96, 48, 96), (2, 1, 10, 6, 16, 8, 2), (3, 1, 72, 130, 72, 136, 0)):
+    for H, G, dim, vdim, DK, DV, rot in ((6, 2, 40, 24, 64, 64, 16), (4, 4, 104, 56, 104, 56, 104), (2, 1, 10, 6, 16, 8, 2), (3, 1, 72, 130, 72, 136, 0)):
         T = 5
         ld = H * dim + G * (dim + vdim) + 3
         row = torch.randn(T, ld, generator=g)
@@ -226,7 +226,7 @@ def _gla_case(T_list, pos_list, H, dim, vdim, rank, tau, z_shift, seed=0, z_scal
     return args, VP, torch.cat(want), want_state, args[6], slots
 
 
-GLA_SIZES = [(3, 32, 64, 16), (2, 24, 40, 5), (1, 128, 72, 20), (5, 64, 8, 1), (2, 160, 136, 33), (1, 256, 64, 16)]
+GLA_SIZES = [(3, 32, 56, 12), (4, 128, 256, 16), (2, 24, 40, 5), (1, 128, 72, 20), (5, 64, 8, 1), (2, 160, 136, 33), (1, 256, 64, 16)]
 
 
 @pytest.mark.parametrize("kind", ["recurrent", "chunked"])
