@@ -1,5 +1,5 @@
 // Paged-KV grouped-query attention for decode: one query token per sequence against a paged
-// fp16 K/V cache with 16-token pages, optional sliding window and learned sink logits.
+// fp16 K/V cache with 16-token pages, optional sliding window, chunks and learned sink logits.
 //
 // Work split: grid = (splits, kv_heads, sequences).  A CTA streams its share of one sequence's
 // pages for one KV head exactly once and serves all G query heads that share that KV head, so the
@@ -24,7 +24,7 @@ struct AttnDecArgs {
   const int* page_table;   // [B][max_pages]
   const int* seq_lens;     // [B] keys to attend (includes the current token)
   const float* sinks;      // [Hq] or null
-  int max_pages, Hq, Hkv, window, S;
+  int max_pages, Hq, Hkv, window, chunk, S;   // chunk > 0: keys of the token's own chunk of that many positions only
   int kv_rep, Hkv_cache;   // virtual KV heads per cache head (splits wide groups), heads in the cache
   int G;                   // query heads per (virtual) KV head
   const float* gate;       // [B][ldg] or null: head h's output is multiplied by sigmoid(gate[b][h])
@@ -117,7 +117,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const __grid_constant_
   pdl_trigger();
   pdl_wait();
   const int len = a.seq_lens[b];
-  const int first = (a.window > 0 && len > a.window) ? len - a.window : 0;
+  const int first = a.chunk > 0 ? (len - 1) / a.chunk * a.chunk : (a.window > 0 && len > a.window) ? len - a.window : 0;
   const int p_first = first >> 4, p_last = (len + 15) >> 4;
   const int per = (p_last - p_first + a.S - 1) / a.S;
   const int pa = p_first + split * per;
@@ -398,16 +398,16 @@ B200_API size_t b200_attn_decode_scratch_floats(int B, int Hq, int Hkv, int hd, 
 // hd: query / key head size, dv: value head size (64..256 and 64..128, multiples of 64).  counters: B * Hq ints, zero before first use.
 B200_API int b200_attn_decode(const float* q, const void* kc, const void* vc, const int* page_table,
                               int max_pages, int n_pages, const int* seq_lens, const float* sinks, int B,
-                              int Hq, int Hkv, int hd, int dv, int window, int S, const float* gate, int ldg, float* out_f32,
+                              int Hq, int Hkv, int hd, int dv, int window, int chunk, int S, const float* gate, int ldg, float* out_f32,
                               void* out_bf16, void* oq, float* od, float* os16, float* scratch, int* counters, int* status,
                               cudaStream_t st) {
-  if (Hkv < 1 || Hq % Hkv || S < 1) return B200_ERR_BAD_ARG;
+  if (Hkv < 1 || Hq % Hkv || S < 1 || chunk < 0 || (chunk && window)) return B200_ERR_BAD_ARG;
   int G = Hq / Hkv, rep = 1;
   while (G % rep || G / rep > 16) rep++;            // a group wider than the 16-row tile is served as several
   AttnDecArgs a;
   a.q = q; a.kc = (const __half*)kc; a.vc = (const __half*)vc; a.page_table = page_table;
   a.seq_lens = seq_lens; a.sinks = sinks; a.max_pages = max_pages; a.Hq = Hq; a.Hkv = Hkv * rep;
-  a.window = window; a.S = S; a.kv_rep = rep; a.Hkv_cache = Hkv; a.G = G / rep; a.gate = gate; a.ldg = ldg;
+  a.window = window; a.chunk = chunk; a.S = S; a.kv_rep = rep; a.Hkv_cache = Hkv; a.G = G / rep; a.gate = gate; a.ldg = ldg;
   a.out_f32 = out_f32; a.out_bf16 = (__nv_bfloat16*)out_bf16;
   a.oq = (int8_t*)oq; a.od = od; a.os16 = os16;
   a.part_acc = scratch;

@@ -1,7 +1,10 @@
 // Causal grouped-query flash attention for prefill on the 5th-generation tensor cores.
 //
 // Head sizes are template parameters (queries / keys DK = 64..256, values DV = 64 or 128, multiples of 64; other sizes are padded
-// in the cache); the figures below are those of DK = DV = 128.  An optional gate per head multiplies the output by a sigmoid.
+// in the cache); the figures below are those of DK = DV = 128.  An optional gate per head (or per output element) multiplies the output
+// by a sigmoid.  Differential attention gives a key/value head two key rows side by side: the query heads of either map load theirs.
+// Latent attention (LATENT): keys and values are plain rows of a workspace that holds the expanded context, and the last columns
+// of every key, the rotated part all heads share, come from the paged latent cache.
 //
 // One CTA = 128 query rows of one head.  Roles: warps 0 and 10 are the TMA producers (a ring of K / V
 // blocks of 64 keys gathered page by page from the paged fp16 cache), warps 1 and 11 issue the two
@@ -19,7 +22,7 @@
 // than 8 (a factor 256, well inside fp16 for P and fp32 for O and the row sum); then the row's owner
 // thread rescales the O row in tensor memory (tcgen05.ld / st) between two PV products.  After the
 // first key blocks of a causal row that is rare, so the steady state has no O traffic at all.
-// Sliding windows, learned sink logits and a context that is longer than the chunk (chunked prefill,
+// Sliding windows, chunks, learned sink logits and a context that is longer than the chunk (chunked prefill,
 // prefix reuse) are handled by the mask and the block range.  Math as in the reference's attention
 // (apps/openagents.com/workers/api/src/cs336-a1-real-gradient-workload.ts:478-518: max-subtract,
 // exp, normalise).  Every wait is bounded; a wait that runs out sets the status word and the CTA
@@ -49,6 +52,13 @@ struct PrefillArgs {
   const float* gate;       // [T_total][ldg] or null: head h's output is multiplied by sigmoid(gate[t][h])
   int ldg;
   int max_pages, Hq, Hkv, window, T_total;
+  int chunk;               // > 0: a query sees its own chunk of that many positions only
+  int maps;                // 2: key/value heads have two key rows of DK columns (query heads in the order (kv head, map, head of the group))
+  int gate_elem;           // the gate has a column per output column instead of one per head
+  float* out_f32;          // written instead of out where given
+  // LATENT
+  const int* base;         // [n_seqs] first workspace row of each sequence
+  int k_boxes, v_col, r_col;   // 64-column boxes of a key's own part; first value column of the workspace; first rotated column of the cache
 };
 
 // fp16 x fp16 -> fp32 instruction descriptor; b_mn: the B operand is MN-major.
@@ -100,9 +110,10 @@ __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.
 template <int DK, int DV>
 constexpr int kv_stages() { return 196608 / (KB * (DK + DV) * 2) < 4 ? 196608 / (KB * (DK + DV) * 2) : 4; }
 
-template <int DK, int DV>
+template <int DK, int DV, bool LATENT>
 __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap tmK,
                                                                    const __grid_constant__ CUtensorMap tmV,
+                                                                   const __grid_constant__ CUtensorMap tmR,
                                                                    const PrefillArgs a) {
   constexpr int K_BYTES = KB * DK * 2, V_BYTES = KB * DV * 2, STAGE_BYTES = K_BYTES + V_BYTES, KV_STAGES = kv_stages<DK, DV>();
   static_assert(256 + DV + DK / 2 <= (int)TMEM_COLS && KV_STAGES >= 2, "head sizes");
@@ -159,10 +170,10 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(const __grid_
   const int q0 = qb * QB;
   const bool live = q0 < qlen;            // a dead CTA still goes through the common exit (it holds tensor memory)
   const int ctx = a.ctx_len[seq], qs = a.q_start[seq];
-  const int kh = h / (a.Hq / a.Hkv);
+  const int row_k = h / (a.Hq / (a.Hkv * a.maps)), kh = row_k / a.maps, k_col = row_k % a.maps * DK;
   const int pos0 = ctx - qlen + q0;       // absolute position of this CTA's first query row
   const int k_hi = min(ctx, pos0 + QB);   // keys [k_lo, k_hi) can matter to some row
-  const int k_lo = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
+  const int k_lo = a.chunk > 0 ? pos0 / a.chunk * a.chunk : a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
   const int jb0 = k_lo / KB, jb1 = live ? (k_hi + KB - 1) / KB : jb0;   // key blocks [jb0, jb1)
   const int nb = jb1 - jb0;
   const uint32_t S_T = tmem_base, O_T = tmem_base + 256;   // S buffers at +0, +128; O at +256
@@ -188,12 +199,29 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(const __grid_
         uint8_t* dst = sKV + (size_t)s * STAGE_BYTES + (is_k ? 0 : K_BYTES);
         const int boxes = (is_k ? DK : DV) / 64;
         const CUtensorMap* tm = is_k ? &tmK : &tmV;
+        if constexpr (LATENT) {
+          const int row = a.base[seq] + (jb0 + j) * KB;             // 128 workspace rows at a time; rows past the context are masked
+          if (!is_k) {
+            for (int c = 0; c < DV / 64; c++) tma_load_2d(smem_u32(dst + c * BOX_BYTES), tm, bar, a.v_col + h * DV + c * 64, row);
+          } else {
+            for (int c = 0; c < a.k_boxes; c++) tma_load_2d(smem_u32(dst + c * BOX_BYTES), tm, bar, (h * a.k_boxes + c) * 64, row);
+#pragma unroll
+            for (int p = 0; p < KB / 16; p++) {
+              const int pi = (jb0 + j) * (KB / 16) + p;
+              const int page = (pi * 16 < ctx) ? pt[pi] : 0;
+              for (int c = a.k_boxes; c < DK / 64; c++)
+                tma_load_2d(smem_u32(dst + c * BOX_BYTES + p * 2048), &tmR, bar, a.r_col + (c - a.k_boxes) * 64, page * 16);
+            }
+          }
+          continue;
+        }
 #pragma unroll
         for (int p = 0; p < KB / 16; p++) {
           const int pi = (jb0 + j) * (KB / 16) + p;
           const int page = (pi * 16 < ctx) ? pt[pi] : 0;          // pages past the context are masked anyway
           const int row = (page * a.Hkv + kh) * 16;
-          for (int hf = 0; hf < boxes; hf++) tma_load_2d(smem_u32(dst + hf * BOX_BYTES + p * 2048), tm, bar, hf * 64, row);
+          for (int hf = 0; hf < boxes; hf++)
+            tma_load_2d(smem_u32(dst + hf * BOX_BYTES + p * 2048), tm, bar, (is_k ? k_col : 0) + hf * 64, row);
         }
       }
     }
@@ -238,6 +266,8 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(const __grid_
     const int hsel = (warp - 2) >> 2;            // 0: keys 0..31 of a block, output columns 0..63; 1: the other half
     const int row = q * 32 + lane;               // query row of this thread (shared with the partner warp's same lane)
     const int qpos = pos0 + row;
+    const int row_lo = a.chunk > 0 ? qpos / a.chunk * a.chunk : a.window > 0 ? qpos - a.window + 1 : 0;     // first key this row sees
+    const int lo_max = a.chunk > 0 ? (pos0 + QB - 1) / a.chunk * a.chunk : a.window > 0 ? pos0 + QB - a.window : 0;   // of the CTA's last row
     const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
     constexpr int HK = KB / 2, HO = DV / 2;
     float m_used = -INFINITY, l = 0.f;     // exponent offset of this row (log2 units) and this warp's part of the row sum
@@ -291,12 +321,12 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(const __grid_
       if (lane == 0) mbar_arrive(smem_u32(s_empty + b));
       // mask, maximum of this half, swap with the partner warp
       const int kb0 = (jb0 + j) * KB;
-      const bool edge = kb0 + KB - 1 > pos0 || kb0 + KB > ctx || (a.window > 0 && kb0 < pos0 + QB - a.window);
+      const bool edge = kb0 + KB - 1 > pos0 || kb0 + KB > ctx || kb0 < lo_max;
       if (edge) {
 #pragma unroll
         for (int i = 0; i < HK; i++) {
           const int kp = kb0 + hsel * HK + i;
-          if (kp > qpos || kp >= ctx || (a.window > 0 && kp <= qpos - a.window)) sv[i] = -INFINITY;
+          if (kp > qpos || kp >= ctx || kp < row_lo) sv[i] = -INFINITY;
         }
       }
       float mx0 = fmaxf(sv[0], sv[1]), mx1 = fmaxf(sv[2], sv[3]);
@@ -371,14 +401,31 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(const __grid_
       if (a.sinks) l += (m_used == -INFINITY) ? 1.f : ex2_approx(a.sinks[h] * kLog2e - m_used);
       float inv = l > 0.f ? 1.f / l : 0.f;
       const bool wr = ok && row < qlen - q0;
-      if (a.gate && wr) inv *= 1.f / (1.f + __expf(-a.gate[(size_t)(qs + q0 + row) * a.ldg + h]));
-      __nv_bfloat16* dst = a.out + (size_t)(qs + q0 + row) * a.Hq * DV + (size_t)h * DV + hsel * HO;
+      if (a.gate && !a.gate_elem && wr) inv *= 1.f / (1.f + __expf(-a.gate[(size_t)(qs + q0 + row) * a.ldg + h]));
+      const size_t at = (size_t)(qs + q0 + row) * a.Hq * DV + (size_t)h * DV + hsel * HO;
+      __nv_bfloat16* dst = a.out + at;
+      const float* gp = a.gate && a.gate_elem ? a.gate + (size_t)(qs + q0 + row) * a.ldg + (size_t)h * DV + hsel * HO : nullptr;
 #pragma unroll
       for (int c = 0; c < HO / 32; c++) {
         uint32_t r[32];
         tmem_ld32(O_T + lane_addr + hsel * HO + c * 32, r);
         tmem_ld_wait();
-        if (wr) {
+        if (wr && gp) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 4) {
+            const float4 g = *(const float4*)(gp + c * 32 + i);
+            r[i] = __float_as_uint(__uint_as_float(r[i]) / (1.f + __expf(-g.x)));
+            r[i + 1] = __float_as_uint(__uint_as_float(r[i + 1]) / (1.f + __expf(-g.y)));
+            r[i + 2] = __float_as_uint(__uint_as_float(r[i + 2]) / (1.f + __expf(-g.z)));
+            r[i + 3] = __float_as_uint(__uint_as_float(r[i + 3]) / (1.f + __expf(-g.w)));
+          }
+        }
+        if (wr && a.out_f32) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 4)
+            *(float4*)(a.out_f32 + at + c * 32 + i) = make_float4(__uint_as_float(r[i]) * inv, __uint_as_float(r[i + 1]) * inv,
+                                                                  __uint_as_float(r[i + 2]) * inv, __uint_as_float(r[i + 3]) * inv);
+        } else if (wr) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
             uint4 v;
@@ -398,17 +445,11 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc05_kernel(const __grid_
   if (threadIdx.x == 0 && *abort_flag && a.status) atomicExch(a.status, (int)B200_ERR_TIMEOUT_MMA);
 }
 
-template <int DK, int DV>
-int launch_prefill(const void* kc, const void* vc, int n_pages, const PrefillArgs& a, int n_seqs, int max_q, cudaStream_t st) {
-  CUtensorMap tk, tv;
-  const uint64_t rows = (uint64_t)n_pages * a.Hkv * 16;
-  int rc = make_tmap_2d(&tk, kc, 2, rows, DK, (uint64_t)DK * 2, 16, 64, true);
-  if (rc) return rc;
-  rc = make_tmap_2d(&tv, vc, 2, rows, DV, (uint64_t)DV * 2, 16, 64, true);
-  if (rc) return rc;
+template <int DK, int DV, bool LATENT>
+int run_prefill(const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tr, const PrefillArgs& a, int n_seqs, int max_q, cudaStream_t st) {
   constexpr size_t smem = 1024 + (size_t)kv_stages<DK, DV>() * KB * (DK + DV) * 2 + 32 * 8 + 2 * 2 * 128 * 4;
   static_assert(smem <= 232448, "shared memory per CTA");
-  auto kern = attn_prefill_tc05_kernel<DK, DV>;
+  auto kern = attn_prefill_tc05_kernel<DK, DV, LATENT>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -416,19 +457,32 @@ int launch_prefill(const void* kc, const void* vc, int n_pages, const PrefillArg
     configured = true;
   }
   dim3 grid((max_q + QB - 1) / QB, a.Hq, n_seqs);
-  return launch_pdl(kern, grid, dim3(384), smem, st, tk, tv, a);
+  return launch_pdl(kern, grid, dim3(384), smem, st, tk, tv, tr, a);
+}
+
+template <int DK, int DV>
+int launch_prefill(const void* kc, const void* vc, int n_pages, const PrefillArgs& a, int n_seqs, int max_q, cudaStream_t st) {
+  CUtensorMap tk, tv;
+  const uint64_t rows = (uint64_t)n_pages * a.Hkv * 16;
+  int rc = make_tmap_2d(&tk, kc, 2, rows, (uint64_t)a.maps * DK, (uint64_t)a.maps * DK * 2, 16, 64, true);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tv, vc, 2, rows, DV, (uint64_t)DV * 2, 16, 64, true);
+  if (rc) return rc;
+  return run_prefill<DK, DV, false>(tk, tv, tk, a, n_seqs, max_q, st);
 }
 
 }  // namespace
 
-// q fp16 [T_total][Hq * dk] (rotated, pre-scaled); kc fp16 [n_pages][Hkv][16][dk], vc [n_pages][Hkv][16][dv];
-// out bf16 [T_total][Hq * dv].  Sequences as in b200_attn_prefill; max_q = longest chunk.
+// q fp16 [T_total][Hq * dk] (rotated, pre-scaled); kc fp16 [n_pages][Hkv][16][maps * dk], vc [n_pages][Hkv][16][dv];
+// out bf16 [T_total][Hq * dv], or the same in fp32 to out_f32.  Sequences as in b200_attn_prefill; max_q = longest chunk.
 B200_API int b200_attn_prefill_tc05(const void* q, const void* kc, const void* vc, const int* page_table, int max_pages,
                                     int n_pages, const int* q_start, const int* q_len, const int* ctx_len, int n_seqs,
                                     int max_q, int T_total, int Hq, int Hkv, int dk, int dv, int window, const float* sinks,
-                                    const float* gate, int ldg, void* out, int* status, cudaStream_t st) {
-  if (Hkv < 1 || Hq % Hkv || n_seqs < 1 || max_q < 1 || !page_table) return B200_ERR_BAD_ARG;
-  PrefillArgs a;
+                                    const float* gate, int ldg, void* out, int chunk, int maps, float* out_f32, int* status, cudaStream_t st) {
+  if (Hkv < 1 || maps < 1 || Hq % (Hkv * maps) || n_seqs < 1 || max_q < 1 || !page_table || chunk < 0 || (chunk && window) || (!out && !out_f32))
+    return B200_ERR_BAD_ARG;
+  PrefillArgs a = {};
+  a.chunk = chunk; a.maps = maps; a.out_f32 = out_f32;
   a.q = (const __half*)q; a.T_total = T_total; a.gate = gate; a.ldg = ldg;
   a.page_table = page_table; a.q_start = q_start; a.q_len = q_len; a.ctx_len = ctx_len; a.sinks = sinks;
   a.out = (__nv_bfloat16*)out; a.status = status; a.max_pages = max_pages; a.Hq = Hq; a.Hkv = Hkv; a.window = window;
@@ -441,6 +495,38 @@ B200_API int b200_attn_prefill_tc05(const void* q, const void* kc, const void* v
     case 192128: return launch_prefill<192, 128>(kc, vc, n_pages, a, n_seqs, max_q, st);
     case 256064: return launch_prefill<256, 64>(kc, vc, n_pages, a, n_seqs, max_q, st);
     case 256128: return launch_prefill<256, 128>(kc, vc, n_pages, a, n_seqs, max_q, st);
+  }
+  return B200_ERR_BAD_ARG;
+}
+
+// The same over an expanded context (latent attention): ws fp16 [ws_rows][ldw] holds, at row base[seq] + key, the keys' own parts (head h at
+// column h * kn) and from v_col on the values (head h at h * dv); the last rr columns of every key lie in the paged cache [n_pages][16][ks] from
+// column r_col on.  q fp16 [T_total][H * (kn + rr)]; gate fp32 [T_total][ldg] (or null) has a column per output column; kn, rr, dv multiples of 64.
+// ws must hold no infinities or NaNs anywhere (rows past a context meet zero weights).
+B200_API int b200_attn_prefill_latent(const void* q, const void* ws, long ws_rows, int ldw, int v_col, const int* base, const void* cache, int n_pages,
+                                      int ks, int r_col, const int* page_table, int max_pages, const int* q_start, const int* q_len, const int* ctx_len,
+                                      int n_seqs, int max_q, int T_total, int H, int kn, int rr, int dv, const float* sinks, const float* gate, int ldg,
+                                      void* out, int* status, cudaStream_t st) {
+  if (H < 1 || n_seqs < 1 || max_q < 1 || kn < 64 || kn % 64 || rr < 64 || rr % 64 || v_col % 8 || r_col % 8 || ldw % 8 || ks % 8 || v_col < H * kn ||
+      ldw < v_col + H * dv || ks < r_col + rr || (gate && (ldg % 4 || ldg < H * dv || ((uintptr_t)gate & 15))))
+    return B200_ERR_BAD_ARG;
+  PrefillArgs a = {};
+  a.q = (const __half*)q; a.T_total = T_total; a.gate = gate; a.ldg = ldg; a.gate_elem = 1; a.maps = 1;
+  a.page_table = page_table; a.q_start = q_start; a.q_len = q_len; a.ctx_len = ctx_len; a.sinks = sinks;
+  a.out = (__nv_bfloat16*)out; a.status = status; a.max_pages = max_pages; a.Hq = H; a.Hkv = H;
+  a.base = base; a.k_boxes = kn / 64; a.v_col = v_col; a.r_col = r_col;
+  CUtensorMap tw, tr;
+  int rc = make_tmap_2d(&tw, ws, 2, (uint64_t)ws_rows, (uint64_t)ldw, (uint64_t)ldw * 2, KB, 64, true);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tr, cache, 2, (uint64_t)n_pages * 16, (uint64_t)ks, (uint64_t)ks * 2, 16, 64, true);
+  if (rc) return rc;
+  switch ((kn + rr) * 1000 + dv) {
+    case 128064: return run_prefill<128, 64, true>(tw, tw, tr, a, n_seqs, max_q, st);
+    case 128128: return run_prefill<128, 128, true>(tw, tw, tr, a, n_seqs, max_q, st);
+    case 192064: return run_prefill<192, 64, true>(tw, tw, tr, a, n_seqs, max_q, st);
+    case 192128: return run_prefill<192, 128, true>(tw, tw, tr, a, n_seqs, max_q, st);
+    case 256064: return run_prefill<256, 64, true>(tw, tw, tr, a, n_seqs, max_q, st);
+    case 256128: return run_prefill<256, 128, true>(tw, tw, tr, a, n_seqs, max_q, st);
   }
   return B200_ERR_BAD_ARG;
 }

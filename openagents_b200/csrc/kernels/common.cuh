@@ -109,6 +109,8 @@ __device__ __forceinline__ float gelu_tanh(float x) {
   return 0.5f * x * (1.f + tanhf(u));
 }
 
+__device__ __forceinline__ float gelu_erf(float x) { return 0.5f * x * (1.f + erff(x * 0.7071067811865476f)); }
+
 // Byte slot of element i (0..7) inside each group of eight quantized activations.  The order is
 // chosen so that `v & 0x0F0F0F0F` / `(v >> 4) & 0x0F0F0F0F` of a repacked 4-bit weight word line up
 // with two consecutive activation words for dp4a.

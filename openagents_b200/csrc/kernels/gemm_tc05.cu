@@ -52,8 +52,11 @@ int make_tmap_2d(CUtensorMap* map, const void* base, int elem_bytes, uint64_t ro
 
 // ACT_SWIGLU_PAIR: B rows are interleaved (gate_0, up_0, gate_1, ...); the epilogue writes
 // silu(gate) * up as bf16, N / 2 values per row of out_bf16 (row stride ldc), nothing else.
-// ACT_RELU2: the square of relu.
-enum { ACT_NONE = 0, ACT_GELU = 1, ACT_SWIGLU_PAIR = 2, ACT_RELU2 = 3 };
+// ACT_RELU2: the square of relu.  ACT_GELU: the tanh form; ACT_GELU_ERF: the exact one.
+enum { ACT_NONE = 0, ACT_GELU = 1, ACT_SWIGLU_PAIR = 2, ACT_RELU2 = 3, ACT_GELU_ERF = 4 };
+__device__ __forceinline__ float activate(int act, float x) {
+  return act == ACT_GELU ? gelu_tanh(x) : act == ACT_GELU_ERF ? gelu_erf(x) : act == ACT_RELU2 ? (x > 0.f ? x * x : 0.f) : x;
+}
 
 struct GemmEpi {
   float* out_f32;            // either or both outputs
@@ -64,6 +67,13 @@ struct GemmEpi {
   int ldc;
   int act;
   int accumulate;            // out_f32 += value
+  float alpha;               // multiplies the product, ahead of everything else
+  int half_out;              // out_bf16 is stored as fp16 instead
+  const float* gate;         // [M][ldg] or null: the result is multiplied by sigmoid(gate[m][n]) (n: output column)
+  int ldg;
+  // Per-head products: head z multiplies columns [z * head_k, +K) of A with rows [z * head_n, +head_n) of B into output columns
+  // [z * head_ldc, +head_n).  0 heads: one product.
+  int heads, head_k, head_n, head_ldc;
   // Split-K (small M): each split adds its partial product into out_f32 with a vector `red`, so
   // out_f32 must already hold the residual (or zeros); bias comes from split 0 only.
   int splitk_red;
@@ -130,7 +140,7 @@ __device__ __forceinline__ void epilogue_chunk_red(const GemmEpi& e, float* stag
       const int row = (lane >> 3) + 4 * i, m = m_warp0 + row;
       if (m >= M) break;
       float4 o = *(const float4*)(stage + row * 32 + ((c4 ^ (row & 7)) << 2));
-      o.x += b.x; o.y += b.y; o.z += b.z; o.w += b.w;
+      o.x = fmaf(o.x, e.alpha, b.x); o.y = fmaf(o.y, e.alpha, b.y); o.z = fmaf(o.z, e.alpha, b.z); o.w = fmaf(o.w, e.alpha, b.w);
       if (!sym) {
         asm volatile("red.relaxed.gpu.global.add.v4.f32 [%0], {%1,%2,%3,%4};" ::"l"(e.out_f32 + (size_t)m * e.ldc + n),
                      "f"(o.x), "f"(o.y), "f"(o.z), "f"(o.w) : "memory");
@@ -185,6 +195,11 @@ __device__ __forceinline__ void epilogue_chunk_combine(const GemmEpi& e, float* 
   __syncwarp();
 }
 
+__device__ __forceinline__ void put16(const GemmEpi& e, size_t at, float x) {
+  if (e.half_out) ((__half*)e.out_bf16)[at] = __float2half(x);
+  else e.out_bf16[at] = __float2bfloat16(x);
+}
+
 // Transposed epilogue: this thread holds, for output column `n` (a weight row), the values of the 32
 // output rows t0..t0+31 (tokens).  Consecutive lanes hold consecutive columns, so each of the 32
 // stores of a warp covers 128 contiguous bytes.
@@ -198,7 +213,7 @@ __device__ __forceinline__ void epilogue_col(const GemmEpi& e, int n, int t0, in
   for (int j = 0; j < 32; j++) {
     const int t = t0 + j;
     if (t >= n_rows) continue;
-    float x = __uint_as_float(r[j]) + b;
+    float x = fmaf(__uint_as_float(r[j]), e.alpha, b);
     if (sym) {
       const int owner = e.sym_mode != SYM_ALLREDUCE ? t / e.rows_per_rank : 0;
       const int lrow = rs_row(e, t);
@@ -212,12 +227,12 @@ __device__ __forceinline__ void epilogue_col(const GemmEpi& e, int n, int t0, in
       asm volatile("red.relaxed.gpu.global.add.f32 [%0], %1;" ::"l"(e.out_f32 + idx), "f"(x) : "memory");
       continue;
     }
-    if (e.act == ACT_GELU) x = gelu_tanh(x);
-    else if (e.act == ACT_RELU2) x = x > 0.f ? x * x : 0.f;
+    x = activate(e.act, x);
+    if (e.gate) x *= 1.f / (1.f + __expf(-e.gate[(size_t)t * e.ldg + n]));
     if (e.resid_f32) x += e.resid_f32[idx];
     if (e.resid_bf16) x += __bfloat162float(e.resid_bf16[idx]);
     if (e.out_f32) e.out_f32[idx] = e.accumulate ? e.out_f32[idx] + x : x;
-    if (e.out_bf16) e.out_bf16[idx] = __float2bfloat16(x);
+    if (e.out_bf16) put16(e, idx, x);
   }
 }
 
@@ -231,7 +246,7 @@ __device__ __forceinline__ void epilogue_row(const GemmEpi& e, int m, int n0, in
   const size_t base = (size_t)m * e.ldc + n0;
   float v[32];
 #pragma unroll
-  for (int j = 0; j < 32; j++) v[j] = __uint_as_float(r[j]);
+  for (int j = 0; j < 32; j++) v[j] = __uint_as_float(r[j]) * e.alpha;
   const bool full = n0 + 32 <= N;
   if (e.splitk_red && e.sym_mode == SYM_NONE) {
     const bool add_bias = e.bias && first_split;
@@ -287,9 +302,20 @@ __device__ __forceinline__ void epilogue_row(const GemmEpi& e, int m, int n0, in
     if (e.act == ACT_GELU) {
 #pragma unroll
       for (int j = 0; j < 32; j++) v[j] = gelu_tanh(v[j]);
+    } else if (e.act == ACT_GELU_ERF) {
+#pragma unroll
+      for (int j = 0; j < 32; j++) v[j] = gelu_erf(v[j]);
     } else if (e.act == ACT_RELU2) {
 #pragma unroll
       for (int j = 0; j < 32; j++) v[j] = v[j] > 0.f ? v[j] * v[j] : 0.f;
+    }
+    if (e.gate) {
+#pragma unroll
+      for (int j = 0; j < 32; j += 4) {
+        const float4 g = *(const float4*)(e.gate + (size_t)m * e.ldg + n0 + j);
+        v[j] *= 1.f / (1.f + __expf(-g.x)); v[j + 1] *= 1.f / (1.f + __expf(-g.y));
+        v[j + 2] *= 1.f / (1.f + __expf(-g.z)); v[j + 3] *= 1.f / (1.f + __expf(-g.w));
+      }
     }
     if (e.resid_f32) {
 #pragma unroll
@@ -328,7 +354,14 @@ __device__ __forceinline__ void epilogue_row(const GemmEpi& e, int m, int n0, in
         uint4 o;
         __nv_bfloat162* p = (__nv_bfloat162*)&o;
 #pragma unroll
-        for (int q = 0; q < 4; q++) p[q] = __floats2bfloat162_rn(v[j + 2 * q], v[j + 2 * q + 1]);
+        for (int q = 0; q < 4; q++) {
+          if (e.half_out) {
+            const __half2 h2 = __floats2half2_rn(v[j + 2 * q], v[j + 2 * q + 1]);
+            p[q] = *(const __nv_bfloat162*)&h2;
+          } else {
+            p[q] = __floats2bfloat162_rn(v[j + 2 * q], v[j + 2 * q + 1]);
+          }
+        }
         *(uint4*)(e.out_bf16 + base + j) = o;
       }
     }
@@ -338,12 +371,12 @@ __device__ __forceinline__ void epilogue_row(const GemmEpi& e, int m, int n0, in
       if (n0 + j >= N) continue;
       float x = v[j];
       if (e.bias) x += e.bias[n0 + j];
-      if (e.act == ACT_GELU) x = gelu_tanh(x);
-      else if (e.act == ACT_RELU2) x = x > 0.f ? x * x : 0.f;
+      x = activate(e.act, x);
+      if (e.gate) x *= 1.f / (1.f + __expf(-e.gate[(size_t)m * e.ldg + n0 + j]));
       if (e.resid_f32) x += e.resid_f32[base + j];
       if (e.resid_bf16) x += __bfloat162float(e.resid_bf16[base + j]);
       if (e.out_f32) e.out_f32[base + j] = e.accumulate ? e.out_f32[base + j] + x : x;
-      if (e.out_bf16) e.out_bf16[base + j] = __float2bfloat16(x);
+      if (e.out_bf16) put16(e, base + j, x);
     }
   }
 }
@@ -388,7 +421,8 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int KB = (K + BKS - 1) / BKS;               // K in stage units
   int tiles_m = (M + BM - 1) / BM;
-  const int tiles_n = (N + BN - 1) / BN;
+  const int tiles_head = epi.heads ? (epi.head_n + BN - 1) / BN : 0;      // column tiles of one head
+  const int tiles_n = epi.heads ? epi.heads * tiles_head : (N + BN - 1) / BN;
   int n_tiles = tiles_m * tiles_n * splits;   // work items: (output tile, K split), split fastest
   const int kps = (KB + splits - 1) / splits;
   // fused all-gather: start the walk over m tiles at this rank's own rows
@@ -448,6 +482,7 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
         // read from HBM once and stay in L2, instead of every expert's rows being re-read for each column tile.
         const int m0 = epi.group_rows ? live_m[tile / tiles_n] : ((tile % tiles_m + m_rot) % tiles_m) * BM;
         const int n0 = epi.group_rows ? (tile % tiles_n) * BN : (tile / tiles_m) * BN;
+        const int z = epi.heads ? tile / tiles_m / tiles_head : 0, a_col = z * epi.head_k;
         if (epi.ag_rows_per_rank) {       // rows of this tile come from their owners' all-gather pushes
           const int o0 = m0 / epi.ag_rows_per_rank, o1 = min(m0 + BM - 1, M - 1) / epi.ag_rows_per_rank;
           for (int o = o0; o <= o1 && ok; o++) {
@@ -461,7 +496,7 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
           if (!ok) break;
           asm volatile("fence.proxy.async.global;" ::: "memory");   // peers' stores -> this CTA's TMA reads
         }
-        int b_row = n0;
+        int b_row = epi.heads ? z * epi.head_n + (tile / tiles_m % tiles_head) * BN : n0;
         if (epi.group_rows) b_row += (m0 / epi.group_rows) * epi.group_n;
         const int kb0 = sp * kps, kb1 = min(KB, kb0 + kps);
         for (int kb = kb0; kb < kb1; kb++, it++) {
@@ -479,7 +514,7 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
           } else {
 #pragma unroll
             for (int u = 0; u < KSUB; u++) {      // a block past the end of K is filled with zeros by the TMA unit
-              tma_load_2d(smem_u32(sA + s * A_BYTES + u * A_SUB), &tmA, smem_u32(full + s), kb * BKS + u * BK, m0);
+              tma_load_2d(smem_u32(sA + s * A_BYTES + u * A_SUB), &tmA, smem_u32(full + s), a_col + kb * BKS + u * BK, m0);
               tma_load_2d(smem_u32(sB + s * B_BYTES + u * B_SUB), &tmB, smem_u32(full + s), kb * BKS + u * BK, b_row);
             }
           }
@@ -535,7 +570,10 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
     for (int item = blockIdx.x; item < n_tiles; item += gridDim.x) {
       const int tile = item / splits, sp = item - tile * splits;
       const int m0 = epi.group_rows ? live_m[tile / tiles_n] : ((tile % tiles_m + m_rot) % tiles_m) * BM;
-      const int n0 = epi.group_rows ? (tile % tiles_n) * BN : (tile / tiles_m) * BN;
+      const int z = epi.heads ? tile / tiles_m / tiles_head : 0;
+      const int n0 = epi.heads ? z * epi.head_ldc + (tile / tiles_m % tiles_head) * BN
+                               : epi.group_rows ? (tile % tiles_n) * BN : (tile / tiles_m) * BN;
+      const int n_end = epi.heads ? z * epi.head_ldc + epi.head_n : N;     // columns below this index are written
       int live_end = M;                       // rows below this index are written
       if (epi.group_rows) {
         const int g = m0 / epi.group_rows;
@@ -560,16 +598,16 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
 #pragma unroll
         for (int j = 0; j < BN / 32; j++) {
           const int n = n0 + j * 32 + lane;
-          stage[j * 32 + lane] = n < N ? epi.bias[n] : 0.f;
+          stage[j * 32 + lane] = n < n_end ? epi.bias[n] : 0.f;
         }
         __syncwarp();
       }
       auto process = [&](int c, const uint32_t (&r)[32]) {
-        if (n0 + c * 32 >= N) return;
+        if (n0 + c * 32 >= n_end) return;
         if (epi.moe_mode == 2) epilogue_chunk_combine(epi, stage, m0 + q * 32, live_end, n0 + c * 32, N, r);
         else if (epi.moe_mode == 1 || epi.act == ACT_SWIGLU_PAIR) { if (m < live_end) epilogue_row_swiglu(epi, m, n0 + c * 32, r); }
         else if (red_path) epilogue_chunk_red(epi, stage, m0 + q * 32, n0 + c * 32, live_end, N, r, sp == 0);
-        else epilogue_row(epi, m, n0 + c * 32, live_end, N, r, sp == 0, stage_bias ? stage + c * 32 : nullptr);
+        else epilogue_row(epi, m, n0 + c * 32, live_end, n_end, r, sp == 0, stage_bias ? stage + c * 32 : nullptr);
       };
       // two register buffers: the tensor-memory load of the next 32 columns is in flight while this chunk is finished
       const uint32_t t_addr = tmem_base + ((uint32_t)(q * 32) << 16) + acc * BN;
@@ -631,7 +669,8 @@ static int launch_gemm(const CUtensorMap& ta, const CUtensorMap& tb, const GemmE
     if (err != cudaSuccess) return (int)err;
     configured = true;
   }
-  const int n_tiles = ((N + BN - 1) / BN) * ((M + BM - 1) / BM) * splits;
+  const int tiles_n = e.heads ? e.heads * ((e.head_n + BN - 1) / BN) : (N + BN - 1) / BN;
+  const int n_tiles = tiles_n * ((M + BM - 1) / BM) * splits;
   const int grid = n_tiles < sm_count() ? n_tiles : sm_count();
   return launch_pdl(kern, dim3(grid), dim3(192), smem, st, ta, tb, e, M, N, K, splits, status);
 }
@@ -643,13 +682,14 @@ B200_API int b200_gemm_bf16(const void* A, const void* B, int M, int N, int K, i
                             void* out_bf16, int ldc, const float* bias, const float* resid_f32,
                             const void* resid_bf16, int act, int accumulate, int tile_n, int split_k, int* status,
                             int sym_mode, const SymTable* sym, size_t sym_off, int rows_per_rank, int wait_ready,
-                            int ag_rows_per_rank, int ag_epoch, int mn_major, cudaStream_t st) {
+                            int ag_rows_per_rank, int ag_epoch, int mn_major, float alpha, int half_out, cudaStream_t st) {
   if (M <= 0 || N <= 0 || K <= 0 || (lda % 8) || (ldb % 8) || (!mn_major && (K % 8))) return B200_ERR_BAD_ARG;
   if (mn_major) {
     // D[M][N] = sum_k A[k][m] * B[k][n]: A is [K][M] (row stride lda), B is [K][N] (row stride ldb).  Plain epilogues only.
     if (sym_mode != SYM_NONE || ag_rows_per_rank || tile_n < 0 || split_k > 1 || act == ACT_SWIGLU_PAIR || (M % 8) || (N % 8))
       return B200_ERR_BAD_ARG;
     if ((out_bf16 && (ldc % 8)) || (out_f32 && (ldc % 4)) || (N % 4)) return B200_ERR_BAD_ARG;
+    if (alpha != 1.f || half_out) return B200_ERR_BAD_ARG;
     CUtensorMap ta, tb;
     int rc = make_tmap_2d(&ta, A, 2, (uint64_t)K, (uint64_t)M, (uint64_t)lda * 2, BK, 64, true);
     if (rc) return rc;
@@ -658,6 +698,7 @@ B200_API int b200_gemm_bf16(const void* A, const void* B, int M, int N, int K, i
     GemmEpi e = {};
     e.out_f32 = out_f32; e.out_bf16 = (__nv_bfloat16*)out_bf16; e.bias = bias; e.resid_f32 = resid_f32;
     e.resid_bf16 = (const __nv_bfloat16*)resid_bf16; e.ldc = ldc; e.act = act; e.accumulate = accumulate; e.rows_per_rank = 1;
+    e.alpha = 1.f;
     const long t256 = (long)((N + 255) / 256) * ((M + 127) / 128);
     if ((tile_n == 256 || (tile_n == 0 && N >= 256 && t256 >= 148)))
       return launch_gemm<256, 4, 128, 1, true>(ta, tb, e, M, N, K, 1, status, st);
@@ -708,7 +749,8 @@ B200_API int b200_gemm_bf16(const void* A, const void* B, int M, int N, int K, i
   if (rc) return rc;
   rc = make_tmap_2d(&tb, B, 2, (uint64_t)N, (uint64_t)K, (uint64_t)ldb * 2, (uint32_t)tile_n, BK, true);
   if (rc) return rc;
-  GemmEpi e;
+  GemmEpi e = {};
+  e.alpha = alpha; e.half_out = half_out;
   e.out_f32 = out_f32; e.out_bf16 = (__nv_bfloat16*)out_bf16; e.bias = bias; e.resid_f32 = resid_f32;
   e.resid_bf16 = (const __nv_bfloat16*)resid_bf16; e.ldc = ldc; e.act = act; e.accumulate = accumulate;
   e.sym_mode = sym_mode; e.rows_per_rank = rows_per_rank > 0 ? rows_per_rank : 1; e.sym_off = sym_off;
@@ -748,6 +790,36 @@ B200_API int b200_gemm_bf16(const void* A, const void* B, int M, int N, int K, i
   return B200_ERR_BAD_ARG;
 }
 
+// One small product per head (see GemmEpi): out[m][z * head_ldc + n] = alpha * sum_k A[m][z * head_k + k] * B[z * N + n][k], times
+// sigmoid(gate[m][z * head_ldc + n]) where a gate is given.  A [M][>= (heads - 1) * head_k + K], B [heads * N][K] with row stride
+// ldb; head_k, head_ldc, ldb multiples of 8.  Columns of A past a head's K meet zeros (the tensor map of B ends at K).
+B200_API int b200_gemm_heads(const void* A, const void* B, int M, int heads, int N, int K, int lda, int head_k, int ldb,
+                             float* out_f32, void* out_bf16, int ldc, int head_ldc, float alpha, const float* gate, int ldg,
+                             int half_out, int* status, cudaStream_t st) {
+  if (M <= 0 || heads <= 0 || N <= 0 || K <= 0 || (lda % 8) || (ldb % 8) || (head_k % 8) || (head_ldc % 8) || (K % 8) || (N % 8) || K > head_k)
+    return B200_ERR_BAD_ARG;
+  if ((!out_f32 && !out_bf16) || (out_bf16 && (ldc % 8)) || (out_f32 && (ldc % 4)) || N > head_ldc || ldc < heads * head_ldc ||
+      lda < heads * head_k || (gate && ((ldg % 4) || ldg < heads * head_ldc || ((uintptr_t)gate & 15))))
+    return B200_ERR_BAD_ARG;
+  const long tiles_m = (M + 127) / 128;
+  const int tile_n = N > 128 && (long)heads * ((N + 255) / 256) * tiles_m >= 148 ? 256
+                     : N > 64 && (long)heads * ((N + 127) / 128) * tiles_m >= 100 ? 128 : 64;
+  const bool few_rows = M <= 64;
+  CUtensorMap ta, tb;
+  int rc = make_tmap_2d(&ta, A, 2, (uint64_t)M, (uint64_t)(heads * head_k), (uint64_t)lda * 2, few_rows ? 64 : BM, BK, true);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tb, B, 2, (uint64_t)heads * N, (uint64_t)K, (uint64_t)ldb * 2, (uint32_t)tile_n, BK, true);
+  if (rc) return rc;
+  GemmEpi e = {};
+  e.out_f32 = out_f32; e.out_bf16 = (__nv_bfloat16*)out_bf16; e.ldc = ldc; e.alpha = alpha; e.gate = gate; e.ldg = ldg;
+  e.half_out = half_out; e.heads = heads; e.head_k = head_k; e.head_n = N; e.head_ldc = head_ldc; e.rows_per_rank = 1;
+  switch (tile_n) {
+    case 256: return few_rows ? launch_gemm<256, 5, 64>(ta, tb, e, M, N, K, 1, status, st) : launch_gemm<256, 4>(ta, tb, e, M, N, K, 1, status, st);
+    case 128: return few_rows ? launch_gemm<128, 4, 64, 2>(ta, tb, e, M, N, K, 1, status, st) : launch_gemm<128, 6>(ta, tb, e, M, N, K, 1, status, st);
+  }
+  return few_rows ? launch_gemm<64, 6, 64, 2>(ta, tb, e, M, N, K, 1, status, st) : launch_gemm<64, 8>(ta, tb, e, M, N, K, 1, status, st);
+}
+
 // Grouped GEMM of a mixture-of-experts layer (see GemmEpi).  A [groups * group_rows][K] bf16 (row
 // stride lda) holds each expert's gathered tokens, B [groups * N][K] bf16 its weights, counts[g] the
 // live rows of group g (device memory, final before this kernel starts).
@@ -774,6 +846,7 @@ B200_API int b200_moe_gemm(const void* A, const void* B, int groups, int group_r
   e.out_bf16 = (__nv_bfloat16*)out_bf16; e.ldc = ldc;
   e.group_rows = group_rows; e.group_n = N; e.group_counts = counts; e.moe_mode = mode; e.meta = meta; e.gate_w = gate_w;
   e.rows_per_rank = 1;
+  e.alpha = 1.f;
   if (mode == 2) {
     e.sym_mode = SYM_ALLREDUCE;   // only so that the kernel ends with the cross-rank barrier
     e.sym = *sym;

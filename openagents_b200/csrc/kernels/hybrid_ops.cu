@@ -1,5 +1,6 @@
 // Operators of hybrid decoders (attention and recurrent layers in one stack, norms around both ends of a sublayer): the
-// residual step, the projection finish of an attention layer, attention in exact 32-bit arithmetic for any head size, the
+// residual step, Dynamic Tanh, the projection finish of an attention layer, attention in exact 32-bit arithmetic for any head size, the
+// difference of two attention maps, the
 // 32-bit matrix product, and the last step of the logits.
 //
 // This file is compiled without fast math: divisions, square roots, exponentials and hyperbolic tangents are the IEEE-accurate
@@ -161,12 +162,108 @@ B200_API int b200_norm_residual(float* y, int ldy, const float* gy, float* x, in
                     y_clear, (float4*)zero_a, zero_a ? (int)(zero_a_n / 4) : 0, (float4*)zero_b, zero_b ? (int)(zero_b_n / 4) : 0);
 }
 
+// ------------------------------------------------------------------ Dynamic Tanh
+
+// Per row:  x += emb[ids[t]]             (when emb is given: a looped stack's next pass takes the embedding in again)
+//           h  = tanh(alpha x) * w + b   -> bf16 and/or fp32, columns D..ldh written as zeros
+// No statistics, so rows are only a shape.  zero: a buffer cleared on the side for a K-split projection that adds into it.
+struct DytArgs {
+  float* x;                  // [T][D]
+  int D, ldh;
+  const int* ids;
+  const __nv_bfloat16* emb;  // [vocab][D] or null
+  int vocab;
+  const float* alpha;        // one number
+  const float* w;
+  const float* b;
+  __nv_bfloat16* hb;
+  float* hf;
+  float4* zero;
+  int nz4;
+};
+__device__ __forceinline__ float dyt_one(float x, float alpha, float w, float b) { return fmaf(tanhf(alpha * x), w, b); }
+
+__global__ void __launch_bounds__(256) norm_dyt_kernel(const DytArgs a) {
+  const int t = blockIdx.x, nt = blockDim.x * gridDim.y, i0 = blockIdx.y * blockDim.x + threadIdx.x;
+  const float alpha = *a.alpha;
+  pdl_trigger();
+  pdl_wait();
+  for (int i = (blockIdx.x * gridDim.y + blockIdx.y) * blockDim.x + threadIdx.x; i < a.nz4; i += gridDim.x * nt)
+    a.zero[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+  float* xr = a.x + (size_t)t * a.D;
+  const int id = a.emb ? a.ids[t] : 0;
+  const bool add = a.emb && id >= 0 && id < a.vocab;
+  for (int i = i0; i < a.ldh; i += nt) {
+    float o = 0.f;
+    if (i < a.D) {
+      float v = xr[i];
+      if (add) {
+        v += __bfloat162float(a.emb[(size_t)id * a.D + i]);
+        xr[i] = v;
+      }
+      o = dyt_one(v, alpha, a.w[i], a.b[i]);
+    }
+    if (a.hb) a.hb[(size_t)t * a.ldh + i] = __float2bfloat16(o);
+    if (a.hf) a.hf[(size_t)t * a.ldh + i] = o;
+  }
+}
+// The same on 16-byte accesses (widths that are multiples of 4).
+__global__ void __launch_bounds__(256) norm_dyt_vec_kernel(const DytArgs a) {
+  const int t = blockIdx.x, nt = blockDim.x * gridDim.y, i0 = blockIdx.y * blockDim.x + threadIdx.x;
+  const int D4 = a.D >> 2, l4 = a.ldh >> 2;
+  const float alpha = *a.alpha;
+  pdl_trigger();
+  pdl_wait();
+  for (int i = (blockIdx.x * gridDim.y + blockIdx.y) * blockDim.x + threadIdx.x; i < a.nz4; i += gridDim.x * nt)
+    a.zero[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4* xr = (float4*)(a.x + (size_t)t * a.D);
+  const int id = a.emb ? a.ids[t] : 0;
+  const bool add = a.emb && id >= 0 && id < a.vocab;
+  for (int i = i0; i < l4; i += nt) {
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < D4) {
+      float4 v = xr[i];
+      const float4 w = ((const float4*)a.w)[i], b = ((const float4*)a.b)[i];
+      if (add) {
+        const uint2 e = ((const uint2*)(a.emb + (size_t)id * a.D))[i];
+        const float2 e0 = __bfloat1622float2(*(const __nv_bfloat162*)&e.x), e1 = __bfloat1622float2(*(const __nv_bfloat162*)&e.y);
+        v.x += e0.x; v.y += e0.y; v.z += e1.x; v.w += e1.y;
+        xr[i] = v;
+      }
+      o = make_float4(dyt_one(v.x, alpha, w.x, b.x), dyt_one(v.y, alpha, w.y, b.y), dyt_one(v.z, alpha, w.z, b.z), dyt_one(v.w, alpha, w.w, b.w));
+    }
+    if (a.hb) {
+      const __nv_bfloat162 p0 = __floats2bfloat162_rn(o.x, o.y), p1 = __floats2bfloat162_rn(o.z, o.w);
+      *(uint2*)(a.hb + ((size_t)t * l4 + i) * 4) = make_uint2(*(const uint32_t*)&p0, *(const uint32_t*)&p1);
+    }
+    if (a.hf) ((float4*)a.hf)[(size_t)t * l4 + i] = o;
+  }
+}
+B200_API int b200_norm_dyt(float* x, int T, int D, const int* ids, const void* emb, int vocab, const float* alpha, const float* w,
+                           const float* b, void* hb, float* hf, int ldh, float* zero, long zero_n, cudaStream_t st) {
+  if (T < 1 || D < 1 || ldh < D || !x || !alpha || !w || !b || (!hb && !hf) || (emb && !ids)) return B200_ERR_BAD_ARG;
+  if (zero && (zero_n % 4 || (uintptr_t)zero % 16)) return B200_ERR_BAD_ARG;
+  DytArgs a;
+  a.x = x; a.D = D; a.ldh = ldh; a.ids = ids; a.emb = (const __nv_bfloat16*)emb; a.vocab = vocab; a.alpha = alpha; a.w = w; a.b = b;
+  a.hb = (__nv_bfloat16*)hb; a.hf = hf; a.zero = (float4*)zero; a.nz4 = zero ? (int)(zero_n / 4) : 0;
+  const uintptr_t align = (uintptr_t)x | (uintptr_t)w | (uintptr_t)b | (uintptr_t)hb | (uintptr_t)hf | (uintptr_t)emb;
+  const bool vec = align % 16 == 0 && D % 4 == 0 && ldh % 4 == 0;
+  const int per = vec ? ldh / 4 : ldh, threads = per > 128 ? 256 : 128;
+  // a row has no reduction, so few rows are spread over several blocks each
+  int gy = 1;
+  while (gy * threads < per && (long)T * gy < 2 * 148) gy++;
+  return launch_pdl(vec ? norm_dyt_vec_kernel : norm_dyt_kernel, dim3(T, gy), dim3(threads), 0, st, a);
+}
+
 // ------------------------------------------------------------------ attention: finish of the projections
 
 // One warp per (token, head) of a fused projection row: queries and keys are rotated on their first `rot` dimensions, then
 // (qk_norm) divided by their root mean square over the head; queries are scaled, keys and values go to the paged cache.
 //   style 0: dimension 2i turns with 2i + 1; style 1: i with i + rot / 2.
 // Cache and query rows are padded to DK / DV columns; the padding is written as zeros.
+// maps = 2 (differential attention): a key/value head has two key rows side by side ([map 1, map 2], DK columns each) and H counts
+// the query rows of both maps, in the order (key/value head, map, query head of the group).  q_wide: a query row is as wide as
+// both key rows and zero on the other map's half, so that one product with them gives its own map's scores.
 struct QkvArgs {
   const float* in;         // [T][ld]
   int ld, q_off, k_off, v_off;     // k_off < 0: the layer has no keys and values of its own
@@ -177,8 +274,10 @@ struct QkvArgs {
   double base;
   int H, G, dim, vdim, DK, DV, rot, style, qk_norm, page_size;
   float eps, q_scale;
-  float* q32;              // [T][H][DK] or null
+  float* q32;              // [T][H][DK or maps * DK] or null
   __half* q16;             // [T][H][DK] or null
+  int maps, q_wide;
+  const float* bias;       // added to the row's columns, or null
 };
 constexpr int kQkvPairs = 8;      // pairs per lane: head sizes up to 512
 
@@ -190,21 +289,27 @@ __global__ void __launch_bounds__(128) qkv_finish_kernel(const QkvArgs a, CT* __
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x, lane = threadIdx.x & 31;
-  const int n_heads = a.H + (a.k_off >= 0 ? 2 * a.G : 0);
+  const int KR = a.G * a.maps;                            // key rows
+  const int n_heads = a.H + (a.k_off >= 0 ? KR + a.G : 0);
   const int hh = blockIdx.y * 4 + (threadIdx.x >> 5);
   if (hh >= n_heads) return;
   const int s = a.slot[t];
   const int page = s >= 0 ? s / a.page_size : 0, off = s >= 0 ? s % a.page_size : 0;
   const float* row = a.in + (size_t)t * a.ld;
-  if (hh >= a.H + a.G) {                                  // a value head
+  if (hh >= a.H + KR) {                                   // a value head
     if (s < 0) return;
-    const int g = hh - a.H - a.G;
+    const int g = hh - a.H - KR;
     CT* dst = vc + (((size_t)page * a.G + g) * a.page_size + off) * a.DV;
-    for (int e = lane; e < a.DV; e += 32) put(dst + e, e < a.vdim ? row[a.v_off + g * a.vdim + e] : 0.f);
+    for (int e = lane; e < a.DV; e += 32) {
+      const int c = a.v_off + g * a.vdim + e;
+      put(dst + e, e < a.vdim ? row[c] + (a.bias ? a.bias[c] : 0.f) : 0.f);
+    }
     return;
   }
   const bool is_q = hh < a.H;
-  const float* in = row + (is_q ? a.q_off + hh * a.dim : a.k_off + (hh - a.H) * a.dim);
+  const int col = is_q ? a.q_off + hh * a.dim : a.k_off + (hh - a.H) * a.dim;
+  const float* in = row + col;
+  const float* bs = a.bias ? a.bias + col : nullptr;
   const int half = a.rot >> 1, n_pairs = (a.DK + 1) >> 1;
   const int p = a.pos[t];
   float u[kQkvPairs], w[kQkvPairs];
@@ -217,6 +322,10 @@ __global__ void __launch_bounds__(128) qkv_finish_kernel(const QkvArgs a, CT* __
       const int i0 = (j < half && a.style == 1) ? j : 2 * j;
       const int i1 = (j < half && a.style == 1) ? j + half : 2 * j + 1;
       float x0 = i0 < a.dim ? in[i0] : 0.f, x1 = i1 < a.dim ? in[i1] : 0.f;
+      if (bs) {
+        if (i0 < a.dim) x0 += bs[i0];
+        if (i1 < a.dim) x1 += bs[i1];
+      }
       if (j < half) {
         float cs, sn;
         if (a.tab && p >= 0 && p < a.tab_len) {
@@ -240,8 +349,14 @@ __global__ void __launch_bounds__(128) qkv_finish_kernel(const QkvArgs a, CT* __
   }
   float m = is_q ? a.q_scale : 1.f;
   if (a.qk_norm) m *= 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
-  const size_t q_at = ((size_t)t * a.H + hh) * a.DK;
-  CT* kd = is_q ? nullptr : kc + (((size_t)page * a.G + (hh - a.H)) * a.page_size + off) * a.DK;
+  const int kr = hh - a.H, map = is_q ? hh / (a.H / KR) % a.maps : kr % a.maps;
+  const int qw = a.q_wide ? a.maps * a.DK : a.DK;
+  size_t q_at = ((size_t)t * a.H + hh) * qw;
+  if (is_q && a.q_wide && a.q32)                          // the halves of the other maps
+    for (int e = lane; e < qw; e += 32)
+      if (e / a.DK != map) a.q32[q_at + e] = 0.f;
+  if (a.q_wide) q_at += map * a.DK;
+  CT* kd = is_q ? nullptr : kc + ((((size_t)page * a.G + kr / a.maps) * a.page_size + off) * a.maps + map) * a.DK;
   if (!is_q && s < 0) return;
 #pragma unroll
   for (int k = 0; k < kQkvPairs; k++) {
@@ -265,19 +380,21 @@ __global__ void __launch_bounds__(128) qkv_finish_kernel(const QkvArgs a, CT* __
     }
   }
 }
-// cache_f32: kc / vc hold fp32 instead of fp16; layout [page][G][page_size][DK or DV].
+// cache_f32: kc / vc hold fp32 instead of fp16; layout [page][G][page_size][maps * DK or DV].
 B200_API int b200_qkv_finish(const float* in, int ld, int T, int q_off, int k_off, int v_off, const int* pos, const int* slot,
                              const void* tab, int tab_len, double base, int H, int G, int dim, int vdim, int DK, int DV, int rot,
                              int style, int qk_norm, float eps, float q_scale, int page_size, float* q32, void* q16, void* kc,
-                             void* vc, int cache_f32, cudaStream_t st) {
+                             void* vc, int cache_f32, int maps, int q_wide, const float* bias, cudaStream_t st) {
   if (T < 1 || H < 1 || G < 1 || dim < 1 || vdim < 1 || dim > DK || vdim > DV || DK > 64 * kQkvPairs || (rot & 1) || rot > dim || rot < 0)
     return B200_ERR_BAD_ARG;
   if ((k_off >= 0 && (!kc || !vc)) || (!q32 && !q16) || page_size < 1) return B200_ERR_BAD_ARG;
+  if (maps < 1 || H % (G * maps) || (q_wide && q16)) return B200_ERR_BAD_ARG;
   QkvArgs a;
   a.in = in; a.ld = ld; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off; a.pos = pos; a.slot = slot; a.tab = (const float2*)tab;
   a.tab_len = tab ? tab_len : 0; a.base = base; a.H = H; a.G = G; a.dim = dim; a.vdim = vdim; a.DK = DK; a.DV = DV; a.rot = rot;
   a.style = style; a.qk_norm = qk_norm; a.page_size = page_size; a.eps = eps; a.q_scale = q_scale; a.q32 = q32; a.q16 = (__half*)q16;
-  const int n_heads = H + (k_off >= 0 ? 2 * G : 0);
+  a.maps = maps; a.q_wide = q_wide; a.bias = bias;
+  const int n_heads = H + (k_off >= 0 ? (maps + 1) * G : 0);
   const dim3 grid(T, (n_heads + 3) / 4);
   if (cache_f32) return launch_pdl(qkv_finish_kernel<float>, grid, dim3(128), 0, st, a, (float*)kc, (float*)vc);
   return launch_pdl(qkv_finish_kernel<__half>, grid, dim3(128), 0, st, a, (__half*)kc, (__half*)vc);
@@ -288,7 +405,9 @@ B200_API int b200_qkv_finish(const float* in, int ld, int T, int q_off, int k_of
 // Causal grouped-query attention over the paged cache, prompts and decoding alike: one warp per query row, eight rows per CTA
 // sharing key tiles of 32.  Lane j scores key j of a tile; the weights are then broadcast lane by lane while the lanes hold
 // the output columns.  Everything is fp32 whatever the cache holds.  gate [T][ldg] (or null): the output of head h is
-// multiplied by sigmoid(gate[t][h]).
+// multiplied by sigmoid(gate[t][h]).  chunk > 0: a query sees its own chunk of that many positions only.  sinks [H] (or null): one more
+// term of the denominator per head.  maps: see qkv_finish (query rows are DK wide).  KS: columns of a key row in the cache.  vc null: the
+// values are the first DV columns of the key row (latent attention).
 struct AttnExactArgs {
   const float* q;          // [T][H][DK], scaled
   const int* page_table;
@@ -296,29 +415,33 @@ struct AttnExactArgs {
   const int* q_len;
   const int* ctx_len;
   const float* gate;
-  int ldg, max_pages, H, G, DK, DV;
+  const float* sinks;
+  int ldg, max_pages, H, G, DK, DV, KS, maps, chunk, shared_kv;
   float* out_f32;          // [T][ldo], head h at column h * DV
   __nv_bfloat16* out_bf16;
   int ldo;
 };
-constexpr int kExactRows = 8, kExactKeys = 32, kExactCols = 16;     // columns per lane: value sizes up to 512
+constexpr int kExactRows = 8, kExactKeys = 32;
 
 __device__ __forceinline__ float get(const float* p) { return *p; }
 __device__ __forceinline__ float get(const __half* p) { return __half2float(*p); }
 
-template <typename CT>
+// kExactCols: output columns per lane (value sizes up to 32 times that)
+template <typename CT, int kExactCols>
 __global__ void __launch_bounds__(32 * kExactRows) attn_exact_kernel(const AttnExactArgs a, const CT* __restrict__ kc,
                                                                      const CT* __restrict__ vc) {
   extern __shared__ __align__(16) float sm[];
   float* sQ = sm;                                   // [rows][DK]
   float* sK = sQ + kExactRows * a.DK;               // [keys][DK + 1]
-  float* sV = sK + kExactKeys * (a.DK + 1);         // [keys][DV]
+  const int ldv = a.shared_kv ? a.DK + 1 : a.DV;
+  float* sV = a.shared_kv ? sK : sK + kExactKeys * (a.DK + 1);         // [keys][ldv]
   pdl_trigger();
   pdl_wait();
   const int seq = blockIdx.z, h = blockIdx.y, q0 = blockIdx.x * kExactRows;
   const int qlen = a.q_len[seq];
   if (q0 >= qlen) return;
-  const int ctx = a.ctx_len[seq], qs = a.q_start[seq], kh = h / (a.H / a.G);
+  const int ctx = a.ctx_len[seq], qs = a.q_start[seq], row_k = h / (a.H / (a.G * a.maps));
+  const int kh = row_k / a.maps, k_col = row_k % a.maps * a.DK;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int* pt = a.page_table + (size_t)seq * a.max_pages;
   const int rows = min(kExactRows, qlen - q0), pos0 = ctx - qlen + q0, qpos = pos0 + warp;
@@ -330,22 +453,23 @@ __global__ void __launch_bounds__(32 * kExactRows) attn_exact_kernel(const AttnE
 #pragma unroll
   for (int i = 0; i < kExactCols; i++) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
-  const int k_end = pos0 + rows;                    // keys [0, k_end) matter to some row
-  for (int k0 = 0; k0 < k_end; k0 += kExactKeys) {
+  const int k_end = pos0 + rows;                    // keys [k_begin, k_end) matter to some row
+  const int k_begin = a.chunk > 0 ? pos0 / a.chunk * a.chunk : 0, q_first = a.chunk > 0 ? qpos / a.chunk * a.chunk : 0;
+  for (int k0 = k_begin; k0 < k_end; k0 += kExactKeys) {
     __syncthreads();
     const int nk = min(kExactKeys, k_end - k0);
     for (int i = tid; i < nk * a.DK; i += blockDim.x) {
       const int r = i / a.DK, c = i % a.DK, key = k0 + r;
-      sK[r * (a.DK + 1) + c] = get(kc + (((size_t)pt[key >> 4] * a.G + kh) * 16 + (key & 15)) * a.DK + c);
+      sK[r * (a.DK + 1) + c] = get(kc + (((size_t)pt[key >> 4] * a.G + kh) * 16 + (key & 15)) * a.KS + k_col + c);
     }
-    for (int i = tid; i < nk * a.DV; i += blockDim.x) {
+    for (int i = tid; i < nk * a.DV && !a.shared_kv; i += blockDim.x) {
       const int r = i / a.DV, c = i % a.DV, key = k0 + r;
       sV[r * a.DV + c] = get(vc + (((size_t)pt[key >> 4] * a.G + kh) * 16 + (key & 15)) * a.DV + c);
     }
     __syncthreads();
     if (warp >= rows) continue;
     float s = -INFINITY;
-    if (lane < nk && k0 + lane <= qpos) {
+    if (lane < nk && k0 + lane <= qpos && k0 + lane >= q_first) {
       const float* kr = sK + lane * (a.DK + 1);
       const float* qr = sQ + warp * a.DK;
       s = 0.f;
@@ -361,7 +485,7 @@ __global__ void __launch_bounds__(32 * kExactRows) attn_exact_kernel(const AttnE
     for (int i = 0; i < kExactCols; i++) acc[i] *= corr;
     for (int j = 0; j < nk; j++) {
       const float pj = __shfl_sync(0xffffffffu, p, j);
-      const float* vr = sV + j * a.DV;
+      const float* vr = sV + j * ldv;
 #pragma unroll
       for (int i = 0; i < kExactCols; i++) {
         const int e = lane + 32 * i;
@@ -372,6 +496,10 @@ __global__ void __launch_bounds__(32 * kExactRows) attn_exact_kernel(const AttnE
   if (warp >= rows) return;
   const size_t t = (size_t)(qs + q0 + warp);
   float inv = l > 0.f ? 1.f / l : 0.f;
+  if (a.sinks) {
+    const float sk = a.sinks[h], mn = fmaxf(m, sk), c = m == -INFINITY ? 0.f : expf(m - mn);
+    inv = c / (l * c + expf(sk - mn));
+  }
   if (a.gate) inv *= 1.f / (1.f + expf(-a.gate[t * a.ldg + h]));
 #pragma unroll
   for (int i = 0; i < kExactCols; i++) {
@@ -382,36 +510,91 @@ __global__ void __launch_bounds__(32 * kExactRows) attn_exact_kernel(const AttnE
     if (a.out_bf16) a.out_bf16[at] = __float2bfloat16(acc[i] * inv);
   }
 }
-B200_API int b200_attn_exact(const float* q, const void* kc, const void* vc, int cache_f32, const int* page_table, int max_pages,
-                             const int* q_start, const int* q_len, const int* ctx_len, int n_seqs, int max_q, int H, int G, int DK,
-                             int DV, const float* gate, int ldg, float* out_f32, void* out_bf16, int ldo, cudaStream_t st) {
-  if (G < 1 || H % G || n_seqs < 1 || max_q < 1 || DK < 1 || DV < 1 || DV > 32 * kExactCols || ldo < H * DV) return B200_ERR_BAD_ARG;
-  AttnExactArgs a;
-  a.q = q; a.page_table = page_table; a.q_start = q_start; a.q_len = q_len; a.ctx_len = ctx_len; a.gate = gate; a.ldg = ldg;
-  a.max_pages = max_pages; a.H = H; a.G = G; a.DK = DK; a.DV = DV; a.out_f32 = out_f32; a.out_bf16 = (__nv_bfloat16*)out_bf16; a.ldo = ldo;
-  const size_t smem = 4 * ((size_t)kExactRows * DK + (size_t)kExactKeys * (DK + 1) + (size_t)kExactKeys * DV);
-  if (smem > 200 * 1024) return B200_ERR_BAD_ARG;
-  const dim3 grid((max_q + kExactRows - 1) / kExactRows, H, n_seqs), block(32 * kExactRows);
+template <typename CT, int NC>
+static int launch_exact_nc(dim3 grid, size_t smem, const AttnExactArgs& a, const CT* kc, const CT* vc, cudaStream_t st) {
+  auto kern = attn_exact_kernel<CT, NC>;
   static size_t configured = 48 * 1024;
   if (smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_exact_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_exact_kernel<__half>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = smem;
   }
-  if (cache_f32) return launch_pdl(attn_exact_kernel<float>, grid, block, smem, st, a, (const float*)kc, (const float*)vc);
-  return launch_pdl(attn_exact_kernel<__half>, grid, block, smem, st, a, (const __half*)kc, (const __half*)vc);
+  return launch_pdl(kern, grid, dim3(32 * kExactRows), smem, st, a, kc, vc);
+}
+template <typename CT>
+static int launch_exact(int DV, dim3 grid, size_t smem, const AttnExactArgs& a, const CT* kc, const CT* vc, cudaStream_t st) {
+  if (DV <= 128) return launch_exact_nc<CT, 4>(grid, smem, a, kc, vc, st);
+  if (DV <= 512) return launch_exact_nc<CT, 16>(grid, smem, a, kc, vc, st);
+  return launch_exact_nc<CT, 32>(grid, smem, a, kc, vc, st);
+}
+B200_API int b200_attn_exact(const float* q, const void* kc, const void* vc, int cache_f32, const int* page_table, int max_pages,
+                             const int* q_start, const int* q_len, const int* ctx_len, int n_seqs, int max_q, int H, int G, int DK,
+                             int DV, const float* gate, int ldg, float* out_f32, void* out_bf16, int ldo, int KS, int maps, int chunk,
+                             const float* sinks, cudaStream_t st) {
+  if (G < 1 || maps < 1 || H % (G * maps) || n_seqs < 1 || max_q < 1 || DK < 1 || DV < 1 || DV > 1024 || ldo < H * DV || KS < maps * DK || chunk < 0)
+    return B200_ERR_BAD_ARG;
+  if (!vc && (DV > DK || maps != 1)) return B200_ERR_BAD_ARG;
+  AttnExactArgs a;
+  a.q = q; a.page_table = page_table; a.q_start = q_start; a.q_len = q_len; a.ctx_len = ctx_len; a.gate = gate; a.ldg = ldg;
+  a.max_pages = max_pages; a.H = H; a.G = G; a.DK = DK; a.DV = DV; a.out_f32 = out_f32; a.out_bf16 = (__nv_bfloat16*)out_bf16; a.ldo = ldo;
+  a.KS = KS; a.maps = maps; a.chunk = chunk; a.sinks = sinks; a.shared_kv = vc ? 0 : 1;
+  const size_t smem = 4 * ((size_t)kExactRows * DK + (size_t)kExactKeys * (DK + 1) + (vc ? (size_t)kExactKeys * DV : 0));
+  if (smem > 200 * 1024) return B200_ERR_BAD_ARG;
+  const dim3 grid((max_q + kExactRows - 1) / kExactRows, H, n_seqs);
+  if (cache_f32) return launch_exact<float>(DV, grid, smem, a, (const float*)kc, (const float*)vc, st);
+  return launch_exact<__half>(DV, grid, smem, a, (const __half*)kc, (const __half*)vc, st);
+}
+
+// ------------------------------------------------------------------ differential attention: the difference of two maps
+
+// One warp per (token, head): o = a1 - lambda a2 over the two maps' outputs, divided by its root mean square over the head's values, times
+// `mult`.  in [T][2 H][DV] in qkv_finish's order; out [T][ldo] with head h at column h * DV, padding columns zero.
+__global__ void __launch_bounds__(128) diff_combine_kernel(const float* __restrict__ in, const float* __restrict__ lambda, int H, int G, int vdim, int DV,
+                                                           float eps, float mult, float* __restrict__ out_f32, __nv_bfloat16* __restrict__ out_bf16,
+                                                           int ldo) {
+  const float lam = *lambda;
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (h >= H) return;
+  const int rep = H / G, g = h / rep, r = h % rep;
+  const float* a1 = in + ((size_t)t * 2 * H + (g * 2) * rep + r) * DV;
+  const float* a2 = a1 + (size_t)rep * DV;
+  float ss = 0.f;
+  for (int e = lane; e < vdim; e += 32) {
+    const float o = a1[e] - lam * a2[e];
+    ss += o * o;
+  }
+  const float m = mult / sqrtf(warp_sum(ss) / (float)vdim + eps);
+  for (int e = lane; e < DV; e += 32) {
+    const float o = e < vdim ? (a1[e] - lam * a2[e]) * m : 0.f;
+    const size_t at = (size_t)t * ldo + (size_t)h * DV + e;
+    if (out_f32) out_f32[at] = o;
+    if (out_bf16) out_bf16[at] = __float2bfloat16(o);
+  }
+}
+B200_API int b200_diff_combine(const float* in, const float* lambda, int T, int H, int G, int vdim, int DV, float eps, float mult,
+                               float* out_f32, void* out_bf16, int ldo, cudaStream_t st) {
+  if (T < 1 || G < 1 || H % G || vdim < 1 || vdim > DV || ldo < H * DV || (!out_f32 && !out_bf16)) return B200_ERR_BAD_ARG;
+  return launch_pdl(diff_combine_kernel, dim3(T, (H + 3) / 4), dim3(128), 0, st, in, lambda, H, G, vdim, DV, eps, mult, out_f32,
+                    (__nv_bfloat16*)out_bf16, ldo);
 }
 
 // ------------------------------------------------------------------ matrix product in 32-bit
 
-// C[M][N] = act(A[M][K] W[N][K]^T): fp32 activations, bf16-stored weights (their expansion is exact), fp32 multiply-adds on the
+// C[M][N] = act(alpha A[M][K] W[N][K]^T), times sigmoid(gate[M][N]) where given, added into C (accumulate) or stored: fp32 activations, bf16-stored weights (their expansion is exact), fp32 multiply-adds on the
 // CUDA cores.  The 32-bit mode's projection; 64 x 64 tiles, 16 K columns staged at a time, 4 x 4 outputs per thread.
+// heads > 1: head z multiplies columns z * head_k of A with rows z * N of W into columns z * head_ldc of C.
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W,
-                                                       int ldb, float* __restrict__ C, int ldc, int M, int N, int K, int act) {
+                                                       int ldb, float* __restrict__ C, int ldc, int M, int N, int K, int act, float alpha,
+                                                       int accumulate, const float* __restrict__ gate, int ldg, int head_k, int head_ldc) {
   __shared__ float sA[16][68], sB[16][68];
   pdl_trigger();
   pdl_wait();
+  A += (size_t)blockIdx.z * head_k;
+  W += (size_t)blockIdx.z * N * ldb;
+  C += (size_t)blockIdx.z * head_ldc;
+  if (gate) gate += (size_t)blockIdx.z * head_ldc;
   const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64, tid = threadIdx.x;
   const int tx = tid & 15, ty = tid >> 4;
   float acc[4][4] = {};
@@ -439,17 +622,21 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
     for (int j = 0; j < 4; j++) {
       const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
       if (m >= M || n >= N) continue;
-      float v = acc[i][j];
+      float v = acc[i][j] * alpha;
       if (act == 1) v = v > 0.f ? v * v : 0.f;
-      C[(size_t)m * ldc + n] = v;
+      else if (act == 2) v = gelu_erf(v);
+      if (gate) v *= 1.f / (1.f + expf(-gate[(size_t)m * ldg + n]));
+      float* c = C + (size_t)m * ldc + n;
+      *c = accumulate ? *c + v : v;
     }
 }
-// act: 0 none, 1 the square of relu.
+// act: 0 none, 1 the square of relu, 2 the erf gelu.
 B200_API int b200_gemm_f32(const float* A, int lda, const void* W, int ldb, float* C, int ldc, int M, int N, int K, int act,
-                           cudaStream_t st) {
-  if (M < 1 || N < 1 || K < 1 || lda < K || ldb < K || ldc < N || act < 0 || act > 1) return B200_ERR_BAD_ARG;
-  return launch_pdl(gemm_f32_kernel, dim3((N + 63) / 64, (M + 63) / 64), dim3(256), 0, st, A, lda, (const __nv_bfloat16*)W, ldb, C,
-                    ldc, M, N, K, act);
+                           float alpha, int accumulate, const float* gate, int ldg, int heads, int head_k, int head_ldc, cudaStream_t st) {
+  if (M < 1 || N < 1 || K < 1 || heads < 1 || lda < (heads - 1) * head_k + K || ldb < K || ldc < (heads - 1) * head_ldc + N || act < 0 || act > 2)
+    return B200_ERR_BAD_ARG;
+  return launch_pdl(gemm_f32_kernel, dim3((N + 63) / 64, (M + 63) / 64, heads), dim3(256), 0, st, A, lda, (const __nv_bfloat16*)W, ldb, C,
+                    ldc, M, N, K, act, alpha, accumulate, gate, ldg, head_k, head_ldc);
 }
 
 // ------------------------------------------------------------------ last step of the logits

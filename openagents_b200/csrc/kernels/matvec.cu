@@ -13,7 +13,7 @@
 using namespace b200;
 
 enum { WT_Q4KR = 0, WT_Q6KR = 1, WT_Q8R = 2, WT_BF16 = 3 };
-enum { EPI_STORE = 0, EPI_RESID = 1, EPI_SWIGLU_Q8 = 2, EPI_SWIGLU_F32 = 3, EPI_ALLREDUCE = 4, EPI_ROPE_KV = 5, EPI_RELU2 = 6 };
+enum { EPI_STORE = 0, EPI_RESID = 1, EPI_SWIGLU_Q8 = 2, EPI_SWIGLU_F32 = 3, EPI_ALLREDUCE = 4, EPI_ROPE_KV = 5, EPI_RELU2 = 6, EPI_GELU_ERF = 7 };
 
 struct MatvecArgs {
   const uint8_t* w;     // main plane
@@ -27,6 +27,7 @@ struct MatvecArgs {
   int epi;
   const float* bias;    // [N] or null (dual: [2N])
   const float* resid;   // [nb][ldy] (EPI_RESID)
+  float alpha;          // EPI_RESID: multiplies the product
   float* y;             // [nb][ldy]
   int ldy;
   int8_t* oq;           // EPI_SWIGLU_Q8 outputs
@@ -228,8 +229,10 @@ __device__ __forceinline__ void matvec_epilogue(const MatvecArgs& a, const float
     }
   } else if (a.epi == EPI_RELU2) {
     if (live) a.y[(size_t)b * a.ldy + n] = v > 0.f ? v * v : 0.f;
+  } else if (a.epi == EPI_GELU_ERF) {
+    if (live) a.y[(size_t)b * a.ldy + n] = gelu_erf(v);
   } else if (a.epi == EPI_RESID) {
-    if (live) a.y[(size_t)b * a.ldy + n] = a.resid[(size_t)b * a.ldy + n] + v;
+    if (live) a.y[(size_t)b * a.ldy + n] = fmaf(v, a.alpha, a.resid[(size_t)b * a.ldy + n]);
   } else if (a.epi == EPI_ALLREDUCE) {
     if (live) sym_red_all_f32(a.sym, a.sym_off + ((size_t)b * a.ldy + n) * 4, v);
   } else {
@@ -516,7 +519,7 @@ static int run_matvec(int wt, MatvecArgs& a, cudaStream_t st) {
 B200_API int b200_matvec(int wt, const void* w, const void* w2, int N, int K, int nb, const void* xq,
                          const float* xd, const float* xs16, const float* xf, int epi, const float* bias,
                          const float* resid, float* y, int ldy, void* oq, float* od, float* os16,
-                         const SymTable* sym, size_t sym_off, int wait_ready, cudaStream_t st) {
+                         const SymTable* sym, size_t sym_off, int wait_ready, float alpha, cudaStream_t st) {
   if (nb < 1 || nb > 8 || epi == EPI_ROPE_KV) return B200_ERR_BAD_ARG;
   if (wt == WT_BF16 ? (K % 8 != 0 || (uintptr_t)xf % 16) : (K % 256 != 0 && !(wt == WT_Q8R && K % 32 == 0))) return B200_ERR_BAD_ARG;
   if (epi == EPI_SWIGLU_Q8 && N % 32) return B200_ERR_BAD_ARG;
@@ -533,6 +536,7 @@ B200_API int b200_matvec(int wt, const void* w, const void* w2, int N, int K, in
     a.sym_off = 0;
   }
   a.wait_ready = wait_ready;
+  a.alpha = alpha;
   return run_matvec(wt, a, st);
 }
 

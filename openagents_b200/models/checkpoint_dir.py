@@ -69,7 +69,7 @@ class CheckpointDirSource(WeightSource):
         self.device = device
         ranks = {}
         for name, (_, shape, _, _) in self.file.entries.items():      # sizes only a tensor's shape gives
-            if name.startswith("l") and name.endswith(".mix.a1") and len(shape) == 2 and name[1:-7].isdigit():
+            if name.startswith("l") and name.endswith((".mix.a1", ".mix.dq")) and len(shape) == 2 and name[1:-7].isdigit():
                 ranks[int(name[1:-7])] = shape[0]
         self.cfg = config_from_json(self.json, ranks, name=os.path.basename(os.path.normpath(path)))
         self.metadata: dict = {}
@@ -78,7 +78,7 @@ class CheckpointDirSource(WeightSource):
             e = self.file.entries.get(spec.name)
             if e is None:
                 raise ValueError(f"{path}: tensor {spec.name!r} is missing")
-            if e[1] != tuple(spec.shape):
+            if (e[1] or (1,)) != tuple(spec.shape):        # a number may be stored without an axis
                 raise ValueError(f"{path}: tensor {spec.name!r} has shape {list(e[1])}, expected {list(spec.shape)}")
 
     def has(self, name):
@@ -86,7 +86,7 @@ class CheckpointDirSource(WeightSource):
 
     def get(self, name):
         dt, shape, _, _ = self.file.entries[name]
-        t = _DTYPES[dt][2]
+        t, shape = _DTYPES[dt][2], shape or (1,)
         if t is None:
             raise ValueError(f"tensor {name!r} holds integers")
         return RawTensor(t, shape, self.file.tensor(name).reshape(-1).view(torch.uint8).to(self.device))

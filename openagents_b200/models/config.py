@@ -13,7 +13,8 @@ from dataclasses import asdict, dataclass, replace
 @dataclass(frozen=True)
 class MixerSpec:
     """What mixes tokens in one layer of a hybrid stack.  ``kind`` "attention": softmax attention over the paged cache;
-    "gla": gated linear attention with a decay per key channel and a state slot per sequence."""
+    "latent": softmax attention whose keys and values are projections of one cached latent per token; "gla": gated linear
+    attention with a decay per key channel and a state slot per sequence."""
     kind: str
     heads: int
     dim: int                       # per-head query / key size
@@ -27,16 +28,33 @@ class MixerSpec:
     qk_norm: bool = False          # q and k divided by their root mean square per head, after the rotation
     head_gate: bool = False        # one sigmoid gate per head on the output
     kv_from: int | None = None     # this layer reads the keys and values of an earlier one
+    bias: bool = False             # q, k and v projections have biases
+    chunk: int = 0                 # keys of the query's own chunk of this many positions only (0: all earlier ones)
+    maps: int = 1                  # 2: differential attention, two maps over the same values, the second one subtracted
+    diff: float = 0.0              # the constant part of the second map's weight
+    # latent attention (``dim``: unrotated query / key dimensions, rope_dims of the rot_dim others rotate)
+    rot_dim: int = 0               # query / key dimensions beside ``dim`` whose key part is shared by all heads
+    kv_rank: int = 0               # size of the cached latent
+    q_rank: int = 0                # size of the queries' latent
+    sink: bool = False             # a learned term per head in the softmax's denominator
+    out_gate: bool = False         # a sigmoid gate per output element
     # gla
     tau: float = 1.0               # decay = sigmoid(z)^(1/tau)
     rank: int = 16                 # rank of the decay's projection
 
     def __post_init__(self):
-        if self.kind not in ("attention", "gla"):
+        if self.kind not in ("attention", "latent", "gla"):
             raise ValueError(f"unknown mixer {self.kind!r}")
         if min(self.heads, self.dim, self.vdim) < 1:
             raise ValueError("a mixer's heads and sizes must be positive")
-        if self.kind == "attention":
+        if self.kind == "latent":
+            if min(self.kv_rank, self.q_rank) < 1 or self.rot_dim < 0:
+                raise ValueError("a latent mixer's ranks must be positive")
+            if not 0 <= self.rope_dims <= self.rot_dim or self.rope_dims % 2:
+                raise ValueError("the rotated dimensions must be even and within the rotated part of the head")
+        elif self.kind == "attention":
+            if self.chunk < 0 or self.maps not in (1, 2):
+                raise ValueError("bad chunk size or number of maps")
             if self.kv_heads < 1 or self.heads % self.kv_heads:
                 raise ValueError("the key/value heads must divide the query heads")
             if not 0 <= self.rope_dims <= self.dim or self.rope_dims % 2:
@@ -47,15 +65,16 @@ class MixerSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    """One layer of a hybrid stack: a mixer and, unless ``ffn`` is 0, a feed-forward of that width; a norm before and behind each."""
+    """One layer of a hybrid stack: a mixer and, unless ``ffn`` is 0, a feed-forward of that width; a norm before each and, where the
+    model has them (``ModelConfig.post_norm``), behind each."""
     mixer: MixerSpec
     ffn: int = 0
-    act: str = "relu2"             # the square of relu
+    act: str = "relu2"             # "relu2": the square of relu; "gelu": the exact (erf) gelu
 
 
 @dataclass(frozen=True)
 class ModelConfig:
-    arch: str = "llama"            # llama | gpt2 | gpt-oss | folirax
+    arch: str = "llama"            # llama | gpt2 | gpt-oss | folirax | pesorax
     n_layers: int = 2
     d_model: int = 256
     n_heads: int = 4
@@ -77,6 +96,10 @@ class ModelConfig:
     qkv_bias: bool = False
     # hybrid stacks: the layers one by one (the flat head and width fields above then hold the largest of each)
     layers: tuple[LayerSpec, ...] = ()
+    norm: str = "rms"              # "rms": root-mean-square, weights stored around zero; "dyt": w * tanh(alpha x) + b, no statistics
+    post_norm: bool = True         # a norm behind every sublayer as well
+    residual_mult: float = 1.0     # multiplies what a sublayer adds to the residual (stacks without post_norm)
+    loop: tuple[int, int, int] | None = None     # (start, stop, times): these layers run ``times`` times in a row, the embedding added ahead of every pass but the first
     logit_scale: float = 1.0
     logit_softcap: float = 0.0     # 0 = none
     name: str = "tiny-llama"
@@ -91,6 +114,15 @@ class ModelConfig:
 
     def layer_uses_window(self, i: int) -> bool:
         return self.sliding_window > 0 and i % self.swa_every == 0
+
+    def layer_runs(self) -> list[tuple[int, bool]]:
+        """Hybrid stacks: the layers in the order they run, and whether the embedding is added to the residual ahead of each."""
+        n = len(self.layers)
+        if self.loop is None:
+            return [(i, False) for i in range(n)]
+        a, b, times = self.loop
+        body = [(i, p > 0 and i == a) for p in range(times) for i in range(a, b)]
+        return [(i, False) for i in range(a)] + body + [(i, False) for i in range(b, n)]
 
     @property
     def has_state(self) -> bool:
@@ -237,8 +269,67 @@ def _folirax(c: dict, ranks: dict[int, int], name: str, context: int) -> ModelCo
                        logit_softcap=0.0 if cap is None else _need(c, "logit_softcap", float, ""), name=name)
 
 
+def _pesorax(c: dict, ranks: dict[int, int], name: str, context: int) -> ModelConfig:
+    """Pesorax: chunked differential attention (biased projections, no positions in the scores) and latent attention (a query latent, half-split
+    rotation of a shared key part, sinks, a gate per output element) in any order, Dynamic Tanh ahead of every sublayer, scaled
+    residual branches, erf-gelu feed-forwards, and a span of layers that runs several times."""
+    layers = []
+    for i, e in enumerate(_need(c, "layers", list, "")):
+        w = f"layers[{i}]."
+        mx, kind = _need(e, "mixer", dict, w), _need(e, "type", str, w)
+        w2 = w + "mixer."
+        common = dict(heads=_need(mx, "heads", int, w2), dim=_need(mx, "dim", int, w2), vdim=_need(mx, "vdim", int, w2), scale=_need(mx, "scale", float, w2))
+        if kind == "attention":
+            chunk = 0 if mx.get("mask") is None else _need(_need(mx, "mask", dict, w2), "size", int, w2 + "mask.")
+            if mx.get("mask") is not None and chunk < 1:
+                raise ValueError(f"config: {w2}mask.size must be positive")
+            m = MixerSpec("attention", **common, kv_heads=_need(mx, "kv_heads", int, w2), bias=True, chunk=chunk, maps=2, diff=_need(mx, "diff", float, w2))
+        elif kind == "latent_attention":
+            rot = _need(mx, "rot", dict, w2)
+            rank = _need(mx, "q_rank", int, w2) if mx.get("q_rank") is not None or i not in ranks else ranks[i]
+            m = MixerSpec("latent", **common, rot_dim=_need(mx, "rot_dim", int, w2), kv_rank=_need(mx, "kv_rank", int, w2), q_rank=rank,
+                          rope_base=_need(rot, "base", float, w2 + "rot."), rope_dims=_need(rot, "dims", int, w2 + "rot."), rope_style="half",
+                          sink=True, out_gate=True)
+        else:
+            raise ValueError(f"config: {w}type {kind!r} is not a mixer of this design")
+        mlp = e.get("mlp")
+        if mlp is not None and _need(mlp, "kind", str, w + "mlp.") != "dense":
+            raise ValueError(f"config: {w}mlp.kind {mlp['kind']!r} is not known")
+        layers.append(LayerSpec(m, 0 if mlp is None else _need(mlp, "ff", int, w + "mlp."), "gelu"))
+    if not layers:
+        raise ValueError("config: layers is empty")
+    loop = None
+    if c.get("loop") is not None:
+        lp = _need(c, "loop", dict, "")
+        loop = tuple(_need(lp, k, int, "loop.") for k in ("start", "stop", "times"))
+        if not 0 <= loop[0] < loop[1] <= len(layers) or loop[2] < 1:
+            raise ValueError("config: loop must name a span of layers and a positive number of passes")
+    mx = [l.mixer for l in layers]
+    return ModelConfig(arch="pesorax", n_layers=len(layers), d_model=_need(c, "width", int, ""), vocab=_need(c, "vocab", int, ""),
+                       n_heads=max(m.heads for m in mx), n_kv_heads=max(1, *(m.kv_heads for m in mx)), head_dim=max(m.dim for m in mx),
+                       ffn=max(l.ffn for l in layers), context=context, norm_eps=_need(_need(c, "norm", dict, ""), "eps", float, "norm."),
+                       layers=tuple(layers), norm="dyt", post_norm=False, loop=loop,
+                       residual_mult=1.0 if c.get("residual_mult") is None else _need(c, "residual_mult", float, ""), name=name)
+
+
+def _pesorax_to_json(cfg: ModelConfig) -> dict:
+    layers = []
+    for l in cfg.layers:
+        m = l.mixer
+        mx = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale}
+        if m.kind == "latent":
+            mx.update(rot_dim=m.rot_dim, kv_rank=m.kv_rank, q_rank=m.q_rank, rot={"base": m.rope_base, "dims": m.rope_dims})
+        else:
+            mx.update(kv_heads=m.kv_heads, diff=m.diff, mask={"size": m.chunk} if m.chunk else None)
+        layers.append({"type": "latent_attention" if m.kind == "latent" else "attention", "mixer": mx, "mlp": {"kind": "dense", "ff": l.ffn} if l.ffn else None})
+    return {"architecture": "Pesorax", "layers": layers, "width": cfg.d_model, "vocab": cfg.vocab, "norm": {"eps": cfg.norm_eps},
+            "loop": None if cfg.loop is None else dict(zip(("start", "stop", "times"), cfg.loop)), "residual_mult": cfg.residual_mult}
+
+
 def hybrid_to_json(cfg: ModelConfig) -> dict:
     """The inverse of ``config_from_json``."""
+    if cfg.arch == "pesorax":
+        return _pesorax_to_json(cfg)
     layers = []
     for l in cfg.layers:
         m = l.mixer
@@ -255,12 +346,13 @@ def hybrid_to_json(cfg: ModelConfig) -> dict:
             "ranks": {str(i): l.mixer.rank for i, l in enumerate(cfg.layers) if l.mixer.kind == "gla"}}
 
 
-JSON_ARCHITECTURES = {"Folirax": _folirax}
+JSON_ARCHITECTURES = {"Folirax": _folirax, "Pesorax": _pesorax}
+HYBRID_ARCHS = tuple(a.lower() for a in JSON_ARCHITECTURES)
 
 
 def config_from_json(c: dict, ranks: dict[int, int] | None = None, name: str | None = None, context: int = HYBRID_CONTEXT) -> ModelConfig:
-    """A model configuration from a checkpoint folder's config.json.  ``ranks``: sizes the file leaves to the tensors' shapes (rank
-    of the decay projection by layer)."""
+    """A model configuration from a checkpoint folder's config.json.  ``ranks``: sizes the file may leave to the tensors' shapes, by layer
+    (rank of the decay projection, size of the queries' latent)."""
     arch = _need(c, "architecture", str, "")
     reader = JSON_ARCHITECTURES.get(arch)
     if reader is None:
@@ -305,4 +397,22 @@ def folirax_stack(width: int, ffn: int, vocab: int, groups: int, heads: int, kv_
 FOLIRAX_8B = folirax_stack(4096, 14336, 128256, 8, 32, 8, 128, 16, 128, 256, "folirax-8b-shape")
 FOLIRAX_1B = folirax_stack(2048, 8192, 32000, 4, 16, 4, 128, 8, 128, 256, "folirax-1b-shape")
 
-PRESETS = {c.name: c for c in (TINY_LLAMA, LLAMA3_8B, LLAMA3_70B, GPT2_SMALL, GPT_OSS_20B, FOLIRAX_8B, FOLIRAX_1B)}
+
+
+def pesorax_stack(width: int, ffn: int, vocab: int, groups: int, heads: int, kv_heads: int, dim: int, vdim: int, chunk: int, latent_heads: int,
+                  latent_dim: int, rot_dim: int, latent_vdim: int, kv_rank: int, q_rank: int, name: str, loop: tuple[int, int, int] | None = None) -> ModelConfig:
+    """A regular stack: ``groups`` times (three chunked differential attention layers, then a latent attention layer)."""
+    local = LayerSpec(MixerSpec("attention", heads, dim, vdim, kv_heads=kv_heads, scale=dim ** -0.5, bias=True, chunk=chunk, maps=2, diff=0.5), ffn, "gelu")
+    latent = LayerSpec(MixerSpec("latent", latent_heads, latent_dim, latent_vdim, scale=(latent_dim + rot_dim) ** -0.5, rope_base=500000.0, rope_dims=rot_dim,
+                                 rope_style="half", rot_dim=rot_dim, kv_rank=kv_rank, q_rank=q_rank, sink=True, out_gate=True), ffn, "gelu")
+    layers = (local, local, local, latent) * groups
+    return ModelConfig(arch="pesorax", n_layers=len(layers), d_model=width, n_heads=max(heads, latent_heads), n_kv_heads=kv_heads, head_dim=max(dim, latent_dim),
+                       ffn=ffn, vocab=vocab, context=HYBRID_CONTEXT, norm_eps=1e-5, layers=layers, norm="dyt", post_norm=False, loop=loop, residual_mult=0.5,
+                       name=name)
+
+
+# the same two sizes with differential and latent attention; the smaller one runs its middle layers twice
+PESORAX_8B = pesorax_stack(4096, 14336, 128256, 8, 16, 4, 64, 128, 2048, 32, 128, 64, 128, 512, 1536, "pesorax-8b-shape")
+PESORAX_1B = pesorax_stack(2048, 8192, 32000, 3, 8, 2, 64, 128, 1024, 16, 128, 64, 128, 512, 768, "pesorax-1b-shape", loop=(4, 8, 2))
+
+PRESETS = {c.name: c for c in (TINY_LLAMA, LLAMA3_8B, LLAMA3_70B, GPT2_SMALL, GPT_OSS_20B, FOLIRAX_8B, FOLIRAX_1B, PESORAX_8B, PESORAX_1B)}

@@ -1,19 +1,24 @@
-"""Engine for hybrid stacks: softmax attention over the paged cache and gated linear attention with a state slot per sequence,
-layer by layer in the order the configuration gives, a norm on both sides of every sublayer.
+"""Engine for hybrid stacks: softmax attention over the paged cache (plain, chunked, differential, or in a latent space) and gated linear
+attention with a state slot per sequence, layer by layer in the order the configuration gives.
 
-Batching, pages, state slots, CUDA graphs and the public operations are ``PagedEngine``'s.  A step runs, per sublayer:
-``norm_residual`` (the previous sublayer's norm, the residual sum, this one's norm, in one pass), one fused projection
-(queries, keys, values, gates in one matrix), the mixer, and the output projection into an fp32 row that the next
-``norm_residual`` takes.  The residual stream, norms, rotations, scores, decays and states are fp32 in both modes.
+Batching, pages, state slots, CUDA graphs and the public operations are ``PagedEngine``'s.  Two kinds of residual step: with a norm on both
+sides of every sublayer, ``norm_residual`` (the previous sublayer's norm, the residual sum, this one's norm, in one pass) takes the fp32 row an
+output projection left; with a norm ahead only (Dynamic Tanh), the output projection adds its scaled product into the residual itself and
+``norm_dyt`` reads it.  Per sublayer one fused projection (queries, keys, values, gates, latents in one matrix), the mixer, and the output
+projection.  A looped span of layers runs several times with the same weights; every run has a cache (or state) of its own.  The residual
+stream, norms, rotations, scores, decays and states are fp32 in both modes.
+
+Latent attention: a step's short entries (single decoded tokens, portions of a few) come first in the batch and work in the latent space,
+straight on the cache; the others expand the latents of their context into keys and values and take the prompt kernel.
 
 ``dtype`` "bfloat16": projections and activations in bf16 on the tensor cores (up to ``small_path_tokens`` decoded tokens: the
-bf16 mat-vec on fp32 activations), fp16 keys and values.  "float32": fp32 activations, keys and values throughout, products on
+bf16 mat-vec on fp32 activations), fp16 keys, values and latents.  "float32": fp32 activations and caches throughout, products on
 the CUDA cores (the weights are bf16 numbers, whose expansion is exact).
 """
 from __future__ import annotations
 
 import os
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 
 import torch
 
@@ -22,6 +27,10 @@ from .config import LayerSpec, MixerSpec, ModelConfig
 from .engine import MATVEC_MAX_TOKENS, QGEMM_MAX_TOKENS
 from .paged import PAGE, PagedEngine
 from .qweight import WeightSource
+
+LATENT_CTAS = 592            # most CTAs of a latent decode launch that splits the keys
+SHORT_TOKENS = 16            # latent attention: entries of up to this many new tokens work in the latent space
+ACTS = {None: (ops.EPI_STORE, ops.ACT_NONE, 0), "relu2": (ops.EPI_RELU2, ops.ACT_RELU2, 1), "gelu": (ops.EPI_GELU_ERF, ops.ACT_GELU_ERF, 2)}
 
 
 def _up(n: int, m: int) -> int:
@@ -43,29 +52,75 @@ class _Lin:
 
 
 @dataclass
+class _Norm:
+    """An RMS norm's weight, or Dynamic Tanh's weight, shift and scalar."""
+    w: torch.Tensor
+    b: torch.Tensor | None = None
+    alpha: torch.Tensor | None = None
+
+
+@dataclass
+class _Latent:
+    """A latent mixer's own weights and padded sizes.  CR / RR: columns of the latent and of the rotated key part in the cache; KN: of a head's own key
+    part once expanded; QH: of a head in the query projection; offs: columns of the query latent, the latent, the rotated part and the gate."""
+    CR: int
+    RR: int
+    KN: int
+    QH: int
+    offs: tuple[int, int, int, int]
+    uq: _Lin
+    absorb: torch.Tensor         # [heads * CR][dim]: a head's queries into the latent space
+    value: torch.Tensor          # [heads * DV][CR]: a head's values out of it
+    expand: _Lin | None          # [heads * (KN + DV)][CR]: every head's keys and values of a latent
+    q_norm: torch.Tensor
+    c_norm: torch.Tensor
+
+
+@dataclass
 class _Block:
     spec: LayerSpec
-    norm1: torch.Tensor
-    norm1b: torch.Tensor
+    norm1: _Norm
+    norm1b: _Norm | None
     proj: _Lin
     out: _Lin
-    DK: int = 0                  # attention: padded head sizes of queries / keys and values;  gla: DV is the padded value size
+    DK: int = 0                  # attention: padded head sizes of queries / keys and values;  gla, latent: DV is the padded value size
     DV: int = 0
-    tc: bool = False             # attention: the tensor-core kernels take these head sizes
-    kv: int = -1                 # index of the key / value cache this layer reads
+    tc: bool = False             # attention, latent: the tensor-core kernels take these head sizes
+    bias: torch.Tensor | None = None
+    lam: torch.Tensor | None = None
+    sink: torch.Tensor | None = None
+    lat: _Latent | None = None
     table: torch.Tensor | None = None
     a2: torch.Tensor | None = None
     b2: torch.Tensor | None = None
     o_norm: torch.Tensor | None = None
-    state: torch.Tensor | None = None
-    norm2: torch.Tensor | None = None
-    norm2b: torch.Tensor | None = None
+    norm2: _Norm | None = None
+    norm2b: _Norm | None = None
     up: _Lin | None = None
     down: _Lin | None = None
 
 
+@dataclass
+class _Run:
+    """One pass of a layer: which cache it reads, its state, and whether the embedding joins the residual ahead of it."""
+    block: _Block
+    joins: bool
+    kv: int = -1                 # index among the key / value caches (latent mixers: among the latent caches)
+    state: torch.Tensor | None = None
+
+
+@dataclass
+class _Plan:
+    """Layout of a step that is not a decode step: its first ``n_short`` entries (``t_short`` tokens) work in the latent space, the others expand
+    their context, in groups [first, last, longest portion, longest context, rows] that fit the workspace."""
+    n_short: int = 0
+    t_short: int = 0
+    short_pages: int = 1
+    groups: list = field(default_factory=list)
+
+
 class HybridEngine(PagedEngine):
-    ARCHS = ("folirax",)
+    ARCHS = ("folirax", "pesorax")
     world = 1                    # one GPU; the serving layer asks
     vocab_sharded = False
 
@@ -80,6 +135,10 @@ class HybridEngine(PagedEngine):
         slots = 0 if not cfg.has_state else (state_slots if state_slots is not None else max_batch + max(4, max_batch // 4))
         self._init_paged(device, max_batch, max_ctx, n_pages, max_tokens, canaries, state_slots=slots)
         self.dp = _up(self.d, 8)
+        # Dynamic Tanh has no statistics of a row, so the residual itself can carry the padding (zeros stay zeros)
+        self.dx = self.dp if cfg.norm == "dyt" else self.d
+        if cfg.post_norm != (cfg.norm == "rms") or (cfg.post_norm and cfg.loop is not None):
+            raise ValueError("norms on both sides go with RMS norms and without a loop, Dynamic Tanh with a norm ahead only")
         # Decode batches up to this size take the mat-vec kernels.  Measured (ms per step, one token, mat-vec / GEMM): width 2048
         # 1.04 / 1.30, width 4096 4.41 / 4.19; the GEMM costs the same at eight tokens, the mat-vec grows with each.
         self.small_path_tokens = min(MATVEC_MAX_TOKENS, int(os.environ.get("B200_SMALL_PATH_TOKENS", 1)))
@@ -96,56 +155,133 @@ class HybridEngine(PagedEngine):
     def _matrix(self, src: WeightSource, name: str) -> torch.Tensor:
         return src.get(name).to_float().to(torch.bfloat16)
 
-    def _vector(self, src: WeightSource, name: str, centred: bool = False) -> torch.Tensor:
-        v = src.get(name).to_float().to(self.device).contiguous()
-        return v + 1.0 if centred else v
+    def _vector(self, src: WeightSource, name: str) -> torch.Tensor:
+        return src.get(name).to_float().to(self.device).contiguous()
+
+    def _norm(self, src: WeightSource, name: str) -> _Norm:
+        w = self._vector(src, name)
+        if self.cfg.norm == "rms":
+            return _Norm(w + 1.0)                        # stored around zero
+        pad = lambda v: torch.nn.functional.pad(v, (0, self.dx - self.d))        # noqa: E731
+        return _Norm(pad(w), pad(self._vector(src, name + ".b")), self._vector(src, name + ".alpha"))
 
     def _out_proj(self, src: WeightSource, name: str, heads: int, vdim: int, pad: int) -> _Lin:
         """The output projection with every head's columns padded to the mixer's output row."""
         w = self._matrix(src, name).view(self.d, heads, vdim)
         return self._lin(torch.nn.functional.pad(w, (0, pad - vdim)).reshape(self.d, heads * pad))
 
+    def _table(self, m: MixerSpec):
+        """(cos, sin) of every position of the cache, shared by the layers with the same rotation."""
+        if not m.rope_dims:
+            return None
+        key = (m.rope_base, m.rope_dims)
+        if key not in self._tables:
+            self._tables[key] = ops.rope_table(self.max_pages * PAGE, m.rope_dims, m.rope_base, self.device)
+        return self._tables[key]
+
     def _load(self, src: WeightSource):
         cfg = self.cfg
-        self.emb = self._matrix(src, "embed").to(self.device).contiguous()
+        emb = self._matrix(src, "embed")
+        self.emb = torch.nn.functional.pad(emb, (0, self.dx - self.d)).to(self.device).contiguous()
         self.blocks: list[_Block] = []
-        tables: dict[tuple, torch.Tensor] = {}
-        n_kv = 0
+        self._tables: dict[tuple, torch.Tensor] = {}
         for i, spec in enumerate(cfg.layers):
-            m, p = spec.mixer, f"l{i}."
-            names = ["q", "k", "v", "g", "a1"] if m.kind == "gla" else ["q"] + (["k", "v"] if m.kv_from is None else []) + (["g"] if m.head_gate else [])
-            proj = self._lin(torch.cat([self._matrix(src, f"{p}mix.{n}") for n in names]))
-            b = _Block(spec, self._vector(src, p + "norm1", True), self._vector(src, p + "norm1b", True), proj, None)
-            if m.kind == "gla":
-                b.DV = _up(m.vdim, 8)
-                b.a2 = src.get(p + "mix.a2").to_float().to(self.device).t().contiguous()
-                b.b2, b.o_norm = self._vector(src, p + "mix.a2.b"), self._vector(src, p + "mix.norm")
-                b.state = torch.zeros((self.state_slots, m.heads, m.dim, b.DV), dtype=torch.float32, device=self.device)
-            else:
-                b.DK, b.DV, b.tc = self._head_pad(m)
-                if m.kv_from is None:
-                    b.kv, n_kv = n_kv, n_kv + 1
-                else:
-                    b.kv = self.blocks[m.kv_from].kv
-                if m.rope_dims:
-                    key = (m.rope_base, m.rope_dims)
-                    if key not in tables:
-                        tables[key] = ops.rope_table(self.max_pages * PAGE, m.rope_dims, m.rope_base, self.device)
-                    b.table = tables[key]
-            b.out = self._out_proj(src, p + "mix.o", m.heads, m.vdim, b.DV)
+            p = f"l{i}."
+            b = {"gla": self._load_gla, "attention": self._load_attention, "latent": self._load_latent}[spec.mixer.kind](src, p + "mix.", spec)
+            b.norm1 = self._norm(src, p + "norm1")
+            if cfg.post_norm:
+                b.norm1b = self._norm(src, p + "norm1b")
             if spec.ffn:
-                b.norm2, b.norm2b = self._vector(src, p + "norm2", True), self._vector(src, p + "norm2b", True)
+                b.norm2 = self._norm(src, p + "norm2")
+                if cfg.post_norm:
+                    b.norm2b = self._norm(src, p + "norm2b")
                 b.up, b.down = self._lin(self._matrix(src, p + "mlp.up")), self._lin(self._matrix(src, p + "mlp.down"))
             self.blocks.append(b)
-        self.final_norm = self._vector(src, "final.norm", True)
+        self.runs: list[_Run] = []
+        self.kv_specs: list[_Block] = []                 # one key / value cache each
+        self.latent_specs: list[_Block] = []             # one latent cache each
+        at: dict[int, int] = {}                          # layer -> cache of its latest run
+        for i, joins in cfg.layer_runs():
+            b, m = self.blocks[i], cfg.layers[i].mixer
+            run = _Run(b, joins)
+            if m.kind == "gla":
+                run.state = torch.zeros((self.state_slots, m.heads, m.dim, b.DV), dtype=torch.float32, device=self.device)
+            else:
+                own = self.latent_specs if m.kind == "latent" else self.kv_specs
+                if m.kind == "attention" and m.kv_from is not None:
+                    run.kv = at[m.kv_from]
+                else:
+                    run.kv = at[i] = len(own)
+                    own.append(b)
+            self.runs.append(run)
+        self.final_norm = self._norm(src, "final.norm")
         self.head = self._lin(self._matrix(src, "head"))
         torch.cuda.synchronize(self.device)
 
+    def _load_gla(self, src: WeightSource, p: str, spec: LayerSpec) -> _Block:
+        m = spec.mixer
+        b = _Block(spec, None, None, self._lin(torch.cat([self._matrix(src, p + n) for n in ("q", "k", "v", "g", "a1")])), None, DV=_up(m.vdim, 8))
+        b.a2 = src.get(p + "a2").to_float().to(self.device).t().contiguous()
+        b.b2, b.o_norm = self._vector(src, p + "a2.b"), self._vector(src, p + "norm")
+        b.out = self._out_proj(src, p + "o", m.heads, m.vdim, b.DV)
+        return b
+
+    def _load_attention(self, src: WeightSource, p: str, spec: LayerSpec) -> _Block:
+        m = spec.mixer
+        own = ["k", "v"] if m.kv_from is None else []
+        parts = {n: self._matrix(src, p + n) for n in ["q"] + own + (["g"] if m.head_gate else [])}
+        biases = {n: self._vector(src, f"{p}{n}.b") for n in ["q"] + own} if m.bias else {}
+        if m.maps > 1:                                   # query rows (head, map) -> (key/value head, map, head of the group)
+            regroup = lambda w: w.view(m.kv_heads, m.heads // m.kv_heads, m.maps, m.dim, -1).transpose(1, 2).reshape(w.shape)      # noqa: E731
+            parts["q"] = regroup(parts["q"])
+            if m.bias:
+                biases["q"] = regroup(biases["q"])
+        b = _Block(spec, None, None, self._lin(torch.cat(list(parts.values()))), None)
+        if m.bias:
+            b.bias = torch.zeros(b.proj.N, dtype=torch.float32, device=self.device)
+            v = torch.cat(list(biases.values()))
+            b.bias[: v.numel()] = v
+        if m.maps > 1:
+            dot = lambda x, y: torch.exp((self._vector(src, p + x).double() * self._vector(src, p + y).double()).sum())      # noqa: E731
+            b.lam = (dot("lq1", "lk1") - dot("lq2", "lk2") + m.diff).float().view(1)
+        b.DK, b.DV, b.tc = self._head_pad(m)
+        b.table = self._table(m)
+        b.out = self._out_proj(src, p + "o", m.heads, m.vdim, b.DV)
+        return b
+
+    def _load_latent(self, src: WeightSource, p: str, spec: LayerSpec) -> _Block:
+        m, pad = spec.mixer, torch.nn.functional.pad
+        unit = 8 if self.exact else 64
+        CR, RR, KN, DV = _up(m.kv_rank, unit), _up(max(m.rot_dim, 1), unit), _up(m.dim, unit), _up(m.vdim, unit)
+        QH, QR = _up(m.dim + m.rot_dim, 8), _up(m.q_rank, 8)
+        tc = not self.exact and KN + RR <= 256 and DV <= 128 and ops.latent_decode_ok(m.heads, CR, RR)
+        if not tc and (CR > 1024 or 4 * (8 * (CR + RR) + 32 * (CR + RR + 1)) > 200 * 1024):
+            raise ValueError(f"latents of {m.kv_rank} + {m.rot_dim} are beyond the attention kernels")
+        heads = lambda w, n, to: pad(w.view(m.heads, n, -1), (0, 0, 0, to - n)).reshape(m.heads * to, -1)      # noqa: E731   (rows per head, padded)
+        dkv = self._matrix(src, p + "dkv")
+        parts = [pad(self._matrix(src, p + "dq"), (0, 0, 0, QR - m.q_rank)), pad(dkv, (0, 0, 0, _up(dkv.shape[0], 8) - dkv.shape[0]))]
+        offs = (0, QR, QR + m.kv_rank, QR + parts[1].shape[0])
+        if m.out_gate:
+            parts.append(heads(self._matrix(src, p + "g"), m.vdim, DV))
+        uk, uv = self._matrix(src, p + "uk"), self._matrix(src, p + "uv")
+        to_rank = (0, CR - m.kv_rank)
+        absorb = pad(uk.view(m.heads, m.dim, m.kv_rank).transpose(1, 2), (0, _up(m.dim, 8) - m.dim, 0, CR - m.kv_rank)).reshape(m.heads * CR, -1)
+        value = pad(heads(uv, m.vdim, DV), to_rank)
+        expand = self._lin(torch.cat([pad(heads(uk, m.dim, KN), to_rank), value])) if tc else None
+        lat = _Latent(CR, RR, KN, QH, offs, self._lin(pad(heads(self._matrix(src, p + "uq"), m.dim + m.rot_dim, QH), (0, QR - m.q_rank))),
+                      absorb.to(self.device).contiguous(), value.to(self.device).contiguous(), expand, self._vector(src, p + "dq.norm"),
+                      self._vector(src, p + "dkv.norm"))
+        b = _Block(spec, None, None, self._lin(torch.cat(parts)), self._out_proj(src, p + "o", m.heads, m.vdim, DV), DV=DV, tc=tc, lat=lat)
+        b.table = self._table(m)
+        if m.sink:
+            b.sink = self._vector(src, p + "sink")
+        return b
+
     def _head_pad(self, m: MixerSpec) -> tuple[int, int, bool]:
-        """Padded head sizes in the cache, and whether the tensor-core attention kernels take them (else, and always in the 32-bit
-        mode, the any-size kernel runs)."""
+        """Padded head sizes in the cache (keys: per map), and whether the tensor-core attention kernels take them (else, and always in
+        the 32-bit mode, the any-size kernel runs)."""
         dk, dv = _up(m.dim, 64), _up(m.vdim, 64)
-        if self.exact or dk > 256 or dv > 128:
+        if self.exact or m.maps * dk > 256 or dv > 128:
             return _up(m.dim, 8), _up(m.vdim, 8), False
         return dk, dv, True
 
@@ -153,6 +289,8 @@ class HybridEngine(PagedEngine):
         n = self.head.w.numel()
         for b in self.blocks:
             n += b.proj.w.numel() + b.out.w.numel() + (b.up.w.numel() + b.down.w.numel() if b.up is not None else 0)
+            if b.lat is not None:                        # what a decode step reads
+                n += b.lat.uq.w.numel() + b.lat.absorb.numel() + b.lat.value.numel()
         return 2 * n
 
     def scratch_bytes(self) -> int:
@@ -163,29 +301,51 @@ class HybridEngine(PagedEngine):
         T, d, dev = self.max_tokens, self.dp, self.device
         f32, bf = torch.float32, torch.bfloat16
         self._alloc_batch()
-        own = [b for b in self.blocks if b.spec.mixer.kind == "attention" and b.spec.mixer.kv_from is None]
         ct = f32 if self.exact else torch.float16
-        self.kc = [torch.zeros((self.n_pages, b.spec.mixer.kv_heads, PAGE, b.DK), dtype=ct, device=dev) for b in own]
-        self.vc = [torch.zeros((self.n_pages, b.spec.mixer.kv_heads, PAGE, b.DV), dtype=ct, device=dev) for b in own]
+        self.kc = [torch.zeros((self.n_pages, b.spec.mixer.kv_heads, PAGE, b.spec.mixer.maps * b.DK), dtype=ct, device=dev) for b in self.kv_specs]
+        self.vc = [torch.zeros((self.n_pages, b.spec.mixer.kv_heads, PAGE, b.DV), dtype=ct, device=dev) for b in self.kv_specs]
+        self.lc = [torch.zeros((self.n_pages, PAGE, b.lat.CR + b.lat.RR), dtype=ct, device=dev) for b in self.latent_specs]
         ws = self._ws
         n_proj = max(b.proj.N for b in self.blocks)
         n_mix = max(b.out.K for b in self.blocks)
         n_ffn = max((b.up.N for b in self.blocks if b.up is not None), default=8)
-        attn = [b for b in self.blocks if b.spec.mixer.kind == "attention"]
-        n_q = max((b.spec.mixer.heads * b.DK for b in attn), default=8)
-        n_q32 = max((b.spec.mixer.heads * b.DK for b in attn if not b.tc), default=0)      # rows of a prompt in fp32
-        self.x = ws("x", (T, self.d), f32)
-        self.y = ws("y", (T, d), f32, zero=True)
+        attn = [(b, b.spec.mixer, b.spec.mixer.heads * b.spec.mixer.maps) for b in self.blocks if b.spec.mixer.kind == "attention"]
+        lat = [(b, b.spec.mixer, b.lat) for b in self.blocks if b.lat is not None]
+        n_q = max((hq * m.maps * b.DK for b, m, hq in attn), default=8)
+        n_q32 = max((hq * b.DK for b, m, hq in attn if not b.tc), default=0)                # rows of a prompt in fp32
+        n_q16 = max([hq * b.DK for b, m, hq in attn if b.tc] + [m.heads * (L.KN + L.RR) for b, m, L in lat if b.tc], default=0)
+        self.x = ws("x", (T, self.dx), f32)
+        self.y = ws("y", (T if self.cfg.post_norm else 1, d), f32, zero=True)
         self.proj = ws("proj", (T * n_proj,), f32, zero=True)
         self.q32 = ws("q32", (max(T * n_q32, self.max_batch * n_q),), f32)
-        self.q16 = ws("q16", (T * n_q if any(b.tc for b in attn) else 8,), torch.float16)
-        tc = [(b.spec.mixer, b.DV) for b in attn if b.tc]
-        self.attn_scratch = ws("attn_scratch", (max((ops.attn_decode_scratch_floats(self.max_batch, m.heads, m.kv_heads, dv, self.max_splits)
-                                                     for m, dv in tc), default=4),), f32)
-        self.attn_counters = ws("attn_counters", (self.max_batch * max((m.heads for m, _ in tc), default=1),), torch.int32, zero=True)
+        self.q16 = ws("q16", (max(8, T * n_q16),), torch.float16)
+        self.maps_out = ws("maps_out", (T * max((hq * b.DV for b, m, hq in attn if m.maps > 1), default=0),), f32)
+        tc = [(m, b.DV, hq) for b, m, hq in attn if b.tc]
+        self.attn_scratch = ws("attn_scratch", (max((ops.attn_decode_scratch_floats(self.max_batch, hq, m.kv_heads, dv, self.max_splits)
+                                                     for m, dv, hq in tc), default=4),), f32)
+        self.attn_counters = ws("attn_counters", (self.max_batch * max((hq for _, _, hq in tc), default=1),), torch.int32, zero=True)
         gla = [b for b in self.blocks if b.spec.mixer.kind == "gla"]
         self.gla_ws = ws("gla_ws", (max((ops.gla_chunk_bytes(T, self.max_batch, m.heads, m.dim, dv, m.rank)
                                          for m, dv in ((b.spec.mixer, b.DV) for b in gla)), default=0) if not self.exact else 0,), torch.uint8)
+        # latent attention: rows in the latent space (all of a step's where the any-size kernel runs), and the expanded context of the others
+        self.short_rows = min(T, max(self.max_batch, 256))
+        rows = lambda b: self.short_rows if b.tc else T                                      # noqa: E731
+        widest = lambda f: max((f(b, m, L) for b, m, L in lat), default=0)                   # noqa: E731
+        self.cq = ws("cq", (T * widest(lambda b, m, L: L.uq.K),), f32 if self.exact else bf)
+        self.cq1 = ws("cq1", (MATVEC_MAX_TOKENS * widest(lambda b, m, L: L.uq.K) if not self.exact else 0,), f32)
+        self.uq32 = ws("uq32", (T * widest(lambda b, m, L: L.uq.N),), f32)
+        self.uq16 = ws("uq16", (widest(lambda b, m, L: T * L.uq.N) if not self.exact else 0,), bf)
+        self.q_lat = ws("q_lat", (widest(lambda b, m, L: rows(b) * m.heads * (L.CR + L.RR)),), f32)
+        self.o_lat = ws("o_lat", (widest(lambda b, m, L: rows(b) * m.heads * L.CR),), f32)
+        big_lat = any(b.tc for b, _, _ in lat)
+        self.ctx_rows = _up(max(T, self.max_pages * PAGE), 128) if big_lat else 0
+        self.ctx_lat = ws("ctx_lat", (self.ctx_rows * widest(lambda b, m, L: L.CR),), bf)
+        self.ctx_kv = ws("ctx_kv", (self.ctx_rows * widest(lambda b, m, L: m.heads * (L.KN + b.DV)),), torch.float16, zero=True)
+        # rows x shares stays below LATENT_CTAS wherever there is more than one share
+        self.lat_scratch = ws("lat_scratch", (widest(lambda b, m, L: ops.latent_decode_scratch_floats(LATENT_CTAS // 2, m.heads, L.CR, 2) if b.tc else 0),), f32)
+        self.row_seq = ws("row_seq", (T,), torch.int32, zero=True)
+        self.ctx_base = ws("ctx_base", (self.max_batch,), torch.int32, zero=True)
+        self._plan = _Plan()
         small = self.max_batch if not self.exact else T            # rows of the fp32 activations
         self.hf = ws("hf", (small * d,), f32)
         self.mf = ws("mf", (small * n_mix,), f32)
@@ -199,58 +359,166 @@ class HybridEngine(PagedEngine):
         self.argmax_scratch = ops.argmax_scratch(self.max_batch, dev)
         self.iota = torch.arange(self.max_batch, dtype=torch.int32, device=dev)
         self.ones = torch.ones(self.max_batch, dtype=torch.int32, device=dev)
-        k_max = max(d, n_mix, n_ffn)
+        k_max = max(d, n_mix, n_ffn, widest(lambda b, m, L: L.uq.K))
         # the bf16 mat-vec keeps its fp32 activations in shared memory
         self.matvec_rows = max((n for n in (1, 2, 4, 8) if n * (k_max * 4 + 256) <= 200 * 1024), default=0)
 
+    def _caches(self):
+        return [*self.kc, *self.vc, *self.lc]
+
+    # ------------------------------------------------------------------ batch layout (latent attention)
+    def _batch_order(self, q_len):
+        if not self.ctx_rows or all(n == 1 for n in q_len):
+            return None
+        order = sorted(range(len(q_len)), key=q_len.__getitem__)
+        return None if order == list(range(len(q_len))) else order
+
+    def _plan_batch(self, q_len, ctx):
+        if not self.ctx_rows:
+            return
+        p = self._plan = _Plan()
+        for n, c in zip(q_len, ctx):                     # shortest first
+            if n > SHORT_TOKENS or p.t_short + n > self.short_rows:
+                break
+            p.n_short, p.t_short, p.short_pages = p.n_short + 1, p.t_short + n, max(p.short_pages, (c + PAGE - 1) // PAGE)
+        rows = [b for b in range(p.n_short) for _ in range(q_len[b])]
+        base = [0] * len(q_len)
+        for b in range(p.n_short, len(q_len)):
+            if not p.groups or p.groups[-1][4] + ctx[b] > self.ctx_rows:
+                p.groups.append([b, b, 0, 0, 0])
+            g = p.groups[-1]
+            base[b] = g[4]
+            p.groups[-1] = [g[0], b + 1, max(g[2], q_len[b]), max(g[3], ctx[b]), g[4] + ctx[b]]
+        if rows:
+            self.row_seq[: len(rows)].copy_(torch.tensor(rows, dtype=torch.int32).pin_memory(), non_blocking=True)
+        self.ctx_base[: len(base)].copy_(torch.tensor(base, dtype=torch.int32).pin_memory(), non_blocking=True)
+
+    def _latent_splits(self, rows: int, heads: int, pages: int) -> int:
+        """Shares of the keys per row in the latent decode kernel: the fewest rounds over the SMs, a round costing its key blocks and a fixed set-up."""
+        ctas, blocks = rows * ((heads + 31) // 32), max(1, (min(pages, self.max_pages) * PAGE + 63) // 64)
+        cost = lambda s: -(-ctas * s // 148) * (-(-blocks // s) + 2)                       # noqa: E731
+        return min(range(1, max(1, min(self.max_splits, blocks, LATENT_CTAS // ctas)) + 1), key=cost)
+
     # ------------------------------------------------------------------ building blocks
-    def _mm(self, a: torch.Tensor, L: _Lin, out: torch.Tensor, act: int = 0, add: bool = False):
+    def _mm(self, a: torch.Tensor, L: _Lin, out: torch.Tensor, act: str | None = None, add: bool = False, into: float | None = None):
         """out = act(a W^T).  fp32 activations: mat-vec for a few rows, else the 32-bit product; bf16: the tensor-core GEMM (``add``:
-        the output was zeroed ahead, K may be split)."""
+        the output was zeroed ahead, K may be split).  ``into``: out += into * (a W^T)."""
         T = a.shape[0]
+        epi, gact, fact = ACTS[act]
         if a.dtype == torch.float32:
             if T <= self.matvec_rows:
-                ops.matvec(ops.WT_BF16, L.w, None, L.N, L.K, T, xf=a, epi=ops.EPI_RELU2 if act else ops.EPI_STORE, y=out, ldy=out.stride(0))
+                if into is not None:
+                    ops.matvec(ops.WT_BF16, L.w, None, L.N, L.K, T, xf=a, epi=ops.EPI_RESID, resid=out, y=out, ldy=out.stride(0), alpha=into)
+                else:
+                    ops.matvec(ops.WT_BF16, L.w, None, L.N, L.K, T, xf=a, epi=epi, y=out, ldy=out.stride(0))
             else:
-                ops.gemm_f32(a, L.w, out, act)
+                ops.gemm_f32(a, L.w, out, fact, alpha=1.0 if into is None else into, accumulate=into is not None)
         else:
             f32 = out.dtype == torch.float32
-            ops.gemm_bf16(a, L.w, T, L.N, L.K, lda=a.stride(0), ldb=L.K, out_f32=out if f32 else None, out_bf16=None if f32 else out,
-                          ldc=out.stride(0), act=ops.ACT_RELU2 if act else ops.ACT_NONE, accumulate=add and f32 and not act, status=self.status)
+            ops.gemm_bf16(a, L.w, T, L.N, L.K, lda=a.stride(0), ldb=L.K, out_f32=out if f32 else None, out_bf16=out if out.dtype == torch.bfloat16 else None,
+                          out_f16=out if out.dtype == torch.float16 else None, ldc=out.stride(0), act=gact, alpha=1.0 if into is None else into,
+                          accumulate=into is not None or (add and f32 and not act), status=self.status)
 
-    def _attention(self, b: _Block, proj, T: int, decode: bool, n_seqs: int, max_q: int, pages: int, o32, o16) -> int:
-        cfg, m = self.cfg, b.spec.mixer
-        own = m.kv_from is None
-        k_off = m.heads * m.dim if own else -1
-        v_off = k_off + m.kv_heads * m.dim
-        g_off = v_off + m.kv_heads * m.vdim if own else m.heads * m.dim
-        kc, vc = self.kc[b.kv], self.vc[b.kv]
-        tc_prompt = b.tc and not decode
-        q = (self.q16 if tc_prompt else self.q32)[: T * m.heads * b.DK].view(T, -1)
-        ops.qkv_finish(proj, 0, k_off, v_off, self.pos, self.slot, b.table, m.rope_base, m.heads, m.kv_heads, m.dim, m.vdim, b.DK, b.DV,
+    def _mm_heads(self, a: torch.Tensor, w: torch.Tensor, heads: int, head_k: int, out: torch.Tensor, head_ldc: int, alpha: float = 1.0, gate=None):
+        """One product per head: w [heads * N][K]; head z reads columns z * head_k of ``a`` and writes columns z * head_ldc of ``out``."""
+        N, K = w.shape[0] // heads, w.shape[1]
+        if a.dtype == torch.float32:
+            ops.gemm_f32(a, w, out, alpha=alpha, gate=gate, heads=heads, head_k=head_k, head_ldc=head_ldc)
+        else:
+            ops.gemm_heads(a, w, heads, N, K, head_k, out, head_ldc, alpha=alpha, gate=gate, status=self.status)
+
+    def _attention(self, r: _Run, proj, T: int, decode: bool, n_seqs: int, max_q: int, pages: int, o32, o16) -> int:
+        b, cfg = r.block, self.cfg
+        m = b.spec.mixer
+        own, HQ = m.kv_from is None, m.heads * m.maps
+        k_off = HQ * m.dim if own else -1
+        v_off = k_off + m.kv_heads * m.maps * m.dim
+        g_off = v_off + m.kv_heads * m.vdim if own else HQ * m.dim
+        kc, vc = self.kc[r.kv], self.vc[r.kv]
+        tc_prompt, wide = b.tc and not decode, b.tc and decode and m.maps > 1
+        q = (self.q16 if tc_prompt else self.q32)[: T * HQ * b.DK * (m.maps if wide else 1)].view(T, -1)
+        ops.qkv_finish(proj, 0, k_off, v_off, self.pos, self.slot, b.table, m.rope_base, HQ, m.kv_heads, m.dim, m.vdim, b.DK, b.DV,
                        m.rope_dims, 0 if m.rope_style == "pairs" else 1, m.qk_norm, cfg.norm_eps, m.scale, PAGE, q32=None if tc_prompt else q,
-                       q16=q if tc_prompt else None, kc=kc, vc=vc)
+                       q16=q if tc_prompt else None, kc=kc, vc=vc, maps=m.maps, q_wide=wide, bias=b.bias)
         gate = proj[:, g_off:] if m.head_gate else None
+        out32, out16 = o32, o16
+        if m.maps > 1:
+            out32, out16 = self.maps_out[: T * HQ * b.DV].view(T, -1), None
+        if m.chunk:
+            pages = min(pages, m.chunk // PAGE + 2)
         if tc_prompt:
-            ops.attn_prefill_tc05(q, kc, vc, self.page_table, self.q_start, self.q_len, self.seq_lens, n_seqs, max_q, m.heads, m.kv_heads,
-                                  out_bf16=o16, status=self.status, dk=b.DK, dv=b.DV, gate=gate)
+            ops.attn_prefill_tc05(q, kc, vc, self.page_table, self.q_start, self.q_len, self.seq_lens, n_seqs, max_q, HQ, m.kv_heads,
+                                  out_bf16=out16, out_f32=out32, status=self.status, dk=b.DK, dv=b.DV, gate=gate, chunk=m.chunk, maps=m.maps)
+        elif b.tc:
+            ops.attn_decode(q, kc, vc, self.page_table, self.seq_lens, n_seqs, HQ, m.kv_heads, m.maps * b.DK, dv=b.DV,
+                            S=self._attn_splits(n_seqs, m.kv_heads, pages), gate=gate, out_f32=out32, out_bf16=out16,
+                            scratch=self.attn_scratch, counters=self.attn_counters, status=self.status, chunk=m.chunk)
+        else:
+            qs, ql = (self.iota, self.ones) if decode else (self.q_start, self.q_len)
+            ops.attn_exact(q, kc, vc, self.page_table, qs, ql, self.seq_lens, n_seqs, max_q, HQ, m.kv_heads, b.DK, b.DV, gate=gate,
+                           out_f32=out32, out_bf16=out16, maps=m.maps, chunk=m.chunk)
+        if m.maps == 1:
             return 2
-        if b.tc:
-            ops.attn_decode(q, kc, vc, self.page_table, self.seq_lens, n_seqs, m.heads, m.kv_heads, b.DK, dv=b.DV,
-                            S=self._attn_splits(n_seqs, m.kv_heads, pages), gate=gate, out_f32=o32, out_bf16=o16,
-                            scratch=self.attn_scratch, counters=self.attn_counters, status=self.status)
-            return 2
-        qs, ql = (self.iota, self.ones) if decode else (self.q_start, self.q_len)
-        ops.attn_exact(q, kc, vc, self.page_table, qs, ql, self.seq_lens, n_seqs, max_q, m.heads, m.kv_heads, b.DK, b.DV, gate=gate,
-                       out_f32=o32, out_bf16=o16)
-        return 2
+        ops.diff_combine(out32, b.lam, m.heads, m.kv_heads, m.vdim, b.DV, cfg.norm_eps, 1.0 - m.diff, out_f32=o32, out_bf16=o16)
+        return 3
 
-    def _gla(self, b: _Block, proj, T: int, decode: bool, n_seqs: int, max_q: int, o32, o16) -> int:
+    def _latent(self, r: _Run, proj, T: int, decode: bool, n_seqs: int, max_q: int, pages: int, o32, o16) -> int:
+        b, L, cache = r.block, r.block.lat, self.lc[r.kv]
+        m, style = b.spec.mixer, 0 if b.spec.mixer.rope_style == "pairs" else 1
+        H, W, f32 = m.heads, L.CR + L.RR, o32 is not None
+        q_off, c_off, r_off, g_off = L.offs
+        gate = proj[:, g_off:] if m.out_gate else None
+        cq = (self.cq1 if f32 and not self.exact else self.cq)[: T * L.uq.K].view(T, -1)
+        ops.latent_finish(proj, q_off, c_off, r_off, m.q_rank, m.kv_rank, m.rot_dim, m.rope_dims, style, L.q_norm, L.c_norm, self.cfg.norm_eps, self.pos,
+                          self.slot, b.table, m.rope_base, cq, cache, L.CR, L.RR)
+        # rows in the latent space: all of a decode step's, and all where the tensor-core kernels do not run
+        plan = _Plan(n_seqs, T, pages) if decode or not b.tc else self._plan
+        t1, n = plan.t_short, 2
+        uq = self.uq32[: T * L.uq.N].view(T, -1)
+        a = uq
+        if f32:
+            self._mm(cq, L.uq, uq)
+        else:
+            a = self.uq16[: T * L.uq.N].view(T, -1)
+            ops.gemm_bf16(cq, L.uq.w, T, L.uq.N, L.uq.K, out_f32=uq, out_bf16=a if t1 else None, status=self.status)
+        rot = (self.pos, b.table, m.rope_base, m.scale)
+        if t1:
+            q = self.q_lat[: t1 * H * W].view(t1, H * W)
+            self._mm_heads(a[:t1], L.absorb, H, L.QH, q, W, alpha=m.scale)
+            ops.latent_q(uq[:t1], L.QH, H, m.dim, m.rot_dim, m.rope_dims, style, 0, L.CR, L.RR, W, *rot, q)
+            o = self.o_lat[: t1 * H * L.CR]
+            o = (o if f32 else o.view(torch.bfloat16)[: t1 * H * L.CR]).view(t1, -1)
+            out = dict(out_f32=o) if f32 else dict(out_bf16=o)
+            if b.tc:
+                S = self._latent_splits(t1, H, plan.short_pages)
+                ops.latent_decode(q, cache, self.page_table, None if decode else self.row_seq, self.pos, t1, H, L.CR, L.RR, S, self.lat_scratch, sinks=b.sink,
+                                  status=self.status, **out)
+                n += S > 1
+            else:
+                qs, ql = (self.iota, self.ones) if decode else (self.q_start, self.q_len)
+                ops.attn_exact(q, cache.view(self.n_pages, 1, PAGE, W), None, self.page_table, qs, ql, self.seq_lens, n_seqs, max_q, H, 1, W, L.CR, sinks=b.sink, **out)
+            self._mm_heads(o, L.value, H, L.CR, (o32 if f32 else o16)[:t1], b.DV, gate=None if gate is None else gate[:t1])
+            n += 4
+        if plan.groups:
+            q16 = self.q16[: T * H * (L.KN + L.RR)].view(T, -1)
+            ops.latent_q(uq, L.QH, H, m.dim, m.rot_dim, m.rope_dims, style, L.KN, L.KN, L.RR, L.KN + L.RR, *rot, q16)
+            n += 1
+            for lo, hi, group_q, group_ctx, rows in plan.groups:
+                c, kv = self.ctx_lat[: rows * L.CR].view(rows, -1), self.ctx_kv[: self.ctx_rows * L.expand.N].view(self.ctx_rows, -1)
+                ops.latent_gather(cache, L.CR, self.page_table[lo:], self.seq_lens[lo:], self.ctx_base[lo:], hi - lo, group_ctx, c)
+                self._mm(c, L.expand, kv[:rows])
+                ops.attn_prefill_latent(q16, kv, H * L.KN, self.ctx_base[lo:], cache, L.CR, self.page_table[lo:], self.q_start[lo:], self.q_len[lo:],
+                                        self.seq_lens[lo:], hi - lo, group_q, H, L.KN, L.RR, b.DV, o16, sinks=b.sink, gate=gate, status=self.status)
+                n += 3
+        return n
+
+    def _gla(self, r: _Run, proj, T: int, decode: bool, n_seqs: int, max_q: int, pages: int, o32, o16) -> int:
+        b = r.block
         m = b.spec.mixer
         qk, vv = m.heads * m.dim, m.heads * m.vdim
         offs = (0, qk, 2 * qk, 2 * qk + vv, 2 * qk + 2 * vv)
         qs, ql = (self.iota, self.ones) if decode else (self.q_start, self.q_len)
-        args = (proj, offs, m.rank, b.a2, b.b2, b.o_norm, b.state, qs, ql, self.seq_lens, self.state_slot, n_seqs, m.heads, m.dim, m.vdim, b.DV,
+        args = (proj, offs, m.rank, b.a2, b.b2, b.o_norm, r.state, qs, ql, self.seq_lens, self.state_slot, n_seqs, m.heads, m.dim, m.vdim, b.DV,
                 m.tau, m.dim ** -0.5, self.cfg.norm_eps)
         if decode or self.exact or not ops.gla_chunk_bytes(T, n_seqs, m.heads, m.dim, b.DV, m.rank):
             ops.gla_recurrent(*args, out_f32=o32, out_bf16=o16)
@@ -259,31 +527,41 @@ class HybridEngine(PagedEngine):
         return 3
 
     def _run_layers(self, T: int, decode: bool, n_seqs: int, max_q: int, pages: int) -> int:
-        eps, x, y = self.cfg.norm_eps, self.x[:T], self.y[:T]
         f32 = self.exact or (decode and T <= min(self.small_path_tokens, self.matvec_rows))
+        walk = self._walk_sandwich if self.cfg.post_norm else self._walk_prenorm
+        return walk(T, decode, f32, (decode, n_seqs, max_q, pages))
+
+    def _buffers(self, T: int, f32: bool):
+        """This step's row, the norms' destination, and the per-layer views of the activations."""
         h = (self.hf if f32 else self.hb)[: T * self.dp].view(T, self.dp)
-        hk = dict(hf=h) if f32 else dict(hb=h)
+        views = lambda b: (self.proj[: T * b.proj.N].view(T, b.proj.N), (self.mf if f32 else self.mb)[: T * b.out.K].view(T, b.out.K),      # noqa: E731
+                           (self.ff if f32 else self.fb)[: T * b.up.N].view(T, b.up.N) if b.up is not None else None)
+        return h, dict(hf=h) if f32 else dict(hb=h), views
+
+    def _mix(self, r: _Run, proj, mix, T: int, f32: bool, step) -> int:
+        fn = {"gla": self._gla, "attention": self._attention, "latent": self._latent}[r.block.spec.mixer.kind]
+        return fn(r, proj, T, *step, mix if f32 else None, None if f32 else mix)
+
+    def _walk_sandwich(self, T: int, decode: bool, f32: bool, step) -> int:
+        """A norm on both sides of every sublayer: each residual step waits for the next norm."""
+        eps, x, y = self.cfg.norm_eps, self.x[:T], self.y[:T]
+        h, hk, views = self._buffers(T, f32)
         add = not f32 and T <= QGEMM_MAX_TOKENS          # one row tile: the projections may split K and add into zeroed outputs
         gy, n = None, 0
-        for b in self.blocks:
-            proj = self.proj[: T * b.proj.N].view(T, b.proj.N)
-            mix = (self.mf if f32 else self.mb)[: T * b.out.K].view(T, b.out.K)
-            ops.norm_residual(x, eps, y=y if gy is not None else None, gy=gy, gh=b.norm1, y_clear=add, zero=proj if add else None,
+        for r in self.runs:
+            b = r.block
+            proj, mix, act = views(b)
+            ops.norm_residual(x, eps, y=y if gy is not None else None, gy=gy, gh=b.norm1.w, y_clear=add, zero=proj if add else None,
                               zero2=y if add and gy is None else None, **hk)
             self._mm(h, b.proj, proj, add=add)
-            o = (mix, None) if f32 else (None, mix)
-            if b.spec.mixer.kind == "gla":
-                n += self._gla(b, proj, T, decode, n_seqs, max_q, *o)
-            else:
-                n += self._attention(b, proj, T, decode, n_seqs, max_q, pages, *o)
+            n += self._mix(r, proj, mix, T, f32, step)
             self._mm(mix, b.out, y, add=add)
-            gy, n = b.norm1b, n + 3
-            if b.up is not None:
-                act = (self.ff if f32 else self.fb)[: T * b.up.N].view(T, b.up.N)
-                ops.norm_residual(x, eps, y=y, gy=gy, gh=b.norm2, y_clear=add, **hk)
-                self._mm(h, b.up, act, act=1)
+            gy, n = b.norm1b.w, n + 3
+            if act is not None:
+                ops.norm_residual(x, eps, y=y, gy=gy, gh=b.norm2.w, y_clear=add, **hk)
+                self._mm(h, b.up, act, act=b.spec.act)
                 self._mm(act, b.down, y, add=add)
-                gy, n = b.norm2b, n + 3
+                gy, n = b.norm2b.w, n + 3
         if decode:
             self._tail = gy                              # the last residual step is folded into the final norm
         else:
@@ -292,13 +570,40 @@ class HybridEngine(PagedEngine):
             n += 1
         return n
 
+    def _walk_prenorm(self, T: int, decode: bool, f32: bool, step) -> int:
+        """A norm ahead of every sublayer: output projections add into the residual."""
+        x, mult = self.x[:T], self.cfg.residual_mult
+        h, hk, views = self._buffers(T, f32)
+        add = not f32 and T <= QGEMM_MAX_TOKENS
+        n = 0
+        for r in self.runs:
+            b = r.block
+            proj, mix, act = views(b)
+            self._dyt(x, b.norm1, emb=self.emb if r.joins else None, zero=proj if add else None, **hk)
+            self._mm(h, b.proj, proj, add=add)
+            n += self._mix(r, proj, mix, T, f32, step) + 3
+            self._mm(mix, b.out, x, into=mult)
+            if act is not None:
+                self._dyt(x, b.norm2, **hk)
+                self._mm(h, b.up, act, act=b.spec.act)
+                self._mm(act, b.down, x, into=mult)
+                n += 3
+        self._tail = None
+        return n
+
+    def _dyt(self, x, norm: _Norm, emb=None, **kw):
+        ops.norm_dyt(x, norm.alpha, norm.w, norm.b, ids=self.ids, emb=emb, **kw)
+
     def _head(self, rows: torch.Tensor, nb: int, greedy: bool = True):
         eps = self.cfg.norm_eps
         gy, self._tail = self._tail, None
         f32 = self.exact or nb <= min(MATVEC_MAX_TOKENS, self.matvec_rows) or self.V % 4 != 0
-        y = self.y[:nb] if gy is not None else None
         h = (self.hf if f32 else self.hb)[: nb * self.dp].view(nb, self.dp)
-        ops.norm_residual(rows, eps, y=y, gy=gy, gh=self.final_norm, **(dict(hf=h) if f32 else dict(hb=h)))
+        hk = dict(hf=h) if f32 else dict(hb=h)
+        if self.cfg.norm == "dyt":
+            self._dyt(rows, self.final_norm, **hk)
+        else:
+            ops.norm_residual(rows, eps, y=self.y[:nb] if gy is not None else None, gy=gy, gh=self.final_norm.w, **hk)
         w = _Lin(self.head.w[: self.V])
         out = self.logits[:nb]
         step = max(1, self.matvec_rows) if f32 and not self.exact else nb

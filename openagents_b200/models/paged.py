@@ -315,6 +315,13 @@ class PagedEngine:
             torch.cuda.synchronize()
             self.state_slot.copy_(saved)
 
+    def _batch_order(self, q_len: list[int]) -> list[int] | None:
+        """The order a step's entries are laid out in (None: as given), for models whose kernels want some of them next to one another."""
+        return None
+
+    def _plan_batch(self, q_len: list[int], ctx: list[int]):
+        """Called ahead of every step that is not a decode step, with the new tokens and the context of each entry as laid out."""
+
     # ------------------------------------------------------------------ public operations
     def _caches(self):
         """Every per-page tensor of the model (first axis: page)."""
@@ -352,6 +359,9 @@ class PagedEngine:
         continuation needs; T is then limited by the logits workspace (``max_batch`` rows).  ``positions[b]``: the places among
         sequence b's new tokens whose logits are wanted, in any number (the result is then a tensor of its own, in that order)."""
         B = len(seq_ids)
+        order = self._batch_order([len(t) for t in new_tokens])
+        if order is not None:
+            seq_ids, new_tokens = [seq_ids[i] for i in order], [new_tokens[i] for i in order]
         staged = self._stage_batch(seq_ids, new_tokens)
         ids, pos, slot, q_start, q_len, ctx, table = staged
         T = len(ids)
@@ -362,7 +372,14 @@ class PagedEngine:
         self._embed(T)
         decode = all(n == 1 for n in q_len)
         pages = max((c + PAGE - 1) // PAGE for c in ctx)
+        if not decode or positions is not None:
+            self._plan_batch(q_len, ctx)
         self._run_layers(T, decode and positions is None, B, max(q_len), pages)
+        if order is not None:                         # from here on in the caller's order again
+            back = sorted(range(B), key=order.__getitem__)
+            q_start, q_len = [q_start[i] for i in back], [q_len[i] for i in back]
+            if all_positions:
+                positions = [range(n) for n in q_len]
         if positions is not None:
             at = [s + i for s, want in zip(q_start, positions) for i in want]
             parts = []

@@ -70,26 +70,48 @@ def tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
 def hybrid_tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
     """Hybrid stacks go by their checkpoints' own tensor names.  Norms stored around zero are of kind "bias" (initialised to 0)."""
     d = cfg.d_model
+
+    def norm(name):
+        if cfg.norm == "dyt":
+            return [TensorSpec(name, (d,), "norm"), TensorSpec(name + ".b", (d,), "bias"), TensorSpec(name + ".alpha", (1,), "norm")]
+        return [TensorSpec(name, (d,), "bias")]
     s = [TensorSpec("embed", (cfg.vocab, d), "embed")]
     for i, l in enumerate(cfg.layers):
         p, m = f"l{i}.", l.mixer
-        s += [TensorSpec(p + n, (d,), "bias") for n in (("norm1", "norm1b", "norm2", "norm2b") if l.ffn else ("norm1", "norm1b"))]
+        for n in ("norm1", "norm2") if l.ffn else ("norm1",):
+            s += norm(p + n) + (norm(p + n + "b") if cfg.post_norm else [])
         p += "mix."
-        s.append(TensorSpec(p + "q", (m.heads * m.dim, d), "matrix"))
+        if m.kind == "latent":
+            qk = m.dim + m.rot_dim
+            s += [TensorSpec(p + "dq", (m.q_rank, d), "matrix"), TensorSpec(p + "dq.norm", (m.q_rank,), "norm"),
+                  TensorSpec(p + "uq", (m.heads * qk, m.q_rank), "matrix"), TensorSpec(p + "dkv", (m.kv_rank + m.rot_dim, d), "matrix"),
+                  TensorSpec(p + "dkv.norm", (m.kv_rank,), "norm"), TensorSpec(p + "uk", (m.heads * m.dim, m.kv_rank), "matrix"),
+                  TensorSpec(p + "uv", (m.heads * m.vdim, m.kv_rank), "matrix")]
+            if m.sink:
+                s.append(TensorSpec(p + "sink", (m.heads,), "bias"))
+            if m.out_gate:
+                s.append(TensorSpec(p + "g", (m.heads * m.vdim, d), "matrix"))
+        else:
+            s.append(TensorSpec(p + "q", (m.maps * m.heads * m.dim, d), "matrix"))
         if m.kind == "gla":
             s += [TensorSpec(p + "k", (m.heads * m.dim, d), "matrix"), TensorSpec(p + "v", (m.heads * m.vdim, d), "matrix"),
                   TensorSpec(p + "g", (m.heads * m.vdim, d), "matrix"), TensorSpec(p + "norm", (m.vdim,), "norm"),
                   TensorSpec(p + "a1", (m.rank, d), "matrix"), TensorSpec(p + "a2", (m.heads * m.dim, m.rank), "matrix"),
                   TensorSpec(p + "a2.b", (m.heads * m.dim,), "bias")]
-        else:
+        elif m.kind == "attention":
+            if m.bias:
+                s.append(TensorSpec(p + "q.b", (m.maps * m.heads * m.dim,), "bias"))
             if m.kv_from is None:
-                s += [TensorSpec(p + "k", (m.kv_heads * m.dim, d), "matrix"), TensorSpec(p + "v", (m.kv_heads * m.vdim, d), "matrix")]
+                for n, rows in (("k", m.maps * m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)):
+                    s += [TensorSpec(p + n, (rows, d), "matrix")] + ([TensorSpec(f"{p}{n}.b", (rows,), "bias")] if m.bias else [])
             if m.head_gate:
                 s.append(TensorSpec(p + "g", (m.heads, d), "matrix"))
+            if m.maps == 2:
+                s += [TensorSpec(p + n, (m.dim,), "bias") for n in ("lq1", "lk1", "lq2", "lk2")]
         s.append(TensorSpec(p + "o", (d, m.heads * m.vdim), "matrix"))
         if l.ffn:
             s += [TensorSpec(f"l{i}.mlp.up", (l.ffn, d), "matrix"), TensorSpec(f"l{i}.mlp.down", (d, l.ffn), "matrix")]
-    return s + [TensorSpec("final.norm", (d,), "bias"), TensorSpec("head", (cfg.vocab, d), "output")]
+    return s + norm("final.norm") + [TensorSpec("head", (cfg.vocab, d), "output")]
 
 
 @dataclass(frozen=True)

@@ -14,10 +14,10 @@ import torch
 from .. import _native
 
 WT_Q4KR, WT_Q6KR, WT_Q8R, WT_BF16, WT_MXFP4R = 0, 1, 2, 3, 4
-EPI_STORE, EPI_RESID, EPI_SWIGLU_Q8, EPI_SWIGLU_F32, EPI_ALLREDUCE, EPI_RELU2 = 0, 1, 2, 3, 4, 6
+EPI_STORE, EPI_RESID, EPI_SWIGLU_Q8, EPI_SWIGLU_F32, EPI_ALLREDUCE, EPI_RELU2, EPI_GELU_ERF = 0, 1, 2, 3, 4, 6, 7
 SYM_NONE, SYM_ALLREDUCE, SYM_RSCATTER, SYM_RSCATTER_ROWS = 0, 1, 2, 3
 EMB_F32, EMB_BF16, EMB_Q8R, EMB_Q6KR = 0, 1, 2, 3
-ACT_NONE, ACT_GELU, ACT_SWIGLU_PAIR, ACT_RELU2 = 0, 1, 2, 3
+ACT_NONE, ACT_GELU, ACT_SWIGLU_PAIR, ACT_RELU2, ACT_GELU_ERF = 0, 1, 2, 3, 4
 
 _P = c_void_p
 _SIGS = {
@@ -34,15 +34,17 @@ _SIGS = {
     "b200_matvec_rope_kv": [c_int, _P, _P, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int,
                             c_int, c_float, c_float, _P],
     "b200_matvec": [c_int, _P, _P, c_int, c_int, c_int, _P, _P, _P, _P, c_int, _P, _P, _P, c_int, _P, _P, _P, _P,
-                    c_size_t, c_int, _P],
+                    c_size_t, c_int, c_float, _P],
     "b200_argmax_merge": [_P, _P, c_int, _P, c_size_t, c_int, _P],
-    "b200_attn_decode": [_P, _P, _P, _P, c_int, c_int, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, _P,
+    "b200_attn_decode": [_P, _P, _P, _P, c_int, c_int, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, _P,
                          _P, _P, _P, _P, _P, _P],
     "b200_attn_prefill": [_P, _P, _P, _P, c_int, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P],
     "b200_attn_prefill_tc05": [_P, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P,
-                               c_int, _P, _P, _P],
+                               c_int, _P, c_int, c_int, _P, _P, _P],
+    "b200_attn_prefill_latent": [_P, _P, c_long, c_int, c_int, _P, _P, c_int, c_int, c_int, _P, c_int, _P, _P, _P] + [c_int] * 7 + [_P, _P, c_int, _P, _P, _P],
     "b200_gemm_bf16": [_P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int,
-                       _P, c_int, _P, c_size_t, c_int, c_int, c_int, c_int, c_int, _P],
+                       _P, c_int, _P, c_size_t, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P],
+    "b200_gemm_heads": [_P, _P] + [c_int] * 7 + [_P, _P, c_int, c_int, c_float, _P, c_int, c_int, _P, _P],
     "b200_moe_gemm": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, _P, _P, _P, c_size_t, _P, _P],
     "b200_moe_route_dispatch": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_size_t, c_size_t, c_size_t, c_size_t,
                                 _P, _P, _P, _P, _P],
@@ -59,9 +61,17 @@ _SIGS = {
     "b200_count_mismatch": [_P, _P, c_size_t, _P, _P],
     "b200_norm_residual": [_P, c_int, _P, _P, c_int, c_int, _P, c_float, _P, _P, c_int, c_int, _P, c_long, _P, c_long, _P],
     "b200_qkv_finish": [_P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, c_double, c_int, c_int, c_int, c_int, c_int, c_int,
-                        c_int, c_int, c_int, c_float, c_float, c_int, _P, _P, _P, _P, c_int, _P],
-    "b200_attn_exact": [_P, _P, _P, c_int, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, c_int, _P],
-    "b200_gemm_f32": [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P],
+                        c_int, c_int, c_int, c_float, c_float, c_int, _P, _P, _P, _P, c_int, c_int, c_int, _P, _P],
+    "b200_attn_exact": [_P, _P, _P, c_int, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, c_int, c_int, c_int,
+                        c_int, _P, _P],
+    "b200_gemm_f32": [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, c_int, c_int, c_int, c_int, _P],
+    "b200_norm_dyt": [_P, c_int, c_int, _P, _P, c_int, _P, _P, _P, _P, _P, c_int, _P, c_long, _P],
+    "b200_diff_combine": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_float, _P, _P, c_int, _P],
+    "b200_latent_finish": [_P] + [c_int] * 10 + [_P, _P, c_float, _P, _P, _P, c_int, c_double, _P, _P, c_int, c_int, c_int, _P, c_int, _P],
+    "b200_latent_q": [_P] + [c_int] * 12 + [_P, _P, c_int, c_double, c_float, _P, _P, _P],
+    "b200_latent_gather": [_P, c_int, c_int, _P, c_int, _P, _P, c_int, c_int, _P, _P],
+    "b200_latent_decode": [_P, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, _P, _P],
+    "b200_latent_decode_ok": [c_int, c_int, c_int],
     "b200_logits_finish": [_P, c_size_t, c_float, c_float, _P],
     "b200_gla_chunked": [_P] + [c_int] * 7 + [_P] * 8 + [c_int] * 5 + [c_float] * 3 + [_P, _P, c_int, c_int, c_int, _P, c_size_t, _P],
     "b200_gla_recurrent": [_P] + [c_int] * 7 + [_P] * 8 + [c_int] * 5 + [c_float] * 3 + [_P, _P, c_int, _P],
@@ -82,6 +92,8 @@ def lib():
             fn.restype = c_int
         L.b200_attn_decode_scratch_floats.argtypes = [c_int, c_int, c_int, c_int, c_int]
         L.b200_attn_decode_scratch_floats.restype = c_size_t
+        L.b200_latent_decode_scratch_floats.argtypes = [c_int] * 4
+        L.b200_latent_decode_scratch_floats.restype = c_size_t
         L.b200_gla_chunk_bytes.argtypes = [c_int] * 6
         L.b200_gla_chunk_bytes.restype = c_size_t
         _lib = L
@@ -189,11 +201,11 @@ def sample_topk(logits, temperature, top_k, top_p, u, out_id, scratch):
 
 
 def matvec(wt, w, w2, N, K, nb, xq=None, xd=None, xs16=None, xf=None, epi=EPI_STORE, bias=None, resid=None, y=None,
-           ldy=0, oq=None, od=None, os16=None, sym=None, sym_off=0, wait_ready=False):
-    """Quantized mat-vec for 1..8 tokens (see ``matvec.cu``).  The SwiGLU epilogues read ``w`` as 2N rows interleaved
+           ldy=0, oq=None, od=None, os16=None, sym=None, sym_off=0, wait_ready=False, alpha=1.0):
+    """Quantized mat-vec for 1..8 tokens (see ``matvec.cu``).  ``alpha`` multiplies what EPI_RESID adds.  The SwiGLU epilogues read ``w`` as 2N rows interleaved
     (gate_0, up_0, gate_1, ...)."""
     _check(lib().b200_matvec(wt, _p(w), _p(w2), N, K, nb, _p(xq), _p(xd), _p(xs16), _p(xf), epi, _p(bias), _p(resid),
-                             _p(y), ldy, _p(oq), _p(od), _p(os16), _sym(sym), sym_off, int(wait_ready), _st()), "matvec")
+                             _p(y), ldy, _p(oq), _p(od), _p(os16), _sym(sym), sym_off, int(wait_ready), alpha, _st()), "matvec")
 
 
 def matvec_rope_kv(w, nb, pos, slot, q_out, kc, vc, Hq, Hkv, hd, page_size, theta, q_scale, xq=None, xd=None, xs16=None, xf=None,
@@ -216,11 +228,11 @@ def attn_decode_scratch_floats(B, Hq, Hkv, hd, S):
 
 
 def attn_decode(q, kc, vc, page_table, seq_lens, B, Hq, Hkv, hd, window=0, S=1, sinks=None, out_f32=None, out_bf16=None,
-                oq=None, od=None, os16=None, scratch=None, counters=None, status=None, dv=None, gate=None):
-    """``hd`` / ``dv``: query-key and value head sizes (``dv`` defaults to ``hd``); ``gate``: fp32 [B, >= Hq] view whose sigmoid scales
+                oq=None, od=None, os16=None, scratch=None, counters=None, status=None, dv=None, gate=None, chunk=0):
+    """``chunk`` > 0: keys of the token's own chunk of that many positions only.  ``hd`` / ``dv``: query-key and value head sizes (``dv`` defaults to ``hd``); ``gate``: fp32 [B, >= Hq] view whose sigmoid scales
     each head's output."""
     _check(lib().b200_attn_decode(_p(q), _p(kc), _p(vc), _p(page_table), page_table.shape[1], kc.shape[0], _p(seq_lens), _p(sinks),
-                                  B, Hq, Hkv, hd, hd if dv is None else dv, window, S, _p(gate), 0 if gate is None else gate.stride(0),
+                                  B, Hq, Hkv, hd, hd if dv is None else dv, window, chunk, S, _p(gate), 0 if gate is None else gate.stride(0),
                                   _p(out_f32), _p(out_bf16), _p(oq), _p(od), _p(os16),
                                   _p(scratch), _p(counters), _p(status), _st()), "attn_decode")
 
@@ -233,25 +245,46 @@ def attn_prefill(q, kc, vc, page_table, max_pages, q_start, q_len, ctx_len, n_se
 
 
 def attn_prefill_tc05(q16, kc, vc, page_table, q_start, q_len, ctx_len, n_seqs, max_q_len, Hq, Hkv, window=0, sinks=None,
-                      out_bf16=None, status=None, dk=128, dv=128, gate=None):
-    """Prefill attention on tcgen05 (fp16 q / cache, bf16 out; ``dk`` 64..256 and ``dv`` 64 or 128, multiples of 64); ``gate``: fp32
+                      out_bf16=None, status=None, dk=128, dv=128, gate=None, chunk=0, maps=1, out_f32=None):
+    """``chunk`` > 0: keys of the query's own chunk only; ``maps`` 2: see :func:`qkv_finish`; ``out_f32`` instead of ``out_bf16``.  Prefill attention on tcgen05 (fp16 q / cache, bf16 out; ``dk`` 64..256 and ``dv`` 64 or 128, multiples of 64); ``gate``: fp32
     [T, >= Hq] view whose sigmoid scales each head's output.  See ``attn_prefill_tc05.cu``."""
     _check(lib().b200_attn_prefill_tc05(_p(q16), _p(kc), _p(vc), _p(page_table), page_table.shape[1], kc.shape[0], _p(q_start),
                                         _p(q_len), _p(ctx_len), n_seqs, max_q_len, q16.shape[0], Hq, Hkv, dk, dv, window, _p(sinks),
-                                        _p(gate), 0 if gate is None else gate.stride(0), _p(out_bf16), _p(status), _st()), "attn_prefill_tc05")
+                                        _p(gate), 0 if gate is None else gate.stride(0), _p(out_bf16), chunk, maps, _p(out_f32), _p(status),
+                                        _st()), "attn_prefill_tc05")
+
+
+def attn_prefill_latent(q16, ws, v_col, base, cache, r_col, page_table, q_start, q_len, ctx_len, n_seqs, max_q, H, kn, rr, dv, out_bf16, sinks=None,
+                        gate=None, status=None):
+    """:func:`attn_prefill_tc05` over an expanded context: ``ws`` fp16 [rows, >= H * (kn + dv)] (own key parts, then values from ``v_col`` on; sequence b from
+    row ``base[b]`` on), the shared key part in the columns from ``r_col`` of the paged latent ``cache`` [pages, 16, ks]; ``gate``: fp32 [T, >= H * dv]."""
+    _check(lib().b200_attn_prefill_latent(_p(q16), _p(ws), ws.shape[0], ws.stride(0), v_col, _p(base), _p(cache), cache.shape[0], cache.shape[-1], r_col,
+                                          _p(page_table), page_table.shape[1], _p(q_start), _p(q_len), _p(ctx_len), n_seqs, max_q, q16.shape[0], H, kn, rr, dv,
+                                          _p(sinks), _p(gate), 0 if gate is None else gate.stride(0), _p(out_bf16), _p(status), _st()), "attn_prefill_latent")
 
 
 def gemm_bf16(A, B, M, N, K, lda=None, ldb=None, out_f32=None, out_bf16=None, ldc=None, bias=None, resid_f32=None,
               resid_bf16=None, act=ACT_NONE, accumulate=False, tile_n=0, status=None, sym_mode=SYM_NONE, sym=None,
-              sym_off=0, rows_per_rank=0, split_k=0, wait_ready=False, ag_rows_per_rank=0, ag_epoch=0, mn_major=False):
-    """D[M][N] = A[M][K] @ B[N][K]^T with fused epilogue (see ``gemm_tc05.cu``).  ``ag_rows_per_rank`` > 0: the rows
+              sym_off=0, rows_per_rank=0, split_k=0, wait_ready=False, ag_rows_per_rank=0, ag_epoch=0, mn_major=False, alpha=1.0,
+              out_f16=None):
+    """``alpha`` multiplies the product; ``out_f16`` instead of ``out_bf16``: stored as fp16.  D[M][N] = A[M][K] @ B[N][K]^T with fused epilogue (see ``gemm_tc05.cu``).  ``ag_rows_per_rank`` > 0: the rows
     of A are all-gathered by push (``rmsnorm_allgather``) and each tile waits for its owners' counter to reach ``ag_epoch``.
     ``mn_major``: the operands are given as A [K][M] and B [K][N] (row strides ``lda`` / ``ldb``), i.e. D = A^T B: the weight
     gradient dW = dy^T x straight from dy and x, without transposed copies."""
-    _check(lib().b200_gemm_bf16(_p(A), _p(B), M, N, K, lda or (M if mn_major else K), ldb or (N if mn_major else K), _p(out_f32), _p(out_bf16), ldc or N,
+    _check(lib().b200_gemm_bf16(_p(A), _p(B), M, N, K, lda or (M if mn_major else K), ldb or (N if mn_major else K), _p(out_f32),
+                                _p(out_bf16 if out_f16 is None else out_f16), ldc or N,
                                 _p(bias), _p(resid_f32), _p(resid_bf16), act, int(accumulate), tile_n, split_k, _p(status),
                                 sym_mode, _sym(sym), sym_off, rows_per_rank, int(wait_ready), ag_rows_per_rank, ag_epoch,
-                                int(mn_major), _st()), "gemm_bf16")
+                                int(mn_major), alpha, int(out_f16 is not None), _st()), "gemm_bf16")
+
+
+def gemm_heads(A, B, heads, N, K, head_k, out, head_ldc, alpha=1.0, gate=None, status=None):
+    """One product per head on the tensor cores: ``out[:, z * head_ldc + n] = alpha * A[:, z * head_k: + K] @ B[z * N + n]`` (bf16 operands; fp32, bf16 or
+    fp16 ``out``), times the sigmoid of ``gate`` (fp32, a column per output column)."""
+    f32 = out.dtype == torch.float32
+    _check(lib().b200_gemm_heads(_p(A), _p(B), A.shape[0], heads, N, K, A.stride(0), head_k, B.stride(0), _p(out) if f32 else None, None if f32 else _p(out),
+                                 out.stride(0), head_ldc, alpha, _p(gate), 0 if gate is None else gate.stride(0), int(out.dtype == torch.float16),
+                                 _p(status), _st()), "gemm_heads")
 
 
 def set_pdl(on: bool):
@@ -349,27 +382,88 @@ def norm_residual(x, eps, y=None, gy=None, gh=None, hb=None, hf=None, y_clear=Fa
 
 
 def qkv_finish(proj, q_off, k_off, v_off, pos, slot, table, base, H, G, dim, vdim, DK, DV, rot, style, qk_norm, eps, q_scale, page_size,
-               q32=None, q16=None, kc=None, vc=None):
-    """Rotation, unit-RMS norm and scale of the queries and keys of a fused projection row, and the paged-cache write of keys and
+               q32=None, q16=None, kc=None, vc=None, maps=1, q_wide=False, bias=None):
+    """``bias`` is added to the projection row; ``maps`` 2 (differential attention): ``H`` counts the query rows of both maps, ordered (key/value head, map,
+    head of the group), a cache row holds both maps' keys side by side, and ``q_wide`` pads a query with zeros on the other map's half.  Rotation, unit-RMS norm and scale of the queries and keys of a fused projection row, and the paged-cache write of keys and
     values (``k_off`` < 0: the layer has none); see ``hybrid_ops.cu``."""
     f32 = int(kc is not None and kc.dtype == torch.float32)
     _check(lib().b200_qkv_finish(_p(proj), proj.stride(0), proj.shape[0], q_off, k_off, v_off, _p(pos), _p(slot), _p(table),
                                  0 if table is None else table.shape[0], base, H, G, dim, vdim, DK, DV, rot, style, int(qk_norm), eps,
-                                 q_scale, page_size, _p(q32), _p(q16), _p(kc), _p(vc), f32, _st()), "qkv_finish")
+                                 q_scale, page_size, _p(q32), _p(q16), _p(kc), _p(vc), f32, maps, int(q_wide), _p(bias), _st()), "qkv_finish")
 
 
-def attn_exact(q32, kc, vc, page_table, q_start, q_len, ctx_len, n_seqs, max_q, H, G, DK, DV, gate=None, out_f32=None, out_bf16=None):
-    """Causal attention in 32-bit arithmetic for any head sizes; ``gate``: fp32 [T, >= H] view whose sigmoid scales each head."""
+def attn_exact(q32, kc, vc, page_table, q_start, q_len, ctx_len, n_seqs, max_q, H, G, DK, DV, gate=None, out_f32=None, out_bf16=None, maps=1,
+               chunk=0, sinks=None):
+    """Causal attention in 32-bit arithmetic for any head sizes; ``gate``: fp32 [T, >= H] view whose sigmoid scales each head; ``maps``: see
+    :func:`qkv_finish`; ``vc`` None: the values are the first DV columns of the keys (latent attention)."""
     o = out_f32 if out_f32 is not None else out_bf16
     _check(lib().b200_attn_exact(_p(q32), _p(kc), _p(vc), int(kc.dtype == torch.float32), _p(page_table), page_table.shape[1], _p(q_start),
                                  _p(q_len), _p(ctx_len), n_seqs, max_q, H, G, DK, DV, _p(gate), 0 if gate is None else gate.stride(0),
-                                 _p(out_f32), _p(out_bf16), o.stride(0), _st()), "attn_exact")
+                                 _p(out_f32), _p(out_bf16), o.stride(0), kc.shape[-1], maps, chunk, _p(sinks), _st()), "attn_exact")
 
 
-def gemm_f32(A, W, out, act=0):
-    """``out = act(A @ W^T)`` in true 32-bit: A fp32 [M, K], W bf16 [N, K]; ``act`` 1: the square of relu."""
+def gemm_f32(A, W, out, act=0, alpha=1.0, accumulate=False, gate=None, heads=1, head_k=0, head_ldc=0):
+    """``out = act(alpha * A @ W^T)`` in true 32-bit: A fp32 [M, K], W bf16 [N, K]; ``act`` 1: the square of relu, 2: the erf gelu; times the sigmoid of ``gate``
+    [M, N]; ``accumulate`` adds into ``out``.  ``heads`` > 1: one product per head, as in :func:`gemm_heads`."""
     M, (N, K) = A.shape[0], W.shape
-    _check(lib().b200_gemm_f32(_p(A), A.stride(0), _p(W), W.stride(0), _p(out), out.stride(0), M, N, K, act, _st()), "gemm_f32")
+    _check(lib().b200_gemm_f32(_p(A), A.stride(0), _p(W), W.stride(0), _p(out), out.stride(0), M, N // heads, K, act, alpha, int(accumulate), _p(gate),
+                               0 if gate is None else gate.stride(0), heads, head_k, head_ldc, _st()), "gemm_f32")
+
+
+def norm_dyt(x, alpha, w, b, hb=None, hf=None, ids=None, emb=None, zero=None):
+    """``h = tanh(alpha * x) * w + b`` (Dynamic Tanh) into ``hb`` (bf16) and/or ``hf`` (fp32), padding columns zero; with ``emb`` (bf16 [vocab, D]) the
+    tokens' rows of it are added to ``x`` first; ``zero``: a contiguous fp32 tensor cleared on the side."""
+    T, D = x.shape
+    h = hb if hb is not None else hf
+    _check(lib().b200_norm_dyt(_p(x), T, D, _p(ids), _p(emb), 0 if emb is None else emb.shape[0], _p(alpha), _p(w), _p(b), _p(hb), _p(hf), h.stride(0),
+                               _p(zero), 0 if zero is None else zero.numel(), _st()), "norm_dyt")
+
+
+def diff_combine(maps_out, lam, H, G, vdim, DV, eps, mult, out_f32=None, out_bf16=None):
+    """``o = a1 - lam * a2`` over two maps' outputs (fp32 [T, 2 H DV], :func:`qkv_finish`'s order), divided by its root mean square per head, times ``mult``."""
+    o = out_f32 if out_f32 is not None else out_bf16
+    _check(lib().b200_diff_combine(_p(maps_out), _p(lam), maps_out.shape[0], H, G, vdim, DV, eps, mult, _p(out_f32), _p(out_bf16), o.stride(0), _st()),
+           "diff_combine")
+
+
+# ---------------------------------------------------------------- latent attention (see ``latent_attn.cu``)
+def latent_finish(proj, q_off, c_off, r_off, q_rank, rank, rot_dim, rot, style, q_w, c_w, eps, pos, slot, table, base, cq, cache, CR, RR):
+    """RMS norm of the two latents of a down-projection row and rotation of the shared key part: the query latent to ``cq`` (bf16 or fp32, padded), the
+    rest to the token's row of the paged ``cache`` [pages, 16, CR + RR]."""
+    f32 = cq.dtype == torch.float32
+    _check(lib().b200_latent_finish(_p(proj), proj.stride(0), proj.shape[0], q_off, c_off, r_off, q_rank, rank, rot_dim, rot, style, _p(q_w), _p(c_w), eps,
+                                    _p(pos), _p(slot), _p(table), 0 if table is None else table.shape[0], base, _p(cq) if f32 else None,
+                                    None if f32 else _p(cq), cq.stride(0), CR, RR, _p(cache), int(cache.dtype == torch.float32), _st()), "latent_finish")
+
+
+def latent_q(q, hs, H, dim, rot_dim, rot, style, NC, r_col, RR, width, pos, table, base, scale, out):
+    """Rotation and scale of the queries (fp32 [T, H * hs]) into ``out`` (fp32 or fp16 [T, H, width]): the unrotated part to columns [0, NC) (0: left alone),
+    the rotated one to [r_col, r_col + RR)."""
+    f32 = out.dtype == torch.float32
+    _check(lib().b200_latent_q(_p(q), q.stride(0), hs, q.shape[0], H, dim, rot_dim, rot, style, NC, r_col, RR, width, _p(pos), _p(table),
+                               0 if table is None else table.shape[0], base, scale, _p(out) if f32 else None, None if f32 else _p(out), _st()), "latent_q")
+
+
+def latent_gather(cache, CR, page_table, ctx_len, base, n_seqs, max_ctx, out):
+    """The cached latents (fp16) of whole contexts as rows of ``out`` (bf16 [rows, CR]), sequence b from row ``base[b]`` on."""
+    _check(lib().b200_latent_gather(_p(cache), cache.shape[-1], CR, _p(page_table), page_table.shape[1], _p(ctx_len), _p(base), n_seqs, max_ctx, _p(out),
+                                    _st()), "latent_gather")
+
+
+def latent_decode_ok(H, CR, RR):
+    return bool(lib().b200_latent_decode_ok(H, CR, RR))
+
+
+def latent_decode_scratch_floats(R, H, CR, S):
+    return lib().b200_latent_decode_scratch_floats(R, H, CR, S)
+
+
+def latent_decode(q, cache, page_table, row_seq, pos, R, H, CR, RR, S, scratch, out_f32=None, out_bf16=None, sinks=None, status=None):
+    """Attention of R query rows in the latent space: ``q`` fp32 [R, H, CR + RR] against the paged rows of ``cache``, as keys and as values; row r belongs to
+    sequence ``row_seq[r]`` (None: r) and sees positions 0..``pos[r]``.  ``S``: shares of the keys."""
+    o = out_f32 if out_f32 is not None else out_bf16
+    _check(lib().b200_latent_decode(_p(q), _p(cache), _p(page_table), page_table.shape[1], cache.shape[0], _p(row_seq), _p(pos), _p(sinks), R, H, CR, RR, S,
+                                    _p(scratch), _p(out_f32), _p(out_bf16), o.stride(0), _p(status), _st()), "latent_decode")
 
 
 def logits_finish(logits, scale, cap):

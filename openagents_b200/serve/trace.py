@@ -75,9 +75,10 @@ def parse_args(argv=None):
 def main(argv=None) -> int:
     a = parse_args(argv)
     from .. import _native
+    from ..models.config import HYBRID_ARCHS
     from ..models.registry import peek_architecture
-    if peek_architecture(a.model) == "folirax":
-        _native.use_subset("hybrid")                 # build no more than this family needs
+    if peek_architecture(a.model) in HYBRID_ARCHS:
+        _native.use_subset("hybrid")                 # build no more than these families need
     from ..models.paged import PAGE
     from .backend import CudaBackend
     pages = max(1, (a.max_tokens + PAGE - 1) // PAGE)
