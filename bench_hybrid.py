@@ -1,6 +1,6 @@
-"""Prefill and decode throughput of the hybrid (Folirax) engine at a real model's layer sizes, beside the Llama engine at equal size.
+"""Prefill and decode throughput of the hybrid engine (Folirax, Pesorax) at a real model's layer sizes, beside the Llama engine at equal size.
 
-    python bench.py --workload hybrid [--model folirax-8b-shape] [--steps K] [--warmup W]
+    python bench.py --workload hybrid [--model folirax-8b-shape | pesorax-8b-shape | ...] [--steps K] [--warmup W]
 
 Both engines hold bf16 random weights of the same width, feed-forward, head layout, depth and vocabulary, run the same prompts
 and batches, and are timed with CUDA events: a 2048-token prompt, four of them in one call, and decode steps (replayed graphs
@@ -29,10 +29,12 @@ def peaks() -> tuple[float, float, str]:
 
 
 def like_llama(cfg):
-    """The Llama shape with the hybrid's width, depth, feed-forward, attention heads and vocabulary."""
+    """The Llama shape with the hybrid's width, depth (a looped layer counts every time), feed-forward, vocabulary and attention heads (Pesorax: heads of
+    128, four to a key/value head)."""
     from openagents_b200.models.config import ModelConfig
     m = next(l.mixer for l in cfg.layers if l.mixer.kind == "attention")
-    return ModelConfig(arch="llama", n_layers=cfg.n_layers, d_model=cfg.d_model, n_heads=m.heads, n_kv_heads=m.kv_heads, head_dim=m.dim,
+    heads, kv, dim = (cfg.d_model // 128, cfg.d_model // 512, 128) if cfg.arch == "pesorax" else (m.heads, m.kv_heads, m.dim)
+    return ModelConfig(arch="llama", n_layers=len(cfg.layer_runs()), d_model=cfg.d_model, n_heads=heads, n_kv_heads=kv, head_dim=dim,
                        ffn=cfg.ffn, vocab=cfg.vocab, context=8192, rope_theta=500000.0, name="llama-" + cfg.name)
 
 
@@ -91,26 +93,18 @@ def time_engine(cfg, dev, steps: int, warmup: int) -> dict:
     return out
 
 
-def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
-    """Every kernel of one hybrid layer pair at 2048 prompt tokens and at a 64-sequence decode step, and its Llama counterpart."""
-    from openagents_b200.ops import cuda_ops as ops
-    hbm, flops, _ = peaks()
-    at = next(l.mixer for l in cfg.layers if l.mixer.kind == "attention")
-    gl = next(l.mixer for l in cfg.layers if l.mixer.kind == "gla")
-    d, F, T, B, ctx = cfg.d_model, cfg.ffn, PROMPT, 64, PROMPT
-    H, G, D = at.heads, at.kv_heads, at.dim
-    flush = torch.empty(1 << 30, dtype=torch.uint8, device=dev)
-    st = torch.zeros(1, dtype=torch.int32, device=dev)
-    rnd = lambda *s: torch.randn(*s, device=dev)                       # noqa: E731
-    bf = lambda *s: torch.randn(*s, device=dev).bfloat16()             # noqa: E731
-    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)     # noqa: E731
-    rows: list[dict] = []
+class _Timer:
+    """Median time of a launch with L2 flushed ahead of it, against the slower of its bytes and its FLOPs at the measured rates."""
 
-    def bench(name, fn, nbytes, fl=0.0, like=None):
+    def __init__(self, dev, reps: int):
+        self.hbm, self.flops, _ = peaks()
+        self.reps, self.rows, self.flush = reps, [], torch.empty(1 << 30, dtype=torch.uint8, device=dev)
+
+    def __call__(self, name, fn, nbytes, fl=0.0, like=None):
         ms = []
-        for i in range(reps + 3):
+        for i in range(self.reps + 3):
             torch.cuda.synchronize()
-            flush.zero_()
+            self.flush.zero_()
             a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             a.record()                             # queued behind the flush: the launch itself is not in the time
             fn()
@@ -119,9 +113,134 @@ def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
             if i >= 3:
                 ms.append(a.elapsed_time(b))
         ms.sort()
-        us, roof = ms[len(ms) // 2] * 1e3, max(nbytes / hbm, fl / flops) * 1e6
-        rows.append({"kernel": name, "us": round(us, 1), "roofline_us": round(roof, 1), "of_roofline": round(roof / us, 3), "like": like})
+        us, roof = ms[len(ms) // 2] * 1e3, max(nbytes / self.hbm, fl / self.flops) * 1e6
+        self.rows.append({"kernel": name, "us": round(us, 1), "roofline_us": round(roof, 1), "of_roofline": round(roof / us, 3), "like": like})
 
+
+def time_pesorax_kernels(cfg, dev, reps: int = 12) -> list[dict]:
+    """Every kernel of a differential and a latent layer at 2048 prompt tokens and at decode steps, and its Llama counterpart.  Cached rows are read once, FLOPs
+    are those of the visible keys; attention's reading of keys and values counts once per key/value head."""
+    from openagents_b200.ops import cuda_ops as ops
+    bench = _Timer(dev, reps)
+    df, lt = (next(l.mixer for l in cfg.layers if l.mixer.kind == k) for k in ("attention", "latent"))
+    ref = like_llama(cfg)
+    d, F, T, B, ctx = cfg.d_model, cfg.ffn, PROMPT, 64, PROMPT
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    rnd = lambda *s: torch.randn(*s, device=dev)                       # noqa: E731
+    bf = lambda *s: torch.randn(*s, device=dev).bfloat16()             # noqa: E731
+    hf = lambda *s: torch.randn(*s, device=dev).half()                 # noqa: E731
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)     # noqa: E731
+    pages = (ctx + 15) // 16
+    table = lambda s: i32(list(range(s * pages))).view(s, pages)       # noqa: E731
+    splits = lambda s, g: max(1, min(64, max(1, pages // 24), max((147 + s * g) // (s * g), (2047 + s * g) // (s * g) if s * g >= 148 else 0)))      # noqa: E731
+    H, G, D, V = df.heads, df.kv_heads, df.dim, df.vdim
+    Hq, Gq, Dq = ref.n_heads, ref.n_kv_heads, ref.head_dim
+    for n in (T, B):
+        x, hb, w, al = rnd(n, d), bf(n, d), rnd(d), torch.ones(1, device=dev)
+        bench(f"norm_dyt [{n}]", lambda: ops.norm_dyt(x, al, w, w, hb=hb), n * d * 6, like=f"rmsnorm [{n}]")
+        bench(f"rmsnorm [{n}]", lambda: ops.rmsnorm(x, w, 1e-6, hb=hb), n * d * 6)
+    # ---- differential attention
+    nq, nk, nv = 2 * H * D, 2 * G * D, G * V
+    for n, seqs in ((T, 1), (B, B), (1, 1)):
+        prompt = n == T
+        row, bias, lam = rnd(n, nq + nk + nv), rnd(nq + nk + nv), torch.ones(1, device=dev)
+        pos, slot = i32([ctx - 1] * n if not prompt else list(range(n))), i32(list(range(n)))
+        kc, vc = hf(seqs * pages + 1, G, 16, 2 * D), hf(seqs * pages + 1, G, 16, V)
+        q16, q32 = hf(n, nq), rnd(n, 2 * nq)
+        q = dict(q16=q16) if prompt else dict(q32=q32, q_wide=True)
+        bench(f"qkv_finish two maps [{n}]", lambda: ops.qkv_finish(row, 0, nq, nq + nk, pos, slot, None, 1.0, 2 * H, G, D, V, D, V, 0, 1, False, 1e-6, df.scale, 16, kc=kc,
+                                                                   vc=vc, maps=2, bias=bias, **q), n * ((nq + nk + nv) * 4 + nq * (2 if prompt else 8) + (nk + nv) * 2),
+              like=f"rope_kv [{n}]")
+        ld = (Hq + 2 * Gq) * Dq
+        row2, tabf, kl, vl = rnd(n, ld), ops.rope_table(ctx, Dq, 500000.0, dev), hf(seqs * pages + 1, Gq, 16, Dq), hf(seqs * pages + 1, Gq, 16, Dq)
+        l16, l32 = hf(n, Hq * Dq), rnd(n, Hq * Dq)
+        bench(f"rope_kv [{n}]", lambda: ops.rope_kv(row2, pos, slot, None if prompt else l32, l16 if prompt else None, kl, vl, Hq, Gq, Dq, 16, 500000.0, 0, 0.1, table=tabf),
+              n * (ld * 4 + Hq * Dq * (2 if prompt else 4) + 2 * Gq * Dq * 2))
+        lens, tb, mo, o = i32([ctx] * seqs), table(seqs), rnd(n, 2 * H * V), bf(n, H * V)
+        if prompt:
+            z = i32([0])
+            bench(f"attn_prefill_tc05 two maps [{T}]", lambda: ops.attn_prefill_tc05(q16, kc, vc, tb, z, lens, lens, 1, T, 2 * H, G, out_f32=mo, status=st, dk=D, dv=V,
+                                                                                    chunk=df.chunk, maps=2), T * (nq * 2 + (nk + nv) * 2 + 2 * H * V * 4),
+                  2.0 * min(T, df.chunk) * T / 2 * 2 * H * (D + V), like=f"attn_prefill_tc05 [{T}]")
+            ol = bf(T, Hq * Dq)
+            bench(f"attn_prefill_tc05 [{T}]", lambda: ops.attn_prefill_tc05(l16, kl, vl, tb, z, lens, lens, 1, T, Hq, Gq, out_bf16=ol, status=st, dk=Dq, dv=Dq),
+                  T * (Hq + Gq) * Dq * 4, 4.0 * T * T / 2 * Hq * Dq)
+        else:
+            S = splits(n, G)
+            sc, cnt = rnd(ops.attn_decode_scratch_floats(n, 2 * H, G, V, S)), torch.zeros(n * 2 * H, dtype=torch.int32, device=dev)
+            bench(f"attn_decode two maps [{n} x {ctx}]", lambda: ops.attn_decode(q32, kc, vc, tb, lens, n, 2 * H, G, 2 * D, dv=V, S=S, out_f32=mo, scratch=sc, counters=cnt,
+                                                                                status=st, chunk=df.chunk), n * min(ctx, df.chunk) * (nk + nv) * 2,
+                  like=f"attn_decode [{n} x {ctx}]")
+            ol, S2 = bf(n, Hq * Dq), splits(n, Gq)
+            sc2, cnt2 = rnd(ops.attn_decode_scratch_floats(n, Hq, Gq, Dq, S2)), torch.zeros(n * Hq, dtype=torch.int32, device=dev)
+            bench(f"attn_decode [{n} x {ctx}]", lambda: ops.attn_decode(l32, kl, vl, tb, lens, n, Hq, Gq, Dq, S=S2, out_bf16=ol, scratch=sc2, counters=cnt2, status=st),
+                  n * ctx * Gq * Dq * 4)
+        bench(f"diff_combine [{n}]", lambda: ops.diff_combine(mo, lam, H, G, V, V, 1e-6, 0.5, out_bf16=o), n * H * V * 10, like=f"rmsnorm [{n if n > 1 else B}]")
+    # ---- latent attention
+    HL, DL, RL, VL, C, Q = lt.heads, lt.dim, lt.rot_dim, lt.vdim, lt.kv_rank, lt.q_rank
+    W, hs, n_proj = C + RL, DL + RL, Q + C + RL + HL * VL
+    tab = ops.rope_table(ctx, lt.rope_dims, lt.rope_base, dev)
+    for n, seqs in ((T, 1), (B, B), (1, 1)):
+        prompt = n == T
+        row, qw, cw = rnd(n, n_proj), rnd(Q), rnd(C)
+        pos, slot = i32([ctx - 1] * n if not prompt else list(range(n))), i32(list(range(n)))
+        cache, cq, uq, uq16 = hf(seqs * pages + 1, 16, W), bf(n, Q), rnd(n, HL * hs), bf(n, HL * hs)
+        tb, lens, gate, sink = table(seqs), i32([ctx] * seqs), row[:, Q + W:], rnd(HL)
+        bench(f"latent_finish [{n}]", lambda: ops.latent_finish(row, 0, Q, Q + C, Q, C, RL, lt.rope_dims, 1, qw, cw, 1e-6, pos, slot, tab, lt.rope_base, cq, cache, C, RL),
+              n * ((Q + W) * 4 + Q * 2 + W * 2), like=f"rope_kv [{n}]")
+        o = bf(n, HL * VL)
+        if prompt:
+            q16, z, base, c, kv = hf(n, HL * hs), i32([0]), i32([0]), bf(n, C), hf(n, HL * (DL + VL))
+            bench(f"latent_q [{n}]", lambda: ops.latent_q(uq, hs, HL, DL, RL, lt.rope_dims, 1, DL, DL, RL, hs, pos, tab, lt.rope_base, 0.1, q16), n * HL * hs * 6, like=f"rope_kv [{n}]")
+            bench(f"latent_gather [{n}]", lambda: ops.latent_gather(cache, C, tb, lens, base, 1, n, c), n * C * 4, like=f"rope_kv [{n}]")
+            we = bf(HL * (DL + VL), C)
+            bench(f"gemm expand [{n} x {HL * (DL + VL)} x {C}]", lambda: ops.gemm_bf16(c, we, n, HL * (DL + VL), C, out_f16=kv, status=st), n * (C + HL * (DL + VL)) * 2 + we.numel() * 2,
+                  2.0 * n * C * HL * (DL + VL), like=f"gemm qkv [{n}]")
+            bench(f"attn_prefill_latent [{n}]", lambda: ops.attn_prefill_latent(q16, kv, HL * DL, base, cache, C, tb, z, lens, lens, 1, n, HL, DL, RL, VL, o, sinks=sink, gate=gate,
+                                                                               status=st), n * HL * (hs + DL + VL + VL) * 2 + n * HL * VL * 4, 2.0 * n * n / 2 * HL * (hs + VL),
+                  like=f"attn_prefill_tc05 [{T}]")
+        else:
+            ql, ol = rnd(n, HL * W), bf(n, HL * C)
+            wa, wv = bf(HL * C, DL), bf(HL * VL, C)
+            if n > 1:
+                bench(f"gemm_heads absorb [{n}]", lambda: ops.gemm_heads(uq16, wa, HL, C, DL, hs, ql, W, alpha=0.1, status=st), wa.numel() * 2 + n * HL * (DL * 2 + C * 4),
+                      2.0 * n * wa.numel(), like=f"gemm qkv [{n}]")
+                bench(f"gemm_heads value [{n}]", lambda: ops.gemm_heads(ol, wv, HL, VL, C, C, o, VL, gate=gate, status=st), wv.numel() * 2 + n * HL * (C * 2 + VL * 6),
+                      2.0 * n * wv.numel(), like=f"gemm qkv [{n}]")
+            bench(f"latent_q [{n}]", lambda: ops.latent_q(uq, hs, HL, DL, RL, lt.rope_dims, 1, 0, C, RL, W, pos, tab, lt.rope_base, 0.1, ql), n * HL * RL * 8, like=f"rope_kv [{n}]")
+            ctas, blocks = n * ((HL + 31) // 32), ctx // 64
+            S = min(range(1, min(64, blocks, max(1, 592 // ctas)) + 1), key=lambda s: -(-ctas * s // 148) * (-(-blocks // s) + 2))
+            sc = rnd(max(1, ops.latent_decode_scratch_floats(n, HL, C, S)))
+            bench(f"latent_decode [{n} x {ctx}] ({S} shares)", lambda: ops.latent_decode(ql, cache, tb, None, pos, n, HL, C, RL, S, sc, out_bf16=ol, sinks=sink, status=st),
+                  n * (ctx * W * 2 + HL * (W * 4 + C * 2)), 2.0 * n * ctx * HL * (W + C), like=f"attn_decode [{n} x {ctx}]")
+    # ---- products
+    for n in (T, B):
+        a, up, dn, gu, x, act = bf(n, d), bf(F, d), bf(d, F), bf(2 * F, d), rnd(n, d), bf(n, F)
+        bench(f"gemm gelu up [{n} x {F} x {d}]", lambda: ops.gemm_bf16(a, up, n, F, d, out_bf16=act, act=ops.ACT_GELU_ERF, status=st), (F * d + n * (d + F)) * 2, 2.0 * n * F * d,
+              like=f"gemm swiglu gate/up [{n}]")
+        bench(f"gemm swiglu gate/up [{n}]", lambda: ops.gemm_bf16(a, gu, n, 2 * F, d, out_bf16=act, ldc=F, act=ops.ACT_SWIGLU_PAIR, status=st), (2 * F * d + n * (d + F)) * 2, 4.0 * n * F * d)
+        bench(f"gemm down, scaled residual [{n}]", lambda: ops.gemm_bf16(act, dn, n, d, F, out_f32=x, accumulate=True, alpha=0.5, status=st), (F * d + n * F) * 2 + n * d * 8,
+              2.0 * n * F * d, like=f"gemm down, residual [{n}]")
+        bench(f"gemm down, residual [{n}]", lambda: ops.gemm_bf16(act, dn, n, d, F, out_f32=x, resid_f32=x, status=st), (F * d + n * F) * 2 + n * d * 8, 2.0 * n * F * d)
+        for nm, N, K in (("gemm differential qkv", nq + nk + nv, d), ("gemm latent down", n_proj, d), ("gemm latent queries", HL * hs, Q), ("gemm qkv", (Hq + 2 * Gq) * Dq, d)):
+            wt, ai, o3 = bf(N, K), bf(n, K), torch.zeros(n, N, device=dev)
+            bench(f"{nm} [{n}]", lambda: ops.gemm_bf16(ai, wt, n, N, K, out_f32=o3, accumulate=n <= 64 and K == d, status=st), N * K * 2 + n * (K * 2 + N * 4), 2.0 * n * N * K,
+                  like=None if nm == "gemm qkv" else f"gemm qkv [{n}]")
+    return bench.rows
+
+
+def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
+    """Every kernel of one hybrid layer pair at 2048 prompt tokens and at a 64-sequence decode step, and its Llama counterpart."""
+    from openagents_b200.ops import cuda_ops as ops
+    bench = _Timer(dev, reps)
+    at = next(l.mixer for l in cfg.layers if l.mixer.kind == "attention")
+    gl = next(l.mixer for l in cfg.layers if l.mixer.kind == "gla")
+    d, F, T, B, ctx = cfg.d_model, cfg.ffn, PROMPT, 64, PROMPT
+    H, G, D = at.heads, at.kv_heads, at.dim
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    rnd = lambda *s: torch.randn(*s, device=dev)                       # noqa: E731
+    bf = lambda *s: torch.randn(*s, device=dev).bfloat16()             # noqa: E731
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)     # noqa: E731
     # ---- norms and residual
     for n in (T, B):
         x, y, hb, gn = rnd(n, d), rnd(n, d), bf(n, d), rnd(d)
@@ -188,7 +307,7 @@ def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
             bench(f"{nm} [{n} x {N} x {d}]", lambda: ops.gemm_bf16(a, wt, n, N, d, out_f32=o3, accumulate=n <= 64, status=st), N * d * 2 + n * (d * 2 + N * 4), 2.0 * n * N * d)
     lg = rnd(B, cfg.vocab)
     bench(f"logits_finish [{B} x {cfg.vocab}]", lambda: ops.logits_finish(lg, 0.5, 30.0), 8 * B * cfg.vocab)
-    return rows
+    return bench.rows
 
 
 def run(args) -> dict:
@@ -198,4 +317,4 @@ def run(args) -> dict:
     cfg = PRESETS[args.model]
     ours, llama = time_engine(cfg, dev, args.steps, max(3, args.warmup)), time_engine(like_llama(cfg), dev, args.steps, max(3, args.warmup))
     return {"workload": "hybrid", "model": cfg.name, "dtype": "bf16", "data": "synthetic", "prompt": PROMPT, "peaks": peaks()[2], "hybrid": ours,
-            "llama_equal_size": llama, "kernels": time_kernels(cfg, dev)}
+            "llama_equal_size": llama, "kernels": (time_pesorax_kernels if cfg.arch == "pesorax" else time_kernels)(cfg, dev)}

@@ -119,6 +119,25 @@ class _Plan:
     groups: list = field(default_factory=list)
 
 
+def plan_latent_batch(q_len: list[int], ctx: list[int], short_rows: int, ctx_rows: int) -> tuple[_Plan, list[int], list[int]]:
+    """Layout of a step whose entries (new tokens, context) come shortest first: the plan, the entry of each short token's row, and every other entry's first
+    row in its group's workspace of ``ctx_rows``."""
+    p = _Plan()
+    for n, c in zip(q_len, ctx):
+        if n > SHORT_TOKENS or p.t_short + n > short_rows:
+            break
+        p.n_short, p.t_short, p.short_pages = p.n_short + 1, p.t_short + n, max(p.short_pages, (c + PAGE - 1) // PAGE)
+    rows = [b for b in range(p.n_short) for _ in range(q_len[b])]
+    base = [0] * len(q_len)
+    for b in range(p.n_short, len(q_len)):
+        if not p.groups or p.groups[-1][4] + ctx[b] > ctx_rows:
+            p.groups.append([b, b, 0, 0, 0])
+        g = p.groups[-1]
+        base[b] = g[4]
+        p.groups[-1] = [g[0], b + 1, max(g[2], q_len[b]), max(g[3], ctx[b]), g[4] + ctx[b]]
+    return p, rows, base
+
+
 class HybridEngine(PagedEngine):
     ARCHS = ("folirax", "pesorax")
     world = 1                    # one GPU; the serving layer asks
@@ -376,19 +395,7 @@ class HybridEngine(PagedEngine):
     def _plan_batch(self, q_len, ctx):
         if not self.ctx_rows:
             return
-        p = self._plan = _Plan()
-        for n, c in zip(q_len, ctx):                     # shortest first
-            if n > SHORT_TOKENS or p.t_short + n > self.short_rows:
-                break
-            p.n_short, p.t_short, p.short_pages = p.n_short + 1, p.t_short + n, max(p.short_pages, (c + PAGE - 1) // PAGE)
-        rows = [b for b in range(p.n_short) for _ in range(q_len[b])]
-        base = [0] * len(q_len)
-        for b in range(p.n_short, len(q_len)):
-            if not p.groups or p.groups[-1][4] + ctx[b] > self.ctx_rows:
-                p.groups.append([b, b, 0, 0, 0])
-            g = p.groups[-1]
-            base[b] = g[4]
-            p.groups[-1] = [g[0], b + 1, max(g[2], q_len[b]), max(g[3], ctx[b]), g[4] + ctx[b]]
+        self._plan, rows, base = plan_latent_batch(q_len, ctx, self.short_rows, self.ctx_rows)
         if rows:
             self.row_seq[: len(rows)].copy_(torch.tensor(rows, dtype=torch.int32).pin_memory(), non_blocking=True)
         self.ctx_base[: len(base)].copy_(torch.tensor(base, dtype=torch.int32).pin_memory(), non_blocking=True)

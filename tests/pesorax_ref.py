@@ -195,7 +195,7 @@ def random_weights(cfg, seed=0):
 
     def put(name, *shape, std=None, mean=0.0):
         s = shape[-1] ** -0.5 if std is None else std
-        W[name] = (torch.randn(*shape, generator=g, dtype=torch.float64) * s + mean).to(torch.bfloat16).double()
+        W[name] = (torch.randn(shape, generator=g, dtype=torch.float64) * s + mean).to(torch.bfloat16).double()
 
     def norm(name):
         put(name, d, std=0.3, mean=1.0)
