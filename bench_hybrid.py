@@ -208,8 +208,8 @@ def time_pesorax_kernels(cfg, dev, reps: int = 12) -> list[dict]:
                 bench(f"gemm_heads value [{n}]", lambda: ops.gemm_heads(ol, wv, HL, VL, C, C, o, VL, gate=gate, status=st), wv.numel() * 2 + n * HL * (C * 2 + VL * 6),
                       2.0 * n * wv.numel(), like=f"gemm qkv [{n}]")
             bench(f"latent_q [{n}]", lambda: ops.latent_q(uq, hs, HL, DL, RL, lt.rope_dims, 1, 0, C, RL, W, pos, tab, lt.rope_base, 0.1, ql), n * HL * RL * 8, like=f"rope_kv [{n}]")
-            ctas, blocks = n * ((HL + 31) // 32), ctx // 64
-            S = min(range(1, min(64, blocks, max(1, 592 // ctas)) + 1), key=lambda s: -(-ctas * s // 148) * (-(-blocks // s) + 2))
+            ctas, blocks = n * ((HL + 31) // 32), ctx // 128
+            S = min(range(1, min(64, blocks, max(1, 592 // ctas)) + 1), key=lambda s: -(-ctas * s // 148) * (-(-blocks // s) + 1))
             sc = rnd(max(1, ops.latent_decode_scratch_floats(n, HL, C, S)))
             bench(f"latent_decode [{n} x {ctx}] ({S} shares)", lambda: ops.latent_decode(ql, cache, tb, None, pos, n, HL, C, RL, S, sc, out_bf16=ol, sinks=sink, status=st),
                   n * (ctx * W * 2 + HL * (W * 4 + C * 2)), 2.0 * n * ctx * HL * (W + C), like=f"attn_decode [{n} x {ctx}]")

@@ -110,6 +110,14 @@ __device__ __forceinline__ float gelu_tanh(float x) {
 }
 
 __device__ __forceinline__ float gelu_erf(float x) { return 0.5f * x * (1.f + erff(x * 0.7071067811865476f)); }
+// The same to about 1e-7 of x, for epilogues whose result is rounded to 16 bits: the complementary error function by formula 7.1.26 of
+// Abramowitz and Stegun, Handbook of Mathematical Functions (a polynomial in 1 / (1 + p z) times exp(-z^2)).
+__device__ __forceinline__ float gelu_erf_fast(float x) {
+  const float z = fabsf(x) * 0.7071067811865476f, t = __fdividef(1.f, fmaf(0.3275911f, z, 1.f));
+  const float p = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.061405429f, -1.453152027f), 1.421413741f), -0.284496736f), 0.254829592f);
+  const float h = x * 0.5f * p * __expf(-z * z);
+  return x > 0.f ? x - h : h;
+}
 
 // Byte slot of element i (0..7) inside each group of eight quantized activations.  The order is
 // chosen so that `v & 0x0F0F0F0F` / `(v >> 4) & 0x0F0F0F0F` of a repacked 4-bit weight word line up

@@ -55,7 +55,7 @@ int make_tmap_2d(CUtensorMap* map, const void* base, int elem_bytes, uint64_t ro
 // ACT_RELU2: the square of relu.  ACT_GELU: the tanh form; ACT_GELU_ERF: the exact one.
 enum { ACT_NONE = 0, ACT_GELU = 1, ACT_SWIGLU_PAIR = 2, ACT_RELU2 = 3, ACT_GELU_ERF = 4 };
 __device__ __forceinline__ float activate(int act, float x) {
-  return act == ACT_GELU ? gelu_tanh(x) : act == ACT_GELU_ERF ? gelu_erf(x) : act == ACT_RELU2 ? (x > 0.f ? x * x : 0.f) : x;
+  return act == ACT_GELU ? gelu_tanh(x) : act == ACT_GELU_ERF ? gelu_erf_fast(x) : act == ACT_RELU2 ? (x > 0.f ? x * x : 0.f) : x;
 }
 
 struct GemmEpi {
@@ -304,7 +304,7 @@ __device__ __forceinline__ void epilogue_row(const GemmEpi& e, int m, int n0, in
       for (int j = 0; j < 32; j++) v[j] = gelu_tanh(v[j]);
     } else if (e.act == ACT_GELU_ERF) {
 #pragma unroll
-      for (int j = 0; j < 32; j++) v[j] = gelu_erf(v[j]);
+      for (int j = 0; j < 32; j++) v[j] = gelu_erf_fast(v[j]);
     } else if (e.act == ACT_RELU2) {
 #pragma unroll
       for (int j = 0; j < 32; j++) v[j] = v[j] > 0.f ? v[j] * v[j] : 0.f;

@@ -380,6 +380,61 @@ __global__ void __launch_bounds__(128) qkv_finish_kernel(const QkvArgs a, CT* __
     }
   }
 }
+// The same where nothing rotates and nothing is normed: a thread takes four columns of one output row (head sizes and offsets that are multiples of 4).
+__device__ __forceinline__ void put4(float* p, float4 v) { *(float4*)p = v; }
+__device__ __forceinline__ void put4(__half* p, float4 v) {
+  const __half2 a = __floats2half2_rn(v.x, v.y), b = __floats2half2_rn(v.z, v.w);
+  *(uint2*)p = make_uint2(*(const uint32_t*)&a, *(const uint32_t*)&b);
+}
+template <typename CT>
+__global__ void __launch_bounds__(256) qkv_copy_kernel(const QkvArgs a, CT* __restrict__ kc, CT* __restrict__ vc) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, i = blockIdx.y * 256 + threadIdx.x;
+  const int KR = a.G * a.maps, qw = a.q_wide ? a.maps * a.DK : a.DK, q4 = qw >> 2, k4 = a.DK >> 2, v4 = a.DV >> 2;
+  const int nq = a.H * q4, nk = a.k_off >= 0 ? KR * k4 : 0, nv = a.k_off >= 0 ? a.G * v4 : 0;
+  if (i >= nq + nk + nv) return;
+  const float* row = a.in + (size_t)t * a.ld;
+  int hh, c, col;
+  bool in;                                                // within the head's own columns (else padding, or the other map's half)
+  if (i < nq) {
+    hh = i / q4;
+    c = (i - hh * q4) << 2;
+    const int cc = a.q_wide ? c - hh / (a.H / KR) % a.maps * a.DK : c;
+    in = cc >= 0 && cc < a.dim;
+    col = a.q_off + hh * a.dim + cc;
+  } else if (i < nq + nk) {
+    hh = (i - nq) / k4;
+    c = (i - nq - hh * k4) << 2;
+    in = c < a.dim;
+    col = a.k_off + hh * a.dim + c;
+  } else {
+    hh = (i - nq - nk) / v4;
+    c = (i - nq - nk - hh * v4) << 2;
+    in = c < a.vdim;
+    col = a.v_off + hh * a.vdim + c;
+  }
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (in) {
+    v = *(const float4*)(row + col);
+    if (a.bias) {
+      const float4 b = *(const float4*)(a.bias + col);
+      v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+    }
+  }
+  if (i < nq) {
+    v.x *= a.q_scale; v.y *= a.q_scale; v.z *= a.q_scale; v.w *= a.q_scale;
+    const size_t at = ((size_t)t * a.H + hh) * qw + c;
+    if (a.q32) put4(a.q32 + at, v);
+    if (a.q16) put4(a.q16 + at, v);
+    return;
+  }
+  const int s = a.slot[t];
+  if (s < 0) return;
+  const int page = s / a.page_size, off = s % a.page_size;
+  if (i < nq + nk) put4(kc + ((((size_t)page * a.G + hh / a.maps) * a.page_size + off) * a.maps + hh % a.maps) * a.DK + c, v);
+  else put4(vc + (((size_t)page * a.G + hh) * a.page_size + off) * a.DV + c, v);
+}
 // cache_f32: kc / vc hold fp32 instead of fp16; layout [page][G][page_size][maps * DK or DV].
 B200_API int b200_qkv_finish(const float* in, int ld, int T, int q_off, int k_off, int v_off, const int* pos, const int* slot,
                              const void* tab, int tab_len, double base, int H, int G, int dim, int vdim, int DK, int DV, int rot,
@@ -394,6 +449,13 @@ B200_API int b200_qkv_finish(const float* in, int ld, int T, int q_off, int k_of
   a.tab_len = tab ? tab_len : 0; a.base = base; a.H = H; a.G = G; a.dim = dim; a.vdim = vdim; a.DK = DK; a.DV = DV; a.rot = rot;
   a.style = style; a.qk_norm = qk_norm; a.page_size = page_size; a.eps = eps; a.q_scale = q_scale; a.q32 = q32; a.q16 = (__half*)q16;
   a.maps = maps; a.q_wide = q_wide; a.bias = bias;
+  if (rot == 0 && !qk_norm && ((ld | q_off | dim | vdim | DK | DV) & 3) == 0 && (k_off < 0 || ((k_off | v_off) & 3) == 0) &&
+      (((uintptr_t)in | (uintptr_t)bias | (uintptr_t)q32 | (uintptr_t)q16 | (uintptr_t)kc | (uintptr_t)vc) & 15) == 0) {
+    const int quads = (H * (q_wide ? maps : 1) * DK + (k_off >= 0 ? G * (maps * DK + DV) : 0)) / 4;
+    const dim3 g(T, (quads + 255) / 256);
+    if (cache_f32) return launch_pdl(qkv_copy_kernel<float>, g, dim3(256), 0, st, a, (float*)kc, (float*)vc);
+    return launch_pdl(qkv_copy_kernel<__half>, g, dim3(256), 0, st, a, (__half*)kc, (__half*)vc);
+  }
   const int n_heads = H + (k_off >= 0 ? (maps + 1) * G : 0);
   const dim3 grid(T, (n_heads + 3) / 4);
   if (cache_f32) return launch_pdl(qkv_finish_kernel<float>, grid, dim3(128), 0, st, a, (float*)kc, (float*)vc);
@@ -637,6 +699,95 @@ B200_API int b200_gemm_f32(const float* A, int lda, const void* W, int ldb, floa
     return B200_ERR_BAD_ARG;
   return launch_pdl(gemm_f32_kernel, dim3((N + 63) / 64, (M + 63) / 64, heads), dim3(256), 0, st, A, lda, (const __nv_bfloat16*)W, ldb, C,
                     ldc, M, N, K, act, alpha, accumulate, gate, ldg, head_k, head_ldc);
+}
+
+// ------------------------------------------------------------------ one small mat-vec per head
+
+// out[t][z * head_ldc + n] = alpha * sum_k A[t][z * head_k + k] W[z * N + n][k], times sigmoid(gate[t][z * head_ldc + n]) where given: gemm_f32's
+// per-head product for 1..8 rows.  LPR lanes share a weight row (LPR * 8 columns per pass); a group of them holds four rows in flight.
+template <int T, int LPR>
+__global__ void __launch_bounds__(256) head_matvec_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W, int ldb,
+                                                          float* __restrict__ out, int ldc, int rows, int N, int K, float alpha,
+                                                          const float* __restrict__ gate, int ldg, int head_k, int head_ldc) {
+  extern __shared__ __align__(16) float xs[];          // [T][K]
+  const int z = blockIdx.y, grp = threadIdx.x / LPR, gl = threadIdx.x % LPR, n0 = (blockIdx.x * (256 / LPR) + grp) * 4;
+  const __nv_bfloat16* w = W + (size_t)z * N * ldb;
+  uint4 q[4];
+  auto fetch = [&](int k) {
+#pragma unroll
+    for (int r = 0; r < 4; r++) q[r] = ldg_stream(w + (size_t)min(n0 + r, N - 1) * ldb + k);
+  };
+  const bool live = n0 < N;
+  if (live && gl * 8 < K) fetch(gl * 8);               // weights do not wait for the kernel before this one
+  pdl_trigger();
+  pdl_wait();
+  for (int i = threadIdx.x; i < T * K; i += 256) {
+    const int t = i / K, k = i - t * K;
+    xs[i] = t < rows ? A[(size_t)t * lda + (size_t)z * head_k + k] : 0.f;
+  }
+  __syncthreads();
+  float acc[4][T];
+#pragma unroll
+  for (int r = 0; r < 4; r++)
+#pragma unroll
+    for (int t = 0; t < T; t++) acc[r][t] = 0.f;
+  for (int k = gl * 8; k < K && live; k += LPR * 8) {
+    if (k != gl * 8) fetch(k);
+#pragma unroll
+    for (int t = 0; t < T; t++) {
+      const float4 x0 = *(const float4*)(xs + t * K + k), x1 = *(const float4*)(xs + t * K + k + 4);
+#pragma unroll
+      for (int r = 0; r < 4; r++) {
+        const __nv_bfloat162* p = (const __nv_bfloat162*)&q[r];
+        float2 f;
+        f = __bfloat1622float2(p[0]); acc[r][t] += f.x * x0.x + f.y * x0.y;
+        f = __bfloat1622float2(p[1]); acc[r][t] += f.x * x0.z + f.y * x0.w;
+        f = __bfloat1622float2(p[2]); acc[r][t] += f.x * x1.x + f.y * x1.y;
+        f = __bfloat1622float2(p[3]); acc[r][t] += f.x * x1.z + f.y * x1.w;
+      }
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < 4; r++)
+#pragma unroll
+    for (int t = 0; t < T; t++) {
+#pragma unroll
+      for (int o = LPR / 2; o > 0; o >>= 1) acc[r][t] += __shfl_xor_sync(0xffffffffu, acc[r][t], o);
+    }
+  if (gl != 0 || !live) return;
+#pragma unroll
+  for (int r = 0; r < 4; r++)
+#pragma unroll
+    for (int t = 0; t < T; t++) {
+      if (n0 + r >= N || t >= rows) continue;
+      const int c = z * head_ldc + n0 + r;
+      float v = acc[r][t] * alpha;
+      if (gate) v *= 1.f / (1.f + expf(-gate[(size_t)t * ldg + c]));
+      out[(size_t)t * ldc + c] = v;
+    }
+}
+template <int T>
+static int launch_head_matvec(const float* A, int lda, const __nv_bfloat16* W, int ldb, float* out, int ldc, int rows, int heads, int N, int K, float alpha,
+                              const float* gate, int ldg, int head_k, int head_ldc, cudaStream_t st) {
+  const size_t smem = (size_t)T * K * 4;
+  const int lpr = K <= 64 ? 8 : K <= 128 ? 16 : 32;
+  const dim3 grid((N + 1024 / lpr - 1) / (1024 / lpr), heads);
+  auto kern = lpr == 8 ? head_matvec_kernel<T, 8> : lpr == 16 ? head_matvec_kernel<T, 16> : head_matvec_kernel<T, 32>;
+  return launch_pdl(kern, grid, dim3(256), smem, st, A, lda, W, ldb, out, ldc, rows, N, K, alpha, gate, ldg, head_k, head_ldc);
+}
+// A fp32 [rows][lda], W bf16 [heads * N][ldb]; rows <= 8, K a multiple of 8 (48 KB of activations at most).
+B200_API int b200_head_matvec(const float* A, int lda, const void* W, int ldb, float* out, int ldc, int rows, int heads, int N, int K, float alpha,
+                              const float* gate, int ldg, int head_k, int head_ldc, cudaStream_t st) {
+  if (rows < 1 || rows > 8 || heads < 1 || N < 1 || K < 8 || K % 8 || ldb % 8 || ((uintptr_t)W & 15) || K > head_k || N > head_ldc) return B200_ERR_BAD_ARG;
+  const int T = rows <= 1 ? 1 : rows <= 2 ? 2 : rows <= 4 ? 4 : 8;
+  if ((size_t)T * K * 4 > 48 * 1024) return B200_ERR_BAD_ARG;
+  const __nv_bfloat16* w = (const __nv_bfloat16*)W;
+  switch (T) {
+    case 1: return launch_head_matvec<1>(A, lda, w, ldb, out, ldc, rows, heads, N, K, alpha, gate, ldg, head_k, head_ldc, st);
+    case 2: return launch_head_matvec<2>(A, lda, w, ldb, out, ldc, rows, heads, N, K, alpha, gate, ldg, head_k, head_ldc, st);
+    case 4: return launch_head_matvec<4>(A, lda, w, ldb, out, ldc, rows, heads, N, K, alpha, gate, ldg, head_k, head_ldc, st);
+  }
+  return launch_head_matvec<8>(A, lda, w, ldb, out, ldc, rows, heads, N, K, alpha, gate, ldg, head_k, head_ldc, st);
 }
 
 // ------------------------------------------------------------------ last step of the logits

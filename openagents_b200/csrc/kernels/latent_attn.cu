@@ -54,28 +54,64 @@ struct LatentFinishArgs {
   __nv_bfloat16* cq16;
   int ldq, CR, RR;
 };
+constexpr int kFinishQ = 6, kFinishC = 3;
 template <typename CT>
 __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinishArgs a, CT* __restrict__ cache) {
-  __shared__ float red[32];
+  __shared__ float2 red[8];
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x, nt = blockDim.x;
   const float* row = a.in + (size_t)t * a.ld;
+  // both latents are held in registers (the first kFinishQ / kFinishC columns per thread; longer ones are read again)
+  float vq[kFinishQ], vc[kFinishC];
+  const int s = a.slot[t], p = a.pos[t];
+#pragma unroll
+  for (int k = 0; k < kFinishQ; k++) {
+    const int i = threadIdx.x + k * nt;
+    vq[k] = i < a.q_rank ? row[a.q_off + i] : 0.f;
+  }
+#pragma unroll
+  for (int k = 0; k < kFinishC; k++) {
+    const int i = threadIdx.x + k * nt;
+    vc[k] = i < a.rank ? row[a.c_off + i] : 0.f;
+  }
   float sq = 0.f, sc = 0.f;
-  for (int i = threadIdx.x; i < a.q_rank; i += nt) { const float v = row[a.q_off + i]; sq += v * v; }
-  for (int i = threadIdx.x; i < a.rank; i += nt) { const float v = row[a.c_off + i]; sc += v * v; }
-  const float rq = 1.f / sqrtf(block_sum(sq, red) / (float)a.q_rank + a.eps);
-  const float rc = 1.f / sqrtf(block_sum(sc, red) / (float)a.rank + a.eps);
-  for (int i = threadIdx.x; i < a.ldq; i += nt) {
-    const float v = i < a.q_rank ? row[a.q_off + i] * rq * a.q_w[i] : 0.f;
+#pragma unroll
+  for (int k = 0; k < kFinishQ; k++) sq += vq[k] * vq[k];
+#pragma unroll
+  for (int k = 0; k < kFinishC; k++) sc += vc[k] * vc[k];
+  for (int i = threadIdx.x + kFinishQ * nt; i < a.q_rank; i += nt) { const float v = row[a.q_off + i]; sq += v * v; }
+  for (int i = threadIdx.x + kFinishC * nt; i < a.rank; i += nt) { const float v = row[a.c_off + i]; sc += v * v; }
+  sq = warp_sum(sq);
+  sc = warp_sum(sc);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(sq, sc);
+  __syncthreads();
+  sq = sc = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; w++) {
+    const float2 e = red[w];
+    sq += e.x;
+    sc += e.y;
+  }
+  const float rq = 1.f / sqrtf(sq / (float)a.q_rank + a.eps), rc = 1.f / sqrtf(sc / (float)a.rank + a.eps);
+  auto put_q = [&](int i, float v) {
     if (a.cq32) a.cq32[(size_t)t * a.ldq + i] = v;
     if (a.cq16) a.cq16[(size_t)t * a.ldq + i] = __float2bfloat16(v);
+  };
+#pragma unroll
+  for (int k = 0; k < kFinishQ; k++) {
+    const int i = threadIdx.x + k * nt;
+    if (i < a.ldq) put_q(i, i < a.q_rank ? vq[k] * rq * a.q_w[i] : 0.f);
   }
-  const int s = a.slot[t];
+  for (int i = threadIdx.x + kFinishQ * nt; i < a.ldq; i += nt) put_q(i, i < a.q_rank ? row[a.q_off + i] * rq * a.q_w[i] : 0.f);
   if (s < 0) return;
   CT* dst = cache + (size_t)s * (a.CR + a.RR);
-  for (int i = threadIdx.x; i < a.CR; i += nt) put(dst + i, i < a.rank ? row[a.c_off + i] * rc * a.c_w[i] : 0.f);
-  const int p = a.pos[t];
+#pragma unroll
+  for (int k = 0; k < kFinishC; k++) {
+    const int i = threadIdx.x + k * nt;
+    if (i < a.CR) put(dst + i, i < a.rank ? vc[k] * rc * a.c_w[i] : 0.f);
+  }
+  for (int i = threadIdx.x + kFinishC * nt; i < a.CR; i += nt) put(dst + i, i < a.rank ? row[a.c_off + i] * rc * a.c_w[i] : 0.f);
   for (int i = threadIdx.x; i < a.RR; i += nt)
     put(dst + a.CR + i, i < a.rot_dim ? rotated(row + a.r_off, i, a.rot, a.style, a.tab, a.tab_len, a.base, p) : 0.f);
 }
@@ -180,15 +216,16 @@ B200_API int b200_latent_gather(const void* cache, int KS, int CR, const int* pa
 
 // One CTA = (share of the keys, group of N heads, query row).  The cached rows are the 128-row operand of both products and the heads the narrow
 // one, so a product costs what its heads need:
-//   S^T [keys][N]  = C [64 keys][CR + RR] Q'^T          (K-major A; operand rows 64..127 are whatever follows in shared memory: their
-//                                                        accumulator rows are never read)
-//   O^T [dims][N] += C^T [128 dims][64 keys] P^T        per 128 latent dimensions (MN-major A: the same bytes, read the other way)
-// Roles: warps 0..7 softmax, rescale and output; warps 8..11 fetch one 16-token page of a 64-key block each; warp 12 issues the first product, warp 13
-// the second.  Scores, weights and sums are fp32; P is fp16.  A head's exponent offset moves only when its maximum has grown by more than 8 (log2).
+//   S^T [keys][N]  = C [128 keys][CR + RR] Q'^T         (K-major A)
+//   O^T [dims][N] += C^T [128 dims][128 keys] P^T       per 128 latent dimensions (MN-major A: the same bytes, read the other way)
+// Roles: warps 0..7 softmax, rescale and output; warps 8..11 fetch two 16-token pages of a 128-key block each; warp 12 issues the first product, warp 13
+// the second.  A block is 147 KB at 512 + 64 columns, so shared memory holds little more than one: it is handed over in pairs of 64-column boxes, the
+// first product follows the copies pair by pair, and the second gives each pair back as soon as it is done with it.  Scores, weights and sums are fp32; P is fp16.  A head's exponent offset moves only when its maximum has grown by more than 8 (log2).
 // Every wait is bounded; one that runs out sets the status word and the CTA leaves through the common exit.
 namespace {
 
-constexpr int kLKeys = 64, kLBox = kLKeys * 128, kLThreads = 448;
+constexpr int kLPairs = 8;                             // pairs of boxes in shared memory at most
+constexpr int kLKeys = 128, kLBox = kLKeys * 128, kLThreads = 448;
 constexpr float kRescaleStep = 8.f;
 
 struct LatentDecArgs {
@@ -197,7 +234,7 @@ struct LatentDecArgs {
   const int* row_seq;      // [R] sequence of each row, or null: row r is sequence r
   const int* pos;          // [R] position of each row: it sees keys 0..pos
   const float* sinks;      // [H] or null
-  int max_pages, H, CR, RR, S, stages;
+  int max_pages, H, CR, RR, S, pairs;      // pairs: slots of the ring
   float* part;             // S > 1: [R][S][H][CR], then [R][S][H][2] (offset, sum)
   float* part_ml;
   float* out_f32;          // [R][ldo], head h at column h * CR
@@ -244,9 +281,14 @@ __device__ __forceinline__ bool meet(bool ok) {
                : "=r"(r) : "r"((uint32_t)ok) : "memory");
   return r != 0;
 }
-// NC values per lane -> lane's result: reduction over the 32 lanes of column `col` (returned).  Halves are exchanged, so it takes about NC shuffles.
-template <int NC, bool MAX>
-__device__ __forceinline__ float reduce_columns(const float (&in)[NC], int lane, int& col) {
+__device__ __forceinline__ float lanes_max(float v) {
+  float r;
+  asm("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(r) : "f"(v));
+  return r;
+}
+// NC values per lane -> the sum over the 32 lanes of column `col` (returned).  Halves are exchanged, so it takes about NC shuffles.
+template <int NC>
+__device__ __forceinline__ float sum_columns(const float (&in)[NC], int lane, int& col) {
   float v[NC];
 #pragma unroll
   for (int i = 0; i < NC; i++) v[i] = in[i];
@@ -261,15 +303,11 @@ __device__ __forceinline__ float reduce_columns(const float (&in)[NC], int lane,
     for (int i = 0; i < NC / 2; i++) {
       if (i >= h) continue;
       const float keep = up ? v[i + h] : v[i], give = up ? v[i] : v[i + h];
-      const float got = __shfl_xor_sync(0xffffffffu, give, off);
-      v[i] = MAX ? fmaxf(keep, got) : keep + got;
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, off);
     }
   }
 #pragma unroll
-  for (; off > 0; off >>= 1) {
-    const float got = __shfl_xor_sync(0xffffffffu, v[0], off);
-    v[0] = MAX ? fmaxf(v[0], got) : v[0] + got;
-  }
+  for (; off > 0; off >>= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], off);
   return v[0];
 }
 
@@ -279,37 +317,41 @@ __global__ void __launch_bounds__(kLThreads, 1) latent_decode_kernel(const __gri
   constexpr uint32_t TMEM_COLS = 256;                  // S: 2 x N, O: up to 5 x N
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
-  const int boxes = (a.CR + a.RR) >> 6, stage_bytes = boxes * kLBox, W = a.CR + a.RR;
-  uint8_t* sC = smem;                                  // stages x boxes x [64 keys][128 bytes]
-  uint8_t* sQ = sC + a.stages * stage_bytes;           // boxes x [N][128 bytes]
-  uint8_t* sP = sQ + boxes * N * 128;                  // 2 x [N][64 keys]
+  const int boxes = (a.CR + a.RR) >> 6, c_boxes = a.CR >> 6, W = a.CR + a.RR;
+  const int nt = (a.CR + 127) >> 7;                    // 128-dimension tiles of the output = pairs of a block (the last may be half)
+  uint8_t* sC = smem;                                  // pairs x 2 x [128 keys][128 bytes]
+  uint8_t* sR = sC + a.pairs * 2 * kLBox;              // the rotated parts' boxes, one block of them
+  uint8_t* sQ = sR + (boxes - c_boxes) * kLBox;        // boxes x [N][128 bytes]
+  uint8_t* sP = sQ + boxes * N * 128;                  // 2 key halves x [N][64 keys]
   uint64_t* bars = (uint64_t*)(sP + 2 * N * 128);
-  uint64_t* kv_full = bars;                            // [4]
-  uint64_t* kv_empty = bars + 4;                       // [4]
-  uint64_t* s_full = bars + 8;                         // [2]
-  uint64_t* s_empty = bars + 10;                       // [2]
-  uint64_t* p_full = bars + 12;                        // [2]
-  uint64_t* pv_done = bars + 14;                       // [2]
-  uint32_t* tmem_holder = (uint32_t*)(bars + 16);
+  uint64_t* c_full = bars;                             // [pairs]
+  uint64_t* c_empty = bars + kLPairs;                  // [pairs]
+  uint64_t* r_full = bars + 2 * kLPairs;
+  uint64_t* r_empty = r_full + 1;
+  uint64_t* s_full = r_full + 2;                       // [2]
+  uint64_t* s_empty = r_full + 4;                      // [2]
+  uint64_t* p_full = r_full + 6;
+  uint64_t* pv_done = r_full + 7;
+  uint32_t* tmem_holder = (uint32_t*)(r_full + 8);
   volatile int* abort_flag = (volatile int*)(tmem_holder + 1);
-  volatile int* any_scale = (volatile int*)(tmem_holder + 2);
-  float* s_part = (float*)(bars + 18);                 // [2 quarters][N] maxima, then sums
-  float* s_m = s_part + 2 * N;                         // [N] exponent offsets
-  float* s_sc = s_m + N;                               // [N] rescale factors, then 1 / sum
+  float* s_part = (float*)(r_full + 10);               // [2 (block parity)][4 quarters][N] maxima, then sums
+  float* s_inv = s_part + 8 * N;                       // [N] 1 / sum
 
   const int split = blockIdx.x, h0 = blockIdx.y * N, row = blockIdx.z;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (tid == 0) {
-    for (int s = 0; s < 4; s++) {
-      mbar_init(smem_u32(kv_full + s), 4);
-      mbar_init(smem_u32(kv_empty + s), 1);
+    for (int s = 0; s < kLPairs; s++) {
+      mbar_init(smem_u32(c_full + s), 4);
+      mbar_init(smem_u32(c_empty + s), 1);
     }
+    mbar_init(smem_u32(r_full), 4);
+    mbar_init(smem_u32(r_empty), 1);
     for (int s = 0; s < 2; s++) {
       mbar_init(smem_u32(s_full + s), 1);
-      mbar_init(smem_u32(s_empty + s), 4);
-      mbar_init(smem_u32(p_full + s), 8);
-      mbar_init(smem_u32(pv_done + s), 1);
+      mbar_init(smem_u32(s_empty + s), 8);
     }
+    mbar_init(smem_u32(p_full), 8);
+    mbar_init(smem_u32(pv_done), 1);
     *abort_flag = 0;
     fence_barrier_init();
     tma_prefetch_desc(&tm);
@@ -329,178 +371,206 @@ __global__ void __launch_bounds__(kLThreads, 1) latent_decode_kernel(const __gri
   const int blocks = (len + kLKeys - 1) / kLKeys, per = (blocks + a.S - 1) / a.S;
   const int j0 = split * per, nb = max(0, min(blocks, j0 + per) - j0);
   const int* pt = a.page_table + (size_t)(a.row_seq ? a.row_seq[row] : row) * a.max_pages;
-  const int nt = (a.CR + 127) >> 7;                    // 128-dimension tiles of the output
 
-  auto fetch = [&](int j) {                            // one lane of warps 8..11: this warp's page of block j
-    const int s = j % a.stages, p = warp - 8, pi = (j0 + j) * (kLKeys / 16) + p;
-    const int r = (pi * 16 < len ? pt[pi] : 0) * 16;   // pages past the context are masked
-    const uint32_t bar = smem_u32(kv_full + s);
-    mbar_expect_tx(bar, boxes * 2048);
-    uint8_t* dst = sC + (size_t)s * stage_bytes + p * 2048;
-    for (int c = 0; c < boxes; c++) tma_load_2d(smem_u32(dst + c * kLBox), &tm, bar, c * 64, r);
+  // one lane of warps 8..11: this warp's two pages of one part of block j (i = -1: the rotated boxes, else pair i)
+  auto fetch = [&](int j, int i) {
+    const int slot = i < 0 ? 0 : (j * nt + i) % a.pairs, b0 = i < 0 ? c_boxes : 2 * i, n_box = (i < 0 ? boxes : min(2 * i + 2, c_boxes)) - b0;
+    const uint32_t bar = smem_u32(i < 0 ? r_full : c_full + slot);
+    uint8_t* dst = i < 0 ? sR : sC + (size_t)slot * 2 * kLBox;
+    mbar_expect_tx(bar, n_box * 4096);
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+      const int p = (warp - 8) * 2 + h, pi = (j0 + j) * (kLKeys / 16) + p;
+      const int r = (pi * 16 < len ? pt[pi] : 0) * 16;                    // pages past the context are masked
+      for (int c = 0; c < n_box; c++) tma_load_2d(smem_u32(dst + c * kLBox + p * 2048), &tm, bar, (b0 + c) * 64, r);
+    }
   };
   const bool producer = warp >= 8 && warp < 12;
   if (producer) {
     if (lane == 0)
-      for (int j = 0; j < min(nb, a.stages); j++) fetch(j);
+      for (int i = -1; i < nt && nb > 0; i++) fetch(0, i);               // the first block: the ring is empty and holds all of it
     __syncwarp();
   } else {
     // queries: fp32 -> fp16, 128-byte-swizzled rows of 64 columns; heads past the last are zeros
-    const int t = warp < 8 ? tid : tid - 128, n_t = kLThreads - 128;
-    for (int i = t; i < N * (W >> 1); i += n_t) {
-      const int n = i / (W >> 1), c = (i % (W >> 1)) * 2, cc = c & 63;
-      float2 v = make_float2(0.f, 0.f);
-      if (h0 + n < a.H) v = *(const float2*)(a.q + ((size_t)row * a.H + h0 + n) * W + c);
-      *(__half2*)(sQ + (c >> 6) * (N * 128) + n * 128 + (((cc >> 3) ^ (n & 7)) << 4) + (cc & 7) * 2) = __floats2half2_rn(v.x, v.y);
+    const int t = warp < 8 ? tid : tid - 128, n_t = kLThreads - 128, q4 = W >> 2;
+#pragma unroll 4
+    for (int i = t; i < N * q4; i += n_t) {
+      const int n = i / q4, c = (i - n * q4) * 4, cc = c & 63;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (h0 + n < a.H) v = *(const float4*)(a.q + ((size_t)row * a.H + h0 + n) * W + c);
+      const __half2 x = __floats2half2_rn(v.x, v.y), y = __floats2half2_rn(v.z, v.w);
+      *(uint2*)(sQ + (c >> 6) * (N * 128) + n * 128 + (((cc >> 3) ^ (n & 7)) << 4) + (cc & 7) * 2) =
+          make_uint2(*(const uint32_t*)&x, *(const uint32_t*)&y);
     }
     fence_proxy_async_smem();
   }
   __syncthreads();
 
   if (producer) {
-    if (lane == 0)
-      for (int j = a.stages; j < nb; j++) {
-        if (!mbar_wait(smem_u32(kv_empty + j % a.stages), ((j / a.stages) & 1) ^ 1, abort_flag)) break;
-        fetch(j);
-      }
+    if (lane == 0) {
+      bool ok = true;
+      for (int j = 1; j < nb && ok; j++)
+        for (int i = -1; i < nt && ok; i++) {          // the rotated parts first: they are given back first
+          const int t = j * nt + i;
+          ok = i < 0 ? mbar_wait(smem_u32(r_empty), (j & 1) ^ 1, abort_flag)
+                     : mbar_wait(smem_u32(c_empty + t % a.pairs), ((t / a.pairs) & 1) ^ 1, abort_flag);
+          if (ok) fetch(j, i);
+        }
+    }
   } else if (warp == 12) {
-    if (lane == 0)
-      for (int j = 0; j < nb; j++) {
-        const int s = j % a.stages, b = j & 1;
-        if (!mbar_wait(smem_u32(kv_full + s), (j / a.stages) & 1, abort_flag)) break;
+    if (lane == 0) {
+      bool ok = true;
+      const uint32_t qa = smem_u32(sQ);
+      for (int j = 0; j < nb && ok; j++) {
+        const int b = j & 1;
         if (!mbar_wait(smem_u32(s_empty + b), ((j >> 1) & 1) ^ 1, abort_flag)) break;
-        tc_fence_after();
-        const uint32_t ca = smem_u32(sC + (size_t)s * stage_bytes), qa = smem_u32(sQ);
-        for (int c = 0; c < boxes; c++) {
-          const uint64_t ad = smem_desc_sw128(ca + c * kLBox), qd = smem_desc_sw128(qa + c * (N * 128));
+        for (int i = -1; i < nt && ok; i++) {
+          const int t = j * nt + i, slot = i < 0 ? 0 : t % a.pairs, b0 = i < 0 ? c_boxes : 2 * i, b1 = i < 0 ? boxes : min(2 * i + 2, c_boxes);
+          ok = i < 0 ? mbar_wait(smem_u32(r_full), j & 1, abort_flag) : mbar_wait(smem_u32(c_full + slot), (t / a.pairs) & 1, abort_flag);
+          if (!ok) break;
+          tc_fence_after();
+          const uint32_t ca = smem_u32(i < 0 ? sR : sC + (size_t)slot * 2 * kLBox);
+          for (int c = b0; c < b1; c++) {
+            const uint64_t ad = smem_desc_sw128(ca + (c - b0) * kLBox), qd = smem_desc_sw128(qa + c * (N * 128));
 #pragma unroll
-          for (int k = 0; k < 4; k++) umma_bf16(S_T + b * N, ad + 2 * k, qd + 2 * k, idesc_lat(N, false), (c | k) ? 1u : 0u);
+            for (int k = 0; k < 4; k++) umma_bf16(S_T + b * N, ad + 2 * k, qd + 2 * k, idesc_lat(N, false), (i >= 0 || c > b0 || k) ? 1u : 0u);
+          }
+          if (i < 0) umma_commit(smem_u32(r_empty));   // the rotated parts are no values: nobody else reads them
         }
-        umma_commit(smem_u32(s_full + b));
+        if (ok) umma_commit(smem_u32(s_full + b));
       }
+    }
   } else if (warp == 13) {
-    if (lane == 0)
-      for (int j = 0; j < nb; j++) {
-        const int s = j % a.stages, b = j & 1;
-        if (!mbar_wait(smem_u32(kv_full + s), (j / a.stages) & 1, abort_flag)) break;
-        if (!mbar_wait(smem_u32(p_full + b), (j >> 1) & 1, abort_flag)) break;
+    if (lane == 0) {
+      bool ok = true;
+      // the page of the partial results is looked up while there is time
+      if (a.S > 1) asm volatile("prefetch.global.L2 [%0];" ::"l"(a.part + (((size_t)row * a.S + split) * a.H + h0) * a.CR));
+      for (int j = 0; j < nb && ok; j++) {
+        for (int i = 0; i < nt && ok; i++) ok = mbar_wait(smem_u32(c_full + (j * nt + i) % a.pairs), ((j * nt + i) / a.pairs) & 1, abort_flag);
+        if (!ok || !mbar_wait(smem_u32(p_full), j & 1, abort_flag)) break;
         tc_fence_after();
-        const uint32_t ca = smem_u32(sC + (size_t)s * stage_bytes);
-        const uint64_t pd = smem_desc_sw128(smem_u32(sP + b * N * 128));
+        const uint64_t pd = smem_desc_sw128(smem_u32(sP));
         for (int i = 0; i < nt; i++) {
-          const uint64_t ad = smem_desc_sw128_mn(ca + 2 * i * kLBox, kLBox);
+          const int slot = (j * nt + i) % a.pairs;
+          const uint64_t ad = smem_desc_sw128_mn(smem_u32(sC + (size_t)slot * 2 * kLBox), kLBox);
 #pragma unroll
-          for (int k = 0; k < 4; k++) umma_bf16(O_T + i * N, ad + 128 * k, pd + 2 * k, idesc_lat(N, true), (j | k) ? 1u : 0u);
+          for (int k = 0; k < 8; k++)
+            umma_bf16(O_T + i * N, ad + 128 * k, pd + (k >> 2) * (N * 8) + 2 * (k & 3), idesc_lat(N, true), (j | k) ? 1u : 0u);
+          umma_commit(smem_u32(c_empty + slot));
         }
-        umma_commit(smem_u32(pv_done + b));
-        umma_commit(smem_u32(kv_empty + s));
+        umma_commit(smem_u32(pv_done));
       }
+    }
   } else {
     const int q = warp & 3, half = warp >> 2, c0 = half * NC;
     const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
-    const bool scorer = q < 2;                         // the two lane quarters that hold the 64 keys
     const int key_in = q * 32 + lane;
-    float m_used = -INFINITY;                          // threads 0..N-1: the head's exponent offset (log2 units)
-    float l[NC];
+    float m_used[NC], l[NC];                           // this warp's heads: exponent offset (log2 units, the same in every thread), part of the sum
 #pragma unroll
-    for (int i = 0; i < NC; i++) l[i] = 0.f;
+    for (int i = 0; i < NC; i++) {
+      m_used[i] = -INFINITY;
+      l[i] = 0.f;
+    }
     bool ok = true;
     for (int j = 0; j < nb; j++) {
       const int b = j & 1;
       ok = ok && mbar_wait(smem_u32(s_full + b), (j >> 1) & 1, abort_flag);
-      if (j >= 2) ok = ok && mbar_wait(smem_u32(pv_done + b), ((j - 2) >> 1) & 1, abort_flag);      // P buffer b is free again
+      if (j > 0) ok = ok && mbar_wait(smem_u32(pv_done), (j - 1) & 1, abort_flag);      // P is free again, O is at rest
       ok = __all_sync(0xffffffffu, ok);
       tc_fence_after();
       float x[NC];
-      if (scorer) {
+      bool behind = false;
+      {
         uint32_t r[NC];
         tmem_ld<NC>(S_T + b * N + lane_addr + c0, r);
         tmem_ld_wait();
         const bool seen = (j0 + j) * kLKeys + key_in < len;
 #pragma unroll
         for (int i = 0; i < NC; i++) x[i] = seen ? __uint_as_float(r[i]) * kLog2e : -INFINITY;
-        int col;
-        const float mx = reduce_columns<NC, true>(x, lane, col);
-        s_part[q * N + c0 + col] = mx;                 // the lanes of a column hold the same value
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(smem_u32(s_empty + b));
-      }
-      if (!meet(ok)) break;
-      if (tid < 32) {
-        float sc = 1.f;
-        if (tid < N) {
-          const float mx = fmaxf(s_part[tid], s_part[N + tid]);
-          if (m_used == -INFINITY) {
-            m_used = mx;
-          } else if (mx > m_used + kRescaleStep) {
-            sc = ex2(m_used - mx);
-            m_used = mx;
-          }
-          s_m[tid] = m_used == -INFINITY ? 0.f : m_used;
-          s_sc[tid] = sc;
-        }
-        const unsigned moved = __ballot_sync(0xffffffffu, sc != 1.f);
-        if (tid == 0) *any_scale = moved != 0u;
-      }
-      meet(true);
-      if (*any_scale && j > 0) {
-        ok = mbar_wait(smem_u32(pv_done + ((j - 1) & 1)), ((j - 1) >> 1) & 1, abort_flag);
-        ok = __all_sync(0xffffffffu, ok);
-        tc_fence_after();
-        for (int i = 0; i < nt; i++) {
-          uint32_t r[NC];
-          tmem_ld<NC>(O_T + i * N + lane_addr + c0, r);
-          tmem_ld_wait();
 #pragma unroll
-          for (int k = 0; k < NC; k++) r[k] = __float_as_uint(__uint_as_float(r[k]) * s_sc[c0 + k]);
-          tmem_st<NC>(O_T + i * N + lane_addr + c0, r);
-        }
-        tmem_st_wait();
+        for (int i = 0; i < NC; i++) behind |= x[i] > m_used[i] + kRescaleStep;      // also while no offset is set
+        behind = __any_sync(0xffffffffu, behind);
       }
-      if (scorer) {
-        uint8_t* p = sP + b * N * 128;
+      if (!meet(ok && !behind)) {                      // some offset has to move (always in the first block), or something failed
+        float* part = s_part + b * 4 * N;
 #pragma unroll
         for (int i = 0; i < NC; i++) {
-          const int n = c0 + i;
-          const float w = ex2(x[i] - s_m[n]);
-          l[i] = l[i] * s_sc[n] + w;
-          *(__half*)(p + n * 128 + (((key_in >> 3) ^ (n & 7)) << 4) + (key_in & 7) * 2) = __float2half(w);
+          const float mx = lanes_max(x[i]);            // over this warp's keys
+          if (lane == 0) part[q * N + c0 + i] = mx;
+        }
+        if (!meet(ok)) break;
+        float sc[NC];
+        bool moved = false;
+#pragma unroll
+        for (int i = 0; i < NC; i++) {
+          const float* p = part + c0 + i;
+          const float top = fmaxf(fmaxf(p[0], p[N]), fmaxf(p[2 * N], p[3 * N])), old = m_used[i];
+          const bool up = top > old + kRescaleStep;
+          m_used[i] = up ? top : old;
+          sc[i] = up && old != -INFINITY ? ex2(old - top) : 1.f;
+          moved |= sc[i] != 1.f;
+        }
+        if (moved) {                                   // uniform: every thread of the warp sees the same maxima
+          for (int i = 0; i < nt; i++) {
+            uint32_t r[NC];
+            tmem_ld<NC>(O_T + i * N + lane_addr + c0, r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int k = 0; k < NC; k++) r[k] = __float_as_uint(__uint_as_float(r[k]) * sc[k]);
+            tmem_st<NC>(O_T + i * N + lane_addr + c0, r);
+          }
+          tmem_st_wait();
+#pragma unroll
+          for (int i = 0; i < NC; i++) l[i] *= sc[i];
+        }
+      }
+      {
+        uint8_t* p = sP + (key_in >> 6) * (N * 128) + c0 * 128 + (key_in & 7) * 2;
+        const int chunk = (key_in & 63) >> 3;
+#pragma unroll
+        for (int i = 0; i < NC; i++) {
+          const float w = ex2(x[i] - m_used[i]);       // finite: the first block has a visible key
+          l[i] += w;
+          *(__half*)(p + i * 128 + ((chunk ^ (i & 7)) << 4)) = __float2half(w);      // c0 is a multiple of 8
         }
         fence_proxy_async_smem();
       }
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(smem_u32(p_full + b));
+      if (lane == 0) mbar_arrive(smem_u32(p_full));
     }
     if (nb > 0) {
-      ok = ok && mbar_wait(smem_u32(pv_done + ((nb - 1) & 1)), ((nb - 1) >> 1) & 1, abort_flag);
+      ok = ok && mbar_wait(smem_u32(pv_done), (nb - 1) & 1, abort_flag);
       ok = __all_sync(0xffffffffu, ok);
     }
-    if (scorer) {
+    // the sums of the four lane quarters, then the offsets, to shared memory (the buffer the last block did not use, then the other one)
+    float* part = s_part + (nb & 1) * 4 * N;
+    float* offs = s_part + ((nb & 1) ^ 1) * 4 * N;
+    {
       int col;
-      const float sum = reduce_columns<NC, false>(l, lane, col);
-      s_part[q * N + c0 + col] = sum;
+      const float sum = sum_columns<NC>(l, lane, col);
+      part[q * N + c0 + col] = sum;                    // the lanes of a column hold the same value
     }
     if (meet(ok)) {
+      if (q == 0 && lane == 0) {
+#pragma unroll
+        for (int i = 0; i < NC; i++) offs[c0 + i] = m_used[i];
+      }
+      meet(true);
       tc_fence_after();
       const size_t p_row = ((size_t)row * a.S + split) * a.H;
-      if (tid < N) {
-        float sum = s_part[tid] + s_part[N + tid];
+      if (tid < N && h0 + tid < a.H) {
+        const float sum = (part[tid] + part[N + tid]) + (part[2 * N + tid] + part[3 * N + tid]), m = offs[tid];
         if (a.S > 1) {
-          if (h0 + tid < a.H) {
-            a.part_ml[(p_row + h0 + tid) * 2] = m_used;
-            a.part_ml[(p_row + h0 + tid) * 2 + 1] = sum;
-          }
+          *(float2*)(a.part_ml + (p_row + h0 + tid) * 2) = make_float2(m, sum);
+        } else if (a.sinks) {
+          const float sk = a.sinks[h0 + tid] * kLog2e, mx = fmaxf(m, sk), c = ex2(m - mx);
+          s_inv[tid] = c / (sum * c + ex2(sk - mx));
         } else {
-          float inv;
-          if (a.sinks && h0 + tid < a.H) {
-            const float sk = a.sinks[h0 + tid] * kLog2e, mx = fmaxf(m_used, sk), c = ex2(m_used - mx);
-            inv = c / (sum * c + ex2(sk - mx));
-          } else {
-            inv = sum > 0.f ? 1.f / sum : 0.f;
-          }
-          s_sc[tid] = inv;
+          s_inv[tid] = sum > 0.f ? 1.f / sum : 0.f;
         }
       }
       meet(true);
@@ -519,8 +589,8 @@ __global__ void __launch_bounds__(kLThreads, 1) latent_decode_kernel(const __gri
             a.part[(p_row + h) * a.CR + d] = v;
           } else {
             const size_t at = (size_t)row * a.ldo + (size_t)h * a.CR + d;
-            if (a.out_f32) a.out_f32[at] = v * s_sc[c0 + k];
-            if (a.out_bf16) a.out_bf16[at] = __float2bfloat16(v * s_sc[c0 + k]);
+            if (a.out_f32) a.out_f32[at] = v * s_inv[c0 + k];
+            if (a.out_bf16) a.out_bf16[at] = __float2bfloat16(v * s_inv[c0 + k]);
           }
         }
       }
@@ -533,47 +603,71 @@ __global__ void __launch_bounds__(kLThreads, 1) latent_decode_kernel(const __gri
 }
 
 // Shares of the keys -> one output row per (row, head), with the sink's term.
+constexpr int kLShares = 64;
 __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentDecArgs a) {
+  __shared__ float s_w[kLShares];
   pdl_trigger();
   pdl_wait();
-  const int h = blockIdx.x, row = blockIdx.y;
+  const int h = blockIdx.x, row = blockIdx.y, lane = threadIdx.x & 31;
   const size_t p0 = (size_t)row * a.S * a.H + h;
-  float M = -INFINITY;
-  for (int s = 0; s < a.S; s++) M = fmaxf(M, a.part_ml[(p0 + (size_t)s * a.H) * 2]);
-  const float sk = a.sinks ? a.sinks[h] * kLog2e : -INFINITY, mx = fmaxf(M, sk);
-  float L = a.sinks ? ex2(sk - mx) : 0.f;
-  for (int s = 0; s < a.S; s++) {
-    const float m = a.part_ml[(p0 + (size_t)s * a.H) * 2];
-    if (m != -INFINITY) L += a.part_ml[(p0 + (size_t)s * a.H) * 2 + 1] * ex2(m - mx);
+  // every warp reads the shares' offsets and sums: one or two per lane
+  float2 ml[kLShares / 32];
+  float M = a.sinks ? a.sinks[h] * kLog2e : -INFINITY;
+#pragma unroll
+  for (int k = 0; k < kLShares / 32; k++) {
+    const int s = lane + 32 * k;
+    ml[k] = s < a.S ? *(const float2*)(a.part_ml + (p0 + (size_t)s * a.H) * 2) : make_float2(-INFINITY, 0.f);
   }
+#pragma unroll
+  for (int k = 0; k < kLShares / 32; k++) M = fmaxf(M, ml[k].x);
+  M = warp_max(M);
+  float L = 0.f, w[kLShares / 32];
+#pragma unroll
+  for (int k = 0; k < kLShares / 32; k++) {
+    w[k] = ml[k].x == -INFINITY ? 0.f : ex2(ml[k].x - M);
+    L += ml[k].y * w[k];
+  }
+  L = warp_sum(L);
+  if (a.sinks) L += ex2(a.sinks[h] * kLog2e - M);
   const float inv = L > 0.f ? 1.f / L : 0.f;
-  for (int d = threadIdx.x; d < a.CR; d += blockDim.x) {
-    float v = 0.f;
+  if (threadIdx.x < 32) {
+#pragma unroll
+    for (int k = 0; k < kLShares / 32; k++) s_w[lane + 32 * k] = w[k] * inv;
+  }
+  __syncthreads();
+  for (int d = threadIdx.x * 4; d < a.CR; d += blockDim.x * 4) {
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
     for (int s = 0; s < a.S; s++) {
-      const size_t p = p0 + (size_t)s * a.H;
-      const float m = a.part_ml[p * 2];
-      if (m != -INFINITY) v += a.part[p * a.CR + d] * ex2(m - mx);       // a share without keys has written nothing
+      const float f = s_w[s];
+      if (f == 0.f) continue;                          // a share without keys has written nothing
+      const float4 v = *(const float4*)(a.part + (p0 + (size_t)s * a.H) * a.CR + d);
+      o.x = fmaf(v.x, f, o.x); o.y = fmaf(v.y, f, o.y); o.z = fmaf(v.z, f, o.z); o.w = fmaf(v.w, f, o.w);
     }
     const size_t at = (size_t)row * a.ldo + (size_t)h * a.CR + d;
-    if (a.out_f32) a.out_f32[at] = v * inv;
-    if (a.out_bf16) a.out_bf16[at] = __float2bfloat16(v * inv);
+    if (a.out_f32) *(float4*)(a.out_f32 + at) = o;
+    if (a.out_bf16) {
+      const __nv_bfloat162 x = __floats2bfloat162_rn(o.x, o.y), y = __floats2bfloat162_rn(o.z, o.w);
+      *(uint2*)(a.out_bf16 + at) = make_uint2(*(const uint32_t*)&x, *(const uint32_t*)&y);
+    }
   }
 }
 
-size_t latent_smem(int N, int W, int stages) {
-  return 1024 + (size_t)stages * (W / 64) * kLBox + (size_t)(W / 64) * N * 128 + 2 * N * 128 + 18 * 8 + 4 * N * 4 + 8192;
+size_t latent_smem(int N, int CR, int RR, int pairs) {
+  const size_t boxes = (CR + RR) / 64;
+  return 1024 + (size_t)pairs * 2 * kLBox + (RR / 64) * kLBox + boxes * N * 128 + 2 * N * 128 + (2 * kLPairs + 12) * 8 + 9 * N * 4;
 }
-int latent_stages(int N, int W) {
-  int s = 4;
-  while (s > 1 && latent_smem(N, W, s) > 220 * 1024) s--;
-  return s;
+// Slots of the ring of pairs: as many as fit, 0 where not even one block does.
+int latent_pairs(int N, int CR, int RR) {
+  int p = kLPairs;
+  while (p > 0 && latent_smem(N, CR, RR, p) > 226 * 1024) p--;
+  return p >= (CR + 127) / 128 ? p : 0;
 }
 
 template <int N>
 int launch_latent(const CUtensorMap& tm, LatentDecArgs& a, int R, cudaStream_t st) {
-  const int W = a.CR + a.RR;
-  a.stages = latent_stages(N, W);
-  const size_t smem = latent_smem(N, W, a.stages);
+  a.pairs = latent_pairs(N, a.CR, a.RR);
+  const size_t smem = latent_smem(N, a.CR, a.RR, a.pairs);
   auto kern = latent_decode_kernel<N>;
   static size_t configured = 48 * 1024;
   if (smem > configured) {
@@ -590,7 +684,7 @@ int launch_latent(const CUtensorMap& tm, LatentDecArgs& a, int R, cudaStream_t s
 
 // Whether the tensor-core decode kernel takes these (padded) sizes.
 B200_API int b200_latent_decode_ok(int H, int CR, int RR) {
-  return CR >= 64 && CR % 64 == 0 && RR >= 64 && RR % 64 == 0 && CR <= 512 && latent_smem(H <= 16 ? 16 : 32, CR + RR, 2) <= 220 * 1024;
+  return CR >= 64 && CR % 64 == 0 && RR >= 64 && RR % 64 == 0 && CR <= 512 && latent_pairs(H <= 16 ? 16 : 32, CR, RR) > 0;
 }
 B200_API size_t b200_latent_decode_scratch_floats(int R, int H, int CR, int S) { return S > 1 ? (size_t)R * S * H * (CR + 2) : 0; }
 
@@ -598,7 +692,7 @@ B200_API size_t b200_latent_decode_scratch_floats(int R, int H, int CR, int S) {
 B200_API int b200_latent_decode(const float* q, const void* cache, const int* page_table, int max_pages, int n_pages, const int* row_seq,
                                 const int* pos, const float* sinks, int R, int H, int CR, int RR, int S, float* scratch, float* out_f32,
                                 void* out_bf16, int ldo, int* status, cudaStream_t st) {
-  if (R < 1 || H < 1 || S < 1 || !b200_latent_decode_ok(H, CR, RR) || (S > 1 && !scratch) || ldo < H * CR || (!out_f32 && !out_bf16))
+  if (R < 1 || H < 1 || S < 1 || S > kLShares || ldo % 4 || !b200_latent_decode_ok(H, CR, RR) || (S > 1 && !scratch) || ldo < H * CR || (!out_f32 && !out_bf16))
     return B200_ERR_BAD_ARG;
   CUtensorMap tm;
   const int rc = make_tmap_2d(&tm, cache, 2, (uint64_t)n_pages * 16, (uint64_t)(CR + RR), (uint64_t)(CR + RR) * 2, 16, 64, true);

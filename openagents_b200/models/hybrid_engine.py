@@ -401,9 +401,9 @@ class HybridEngine(PagedEngine):
         self.ctx_base[: len(base)].copy_(torch.tensor(base, dtype=torch.int32).pin_memory(), non_blocking=True)
 
     def _latent_splits(self, rows: int, heads: int, pages: int) -> int:
-        """Shares of the keys per row in the latent decode kernel: the fewest rounds over the SMs, a round costing its key blocks and a fixed set-up."""
-        ctas, blocks = rows * ((heads + 31) // 32), max(1, (min(pages, self.max_pages) * PAGE + 63) // 64)
-        cost = lambda s: -(-ctas * s // 148) * (-(-blocks // s) + 2)                       # noqa: E731
+        """Shares of the keys per row in the latent decode kernel: the fewest rounds over the SMs, a round costing its blocks of 128 keys and a fixed set-up."""
+        ctas, blocks = rows * ((heads + 31) // 32), max(1, (min(pages, self.max_pages) * PAGE + 127) // 128)
+        cost = lambda s: -(-ctas * s // 148) * (-(-blocks // s) + 1)                       # noqa: E731
         return min(range(1, max(1, min(self.max_splits, blocks, LATENT_CTAS // ctas)) + 1), key=cost)
 
     # ------------------------------------------------------------------ building blocks
@@ -429,7 +429,9 @@ class HybridEngine(PagedEngine):
     def _mm_heads(self, a: torch.Tensor, w: torch.Tensor, heads: int, head_k: int, out: torch.Tensor, head_ldc: int, alpha: float = 1.0, gate=None):
         """One product per head: w [heads * N][K]; head z reads columns z * head_k of ``a`` and writes columns z * head_ldc of ``out``."""
         N, K = w.shape[0] // heads, w.shape[1]
-        if a.dtype == torch.float32:
+        if a.dtype == torch.float32 and a.shape[0] <= MATVEC_MAX_TOKENS and K <= 1536:
+            ops.head_matvec(a, w, out, heads, head_k, head_ldc, alpha=alpha, gate=gate)
+        elif a.dtype == torch.float32:
             ops.gemm_f32(a, w, out, alpha=alpha, gate=gate, heads=heads, head_k=head_k, head_ldc=head_ldc)
         else:
             ops.gemm_heads(a, w, heads, N, K, head_k, out, head_ldc, alpha=alpha, gate=gate, status=self.status)

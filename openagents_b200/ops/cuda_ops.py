@@ -65,6 +65,7 @@ _SIGS = {
     "b200_attn_exact": [_P, _P, _P, c_int, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, c_int, c_int, c_int,
                         c_int, _P, _P],
     "b200_gemm_f32": [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, c_int, c_int, c_int, c_int, _P],
+    "b200_head_matvec": [_P, c_int, _P, c_int, _P] + [c_int] * 5 + [c_float, _P, c_int, c_int, c_int, _P],
     "b200_norm_dyt": [_P, c_int, c_int, _P, _P, c_int, _P, _P, _P, _P, _P, c_int, _P, c_long, _P],
     "b200_diff_combine": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_float, _P, _P, c_int, _P],
     "b200_latent_finish": [_P] + [c_int] * 10 + [_P, _P, c_float, _P, _P, _P, c_int, c_double, _P, _P, c_int, c_int, c_int, _P, c_int, _P],
@@ -408,6 +409,12 @@ def gemm_f32(A, W, out, act=0, alpha=1.0, accumulate=False, gate=None, heads=1, 
     M, (N, K) = A.shape[0], W.shape
     _check(lib().b200_gemm_f32(_p(A), A.stride(0), _p(W), W.stride(0), _p(out), out.stride(0), M, N // heads, K, act, alpha, int(accumulate), _p(gate),
                                0 if gate is None else gate.stride(0), heads, head_k, head_ldc, _st()), "gemm_f32")
+
+
+def head_matvec(A, W, out, heads, head_k, head_ldc, alpha=1.0, gate=None):
+    """:func:`gemm_heads` for 1..8 fp32 rows on the CUDA cores: ``W`` bf16 [heads * N, K]."""
+    _check(lib().b200_head_matvec(_p(A), A.stride(0), _p(W), W.stride(0), _p(out), out.stride(0), A.shape[0], heads, W.shape[0] // heads, W.shape[1], alpha,
+                                  _p(gate), 0 if gate is None else gate.stride(0), head_k, head_ldc, _st()), "head_matvec")
 
 
 def norm_dyt(x, alpha, w, b, hb=None, hf=None, ids=None, emb=None, zero=None):

@@ -103,6 +103,12 @@ def test_one_product_per_head(heads, N, K, head_k, head_ldc):
             ops.gemm_f32(a.float().to(DEV), w.to(DEV), out, alpha=0.7, gate=gd, heads=heads, head_k=head_k, head_ldc=head_ldc)
             got = out.view(M, heads, head_ldc)
             assert rel(got[..., :N], ref) < 1e-6 and (got[..., N:] == 9.0).all()
+            for rows in (1, 2, 3, 8):
+                if rows <= M:
+                    out = torch.full((M, heads * head_ldc), 9.0, device=DEV)
+                    ops.head_matvec(a[:rows].float().to(DEV), w.to(DEV), out, heads, head_k, head_ldc, alpha=0.7, gate=None if gd is None else gd[:rows])
+                    got = out.view(M, heads, head_ldc)
+                    assert rel(got[:rows, :, :N], ref[:rows]) < 1e-6 and (got[..., N:] == 9.0).all() and (got[rows:] == 9.0).all()
 
 
 # ---------------------------------------------------------------- chunked differential attention
