@@ -68,6 +68,7 @@ struct GemmEpi {
   int act;
   int accumulate;            // out_f32 += value
   float alpha;               // multiplies the product, ahead of everything else
+  const float* col_scale;    // [N] or null: multiplies what is stored or added, last (but for the residual)
   int half_out;              // out_bf16 is stored as fp16 instead
   const float* gate;         // [M][ldg] or null: the result is multiplied by sigmoid(gate[m][n]) (n: output column)
   int ldg;
@@ -135,12 +136,14 @@ __device__ __forceinline__ void epilogue_chunk_red(const GemmEpi& e, float* stag
     const bool sym = e.sym_mode != SYM_NONE;
     float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
     if (e.bias && first_split && (!sym || e.sym.rank == 0)) b = *(const float4*)(e.bias + n);
+    const float4 cs = e.col_scale ? *(const float4*)(e.col_scale + n) : make_float4(1.f, 1.f, 1.f, 1.f);
 #pragma unroll
     for (int i = 0; i < 8; i++) {
       const int row = (lane >> 3) + 4 * i, m = m_warp0 + row;
       if (m >= M) break;
       float4 o = *(const float4*)(stage + row * 32 + ((c4 ^ (row & 7)) << 2));
       o.x = fmaf(o.x, e.alpha, b.x); o.y = fmaf(o.y, e.alpha, b.y); o.z = fmaf(o.z, e.alpha, b.z); o.w = fmaf(o.w, e.alpha, b.w);
+      if (e.col_scale) { o.x *= cs.x; o.y *= cs.y; o.z *= cs.z; o.w *= cs.w; }
       if (!sym) {
         asm volatile("red.relaxed.gpu.global.add.v4.f32 [%0], {%1,%2,%3,%4};" ::"l"(e.out_f32 + (size_t)m * e.ldc + n),
                      "f"(o.x), "f"(o.y), "f"(o.z), "f"(o.w) : "memory");
@@ -156,12 +159,13 @@ __device__ __forceinline__ void epilogue_chunk_red(const GemmEpi& e, float* stag
 
 // moe_mode 1: 32 accumulator columns are 16 (gate, up) pairs of one row.
 __device__ __forceinline__ void epilogue_row_swiglu(const GemmEpi& e, int m, int n0, const uint32_t (&r)[32]) {
+  const float w = e.moe_mode == 1 && e.gate_w ? e.gate_w[m] : 1.f;
   uint4 o[2];
   __nv_bfloat162* p = (__nv_bfloat162*)o;
 #pragma unroll
   for (int j = 0; j < 8; j++) {
-    const float g0 = __uint_as_float(r[4 * j]), u0 = __uint_as_float(r[4 * j + 1]);
-    const float g1 = __uint_as_float(r[4 * j + 2]), u1 = __uint_as_float(r[4 * j + 3]);
+    const float g0 = w * __uint_as_float(r[4 * j]), u0 = w * __uint_as_float(r[4 * j + 1]);
+    const float g1 = w * __uint_as_float(r[4 * j + 2]), u1 = w * __uint_as_float(r[4 * j + 3]);
     p[j] = __floats2bfloat162_rn(silu(g0) * u0, silu(g1) * u1);
   }
   uint4* dst = (uint4*)(e.out_bf16 + (size_t)m * e.ldc + (n0 >> 1));
@@ -181,14 +185,15 @@ __device__ __forceinline__ void epilogue_chunk_combine(const GemmEpi& e, float* 
   __syncwarp();
   const int c4 = lane & 7, n = n0 + c4 * 4;
   if (n < N) {
+    const float4 cs = e.col_scale ? *(const float4*)(e.col_scale + n) : make_float4(1.f, 1.f, 1.f, 1.f);
 #pragma unroll
     for (int i = 0; i < 8; i++) {
       const int row = (lane >> 3) + 4 * i, m = m_warp0 + row;
       if (m >= live_end) break;
       const int dst = e.meta[2 * m], tok = e.meta[2 * m + 1];
-      const float w = e.gate_w[m];
+      const float w = e.gate_w ? e.gate_w[m] : 1.f;
       float4 o = *(const float4*)(stage + row * 32 + ((c4 ^ (row & 7)) << 2));
-      o.x *= w; o.y *= w; o.z *= w; o.w *= w;
+      o.x *= w * cs.x; o.y *= w * cs.y; o.z *= w * cs.z; o.w *= w * cs.w;
       sym_red_to_f32x4(e.sym, dst, e.sym_off + ((size_t)tok * e.ldc + n) * 4, o);
     }
   }
@@ -207,7 +212,7 @@ __device__ __forceinline__ void epilogue_col(const GemmEpi& e, int n, int t0, in
                                              const uint32_t (&r)[32], bool first_split) {
   if (n >= n_cols) return;
   const bool sym = e.sym_mode != SYM_NONE;
-  const float b = (e.bias && first_split && (!sym || e.sym.rank == 0)) ? e.bias[n] : 0.f;
+  const float b = (e.bias && first_split && (!sym || e.sym.rank == 0)) ? e.bias[n] : 0.f, cs = e.col_scale ? e.col_scale[n] : 1.f;
   // fully unrolled with a predicate per row: an index that is not a compile-time constant would put r[] on the stack
 #pragma unroll
   for (int j = 0; j < 32; j++) {
@@ -224,11 +229,12 @@ __device__ __forceinline__ void epilogue_col(const GemmEpi& e, int n, int t0, in
     }
     const size_t idx = (size_t)t * e.ldc + n;
     if (e.splitk_red) {
-      asm volatile("red.relaxed.gpu.global.add.f32 [%0], %1;" ::"l"(e.out_f32 + idx), "f"(x) : "memory");
+      asm volatile("red.relaxed.gpu.global.add.f32 [%0], %1;" ::"l"(e.out_f32 + idx), "f"(x * cs) : "memory");
       continue;
     }
     x = activate(e.act, x);
     if (e.gate) x *= 1.f / (1.f + __expf(-e.gate[(size_t)t * e.ldg + n]));
+    x *= cs;
     if (e.resid_f32) x += e.resid_f32[idx];
     if (e.resid_bf16) x += __bfloat162float(e.resid_bf16[idx]);
     if (e.out_f32) e.out_f32[idx] = e.accumulate ? e.out_f32[idx] + x : x;
@@ -257,6 +263,10 @@ __device__ __forceinline__ void epilogue_row(const GemmEpi& e, int m, int n0, in
       if (add_bias) {
         const float4 b = *(const float4*)(e.bias + n0 + j);
         o.x += b.x; o.y += b.y; o.z += b.z; o.w += b.w;
+      }
+      if (e.col_scale) {
+        const float4 c = *(const float4*)(e.col_scale + n0 + j);
+        o.x *= c.x; o.y *= c.y; o.z *= c.z; o.w *= c.w;
       }
       asm volatile("red.relaxed.gpu.global.add.v4.f32 [%0], {%1,%2,%3,%4};" ::"l"(e.out_f32 + base + j), "f"(o.x),
                    "f"(o.y), "f"(o.z), "f"(o.w) : "memory");
@@ -317,6 +327,13 @@ __device__ __forceinline__ void epilogue_row(const GemmEpi& e, int m, int n0, in
         v[j + 2] *= 1.f / (1.f + __expf(-g.z)); v[j + 3] *= 1.f / (1.f + __expf(-g.w));
       }
     }
+    if (e.col_scale) {
+#pragma unroll
+      for (int j = 0; j < 32; j += 4) {
+        const float4 b = *(const float4*)(e.col_scale + n0 + j);
+        v[j] *= b.x; v[j + 1] *= b.y; v[j + 2] *= b.z; v[j + 3] *= b.w;
+      }
+    }
     if (e.resid_f32) {
 #pragma unroll
       for (int j = 0; j < 32; j += 4) {
@@ -373,6 +390,7 @@ __device__ __forceinline__ void epilogue_row(const GemmEpi& e, int m, int n0, in
       if (e.bias) x += e.bias[n0 + j];
       x = activate(e.act, x);
       if (e.gate) x *= 1.f / (1.f + __expf(-e.gate[(size_t)m * e.ldg + n0 + j]));
+      if (e.col_scale) x *= e.col_scale[n0 + j];
       if (e.resid_f32) x += e.resid_f32[base + j];
       if (e.resid_bf16) x += __bfloat162float(e.resid_bf16[base + j]);
       if (e.out_f32) e.out_f32[base + j] = e.accumulate ? e.out_f32[base + j] + x : x;
@@ -682,14 +700,15 @@ B200_API int b200_gemm_bf16(const void* A, const void* B, int M, int N, int K, i
                             void* out_bf16, int ldc, const float* bias, const float* resid_f32,
                             const void* resid_bf16, int act, int accumulate, int tile_n, int split_k, int* status,
                             int sym_mode, const SymTable* sym, size_t sym_off, int rows_per_rank, int wait_ready,
-                            int ag_rows_per_rank, int ag_epoch, int mn_major, float alpha, int half_out, cudaStream_t st) {
+                            int ag_rows_per_rank, int ag_epoch, int mn_major, float alpha, int half_out, const float* col_scale,
+                            cudaStream_t st) {
   if (M <= 0 || N <= 0 || K <= 0 || (lda % 8) || (ldb % 8) || (!mn_major && (K % 8))) return B200_ERR_BAD_ARG;
   if (mn_major) {
     // D[M][N] = sum_k A[k][m] * B[k][n]: A is [K][M] (row stride lda), B is [K][N] (row stride ldb).  Plain epilogues only.
     if (sym_mode != SYM_NONE || ag_rows_per_rank || tile_n < 0 || split_k > 1 || act == ACT_SWIGLU_PAIR || (M % 8) || (N % 8))
       return B200_ERR_BAD_ARG;
     if ((out_bf16 && (ldc % 8)) || (out_f32 && (ldc % 4)) || (N % 4)) return B200_ERR_BAD_ARG;
-    if (alpha != 1.f || half_out) return B200_ERR_BAD_ARG;
+    if (alpha != 1.f || half_out || col_scale) return B200_ERR_BAD_ARG;
     CUtensorMap ta, tb;
     int rc = make_tmap_2d(&ta, A, 2, (uint64_t)K, (uint64_t)M, (uint64_t)lda * 2, BK, 64, true);
     if (rc) return rc;
@@ -705,7 +724,7 @@ B200_API int b200_gemm_bf16(const void* A, const void* B, int M, int N, int K, i
     return launch_gemm<128, 6, 128, 1, true>(ta, tb, e, M, N, K, 1, status, st);
   }
   if ((out_bf16 && (ldc % 8)) || (out_f32 && (ldc % 4))) return B200_ERR_BAD_ARG;
-  if (N % 4) return B200_ERR_BAD_ARG;
+  if (N % 4 || (col_scale && (sym_mode != SYM_NONE || act == ACT_SWIGLU_PAIR || ((uintptr_t)col_scale & 15)))) return B200_ERR_BAD_ARG;
   if (sym_mode != SYM_NONE && (!sym || (ldc % 4) || (sym_off % 16))) return B200_ERR_BAD_ARG;
   if (ag_rows_per_rank < 0 || (ag_rows_per_rank > 0 && (!sym || tile_n == -1))) return B200_ERR_BAD_ARG;
   if (act == ACT_SWIGLU_PAIR && (!out_bf16 || out_f32 || bias || resid_f32 || resid_bf16 || accumulate || sym_mode != SYM_NONE ||
@@ -750,7 +769,7 @@ B200_API int b200_gemm_bf16(const void* A, const void* B, int M, int N, int K, i
   rc = make_tmap_2d(&tb, B, 2, (uint64_t)N, (uint64_t)K, (uint64_t)ldb * 2, (uint32_t)tile_n, BK, true);
   if (rc) return rc;
   GemmEpi e = {};
-  e.alpha = alpha; e.half_out = half_out;
+  e.alpha = alpha; e.half_out = half_out; e.col_scale = col_scale;
   e.out_f32 = out_f32; e.out_bf16 = (__nv_bfloat16*)out_bf16; e.bias = bias; e.resid_f32 = resid_f32;
   e.resid_bf16 = (const __nv_bfloat16*)resid_bf16; e.ldc = ldc; e.act = act; e.accumulate = accumulate;
   e.sym_mode = sym_mode; e.rows_per_rank = rows_per_rank > 0 ? rows_per_rank : 1; e.sym_off = sym_off;
@@ -824,19 +843,25 @@ B200_API int b200_gemm_heads(const void* A, const void* B, int M, int heads, int
 // stride lda) holds each expert's gathered tokens, B [groups * N][K] bf16 its weights, counts[g] the
 // live rows of group g (device memory, final before this kernel starts).
 //   mode 1: B rows are interleaved (gate_0, up_0, gate_1, ...), N = 2 * ffn; out_bf16 [rows][ldc] gets
-//           silu(gate) * up, N / 2 columns per row.
+//           silu(gate) * up, N / 2 columns per row; with gate_w, row m's weight multiplies the expert's INPUT
+//           (gate and up ahead of the activation).
 //   mode 2: N = d_model; row m is added, scaled by gate_w[m], into token meta[2m+1] of rank meta[2m]:
 //           fp32 [tokens][ldc] at byte offset sym_off of that rank's symmetric heap.  The kernel ends
-//           with the cross-rank barrier, so afterwards every rank's residual stream is complete.
+//           with the cross-rank barrier, so afterwards every rank's residual stream is complete.  gate_w null:
+//           weights of one.  sym null: one rank, sym_off is the destination's address.  col_scale [N] (or null)
+//           multiplies what is added.
+// live_rows: the most rows all groups hold together (0: unknown), which bounds the list of live tiles.
 B200_API int b200_moe_gemm(const void* A, const void* B, int groups, int group_rows, int N, int K, int lda, int ldb,
                            const int* counts, int mode, void* out_bf16, int ldc, const int* meta, const float* gate_w,
-                           const SymTable* sym, size_t sym_off, int* status, cudaStream_t st) {
+                           const SymTable* sym, size_t sym_off, const float* col_scale, long live_rows, int* status, cudaStream_t st) {
   if (groups <= 0 || group_rows <= 0 || group_rows % BM || N <= 0 || K <= 0 || (lda % 8) || (ldb % 8) || (K % 8) || (N % 4))
     return B200_ERR_BAD_ARG;
-  if (mode == 1 ? (!out_bf16 || (ldc % 8) || (N % 32)) : (mode != 2 || !meta || !gate_w || !sym || (ldc % 4) || (sym_off % 16)))
+  if (mode == 1 ? (!out_bf16 || (ldc % 8) || (N % 32)) : (mode != 2 || !meta || (ldc % 4) || (sym_off % 16)))
     return B200_ERR_BAD_ARG;
   const int M = groups * group_rows;
-  if ((long)groups * (group_rows / BM) > kMaxLiveTiles) return B200_ERR_BAD_ARG;
+  if (mode == 2 && !sym && !sym_off) return B200_ERR_BAD_ARG;
+  const long tiles = (long)groups * (group_rows / BM), live_tiles = live_rows > 0 ? live_rows / BM + groups : tiles;
+  if (min(tiles, live_tiles) > kMaxLiveTiles || ((uintptr_t)col_scale & 15)) return B200_ERR_BAD_ARG;
   CUtensorMap ta, tb;
   int rc = make_tmap_2d(&ta, A, 2, (uint64_t)M, (uint64_t)K, (uint64_t)lda * 2, BM, BK, true);
   if (rc) return rc;
@@ -847,7 +872,10 @@ B200_API int b200_moe_gemm(const void* A, const void* B, int groups, int group_r
   e.group_rows = group_rows; e.group_n = N; e.group_counts = counts; e.moe_mode = mode; e.meta = meta; e.gate_w = gate_w;
   e.rows_per_rank = 1;
   e.alpha = 1.f;
-  if (mode == 2) {
+  e.col_scale = mode == 2 ? col_scale : nullptr;
+  if (mode == 2 && !sym) {            // the rows' own memory: the offset is an address
+    e.sym_off = sym_off;
+  } else if (mode == 2) {
     e.sym_mode = SYM_ALLREDUCE;   // only so that the kernel ends with the cross-rank barrier
     e.sym = *sym;
     e.sym_off = sym_off;

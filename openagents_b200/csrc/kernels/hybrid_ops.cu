@@ -255,6 +255,236 @@ B200_API int b200_norm_dyt(float* x, int T, int D, const int* ids, const void* e
   return launch_pdl(vec ? norm_dyt_vec_kernel : norm_dyt_kernel, dim3(T, gy), dim3(threads), 0, st, a);
 }
 
+// ------------------------------------------------------------------ depth average and the norms behind it
+
+// Per row:  x = sum over j < n of w[j] * X_j   (X_j: row t of xs + j * stride; the embedding output and every layer's result so far)
+//           out = x + add                     (the next layer adds its results to this row: `add` is a bias they carry, or null)
+//           h1 = x / rms(x) * g1, h2 = x / rms(x) * g2   (two norms of the same x; each given or not; bf16 or fp32)
+// Rows are ld floats apart in xs, out and h, D of them live; the others are written as zeros.  zero: a buffer cleared on the side.
+struct DepthArgs {
+  const float* xs;
+  size_t stride;
+  const float* w;          // [n] or null (n = 1: x = X_0)
+  int n, D, ld;
+  float* out;              // or null
+  const float* add;        // [D] or null
+  const float* g1;         // [D] or null
+  const float* g2;
+  float eps;
+  __nv_bfloat16* hb1;
+  __nv_bfloat16* hb2;
+  float* hf1;
+  float* hf2;
+  float4* zero;
+  int nz4;
+};
+__global__ void __launch_bounds__(256) depth_norm_kernel(const DepthArgs a) {
+  extern __shared__ float depth_row[];               // [D]
+  __shared__ float red[32];
+  const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+  pdl_trigger();
+  pdl_wait();
+  for (int i = blockIdx.x * nt + tid; i < a.nz4; i += gridDim.x * nt) a.zero[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+  const size_t at = (size_t)t * a.ld;
+  float ss = 0.f;
+  for (int i = tid; i < a.ld; i += nt) {
+    float v = 0.f;
+    if (i < a.D) {
+      const float* x = a.xs + at + i;
+      if (!a.w) v = *x;
+      else
+        for (int j = 0; j < a.n; j++) v = fmaf(a.w[j], x[j * a.stride], v);
+      depth_row[i] = v;
+      ss += v * v;
+    }
+    if (a.out) a.out[at + i] = i < a.D && a.add ? v + a.add[i] : v;
+  }
+  if (!a.g1 && !a.g2) return;
+  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)a.D + a.eps);
+  for (int i = tid; i < a.ld; i += nt) {               // every thread meets the elements it wrote
+    const float v = i < a.D ? depth_row[i] * r : 0.f;
+    if (a.g1) {
+      const float o = i < a.D ? v * a.g1[i] : 0.f;
+      if (a.hb1) a.hb1[at + i] = __float2bfloat16(o);
+      if (a.hf1) a.hf1[at + i] = o;
+    }
+    if (a.g2) {
+      const float o = i < a.D ? v * a.g2[i] : 0.f;
+      if (a.hb2) a.hb2[at + i] = __float2bfloat16(o);
+      if (a.hf2) a.hf2[at + i] = o;
+    }
+  }
+}
+// The same on 16-byte accesses with the row in registers (widths that are multiples of 4).
+template <int R>
+__global__ void __launch_bounds__(256) depth_norm_vec_kernel(const DepthArgs a) {
+  __shared__ float red[32];
+  const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x, D4 = a.D >> 2, l4 = a.ld >> 2;
+  const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+  pdl_trigger();
+  pdl_wait();
+  for (int i = blockIdx.x * nt + tid; i < a.nz4; i += gridDim.x * nt) a.zero[i] = z;
+  const size_t at = (size_t)t * l4;
+  float4 v[R];
+#pragma unroll
+  for (int k = 0; k < R; k++) v[k] = z;
+  const float4* x = (const float4*)a.xs + at;
+  const size_t s4 = a.stride >> 2;
+  if (!a.w) {
+#pragma unroll
+    for (int k = 0; k < R; k++)
+      if (tid + k * nt < D4) v[k] = x[tid + k * nt];
+  } else {
+    constexpr int U = R >= 4 ? 2 : 8 / R;             // layers in flight
+    for (int j0 = 0; j0 < a.n; j0 += U) {
+      float4 e[U][R];
+      float w[U];
+#pragma unroll
+      for (int u = 0; u < U; u++) {
+        w[u] = j0 + u < a.n ? a.w[j0 + u] : 0.f;
+#pragma unroll
+        for (int k = 0; k < R; k++) e[u][k] = j0 + u < a.n && tid + k * nt < D4 ? x[(j0 + u) * s4 + tid + k * nt] : z;
+      }
+#pragma unroll
+      for (int u = 0; u < U; u++)
+#pragma unroll
+        for (int k = 0; k < R; k++) {
+          v[k].x = fmaf(w[u], e[u][k].x, v[k].x);
+          v[k].y = fmaf(w[u], e[u][k].y, v[k].y);
+          v[k].z = fmaf(w[u], e[u][k].z, v[k].z);
+          v[k].w = fmaf(w[u], e[u][k].w, v[k].w);
+        }
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < R; k++) {
+    const int i = tid + k * nt;
+    ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    if (a.out && i < l4) {
+      const float4 b = a.add && i < D4 ? ((const float4*)a.add)[i] : z;
+      ((float4*)a.out)[at + i] = make_float4(v[k].x + b.x, v[k].y + b.y, v[k].z + b.z, v[k].w + b.w);
+    }
+  }
+  if (!a.g1 && !a.g2) return;
+  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)a.D + a.eps);
+  auto put = [&](const float* g, __nv_bfloat16* hb, float* hf) {
+#pragma unroll
+    for (int k = 0; k < R; k++) {
+      const int i = tid + k * nt;
+      if (i >= l4) continue;
+      const float4 w = i < D4 ? ((const float4*)g)[i] : z;
+      const float4 o = make_float4(v[k].x * r * w.x, v[k].y * r * w.y, v[k].z * r * w.z, v[k].w * r * w.w);
+      if (hb) {
+        const __nv_bfloat162 p0 = __floats2bfloat162_rn(o.x, o.y), p1 = __floats2bfloat162_rn(o.z, o.w);
+        *(uint2*)(hb + (at + i) * 4) = make_uint2(*(const uint32_t*)&p0, *(const uint32_t*)&p1);
+      }
+      if (hf) ((float4*)hf)[at + i] = o;
+    }
+  };
+  if (a.g1) put(a.g1, a.hb1, a.hf1);
+  if (a.g2) put(a.g2, a.hb2, a.hf2);
+}
+// xs fp32: n slabs `stride` floats apart, rows ld apart.  Outputs share ld.
+B200_API int b200_depth_norm(const float* xs, size_t stride, const float* w, int n, int T, int D, int ld, float* out, const float* add,
+                             const float* g1, const float* g2, float eps, void* hb1, void* hb2, float* hf1, float* hf2, float* zero,
+                             long zero_n, cudaStream_t st) {
+  if (T < 1 || D < 1 || ld < D || n < 1 || !xs || (!w && n != 1) || (g1 && !hb1 && !hf1) || (g2 && !hb2 && !hf2)) return B200_ERR_BAD_ARG;
+  if (zero && (zero_n % 4 || (uintptr_t)zero % 16)) return B200_ERR_BAD_ARG;
+  DepthArgs a;
+  a.xs = xs; a.stride = stride; a.w = w; a.n = n; a.D = D; a.ld = ld; a.out = out; a.add = add; a.g1 = g1; a.g2 = g2; a.eps = eps;
+  a.hb1 = (__nv_bfloat16*)hb1; a.hb2 = (__nv_bfloat16*)hb2; a.hf1 = hf1; a.hf2 = hf2; a.zero = (float4*)zero; a.nz4 = zero ? (int)(zero_n / 4) : 0;
+  const uintptr_t align = (uintptr_t)xs | (uintptr_t)out | (uintptr_t)add | (uintptr_t)g1 | (uintptr_t)g2 | (uintptr_t)hb1 | (uintptr_t)hb2 |
+                          (uintptr_t)hf1 | (uintptr_t)hf2;
+  if (align % 16 == 0 && D % 4 == 0 && ld % 4 == 0 && stride % 4 == 0 && ld <= 256 * 4 * 8) {
+    const int n4 = ld / 4, nt = n4 > 128 ? 256 : n4 > 64 ? 128 : 64, R = (n4 + nt - 1) / nt;
+    auto kern = R <= 1 ? depth_norm_vec_kernel<1> : R <= 2 ? depth_norm_vec_kernel<2> : R <= 4 ? depth_norm_vec_kernel<4> : depth_norm_vec_kernel<8>;
+    return launch_pdl(kern, dim3(T), dim3(nt), 0, st, a);
+  }
+  const size_t smem = (size_t)D * 4;
+  if (smem > 200 * 1024) return B200_ERR_BAD_ARG;
+  static size_t configured = 48 * 1024;
+  if (smem > configured) {
+    cudaError_t e = cudaFuncSetAttribute(depth_norm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    configured = smem;
+  }
+  return launch_pdl(depth_norm_kernel, dim3(T), dim3(256), smem, st, a);
+}
+
+// ------------------------------------------------------------------ PolyNorm
+
+// Per row of F values z:  a N(z) + b N(z^2) + c N(z^3) + e, N dividing a row by its root mean square (powers element by element), with
+// coef = (a, b, c, e).  in fp32 [T][ldi]; out bf16 or fp32 [T][ldo], columns F..ldo zero.
+constexpr int kPolyRegs = 8;
+__global__ void __launch_bounds__(512) poly_norm_kernel(const float* __restrict__ in, int ldi, int F, const float* __restrict__ coef, float eps,
+                                                        __nv_bfloat16* __restrict__ ob, float* __restrict__ of, int ldo, int vec) {
+  __shared__ float red[3][32];
+  const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+  const float ca = coef[0], cb = coef[1], cc = coef[2], ce = coef[3];
+  pdl_trigger();
+  pdl_wait();
+  const float* zr = in + (size_t)t * ldi;
+  const int F4 = F >> 2;
+  float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+  auto stat = [&](float z) {
+    const float z2 = z * z;
+    s2 += z2;
+    s4 = fmaf(z2, z2, s4);
+    s6 = fmaf(z2 * z2, z2, s6);
+  };
+  float4 v[kPolyRegs];                                  // vec: the first part of the row stays in registers
+  if (vec) {
+#pragma unroll
+    for (int k = 0; k < kPolyRegs; k++) {
+      const int i = tid + k * nt;
+      v[k] = i < F4 ? ((const float4*)zr)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int k = 0; k < kPolyRegs; k++) { stat(v[k].x); stat(v[k].y); stat(v[k].z); stat(v[k].w); }
+    for (int i = tid + kPolyRegs * nt; i < F4; i += nt) {
+      const float4 e = ((const float4*)zr)[i];
+      stat(e.x); stat(e.y); stat(e.z); stat(e.w);
+    }
+  } else {
+    for (int i = tid; i < F; i += nt) stat(zr[i]);
+  }
+  const int lane = tid & 31, w = tid >> 5, nw = nt >> 5;
+  s2 = warp_sum(s2); s4 = warp_sum(s4); s6 = warp_sum(s6);
+  if (lane == 0) { red[0][w] = s2; red[1][w] = s4; red[2][w] = s6; }
+  __syncthreads();
+  s2 = warp_sum(lane < nw ? red[0][lane] : 0.f);
+  s4 = warp_sum(lane < nw ? red[1][lane] : 0.f);
+  s6 = warp_sum(lane < nw ? red[2][lane] : 0.f);
+  const float a1 = ca / sqrtf(s2 / (float)F + eps), a2 = cb / sqrtf(s4 / (float)F + eps), a3 = cc / sqrtf(s6 / (float)F + eps);
+  auto f = [&](float z) { return fmaf(z, fmaf(z, fmaf(z, a3, a2), a1), ce); };
+  if (vec) {
+    auto store = [&](int i, float4 z) {
+      const float4 o = make_float4(f(z.x), f(z.y), f(z.z), f(z.w));
+      if (ob) {
+        const __nv_bfloat162 p0 = __floats2bfloat162_rn(o.x, o.y), p1 = __floats2bfloat162_rn(o.z, o.w);
+        *(uint2*)(ob + (size_t)t * ldo + 4 * i) = make_uint2(*(const uint32_t*)&p0, *(const uint32_t*)&p1);
+      }
+      if (of) *(float4*)(of + (size_t)t * ldo + 4 * i) = o;
+    };
+#pragma unroll
+    for (int k = 0; k < kPolyRegs; k++)
+      if (tid + k * nt < F4) store(tid + k * nt, v[k]);
+    for (int i = tid + kPolyRegs * nt; i < F4; i += nt) store(i, ((const float4*)zr)[i]);
+  }
+  for (int i = (vec ? F : 0) + tid; i < ldo; i += nt) {
+    const float o = i < F ? f(zr[i]) : 0.f;
+    if (ob) ob[(size_t)t * ldo + i] = __float2bfloat16(o);
+    if (of) of[(size_t)t * ldo + i] = o;
+  }
+}
+B200_API int b200_poly_norm(const float* in, int ldi, int T, int F, const float* coef, float eps, void* ob, float* of, int ldo, cudaStream_t st) {
+  if (T < 1 || F < 1 || ldi < F || ldo < F || !in || !coef || (!ob && !of) || of == in) return B200_ERR_BAD_ARG;
+  const int vec = F % 4 == 0 && ldi % 4 == 0 && ldo % 4 == 0 && (((uintptr_t)in | (uintptr_t)ob | (uintptr_t)of) & 15) == 0;
+  const int threads = F >= 4096 ? 512 : F >= 1024 ? 256 : 128;
+  return launch_pdl(poly_norm_kernel, dim3(T), dim3(threads), 0, st, in, ldi, F, coef, eps, (__nv_bfloat16*)ob, of, ldo, vec);
+}
+
 // ------------------------------------------------------------------ attention: finish of the projections
 
 // One warp per (token, head) of a fused projection row: queries and keys are rotated on their first `rot` dimensions, then
@@ -266,7 +496,7 @@ B200_API int b200_norm_dyt(float* x, int T, int D, const int* ids, const void* e
 // both key rows and zero on the other map's half, so that one product with them gives its own map's scores.
 struct QkvArgs {
   const float* in;         // [T][ld]
-  int ld, q_off, k_off, v_off;     // k_off < 0: the layer has no keys and values of its own
+  int ld, q_off, k_off, v_off;     // k_off < 0: the layer has no keys and values of its own; v_off < 0: its values are its keys
   const int* pos;
   const int* slot;         // physical cache slot (page * page_size + offset); < 0: no cache write
   const float2* tab;       // [tab_len][rot / 2] (cos, sin)
@@ -290,7 +520,7 @@ __global__ void __launch_bounds__(128) qkv_finish_kernel(const QkvArgs a, CT* __
   pdl_wait();
   const int t = blockIdx.x, lane = threadIdx.x & 31;
   const int KR = a.G * a.maps;                            // key rows
-  const int n_heads = a.H + (a.k_off >= 0 ? KR + a.G : 0);
+  const int n_heads = a.H + (a.k_off >= 0 ? KR + (a.v_off >= 0 ? a.G : 0) : 0);
   const int hh = blockIdx.y * 4 + (threadIdx.x >> 5);
   if (hh >= n_heads) return;
   const int s = a.slot[t];
@@ -392,7 +622,7 @@ __global__ void __launch_bounds__(256) qkv_copy_kernel(const QkvArgs a, CT* __re
   pdl_wait();
   const int t = blockIdx.x, i = blockIdx.y * 256 + threadIdx.x;
   const int KR = a.G * a.maps, qw = a.q_wide ? a.maps * a.DK : a.DK, q4 = qw >> 2, k4 = a.DK >> 2, v4 = a.DV >> 2;
-  const int nq = a.H * q4, nk = a.k_off >= 0 ? KR * k4 : 0, nv = a.k_off >= 0 ? a.G * v4 : 0;
+  const int nq = a.H * q4, nk = a.k_off >= 0 ? KR * k4 : 0, nv = a.k_off >= 0 && a.v_off >= 0 ? a.G * v4 : 0;
   if (i >= nq + nk + nv) return;
   const float* row = a.in + (size_t)t * a.ld;
   int hh, c, col;
@@ -442,21 +672,21 @@ B200_API int b200_qkv_finish(const float* in, int ld, int T, int q_off, int k_of
                              void* vc, int cache_f32, int maps, int q_wide, const float* bias, cudaStream_t st) {
   if (T < 1 || H < 1 || G < 1 || dim < 1 || vdim < 1 || dim > DK || vdim > DV || DK > 64 * kQkvPairs || (rot & 1) || rot > dim || rot < 0)
     return B200_ERR_BAD_ARG;
-  if ((k_off >= 0 && (!kc || !vc)) || (!q32 && !q16) || page_size < 1) return B200_ERR_BAD_ARG;
+  if ((k_off >= 0 && (!kc || (v_off >= 0 && !vc))) || (!q32 && !q16) || page_size < 1) return B200_ERR_BAD_ARG;
   if (maps < 1 || H % (G * maps) || (q_wide && q16)) return B200_ERR_BAD_ARG;
   QkvArgs a;
   a.in = in; a.ld = ld; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off; a.pos = pos; a.slot = slot; a.tab = (const float2*)tab;
   a.tab_len = tab ? tab_len : 0; a.base = base; a.H = H; a.G = G; a.dim = dim; a.vdim = vdim; a.DK = DK; a.DV = DV; a.rot = rot;
   a.style = style; a.qk_norm = qk_norm; a.page_size = page_size; a.eps = eps; a.q_scale = q_scale; a.q32 = q32; a.q16 = (__half*)q16;
   a.maps = maps; a.q_wide = q_wide; a.bias = bias;
-  if (rot == 0 && !qk_norm && ((ld | q_off | dim | vdim | DK | DV) & 3) == 0 && (k_off < 0 || ((k_off | v_off) & 3) == 0) &&
+  if (rot == 0 && !qk_norm && ((ld | q_off | dim | vdim | DK | DV) & 3) == 0 && (k_off < 0 || ((k_off | max(v_off, 0)) & 3) == 0) &&
       (((uintptr_t)in | (uintptr_t)bias | (uintptr_t)q32 | (uintptr_t)q16 | (uintptr_t)kc | (uintptr_t)vc) & 15) == 0) {
-    const int quads = (H * (q_wide ? maps : 1) * DK + (k_off >= 0 ? G * (maps * DK + DV) : 0)) / 4;
+    const int quads = (H * (q_wide ? maps : 1) * DK + (k_off >= 0 ? G * (maps * DK + (v_off >= 0 ? DV : 0)) : 0)) / 4;
     const dim3 g(T, (quads + 255) / 256);
     if (cache_f32) return launch_pdl(qkv_copy_kernel<float>, g, dim3(256), 0, st, a, (float*)kc, (float*)vc);
     return launch_pdl(qkv_copy_kernel<__half>, g, dim3(256), 0, st, a, (__half*)kc, (__half*)vc);
   }
-  const int n_heads = H + (k_off >= 0 ? (maps + 1) * G : 0);
+  const int n_heads = H + (k_off >= 0 ? (maps + (v_off >= 0)) * G : 0);
   const dim3 grid(T, (n_heads + 3) / 4);
   if (cache_f32) return launch_pdl(qkv_finish_kernel<float>, grid, dim3(128), 0, st, a, (float*)kc, (float*)vc);
   return launch_pdl(qkv_finish_kernel<__half>, grid, dim3(128), 0, st, a, (__half*)kc, (__half*)vc);
@@ -469,7 +699,9 @@ B200_API int b200_qkv_finish(const float* in, int ld, int T, int q_off, int k_of
 // the output columns.  Everything is fp32 whatever the cache holds.  gate [T][ldg] (or null): the output of head h is
 // multiplied by sigmoid(gate[t][h]).  chunk > 0: a query sees its own chunk of that many positions only.  sinks [H] (or null): one more
 // term of the denominator per head.  maps: see qkv_finish (query rows are DK wide).  KS: columns of a key row in the cache.  vc null: the
-// values are the first DV columns of the key row (latent attention).
+// values are the first DV columns of the key row (latent attention).  window > 0: a query sees that many positions, itself the last.
+// slopes [H] (or null): slopes[h] times the distance is taken off a score.  slices > 1 (mixed heads, values are keys): a key row is that many
+// heads' keys of DK columns side by side, a query row is as wide and meets all of them, and the values are the slice of the head's own group.
 struct AttnExactArgs {
   const float* q;          // [T][H][DK], scaled
   const int* page_table;
@@ -478,7 +710,8 @@ struct AttnExactArgs {
   const int* ctx_len;
   const float* gate;
   const float* sinks;
-  int ldg, max_pages, H, G, DK, DV, KS, maps, chunk, shared_kv;
+  const float* slopes;
+  int ldg, max_pages, H, G, DK, DV, KS, maps, chunk, shared_kv, window, slices;
   float* out_f32;          // [T][ldo], head h at column h * DV
   __nv_bfloat16* out_bf16;
   int ldo;
@@ -493,8 +726,9 @@ template <typename CT, int kExactCols>
 __global__ void __launch_bounds__(32 * kExactRows) attn_exact_kernel(const AttnExactArgs a, const CT* __restrict__ kc,
                                                                      const CT* __restrict__ vc) {
   extern __shared__ __align__(16) float sm[];
-  float* sQ = sm;                                   // [rows][DK]
-  float* sK = sQ + kExactRows * a.DK;               // [keys][DK + 1]
+  float* sQ = sm;                                   // [rows][QW]
+  const int QW = a.DK * a.slices;                   // columns of a query row
+  float* sK = sQ + kExactRows * QW;                 // [keys][DK + 1]
   const int ldv = a.shared_kv ? a.DK + 1 : a.DV;
   float* sV = a.shared_kv ? sK : sK + kExactKeys * (a.DK + 1);         // [keys][ldv]
   pdl_trigger();
@@ -503,40 +737,47 @@ __global__ void __launch_bounds__(32 * kExactRows) attn_exact_kernel(const AttnE
   const int qlen = a.q_len[seq];
   if (q0 >= qlen) return;
   const int ctx = a.ctx_len[seq], qs = a.q_start[seq], row_k = h / (a.H / (a.G * a.maps));
-  const int kh = row_k / a.maps, k_col = row_k % a.maps * a.DK;
+  const int kh = row_k / a.maps, own = h / (a.H / a.slices);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int* pt = a.page_table + (size_t)seq * a.max_pages;
   const int rows = min(kExactRows, qlen - q0), pos0 = ctx - qlen + q0, qpos = pos0 + warp;
-  for (int i = tid; i < rows * a.DK; i += blockDim.x) {
-    const int r = i / a.DK, c = i % a.DK;
-    sQ[i] = a.q[((size_t)(qs + q0 + r) * a.H + h) * a.DK + c];
+  for (int i = tid; i < rows * QW; i += blockDim.x) {
+    const int r = i / QW, c = i % QW;
+    sQ[i] = a.q[((size_t)(qs + q0 + r) * a.H + h) * QW + c];
   }
   float acc[kExactCols];
 #pragma unroll
   for (int i = 0; i < kExactCols; i++) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
+  const float slope = a.slopes ? a.slopes[h] : 0.f;
   const int k_end = pos0 + rows;                    // keys [k_begin, k_end) matter to some row
-  const int k_begin = a.chunk > 0 ? pos0 / a.chunk * a.chunk : 0, q_first = a.chunk > 0 ? qpos / a.chunk * a.chunk : 0;
+  const int k_begin = a.chunk > 0 ? pos0 / a.chunk * a.chunk : a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
+  const int q_first = a.chunk > 0 ? qpos / a.chunk * a.chunk : a.window > 0 ? qpos - a.window + 1 : 0;
   for (int k0 = k_begin; k0 < k_end; k0 += kExactKeys) {
-    __syncthreads();
     const int nk = min(kExactKeys, k_end - k0);
-    for (int i = tid; i < nk * a.DK; i += blockDim.x) {
-      const int r = i / a.DK, c = i % a.DK, key = k0 + r;
-      sK[r * (a.DK + 1) + c] = get(kc + (((size_t)pt[key >> 4] * a.G + kh) * 16 + (key & 15)) * a.KS + k_col + c);
+    const bool seen = warp < rows && lane < nk && k0 + lane <= qpos && k0 + lane >= q_first;
+    float s = seen ? -slope * (float)(qpos - k0 - lane) : -INFINITY;
+    for (int u = 1; u <= a.slices; u++) {           // the own slice comes last: its keys are then the values
+      const int sl = (own + u) % a.slices, k_col = (a.slices > 1 ? sl : row_k % a.maps) * a.DK;
+      __syncthreads();
+      for (int i = tid; i < nk * a.DK; i += blockDim.x) {
+        const int r = i / a.DK, c = i % a.DK, key = k0 + r;
+        sK[r * (a.DK + 1) + c] = get(kc + (((size_t)pt[key >> 4] * a.G + kh) * 16 + (key & 15)) * a.KS + k_col + c);
+      }
+      for (int i = tid; i < nk * a.DV && !a.shared_kv; i += blockDim.x) {
+        const int r = i / a.DV, c = i % a.DV, key = k0 + r;
+        sV[r * a.DV + c] = get(vc + (((size_t)pt[key >> 4] * a.G + kh) * 16 + (key & 15)) * a.DV + c);
+      }
+      __syncthreads();
+      if (seen) {
+        const float* kr = sK + lane * (a.DK + 1);
+        const float* qr = sQ + warp * QW + (a.slices > 1 ? sl * a.DK : 0);
+        float dot = 0.f;
+        for (int c = 0; c < a.DK; c++) dot = fmaf(qr[c], kr[c], dot);
+        s += dot;
+      }
     }
-    for (int i = tid; i < nk * a.DV && !a.shared_kv; i += blockDim.x) {
-      const int r = i / a.DV, c = i % a.DV, key = k0 + r;
-      sV[r * a.DV + c] = get(vc + (((size_t)pt[key >> 4] * a.G + kh) * 16 + (key & 15)) * a.DV + c);
-    }
-    __syncthreads();
     if (warp >= rows) continue;
-    float s = -INFINITY;
-    if (lane < nk && k0 + lane <= qpos && k0 + lane >= q_first) {
-      const float* kr = sK + lane * (a.DK + 1);
-      const float* qr = sQ + warp * a.DK;
-      s = 0.f;
-      for (int c = 0; c < a.DK; c++) s = fmaf(qr[c], kr[c], s);
-    }
     const float mn = fmaxf(m, warp_max(s));
     if (mn == -INFINITY) continue;
     const float corr = m == -INFINITY ? 0.f : expf(m - mn);
@@ -592,15 +833,16 @@ static int launch_exact(int DV, dim3 grid, size_t smem, const AttnExactArgs& a, 
 B200_API int b200_attn_exact(const float* q, const void* kc, const void* vc, int cache_f32, const int* page_table, int max_pages,
                              const int* q_start, const int* q_len, const int* ctx_len, int n_seqs, int max_q, int H, int G, int DK,
                              int DV, const float* gate, int ldg, float* out_f32, void* out_bf16, int ldo, int KS, int maps, int chunk,
-                             const float* sinks, cudaStream_t st) {
+                             const float* sinks, int window, const float* slopes, int slices, cudaStream_t st) {
   if (G < 1 || maps < 1 || H % (G * maps) || n_seqs < 1 || max_q < 1 || DK < 1 || DV < 1 || DV > 1024 || ldo < H * DV || KS < maps * DK || chunk < 0)
     return B200_ERR_BAD_ARG;
   if (!vc && (DV > DK || maps != 1)) return B200_ERR_BAD_ARG;
+  if (window < 0 || (window && chunk) || slices < 1 || (slices > 1 && (vc || G != 1 || maps != 1 || H % slices || KS < slices * DK))) return B200_ERR_BAD_ARG;
   AttnExactArgs a;
   a.q = q; a.page_table = page_table; a.q_start = q_start; a.q_len = q_len; a.ctx_len = ctx_len; a.gate = gate; a.ldg = ldg;
   a.max_pages = max_pages; a.H = H; a.G = G; a.DK = DK; a.DV = DV; a.out_f32 = out_f32; a.out_bf16 = (__nv_bfloat16*)out_bf16; a.ldo = ldo;
-  a.KS = KS; a.maps = maps; a.chunk = chunk; a.sinks = sinks; a.shared_kv = vc ? 0 : 1;
-  const size_t smem = 4 * ((size_t)kExactRows * DK + (size_t)kExactKeys * (DK + 1) + (vc ? (size_t)kExactKeys * DV : 0));
+  a.KS = KS; a.maps = maps; a.chunk = chunk; a.sinks = sinks; a.shared_kv = vc ? 0 : 1; a.window = window; a.slopes = slopes; a.slices = slices;
+  const size_t smem = 4 * ((size_t)kExactRows * DK * slices + (size_t)kExactKeys * (DK + 1) + (vc ? (size_t)kExactKeys * DV : 0));
   if (smem > 200 * 1024) return B200_ERR_BAD_ARG;
   const dim3 grid((max_q + kExactRows - 1) / kExactRows, H, n_seqs);
   if (cache_f32) return launch_exact<float>(DV, grid, smem, a, (const float*)kc, (const float*)vc, st);
@@ -646,10 +888,11 @@ B200_API int b200_diff_combine(const float* in, const float* lambda, int T, int 
 
 // C[M][N] = act(alpha A[M][K] W[N][K]^T), times sigmoid(gate[M][N]) where given, added into C (accumulate) or stored: fp32 activations, bf16-stored weights (their expansion is exact), fp32 multiply-adds on the
 // CUDA cores.  The 32-bit mode's projection; 64 x 64 tiles, 16 K columns staged at a time, 4 x 4 outputs per thread.
-// heads > 1: head z multiplies columns z * head_k of A with rows z * N of W into columns z * head_ldc of C.
+// col_scale [N] (or null) multiplies what is stored or added.  heads > 1: head z multiplies columns z * head_k of A with rows z * N of W into columns z * head_ldc of C.
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W,
                                                        int ldb, float* __restrict__ C, int ldc, int M, int N, int K, int act, float alpha,
-                                                       int accumulate, const float* __restrict__ gate, int ldg, int head_k, int head_ldc) {
+                                                       int accumulate, const float* __restrict__ gate, int ldg, int head_k, int head_ldc,
+                                                       const float* __restrict__ col_scale) {
   __shared__ float sA[16][68], sB[16][68];
   pdl_trigger();
   pdl_wait();
@@ -688,17 +931,19 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
       if (act == 1) v = v > 0.f ? v * v : 0.f;
       else if (act == 2) v = gelu_erf(v);
       if (gate) v *= 1.f / (1.f + expf(-gate[(size_t)m * ldg + n]));
+      if (col_scale) v *= col_scale[n];
       float* c = C + (size_t)m * ldc + n;
       *c = accumulate ? *c + v : v;
     }
 }
 // act: 0 none, 1 the square of relu, 2 the erf gelu.
 B200_API int b200_gemm_f32(const float* A, int lda, const void* W, int ldb, float* C, int ldc, int M, int N, int K, int act,
-                           float alpha, int accumulate, const float* gate, int ldg, int heads, int head_k, int head_ldc, cudaStream_t st) {
-  if (M < 1 || N < 1 || K < 1 || heads < 1 || lda < (heads - 1) * head_k + K || ldb < K || ldc < (heads - 1) * head_ldc + N || act < 0 || act > 2)
+                           float alpha, int accumulate, const float* gate, int ldg, int heads, int head_k, int head_ldc, const float* col_scale,
+                           cudaStream_t st) {
+  if (M < 1 || N < 1 || K < 1 || heads < 1 || (col_scale && heads > 1) || lda < (heads - 1) * head_k + K || ldb < K || ldc < (heads - 1) * head_ldc + N || act < 0 || act > 2)
     return B200_ERR_BAD_ARG;
   return launch_pdl(gemm_f32_kernel, dim3((N + 63) / 64, (M + 63) / 64, heads), dim3(256), 0, st, A, lda, (const __nv_bfloat16*)W, ldb, C,
-                    ldc, M, N, K, act, alpha, accumulate, gate, ldg, head_k, head_ldc);
+                    ldc, M, N, K, act, alpha, accumulate, gate, ldg, head_k, head_ldc, col_scale);
 }
 
 // ------------------------------------------------------------------ one small mat-vec per head

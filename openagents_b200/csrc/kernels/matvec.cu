@@ -28,6 +28,7 @@ struct MatvecArgs {
   const float* bias;    // [N] or null (dual: [2N])
   const float* resid;   // [nb][ldy] (EPI_RESID)
   float alpha;          // EPI_RESID: multiplies the product
+  const float* col_scale;   // EPI_RESID: [N] or null, multiplies the product too
   float* y;             // [nb][ldy]
   int ldy;
   int8_t* oq;           // EPI_SWIGLU_Q8 outputs
@@ -232,7 +233,7 @@ __device__ __forceinline__ void matvec_epilogue(const MatvecArgs& a, const float
   } else if (a.epi == EPI_GELU_ERF) {
     if (live) a.y[(size_t)b * a.ldy + n] = gelu_erf(v);
   } else if (a.epi == EPI_RESID) {
-    if (live) a.y[(size_t)b * a.ldy + n] = fmaf(v, a.alpha, a.resid[(size_t)b * a.ldy + n]);
+    if (live) a.y[(size_t)b * a.ldy + n] = fmaf(v, a.col_scale ? a.alpha * a.col_scale[n] : a.alpha, a.resid[(size_t)b * a.ldy + n]);
   } else if (a.epi == EPI_ALLREDUCE) {
     if (live) sym_red_all_f32(a.sym, a.sym_off + ((size_t)b * a.ldy + n) * 4, v);
   } else {
@@ -519,7 +520,7 @@ static int run_matvec(int wt, MatvecArgs& a, cudaStream_t st) {
 B200_API int b200_matvec(int wt, const void* w, const void* w2, int N, int K, int nb, const void* xq,
                          const float* xd, const float* xs16, const float* xf, int epi, const float* bias,
                          const float* resid, float* y, int ldy, void* oq, float* od, float* os16,
-                         const SymTable* sym, size_t sym_off, int wait_ready, float alpha, cudaStream_t st) {
+                         const SymTable* sym, size_t sym_off, int wait_ready, float alpha, const float* col_scale, cudaStream_t st) {
   if (nb < 1 || nb > 8 || epi == EPI_ROPE_KV) return B200_ERR_BAD_ARG;
   if (wt == WT_BF16 ? (K % 8 != 0 || (uintptr_t)xf % 16) : (K % 256 != 0 && !(wt == WT_Q8R && K % 32 == 0))) return B200_ERR_BAD_ARG;
   if (epi == EPI_SWIGLU_Q8 && N % 32) return B200_ERR_BAD_ARG;
@@ -537,6 +538,7 @@ B200_API int b200_matvec(int wt, const void* w, const void* w2, int N, int K, in
   }
   a.wait_ready = wait_ready;
   a.alpha = alpha;
+  a.col_scale = col_scale;
   return run_matvec(wt, a, st);
 }
 

@@ -30,6 +30,12 @@ class MixerSpec:
     kv_from: int | None = None     # this layer reads the keys and values of an earlier one
     bias: bool = False             # q, k and v projections have biases
     chunk: int = 0                 # keys of the query's own chunk of this many positions only (0: all earlier ones)
+    window: int = 0                # keys of this many positions only, the query's own the last (0: all earlier ones)
+    tied_kv: bool = False          # the values are the keys: no value projection, one cache
+    out_bias: bool = False         # the output projection has a bias
+    distance_bias: bool = False    # head h of H: 2^(-8 (h + 1) / H) times the distance comes off a score
+    mix_heads: bool = False        # a learned [heads, heads] matrix mixes the heads' scores ahead of the softmax
+    silent_sink: bool = False      # one more term of the softmax's denominator, with a score of 0 and no value
     maps: int = 1                  # 2: differential attention, two maps over the same values, the second one subtracted
     diff: float = 0.0              # the constant part of the second map's weight
     # latent attention (``dim``: unrotated query / key dimensions, rope_dims of the rot_dim others rotate)
@@ -55,6 +61,12 @@ class MixerSpec:
         elif self.kind == "attention":
             if self.chunk < 0 or self.maps not in (1, 2):
                 raise ValueError("bad chunk size or number of maps")
+            if self.window < 0 or (self.window and self.chunk):
+                raise ValueError("bad window size, or a window together with chunks")
+            if self.tied_kv and (self.dim != self.vdim or self.maps > 1 or self.kv_from is not None):
+                raise ValueError("values that are the keys have their size, one map and a cache of their own")
+            if self.mix_heads and (not self.tied_kv or self.rope_dims or self.qk_norm or self.head_gate or self.chunk):
+                raise ValueError("mixed heads go with values that are the keys, without rotation, unit norms, gates and chunks")
             if self.kv_heads < 1 or self.heads % self.kv_heads:
                 raise ValueError("the key/value heads must divide the query heads")
             if not 0 <= self.rope_dims <= self.dim or self.rope_dims % 2:
@@ -64,17 +76,30 @@ class MixerSpec:
 
 
 @dataclass(frozen=True)
+class ExpertSpec:
+    """A mixture of gated feed-forwards (silu) in place of one: each token uses the ``top`` experts with the largest scores, weighted by the sigmoid of
+    their router logits, not renormalised; the weight multiplies what goes into an expert."""
+    experts: int
+    top: int
+
+    def __post_init__(self):
+        if not 1 <= self.top <= self.experts:
+            raise ValueError("a token's experts must be at least one and no more than there are")
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    """One layer of a hybrid stack: a mixer and, unless ``ffn`` is 0, a feed-forward of that width; a norm before each and, where the
-    model has them (``ModelConfig.post_norm``), behind each."""
+    """One layer of a hybrid stack: a mixer and, unless ``ffn`` is 0, a feed-forward of that width (with ``moe``: experts of that width each); a norm
+    before each and, where the model has them (``ModelConfig.post_norm``), behind each."""
     mixer: MixerSpec
     ffn: int = 0
-    act: str = "relu2"             # "relu2": the square of relu; "gelu": the exact (erf) gelu
+    act: str = "relu2"             # "relu2": the square of relu; "gelu": the exact (erf) gelu; "polynorm": unit-RMS powers 1 to 3, mixed; "swiglu"
+    moe: ExpertSpec | None = None
 
 
 @dataclass(frozen=True)
 class ModelConfig:
-    arch: str = "llama"            # llama | gpt2 | gpt-oss | folirax | pesorax
+    arch: str = "llama"            # llama | gpt2 | gpt-oss | folirax | pesorax | kazolorn
     n_layers: int = 2
     d_model: int = 256
     n_heads: int = 4
@@ -96,7 +121,10 @@ class ModelConfig:
     qkv_bias: bool = False
     # hybrid stacks: the layers one by one (the flat head and width fields above then hold the largest of each)
     layers: tuple[LayerSpec, ...] = ()
-    norm: str = "rms"              # "rms": root-mean-square, weights stored around zero; "dyt": w * tanh(alpha x) + b, no statistics
+    norm: str = "rms"              # "rms": root-mean-square, weights stored around zero; "rms1": the same, stored as they are; "dyt": w * tanh(alpha x) + b
+    walk: str = "serial"           # "parallel": mixer and feed-forward of a layer read the same residual (a norm each) and are added together
+    layer_scale: bool = False      # a learned factor per channel on what either adds
+    depth_average: bool = False    # what a layer hands on is a learned mixture of the embedding output and every layer's result so far
     post_norm: bool = True         # a norm behind every sublayer as well
     residual_mult: float = 1.0     # multiplies what a sublayer adds to the residual (stacks without post_norm)
     loop: tuple[int, int, int] | None = None     # (start, stop, times): these layers run ``times`` times in a row, the embedding added ahead of every pass but the first
@@ -326,10 +354,65 @@ def _pesorax_to_json(cfg: ModelConfig) -> dict:
             "loop": None if cfg.loop is None else dict(zip(("start", "stop", "times"), cfg.loop)), "residual_mult": cfg.residual_mult}
 
 
+def _kazolorn(c: dict, ranks: dict[int, int], name: str, context: int) -> ModelConfig:
+    """Kazolorn: sliding-window attention whose keys are its values, with a distance bias, mixed heads and a silent sink; the feed-forward (PolyNorm, or
+    experts whose weights scale their input) in parallel, both scaled per channel; a depth average behind every layer."""
+    layers = []
+    for i, e in enumerate(_need(c, "layers", list, "")):
+        w = f"layers[{i}]."
+        mx, kind = _need(e, "mixer", dict, w), _need(e, "type", str, w)
+        w2 = w + "mixer."
+        if kind != "attention":
+            raise ValueError(f"config: {w}type {kind!r} is not a mixer of this design")
+        window = _need(_need(mx, "mask", dict, w2), "size", int, w2 + "mask.")
+        if window < 1:
+            raise ValueError(f"config: {w2}mask.size must be positive")
+        dim = _need(mx, "dim", int, w2)
+        m = MixerSpec("attention", _need(mx, "heads", int, w2), dim, dim if mx.get("vdim") is None else _need(mx, "vdim", int, w2),
+                      kv_heads=_need(mx, "kv_heads", int, w2), scale=_need(mx, "scale", float, w2), bias=True, out_bias=True, window=window, tied_kv=True,
+                      distance_bias=True, mix_heads=True, silent_sink=True)
+        mlp, ff, moe = e.get("mlp"), 0, None
+        if mlp is not None:
+            kind = _need(mlp, "kind", str, w + "mlp.")
+            if kind == "dense":
+                ff = _need(mlp, "ff", int, w + "mlp.")
+            elif kind == "moe":
+                ff = _need(_need(mlp, "expert", dict, w + "mlp."), "ff", int, w + "mlp.expert.")
+                router = _need(mlp, "router", dict, w + "mlp.")
+                moe = ExpertSpec(_need(router, "experts", int, w + "mlp.router."), _need(router, "top", int, w + "mlp.router."))
+            else:
+                raise ValueError(f"config: {w}mlp.kind {kind!r} is not known")
+            if ff < 1:
+                raise ValueError(f"config: {w}mlp: the width must be positive")
+        layers.append(LayerSpec(m, ff, "swiglu" if moe else "polynorm", moe))
+    if not layers:
+        raise ValueError("config: layers is empty")
+    mx = [l.mixer for l in layers]
+    return ModelConfig(arch="kazolorn", n_layers=len(layers), d_model=_need(c, "width", int, ""), vocab=_need(c, "vocab", int, ""),
+                       n_heads=max(m.heads for m in mx), n_kv_heads=max(m.kv_heads for m in mx), head_dim=max(m.dim for m in mx),
+                       ffn=max(l.ffn for l in layers), context=context, norm_eps=_need(_need(c, "norm", dict, ""), "eps", float, "norm."),
+                       layers=tuple(layers), norm="rms1", post_norm=False, walk="parallel", layer_scale=True, depth_average=True, name=name)
+
+
+def _kazolorn_to_json(cfg: ModelConfig) -> dict:
+    layers = []
+    for l in cfg.layers:
+        m, mlp = l.mixer, None
+        if l.moe:
+            mlp = {"kind": "moe", "expert": {"ff": l.ffn}, "router": {"experts": l.moe.experts, "top": l.moe.top}}
+        elif l.ffn:
+            mlp = {"kind": "dense", "ff": l.ffn}
+        layers.append({"type": "attention", "mlp": mlp, "mixer": {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale,
+                                                                  "mask": {"size": m.window}}})
+    return {"architecture": "Kazolorn", "layers": layers, "width": cfg.d_model, "vocab": cfg.vocab, "norm": {"eps": cfg.norm_eps}}
+
+
 def hybrid_to_json(cfg: ModelConfig) -> dict:
     """The inverse of ``config_from_json``."""
     if cfg.arch == "pesorax":
         return _pesorax_to_json(cfg)
+    if cfg.arch == "kazolorn":
+        return _kazolorn_to_json(cfg)
     layers = []
     for l in cfg.layers:
         m = l.mixer
@@ -346,7 +429,7 @@ def hybrid_to_json(cfg: ModelConfig) -> dict:
             "ranks": {str(i): l.mixer.rank for i, l in enumerate(cfg.layers) if l.mixer.kind == "gla"}}
 
 
-JSON_ARCHITECTURES = {"Folirax": _folirax, "Pesorax": _pesorax}
+JSON_ARCHITECTURES = {"Folirax": _folirax, "Pesorax": _pesorax, "Kazolorn": _kazolorn}
 HYBRID_ARCHS = tuple(a.lower() for a in JSON_ARCHITECTURES)
 
 
@@ -415,4 +498,22 @@ def pesorax_stack(width: int, ffn: int, vocab: int, groups: int, heads: int, kv_
 PESORAX_8B = pesorax_stack(4096, 14336, 128256, 8, 16, 4, 64, 128, 2048, 32, 128, 64, 128, 512, 1536, "pesorax-8b-shape")
 PESORAX_1B = pesorax_stack(2048, 8192, 32000, 3, 8, 2, 64, 128, 1024, 16, 128, 64, 128, 512, 768, "pesorax-1b-shape", loop=(4, 8, 2))
 
-PRESETS = {c.name: c for c in (TINY_LLAMA, LLAMA3_8B, LLAMA3_70B, GPT2_SMALL, GPT_OSS_20B, FOLIRAX_8B, FOLIRAX_1B, PESORAX_8B, PESORAX_1B)}
+
+def kazolorn_stack(width: int, ffn: int, vocab: int, layers: int, heads: int, kv_heads: int, dim: int, window: int, name: str, experts: int = 0, top: int = 0,
+                   expert_ffn: int = 0, dense: int = 1) -> ModelConfig:
+    """A regular stack: ``dense`` layers with one feed-forward, the others (all of them without ``experts``) with a mixture."""
+    m = MixerSpec("attention", heads, dim, dim, kv_heads=kv_heads, scale=dim ** -0.5, bias=True, out_bias=True, window=window, tied_kv=True, distance_bias=True,
+                  mix_heads=True, silent_sink=True)
+    own, mixture = LayerSpec(m, ffn, "polynorm"), LayerSpec(m, expert_ffn, "swiglu", ExpertSpec(experts, top)) if experts else None
+    stack = tuple(mixture if experts and i >= dense else own for i in range(layers))
+    return ModelConfig(arch="kazolorn", n_layers=layers, d_model=width, n_heads=heads, n_kv_heads=kv_heads, head_dim=dim, ffn=max(ffn, expert_ffn), vocab=vocab,
+                       context=HYBRID_CONTEXT, norm_eps=1e-5, layers=stack, norm="rms1", post_norm=False, walk="parallel", layer_scale=True,
+                       depth_average=True, name=name)
+
+
+# layers of the 8B preset's size with one feed-forward each, and a smaller stack whose layers (but the first) have 32 experts of which a token uses four
+KAZOLORN_8B = kazolorn_stack(4096, 14336, 128256, 32, 32, 8, 128, 4096, "kazolorn-8b-shape")
+KAZOLORN_MOE = kazolorn_stack(2048, 8192, 32000, 16, 16, 4, 128, 1024, "kazolorn-moe-shape", experts=32, top=4, expert_ffn=2048)
+
+PRESETS = {c.name: c for c in (TINY_LLAMA, LLAMA3_8B, LLAMA3_70B, GPT2_SMALL, GPT_OSS_20B, FOLIRAX_8B, FOLIRAX_1B, PESORAX_8B, PESORAX_1B, KAZOLORN_8B,
+                               KAZOLORN_MOE)}

@@ -29,7 +29,9 @@ from .paged import PAGE, PagedEngine
 from .qweight import WeightSource
 
 LATENT_CTAS = 592            # most CTAs of a latent decode launch that splits the keys
+MOE_EXPERTS, MOE_TOP = 256, 32   # most experts of a layer, and of a token
 SHORT_TOKENS = 16            # latent attention: entries of up to this many new tokens work in the latent space
+ALONE = ("polynorm", "swiglu")   # activations that are no epilogue of the up projection
 ACTS = {None: (ops.EPI_STORE, ops.ACT_NONE, 0), "relu2": (ops.EPI_RELU2, ops.ACT_RELU2, 1), "gelu": (ops.EPI_GELU_ERF, ops.ACT_GELU_ERF, 2)}
 
 
@@ -77,6 +79,15 @@ class _Latent:
 
 
 @dataclass
+class _Experts:
+    """A mixture's weights; F: the experts' width, padded."""
+    F: int
+    router: torch.Tensor         # fp32 [E][dp]
+    w13: torch.Tensor            # bf16 [E * 2 F][dp], rows interleaved (gate, up)
+    w2: torch.Tensor             # bf16 [E * dp][F]
+
+
+@dataclass
 class _Block:
     spec: LayerSpec
     norm1: _Norm
@@ -98,6 +109,15 @@ class _Block:
     norm2b: _Norm | None = None
     up: _Lin | None = None
     down: _Lin | None = None
+    act: torch.Tensor | None = None              # PolyNorm's four numbers
+    moe: _Experts | None = None
+    mix: torch.Tensor | None = None              # fp32 [heads][heads]
+    slopes: torch.Tensor | None = None           # what a step of distance takes off a score, per head (behind the mixture)
+    silent: torch.Tensor | None = None           # zeros: the scores of the silent sinks
+    out_bias: torch.Tensor | None = None         # times the layer scale: joins the residual ahead of the layer
+    ls1: torch.Tensor | None = None
+    ls2: torch.Tensor | None = None
+    average: torch.Tensor | None = None
 
 
 @dataclass
@@ -139,7 +159,7 @@ def plan_latent_batch(q_len: list[int], ctx: list[int], short_rows: int, ctx_row
 
 
 class HybridEngine(PagedEngine):
-    ARCHS = ("folirax", "pesorax")
+    ARCHS = ("folirax", "pesorax", "kazolorn")
     world = 1                    # one GPU; the serving layer asks
     vocab_sharded = False
 
@@ -155,7 +175,11 @@ class HybridEngine(PagedEngine):
         self._init_paged(device, max_batch, max_ctx, n_pages, max_tokens, canaries, state_slots=slots)
         self.dp = _up(self.d, 8)
         # Dynamic Tanh has no statistics of a row, so the residual itself can carry the padding (zeros stay zeros)
-        self.dx = self.dp if cfg.norm == "dyt" else self.d
+        self.dx = self.dp if cfg.norm != "rms" else self.d
+        self.parallel = cfg.walk == "parallel"
+        if self.parallel != cfg.depth_average or cfg.layer_scale != cfg.depth_average or (cfg.norm == "rms1") != self.parallel or \
+                (self.parallel and cfg.loop is not None) or any(l.act in ALONE or l.mixer.out_bias for l in cfg.layers) and not self.parallel:
+            raise ValueError("a depth average goes with parallel sublayers, layer scales and norms stored as they are, without a loop")
         if cfg.post_norm != (cfg.norm == "rms") or (cfg.post_norm and cfg.loop is not None):
             raise ValueError("norms on both sides go with RMS norms and without a loop, Dynamic Tanh with a norm ahead only")
         # Decode batches up to this size take the mat-vec kernels.  Measured (ms per step, one token, mat-vec / GEMM): width 2048
@@ -181,8 +205,12 @@ class HybridEngine(PagedEngine):
         w = self._vector(src, name)
         if self.cfg.norm == "rms":
             return _Norm(w + 1.0)                        # stored around zero
-        pad = lambda v: torch.nn.functional.pad(v, (0, self.dx - self.d))        # noqa: E731
-        return _Norm(pad(w), pad(self._vector(src, name + ".b")), self._vector(src, name + ".alpha"))
+        if self.cfg.norm == "rms1":
+            return _Norm(self._wide(w))
+        return _Norm(self._wide(w), self._wide(self._vector(src, name + ".b")), self._vector(src, name + ".alpha"))
+
+    def _wide(self, v: torch.Tensor) -> torch.Tensor:
+        return torch.nn.functional.pad(v, (0, self.dp - self.d))
 
     def _out_proj(self, src: WeightSource, name: str, heads: int, vdim: int, pad: int) -> _Lin:
         """The output projection with every head's columns padded to the mixer's output row."""
@@ -214,7 +242,20 @@ class HybridEngine(PagedEngine):
                 b.norm2 = self._norm(src, p + "norm2")
                 if cfg.post_norm:
                     b.norm2b = self._norm(src, p + "norm2b")
-                b.up, b.down = self._lin(self._matrix(src, p + "mlp.up")), self._lin(self._matrix(src, p + "mlp.down"))
+                if spec.moe:
+                    b.moe = self._load_experts(src, p + "mlp.", spec)
+                else:
+                    b.up, b.down = self._lin(self._matrix(src, p + "mlp.up")), self._lin(self._matrix(src, p + "mlp.down"))
+                if spec.act == "polynorm":
+                    b.act = self._vector(src, p + "mlp.act")
+                if cfg.layer_scale:
+                    b.ls2 = self._wide(self._vector(src, p + "ls2"))
+            if cfg.layer_scale:
+                b.ls1 = self._wide(self._vector(src, p + "ls1"))
+            if spec.mixer.out_bias:
+                b.out_bias = self._wide(self._vector(src, p + "mix.o.b")) * b.ls1
+            if cfg.depth_average:
+                b.average = self._vector(src, p + "dwa")
             self.blocks.append(b)
         self.runs: list[_Run] = []
         self.kv_specs: list[_Block] = []                 # one key / value cache each
@@ -247,7 +288,7 @@ class HybridEngine(PagedEngine):
 
     def _load_attention(self, src: WeightSource, p: str, spec: LayerSpec) -> _Block:
         m = spec.mixer
-        own = ["k", "v"] if m.kv_from is None else []
+        own = [] if m.kv_from is not None else ["k"] if m.tied_kv else ["k", "v"]
         parts = {n: self._matrix(src, p + n) for n in ["q"] + own + (["g"] if m.head_gate else [])}
         biases = {n: self._vector(src, f"{p}{n}.b") for n in ["q"] + own} if m.bias else {}
         if m.maps > 1:                                   # query rows (head, map) -> (key/value head, map, head of the group)
@@ -266,7 +307,27 @@ class HybridEngine(PagedEngine):
         b.DK, b.DV, b.tc = self._head_pad(m)
         b.table = self._table(m)
         b.out = self._out_proj(src, p + "o", m.heads, m.vdim, b.DV)
+        if m.mix_heads:
+            b.mix = self._vector(src, p + "talk").view(m.heads, m.heads)
+        if m.distance_bias:
+            slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / m.heads) for h in range(m.heads)], dtype=torch.float64, device=self.device)
+            b.slopes = (slopes if b.mix is None else b.mix.double() @ slopes).float()
+        if m.silent_sink:
+            b.silent = torch.zeros(m.heads, dtype=torch.float32, device=self.device)
         return b
+
+    def _load_experts(self, src: WeightSource, p: str, spec: LayerSpec) -> _Experts:
+        E, F, d, pad = spec.moe.experts, _up(spec.ffn, 16), self.d, torch.nn.functional.pad
+        if E > MOE_EXPERTS or spec.moe.top > MOE_TOP:
+            raise ValueError(f"at most {MOE_EXPERTS} experts, {MOE_TOP} of them per token")
+        w13 = torch.zeros((E, F, 2, self.dp), dtype=torch.bfloat16, device=self.device)
+        w2 = torch.zeros((E, self.dp, F), dtype=torch.bfloat16, device=self.device)
+        for e in range(E):
+            w13[e, : spec.ffn, 0, :d] = self._matrix(src, f"{p}e{e}.gate").to(self.device)
+            w13[e, : spec.ffn, 1, :d] = self._matrix(src, f"{p}e{e}.up").to(self.device)
+            w2[e, :d, : spec.ffn] = self._matrix(src, f"{p}e{e}.down").to(self.device)
+        router = pad(self._vector(src, p + "router").view(E, d), (0, self.dp - d)).contiguous()
+        return _Experts(F, router, w13.view(-1, self.dp), w2.view(-1, F))
 
     def _load_latent(self, src: WeightSource, p: str, spec: LayerSpec) -> _Block:
         m, pad = spec.mixer, torch.nn.functional.pad
@@ -300,6 +361,8 @@ class HybridEngine(PagedEngine):
         """Padded head sizes in the cache (keys: per map), and whether the tensor-core attention kernels take them (else, and always in
         the 32-bit mode, the any-size kernel runs)."""
         dk, dv = _up(m.dim, 64), _up(m.vdim, 64)
+        if m.mix_heads or m.distance_bias:
+            return _up(m.dim, 8), _up(m.vdim, 8), False
         if self.exact or m.maps * dk > 256 or dv > 128:
             return _up(m.dim, 8), _up(m.vdim, 8), False
         return dk, dv, True
@@ -308,6 +371,8 @@ class HybridEngine(PagedEngine):
         n = self.head.w.numel()
         for b in self.blocks:
             n += b.proj.w.numel() + b.out.w.numel() + (b.up.w.numel() + b.down.w.numel() if b.up is not None else 0)
+            if b.moe is not None:
+                n += b.moe.w13.numel() + b.moe.w2.numel() + 2 * b.moe.router.numel()
             if b.lat is not None:                        # what a decode step reads
                 n += b.lat.uq.w.numel() + b.lat.absorb.numel() + b.lat.value.numel()
         return 2 * n
@@ -321,8 +386,9 @@ class HybridEngine(PagedEngine):
         f32, bf = torch.float32, torch.bfloat16
         self._alloc_batch()
         ct = f32 if self.exact else torch.float16
-        self.kc = [torch.zeros((self.n_pages, b.spec.mixer.kv_heads, PAGE, b.spec.mixer.maps * b.DK), dtype=ct, device=dev) for b in self.kv_specs]
-        self.vc = [torch.zeros((self.n_pages, b.spec.mixer.kv_heads, PAGE, b.DV), dtype=ct, device=dev) for b in self.kv_specs]
+        self.kc = [torch.zeros((self.n_pages, *self._key_rows(b)), dtype=ct, device=dev) for b in self.kv_specs]
+        self.vc = [None if b.spec.mixer.tied_kv else torch.zeros((self.n_pages, b.spec.mixer.kv_heads, PAGE, b.DV), dtype=ct, device=dev)
+                   for b in self.kv_specs]
         self.lc = [torch.zeros((self.n_pages, PAGE, b.lat.CR + b.lat.RR), dtype=ct, device=dev) for b in self.latent_specs]
         ws = self._ws
         n_proj = max(b.proj.N for b in self.blocks)
@@ -330,9 +396,10 @@ class HybridEngine(PagedEngine):
         n_ffn = max((b.up.N for b in self.blocks if b.up is not None), default=8)
         attn = [(b, b.spec.mixer, b.spec.mixer.heads * b.spec.mixer.maps) for b in self.blocks if b.spec.mixer.kind == "attention"]
         lat = [(b, b.spec.mixer, b.lat) for b in self.blocks if b.lat is not None]
-        n_q = max((hq * m.maps * b.DK for b, m, hq in attn), default=8)
-        n_q32 = max((hq * b.DK for b, m, hq in attn if not b.tc), default=0)                # rows of a prompt in fp32
-        n_q16 = max([hq * b.DK for b, m, hq in attn if b.tc] + [m.heads * (L.KN + L.RR) for b, m, L in lat if b.tc], default=0)
+        wide = lambda b, m: (m.kv_heads if m.mix_heads else 1) * b.DK                        # noqa: E731   (columns of a prompt's query row)
+        n_q = max((hq * m.maps * wide(b, m) for b, m, hq in attn), default=8)
+        n_q32 = max((hq * wide(b, m) for b, m, hq in attn if not b.tc), default=0)          # rows of a prompt in fp32
+        n_q16 = max([hq * wide(b, m) for b, m, hq in attn if b.tc] + [m.heads * (L.KN + L.RR) for b, m, L in lat if b.tc], default=0)
         self.x = ws("x", (T, self.dx), f32)
         self.y = ws("y", (T if self.cfg.post_norm else 1, d), f32, zero=True)
         self.proj = ws("proj", (T * n_proj,), f32, zero=True)
@@ -378,12 +445,27 @@ class HybridEngine(PagedEngine):
         self.argmax_scratch = ops.argmax_scratch(self.max_batch, dev)
         self.iota = torch.arange(self.max_batch, dtype=torch.int32, device=dev)
         self.ones = torch.ones(self.max_batch, dtype=torch.int32, device=dev)
+        if self.cfg.depth_average:
+            # the embedding output, every layer's result (the row a layer adds into becomes one), and what goes on to the head
+            self.hist = ws("hist", (len(self.runs) + 1, T, d), f32, zero=True)
+            self.hf2, self.hb2 = ws("hf2", (small * d,), f32), ws("hb2", (big * d,), bf)
+            self.z = ws("z", (T * n_ffn,), f32, zero=True)
+        moe = [(b.spec.moe, b.moe) for b in self.blocks if b.moe is not None]
+        if moe:
+            top = max(m.top for m, _ in moe)
+            self.topk_ids, self.topk_w = ws("topk_ids", (T * top,), torch.int32, zero=True), ws("topk_w", (T * top,), f32)
+            self.mid = ws("mid", (max(T * m.top * x.F for m, x in moe),), f32)
         k_max = max(d, n_mix, n_ffn, widest(lambda b, m, L: L.uq.K))
         # the bf16 mat-vec keeps its fp32 activations in shared memory
         self.matvec_rows = max((n for n in (1, 2, 4, 8) if n * (k_max * 4 + 256) <= 200 * 1024), default=0)
 
+    def _key_rows(self, b: _Block) -> tuple[int, int, int]:
+        """A page of a layer's key cache.  Mixed heads: all heads' keys of a token side by side in one row."""
+        m = b.spec.mixer
+        return (1, PAGE, m.kv_heads * b.DK) if m.mix_heads else (m.kv_heads, PAGE, m.maps * b.DK)
+
     def _caches(self):
-        return [*self.kc, *self.vc, *self.lc]
+        return [c for c in (*self.kc, *self.vc, *self.lc) if c is not None]
 
     # ------------------------------------------------------------------ batch layout (latent attention)
     def _batch_order(self, q_len):
@@ -407,24 +489,25 @@ class HybridEngine(PagedEngine):
         return min(range(1, max(1, min(self.max_splits, blocks, LATENT_CTAS // ctas)) + 1), key=cost)
 
     # ------------------------------------------------------------------ building blocks
-    def _mm(self, a: torch.Tensor, L: _Lin, out: torch.Tensor, act: str | None = None, add: bool = False, into: float | None = None):
+    def _mm(self, a: torch.Tensor, L: _Lin, out: torch.Tensor, act: str | None = None, add: bool = False, into: float | None = None,
+            scale: torch.Tensor | None = None):
         """out = act(a W^T).  fp32 activations: mat-vec for a few rows, else the 32-bit product; bf16: the tensor-core GEMM (``add``:
-        the output was zeroed ahead, K may be split).  ``into``: out += into * (a W^T)."""
+        the output was zeroed ahead, K may be split).  ``into``: out += into * (a W^T), times ``scale`` per column."""
         T = a.shape[0]
         epi, gact, fact = ACTS[act]
         if a.dtype == torch.float32:
             if T <= self.matvec_rows:
                 if into is not None:
-                    ops.matvec(ops.WT_BF16, L.w, None, L.N, L.K, T, xf=a, epi=ops.EPI_RESID, resid=out, y=out, ldy=out.stride(0), alpha=into)
+                    ops.matvec(ops.WT_BF16, L.w, None, L.N, L.K, T, xf=a, epi=ops.EPI_RESID, resid=out, y=out, ldy=out.stride(0), alpha=into, col_scale=scale)
                 else:
                     ops.matvec(ops.WT_BF16, L.w, None, L.N, L.K, T, xf=a, epi=epi, y=out, ldy=out.stride(0))
             else:
-                ops.gemm_f32(a, L.w, out, fact, alpha=1.0 if into is None else into, accumulate=into is not None)
+                ops.gemm_f32(a, L.w, out, fact, alpha=1.0 if into is None else into, accumulate=into is not None, col_scale=scale)
         else:
             f32 = out.dtype == torch.float32
             ops.gemm_bf16(a, L.w, T, L.N, L.K, lda=a.stride(0), ldb=L.K, out_f32=out if f32 else None, out_bf16=out if out.dtype == torch.bfloat16 else None,
                           out_f16=out if out.dtype == torch.float16 else None, ldc=out.stride(0), act=gact, alpha=1.0 if into is None else into,
-                          accumulate=into is not None or (add and f32 and not act), status=self.status)
+                          accumulate=into is not None or (add and f32 and not act), status=self.status, col_scale=scale)
 
     def _mm_heads(self, a: torch.Tensor, w: torch.Tensor, heads: int, head_k: int, out: torch.Tensor, head_ldc: int, alpha: float = 1.0, gate=None):
         """One product per head: w [heads * N][K]; head z reads columns z * head_k of ``a`` and writes columns z * head_ldc of ``out``."""
@@ -436,14 +519,28 @@ class HybridEngine(PagedEngine):
         else:
             ops.gemm_heads(a, w, heads, N, K, head_k, out, head_ldc, alpha=alpha, gate=gate, status=self.status)
 
+    def _mixed(self, r: _Run, proj, T: int, decode: bool, n_seqs: int, max_q: int, pages: int, o32, o16) -> int:
+        """Attention with mixed heads: wide queries, one for all key heads of a cache row."""
+        b = r.block
+        m, kc = b.spec.mixer, self.kc[r.kv]
+        q = self.q32[: T * m.heads * m.kv_heads * b.DK].view(T, -1)
+        ops.mixed_finish(proj, m.heads * m.dim, b.bias, b.mix, m.scale, self.slot, m.heads, m.kv_heads, m.dim, b.DK, q, kc)
+        qs, ql = (self.iota, self.ones) if decode else (self.q_start, self.q_len)
+        ops.attn_exact(q, kc, None, self.page_table, qs, ql, self.seq_lens, n_seqs, max_q, m.heads, 1, b.DK, b.DV, out_f32=o32, out_bf16=o16, window=m.window,
+                       sinks=b.silent, slopes=b.slopes, slices=m.kv_heads)
+        return 2
+
     def _attention(self, r: _Run, proj, T: int, decode: bool, n_seqs: int, max_q: int, pages: int, o32, o16) -> int:
         b, cfg = r.block, self.cfg
         m = b.spec.mixer
+        if m.mix_heads:
+            return self._mixed(r, proj, T, decode, n_seqs, max_q, pages, o32, o16)
         own, HQ = m.kv_from is None, m.heads * m.maps
         k_off = HQ * m.dim if own else -1
-        v_off = k_off + m.kv_heads * m.maps * m.dim
-        g_off = v_off + m.kv_heads * m.vdim if own else HQ * m.dim
-        kc, vc = self.kc[r.kv], self.vc[r.kv]
+        v_off = -1 if m.tied_kv else k_off + m.kv_heads * m.maps * m.dim
+        g_off = HQ * m.dim + (m.kv_heads * (m.maps * m.dim + (0 if m.tied_kv else m.vdim)) if own else 0)
+        kc = self.kc[r.kv]
+        vc = kc if m.tied_kv else self.vc[r.kv]
         tc_prompt, wide = b.tc and not decode, b.tc and decode and m.maps > 1
         q = (self.q16 if tc_prompt else self.q32)[: T * HQ * b.DK * (m.maps if wide else 1)].view(T, -1)
         ops.qkv_finish(proj, 0, k_off, v_off, self.pos, self.slot, b.table, m.rope_base, HQ, m.kv_heads, m.dim, m.vdim, b.DK, b.DV,
@@ -455,17 +552,19 @@ class HybridEngine(PagedEngine):
             out32, out16 = self.maps_out[: T * HQ * b.DV].view(T, -1), None
         if m.chunk:
             pages = min(pages, m.chunk // PAGE + 2)
+        if m.window:
+            pages = min(pages, m.window // PAGE + 2)
         if tc_prompt:
             ops.attn_prefill_tc05(q, kc, vc, self.page_table, self.q_start, self.q_len, self.seq_lens, n_seqs, max_q, HQ, m.kv_heads,
-                                  out_bf16=out16, out_f32=out32, status=self.status, dk=b.DK, dv=b.DV, gate=gate, chunk=m.chunk, maps=m.maps)
+                                  out_bf16=out16, out_f32=out32, status=self.status, dk=b.DK, dv=b.DV, gate=gate, chunk=m.chunk, maps=m.maps, window=m.window, sinks=b.silent)
         elif b.tc:
             ops.attn_decode(q, kc, vc, self.page_table, self.seq_lens, n_seqs, HQ, m.kv_heads, m.maps * b.DK, dv=b.DV,
                             S=self._attn_splits(n_seqs, m.kv_heads, pages), gate=gate, out_f32=out32, out_bf16=out16,
-                            scratch=self.attn_scratch, counters=self.attn_counters, status=self.status, chunk=m.chunk)
+                            scratch=self.attn_scratch, counters=self.attn_counters, status=self.status, chunk=m.chunk, window=m.window, sinks=b.silent)
         else:
             qs, ql = (self.iota, self.ones) if decode else (self.q_start, self.q_len)
             ops.attn_exact(q, kc, vc, self.page_table, qs, ql, self.seq_lens, n_seqs, max_q, HQ, m.kv_heads, b.DK, b.DV, gate=gate,
-                           out_f32=out32, out_bf16=out16, maps=m.maps, chunk=m.chunk)
+                           out_f32=out32, out_bf16=out16, maps=m.maps, chunk=m.chunk, window=m.window, sinks=b.silent, slopes=b.slopes)
         if m.maps == 1:
             return 2
         ops.diff_combine(out32, b.lam, m.heads, m.kv_heads, m.vdim, b.DV, cfg.norm_eps, 1.0 - m.diff, out_f32=o32, out_bf16=o16)
@@ -537,7 +636,7 @@ class HybridEngine(PagedEngine):
 
     def _run_layers(self, T: int, decode: bool, n_seqs: int, max_q: int, pages: int) -> int:
         f32 = self.exact or (decode and T <= min(self.small_path_tokens, self.matvec_rows))
-        walk = self._walk_sandwich if self.cfg.post_norm else self._walk_prenorm
+        walk = self._walk_parallel if self.parallel else self._walk_sandwich if self.cfg.post_norm else self._walk_prenorm
         return walk(T, decode, f32, (decode, n_seqs, max_q, pages))
 
     def _buffers(self, T: int, f32: bool):
@@ -600,6 +699,47 @@ class HybridEngine(PagedEngine):
         self._tail = None
         return n
 
+    def _walk_parallel(self, T: int, decode: bool, f32: bool, step) -> int:
+        """Mixer and feed-forward of a layer read the same residual row and add into a copy of it, which then is the layer's result; the depth average over
+        the results so far makes the next layer's row, and its two norms, in one pass."""
+        eps, D = self.cfg.norm_eps, self.d
+        h, _, views = self._buffers(T, f32)
+        h2 = (self.hf2 if f32 else self.hb2)[: T * self.dp].view(T, self.dp)
+        add = not f32 and T <= QGEMM_MAX_TOKENS
+        n, weights = 0, None
+        for i, r in enumerate(self.runs):
+            b = r.block
+            proj, mix, act = views(b)
+            out = self.hist[i + 1, :T]
+            ff = b.norm2 is not None
+            ops.depth_norm(self.hist[: i + 1, :T], D, eps, weights=weights, out=out, add=b.out_bias, g1=b.norm1.w, h1=h, g2=b.norm2.w if ff else None,
+                           h2=h2 if ff else None, zero=proj if add else None)
+            self._mm(h, b.proj, proj, add=add)
+            n += self._mix(r, proj, mix, T, f32, step) + 3
+            self._mm(mix, b.out, out, into=1.0, scale=b.ls1)
+            if b.moe is not None:
+                n += self._experts(b, h2, out)
+            elif ff:
+                z = self.z[: T * b.up.N].view(T, -1)
+                self._mm(h2, b.up, z)
+                ops.poly_norm(z, b.spec.ffn, b.act, eps, act)
+                self._mm(act, b.down, out, into=1.0, scale=b.ls2)
+                n += 3
+            weights = b.average
+        ops.depth_norm(self.hist[: len(self.runs) + 1, :T], D, weights=weights, out=self.x[:T])
+        self._tail = None
+        return n + 1
+
+    def _experts(self, b: _Block, h, out) -> int:
+        """The chosen experts' sum, scaled per channel, into ``out``."""
+        T, top, x = h.shape[0], b.spec.moe.top, b.moe
+        ids, w = self.topk_ids[: T * top].view(T, top), self.topk_w[: T * top].view(T, top)
+        ops.moe_choose(h, x.router, top, ids, w, score=ops.SCORE_SIGMOID)
+        mid = self.mid[: T * top * x.F]
+        ops.expert_gate_up(h if h.dtype == torch.float32 else h.float(), x.w13, x.F, ids, w, mid)
+        ops.expert_down(mid, x.w2, self.dp, ids, out, scale=b.ls2)
+        return 3
+
     def _dyt(self, x, norm: _Norm, emb=None, **kw):
         ops.norm_dyt(x, norm.alpha, norm.w, norm.b, ids=self.ids, emb=emb, **kw)
 
@@ -611,6 +751,8 @@ class HybridEngine(PagedEngine):
         hk = dict(hf=h) if f32 else dict(hb=h)
         if self.cfg.norm == "dyt":
             self._dyt(rows, self.final_norm, **hk)
+        elif self.cfg.norm == "rms1":
+            ops.depth_norm(rows[None], self.d, eps, g1=self.final_norm.w, h1=h)
         else:
             ops.norm_residual(rows, eps, y=self.y[:nb] if gy is not None else None, gy=gy, gh=self.final_norm.w, **hk)
         w = _Lin(self.head.w[: self.V])
@@ -628,4 +770,4 @@ class HybridEngine(PagedEngine):
         return n
 
     def _embed(self, T: int):
-        ops.embedding(self.ids, self.x[:T], ops.EMB_BF16, self.emb, vocab_n=self.V)
+        ops.embedding(self.ids, self.hist[0, :T] if self.parallel else self.x[:T], ops.EMB_BF16, self.emb, vocab_n=self.V)

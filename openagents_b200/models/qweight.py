@@ -98,7 +98,7 @@ class RandomSource(WeightSource):
         t = self.plan.type_for(s)
         rows = s.shape[0]
         # Quantize in row chunks so a 128256 x 4096 table never needs several fp32 copies at once.
-        if len(s.shape) >= 2 and s.kind not in ("norm", "bias", "sink"):
+        if len(s.shape) >= 2 and s.kind not in ("norm", "bias", "sink", "average"):
             x = init_tensor(s, self.seed, device=self.device)
             chunks = [tc.quantize(c, t) for c in x.split(max(1, (1 << 24) // max(1, x[0].numel())))]
             del x

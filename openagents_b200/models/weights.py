@@ -18,7 +18,7 @@ from .config import ModelConfig
 class TensorSpec:
     name: str
     shape: tuple[int, ...]
-    kind: str   # "matrix" | "embed" | "output" | "norm" | "bias" | "expert" | "router" | "sink" | "pos"
+    kind: str   # "matrix" | "embed" | "output" | "norm" | "bias" | "expert" | "router" | "sink" | "pos" | "average"
 
 
 def tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
@@ -74,7 +74,7 @@ def hybrid_tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
     def norm(name):
         if cfg.norm == "dyt":
             return [TensorSpec(name, (d,), "norm"), TensorSpec(name + ".b", (d,), "bias"), TensorSpec(name + ".alpha", (1,), "norm")]
-        return [TensorSpec(name, (d,), "bias")]
+        return [TensorSpec(name, (d,), "norm" if cfg.norm == "rms1" else "bias")]
     s = [TensorSpec("embed", (cfg.vocab, d), "embed")]
     for i, l in enumerate(cfg.layers):
         p, m = f"l{i}.", l.mixer
@@ -102,15 +102,30 @@ def hybrid_tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
             if m.bias:
                 s.append(TensorSpec(p + "q.b", (m.maps * m.heads * m.dim,), "bias"))
             if m.kv_from is None:
-                for n, rows in (("k", m.maps * m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)):
+                for n, rows in [("k", m.maps * m.kv_heads * m.dim)] + ([] if m.tied_kv else [("v", m.kv_heads * m.vdim)]):
                     s += [TensorSpec(p + n, (rows, d), "matrix")] + ([TensorSpec(f"{p}{n}.b", (rows,), "bias")] if m.bias else [])
             if m.head_gate:
                 s.append(TensorSpec(p + "g", (m.heads, d), "matrix"))
             if m.maps == 2:
                 s += [TensorSpec(p + n, (m.dim,), "bias") for n in ("lq1", "lk1", "lq2", "lk2")]
+            if m.mix_heads:
+                s.append(TensorSpec(p + "talk", (m.heads, m.heads), "sink"))
         s.append(TensorSpec(p + "o", (d, m.heads * m.vdim), "matrix"))
-        if l.ffn:
-            s += [TensorSpec(f"l{i}.mlp.up", (l.ffn, d), "matrix"), TensorSpec(f"l{i}.mlp.down", (d, l.ffn), "matrix")]
+        if m.out_bias:
+            s.append(TensorSpec(p + "o.b", (d,), "bias"))
+        p = f"l{i}.mlp."
+        if l.moe:
+            for e in range(l.moe.experts):
+                s += [TensorSpec(f"{p}e{e}.{n}", shape, "matrix") for n, shape in (("gate", (l.ffn, d)), ("up", (l.ffn, d)), ("down", (d, l.ffn)))]
+            s.append(TensorSpec(p + "router", (l.moe.experts, d), "router"))
+        elif l.ffn:
+            s += [TensorSpec(p + "up", (l.ffn, d), "matrix"), TensorSpec(p + "down", (d, l.ffn), "matrix")]
+            if l.act == "polynorm":
+                s.append(TensorSpec(p + "act", (4,), "norm"))
+        if cfg.layer_scale:
+            s += [TensorSpec(f"l{i}.{n}", (d,), "norm") for n in (("ls1", "ls2") if l.ffn else ("ls1",))]
+        if cfg.depth_average:
+            s.append(TensorSpec(f"l{i}.dwa", (i + 2,), "average"))
     return s + norm("final.norm") + [TensorSpec("head", (cfg.vocab, d), "output")]
 
 
@@ -124,7 +139,7 @@ class QuantPlan:
     router: GgmlType = GgmlType.F32
 
     def type_for(self, spec: TensorSpec) -> GgmlType:
-        if spec.kind in ("norm", "bias", "sink", "pos"):
+        if spec.kind in ("norm", "bias", "sink", "pos", "average"):
             return GgmlType.F32
         t = {"matrix": self.matrix, "embed": self.embed, "output": self.output,
              "expert": self.expert, "router": self.router}[spec.kind]
@@ -145,6 +160,10 @@ def init_tensor(spec: TensorSpec, seed: int, device="cpu", std: float = 0.02) ->
         return torch.ones(spec.shape, dtype=torch.float32, device=device)
     if spec.kind == "bias":
         return torch.zeros(spec.shape, dtype=torch.float32, device=device)
+    if spec.kind == "average":             # the latest result, and a little of the others
+        w = torch.full(spec.shape, 0.1 / spec.shape[0], dtype=torch.float32, device=device)
+        w[-1] += 0.9
+        return w
     g = torch.Generator(device=device)
     g.manual_seed((seed * 1000003 + zlib.crc32(spec.name.encode())) & 0x7FFFFFFF)
     return torch.randn(spec.shape, generator=g, dtype=torch.float32, device=device) * std

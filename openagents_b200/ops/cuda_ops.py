@@ -17,6 +17,7 @@ WT_Q4KR, WT_Q6KR, WT_Q8R, WT_BF16, WT_MXFP4R = 0, 1, 2, 3, 4
 EPI_STORE, EPI_RESID, EPI_SWIGLU_Q8, EPI_SWIGLU_F32, EPI_ALLREDUCE, EPI_RELU2, EPI_GELU_ERF = 0, 1, 2, 3, 4, 6, 7
 SYM_NONE, SYM_ALLREDUCE, SYM_RSCATTER, SYM_RSCATTER_ROWS = 0, 1, 2, 3
 EMB_F32, EMB_BF16, EMB_Q8R, EMB_Q6KR = 0, 1, 2, 3
+SCORE_SOFTMAX, SCORE_SIGMOID = 0, 1
 ACT_NONE, ACT_GELU, ACT_SWIGLU_PAIR, ACT_RELU2, ACT_GELU_ERF = 0, 1, 2, 3, 4
 
 _P = c_void_p
@@ -34,7 +35,7 @@ _SIGS = {
     "b200_matvec_rope_kv": [c_int, _P, _P, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int,
                             c_int, c_float, c_float, _P],
     "b200_matvec": [c_int, _P, _P, c_int, c_int, c_int, _P, _P, _P, _P, c_int, _P, _P, _P, c_int, _P, _P, _P, _P,
-                    c_size_t, c_int, c_float, _P],
+                    c_size_t, c_int, c_float, _P, _P],
     "b200_argmax_merge": [_P, _P, c_int, _P, c_size_t, c_int, _P],
     "b200_attn_decode": [_P, _P, _P, _P, c_int, c_int, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, _P,
                          _P, _P, _P, _P, _P, _P],
@@ -43,11 +44,16 @@ _SIGS = {
                                c_int, _P, c_int, c_int, _P, _P, _P],
     "b200_attn_prefill_latent": [_P, _P, c_long, c_int, c_int, _P, _P, c_int, c_int, c_int, _P, c_int, _P, _P, _P] + [c_int] * 7 + [_P, _P, c_int, _P, _P, _P],
     "b200_gemm_bf16": [_P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int,
-                       _P, c_int, _P, c_size_t, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P],
+                       _P, c_int, _P, c_size_t, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, _P],
     "b200_gemm_heads": [_P, _P] + [c_int] * 7 + [_P, _P, c_int, c_int, c_float, _P, c_int, c_int, _P, _P],
-    "b200_moe_gemm": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, _P, _P, _P, c_size_t, _P, _P],
+    "b200_moe_gemm": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, _P, _P, _P, c_size_t, _P, c_long, _P, _P],
     "b200_moe_route_dispatch": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_size_t, c_size_t, c_size_t, c_size_t,
-                                _P, _P, _P, _P, _P],
+                                _P, _P, c_int, _P, _P, _P],
+    "b200_expert_gate_up": [_P, c_int, c_int, _P, c_int, _P, _P, c_int, _P, _P],
+    "b200_expert_down": [_P, c_int, c_int, _P, c_int, _P, c_int, _P, _P, c_int, _P],
+    "b200_depth_norm": [_P, c_size_t, _P, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_float, _P, _P, _P, _P, _P, c_long, _P],
+    "b200_poly_norm": [_P, c_int, c_int, c_int, _P, c_float, _P, _P, c_int, _P],
+    "b200_mixed_finish": [_P] + [c_int] * 3 + [_P, _P, c_float, _P] + [c_int] * 5 + [_P, _P, _P, c_int, _P],
     "b200_moe_zero": [_P, c_int, _P],
     "b200_set_pdl": [c_int],
     "b200_set_prefetch": [c_int],
@@ -63,8 +69,8 @@ _SIGS = {
     "b200_qkv_finish": [_P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, c_double, c_int, c_int, c_int, c_int, c_int, c_int,
                         c_int, c_int, c_int, c_float, c_float, c_int, _P, _P, _P, _P, c_int, c_int, c_int, _P, _P],
     "b200_attn_exact": [_P, _P, _P, c_int, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, c_int, c_int, c_int,
-                        c_int, _P, _P],
-    "b200_gemm_f32": [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, c_int, c_int, c_int, c_int, _P],
+                        c_int, _P, c_int, _P, c_int, _P],
+    "b200_gemm_f32": [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, c_int, c_int, c_int, c_int, _P, _P],
     "b200_head_matvec": [_P, c_int, _P, c_int, _P] + [c_int] * 5 + [c_float, _P, c_int, c_int, c_int, _P],
     "b200_norm_dyt": [_P, c_int, c_int, _P, _P, c_int, _P, _P, _P, _P, _P, c_int, _P, c_long, _P],
     "b200_diff_combine": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_float, _P, _P, c_int, _P],
@@ -202,11 +208,11 @@ def sample_topk(logits, temperature, top_k, top_p, u, out_id, scratch):
 
 
 def matvec(wt, w, w2, N, K, nb, xq=None, xd=None, xs16=None, xf=None, epi=EPI_STORE, bias=None, resid=None, y=None,
-           ldy=0, oq=None, od=None, os16=None, sym=None, sym_off=0, wait_ready=False, alpha=1.0):
-    """Quantized mat-vec for 1..8 tokens (see ``matvec.cu``).  ``alpha`` multiplies what EPI_RESID adds.  The SwiGLU epilogues read ``w`` as 2N rows interleaved
+           ldy=0, oq=None, od=None, os16=None, sym=None, sym_off=0, wait_ready=False, alpha=1.0, col_scale=None):
+    """Quantized mat-vec for 1..8 tokens (see ``matvec.cu``).  ``alpha`` (a number) and ``col_scale`` [N] multiply what EPI_RESID adds.  The SwiGLU epilogues read ``w`` as 2N rows interleaved
     (gate_0, up_0, gate_1, ...)."""
     _check(lib().b200_matvec(wt, _p(w), _p(w2), N, K, nb, _p(xq), _p(xd), _p(xs16), _p(xf), epi, _p(bias), _p(resid),
-                             _p(y), ldy, _p(oq), _p(od), _p(os16), _sym(sym), sym_off, int(wait_ready), alpha, _st()), "matvec")
+                             _p(y), ldy, _p(oq), _p(od), _p(os16), _sym(sym), sym_off, int(wait_ready), alpha, _p(col_scale), _st()), "matvec")
 
 
 def matvec_rope_kv(w, nb, pos, slot, q_out, kc, vc, Hq, Hkv, hd, page_size, theta, q_scale, xq=None, xd=None, xs16=None, xf=None,
@@ -267,8 +273,8 @@ def attn_prefill_latent(q16, ws, v_col, base, cache, r_col, page_table, q_start,
 def gemm_bf16(A, B, M, N, K, lda=None, ldb=None, out_f32=None, out_bf16=None, ldc=None, bias=None, resid_f32=None,
               resid_bf16=None, act=ACT_NONE, accumulate=False, tile_n=0, status=None, sym_mode=SYM_NONE, sym=None,
               sym_off=0, rows_per_rank=0, split_k=0, wait_ready=False, ag_rows_per_rank=0, ag_epoch=0, mn_major=False, alpha=1.0,
-              out_f16=None):
-    """``alpha`` multiplies the product; ``out_f16`` instead of ``out_bf16``: stored as fp16.  D[M][N] = A[M][K] @ B[N][K]^T with fused epilogue (see ``gemm_tc05.cu``).  ``ag_rows_per_rank`` > 0: the rows
+              out_f16=None, col_scale=None):
+    """``alpha`` multiplies the product, ``col_scale`` [N] what is stored or added; ``out_f16`` instead of ``out_bf16``: stored as fp16.  D[M][N] = A[M][K] @ B[N][K]^T with fused epilogue (see ``gemm_tc05.cu``).  ``ag_rows_per_rank`` > 0: the rows
     of A are all-gathered by push (``rmsnorm_allgather``) and each tile waits for its owners' counter to reach ``ag_epoch``.
     ``mn_major``: the operands are given as A [K][M] and B [K][N] (row strides ``lda`` / ``ldb``), i.e. D = A^T B: the weight
     gradient dW = dy^T x straight from dy and x, without transposed copies."""
@@ -276,7 +282,7 @@ def gemm_bf16(A, B, M, N, K, lda=None, ldb=None, out_f32=None, out_bf16=None, ld
                                 _p(out_bf16 if out_f16 is None else out_f16), ldc or N,
                                 _p(bias), _p(resid_f32), _p(resid_bf16), act, int(accumulate), tile_n, split_k, _p(status),
                                 sym_mode, _sym(sym), sym_off, rows_per_rank, int(wait_ready), ag_rows_per_rank, ag_epoch,
-                                int(mn_major), alpha, int(out_f16 is not None), _st()), "gemm_bf16")
+                                int(mn_major), alpha, int(out_f16 is not None), _p(col_scale), _st()), "gemm_bf16")
 
 
 def gemm_heads(A, B, heads, N, K, head_k, out, head_ldc, alpha=1.0, gate=None, status=None):
@@ -326,22 +332,42 @@ def qgemm(w, x_bf16, T, out_f32=None, out_bf16=None, ldo=None, bias=None, epi=QE
 
 # ---------------------------------------------------------------- mixture of experts
 def moe_route_dispatch(h_bf16, h_f32, router_w, router_b, top_k, E_local, C, recv_x_off, recv_meta_off, recv_w_off, counts_off,
-                       sym, topk_ids=None, topk_w=None, status=None):
-    """Router + top-k + softmax + expert-parallel dispatch of ``h_bf16`` [T][d] (see ``moe.cu``); the router
-    (fp32 weights) reads ``h_f32`` when given."""
-    T, d = h_bf16.shape
+                       sym, topk_ids=None, topk_w=None, status=None, score=SCORE_SOFTMAX):
+    """Router + top-k + weights (``score``: softmax over the chosen, or each one's sigmoid) + expert-parallel dispatch of ``h_bf16`` [T][d] (see
+    ``moe.cu``); the router (fp32 weights) reads ``h_f32`` when given.  ``sym`` None: one rank, the offsets are addresses."""
+    T, d = (h_bf16 if h_bf16 is not None else h_f32).shape
     E = router_w.shape[0]
     _check(lib().b200_moe_route_dispatch(_p(h_bf16), _p(h_f32), _p(router_w), _p(router_b), T, d, E, top_k, E_local, C, recv_x_off,
-                                         recv_meta_off, recv_w_off, counts_off, _p(topk_ids), _p(topk_w), _sym(sym),
+                                         recv_meta_off, recv_w_off, counts_off, _p(topk_ids), _p(topk_w), score, _sym(sym),
                                          _p(status), _st()), "moe_route_dispatch")
 
 
 def moe_gemm(A, B, groups, group_rows, N, K, counts, mode, out_bf16=None, ldc=0, meta=None, gate_w=None, sym=None,
-             sym_off=0, status=None, lda=None, ldb=None):
+             sym_off=0, status=None, lda=None, ldb=None, col_scale=None, live_rows=0):
     """Grouped expert GEMM (see ``gemm_tc05.cu``): mode 1 = gate/up with fused SwiGLU, mode 2 = down
-    projection fused with the weighted combine into the source ranks' residual streams."""
+    projection fused with the weighted combine into the source ranks' residual streams.  Mode 1 with ``gate_w``: the weight multiplies
+    the expert's input.  Mode 2 without ``sym``: ``sym_off`` is the address of the fp32 [tokens, ldc] destination; ``col_scale`` [N] multiplies
+    what is added.  ``live_rows``: the most rows all groups hold together."""
     _check(lib().b200_moe_gemm(_p(A), _p(B), groups, group_rows, N, K, lda or K, ldb or K, _p(counts), mode, _p(out_bf16),
-                               ldc, _p(meta), _p(gate_w), _sym(sym), sym_off, _p(status), _st()), "moe_gemm")
+                               ldc, _p(meta), _p(gate_w), _sym(sym), sym_off, _p(col_scale), live_rows, _p(status), _st()), "moe_gemm")
+
+
+def moe_choose(h, router_w, top_k, ids, w, score=SCORE_SOFTMAX):
+    """The choice alone: expert ids (int32) and weights (fp32), [T, top_k], of the rows ``h`` (bf16 or fp32)."""
+    f32, E = h.dtype == torch.float32, router_w.shape[0]
+    moe_route_dispatch(None if f32 else h, h if f32 else None, router_w, None, top_k, E, 0, 0, 0, 0, 0, None, topk_ids=ids, topk_w=w, score=score)
+
+
+def expert_gate_up(x, w13, F, ids, weights, mid):
+    """``mid[t, s] = silu(w g) * (w u)`` for the chosen experts of fp32 rows ``x`` [T, K]; ``w13`` bf16 [E * 2 F, K], rows interleaved (gate, up); ``ids`` /
+    ``weights`` [T, top] (None: weights of one)."""
+    _check(lib().b200_expert_gate_up(_p(x), x.shape[0], x.shape[1], _p(w13), F, _p(ids), _p(weights), ids.shape[1], _p(mid), _st()), "expert_gate_up")
+
+
+def expert_down(mid, w2, N, ids, out, scale=None):
+    """``out[t] += scale * sum_s W_down[ids[t, s]] mid[t, s]``; ``w2`` bf16 [E * N, F]."""
+    T, top = ids.shape
+    _check(lib().b200_expert_down(_p(mid), T, w2.shape[1], _p(w2), N, _p(ids), top, _p(scale), _p(out), out.stride(0), _st()), "expert_down")
 
 
 def moe_zero(t):
@@ -394,27 +420,55 @@ def qkv_finish(proj, q_off, k_off, v_off, pos, slot, table, base, H, G, dim, vdi
 
 
 def attn_exact(q32, kc, vc, page_table, q_start, q_len, ctx_len, n_seqs, max_q, H, G, DK, DV, gate=None, out_f32=None, out_bf16=None, maps=1,
-               chunk=0, sinks=None):
+               chunk=0, sinks=None, window=0, slopes=None, slices=1):
     """Causal attention in 32-bit arithmetic for any head sizes; ``gate``: fp32 [T, >= H] view whose sigmoid scales each head; ``maps``: see
-    :func:`qkv_finish`; ``vc`` None: the values are the first DV columns of the keys (latent attention)."""
+    :func:`qkv_finish`; ``vc`` None: the values are the first DV columns of the keys (latent attention); ``slopes`` [H]: times the distance, taken off
+    the scores; ``slices``: see :func:`mixed_finish`."""
     o = out_f32 if out_f32 is not None else out_bf16
     _check(lib().b200_attn_exact(_p(q32), _p(kc), _p(vc), int(kc.dtype == torch.float32), _p(page_table), page_table.shape[1], _p(q_start),
                                  _p(q_len), _p(ctx_len), n_seqs, max_q, H, G, DK, DV, _p(gate), 0 if gate is None else gate.stride(0),
-                                 _p(out_f32), _p(out_bf16), o.stride(0), kc.shape[-1], maps, chunk, _p(sinks), _st()), "attn_exact")
+                                 _p(out_f32), _p(out_bf16), o.stride(0), kc.shape[-1], maps, chunk, _p(sinks), window, _p(slopes), slices, _st()), "attn_exact")
 
 
-def gemm_f32(A, W, out, act=0, alpha=1.0, accumulate=False, gate=None, heads=1, head_k=0, head_ldc=0):
+def gemm_f32(A, W, out, act=0, alpha=1.0, accumulate=False, gate=None, heads=1, head_k=0, head_ldc=0, col_scale=None):
     """``out = act(alpha * A @ W^T)`` in true 32-bit: A fp32 [M, K], W bf16 [N, K]; ``act`` 1: the square of relu, 2: the erf gelu; times the sigmoid of ``gate``
-    [M, N]; ``accumulate`` adds into ``out``.  ``heads`` > 1: one product per head, as in :func:`gemm_heads`."""
+    [M, N] and by ``col_scale`` [N]; ``accumulate`` adds into ``out``.  ``heads`` > 1: one product per head, as in :func:`gemm_heads`."""
     M, (N, K) = A.shape[0], W.shape
     _check(lib().b200_gemm_f32(_p(A), A.stride(0), _p(W), W.stride(0), _p(out), out.stride(0), M, N // heads, K, act, alpha, int(accumulate), _p(gate),
-                               0 if gate is None else gate.stride(0), heads, head_k, head_ldc, _st()), "gemm_f32")
+                               0 if gate is None else gate.stride(0), heads, head_k, head_ldc, _p(col_scale), _st()), "gemm_f32")
 
 
 def head_matvec(A, W, out, heads, head_k, head_ldc, alpha=1.0, gate=None):
     """:func:`gemm_heads` for 1..8 fp32 rows on the CUDA cores: ``W`` bf16 [heads * N, K]."""
     _check(lib().b200_head_matvec(_p(A), A.stride(0), _p(W), W.stride(0), _p(out), out.stride(0), A.shape[0], heads, W.shape[0] // heads, W.shape[1], alpha,
                                   _p(gate), 0 if gate is None else gate.stride(0), head_k, head_ldc, _st()), "head_matvec")
+
+
+def depth_norm(xs, D, eps=0.0, weights=None, out=None, add=None, g1=None, g2=None, h1=None, h2=None, zero=None):
+    """``x = sum_j weights[j] * xs[j]`` over the slabs of ``xs`` (fp32 [n, >= T, ld], D columns live; a slice along the rows is fine; ``weights`` None: one
+    slab as it is); ``out`` [T, ld] = x + ``add``; ``h1`` / ``h2`` (both bf16 or fp32, [T, ld]) = x over its root mean square, times ``g1`` / ``g2``."""
+    n, T, ld = xs.shape
+    f32 = next((h.dtype == torch.float32 for h in (h1, h2) if h is not None), False)
+    b, f = (lambda h: None if f32 else _p(h)), (lambda h: _p(h) if f32 else None)                   # noqa: E731
+    _check(lib().b200_depth_norm(_p(xs), xs.stride(0), _p(weights), n, T, D, ld, _p(out), _p(add), _p(g1), _p(g2), eps, b(h1), b(h2), f(h1), f(h2),
+                                 _p(zero), 0 if zero is None else zero.numel(), _st()), "depth_norm")
+
+
+def poly_norm(z, F, coef, eps, out):
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` per row of ``z`` (fp32 [T, >= F]), N dividing by the root mean square, ``coef`` = (a, b, c, e); ``out`` bf16 or fp32,
+    columns beyond F zero."""
+    f32 = out.dtype == torch.float32
+    _check(lib().b200_poly_norm(_p(z), z.stride(0), z.shape[0], F, _p(coef), eps, None if f32 else _p(out), _p(out) if f32 else None, out.stride(0), _st()),
+           "poly_norm")
+
+
+def mixed_finish(proj, k_off, bias, mix, scale, slot, H, G, dim, DK, q, kc):
+    """Queries and keys of an attention layer whose heads' scores are mixed: a cache row holds all G heads' keys of DK columns side by side (they are the
+    values too), and a query row ``q`` (fp32 or fp16 [T, H, G * DK]) holds, per key head, the ``mix`` [H, H] weighted sum of that group's scaled
+    queries, so that its product with a cache row is the mixed score.  ``proj`` fp32 [T, >= (H + G) * dim], keys from column ``k_off`` on."""
+    f32, c32 = q.dtype == torch.float32, kc.dtype == torch.float32
+    _check(lib().b200_mixed_finish(_p(proj), proj.stride(0), proj.shape[0], k_off, _p(bias), _p(mix), scale, _p(slot), H, G, dim, DK, kc.shape[2],
+                                   _p(q) if f32 else None, None if f32 else _p(q), _p(kc), int(c32), _st()), "mixed_finish")
 
 
 def norm_dyt(x, alpha, w, b, hb=None, hf=None, ids=None, emb=None, zero=None):
