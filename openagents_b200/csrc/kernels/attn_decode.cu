@@ -14,6 +14,7 @@
 // The softmax follows the reference formulation (max-subtract, exp, normalise:
 // apps/openagents.com/workers/api/src/cs336-a1-real-gradient-workload.ts:478-518).
 #include "tc05.cuh"
+#include "warp_mma.cuh"
 
 using namespace b200;
 
@@ -57,25 +58,6 @@ __device__ __forceinline__ void write_out(const AttnDecArgs& a, int b, int h, in
     quantize_block32(o, lane, a.oq + row + (size_t)blk * 32, a.od + (size_t)b * nblk + blk,
                      a.os16 + ((size_t)b * nblk + blk) * 2);
   }
-}
-
-__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x4_t(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_h2(float x, float y) {
-  __half2 h = __floats2half2_rn(x, y);
-  return *(uint32_t*)&h;
 }
 
 constexpr int kStages = 8;   // pages in flight per CTA (two per warp)

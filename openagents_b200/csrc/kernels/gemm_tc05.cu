@@ -48,6 +48,19 @@ int make_tmap_2d(CUtensorMap* map, const void* base, int elem_bytes, uint64_t ro
   return r == CUDA_SUCCESS ? 0 : (int)r;
 }
 
+int make_tmap_rows8(CUtensorMap* map, const void* base, uint64_t rows, uint64_t cols, uint32_t col_boxes) {
+  EncodeTiledFn enc = get_encode_tiled();
+  if (!enc) return -1;
+  if (((uintptr_t)base & 15) || cols % 64 || rows % 8 || col_boxes < 1 || col_boxes > 256) return -2;
+  cuuint64_t dims[4] = {64, 8, cols / 64, rows / 8};
+  cuuint64_t strides[3] = {cols * 2, 128, cols * 16};
+  cuuint32_t box[4] = {64, 8, col_boxes, 2};
+  cuuint32_t estr[4] = {1, 1, 1, 1};
+  CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : (int)r;
+}
+
 }  // namespace b200
 
 // ACT_SWIGLU_PAIR: B rows are interleaved (gate_0, up_0, gate_1, ...); the epilogue writes

@@ -273,7 +273,6 @@ __device__ __forceinline__ void tmem_st(uint32_t taddr, const uint32_t (&r)[NC])
                  ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]),
                    "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]) : "memory");
 }
-__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 // The 256 softmax threads meet, and all learn whether every one of them is fine.
 __device__ __forceinline__ bool meet(bool ok) {
   uint32_t r;

@@ -5,13 +5,24 @@
 //   sum_g T[h][g] (q_g . k_c(g)) = Q'_h . K,   K = [k_0 | k_1 | ...] (all key heads of a token side by side),
 //                                              Q'_h = [sum over g of group 0 of T[h][g] q_g | the same of group 1 | ...]
 // Prompts take the first form: every head then attends on its own, with wide queries on a key row that all heads share, whose slice of the
-// head's group is the value.  Distances: the biases of the mixture add up to one slope per head.
+// head's group is the value; the tensor cores have the room for the longer products.  Decoding takes the second: a token's raw scores fit one warp's
+// registers, so that the mixture is one more small product there.  Distances: the biases of the mixture add up to one slope per head.
 // A cache row is K: [page][16][G * DK], fp16 (or fp32 in the 32-bit mode).
 //
 // This file is compiled without fast math.
-#include "common.cuh"
+#include "tc05.cuh"
+#include "warp_mma.cuh"
 
 using namespace b200;
+using namespace b200::tc;
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+// A wait that ran out leaves copies in flight: give them time to land before the shared memory goes to another block.
+__device__ __forceinline__ void drain_after_abort() {
+  const unsigned long long t0 = globaltimer_ns();
+  while (globaltimer_ns() - t0 < 2000000ull) __nanosleep(1000);
+}
 
 // ------------------------------------------------------------------ finish of the projections
 
@@ -121,4 +132,784 @@ B200_API int b200_mixed_finish(const float* in, int ld, int T, int k_off, const 
   a.in = in; a.ld = ld; a.k_off = k_off; a.bias = bias; a.mix = mix; a.q_scale = q_scale; a.slot = slot; a.H = H; a.G = G; a.dim = dim; a.DK = DK;
   a.page_size = page_size; a.q32 = q32; a.q16 = (__half*)q16;
   return cache_f32 ? launch_mixed_finish(T, a, (float*)kc, st) : launch_mixed_finish(T, a, (__half*)kc, st);
+}
+
+// ------------------------------------------------------------------ decoding: one query token per sequence
+
+// Grid (shares of the keys, value parts, sequences).  Pages come whole, all key heads of 16 tokens, in one TMA copy each: [2][W / 64][8 rows][128
+// bytes], swizzled, into a ring whose slots are a multiple of the warps; a warp takes every nw-th page of the CTA's share (so a slot is always the same
+// warp's) and works on it alone:
+//   raw scores      S^T = K Q^T per key head, 16 keys x 8 query heads a tile
+//   mixture         S^T T^T on bf16 products: the scores as three bf16 pieces (24 bits: fp32's own), T is stored in bf16
+//   softmax         running, in base 2; a head's offset moves only when its maximum has grown by 2^8
+//   output          O^T += K^T P^T, the transposed weights coming from movmatrix
+// A group's query heads are padded to RP of 1, 2, 4 or a multiple of 8.  Where a tile's eight heads belong to several groups, the raw product runs
+// over all their keys with the other groups' queries as zeros, and the output product puts 8 keys of two groups into one step of 16.
+// Heads beyond what a warp's registers hold as outputs are served by several CTAs (value parts), each mixing for its own tiles.
+struct MixedDecArgs {
+  const float* q;          // [B][H * DK], scaled
+  const float* mix;        // [H][H]
+  const float* slopes;     // [H], of the mixed scores
+  const float* sinks;      // [H] or null
+  const int* page_table;
+  const int* seq_lens;
+  int max_pages, H, G, rp, window, S, nslot;
+  float* out_f32;          // [B][H * DK]
+  __nv_bfloat16* out_bf16;
+  float* part_acc;         // [B][parts][S][8 NTV][DK]
+  float* part_ml;          // [B][parts][S][8 NTV][2]
+  int* counters;           // [B][parts], zero before first use, left zero
+  int* status;
+};
+__device__ __forceinline__ float2 split_bf16(float x, float y, uint32_t& packed) {      // the pair's bf16 values, and what they leave
+  const __nv_bfloat162 p = __floats2bfloat162_rn(x, y);
+  packed = *(const uint32_t*)&p;
+  const float2 f = __bfloat1622float2(p);
+  return make_float2(x - f.x, y - f.y);
+}
+
+// NT: tiles of eight (padded) query heads, an even number; NTV: those whose outputs this CTA keeps
+template <int DK, int NT, int NTV>
+__global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant__ CUtensorMap tm, const MixedDecArgs a) {
+  constexpr int QLD = DK + 8, KB = DK / 64;
+  extern __shared__ uint8_t dyn_raw[];
+  __shared__ float s_ml[8][NTV * 8][2];
+  __shared__ int s_last;
+  __shared__ int s_abort;
+  uint8_t* ring = (uint8_t*)(((uintptr_t)dyn_raw + 1023) & ~(uintptr_t)1023);
+  const int W = a.G * DK, page_bytes = 32 * W, NB = W / 64, nw = blockDim.x >> 5;
+  float* s_acc = (float*)ring;                                           // [nw][NTV * 8][DK], once the pages are done with
+  const size_t ring_bytes = max((size_t)a.nslot * page_bytes, (size_t)nw * NTV * 8 * DK * 4);
+  uint64_t* bars = (uint64_t*)(ring + ring_bytes);
+  __half* sQ = (__half*)(bars + ((a.nslot + 1) & ~1));                   // [8 NT + 1][QLD], the last row zeros
+  uint2* sT = (uint2*)(sQ + (8 * NT + 1) * QLD + 8 * ((8 * NT + 1) & 1));             // [NT / 2][NTV][32]
+  int* s_pid = (int*)(sT + NT / 2 * NTV * 32);
+
+  const int split = blockIdx.x, part = blockIdx.y, b = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
+  const int rp = a.rp, rep = a.H / a.G, live = a.G * rp, nsub = rp < 8 ? 8 / rp : 1;      // live: padded heads that exist
+  auto head_of = [&](int slot) { return slot < live && slot % rp < rep ? slot / rp * rep + slot % rp : -1; };
+  if (tid == 0) {
+    for (int s = 0; s < a.nslot; s++) mbar_init(smem_u32(bars + s), 1);
+    s_abort = 0;
+    fence_barrier_init();
+    tma_prefetch_desc(&tm);
+  }
+  // the mixture as B operand: rows the raw slots, columns this part's slots (weights: nothing to wait for)
+  for (int i = tid; i < NT / 2 * NTV * 32; i += blockDim.x) {
+    const int l = i & 31, nt = (i >> 5) % NTV, kk = (i >> 5) / NTV, ho = head_of((part * NTV + nt) * 8 + (l >> 2));
+    uint32_t w[2];
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+      const int k = kk * 16 + e * 8 + (l & 3) * 2, h0 = head_of(k), h1 = head_of(k + 1);
+      const __nv_bfloat162 v = __floats2bfloat162_rn(ho >= 0 && h0 >= 0 ? a.mix[ho * a.H + h0] : 0.f, ho >= 0 && h1 >= 0 ? a.mix[ho * a.H + h1] : 0.f);
+      w[e] = *(const uint32_t*)&v;
+    }
+    sT[i] = make_uint2(w[0], w[1]);
+  }
+  pdl_trigger();
+  pdl_wait();
+  const int len = a.seq_lens[b];
+  const int first = a.window > 0 && len > a.window ? len - a.window : 0;
+  const int p_first = first >> 4, p_last = (len + 15) >> 4;
+  const int per = (p_last - p_first + a.S - 1) / a.S;
+  const int pa = p_first + split * per, np = max(0, min(p_last, pa + per) - pa);
+  const int* pt = a.page_table + (size_t)b * a.max_pages;
+  for (int i = tid; i < np; i += blockDim.x) s_pid[i] = pt[pa + i];
+  __syncthreads();
+  auto issue = [&](int i) {   // one lane: page i of the share into its slot
+    const uint32_t bar = smem_u32(bars + i % a.nslot);
+    mbar_expect_tx(bar, page_bytes);
+    tma_load_4d(smem_u32(ring + (size_t)(i % a.nslot) * page_bytes), &tm, bar, 0, 0, 0, s_pid[i] * 2);
+  };
+  if (lane == 0)
+    for (int i = warp; i < min(np, a.nslot); i += nw) issue(i);
+  for (int i = tid; i < (8 * NT + 1) * (DK / 2); i += blockDim.x) {
+    const int slot = i / (DK / 2), c = i % (DK / 2) * 2, h = slot < 8 * NT ? head_of(slot) : -1;
+    const float2 v = h >= 0 ? *(const float2*)(a.q + ((size_t)b * a.H + h) * DK + c) : make_float2(0.f, 0.f);
+    *(__half2*)(sQ + slot * QLD + c) = __floats2half2_rn(v.x, v.y);
+  }
+  __syncthreads();
+
+  float o[NTV][DK / 16][4], mu[NTV][2], l[NTV][2], sl[NTV][2];
+#pragma unroll
+  for (int nt = 0; nt < NTV; nt++) {
+#pragma unroll
+    for (int m = 0; m < DK / 16; m++) o[nt][m][0] = o[nt][m][1] = o[nt][m][2] = o[nt][m][3] = 0.f;
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+      const int h = head_of((part * NTV + nt) * 8 + 2 * t4 + e);
+      mu[nt][e] = -INFINITY;
+      l[nt][e] = 0.f;
+      sl[nt][e] = h >= 0 && a.slopes ? a.slopes[h] * kLog2e : 0.f;
+    }
+  }
+  const int mi = lane >> 3, r8 = lane & 7;              // ldmatrix: tile and row of this lane's address
+  for (int i = warp; i < np; i += nw) {
+    const int s = i % a.nslot;
+    bool ok = mbar_wait(smem_u32(bars + s), (uint32_t)((i / a.nslot) & 1), &s_abort);
+    ok = __all_sync(0xffffffffu, ok);
+    if (!ok) break;
+    const uint32_t page = smem_u32(ring) + (uint32_t)(s * page_bytes);
+    // 16 bytes of key row `row` of the page: piece `ch` of key head c
+    auto piece = [&](int row, int c, int ch) {
+      return page + (uint32_t)((row >> 3) * NB + c * KB + (ch >> 3)) * 1024u + (uint32_t)(row & 7) * 128u + (uint32_t)(((ch & 7) ^ (row & 7)) << 4);
+    };
+    float sc[NT][4];
+#pragma unroll
+    for (int j = 0; j < NT; j++) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+    for (int u = 0; u < nsub; u++)
+#pragma unroll 1
+      for (int kk = 0; kk < DK / 32; kk++)
+#pragma unroll
+        for (int j = 0; j < NT; j++) {
+          const int c = rp < 8 ? j * nsub + u : j * 8 / rp;
+          if (c >= a.G) continue;
+          uint32_t k0[4], k1[4], q[4];
+          const int row = r8 + (mi & 1) * 8, slot = j * 8 + r8;
+          ldsm_x4(piece(row, c, kk * 4 + (mi >> 1)), k0[0], k0[1], k0[2], k0[3]);
+          ldsm_x4(piece(row, c, kk * 4 + 2 + (mi >> 1)), k1[0], k1[1], k1[2], k1[3]);
+          ldsm_x4(smem_u32(sQ + (slot / rp == c ? slot : 8 * NT) * QLD + kk * 32 + mi * 8), q[0], q[1], q[2], q[3]);
+          mma16816(sc[j], k0, q[0], q[1]);
+          mma16816(sc[j], k1, q[2], q[3]);
+        }
+    float d[NTV][4];
+#pragma unroll
+    for (int nt = 0; nt < NTV; nt++) d[nt][0] = d[nt][1] = d[nt][2] = d[nt][3] = 0.f;
+#pragma unroll
+    for (int kk = 0; kk < NT / 2; kk++) {
+      uint32_t hi[4], md[4], lo[4];
+#pragma unroll
+      for (int x = 0; x < 4; x++) {
+        const float* v = &sc[2 * kk + (x >> 1)][(x & 1) * 2];
+        float2 r = split_bf16(v[0], v[1], hi[x]);
+        r = split_bf16(r.x, r.y, md[x]);
+        split_bf16(r.x, r.y, lo[x]);
+      }
+      uint2 w[NTV];
+#pragma unroll
+      for (int nt = 0; nt < NTV; nt++) w[nt] = sT[(kk * NTV + nt) * 32 + lane];
+#pragma unroll
+      for (int nt = 0; nt < NTV; nt++) mma16816_bf16(d[nt], lo, w[nt].x, w[nt].y);
+#pragma unroll
+      for (int nt = 0; nt < NTV; nt++) mma16816_bf16(d[nt], md, w[nt].x, w[nt].y);
+#pragma unroll
+      for (int nt = 0; nt < NTV; nt++) mma16816_bf16(d[nt], hi, w[nt].x, w[nt].y);
+    }
+    const int t0 = (pa + i) * 16 + g4, t1 = t0 + 8;
+    const bool in0 = t0 >= first && t0 < len, in1 = t1 >= first && t1 < len;
+    const float f0 = (float)(len - 1 - t0), f1 = (float)(len - 1 - t1);
+    bool grown = false;
+#pragma unroll
+    for (int nt = 0; nt < NTV; nt++)
+#pragma unroll
+      for (int e = 0; e < 2; e++) {
+        d[nt][e] = in0 ? fmaf(d[nt][e], kLog2e, -sl[nt][e] * f0) : -INFINITY;
+        d[nt][e + 2] = in1 ? fmaf(d[nt][e + 2], kLog2e, -sl[nt][e] * f1) : -INFINITY;
+        grown |= fmaxf(d[nt][e], d[nt][e + 2]) > mu[nt][e] + 8.f;
+      }
+    if (__any_sync(0xffffffffu, grown)) {
+#pragma unroll
+      for (int nt = 0; nt < NTV; nt++)
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+          float mx = fmaxf(d[nt][e], d[nt][e + 2]);
+          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 4));
+          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
+          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 16));
+          mx = fmaxf(mx, mu[nt][e]);
+          const float c = mu[nt][e] == -INFINITY ? 0.f : ex2_approx(mu[nt][e] - mx);
+          mu[nt][e] = mx;
+          l[nt][e] *= c;
+#pragma unroll
+          for (int m = 0; m < DK / 16; m++) {
+            o[nt][m][e] *= c;
+            o[nt][m][e + 2] *= c;
+          }
+        }
+    }
+#pragma unroll
+    for (int nt = 0; nt < NTV; nt++) {
+      float p[4];
+#pragma unroll
+      for (int e = 0; e < 2; e++) {
+        const float off = mu[nt][e] == -INFINITY ? 0.f : mu[nt][e];
+        p[e] = ex2_approx(d[nt][e] - off);
+        p[e + 2] = ex2_approx(d[nt][e + 2] - off);
+        l[nt][e] += p[e] + p[e + 2];
+      }
+      const uint32_t w[2] = {transpose_8x8(pack_h2(p[0], p[1])), transpose_8x8(pack_h2(p[2], p[3]))};      // keys 0..7, 8..15 of head g4
+      const int tile = part * NTV + nt;
+      if (tile * 8 >= live) continue;
+      if (rp >= 8) {
+        const int c = tile * 8 / rp;
+#pragma unroll
+        for (int m = 0; m < DK / 16; m++) {
+          uint32_t k[4];
+          ldsm_x4_t(piece(r8 + (mi >> 1) * 8, c, m * 2 + (mi & 1)), k[0], k[1], k[2], k[3]);
+          mma16816(o[nt][m], k, w[0], w[1]);
+        }
+      } else {
+#pragma unroll 1
+        for (int pr = 0; pr < max(1, nsub >> 1); pr++) {
+          const int c0 = tile * nsub + 2 * pr, c1 = min(c0 + 1, a.G - 1);
+          if (c0 >= a.G) break;
+          const bool own0 = g4 / rp == 2 * pr, own1 = g4 / rp == 2 * pr + 1;
+#pragma unroll
+          for (int kg = 0; kg < 2; kg++)
+#pragma unroll
+            for (int m = 0; m < DK / 16; m++) {
+              uint32_t k[4];
+              ldsm_x4_t(piece(r8 + kg * 8, mi < 2 ? c0 : c1, m * 2 + (mi & 1)), k[0], k[1], k[2], k[3]);
+              mma16816(o[nt][m], k, own0 ? w[kg] : 0u, own1 ? w[kg] : 0u);
+            }
+        }
+      }
+    }
+    __syncwarp();
+    if (lane == 0 && i + a.nslot < np) issue(i + a.nslot);
+  }
+  if (tid == 0 && s_abort && a.status) atomicExch(a.status, (int)B200_ERR_TIMEOUT_TMA);
+  if (s_abort) drain_after_abort();
+  __syncthreads();                                      // every page has been read: the ring becomes the partial outputs
+#pragma unroll
+  for (int nt = 0; nt < NTV; nt++)
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+      float v = l[nt][e];
+      v += __shfl_xor_sync(0xffffffffu, v, 4);
+      v += __shfl_xor_sync(0xffffffffu, v, 8);
+      v += __shfl_xor_sync(0xffffffffu, v, 16);
+      const int slot = nt * 8 + 2 * t4 + e;
+      if (g4 == 0) {
+        s_ml[warp][slot][0] = mu[nt][e];
+        s_ml[warp][slot][1] = v;
+      }
+      float* acc = s_acc + ((size_t)warp * NTV * 8 + slot) * DK;
+#pragma unroll
+      for (int m = 0; m < DK / 16; m++) {
+        acc[m * 16 + g4] = o[nt][m][e];
+        acc[m * 16 + g4 + 8] = o[nt][m][e + 2];
+      }
+    }
+  __syncthreads();
+  const int parts = gridDim.y, n_out = NTV * 8 * DK;
+  const size_t row = ((size_t)b * parts + part) * a.S;
+  auto finish = [&](int slot, int e, float M, float L, float A) {
+    const int h = head_of(part * NTV * 8 + slot);
+    if (h < 0) return;
+    if (a.sinks) {
+      const float sk = a.sinks[h] * kLog2e, M2 = fmaxf(M, sk), c = M == -INFINITY ? 0.f : ex2_approx(M - M2);
+      L = L * c + ex2_approx(sk - M2);
+      A *= c;
+    }
+    const float v = L > 0.f ? A / L : 0.f;
+    const size_t at = ((size_t)b * a.H + h) * DK + e;
+    if (a.out_f32) a.out_f32[at] = v;
+    if (a.out_bf16) a.out_bf16[at] = __float2bfloat16(v);
+  };
+  for (int x = tid; x < n_out; x += blockDim.x) {
+    const int slot = x / DK, e = x % DK;
+    float M = -INFINITY, L = 0.f, A = 0.f;
+    for (int w = 0; w < nw; w++) M = fmaxf(M, s_ml[w][slot][0]);
+    for (int w = 0; w < nw; w++) {
+      const float c = s_ml[w][slot][0] == -INFINITY ? 0.f : ex2_approx(s_ml[w][slot][0] - M);
+      L += s_ml[w][slot][1] * c;
+      A += s_acc[((size_t)w * NTV * 8 + slot) * DK + e] * c;
+    }
+    if (a.S == 1) {
+      finish(slot, e, M, L, A);
+    } else {
+      a.part_acc[(row + split) * n_out + x] = A;
+      if (e == 0) {
+        a.part_ml[((row + split) * NTV * 8 + slot) * 2] = M;
+        a.part_ml[((row + split) * NTV * 8 + slot) * 2 + 1] = L;
+      }
+    }
+  }
+  if (a.S == 1) return;
+  __threadfence();
+  __syncthreads();
+  if (tid == 0) {                                        // the CTA that comes last merges the shares
+    int* cnt = a.counters + (size_t)b * parts + part;
+    s_last = atomicAdd(cnt, 1) == a.S - 1;
+    if (s_last) *cnt = 0;
+  }
+  __syncthreads();
+  if (!s_last) return;
+  __threadfence();
+  for (int x = tid; x < n_out; x += blockDim.x) {
+    const int slot = x / DK, e = x % DK;
+    float M = -INFINITY, L = 0.f, A = 0.f;
+    for (int s = 0; s < a.S; s++) M = fmaxf(M, __ldcg(a.part_ml + ((row + s) * NTV * 8 + slot) * 2));
+    for (int s = 0; s < a.S; s++) {
+      const float* ml = a.part_ml + ((row + s) * NTV * 8 + slot) * 2;
+      const float m = __ldcg(ml), c = m == -INFINITY ? 0.f : ex2_approx(m - M);
+      L += __ldcg(ml + 1) * c;
+      A += __ldcg(a.part_acc + (row + s) * n_out + x) * c;
+    }
+    finish(slot, e, M, L, A);
+  }
+}
+
+// Padded group size, tiles of eight padded heads (even), and tiles a CTA keeps the outputs of; false: sizes the kernel does not take.
+static bool mixed_decode_plan(int H, int G, int DK, int& rp, int& nt, int& ntv) {
+  if (G < 1 || H < 1 || H % G || (DK != 64 && DK != 128)) return false;
+  const int rep = H / G;
+  rp = rep <= 1 ? 1 : rep <= 2 ? 2 : rep <= 4 ? 4 : (rep + 7) / 8 * 8;
+  const int tiles = (G * rp + 7) / 8;
+  nt = tiles <= 2 ? 2 : tiles <= 4 ? 4 : 8;
+  ntv = DK == 128 && nt == 8 ? 4 : nt;
+  return tiles <= 8 && G * DK <= 1536;
+}
+B200_API int b200_mixed_decode_ok(int H, int G, int DK) {
+  int rp, nt, ntv;
+  return mixed_decode_plan(H, G, DK, rp, nt, ntv) ? 1 : 0;
+}
+B200_API size_t b200_mixed_decode_scratch_floats(int B, int H, int G, int DK, int S) {
+  int rp, nt, ntv;
+  if (!mixed_decode_plan(H, G, DK, rp, nt, ntv)) return 0;
+  return (size_t)B * S * nt * 8 * (DK + 2);
+}
+template <int DK, int NT, int NTV>
+static int launch_mixed_decode(MixedDecArgs a, const void* kc, int n_pages, int B, float* scratch, cudaStream_t st) {
+  const int W = a.G * DK, page = 32 * W, parts = NT / NTV;
+  constexpr int kOut = NTV * 8 * DK * 4;
+  // two CTAs of four warps to an SM where half its shared memory holds enough pages, else one of up to eight
+  const size_t fixed = 1024 + 34 * 8 + (8 * NT + 2) * (DK + 8) * 2 + 16 + NT / 2 * NTV * 256 + ((size_t)a.max_pages + 1) * 4;
+  if (fixed > 100 * 1024) return B200_ERR_BAD_ARG;
+  int nw = 0;
+  if (fixed + 8 * (size_t)page <= 106 * 1024 && fixed + 4 * (size_t)kOut <= 106 * 1024) {
+    nw = 4;
+    a.nslot = (106 * 1024 - fixed) / page >= 16 ? 16 : (int)((106 * 1024 - fixed) / page) / 4 * 4;
+  } else {
+    const size_t room = 220 * 1024 - fixed;
+    const int cap = (int)(room / page < 16 ? room / page : 16);
+    for (int w = 8; w >= 2; w--)
+      if (cap >= w && (size_t)w * kOut <= room && (!nw || cap / w * w > a.nslot)) {
+        nw = w;
+        a.nslot = cap / w * w;
+      }
+    if (!nw) return B200_ERR_BAD_ARG;
+  }
+  a.part_acc = scratch;
+  a.part_ml = scratch ? scratch + (size_t)B * parts * a.S * NTV * 8 * DK : nullptr;
+  const size_t ring = (size_t)a.nslot * page > (size_t)nw * kOut ? (size_t)a.nslot * page : (size_t)nw * kOut, smem = fixed + ring;
+  auto kern = mixed_decode_kernel<DK, NT, NTV>;
+  static size_t configured = 0;
+  if (smem > configured) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    configured = smem;
+  }
+  CUtensorMap tm;
+  const int rc = make_tmap_rows8(&tm, kc, (uint64_t)n_pages * 16, W, W / 64);
+  if (rc) return rc;
+  return launch_pdl(kern, dim3(a.S, parts, B), dim3(32 * nw), smem, st, tm, a);
+}
+// q fp32 [B][H][DK], scaled; mix fp32 [H][H] (bf16 values); kc fp16 [n_pages][16][G * DK]; sizes as b200_mixed_decode_ok has them.  S: shares of the
+// keys (scratch and counters [2 B], zero before first use, where there are several).
+B200_API int b200_mixed_decode(const float* q, const void* kc, const float* mix, const float* slopes, const float* sinks, const int* page_table,
+                               int max_pages, int n_pages, const int* seq_lens, int B, int H, int G, int DK, int window, int S, float* out_f32,
+                               void* out_bf16, float* scratch, int* counters, int* status, cudaStream_t st) {
+  MixedDecArgs a = {};
+  int nt, ntv;
+  if (B < 1 || S < 1 || window < 0 || max_pages < 1 || !q || !kc || !mix || (!out_f32 && !out_bf16) || (S > 1 && (!scratch || !counters)) ||
+      !mixed_decode_plan(H, G, DK, a.rp, nt, ntv) || ((uintptr_t)q & 7))
+    return B200_ERR_BAD_ARG;
+  a.q = q; a.mix = mix; a.slopes = slopes; a.sinks = sinks; a.page_table = page_table; a.seq_lens = seq_lens; a.max_pages = max_pages; a.H = H; a.G = G;
+  a.window = window; a.S = S; a.out_f32 = out_f32; a.out_bf16 = (__nv_bfloat16*)out_bf16; a.counters = counters; a.status = status;
+  if (DK == 64) {
+    if (nt == 2) return launch_mixed_decode<64, 2, 2>(a, kc, n_pages, B, scratch, st);
+    if (nt == 4) return launch_mixed_decode<64, 4, 4>(a, kc, n_pages, B, scratch, st);
+    return launch_mixed_decode<64, 8, 8>(a, kc, n_pages, B, scratch, st);
+  }
+  if (nt == 2) return launch_mixed_decode<128, 2, 2>(a, kc, n_pages, B, scratch, st);
+  if (nt == 4) return launch_mixed_decode<128, 4, 4>(a, kc, n_pages, B, scratch, st);
+  return launch_mixed_decode<128, 8, 4>(a, kc, n_pages, B, scratch, st);
+}
+
+// ------------------------------------------------------------------ prompts: wide queries on the 5th-generation tensor cores
+
+// One CTA = 128 query rows of one head against blocks of 128 keys, in the manner of attn_prefill_tc05.cu: two TMA warps, one warp that issues the
+// score products, one for the output products, eight softmax warps (two to a tensor-memory quarter, half of a block's keys and of the output columns
+// each).  What differs:
+//   - a score is a product over G slices (a key head's DK columns each); slices are the entries of the ring, [16 groups][DK / 64][8 rows][128
+//     bytes] = 128 keys, one TMA copy per page.  The head's own slice comes last in a block: it is the value operand too, and its entry is given back
+//     by the output product instead of the score product.
+//   - the wide query row lies in tensor memory as far as that reaches (QT slices), the rest in shared memory, both read as the A operand.
+//   - where the slices leave no room for two score accumulators (NS = 1), a block's score product waits for the output product before it.
+//   - slopes: one multiply-add per score, the block's part of the distance joins the exponent's offset.
+constexpr int QB = 128, KEYS = 128;
+constexpr uint32_t kTmemCols = 512;
+constexpr float kRescale = 8.f;                   // log2 units
+
+struct MixedPreArgs {
+  const __half* q;         // [T_total][H][G * DK], mixed and scaled
+  const float* slopes;     // [H] or null
+  const float* sinks;      // [H] or null
+  const int* page_table;
+  const int* q_start;
+  const int* q_len;
+  const int* ctx_len;
+  int max_pages, H, G, T_total, window, QT, R;    // R: ring entries
+  __nv_bfloat16* out;      // [T_total][H * DK]
+  float* out_f32;          // instead of out where given
+  int* status;
+};
+
+template <int DK, int NS>
+__global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmQ,
+                                                               const MixedPreArgs a) {
+  constexpr int CB = DK / 64, SLICE = KEYS * DK * 2, GROUP = CB * 1024;        // GROUP: bytes of eight key rows of a slice
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+  const int QS = a.G - a.QT, R = a.R;
+  uint8_t* sQ = smem;                                     // QS slices of the queries, [CB][128 rows][128 bytes] each
+  uint8_t* sK = sQ + (size_t)QS * SLICE;                  // R ring entries
+  uint64_t* bars = (uint64_t*)(sK + (size_t)R * SLICE);
+  uint64_t* q_full = bars;                                // [1] the part in tensor memory
+  uint64_t* qs_full = bars + 1;                           // [1] the part in shared memory
+  uint64_t* s_full = bars + 2;                            // [2]
+  uint64_t* s_empty = bars + 4;                           // [2]
+  uint64_t* p_full = bars + 6;                            // [2]
+  uint64_t* pv_done = bars + 8;                           // [2]
+  uint64_t* x_full = bars + 10;                           // [4 quarters][2]
+  uint32_t* tmem_holder = (uint32_t*)(bars + 18);
+  volatile int* abort_flag = (volatile int*)(tmem_holder + 1);
+  uint64_t* k_full = bars + 20;                           // [R]
+  uint64_t* k_empty = k_full + R;                         // [R]
+  float* xch = (float*)(bars + 20 + 2 * R);               // [NS][2 (half)][128 rows]
+
+  const int seq = blockIdx.z, h = blockIdx.y, qb = gridDim.x - 1 - blockIdx.x;   // longest (latest) query blocks first
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x == 0) {
+    mbar_init(smem_u32(q_full), 4);
+    mbar_init(smem_u32(qs_full), 1);
+    for (int s = 0; s < R; s++) {
+      mbar_init(smem_u32(k_full + s), 1);
+      mbar_init(smem_u32(k_empty + s), 1);
+    }
+    for (int s = 0; s < 2; s++) {
+      mbar_init(smem_u32(s_full + s), 1);
+      mbar_init(smem_u32(s_empty + s), 8);
+      mbar_init(smem_u32(p_full + s), 8);
+      mbar_init(smem_u32(pv_done + s), 1);
+    }
+    for (int s = 0; s < 8; s++) mbar_init(smem_u32(x_full + s), 2);
+    *abort_flag = 0;
+    fence_barrier_init();
+    tma_prefetch_desc(&tmK);
+    tma_prefetch_desc(&tmQ);
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(tmem_holder), kTmemCols);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_holder;
+  pdl_trigger();
+  pdl_wait();
+
+  const int qlen = a.q_len[seq], q0 = qb * QB;
+  const bool live = q0 < qlen;            // a dead CTA still goes through the common exit (it holds tensor memory)
+  const int ctx = a.ctx_len[seq], qs = a.q_start[seq], G = a.G, W = G * DK;
+  const int own = h / (a.H / G);
+  const int pos0 = ctx - qlen + q0;       // absolute position of this CTA's first query row
+  const int k_hi = min(ctx, pos0 + QB), k_lo = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
+  const int jb0 = k_lo / KEYS, nb = live ? (k_hi + KEYS - 1) / KEYS - jb0 : 0;
+  const uint32_t S_T = tmem_base, O_T = tmem_base + NS * KEYS, Q_T = O_T + DK;
+
+  if (warp == 0 || warp == 10) {
+    // entries e = j * G + u in order (block j, u-th slice of it).  Slots are shared out, not entries: a slot's uses must be waited for one after the other by
+    // one thread (a parity tells neighbouring phases apart, no more), and entries are not given back in order (the own slices come later).
+    if (lane == 0 && nb > 0) {
+      const int* pt = a.page_table + (size_t)seq * a.max_pages;
+      if (warp == 0 && QS > 0) {
+        const uint32_t bar = smem_u32(qs_full);
+        mbar_expect_tx(bar, QS * SLICE);
+        for (int u = a.QT; u < G; u++)
+          for (int c = 0; c < CB; c++)
+            tma_load_2d(smem_u32(sQ + (size_t)(u - a.QT) * SLICE + c * (QB * 128)), &tmQ, bar, h * W + (own + 1 + u) % G * DK + c * 64, qs + q0);
+      }
+      for (int e = 0; e < nb * G; e++) {
+        const int j = e / G, sl = (own + 1 + e - j * G) % G, s = e % R;
+        if ((s & 1) != (warp == 0 ? 0 : 1)) continue;
+        if (!mbar_wait(smem_u32(k_empty + s), (uint32_t)((e / R) & 1) ^ 1, abort_flag)) break;
+        const uint32_t bar = smem_u32(k_full + s), dst = smem_u32(sK + (size_t)s * SLICE);
+        mbar_expect_tx(bar, SLICE);
+#pragma unroll
+        for (int p = 0; p < KEYS / 16; p++) {
+          const int pi = (jb0 + j) * (KEYS / 16) + p;
+          tma_load_4d(dst + p * 2 * GROUP, &tmK, bar, 0, 0, sl * CB, (pi * 16 < ctx ? pt[pi] : 0) * 2);      // pages past the context are masked anyway
+        }
+      }
+    }
+  } else if (warp == 1) {
+    if (lane == 0 && nb > 0) {
+      constexpr uint32_t idesc = idesc_f16(QB, KEYS, false);
+      bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag) && (QS == 0 || mbar_wait(smem_u32(qs_full), 0, abort_flag));
+      for (int j = 0; j < nb && ok; j++) {
+        const int b = j % NS, use = j / NS;
+        if (!mbar_wait(smem_u32(s_empty + b), (uint32_t)(use & 1) ^ 1, abort_flag)) break;
+        if (j >= NS && !mbar_wait(smem_u32(pv_done + b), (uint32_t)(use - 1) & 1, abort_flag)) break;      // the weights before lie in this accumulator
+        for (int u = 0; u < G; u++) {
+          const int e = j * G + u, s = e % R;
+          ok = mbar_wait(smem_u32(k_full + s), (uint32_t)(e / R) & 1, abort_flag);
+          if (!ok) break;
+          tc_fence_after();
+          const uint32_t ka = smem_u32(sK + (size_t)s * SLICE);
+          if (u < a.QT) {
+#pragma unroll
+            for (int kk = 0; kk < DK / 16; kk++)
+              umma_ts(S_T + b * KEYS, Q_T + u * (DK / 2) + 8 * kk, smem_desc_sw128_strided(ka + (kk >> 2) * 1024, 16, GROUP) + 2 * (kk & 3), idesc,
+                      u != 0 || kk != 0 ? 1u : 0u);
+          } else {
+            const uint32_t qa = smem_u32(sQ + (size_t)(u - a.QT) * SLICE);
+#pragma unroll
+            for (int kk = 0; kk < DK / 16; kk++)
+              umma_bf16(S_T + b * KEYS, smem_desc_sw128(qa + (kk >> 2) * (QB * 128)) + 2 * (kk & 3),
+                        smem_desc_sw128_strided(ka + (kk >> 2) * 1024, 16, GROUP) + 2 * (kk & 3), idesc, u != 0 || kk != 0 ? 1u : 0u);
+          }
+          if (u != G - 1) umma_commit(smem_u32(k_empty + s));
+        }
+        umma_commit(smem_u32(s_full + b));
+      }
+    }
+  } else if (warp == 11) {
+    if (lane == 0 && nb > 0) {
+      constexpr uint32_t idesc = idesc_f16(QB, DK, true);
+      for (int j = 0; j < nb; j++) {
+        const int b = j % NS, e = j * G + G - 1, s = e % R;
+        if (!mbar_wait(smem_u32(p_full + b), (uint32_t)(j / NS) & 1, abort_flag)) break;      // weights written, output rows rescaled if needed
+        if (!mbar_wait(smem_u32(k_full + s), (uint32_t)(e / R) & 1, abort_flag)) break;       // (landed long ago: the scores needed it; only now is the parity its own)
+        tc_fence_after();
+        const uint32_t va = smem_u32(sK + (size_t)s * SLICE);
+#pragma unroll
+        for (int kk = 0; kk < KEYS / 16; kk++)
+          umma_ts(O_T, S_T + b * KEYS + (kk >> 2) * 64 + 8 * (kk & 3), smem_desc_sw128_strided(va + kk * 2 * GROUP, 1024, GROUP), idesc,
+                  (j != 0 || kk != 0) ? 1u : 0u);
+        umma_commit(smem_u32(pv_done + b));
+        umma_commit(smem_u32(k_empty + s));
+      }
+    }
+  } else if (warp < 10 && nb > 0) {
+    const int q = warp & 3;                      // tensor-memory lane quarter this warp may read
+    const int hsel = (warp - 2) >> 2;            // which half of a block's keys and of the output columns
+    const int row = q * 32 + lane, qpos = pos0 + row;
+    const int row_lo = a.window > 0 ? qpos - a.window + 1 : 0, lo_max = a.window > 0 ? pos0 + QB - a.window : 0;      // first key of this row, of the last row
+    const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
+    constexpr int HK = KEYS / 2, HO = DK / 2;
+    const float slope = a.slopes ? a.slopes[h] : 0.f;
+    float m_used = -INFINITY, l = 0.f;           // exponent offset of this row (log2 units), this warp's part of the row sum
+    bool ok = true;
+    if (hsel == 0) {
+      const bool in = qs + q0 + row < a.T_total;
+      const __half* qrow = a.q + ((size_t)(qs + q0 + (in ? row : 0)) * a.H + h) * W;
+      for (int u = 0; u < a.QT; u++) {
+        const uint4* src = (const uint4*)(qrow + (own + 1 + u) % G * DK);
+#pragma unroll
+        for (int c = 0; c < CB; c++) {
+          uint32_t r[32];
+#pragma unroll
+          for (int i = 0; i < 8; i++) {
+            const uint4 v = in ? src[c * 8 + i] : make_uint4(0u, 0u, 0u, 0u);
+            r[4 * i] = v.x; r[4 * i + 1] = v.y; r[4 * i + 2] = v.z; r[4 * i + 3] = v.w;
+          }
+          tmem_st32(Q_T + lane_addr + u * (DK / 2) + c * 32, r);
+          tmem_st_wait();
+        }
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(q_full));
+    }
+    // both warps of a pair have written their half to xch; `n`: how many times barrier bb has been used
+    auto pair_sync = [&](int bb, int n) -> bool {
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(x_full + q * 2 + bb));
+      const bool k = mbar_wait(smem_u32(x_full + q * 2 + bb), (uint32_t)n & 1, abort_flag);
+      return __all_sync(0xffffffffu, k && !*abort_flag);
+    };
+    for (int j = 0; j < nb; j++) {
+      const int b = j % NS, use = j / NS;
+      ok = mbar_wait(smem_u32(s_full + b), (uint32_t)use & 1, abort_flag);
+      ok = __all_sync(0xffffffffu, ok && !*abort_flag);
+      if (!ok) break;
+      tc_fence_after();
+      float sv[HK];
+      {
+        uint32_t r[32];
+#pragma unroll
+        for (int c = 0; c < HK / 32; c++) {
+          tmem_ld32(S_T + b * KEYS + lane_addr + hsel * HK + c * 32, r);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; i++) sv[c * 32 + i] = fmaf(slope, (float)(c * 32 + i), __uint_as_float(r[i]));
+        }
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(s_empty + b));
+      const int kb0 = (jb0 + j) * KEYS;
+      const float base = slope * (float)(kb0 + hsel * HK - qpos);      // the distance's part that all of this warp's keys of the block share
+      if (kb0 + KEYS - 1 > pos0 || kb0 + KEYS > ctx || kb0 < lo_max) {
+#pragma unroll
+        for (int i = 0; i < HK; i++) {
+          const int kp = kb0 + hsel * HK + i;
+          if (kp > qpos || kp >= ctx || kp < row_lo) sv[i] = -INFINITY;
+        }
+      }
+      float mx0 = fmaxf(sv[0], sv[1]), mx1 = fmaxf(sv[2], sv[3]);
+#pragma unroll
+      for (int i = 4; i < HK; i += 4) {
+        mx0 = max3(mx0, sv[i], sv[i + 1]);
+        mx1 = max3(mx1, sv[i + 2], sv[i + 3]);
+      }
+      const float mine = fmaxf(mx0, mx1) + base;
+      float* xb = xch + b * 256;
+      xb[hsel * 128 + row] = mine;
+      ok = pair_sync(b, use);
+      if (!ok) break;
+      const float bmax = fmaxf(mine, xb[(hsel ^ 1) * 128 + row]) * kLog2e;
+      const bool unset = m_used == -INFINITY;
+      const bool behind = bmax > m_used + kRescale;
+      if (j > 0 && __any_sync(0xffffffffu, behind && !unset)) {
+        const float m_new = fmaxf(m_used, bmax);
+        const float scale = (m_new == -INFINITY) ? 1.f : ex2_approx(m_used - m_new);
+        ok = mbar_wait(smem_u32(pv_done + (j - 1) % NS), (uint32_t)((j - 1) / NS) & 1, abort_flag);       // the output product before has finished
+        ok = __all_sync(0xffffffffu, ok && !*abort_flag);
+        if (!ok) break;
+        tc_fence_after();
+#pragma unroll
+        for (int c = 0; c < HO / 32; c++) {
+          uint32_t r[32];
+          tmem_ld32(O_T + lane_addr + hsel * HO + c * 32, r);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; i++) r[i] = __float_as_uint(__uint_as_float(r[i]) * scale);
+          tmem_st32(O_T + lane_addr + hsel * HO + c * 32, r);
+        }
+        tmem_st_wait();
+        tc_fence_before();
+        l *= scale;
+        m_used = m_new;
+      } else if (unset) {
+        m_used = bmax;                             // nothing accumulated yet under the old offset
+      }
+      const float off = (m_used == -INFINITY) ? 0.f : fmaf(base, kLog2e, -m_used);
+      float sum0 = 0.f, sum1 = 0.f, sum2 = 0.f, sum3 = 0.f;
+      uint32_t pw[HK / 2];
+#pragma unroll
+      for (int i = 0; i < HK / 2; i++) {
+        const float p0 = ex2_approx(fmaf(sv[2 * i], kLog2e, off)), p1 = ex2_approx(fmaf(sv[2 * i + 1], kLog2e, off));
+        if (i & 1) { sum2 += p0; sum3 += p1; } else { sum0 += p0; sum1 += p1; }
+        const __half2 hh = __floats2half2_rn(p0, p1);
+        pw[i] = *(const uint32_t*)&hh;
+      }
+      tmem_st32(S_T + b * KEYS + lane_addr + hsel * HK, pw);
+      tmem_st_wait();
+      l += (sum0 + sum1) + (sum2 + sum3);
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(p_full + b));
+    }
+    if (ok) {
+      ok = mbar_wait(smem_u32(pv_done + (nb - 1) % NS), (uint32_t)((nb - 1) / NS) & 1, abort_flag);          // the last output product
+      ok = __all_sync(0xffffffffu, ok && !*abort_flag);
+    }
+    if (__all_sync(0xffffffffu, ok)) {
+      const int b = nb % NS;                       // the buffer the last block did not use (or the only one, whose readers are done)
+      float* xl = xch + b * 256;
+      xl[hsel * 128 + row] = l;
+      ok = pair_sync(b, nb / NS);
+      l += xl[(hsel ^ 1) * 128 + row];
+      tc_fence_after();
+      if (a.sinks) l += (m_used == -INFINITY) ? 1.f : ex2_approx(a.sinks[h] * kLog2e - m_used);
+      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const bool wr = ok && row < qlen - q0;
+      const size_t at = (size_t)(qs + q0 + row) * a.H * DK + (size_t)h * DK + hsel * HO;
+#pragma unroll
+      for (int c = 0; c < HO / 32; c++) {
+        uint32_t r[32];
+        tmem_ld32(O_T + lane_addr + hsel * HO + c * 32, r);
+        tmem_ld_wait();
+        if (wr && a.out_f32) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 4)
+            *(float4*)(a.out_f32 + at + c * 32 + i) = make_float4(__uint_as_float(r[i]) * inv, __uint_as_float(r[i + 1]) * inv,
+                                                                  __uint_as_float(r[i + 2]) * inv, __uint_as_float(r[i + 3]) * inv);
+        } else if (wr) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 8) {
+            uint4 v;
+            __nv_bfloat162* p = (__nv_bfloat162*)&v;
+#pragma unroll
+            for (int k = 0; k < 4; k++) p[k] = __floats2bfloat162_rn(__uint_as_float(r[i + 2 * k]) * inv, __uint_as_float(r[i + 2 * k + 1]) * inv);
+            *(uint4*)(a.out + at + c * 32 + i) = v;
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (*abort_flag) drain_after_abort();
+  if (warp == 1) tmem_dealloc(tmem_base, kTmemCols);
+  if (threadIdx.x == 0 && *abort_flag && a.status) atomicExch(a.status, (int)B200_ERR_TIMEOUT_MMA);
+}
+
+// Score accumulators, slices of the queries in tensor memory, ring entries; false: sizes the kernel does not take.
+static bool mixed_prefill_plan(int G, int DK, int& ns, int& qt, int& r) {
+  if (G < 1 || (DK != 64 && DK != 128)) return false;
+  const int slice = KEYS * DK * 2;
+  for (ns = 2; ns >= 1; ns--) {
+    const int most = (232448 - 1024 - 36 * 8 - ns * 1024) / slice;
+    qt = (512 - ns * KEYS - DK) / (DK / 2);
+    if (qt > G) qt = G;
+    r = most - (G - qt);
+    if (r > 8) r = 8;
+    if (r >= 3) return true;
+  }
+  return false;
+}
+B200_API int b200_mixed_prefill_ok(int G, int DK) {
+  int ns, qt, r;
+  return mixed_prefill_plan(G, DK, ns, qt, r) ? 1 : 0;
+}
+template <int DK, int NS>
+static int launch_mixed_prefill(const CUtensorMap& tk, const CUtensorMap& tq, const MixedPreArgs& a, int n_seqs, int max_q, cudaStream_t st) {
+  const size_t smem = 1024 + (size_t)(a.G - a.QT + a.R) * KEYS * DK * 2 + (20 + 2 * a.R) * 8 + NS * 1024;
+  if (smem > 232448) return B200_ERR_BAD_ARG;
+  auto kern = mixed_prefill_kernel<DK, NS>;
+  static size_t configured = 0;
+  if (smem > configured) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    configured = smem;
+  }
+  return launch_pdl(kern, dim3((max_q + QB - 1) / QB, a.H, n_seqs), dim3(384), smem, st, tk, tq, a);
+}
+// q fp16 [T_total][H][G * DK] (mixed, scaled); kc fp16 [n_pages][16][G * DK], whole pages of finite numbers; out bf16 [T_total][H * DK], or the same
+// in fp32 to out_f32.  max_q: the longest portion.
+B200_API int b200_mixed_prefill(const void* q, const void* kc, const float* slopes, const float* sinks, const int* page_table, int max_pages, int n_pages,
+                                const int* q_start, const int* q_len, const int* ctx_len, int n_seqs, int max_q, int T_total, int H, int G, int DK,
+                                int window, void* out, float* out_f32, int* status, cudaStream_t st) {
+  int ns, qt, r;
+  if (n_seqs < 1 || max_q < 1 || T_total < 1 || H < 1 || window < 0 || !q || !kc || !page_table || (!out && !out_f32) || G < 1 || H % G ||
+      !mixed_prefill_plan(G, DK, ns, qt, r))
+    return B200_ERR_BAD_ARG;
+  MixedPreArgs a = {};
+  a.q = (const __half*)q; a.slopes = slopes; a.sinks = sinks; a.page_table = page_table; a.q_start = q_start; a.q_len = q_len; a.ctx_len = ctx_len;
+  a.max_pages = max_pages; a.H = H; a.G = G; a.T_total = T_total; a.window = window; a.QT = qt; a.R = r; a.out = (__nv_bfloat16*)out; a.out_f32 = out_f32;
+  a.status = status;
+  CUtensorMap tk, tq;
+  int rc = make_tmap_rows8(&tk, kc, (uint64_t)n_pages * 16, (uint64_t)G * DK, DK / 64);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tq, q, 2, (uint64_t)T_total, (uint64_t)H * G * DK, (uint64_t)H * G * DK * 2, QB, 64, true);
+  if (rc) return rc;
+  if (DK == 64) return ns == 2 ? launch_mixed_prefill<64, 2>(tk, tq, a, n_seqs, max_q, st) : launch_mixed_prefill<64, 1>(tk, tq, a, n_seqs, max_q, st);
+  return ns == 2 ? launch_mixed_prefill<128, 2>(tk, tq, a, n_seqs, max_q, st) : launch_mixed_prefill<128, 1>(tk, tq, a, n_seqs, max_q, st);
 }

