@@ -1,6 +1,7 @@
-"""Prefill and decode throughput of the hybrid engine (Folirax, Pesorax) at a real model's layer sizes, beside the Llama engine at equal size.
+"""Prefill and decode throughput of the hybrid engine (Folirax, Pesorax, Kazolorn) at a real model's layer sizes, beside the closest other engine at equal size:
+the Llama engine, or, for a stack with experts, the mixture-of-experts engine.
 
-    python bench.py --workload hybrid [--model folirax-8b-shape | pesorax-8b-shape | ...] [--steps K] [--warmup W]
+    python bench.py --workload hybrid [--model folirax-8b-shape | pesorax-8b-shape | kazolorn-8b-shape | kazolorn-moe-shape | ...] [--steps K] [--warmup W]
 
 Both engines hold bf16 random weights of the same width, feed-forward, head layout, depth and vocabulary, run the same prompts
 and batches, and are timed with CUDA events: a 2048-token prompt, four of them in one call, and decode steps (replayed graphs
@@ -33,6 +34,11 @@ def like_llama(cfg):
     128, four to a key/value head)."""
     from openagents_b200.models.config import ModelConfig
     m = next(l.mixer for l in cfg.layers if l.mixer.kind == "attention")
+    moe = next((l for l in cfg.layers if l.moe), None)
+    if moe is not None:              # the same experts, heads and windows, a mixture in every layer
+        return ModelConfig(arch="gpt-oss", n_layers=len(cfg.layers), d_model=cfg.d_model, n_heads=m.heads, n_kv_heads=m.kv_heads, head_dim=m.dim, ffn=moe.ffn,
+                           vocab=cfg.vocab, context=8192, rope_theta=150000.0, rope_style="half", n_experts=moe.moe.experts, top_k=moe.moe.top,
+                           sliding_window=m.window, swa_every=1, attn_sinks=True, name="moe-" + cfg.name)
     heads, kv, dim = (cfg.d_model // 128, cfg.d_model // 512, 128) if cfg.arch == "pesorax" else (m.heads, m.kv_heads, m.dim)
     return ModelConfig(arch="llama", n_layers=len(cfg.layer_runs()), d_model=cfg.d_model, n_heads=heads, n_kv_heads=kv, head_dim=dim,
                        ffn=cfg.ffn, vocab=cfg.vocab, context=8192, rope_theta=500000.0, name="llama-" + cfg.name)
@@ -41,9 +47,9 @@ def like_llama(cfg):
 def time_engine(cfg, dev, steps: int, warmup: int) -> dict:
     from openagents_b200.models.qweight import RandomSource
     from openagents_b200.models.registry import build_engine
-    from openagents_b200.models.weights import PLAN_BF16
+    from openagents_b200.models.weights import PLAN_BF16, PLAN_MOE
     B = max(BATCHES)
-    eng = build_engine(RandomSource(cfg, PLAN_BF16, 0, dev), dev, B, PROMPT + 2 * (steps + warmup) * len(BATCHES) + 64, 4 * PROMPT)
+    eng = build_engine(RandomSource(cfg, PLAN_MOE if cfg.n_experts else PLAN_BF16, 0, dev), dev, B, PROMPT + 2 * (steps + warmup) * len(BATCHES) + 64, 4 * PROMPT)
     g = torch.Generator().manual_seed(1)
     prompts = torch.randint(0, cfg.vocab, (B, PROMPT), generator=g).tolist()
 
@@ -229,6 +235,120 @@ def time_pesorax_kernels(cfg, dev, reps: int = 12) -> list[dict]:
     return bench.rows
 
 
+def time_kazolorn_kernels(cfg, dev, reps: int = 12) -> list[dict]:
+    """Every kernel of a Kazolorn layer at 2048 prompt tokens and at decode steps, and its counterpart in the closest engine's layer.  Cached rows are read once; FLOPs
+    of the attention are the design's own (raw scores, mixture, output of the visible keys), whatever form the kernel computes them in."""
+    from openagents_b200.ops import cuda_ops as ops
+    bench = _Timer(dev, reps)
+    m = cfg.layers[0].mixer
+    H, G, D, win = m.heads, m.kv_heads, m.dim, m.window
+    dense, mix = next((l for l in cfg.layers if l.ffn and not l.moe), None), next((l for l in cfg.layers if l.moe), None)
+    d, T, B, ctx = cfg.d_model, PROMPT, 64, PROMPT
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    rnd = lambda *s: torch.randn(*s, device=dev)                       # noqa: E731
+    bf = lambda *s: torch.randn(*s, device=dev).bfloat16()             # noqa: E731
+    hf = lambda *s: torch.randn(*s, device=dev).half()                 # noqa: E731
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)     # noqa: E731
+    pages, slabs, ls = (ctx + 15) // 16, (len(cfg.layers) + 2) // 2, rnd(d)
+    for n in (T, B, 1):
+        xs, w, g, h1, h2 = rnd(slabs + 1, n, d), rnd(slabs), rnd(d), bf(n, d), bf(n, d)
+        bench(f"depth_norm of {slabs} [{n}]", lambda: ops.depth_norm(xs[:slabs], d, 1e-6, weights=w, out=xs[slabs], add=g, g1=g, g2=g, h1=h1, h2=h2), n * d * (4 * slabs + 8),
+              like=f"rmsnorm [{n}]")
+        x = rnd(n, d)
+        bench(f"rmsnorm [{n}]", lambda: ops.rmsnorm(x, g, 1e-6, hb=h1), n * d * 6)
+        del xs
+    # ---- attention
+    nq, nk = H * D, G * D
+    for n, seqs in ((T, 1), (B, B), (1, 1)):
+        prompt = n == T
+        row, bias, mixw, slopes, zero = rnd(n, nq + nk), rnd(nq + nk), rnd(H, H).bfloat16().float(), rnd(H).abs() * 0.01, torch.zeros(H, device=dev)
+        pos, slot = i32([ctx - 1] * n if not prompt else list(range(n))), i32(list(range(n)))
+        kc = hf(seqs * pages + 1, 1, 16, nk)
+        table, lens, o = i32(list(range(seqs * pages))).view(seqs, pages), i32([ctx] * seqs), bf(n, nq)
+        ld = (H + 2 * G) * D
+        row2, tabf, kl, vl = rnd(n, ld), ops.rope_table(ctx, D, 500000.0, dev), hf(seqs * pages + 1, G, 16, D), hf(seqs * pages + 1, G, 16, D)
+        l16, l32 = hf(n, nq), rnd(n, nq)
+        seen = min(ctx, win)
+        if prompt:
+            q16, z = hf(n, H * nk), i32([0])
+            bench(f"mixed_finish [{n}]", lambda: ops.mixed_finish(row, nq, bias, mixw, 0.1, slot, H, G, D, D, q16, kc), n * ((nq + nk) * 4 + H * nk * 2 + nk * 2), like=f"rope_kv [{n}]")
+            pairs = sum(min(t + 1, win) for t in range(T))
+            bench(f"mixed_prefill [{n}]", lambda: ops.mixed_prefill(q16, kc, slopes, table, z, lens, lens, 1, n, H, G, D, window=win, sinks=zero, out_bf16=o, status=st),
+                  n * (nq * 4 + nk * 2), 2.0 * pairs * H * (2 * D + H), like=f"attn_prefill_tc05 [{n}]")
+            bench(f"attn_prefill_tc05 [{n}]", lambda: ops.attn_prefill_tc05(l16, kl, vl, table, z, lens, lens, 1, n, H, G, window=0 if win >= T else win, out_bf16=o, status=st, dk=D, dv=D),
+                  n * (H + G) * D * 4, 4.0 * pairs * H * D)
+        else:
+            bench(f"qkv_finish keys only [{n}]", lambda: ops.qkv_finish(row, 0, nq, -1, pos, slot, None, 1.0, H, 1, D, D, D, D, 0, 1, False, 0.0, 0.1, 16, q32=l32, kc=kc, maps=G,
+                                                                        bias=bias), n * ((nq + nk) * 4 + nq * 4 + nk * 2), like=f"rope_kv [{n}]")
+            from openagents_b200.models.hybrid_engine import HybridEngine
+            e = HybridEngine.__new__(HybridEngine)
+            e.max_splits = 64
+            S = e._mixed_splits(n, min(pages, win // 16 + 2))
+            sc = rnd(ops.mixed_decode_scratch_floats(n, H, G, D, S))
+            bench(f"mixed_decode [{n} x {seen}] ({S} shares)", lambda: ops.mixed_decode(l32, kc, mixw, slopes, table, lens, n, H, G, D, window=win, S=S, sinks=zero, out_bf16=o,
+                                                                                     scratch=sc, status=st), n * (seen * nk * 2 + nq * 6),
+                  2.0 * n * seen * H * (2 * D + H), like=f"attn_decode [{n} x {seen}]")
+            e.attn_target_ctas = 0
+            S2 = e._attn_splits(n, G, min(pages, win // 16 + 2))
+            sc2, cnt2 = rnd(ops.attn_decode_scratch_floats(n, H, G, D, S2)), torch.zeros(n * H, dtype=torch.int32, device=dev)
+            bench(f"attn_decode [{n} x {seen}]", lambda: ops.attn_decode(l32, kl, vl, table, lens, n, H, G, D, window=0 if win >= ctx else win, S=S2, out_bf16=o, scratch=sc2, counters=cnt2,
+                                                                      status=st), n * (seen * G * D * 4 + nq * 6))
+        bench(f"rope_kv [{n}]", lambda: ops.rope_kv(row2, pos, slot, None if prompt else l32, l16 if prompt else None, kl, vl, H, G, D, 16, 500000.0, 0, 0.1, table=tabf),
+              n * (ld * 4 + nq * (2 if prompt else 4) + 2 * nk * 2))
+        del kc, kl, vl
+    # ---- products
+    for n in (T, B):
+        a, x = bf(n, d), rnd(n, d)
+        for nm, N, like in (("gemm queries and keys", nq + nk, True), ("gemm qkv", nq + 2 * nk, False)):
+            wt, o3 = bf(N, d), torch.zeros(n, N, device=dev)
+            bench(f"{nm} [{n}]", lambda: ops.gemm_bf16(a, wt, n, N, d, out_f32=o3, accumulate=n <= 64, status=st), N * d * 2 + n * (d * 2 + N * 4), 2.0 * n * N * d,
+                  like=f"gemm qkv [{n}]" if like else None)
+        wo, ao = bf(d, nq), bf(n, nq)
+        bench(f"gemm output, layer scale [{n}]", lambda: ops.gemm_bf16(ao, wo, n, d, nq, out_f32=x, accumulate=True, col_scale=ls, status=st), wo.numel() * 2 + n * (nq * 2 + d * 8),
+              2.0 * n * d * nq, like=f"gemm output, residual [{n}]")
+        bench(f"gemm output, residual [{n}]", lambda: ops.gemm_bf16(ao, wo, n, d, nq, out_f32=x, resid_f32=x, status=st), wo.numel() * 2 + n * (nq * 2 + d * 8), 2.0 * n * d * nq)
+        if dense:
+            F = dense.ffn
+            up, dn, gu, z, act, coef = bf(F, d), bf(d, F), bf(2 * F, d), rnd(n, F), bf(n, F), rnd(4)
+            bench(f"gemm up [{n}]", lambda: ops.gemm_bf16(a, up, n, F, d, out_f32=z, status=st), (F * d + n * d) * 2 + n * F * 4, 2.0 * n * F * d, like=f"gemm swiglu gate/up [{n}]")
+            bench(f"gemm swiglu gate/up [{n}]", lambda: ops.gemm_bf16(a, gu, n, 2 * F, d, out_bf16=act, ldc=F, act=ops.ACT_SWIGLU_PAIR, status=st), (2 * F * d + n * (d + F)) * 2,
+                  4.0 * n * F * d)
+            bench(f"poly_norm [{n}]", lambda: ops.poly_norm(z, F, coef, 1e-6, act), n * F * 6, like=f"rmsnorm [{n}]")
+            bench(f"gemm down, layer scale [{n}]", lambda: ops.gemm_bf16(act, dn, n, d, F, out_f32=x, accumulate=True, col_scale=ls, status=st), (F * d + n * F) * 2 + n * d * 8,
+                  2.0 * n * F * d, like=f"gemm down, residual [{n}]")
+            bench(f"gemm down, residual [{n}]", lambda: ops.gemm_bf16(act, dn, n, d, F, out_f32=x, resid_f32=x, status=st), (F * d + n * F) * 2 + n * d * 8, 2.0 * n * F * d)
+            del up, dn, gu, z, act
+    # ---- experts
+    if mix:
+        E, top, F = mix.moe.experts, mix.moe.top, mix.ffn
+        w13, w2, router = bf(E * 2 * F, d) * 0.02, bf(E * d, F) * 0.02, rnd(E, d) * 0.02
+        for n in (T, B):
+            cap = (n + 127) // 128 * 128
+            rx, mid, meta, rw = bf(E * cap, d), bf(E * cap, F), torch.zeros(E * cap, 2, dtype=torch.int32, device=dev), rnd(E * cap)
+            h, x, ids, w = bf(n, d), rnd(n, d), torch.zeros(n, top, dtype=torch.int32, device=dev), rnd(n, top)
+            cnt = torch.zeros(64, E, dtype=torch.int32, device=dev)
+            used = min(E, n * top)
+            for nm, score, like in (("route and dispatch, sigmoid", ops.SCORE_SIGMOID, "route and dispatch, softmax"), ("route and dispatch, softmax", ops.SCORE_SOFTMAX, None)):
+                cnt.zero_()
+                turn = iter(range(64))
+                bench(f"{nm} [{n}]", lambda: ops.moe_route_dispatch(h, None, router, None, top, E, cap, rx.data_ptr(), meta.data_ptr(), rw.data_ptr(), cnt[next(turn)].data_ptr(), None,
+                                                                    topk_ids=ids, topk_w=w, status=st, score=score), n * d * 2 * (1 + top) + E * d * 4, like=like and f"{like} [{n}]")
+            for nm, gw, like in (("experts gate/up, weight on the input", rw, "experts gate/up"), ("experts gate/up", None, None)):
+                bench(f"{nm} [{n}]", lambda: ops.moe_gemm(rx, w13, E, cap, 2 * F, d, cnt[0], 1, out_bf16=mid, ldc=F, gate_w=gw, status=st, live_rows=n * top),
+                      used * 2 * F * d * 2 + n * top * (d + F) * 2, 4.0 * n * top * F * d, like=like and f"{like} [{n}]")
+            for nm, gw, sc, like in (("experts down, layer scale", None, ls, "experts down"), ("experts down", rw, None, None)):
+                bench(f"{nm} [{n}]", lambda: ops.moe_gemm(mid, w2, E, cap, d, F, cnt[0], 2, ldc=d, meta=meta, gate_w=gw, sym_off=x.data_ptr(), col_scale=sc, status=st, live_rows=n * top),
+                      used * F * d * 2 + n * top * (F * 2 + d * 4), 2.0 * n * top * F * d, like=like and f"{like} [{n}]")
+        h, x, ids, w, mid = rnd(1, d), rnd(1, d), i32([list(range(top))]), rnd(1, top), rnd(1, top, F)
+        bench("expert_gate_up [1]", lambda: ops.expert_gate_up(h, w13, F, ids, w, mid), top * 2 * F * d * 2, like="matvec swiglu [1]")
+        bench("expert_down [1]", lambda: ops.expert_down(mid, w2, d, ids, x, scale=ls), top * F * d * 2, like="matvec down [1]")
+        F4 = top * F
+        gu, dn, act = bf(2 * F4, d), bf(d, F4), rnd(1, F4)
+        bench("matvec swiglu [1]", lambda: ops.matvec(ops.WT_BF16, gu, None, F4, d, 1, xf=h, epi=ops.EPI_SWIGLU_F32, y=act, ldy=F4), 2 * F4 * d * 2)
+        bench("matvec down [1]", lambda: ops.matvec(ops.WT_BF16, dn, None, d, F4, 1, xf=act, epi=ops.EPI_RESID, resid=x, y=x, ldy=d), F4 * d * 2)
+    return bench.rows
+
+
 def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
     """Every kernel of one hybrid layer pair at 2048 prompt tokens and at a 64-sequence decode step, and its Llama counterpart."""
     from openagents_b200.ops import cuda_ops as ops
@@ -315,6 +435,8 @@ def run(args) -> dict:
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
     cfg = PRESETS[args.model]
-    ours, llama = time_engine(cfg, dev, args.steps, max(3, args.warmup)), time_engine(like_llama(cfg), dev, args.steps, max(3, args.warmup))
+    llama_cfg = like_llama(cfg)
+    ours, llama = time_engine(cfg, dev, args.steps, max(3, args.warmup)), time_engine(llama_cfg, dev, args.steps, max(3, args.warmup))
     return {"workload": "hybrid", "model": cfg.name, "dtype": "bf16", "data": "synthetic", "prompt": PROMPT, "peaks": peaks()[2], "hybrid": ours,
-            "llama_equal_size": llama, "kernels": (time_pesorax_kernels if cfg.arch == "pesorax" else time_kernels)(cfg, dev)}
+            "moe_equal_size" if llama_cfg.n_experts else "llama_equal_size": llama,
+            "kernels": {"pesorax": time_pesorax_kernels, "kazolorn": time_kazolorn_kernels}.get(cfg.arch, time_kernels)(cfg, dev)}

@@ -156,9 +156,8 @@ struct MixedDecArgs {
   int max_pages, H, G, rp, window, S, nslot;
   float* out_f32;          // [B][H * DK]
   __nv_bfloat16* out_bf16;
-  float* part_acc;         // [B][parts][S][8 NTV][DK]
-  float* part_ml;          // [B][parts][S][8 NTV][2]
-  int* counters;           // [B][parts], zero before first use, left zero
+  float* part_acc;         // [B][S][8 NT][DK]
+  float* part_ml;          // [B][S][8 NT][2]
   int* status;
 };
 __device__ __forceinline__ float2 split_bf16(float x, float y, uint32_t& packed) {      // the pair's bf16 values, and what they leave
@@ -174,7 +173,6 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
   constexpr int QLD = DK + 8, KB = DK / 64;
   extern __shared__ uint8_t dyn_raw[];
   __shared__ float s_ml[8][NTV * 8][2];
-  __shared__ int s_last;
   __shared__ int s_abort;
   uint8_t* ring = (uint8_t*)(((uintptr_t)dyn_raw + 1023) & ~(uintptr_t)1023);
   const int W = a.G * DK, page_bytes = 32 * W, NB = W / 64, nw = blockDim.x >> 5;
@@ -251,28 +249,33 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
     ok = __all_sync(0xffffffffu, ok);
     if (!ok) break;
     const uint32_t page = smem_u32(ring) + (uint32_t)(s * page_bytes);
-    // 16 bytes of key row `row` of the page: piece `ch` of key head c
-    auto piece = [&](int row, int c, int ch) {
-      return page + (uint32_t)((row >> 3) * NB + c * KB + (ch >> 3)) * 1024u + (uint32_t)(row & 7) * 128u + (uint32_t)(((ch & 7) ^ (row & 7)) << 4);
-    };
+    // key row `row` of the page at key head c, and 16-byte piece `ch` of it (r8: the row's place among its eight)
+    auto row_at = [&](int row, int c) { return page + (uint32_t)((row >> 3) * NB + c * KB) * 1024u + (uint32_t)r8 * 128u; };
+    auto piece_at = [&](int ch) { return (uint32_t)(ch >> 3) * 1024u + (uint32_t)(((ch & 7) ^ r8) << 4); };
     float sc[NT][4];
 #pragma unroll
     for (int j = 0; j < NT; j++) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
-    for (int u = 0; u < nsub; u++)
 #pragma unroll 1
+    for (int u = 0; u < nsub; u++) {
+      uint32_t ka[NT], qa[NT];                            // tile j: this lane's key row of the u-th head the tile meets, its query row
+#pragma unroll
+      for (int j = 0; j < NT; j++) {
+        const int c = rp < 8 ? j * nsub + u : j * 8 / rp;
+        ka[j] = row_at(r8 + (mi & 1) * 8, min(c, a.G - 1));       // (a head that is not there meets zero queries)
+        qa[j] = smem_u32(sQ + ((rp >= 8 || r8 / rp == u) ? j * 8 + r8 : 8 * NT) * QLD + mi * 8);
+      }
+#pragma unroll
       for (int kk = 0; kk < DK / 32; kk++)
 #pragma unroll
         for (int j = 0; j < NT; j++) {
-          const int c = rp < 8 ? j * nsub + u : j * 8 / rp;
-          if (c >= a.G) continue;
           uint32_t k0[4], k1[4], q[4];
-          const int row = r8 + (mi & 1) * 8, slot = j * 8 + r8;
-          ldsm_x4(piece(row, c, kk * 4 + (mi >> 1)), k0[0], k0[1], k0[2], k0[3]);
-          ldsm_x4(piece(row, c, kk * 4 + 2 + (mi >> 1)), k1[0], k1[1], k1[2], k1[3]);
-          ldsm_x4(smem_u32(sQ + (slot / rp == c ? slot : 8 * NT) * QLD + kk * 32 + mi * 8), q[0], q[1], q[2], q[3]);
+          ldsm_x4(ka[j] + piece_at(kk * 4 + (mi >> 1)), k0[0], k0[1], k0[2], k0[3]);
+          ldsm_x4(ka[j] + piece_at(kk * 4 + 2 + (mi >> 1)), k1[0], k1[1], k1[2], k1[3]);
+          ldsm_x4(qa[j] + kk * 64, q[0], q[1], q[2], q[3]);
           mma16816(sc[j], k0, q[0], q[1]);
           mma16816(sc[j], k1, q[2], q[3]);
         }
+    }
     float d[NTV][4];
 #pragma unroll
     for (int nt = 0; nt < NTV; nt++) d[nt][0] = d[nt][1] = d[nt][2] = d[nt][3] = 0.f;
@@ -340,29 +343,29 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
       }
       const uint32_t w[2] = {transpose_8x8(pack_h2(p[0], p[1])), transpose_8x8(pack_h2(p[2], p[3]))};      // keys 0..7, 8..15 of head g4
       const int tile = part * NTV + nt;
-      if (tile * 8 >= live) continue;
       if (rp >= 8) {
-        const int c = tile * 8 / rp;
+        const uint32_t at = row_at(r8 + (mi >> 1) * 8, min(tile * 8 / rp, a.G - 1));
 #pragma unroll
         for (int m = 0; m < DK / 16; m++) {
           uint32_t k[4];
-          ldsm_x4_t(piece(r8 + (mi >> 1) * 8, c, m * 2 + (mi & 1)), k[0], k[1], k[2], k[3]);
+          ldsm_x4_t(at + piece_at(m * 2 + (mi & 1)), k[0], k[1], k[2], k[3]);
           mma16816(o[nt][m], k, w[0], w[1]);
         }
       } else {
 #pragma unroll 1
-        for (int pr = 0; pr < max(1, nsub >> 1); pr++) {
-          const int c0 = tile * nsub + 2 * pr, c1 = min(c0 + 1, a.G - 1);
-          if (c0 >= a.G) break;
-          const bool own0 = g4 / rp == 2 * pr, own1 = g4 / rp == 2 * pr + 1;
+        for (int pr = 0; pr < nsub >> 1; pr++) {
+          const int c = min(tile * nsub + 2 * pr + (mi >> 1), a.G - 1), sub = g4 / rp - 2 * pr;
+          const uint32_t at = row_at(r8, c);
 #pragma unroll
-          for (int kg = 0; kg < 2; kg++)
+          for (int kg = 0; kg < 2; kg++) {
+            const uint32_t b0 = sub == 0 ? w[kg] : 0u, b1 = sub == 1 ? w[kg] : 0u;
 #pragma unroll
             for (int m = 0; m < DK / 16; m++) {
               uint32_t k[4];
-              ldsm_x4_t(piece(r8 + kg * 8, mi < 2 ? c0 : c1, m * 2 + (mi & 1)), k[0], k[1], k[2], k[3]);
-              mma16816(o[nt][m], k, own0 ? w[kg] : 0u, own1 ? w[kg] : 0u);
+              ldsm_x4_t(at + (uint32_t)(kg * NB) * 1024u + piece_at(m * 2 + (mi & 1)), k[0], k[1], k[2], k[3]);
+              mma16816(o[nt][m], k, b0, b1);
             }
+          }
         }
       }
     }
@@ -393,8 +396,8 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
       }
     }
   __syncthreads();
-  const int parts = gridDim.y, n_out = NTV * 8 * DK;
-  const size_t row = ((size_t)b * parts + part) * a.S;
+  const int n_slots = gridDim.y * NTV * 8, n_out = NTV * 8 * DK;
+  const size_t row = ((size_t)b * a.S + split) * n_slots + part * NTV * 8;
   auto finish = [&](int slot, int e, float M, float L, float A) {
     const int h = head_of(part * NTV * 8 + slot);
     if (h < 0) return;
@@ -420,36 +423,52 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
     if (a.S == 1) {
       finish(slot, e, M, L, A);
     } else {
-      a.part_acc[(row + split) * n_out + x] = A;
+      a.part_acc[(row + slot) * DK + e] = A;
       if (e == 0) {
-        a.part_ml[((row + split) * NTV * 8 + slot) * 2] = M;
-        a.part_ml[((row + split) * NTV * 8 + slot) * 2 + 1] = L;
+        a.part_ml[(row + slot) * 2] = M;
+        a.part_ml[(row + slot) * 2 + 1] = L;
       }
     }
   }
-  if (a.S == 1) return;
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) {                                        // the CTA that comes last merges the shares
-    int* cnt = a.counters + (size_t)b * parts + part;
-    s_last = atomicAdd(cnt, 1) == a.S - 1;
-    if (s_last) *cnt = 0;
+}
+// The shares of one (sequence, head): a thread per output column.
+template <int DK>
+__global__ void __launch_bounds__(DK) mixed_merge_kernel(const float* __restrict__ acc, const float* __restrict__ ml, const float* __restrict__ sinks,
+                                                         int H, int rep, int rp, int n_slots, int S, float* __restrict__ out_f32,
+                                                         __nv_bfloat16* __restrict__ out_bf16) {
+  pdl_trigger();
+  pdl_wait();
+  const int h = blockIdx.x, b = blockIdx.y, e = threadIdx.x, slot = h / rep * rp + h % rep, lane = e & 31;
+  const size_t row = (size_t)b * S;
+  // lane s holds share s (up to 64 shares: two each)
+  float m[2], l[2], M = sinks ? sinks[h] * kLog2e : -INFINITY;
+#pragma unroll
+  for (int k = 0; k < 2; k++) {
+    const int s = lane + 32 * k;
+    m[k] = s < S ? ml[((row + s) * n_slots + slot) * 2] : -INFINITY;
+    l[k] = s < S ? ml[((row + s) * n_slots + slot) * 2 + 1] : 0.f;
   }
-  __syncthreads();
-  if (!s_last) return;
-  __threadfence();
-  for (int x = tid; x < n_out; x += blockDim.x) {
-    const int slot = x / DK, e = x % DK;
-    float M = -INFINITY, L = 0.f, A = 0.f;
-    for (int s = 0; s < a.S; s++) M = fmaxf(M, __ldcg(a.part_ml + ((row + s) * NTV * 8 + slot) * 2));
-    for (int s = 0; s < a.S; s++) {
-      const float* ml = a.part_ml + ((row + s) * NTV * 8 + slot) * 2;
-      const float m = __ldcg(ml), c = m == -INFINITY ? 0.f : ex2_approx(m - M);
-      L += __ldcg(ml + 1) * c;
-      A += __ldcg(a.part_acc + (row + s) * n_out + x) * c;
-    }
-    finish(slot, e, M, L, A);
+  M = fmaxf(M, warp_max(fmaxf(m[0], m[1])));
+  float c[2], L = 0.f;
+#pragma unroll
+  for (int k = 0; k < 2; k++) {
+    c[k] = m[k] == -INFINITY ? 0.f : ex2_approx(m[k] - M);
+    L += l[k] * c[k];
   }
+  L = warp_sum(L);
+  if (sinks) L += ex2_approx(sinks[h] * kLog2e - M);
+  float A = 0.f;
+  for (int s0 = 0; s0 < S; s0 += 8) {
+    float v[8];
+#pragma unroll
+    for (int i = 0; i < 8; i++) v[i] = s0 + i < S ? acc[((row + s0 + i) * n_slots + slot) * DK + e] : 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; i++) A = fmaf(v[i], __shfl_sync(0xffffffffu, s0 < 32 ? c[0] : c[1], (s0 + i) & 31), A);
+  }
+  const float v = L > 0.f ? A / L : 0.f;
+  const size_t at = ((size_t)b * H + h) * DK + e;
+  if (out_f32) out_f32[at] = v;
+  if (out_bf16) out_bf16[at] = __float2bfloat16(v);
 }
 
 // Padded group size, tiles of eight padded heads (even), and tiles a CTA keeps the outputs of; false: sizes the kernel does not take.
@@ -493,7 +512,7 @@ static int launch_mixed_decode(MixedDecArgs a, const void* kc, int n_pages, int 
     if (!nw) return B200_ERR_BAD_ARG;
   }
   a.part_acc = scratch;
-  a.part_ml = scratch ? scratch + (size_t)B * parts * a.S * NTV * 8 * DK : nullptr;
+  a.part_ml = scratch ? scratch + (size_t)B * a.S * NT * 8 * DK : nullptr;
   const size_t ring = (size_t)a.nslot * page > (size_t)nw * kOut ? (size_t)a.nslot * page : (size_t)nw * kOut, smem = fixed + ring;
   auto kern = mixed_decode_kernel<DK, NT, NTV>;
   static size_t configured = 0;
@@ -505,20 +524,23 @@ static int launch_mixed_decode(MixedDecArgs a, const void* kc, int n_pages, int 
   CUtensorMap tm;
   const int rc = make_tmap_rows8(&tm, kc, (uint64_t)n_pages * 16, W, W / 64);
   if (rc) return rc;
-  return launch_pdl(kern, dim3(a.S, parts, B), dim3(32 * nw), smem, st, tm, a);
+  const int err = launch_pdl(kern, dim3(a.S, parts, B), dim3(32 * nw), smem, st, tm, a);
+  if (err || a.S == 1) return err;
+  return launch_pdl(mixed_merge_kernel<DK>, dim3(a.H, B), dim3(DK), 0, st, (const float*)a.part_acc, (const float*)a.part_ml, a.sinks, a.H, a.H / a.G, a.rp, NT * 8,
+                    a.S, a.out_f32, a.out_bf16);
 }
 // q fp32 [B][H][DK], scaled; mix fp32 [H][H] (bf16 values); kc fp16 [n_pages][16][G * DK]; sizes as b200_mixed_decode_ok has them.  S: shares of the
-// keys (scratch and counters [2 B], zero before first use, where there are several).
+// keys, at most 64 (scratch where there are several).
 B200_API int b200_mixed_decode(const float* q, const void* kc, const float* mix, const float* slopes, const float* sinks, const int* page_table,
                                int max_pages, int n_pages, const int* seq_lens, int B, int H, int G, int DK, int window, int S, float* out_f32,
-                               void* out_bf16, float* scratch, int* counters, int* status, cudaStream_t st) {
+                               void* out_bf16, float* scratch, int* status, cudaStream_t st) {
   MixedDecArgs a = {};
   int nt, ntv;
-  if (B < 1 || S < 1 || window < 0 || max_pages < 1 || !q || !kc || !mix || (!out_f32 && !out_bf16) || (S > 1 && (!scratch || !counters)) ||
+  if (B < 1 || S < 1 || S > 64 || window < 0 || max_pages < 1 || !q || !kc || !mix || (!out_f32 && !out_bf16) || (S > 1 && !scratch) ||
       !mixed_decode_plan(H, G, DK, a.rp, nt, ntv) || ((uintptr_t)q & 7))
     return B200_ERR_BAD_ARG;
   a.q = q; a.mix = mix; a.slopes = slopes; a.sinks = sinks; a.page_table = page_table; a.seq_lens = seq_lens; a.max_pages = max_pages; a.H = H; a.G = G;
-  a.window = window; a.S = S; a.out_f32 = out_f32; a.out_bf16 = (__nv_bfloat16*)out_bf16; a.counters = counters; a.status = status;
+  a.window = window; a.S = S; a.out_f32 = out_f32; a.out_bf16 = (__nv_bfloat16*)out_bf16; a.status = status;
   if (DK == 64) {
     if (nt == 2) return launch_mixed_decode<64, 2, 2>(a, kc, n_pages, B, scratch, st);
     if (nt == 4) return launch_mixed_decode<64, 4, 4>(a, kc, n_pages, B, scratch, st);
@@ -634,16 +656,26 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
           for (int c = 0; c < CB; c++)
             tma_load_2d(smem_u32(sQ + (size_t)(u - a.QT) * SLICE + c * (QB * 128)), &tmQ, bar, h * W + (own + 1 + u) % G * DK + c * 64, qs + q0);
       }
-      for (int e = 0; e < nb * G; e++) {
-        const int j = e / G, sl = (own + 1 + e - j * G) % G, s = e % R;
-        if ((s & 1) != (warp == 0 ? 0 : 1)) continue;
-        if (!mbar_wait(smem_u32(k_empty + s), (uint32_t)((e / R) & 1) ^ 1, abort_flag)) break;
-        const uint32_t bar = smem_u32(k_full + s), dst = smem_u32(sK + (size_t)s * SLICE);
-        mbar_expect_tx(bar, SLICE);
+      bool ok = true;
+      int s = 0, ph = 1;                           // slot and parity of entry e
+      for (int j = 0; j < nb && ok; j++) {
+        int page[KEYS / 16];                       // read together: one at a time, their latency would bound the copies
 #pragma unroll
         for (int p = 0; p < KEYS / 16; p++) {
           const int pi = (jb0 + j) * (KEYS / 16) + p;
-          tma_load_4d(dst + p * 2 * GROUP, &tmK, bar, 0, 0, sl * CB, (pi * 16 < ctx ? pt[pi] : 0) * 2);      // pages past the context are masked anyway
+          page[p] = pi * 16 < ctx ? pt[pi] * 2 : 0;                 // pages past the context are masked anyway
+        }
+        int sl = own;
+        for (int u = 0; u < G; u++) {
+          sl = sl + 1 == G ? 0 : sl + 1;
+          if ((s & 1) == (warp == 0 ? 0 : 1)) {
+            if (!mbar_wait(smem_u32(k_empty + s), ph, abort_flag)) { ok = false; break; }
+            const uint32_t bar = smem_u32(k_full + s), dst = smem_u32(sK + (size_t)s * SLICE);
+            mbar_expect_tx(bar, SLICE);
+#pragma unroll
+            for (int p = 0; p < KEYS / 16; p++) tma_load_4d(dst + p * 2 * GROUP, &tmK, bar, 0, 0, sl * CB, page[p]);
+          }
+          if (++s == R) { s = 0; ph ^= 1; }
         }
       }
     }

@@ -415,7 +415,6 @@ class HybridEngine(PagedEngine):
         # rows x shares stays below MIXED_CTAS wherever there is more than one share
         self.mixed_scratch = ws("mixed_scratch", (max((ops.mixed_decode_scratch_floats(max(self.max_batch, MIXED_CTAS), m.heads, m.kv_heads, b.DK, 1)
                                                        for b, m, _ in attn if b.dec), default=0),), f32)
-        self.mixed_counters = ws("mixed_counters", (2 * self.max_batch if any(b.dec for b, _, _ in attn) else 0,), torch.int32, zero=True)
         self.attn_scratch = ws("attn_scratch", (max((ops.attn_decode_scratch_floats(self.max_batch, hq, m.kv_heads, dv, self.max_splits)
                                                      for m, dv, hq in tc), default=4),), f32)
         self.attn_counters = ws("attn_counters", (self.max_batch * max((hq for _, _, hq in tc), default=1),), torch.int32, zero=True)
@@ -550,10 +549,10 @@ class HybridEngine(PagedEngine):
             q = self.q32[: T * H * b.DK].view(T, -1)
             ops.qkv_finish(proj, 0, k_off, -1, self.pos, self.slot, None, 1.0, H, 1, m.dim, m.vdim, b.DK, b.DV, 0, 1, False, 0.0, m.scale, PAGE, q32=q, kc=kc,
                            maps=G, bias=b.bias)
-            ops.mixed_decode(q, kc, b.mix, b.slopes, self.page_table, self.seq_lens, T, H, G, b.DK, window=m.window,
-                             S=self._mixed_splits(T, min(pages, m.window // PAGE + 2) if m.window else pages), sinks=b.silent, out_f32=o32, out_bf16=o16,
-                             scratch=self.mixed_scratch, counters=self.mixed_counters, status=self.status)
-            return 2
+            S = self._mixed_splits(T, min(pages, m.window // PAGE + 2) if m.window else pages)
+            ops.mixed_decode(q, kc, b.mix, b.slopes, self.page_table, self.seq_lens, T, H, G, b.DK, window=m.window, S=S, sinks=b.silent, out_f32=o32, out_bf16=o16,
+                             scratch=self.mixed_scratch, status=self.status)
+            return 2 + (S > 1)
         tc = b.tc and not decode
         q = (self.q16 if tc else self.q32)[: T * H * G * b.DK].view(T, -1)
         ops.mixed_finish(proj, k_off, b.bias, b.mix, m.scale, self.slot, H, G, m.dim, b.DK, q, kc)

@@ -54,7 +54,7 @@ _SIGS = {
     "b200_depth_norm": [_P, c_size_t, _P, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_float, _P, _P, _P, _P, _P, c_long, _P],
     "b200_poly_norm": [_P, c_int, c_int, c_int, _P, c_float, _P, _P, c_int, _P],
     "b200_mixed_finish": [_P] + [c_int] * 3 + [_P, _P, c_float, _P] + [c_int] * 5 + [_P, _P, _P, c_int, _P],
-    "b200_mixed_decode": [_P] * 6 + [c_int, c_int, _P] + [c_int] * 6 + [_P] * 6,
+    "b200_mixed_decode": [_P] * 6 + [c_int, c_int, _P] + [c_int] * 6 + [_P] * 5,
     "b200_mixed_decode_ok": [c_int] * 3,
     "b200_mixed_prefill": [_P] * 5 + [c_int, c_int, _P, _P, _P] + [c_int] * 7 + [_P] * 4,
     "b200_mixed_prefill_ok": [c_int] * 2,
@@ -489,12 +489,11 @@ def mixed_decode_scratch_floats(B, H, G, DK, S):
     return lib().b200_mixed_decode_scratch_floats(B, H, G, DK, S)
 
 
-def mixed_decode(q, kc, mix, slopes, page_table, seq_lens, B, H, G, DK, window=0, S=1, sinks=None, out_f32=None, out_bf16=None, scratch=None, counters=None,
-                 status=None):
+def mixed_decode(q, kc, mix, slopes, page_table, seq_lens, B, H, G, DK, window=0, S=1, sinks=None, out_f32=None, out_bf16=None, scratch=None, status=None):
     """One query token per sequence, heads mixed on the scores (see ``mixed_attn.cu``): ``q`` fp32 [B, H, DK], scaled and not mixed; ``kc`` fp16 [pages, 1, 16,
-    G * DK], keys and values; ``slopes`` [H]: of the mixed scores.  ``S``: shares of the keys (``counters``: int32 [2 B], zero)."""
+    G * DK], keys and values; ``slopes`` [H]: of the mixed scores.  ``S``: shares of the keys, at most 64."""
     _check(lib().b200_mixed_decode(_p(q), _p(kc), _p(mix), _p(slopes), _p(sinks), _p(page_table), page_table.shape[1], kc.shape[0], _p(seq_lens), B, H, G, DK,
-                                   window, S, _p(out_f32), _p(out_bf16), _p(scratch), _p(counters), _p(status), _st()), "mixed_decode")
+                                   window, S, _p(out_f32), _p(out_bf16), _p(scratch), _p(status), _st()), "mixed_decode")
 
 
 def mixed_prefill(q16, kc, slopes, page_table, q_start, q_len, ctx_len, n_seqs, max_q, H, G, DK, window=0, sinks=None, out_bf16=None, out_f32=None, status=None):

@@ -219,13 +219,12 @@ def mixed(kernel, qs, ks, mix, scale, window, bias=None):
     out = torch.full((T, H * DK), 9.0, device=DEV)
     row, slot = row[last].contiguous(), slot[last].contiguous()
     if kernel == "decode":
-        for S in (1, 3):
+        for S in (1, 3, 37):
             q32, before = torch.full((T, H * DK), 7.0, device=DEV), kc.clone()
             ops.qkv_finish(row, 0, nq, -1, slot, slot, None, 1.0, H, 1, dim, dim, DK, DK, 0, 1, False, 0.0, scale, 16, q32=q32, kc=kc, maps=G, bias=bias.to(DEV))
             assert torch.equal(kc, before)               # the very rows the other finish writes
             ops.mixed_decode(q32, kc, mix.to(DEV), slopes, tab, ctx, B, H, G, DK, S=S, out_f32=out, status=st, window=window, sinks=args["sinks"],
-                             scratch=torch.full((ops.mixed_decode_scratch_floats(B, H, G, DK, S),), float("nan"), device=DEV),
-                             counters=torch.zeros(2 * B, dtype=torch.int32, device=DEV))
+                             scratch=torch.full((ops.mixed_decode_scratch_floats(B, H, G, DK, S),), float("nan"), device=DEV))
             assert S == 1 or (out.cpu() - first).abs().max() <= 2e-3 * first.abs().max()
             first = out.clone().cpu()
     elif kernel == "tc05":
