@@ -27,14 +27,6 @@ struct AttnPreArgs {
   float* lse;               // [T_total][Hq] natural-log sum-exp (training backward), or null
 };
 
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src));
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() {
-  asm volatile("cp.async.wait_group %0;" ::"n"(N));
-}
 template <int HD>
 __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnPreArgs a) {
   constexpr int ROW_B = HD * 2;          // bytes per row

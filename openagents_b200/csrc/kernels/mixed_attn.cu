@@ -553,12 +553,13 @@ B200_API int b200_mixed_decode(const float* q, const void* kc, const float* mix,
 
 // ------------------------------------------------------------------ prompts: wide queries on the 5th-generation tensor cores
 
-// One CTA = 128 query rows of one head against blocks of 128 keys, in the manner of attn_prefill_tc05.cu: two TMA warps, one warp that issues the
-// score products, one for the output products, eight softmax warps (two to a tensor-memory quarter, half of a block's keys and of the output columns
-// each).  What differs:
-//   - a score is a product over G slices (a key head's DK columns each); slices are the entries of the ring, [16 groups][DK / 64][8 rows][128
-//     bytes] = 128 keys, one TMA copy per page.  The head's own slice comes last in a block: it is the value operand too, and its entry is given back
-//     by the output product instead of the score product.
+// One CTA = 128 query rows of one head against blocks of 128 keys, in the manner of attn_prefill_tc05.cu: two warps that copy keys, one warp that issues
+// the score products, one for the output products, eight softmax warps (two to a tensor-memory quarter, half of a block's keys and of the output
+// columns each).  What differs:
+//   - a score is a product over G slices (a key head's DK columns each); slices of 128 keys are the entries of the ring.  The head's own slice comes
+//     last in a block: it is the value operand too, and its entry is given back by the output product instead of the score product.
+//   - a slice is gathered from eight pages.  16-byte asynchronous copies by 64 threads do that in some 500 cycles; TMA copies of a page's part each
+//     (4 KB) took 1600.
 //   - the wide query row lies in tensor memory as far as that reaches (QT slices), the rest in shared memory, both read as the A operand.
 //   - where the slices leave no room for two score accumulators (NS = 1), a block's score product waits for the output product before it.
 //   - slopes: one multiply-add per score, the block's part of the distance joins the exponent's offset.
@@ -568,6 +569,7 @@ constexpr float kRescale = 8.f;                   // log2 units
 
 struct MixedPreArgs {
   const __half* q;         // [T_total][H][G * DK], mixed and scaled
+  const __half* kc;        // [pages][16][G * DK]
   const float* slopes;     // [H] or null
   const float* sinks;      // [H] or null
   const int* page_table;
@@ -581,9 +583,8 @@ struct MixedPreArgs {
 };
 
 template <int DK, int NS>
-__global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmQ,
-                                                               const MixedPreArgs a) {
-  constexpr int CB = DK / 64, SLICE = KEYS * DK * 2, GROUP = CB * 1024;        // GROUP: bytes of eight key rows of a slice
+__global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const MixedPreArgs a) {
+  constexpr int CB = DK / 64, SLICE = KEYS * DK * 2, BOX = KEYS * 128;        // BOX: 64 columns of a slice, [128 rows][128 bytes]
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   const int QS = a.G - a.QT, R = a.R;
@@ -597,19 +598,23 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
   uint64_t* p_full = bars + 6;                            // [2]
   uint64_t* pv_done = bars + 8;                           // [2]
   uint64_t* x_full = bars + 10;                           // [4 quarters][2]
-  uint32_t* tmem_holder = (uint32_t*)(bars + 18);
+  uint64_t* qt_full = bars + 18;                          // [1] queries on their way to tensor memory have landed in the ring
+  uint64_t* qt_empty = bars + 19;                         // [1] and have been read from it
+  uint32_t* tmem_holder = (uint32_t*)(bars + 20);
   volatile int* abort_flag = (volatile int*)(tmem_holder + 1);
-  uint64_t* k_full = bars + 20;                           // [R]
+  uint64_t* k_full = bars + 22;                           // [R]
   uint64_t* k_empty = k_full + R;                         // [R]
-  float* xch = (float*)(bars + 20 + 2 * R);               // [NS][2 (half)][128 rows]
+  float* xch = (float*)(bars + 22 + 2 * R);               // [NS][2 (half)][128 rows]
 
   const int seq = blockIdx.z, h = blockIdx.y, qb = gridDim.x - 1 - blockIdx.x;   // longest (latest) query blocks first
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    mbar_init(smem_u32(q_full), 4);
+    mbar_init(smem_u32(q_full), 8);
     mbar_init(smem_u32(qs_full), 1);
+    mbar_init(smem_u32(qt_full), 1);
+    mbar_init(smem_u32(qt_empty), 8);
     for (int s = 0; s < R; s++) {
-      mbar_init(smem_u32(k_full + s), 1);
+      mbar_init(smem_u32(k_full + s), 64);
       mbar_init(smem_u32(k_empty + s), 1);
     }
     for (int s = 0; s < 2; s++) {
@@ -621,7 +626,6 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
     for (int s = 0; s < 8; s++) mbar_init(smem_u32(x_full + s), 2);
     *abort_flag = 0;
     fence_barrier_init();
-    tma_prefetch_desc(&tmK);
     tma_prefetch_desc(&tmQ);
   }
   if (warp == 1) {
@@ -645,86 +649,117 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
   const uint32_t S_T = tmem_base, O_T = tmem_base + NS * KEYS, Q_T = O_T + DK;
 
   if (warp == 0 || warp == 10) {
-    // entries e = j * G + u in order (block j, u-th slice of it).  Slots are shared out, not entries: a slot's uses must be waited for one after the other by
-    // one thread (a parity tells neighbouring phases apart, no more), and entries are not given back in order (the own slices come later).
-    if (lane == 0 && nb > 0) {
+    // Entries e = j * G + u in order (block j, u-th slice of it), all by both warps: thread x copies 16-byte piece x % 8 of every eighth row.  The
+    // barrier counts the threads whose copies have landed; the fence between those writes and the tensor cores' reads is the issuing warps'.
+    if (nb > 0) {
       const int* pt = a.page_table + (size_t)seq * a.max_pages;
-      if (warp == 0 && QS > 0) {
-        const uint32_t bar = smem_u32(qs_full);
-        mbar_expect_tx(bar, QS * SLICE);
-        for (int u = a.QT; u < G; u++)
-          for (int c = 0; c < CB; c++)
-            tma_load_2d(smem_u32(sQ + (size_t)(u - a.QT) * SLICE + c * (QB * 128)), &tmQ, bar, h * W + (own + 1 + u) % G * DK + c * 64, qs + q0);
-      }
       bool ok = true;
-      int s = 0, ph = 1;                           // slot and parity of entry e
+      // the queries: QT slices through the ring to tensor memory, R at a time, the others to where they stay
+      if (warp == 0 && lane == 0) {
+        auto fetch = [&](uint8_t* to, int u, uint32_t bar) {
+          for (int c = 0; c < CB; c++) tma_load_2d(smem_u32(to + c * BOX), &tmQ, bar, h * W + (own + 1 + u) % G * DK + c * 64, qs + q0);
+        };
+        for (int u0 = 0; u0 < a.QT && ok; u0 += R) {
+          const int n = min(R, a.QT - u0);
+          if (u0 > 0) ok = mbar_wait(smem_u32(qt_empty), (uint32_t)(u0 / R - 1) & 1, abort_flag);
+          if (!ok) break;
+          mbar_expect_tx(smem_u32(qt_full), n * SLICE);
+          for (int i = 0; i < n; i++) fetch(sK + (size_t)i * SLICE, u0 + i, smem_u32(qt_full));
+          if (u0 == 0 && QS > 0) {
+            mbar_expect_tx(smem_u32(qs_full), QS * SLICE);
+            for (int u = a.QT; u < G; u++) fetch(sQ + (size_t)(u - a.QT) * SLICE, u, smem_u32(qs_full));
+          }
+        }
+      }
+      ok = __all_sync(0xffffffffu, ok) && mbar_wait(smem_u32(q_full), 0, abort_flag);      // the ring is free for keys
+      ok = __all_sync(0xffffffffu, ok);
+      const int x = (warp == 0 ? 0 : 32) + lane, r0 = x >> 3, c0 = x & 7;
+      const uint32_t dst0 = smem_u32(sK) + (uint32_t)(r0 * 128 + ((c0 ^ r0) << 4));
+      const __half* src0 = a.kc + (size_t)r0 * W + c0 * 8;
+      int s = 0, ph = 1;                           // slot of the entry and the parity of its being free
       for (int j = 0; j < nb && ok; j++) {
-        int page[KEYS / 16];                       // read together: one at a time, their latency would bound the copies
+        const __half* page[KEYS / 16];             // read together: one at a time, their latency would bound the copies
 #pragma unroll
         for (int p = 0; p < KEYS / 16; p++) {
           const int pi = (jb0 + j) * (KEYS / 16) + p;
-          page[p] = pi * 16 < ctx ? pt[pi] * 2 : 0;                 // pages past the context are masked anyway
+          page[p] = src0 + (size_t)(pi * 16 < ctx ? pt[pi] : 0) * 16 * W;         // pages past the context are masked anyway
         }
         int sl = own;
         for (int u = 0; u < G; u++) {
           sl = sl + 1 == G ? 0 : sl + 1;
-          if ((s & 1) == (warp == 0 ? 0 : 1)) {
-            if (!mbar_wait(smem_u32(k_empty + s), ph, abort_flag)) { ok = false; break; }
-            const uint32_t bar = smem_u32(k_full + s), dst = smem_u32(sK + (size_t)s * SLICE);
-            mbar_expect_tx(bar, SLICE);
+          ok = mbar_wait(smem_u32(k_empty + s), ph, abort_flag);
+          ok = __all_sync(0xffffffffu, ok);
+          if (!ok) break;
+          const uint32_t dst = dst0 + (uint32_t)(s * SLICE);
 #pragma unroll
-            for (int p = 0; p < KEYS / 16; p++) tma_load_4d(dst + p * 2 * GROUP, &tmK, bar, 0, 0, sl * CB, page[p]);
-          }
+          for (int p = 0; p < KEYS / 16; p++)
+#pragma unroll
+            for (int i = 0; i < 2; i++)
+#pragma unroll
+              for (int c = 0; c < CB; c++) cp_async16(dst + c * BOX + (p * 2 + i) * 1024, page[p] + sl * DK + c * 64 + (size_t)i * 8 * W);
+          cp_async_arrive(smem_u32(k_full + s));
           if (++s == R) { s = 0; ph ^= 1; }
         }
       }
+      cp_async_wait_all();
     }
   } else if (warp == 1) {
-    if (lane == 0 && nb > 0) {
+    if (nb > 0) {                                  // the whole warp walks the loop, one lane issues: operands stay warp-uniform
       constexpr uint32_t idesc = idesc_f16(QB, KEYS, false);
+      const bool issuer = elect_one();
+      const uint64_t k0 = smem_desc_sw128(smem_u32(sK)), q0d = smem_desc_sw128(smem_u32(sQ));
       bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag) && (QS == 0 || mbar_wait(smem_u32(qs_full), 0, abort_flag));
+      int s = 0, ph = 0;                           // slot and parity of the entry
       for (int j = 0; j < nb && ok; j++) {
         const int b = j % NS, use = j / NS;
         if (!mbar_wait(smem_u32(s_empty + b), (uint32_t)(use & 1) ^ 1, abort_flag)) break;
         if (j >= NS && !mbar_wait(smem_u32(pv_done + b), (uint32_t)(use - 1) & 1, abort_flag)) break;      // the weights before lie in this accumulator
+        const uint32_t acc = S_T + b * KEYS;
         for (int u = 0; u < G; u++) {
-          const int e = j * G + u, s = e % R;
-          ok = mbar_wait(smem_u32(k_full + s), (uint32_t)(e / R) & 1, abort_flag);
+          ok = mbar_wait(smem_u32(k_full + s), (uint32_t)ph, abort_flag);
           if (!ok) break;
+          fence_proxy_async_smem();
           tc_fence_after();
-          const uint32_t ka = smem_u32(sK + (size_t)s * SLICE);
-          if (u < a.QT) {
+          const uint64_t kd = k0 + (uint64_t)(s * (SLICE >> 4));
+          if (issuer) {
+            if (u < a.QT) {
+              const uint32_t qt = Q_T + u * (DK / 2);
+              umma_ts(acc, qt, kd, idesc, u != 0 ? 1u : 0u);
 #pragma unroll
-            for (int kk = 0; kk < DK / 16; kk++)
-              umma_ts(S_T + b * KEYS, Q_T + u * (DK / 2) + 8 * kk, smem_desc_sw128_strided(ka + (kk >> 2) * 1024, 16, GROUP) + 2 * (kk & 3), idesc,
-                      u != 0 || kk != 0 ? 1u : 0u);
-          } else {
-            const uint32_t qa = smem_u32(sQ + (size_t)(u - a.QT) * SLICE);
+              for (int kk = 1; kk < DK / 16; kk++) umma_ts(acc, qt + 8 * kk, kd + ((kk >> 2) * (BOX >> 4) + 2 * (kk & 3)), idesc, 1u);
+            } else {
+              const uint64_t qd = q0d + (uint64_t)((u - a.QT) * (SLICE >> 4));
 #pragma unroll
-            for (int kk = 0; kk < DK / 16; kk++)
-              umma_bf16(S_T + b * KEYS, smem_desc_sw128(qa + (kk >> 2) * (QB * 128)) + 2 * (kk & 3),
-                        smem_desc_sw128_strided(ka + (kk >> 2) * 1024, 16, GROUP) + 2 * (kk & 3), idesc, u != 0 || kk != 0 ? 1u : 0u);
+              for (int kk = 0; kk < DK / 16; kk++)
+                umma_bf16(acc, qd + ((kk >> 2) * (BOX >> 4) + 2 * (kk & 3)), kd + ((kk >> 2) * (BOX >> 4) + 2 * (kk & 3)), idesc, 1u);
+            }
+            umma_commit(smem_u32(u != G - 1 ? k_empty + s : s_full + b));
           }
-          if (u != G - 1) umma_commit(smem_u32(k_empty + s));
+          __syncwarp();
+          if (++s == R) { s = 0; ph ^= 1; }
         }
-        umma_commit(smem_u32(s_full + b));
       }
     }
   } else if (warp == 11) {
-    if (lane == 0 && nb > 0) {
+    if (nb > 0) {
       constexpr uint32_t idesc = idesc_f16(QB, DK, true);
+      const bool issuer = elect_one();
+      const uint64_t v0 = smem_desc_sw128_mn(smem_u32(sK), BOX);
       for (int j = 0; j < nb; j++) {
         const int b = j % NS, e = j * G + G - 1, s = e % R;
         if (!mbar_wait(smem_u32(p_full + b), (uint32_t)(j / NS) & 1, abort_flag)) break;      // weights written, output rows rescaled if needed
         if (!mbar_wait(smem_u32(k_full + s), (uint32_t)(e / R) & 1, abort_flag)) break;       // (landed long ago: the scores needed it; only now is the parity its own)
+        fence_proxy_async_smem();
         tc_fence_after();
-        const uint32_t va = smem_u32(sK + (size_t)s * SLICE);
+        const uint64_t vd = v0 + (uint64_t)(s * (SLICE >> 4));
+        if (issuer) {
+          umma_ts(O_T, S_T + b * KEYS, vd, idesc, j != 0 ? 1u : 0u);
 #pragma unroll
-        for (int kk = 0; kk < KEYS / 16; kk++)
-          umma_ts(O_T, S_T + b * KEYS + (kk >> 2) * 64 + 8 * (kk & 3), smem_desc_sw128_strided(va + kk * 2 * GROUP, 1024, GROUP), idesc,
-                  (j != 0 || kk != 0) ? 1u : 0u);
-        umma_commit(smem_u32(pv_done + b));
-        umma_commit(smem_u32(k_empty + s));
+          for (int kk = 1; kk < KEYS / 16; kk++) umma_ts(O_T, S_T + b * KEYS + (kk >> 2) * 64 + 8 * (kk & 3), vd + 128 * kk, idesc, 1u);
+          umma_commit(smem_u32(pv_done + b));
+          umma_commit(smem_u32(k_empty + s));
+        }
+        __syncwarp();
       }
     }
   } else if (warp < 10 && nb > 0) {
@@ -737,26 +772,25 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
     const float slope = a.slopes ? a.slopes[h] : 0.f;
     float m_used = -INFINITY, l = 0.f;           // exponent offset of this row (log2 units), this warp's part of the row sum
     bool ok = true;
-    if (hsel == 0) {
-      const bool in = qs + q0 + row < a.T_total;
-      const __half* qrow = a.q + ((size_t)(qs + q0 + (in ? row : 0)) * a.H + h) * W;
-      for (int u = 0; u < a.QT; u++) {
-        const uint4* src = (const uint4*)(qrow + (own + 1 + u) % G * DK);
+    for (int u0 = 0; u0 < a.QT && ok; u0 += R) {   // this row's queries from the ring to tensor memory, every other box by the partner warp
+      ok = mbar_wait(smem_u32(qt_full), (uint32_t)(u0 / R) & 1, abort_flag);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      const int n = min(R, a.QT - u0) * CB;
+      for (int i = hsel; i < n; i += 2) {
+        const uint8_t* src = sK + (size_t)i * BOX + row * 128;
+        uint32_t r[32];
 #pragma unroll
-        for (int c = 0; c < CB; c++) {
-          uint32_t r[32];
-#pragma unroll
-          for (int i = 0; i < 8; i++) {
-            const uint4 v = in ? src[c * 8 + i] : make_uint4(0u, 0u, 0u, 0u);
-            r[4 * i] = v.x; r[4 * i + 1] = v.y; r[4 * i + 2] = v.z; r[4 * i + 3] = v.w;
-          }
-          tmem_st32(Q_T + lane_addr + u * (DK / 2) + c * 32, r);
-          tmem_st_wait();
+        for (int c = 0; c < 8; c++) {
+          const uint4 v = *(const uint4*)(src + ((c ^ (row & 7)) << 4));
+          r[4 * c] = v.x; r[4 * c + 1] = v.y; r[4 * c + 2] = v.z; r[4 * c + 3] = v.w;
         }
+        tmem_st32(Q_T + lane_addr + (u0 * CB + i) * 32, r);
       }
+      tmem_st_wait();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(smem_u32(q_full));
+      if (lane == 0) mbar_arrive(smem_u32(u0 + R < a.QT ? qt_empty : q_full));
     }
     // both warps of a pair have written their half to xch; `n`: how many times barrier bb has been used
     auto pair_sync = [&](int bb, int n) -> bool {
@@ -765,7 +799,7 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
       const bool k = mbar_wait(smem_u32(x_full + q * 2 + bb), (uint32_t)n & 1, abort_flag);
       return __all_sync(0xffffffffu, k && !*abort_flag);
     };
-    for (int j = 0; j < nb; j++) {
+    for (int j = 0; j < nb && ok; j++) {
       const int b = j % NS, use = j / NS;
       ok = mbar_wait(smem_u32(s_full + b), (uint32_t)use & 1, abort_flag);
       ok = __all_sync(0xffffffffu, ok && !*abort_flag);
@@ -898,7 +932,7 @@ static bool mixed_prefill_plan(int G, int DK, int& ns, int& qt, int& r) {
   if (G < 1 || (DK != 64 && DK != 128)) return false;
   const int slice = KEYS * DK * 2;
   for (ns = 2; ns >= 1; ns--) {
-    const int most = (232448 - 1024 - 36 * 8 - ns * 1024) / slice;
+    const int most = (232448 - 1024 - 38 * 8 - ns * 1024) / slice;
     qt = (512 - ns * KEYS - DK) / (DK / 2);
     if (qt > G) qt = G;
     r = most - (G - qt);
@@ -912,8 +946,8 @@ B200_API int b200_mixed_prefill_ok(int G, int DK) {
   return mixed_prefill_plan(G, DK, ns, qt, r) ? 1 : 0;
 }
 template <int DK, int NS>
-static int launch_mixed_prefill(const CUtensorMap& tk, const CUtensorMap& tq, const MixedPreArgs& a, int n_seqs, int max_q, cudaStream_t st) {
-  const size_t smem = 1024 + (size_t)(a.G - a.QT + a.R) * KEYS * DK * 2 + (20 + 2 * a.R) * 8 + NS * 1024;
+static int launch_mixed_prefill(const CUtensorMap& tq, const MixedPreArgs& a, int n_seqs, int max_q, cudaStream_t st) {
+  const size_t smem = 1024 + (size_t)(a.G - a.QT + a.R) * KEYS * DK * 2 + (22 + 2 * a.R) * 8 + NS * 1024;
   if (smem > 232448) return B200_ERR_BAD_ARG;
   auto kern = mixed_prefill_kernel<DK, NS>;
   static size_t configured = 0;
@@ -922,26 +956,24 @@ static int launch_mixed_prefill(const CUtensorMap& tk, const CUtensorMap& tq, co
     if (e != cudaSuccess) return (int)e;
     configured = smem;
   }
-  return launch_pdl(kern, dim3((max_q + QB - 1) / QB, a.H, n_seqs), dim3(384), smem, st, tk, tq, a);
+  return launch_pdl(kern, dim3((max_q + QB - 1) / QB, a.H, n_seqs), dim3(384), smem, st, tq, a);
 }
 // q fp16 [T_total][H][G * DK] (mixed, scaled); kc fp16 [n_pages][16][G * DK], whole pages of finite numbers; out bf16 [T_total][H * DK], or the same
 // in fp32 to out_f32.  max_q: the longest portion.
-B200_API int b200_mixed_prefill(const void* q, const void* kc, const float* slopes, const float* sinks, const int* page_table, int max_pages, int n_pages,
+B200_API int b200_mixed_prefill(const void* q, const void* kc, const float* slopes, const float* sinks, const int* page_table, int max_pages,
                                 const int* q_start, const int* q_len, const int* ctx_len, int n_seqs, int max_q, int T_total, int H, int G, int DK,
                                 int window, void* out, float* out_f32, int* status, cudaStream_t st) {
   int ns, qt, r;
-  if (n_seqs < 1 || max_q < 1 || T_total < 1 || H < 1 || window < 0 || !q || !kc || !page_table || (!out && !out_f32) || G < 1 || H % G ||
+  if (n_seqs < 1 || max_q < 1 || T_total < 1 || H < 1 || window < 0 || !q || !kc || ((uintptr_t)kc & 15) || !page_table || (!out && !out_f32) || G < 1 || H % G ||
       !mixed_prefill_plan(G, DK, ns, qt, r))
     return B200_ERR_BAD_ARG;
   MixedPreArgs a = {};
-  a.q = (const __half*)q; a.slopes = slopes; a.sinks = sinks; a.page_table = page_table; a.q_start = q_start; a.q_len = q_len; a.ctx_len = ctx_len;
+  a.q = (const __half*)q; a.kc = (const __half*)kc; a.slopes = slopes; a.sinks = sinks; a.page_table = page_table; a.q_start = q_start; a.q_len = q_len; a.ctx_len = ctx_len;
   a.max_pages = max_pages; a.H = H; a.G = G; a.T_total = T_total; a.window = window; a.QT = qt; a.R = r; a.out = (__nv_bfloat16*)out; a.out_f32 = out_f32;
   a.status = status;
-  CUtensorMap tk, tq;
-  int rc = make_tmap_rows8(&tk, kc, (uint64_t)n_pages * 16, (uint64_t)G * DK, DK / 64);
+  CUtensorMap tq;
+  const int rc = make_tmap_2d(&tq, q, 2, (uint64_t)T_total, (uint64_t)H * G * DK, (uint64_t)H * G * DK * 2, QB, 64, true);
   if (rc) return rc;
-  rc = make_tmap_2d(&tq, q, 2, (uint64_t)T_total, (uint64_t)H * G * DK, (uint64_t)H * G * DK * 2, QB, 64, true);
-  if (rc) return rc;
-  if (DK == 64) return ns == 2 ? launch_mixed_prefill<64, 2>(tk, tq, a, n_seqs, max_q, st) : launch_mixed_prefill<64, 1>(tk, tq, a, n_seqs, max_q, st);
-  return ns == 2 ? launch_mixed_prefill<128, 2>(tk, tq, a, n_seqs, max_q, st) : launch_mixed_prefill<128, 1>(tk, tq, a, n_seqs, max_q, st);
+  if (DK == 64) return ns == 2 ? launch_mixed_prefill<64, 2>(tq, a, n_seqs, max_q, st) : launch_mixed_prefill<64, 1>(tq, a, n_seqs, max_q, st);
+  return ns == 2 ? launch_mixed_prefill<128, 2>(tq, a, n_seqs, max_q, st) : launch_mixed_prefill<128, 1>(tq, a, n_seqs, max_q, st);
 }

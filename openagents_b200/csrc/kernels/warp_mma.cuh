@@ -1,10 +1,21 @@
-// Warp-level matrix instructions: shared-memory fragment loads and the m16n8k16 products.  Attention over one query per sequence has a handful of
+// Warp-level matrix instructions (shared-memory fragment loads and the m16n8k16 products) and 16-byte asynchronous copies.  Attention over one query per sequence has a handful of
 // rows per key head, far from the 128 of a tcgen05 tile, and is bound by the cache's bytes; these fit it.
 #pragma once
 #include "common.cuh"
 
 namespace b200 {
 
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() {
+  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+// Arrives on the mbarrier once every copy this thread has issued so far has landed (one of the arrivals the barrier was made for).
+__device__ __forceinline__ void cp_async_arrive(uint32_t bar) { asm volatile("cp.async.mbarrier.arrive.noinc.shared::cta.b64 [%0];" ::"r"(bar) : "memory"); }
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));

@@ -56,7 +56,7 @@ _SIGS = {
     "b200_mixed_finish": [_P] + [c_int] * 3 + [_P, _P, c_float, _P] + [c_int] * 5 + [_P, _P, _P, c_int, _P],
     "b200_mixed_decode": [_P] * 6 + [c_int, c_int, _P] + [c_int] * 6 + [_P] * 5,
     "b200_mixed_decode_ok": [c_int] * 3,
-    "b200_mixed_prefill": [_P] * 5 + [c_int, c_int, _P, _P, _P] + [c_int] * 7 + [_P] * 4,
+    "b200_mixed_prefill": [_P] * 5 + [c_int, _P, _P, _P] + [c_int] * 7 + [_P] * 4,
     "b200_mixed_prefill_ok": [c_int] * 2,
     "b200_moe_zero": [_P, c_int, _P],
     "b200_set_pdl": [c_int],
@@ -498,8 +498,8 @@ def mixed_decode(q, kc, mix, slopes, page_table, seq_lens, B, H, G, DK, window=0
 
 def mixed_prefill(q16, kc, slopes, page_table, q_start, q_len, ctx_len, n_seqs, max_q, H, G, DK, window=0, sinks=None, out_bf16=None, out_f32=None, status=None):
     """Prompt portions with wide queries: ``q16`` fp16 [T, H * G * DK] from :func:`mixed_finish`, against the same cache rows."""
-    _check(lib().b200_mixed_prefill(_p(q16), _p(kc), _p(slopes), _p(sinks), _p(page_table), page_table.shape[1], kc.shape[0], _p(q_start), _p(q_len),
-                                    _p(ctx_len), n_seqs, max_q, q16.shape[0], H, G, DK, window, _p(out_bf16), _p(out_f32), _p(status), _st()), "mixed_prefill")
+    _check(lib().b200_mixed_prefill(_p(q16), _p(kc), _p(slopes), _p(sinks), _p(page_table), page_table.shape[1], _p(q_start), _p(q_len), _p(ctx_len),
+                                    n_seqs, max_q, q16.shape[0], H, G, DK, window, _p(out_bf16), _p(out_f32), _p(status), _st()), "mixed_prefill")
 
 
 def norm_dyt(x, alpha, w, b, hb=None, hf=None, ids=None, emb=None, zero=None):
