@@ -606,7 +606,7 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
   uint64_t* k_empty = k_full + R;                         // [R]
   float* xch = (float*)(bars + 22 + 2 * R);               // [NS][2 (half)][128 rows]
 
-  const int seq = blockIdx.z, h = blockIdx.y, qb = gridDim.x - 1 - blockIdx.x;   // longest (latest) query blocks first
+  const int seq = blockIdx.z, h = blockIdx.x, qb = gridDim.y - 1 - blockIdx.y;   // every head's longest (latest) query blocks first
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
     mbar_init(smem_u32(q_full), 8);
@@ -647,6 +647,10 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
   const int k_hi = min(ctx, pos0 + QB), k_lo = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
   const int jb0 = k_lo / KEYS, nb = live ? (k_hi + KEYS - 1) / KEYS - jb0 : 0;
   const uint32_t S_T = tmem_base, O_T = tmem_base + NS * KEYS, Q_T = O_T + DK;
+  // what goes to tensor memory passes through the place of the slices that stay in shared memory, where they are as many, else through the ring
+  const bool in_place = QS >= a.QT;
+  uint8_t* sStage = in_place ? sQ : sK;
+  const int stage = in_place ? a.QT : R;
 
   if (warp == 0 || warp == 10) {
     // Entries e = j * G + u in order (block j, u-th slice of it), all by both warps: thread x copies 16-byte piece x % 8 of every eighth row.  The
@@ -654,29 +658,38 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
     if (nb > 0) {
       const int* pt = a.page_table + (size_t)seq * a.max_pages;
       bool ok = true;
-      // the queries: QT slices through the ring to tensor memory, R at a time, the others to where they stay
+      // the queries: QT slices by way of shared memory to tensor memory, `stage` at a time, the others to where they stay
       if (warp == 0 && lane == 0) {
         auto fetch = [&](uint8_t* to, int u, uint32_t bar) {
           for (int c = 0; c < CB; c++) tma_load_2d(smem_u32(to + c * BOX), &tmQ, bar, h * W + (own + 1 + u) % G * DK + c * 64, qs + q0);
         };
-        for (int u0 = 0; u0 < a.QT && ok; u0 += R) {
-          const int n = min(R, a.QT - u0);
-          if (u0 > 0) ok = mbar_wait(smem_u32(qt_empty), (uint32_t)(u0 / R - 1) & 1, abort_flag);
+        for (int u0 = 0; u0 < a.QT && ok; u0 += stage) {
+          const int n = min(stage, a.QT - u0);
+          if (u0 > 0) ok = mbar_wait(smem_u32(qt_empty), (uint32_t)(u0 / stage - 1) & 1, abort_flag);
           if (!ok) break;
           mbar_expect_tx(smem_u32(qt_full), n * SLICE);
-          for (int i = 0; i < n; i++) fetch(sK + (size_t)i * SLICE, u0 + i, smem_u32(qt_full));
-          if (u0 == 0 && QS > 0) {
-            mbar_expect_tx(smem_u32(qs_full), QS * SLICE);
-            for (int u = a.QT; u < G; u++) fetch(sQ + (size_t)(u - a.QT) * SLICE, u, smem_u32(qs_full));
-          }
+          for (int i = 0; i < n; i++) fetch(sStage + (size_t)i * SLICE, u0 + i, smem_u32(qt_full));
         }
       }
-      ok = __all_sync(0xffffffffu, ok) && mbar_wait(smem_u32(q_full), 0, abort_flag);      // the ring is free for keys
+      ok = __all_sync(0xffffffffu, ok);
+      if (!in_place && ok) ok = mbar_wait(smem_u32(q_full), 0, abort_flag);      // the ring is free for keys
       ok = __all_sync(0xffffffffu, ok);
       const int x = (warp == 0 ? 0 : 32) + lane, r0 = x >> 3, c0 = x & 7;
       const uint32_t dst0 = smem_u32(sK) + (uint32_t)(r0 * 128 + ((c0 ^ r0) << 4));
       const __half* src0 = a.kc + (size_t)r0 * W + c0 * 8;
       int s = 0, ph = 1;                           // slot of the entry and the parity of its being free
+      auto fetch_rest = [&]() {                    // the slices that stay in shared memory, once nothing passes through there any more
+        if (QS == 0 || !ok || warp != 0) return;
+        if (in_place) ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(q_full), 0, abort_flag));
+        if (ok && lane == 0) {
+          mbar_expect_tx(smem_u32(qs_full), QS * SLICE);
+          for (int u = a.QT; u < G; u++)
+            for (int c = 0; c < CB; c++)
+              tma_load_2d(smem_u32(sQ + (size_t)(u - a.QT) * SLICE + c * BOX), &tmQ, smem_u32(qs_full), h * W + (own + 1 + u) % G * DK + c * 64, qs + q0);
+        }
+        __syncwarp();
+      };
+      if (!in_place) fetch_rest();
       for (int j = 0; j < nb && ok; j++) {
         const __half* page[KEYS / 16];             // read together: one at a time, their latency would bound the copies
 #pragma unroll
@@ -699,6 +712,7 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
               for (int c = 0; c < CB; c++) cp_async16(dst + c * BOX + (p * 2 + i) * 1024, page[p] + sl * DK + c * 64 + (size_t)i * 8 * W);
           cp_async_arrive(smem_u32(k_full + s));
           if (++s == R) { s = 0; ph ^= 1; }
+          if (in_place && j == 0 && u == min(a.QT, R) - 1) fetch_rest();      // behind the first keys, which need no more than tensor memory's part
         }
       }
       cp_async_wait_all();
@@ -708,7 +722,7 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
       constexpr uint32_t idesc = idesc_f16(QB, KEYS, false);
       const bool issuer = elect_one();
       const uint64_t k0 = smem_desc_sw128(smem_u32(sK)), q0d = smem_desc_sw128(smem_u32(sQ));
-      bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag) && (QS == 0 || mbar_wait(smem_u32(qs_full), 0, abort_flag));
+      bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag);
       int s = 0, ph = 0;                           // slot and parity of the entry
       for (int j = 0; j < nb && ok; j++) {
         const int b = j % NS, use = j / NS;
@@ -716,7 +730,7 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
         if (j >= NS && !mbar_wait(smem_u32(pv_done + b), (uint32_t)(use - 1) & 1, abort_flag)) break;      // the weights before lie in this accumulator
         const uint32_t acc = S_T + b * KEYS;
         for (int u = 0; u < G; u++) {
-          ok = mbar_wait(smem_u32(k_full + s), (uint32_t)ph, abort_flag);
+          ok = mbar_wait(smem_u32(k_full + s), (uint32_t)ph, abort_flag) && (j > 0 || u != a.QT || mbar_wait(smem_u32(qs_full), 0, abort_flag));
           if (!ok) break;
           fence_proxy_async_smem();
           tc_fence_after();
@@ -772,13 +786,13 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
     const float slope = a.slopes ? a.slopes[h] : 0.f;
     float m_used = -INFINITY, l = 0.f;           // exponent offset of this row (log2 units), this warp's part of the row sum
     bool ok = true;
-    for (int u0 = 0; u0 < a.QT && ok; u0 += R) {   // this row's queries from the ring to tensor memory, every other box by the partner warp
-      ok = mbar_wait(smem_u32(qt_full), (uint32_t)(u0 / R) & 1, abort_flag);
+    for (int u0 = 0; u0 < a.QT && ok; u0 += stage) {   // this row's queries to tensor memory, every other box by the partner warp
+      ok = mbar_wait(smem_u32(qt_full), (uint32_t)(u0 / stage) & 1, abort_flag);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
-      const int n = min(R, a.QT - u0) * CB;
+      const int n = min(stage, a.QT - u0) * CB;
       for (int i = hsel; i < n; i += 2) {
-        const uint8_t* src = sK + (size_t)i * BOX + row * 128;
+        const uint8_t* src = sStage + (size_t)i * BOX + row * 128;
         uint32_t r[32];
 #pragma unroll
         for (int c = 0; c < 8; c++) {
@@ -790,7 +804,7 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(smem_u32(u0 + R < a.QT ? qt_empty : q_full));
+      if (lane == 0) mbar_arrive(smem_u32(u0 + stage < a.QT ? qt_empty : q_full));
     }
     // both warps of a pair have written their half to xch; `n`: how many times barrier bb has been used
     auto pair_sync = [&](int bb, int n) -> bool {
@@ -822,11 +836,10 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
       const int kb0 = (jb0 + j) * KEYS;
       const float base = slope * (float)(kb0 + hsel * HK - qpos);      // the distance's part that all of this warp's keys of the block share
       if (kb0 + KEYS - 1 > pos0 || kb0 + KEYS > ctx || kb0 < lo_max) {
+        const int lo = row_lo - kb0 - hsel * HK, hi = min(qpos, ctx - 1) - kb0 - hsel * HK;
 #pragma unroll
-        for (int i = 0; i < HK; i++) {
-          const int kp = kb0 + hsel * HK + i;
-          if (kp > qpos || kp >= ctx || kp < row_lo) sv[i] = -INFINITY;
-        }
+        for (int i = 0; i < HK; i++)
+          if (i < lo || i > hi) sv[i] = -INFINITY;
       }
       float mx0 = fmaxf(sv[0], sv[1]), mx1 = fmaxf(sv[2], sv[3]);
 #pragma unroll
@@ -895,26 +908,31 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
       tc_fence_after();
       if (a.sinks) l += (m_used == -INFINITY) ? 1.f : ex2_approx(a.sinks[h] * kLog2e - m_used);
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      const bool wr = ok && row < qlen - q0;
-      const size_t at = (size_t)(qs + q0 + row) * a.H * DK + (size_t)h * DK + hsel * HO;
+      // 32 rows of HO columns per warp go through shared memory (the ring, whose last reader has finished), so that whole lines leave
+      const int rows = ok ? min(32, qlen - q0 - q * 32) : 0;
+      float* stg = (float*)sK + (size_t)(warp - 2) * 32 * 32;
 #pragma unroll
       for (int c = 0; c < HO / 32; c++) {
         uint32_t r[32];
         tmem_ld32(O_T + lane_addr + hsel * HO + c * 32, r);
         tmem_ld_wait();
-        if (wr && a.out_f32) {
+        __syncwarp();
 #pragma unroll
-          for (int i = 0; i < 32; i += 4)
-            *(float4*)(a.out_f32 + at + c * 32 + i) = make_float4(__uint_as_float(r[i]) * inv, __uint_as_float(r[i + 1]) * inv,
-                                                                  __uint_as_float(r[i + 2]) * inv, __uint_as_float(r[i + 3]) * inv);
-        } else if (wr) {
+        for (int i = 0; i < 8; i++)
+          *(float4*)(stg + lane * 32 + ((i ^ (lane & 7)) << 2)) = make_float4(__uint_as_float(r[4 * i]) * inv, __uint_as_float(r[4 * i + 1]) * inv,
+                                                                             __uint_as_float(r[4 * i + 2]) * inv, __uint_as_float(r[4 * i + 3]) * inv);
+        __syncwarp();
 #pragma unroll
-          for (int i = 0; i < 32; i += 8) {
-            uint4 v;
-            __nv_bfloat162* p = (__nv_bfloat162*)&v;
-#pragma unroll
-            for (int k = 0; k < 4; k++) p[k] = __floats2bfloat162_rn(__uint_as_float(r[i + 2 * k]) * inv, __uint_as_float(r[i + 2 * k + 1]) * inv);
-            *(uint4*)(a.out + at + c * 32 + i) = v;
+        for (int i = 0; i < 8; i++) {
+          const int rr = i * 4 + (lane >> 3), p = lane & 7;
+          if (rr >= rows) continue;
+          const float4 v = *(const float4*)(stg + rr * 32 + ((p ^ (rr & 7)) << 2));
+          const size_t at = ((size_t)(qs + q0 + q * 32 + rr) * a.H + h) * DK + hsel * HO + c * 32 + p * 4;
+          if (a.out_f32) {
+            *(float4*)(a.out_f32 + at) = v;
+          } else {
+            const __nv_bfloat162 x = __floats2bfloat162_rn(v.x, v.y), y = __floats2bfloat162_rn(v.z, v.w);
+            *(uint2*)(a.out + at) = make_uint2(*(const uint32_t*)&x, *(const uint32_t*)&y);
           }
         }
       }
@@ -956,7 +974,7 @@ static int launch_mixed_prefill(const CUtensorMap& tq, const MixedPreArgs& a, in
     if (e != cudaSuccess) return (int)e;
     configured = smem;
   }
-  return launch_pdl(kern, dim3((max_q + QB - 1) / QB, a.H, n_seqs), dim3(384), smem, st, tq, a);
+  return launch_pdl(kern, dim3(a.H, (max_q + QB - 1) / QB, n_seqs), dim3(384), smem, st, tq, a);
 }
 // q fp16 [T_total][H][G * DK] (mixed, scaled); kc fp16 [n_pages][16][G * DK], whole pages of finite numbers; out bf16 [T_total][H * DK], or the same
 // in fp32 to out_f32.  max_q: the longest portion.
