@@ -284,8 +284,8 @@ def time_kazolorn_kernels(cfg, dev, reps: int = 12) -> list[dict]:
             e = HybridEngine.__new__(HybridEngine)
             e.max_splits = 64
             S = e._mixed_splits(n, min(pages, win // 16 + 2))
-            sc = rnd(ops.mixed_decode_scratch_floats(n, H, G, D, S))
-            bench(f"mixed_decode [{n} x {seen}] ({S} shares)", lambda: ops.mixed_decode(l32, kc, mixw, slopes, table, lens, n, H, G, D, window=win, S=S, sinks=zero, out_bf16=o,
+            sc, prep = rnd(ops.mixed_decode_scratch_floats(n, H, G, D, S)), ops.mixed_decode_prepare(mixw, slopes, H, G, D)
+            bench(f"mixed_decode [{n} x {seen}] ({S} shares)", lambda: ops.mixed_decode(l32, kc, prep, table, lens, n, H, G, D, window=win, S=S, sinks=zero, out_bf16=o,
                                                                                      scratch=sc, status=st), n * (seen * nk * 2 + nq * 6),
                   2.0 * n * seen * H * (2 * D + H), like=f"attn_decode [{n} x {seen}]")
             e.attn_target_ctas = 0

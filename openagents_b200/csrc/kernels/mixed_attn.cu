@@ -136,20 +136,17 @@ B200_API int b200_mixed_finish(const float* in, int ld, int T, int k_off, const 
 
 // ------------------------------------------------------------------ decoding: one query token per sequence
 
-// Grid (shares of the keys, value parts, sequences).  Pages come whole, all key heads of 16 tokens, in one TMA copy each: [2][W / 64][8 rows][128
-// bytes], swizzled, into a ring whose slots are a multiple of the warps; a warp takes every nw-th page of the CTA's share (so a slot is always the same
-// warp's) and works on it alone:
-//   raw scores      S^T = K Q^T per key head, 16 keys x 8 query heads a tile
+// Grid (shares of the keys, sequences).  Pages come whole, all key heads of 16 tokens, in one TMA copy each: [2][W / 64][8 rows][128 bytes], swizzled,
+// into a ring.  Two warps work on a page, each for half of the query heads (a slot of the ring is always the same pair's):
+//   raw scores      S^T = K Q^T per key head, 16 keys x 8 query heads a tile; the two warps swap theirs through shared memory
 //   mixture         S^T T^T on bf16 products: the scores as three bf16 pieces (24 bits: fp32's own), T is stored in bf16
 //   softmax         running, in base 2; a head's offset moves only when its maximum has grown by 2^8
 //   output          O^T += K^T P^T, the transposed weights coming from movmatrix
 // A group's query heads are padded to RP of 1, 2, 4 or a multiple of 8.  Where a tile's eight heads belong to several groups, the raw product runs
 // over all their keys with the other groups' queries as zeros, and the output product puts 8 keys of two groups into one step of 16.
-// Heads beyond what a warp's registers hold as outputs are served by several CTAs (value parts), each mixing for its own tiles.
 struct MixedDecArgs {
   const float* q;          // [B][H * DK], scaled
-  const float* mix;        // [H][H]
-  const float* slopes;     // [H], of the mixed scores
+  const uint2* mix;        // the mixture as B operand (see mixed_prepare_kernel), then the padded heads' slopes
   const float* sinks;      // [H] or null
   const int* page_table;
   const int* seq_lens;
@@ -166,45 +163,64 @@ __device__ __forceinline__ float2 split_bf16(float x, float y, uint32_t& packed)
   const float2 f = __bfloat1622float2(p);
   return make_float2(x - f.x, y - f.y);
 }
+__device__ __forceinline__ void pair_barrier(int pair) { asm volatile("bar.sync %0, 64;" ::"r"(pair + 1) : "memory"); }
 
-// NT: tiles of eight (padded) query heads, an even number; NTV: those whose outputs this CTA keeps
-template <int DK, int NT, int NTV>
-__global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant__ CUtensorMap tm, const MixedDecArgs a) {
-  constexpr int QLD = DK + 8, KB = DK / 64;
+// Once per layer, at load: out [NT / 2][NT][32 lanes] = the fragments of T^T (rows the raw slots, columns the mixed ones), and [8 NT] slopes in base 2.
+__global__ void mixed_prepare_kernel(const float* __restrict__ mix, const float* __restrict__ slopes, int H, int G, int rp, int NT, uint2* __restrict__ out) {
+  const int rep = H / G, n = NT / 2 * NT * 32;
+  auto head_of = [&](int slot) { return slot < G * rp && slot % rp < rep ? slot / rp * rep + slot % rp : -1; };
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const int l = i & 31, nt = (i >> 5) % NT, kk = (i >> 5) / NT, ho = head_of(nt * 8 + (l >> 2));
+    uint32_t w[2];
+    for (int e = 0; e < 2; e++) {
+      const int k = kk * 16 + e * 8 + (l & 3) * 2, h0 = head_of(k), h1 = head_of(k + 1);
+      const __nv_bfloat162 v = __floats2bfloat162_rn(ho >= 0 && h0 >= 0 ? mix[ho * H + h0] : 0.f, ho >= 0 && h1 >= 0 ? mix[ho * H + h1] : 0.f);
+      w[e] = *(const uint32_t*)&v;
+    }
+    out[i] = make_uint2(w[0], w[1]);
+  }
+  for (int i = threadIdx.x; i < 8 * NT; i += blockDim.x) {
+    const int h = head_of(i);
+    ((float*)(out + n))[i] = h >= 0 && slopes ? slopes[h] * kLog2e : 0.f;
+  }
+}
+
+// NT: tiles of eight (padded) query heads, an even number; THREADS: at most that many (registers).
+template <int DK, int NT, int THREADS>
+__global__ void __launch_bounds__(THREADS, 1) mixed_decode_kernel(const __grid_constant__ CUtensorMap tm, const MixedDecArgs a) {
+  constexpr int QLD = DK + 8, KB = DK / 64, NW = NT / 2, SLOTS = 8 * NT;       // NW: tiles of a warp
   extern __shared__ uint8_t dyn_raw[];
-  __shared__ float s_ml[8][NTV * 8][2];
+  __shared__ float s_ml[THREADS / 64][SLOTS][2];
+  __shared__ int s_fail[THREADS / 64];
   __shared__ int s_abort;
   uint8_t* ring = (uint8_t*)(((uintptr_t)dyn_raw + 1023) & ~(uintptr_t)1023);
-  const int W = a.G * DK, page_bytes = 32 * W, NB = W / 64, nw = blockDim.x >> 5;
-  float* s_acc = (float*)ring;                                           // [nw][NTV * 8][DK], once the pages are done with
-  const size_t ring_bytes = max((size_t)a.nslot * page_bytes, (size_t)nw * NTV * 8 * DK * 4);
+  const int W = a.G * DK, page_bytes = 32 * W, NB = W / 64, pairs = blockDim.x >> 6;
+  float* s_acc = (float*)ring;                                           // [pairs][SLOTS][DK], once the pages are done with
+  const size_t ring_bytes = max((size_t)a.nslot * page_bytes, (size_t)pairs * SLOTS * DK * 4);
   uint64_t* bars = (uint64_t*)(ring + ring_bytes);
-  __half* sQ = (__half*)(bars + ((a.nslot + 1) & ~1));                   // [8 NT + 1][QLD], the last row zeros
-  uint2* sT = (uint2*)(sQ + (8 * NT + 1) * QLD + 8 * ((8 * NT + 1) & 1));             // [NT / 2][NTV][32]
-  int* s_pid = (int*)(sT + NT / 2 * NTV * 32);
+  float4* sX = (float4*)(bars + ((a.nslot + 1) & ~1));                   // [pairs][2][NW][32] raw scores on their way to the partner
+  uint2* sT = (uint2*)(sX + pairs * NT * 32);                            // [NT / 2][NT][32]
+  __half* sQ = (__half*)(sT + NT / 2 * NT * 32);                         // [SLOTS + 1][QLD], the last row zeros
+  int* s_pid = (int*)(sQ + (SLOTS + 1) * QLD);
 
-  const int split = blockIdx.x, part = blockIdx.y, b = blockIdx.z;
+  const int split = blockIdx.x, b = blockIdx.y;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
-  const int rp = a.rp, rep = a.H / a.G, live = a.G * rp, nsub = rp < 8 ? 8 / rp : 1;      // live: padded heads that exist
-  auto head_of = [&](int slot) { return slot < live && slot % rp < rep ? slot / rp * rep + slot % rp : -1; };
+  const int pair = warp >> 1, hf = warp & 1, T0 = hf * NW;               // this warp's first tile
+  const int rp = a.rp, rep = a.H / a.G, nsub = rp < 8 ? 8 / rp : 1;
   if (tid == 0) {
     for (int s = 0; s < a.nslot; s++) mbar_init(smem_u32(bars + s), 1);
     s_abort = 0;
     fence_barrier_init();
     tma_prefetch_desc(&tm);
   }
-  // the mixture as B operand: rows the raw slots, columns this part's slots (weights: nothing to wait for)
-  for (int i = tid; i < NT / 2 * NTV * 32; i += blockDim.x) {
-    const int l = i & 31, nt = (i >> 5) % NTV, kk = (i >> 5) / NTV, ho = head_of((part * NTV + nt) * 8 + (l >> 2));
-    uint32_t w[2];
+  if (tid < pairs) s_fail[tid] = 0;
+  for (int i = tid; i < (SLOTS + 1) * QLD / 8; i += blockDim.x) ((uint4*)sQ)[i] = make_uint4(0u, 0u, 0u, 0u);
+  for (int i = tid; i < NT * NT * 8; i += blockDim.x) ((uint4*)sT)[i] = ((const uint4*)a.mix)[i];           // weights: nothing to wait for
+  float sl[NW][2];
 #pragma unroll
-    for (int e = 0; e < 2; e++) {
-      const int k = kk * 16 + e * 8 + (l & 3) * 2, h0 = head_of(k), h1 = head_of(k + 1);
-      const __nv_bfloat162 v = __floats2bfloat162_rn(ho >= 0 && h0 >= 0 ? a.mix[ho * a.H + h0] : 0.f, ho >= 0 && h1 >= 0 ? a.mix[ho * a.H + h1] : 0.f);
-      w[e] = *(const uint32_t*)&v;
-    }
-    sT[i] = make_uint2(w[0], w[1]);
-  }
+  for (int nt = 0; nt < NW; nt++)
+#pragma unroll
+    for (int e = 0; e < 2; e++) sl[nt][e] = ((const float*)(a.mix + NT * NT * 16))[(T0 + nt) * 8 + 2 * t4 + e];
   pdl_trigger();
   pdl_wait();
   const int len = a.seq_lens[b];
@@ -213,61 +229,57 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
   const int per = (p_last - p_first + a.S - 1) / a.S;
   const int pa = p_first + split * per, np = max(0, min(p_last, pa + per) - pa);
   const int* pt = a.page_table + (size_t)b * a.max_pages;
-  for (int i = tid; i < np; i += blockDim.x) s_pid[i] = pt[pa + i];
-  __syncthreads();
-  auto issue = [&](int i) {   // one lane: page i of the share into its slot
+  auto issue = [&](int i, int page) {   // one lane: page i of the share into its slot
     const uint32_t bar = smem_u32(bars + i % a.nslot);
     mbar_expect_tx(bar, page_bytes);
-    tma_load_4d(smem_u32(ring + (size_t)(i % a.nslot) * page_bytes), &tm, bar, 0, 0, 0, s_pid[i] * 2);
+    tma_load_4d(smem_u32(ring + (size_t)(i % a.nslot) * page_bytes), &tm, bar, 0, 0, 0, page * 2);
   };
-  if (lane == 0)
-    for (int i = warp; i < min(np, a.nslot); i += nw) issue(i);
-  for (int i = tid; i < (8 * NT + 1) * (DK / 2); i += blockDim.x) {
-    const int slot = i / (DK / 2), c = i % (DK / 2) * 2, h = slot < 8 * NT ? head_of(slot) : -1;
-    const float2 v = h >= 0 ? *(const float2*)(a.q + ((size_t)b * a.H + h) * DK + c) : make_float2(0.f, 0.f);
-    *(__half2*)(sQ + slot * QLD + c) = __floats2half2_rn(v.x, v.y);
+  __syncthreads();
+  if (lane == 0 && hf == 0)
+    for (int i = pair; i < min(np, a.nslot); i += pairs) issue(i, pt[pa + i]);
+  for (int i = tid; i < np; i += blockDim.x) s_pid[i] = pt[pa + i];
+  for (int i = tid; i < a.H * (DK / 4); i += blockDim.x) {
+    const int h = i / (DK / 4), c = i % (DK / 4) * 4;
+    const float4 v = ((const float4*)(a.q + (size_t)b * a.H * DK))[i];
+    *(uint2*)(sQ + (h / rep * rp + h % rep) * QLD + c) = make_uint2(pack_h2(v.x, v.y), pack_h2(v.z, v.w));
   }
   __syncthreads();
 
-  float o[NTV][DK / 16][4], mu[NTV][2], l[NTV][2], sl[NTV][2];
+  float o[NW][DK / 16][4], mu[NW][2], l[NW][2];
 #pragma unroll
-  for (int nt = 0; nt < NTV; nt++) {
+  for (int nt = 0; nt < NW; nt++) {
 #pragma unroll
     for (int m = 0; m < DK / 16; m++) o[nt][m][0] = o[nt][m][1] = o[nt][m][2] = o[nt][m][3] = 0.f;
-#pragma unroll
-    for (int e = 0; e < 2; e++) {
-      const int h = head_of((part * NTV + nt) * 8 + 2 * t4 + e);
-      mu[nt][e] = -INFINITY;
-      l[nt][e] = 0.f;
-      sl[nt][e] = h >= 0 && a.slopes ? a.slopes[h] * kLog2e : 0.f;
-    }
+    mu[nt][0] = mu[nt][1] = -INFINITY;
+    l[nt][0] = l[nt][1] = 0.f;
   }
   const int mi = lane >> 3, r8 = lane & 7;              // ldmatrix: tile and row of this lane's address
-  for (int i = warp; i < np; i += nw) {
+  float4* xs = sX + (size_t)pair * NT * 32 + lane;      // [2][NW], 32 apart
+  for (int i = pair; i < np; i += pairs) {
     const int s = i % a.nslot;
     bool ok = mbar_wait(smem_u32(bars + s), (uint32_t)((i / a.nslot) & 1), &s_abort);
     ok = __all_sync(0xffffffffu, ok);
-    if (!ok) break;
+    if (!ok) s_fail[pair] = 1;                           // both warps meet at the barrier below and leave together
     const uint32_t page = smem_u32(ring) + (uint32_t)(s * page_bytes);
     // key row `row` of the page at key head c, and 16-byte piece `ch` of it (r8: the row's place among its eight)
     auto row_at = [&](int row, int c) { return page + (uint32_t)((row >> 3) * NB + c * KB) * 1024u + (uint32_t)r8 * 128u; };
     auto piece_at = [&](int ch) { return (uint32_t)(ch >> 3) * 1024u + (uint32_t)(((ch & 7) ^ r8) << 4); };
-    float sc[NT][4];
+    float sc[NW][4];
 #pragma unroll
-    for (int j = 0; j < NT; j++) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+    for (int j = 0; j < NW; j++) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
 #pragma unroll 1
     for (int u = 0; u < nsub; u++) {
-      uint32_t ka[NT], qa[NT];                            // tile j: this lane's key row of the u-th head the tile meets, its query row
+      uint32_t ka[NW], qa[NW];                            // tile j: this lane's key row of the u-th head the tile meets, its query row
 #pragma unroll
-      for (int j = 0; j < NT; j++) {
-        const int c = rp < 8 ? j * nsub + u : j * 8 / rp;
+      for (int j = 0; j < NW; j++) {
+        const int c = rp < 8 ? (T0 + j) * nsub + u : (T0 + j) * 8 / rp;
         ka[j] = row_at(r8 + (mi & 1) * 8, min(c, a.G - 1));       // (a head that is not there meets zero queries)
-        qa[j] = smem_u32(sQ + ((rp >= 8 || r8 / rp == u) ? j * 8 + r8 : 8 * NT) * QLD + mi * 8);
+        qa[j] = smem_u32(sQ + ((rp >= 8 || r8 / rp == u) ? (T0 + j) * 8 + r8 : SLOTS) * QLD + mi * 8);
       }
 #pragma unroll
       for (int kk = 0; kk < DK / 32; kk++)
 #pragma unroll
-        for (int j = 0; j < NT; j++) {
+        for (int j = 0; j < NW; j++) {
           uint32_t k0[4], k1[4], q[4];
           ldsm_x4(ka[j] + piece_at(kk * 4 + (mi >> 1)), k0[0], k0[1], k0[2], k0[3]);
           ldsm_x4(ka[j] + piece_at(kk * 4 + 2 + (mi >> 1)), k1[0], k1[1], k1[2], k1[3]);
@@ -276,35 +288,54 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
           mma16816(sc[j], k1, q[2], q[3]);
         }
     }
-    float d[NTV][4];
+    // the partner's tiles
+    float ot[NW][4];
 #pragma unroll
-    for (int nt = 0; nt < NTV; nt++) d[nt][0] = d[nt][1] = d[nt][2] = d[nt][3] = 0.f;
+    for (int j = 0; j < NW; j++) xs[(hf * NW + j) * 32] = make_float4(sc[j][0], sc[j][1], sc[j][2], sc[j][3]);
+    pair_barrier(pair);
+    if (*(volatile int*)&s_fail[pair]) break;
 #pragma unroll
-    for (int kk = 0; kk < NT / 2; kk++) {
+    for (int j = 0; j < NW; j++) {
+      const float4 v = xs[((hf ^ 1) * NW + j) * 32];
+      ot[j][0] = v.x; ot[j][1] = v.y; ot[j][2] = v.z; ot[j][3] = v.w;
+    }
+    float d[NW][4];
+#pragma unroll
+    for (int nt = 0; nt < NW; nt++) d[nt][0] = d[nt][1] = d[nt][2] = d[nt][3] = 0.f;
+    auto mix_step = [&](int kk, const float (&x)[4], const float (&y)[4]) {      // raw slots 16 kk .. 16 kk + 15
       uint32_t hi[4], md[4], lo[4];
 #pragma unroll
-      for (int x = 0; x < 4; x++) {
-        const float* v = &sc[2 * kk + (x >> 1)][(x & 1) * 2];
-        float2 r = split_bf16(v[0], v[1], hi[x]);
-        r = split_bf16(r.x, r.y, md[x]);
-        split_bf16(r.x, r.y, lo[x]);
+      for (int p = 0; p < 4; p++) {
+        const float* v = (p < 2 ? x : y) + (p & 1) * 2;
+        float2 r = split_bf16(v[0], v[1], hi[p]);
+        r = split_bf16(r.x, r.y, md[p]);
+        split_bf16(r.x, r.y, lo[p]);
       }
-      uint2 w[NTV];
+      uint2 w[NW];
 #pragma unroll
-      for (int nt = 0; nt < NTV; nt++) w[nt] = sT[(kk * NTV + nt) * 32 + lane];
+      for (int nt = 0; nt < NW; nt++) w[nt] = sT[(kk * NT + T0 + nt) * 32 + lane];
 #pragma unroll
-      for (int nt = 0; nt < NTV; nt++) mma16816_bf16(d[nt], lo, w[nt].x, w[nt].y);
+      for (int nt = 0; nt < NW; nt++) mma16816_bf16(d[nt], lo, w[nt].x, w[nt].y);
 #pragma unroll
-      for (int nt = 0; nt < NTV; nt++) mma16816_bf16(d[nt], md, w[nt].x, w[nt].y);
+      for (int nt = 0; nt < NW; nt++) mma16816_bf16(d[nt], md, w[nt].x, w[nt].y);
 #pragma unroll
-      for (int nt = 0; nt < NTV; nt++) mma16816_bf16(d[nt], hi, w[nt].x, w[nt].y);
+      for (int nt = 0; nt < NW; nt++) mma16816_bf16(d[nt], hi, w[nt].x, w[nt].y);
+    };
+    if constexpr (NW == 1) {
+      if (hf == 0) mix_step(0, sc[0], ot[0]);
+      else mix_step(0, ot[0], sc[0]);
+    } else {
+#pragma unroll
+      for (int k = 0; k < NW / 2; k++) mix_step(hf * (NW / 2) + k, sc[2 * k], sc[2 * k + 1]);
+#pragma unroll
+      for (int k = 0; k < NW / 2; k++) mix_step((hf ^ 1) * (NW / 2) + k, ot[2 * k], ot[2 * k + 1]);
     }
     const int t0 = (pa + i) * 16 + g4, t1 = t0 + 8;
     const bool in0 = t0 >= first && t0 < len, in1 = t1 >= first && t1 < len;
     const float f0 = (float)(len - 1 - t0), f1 = (float)(len - 1 - t1);
     bool grown = false;
 #pragma unroll
-    for (int nt = 0; nt < NTV; nt++)
+    for (int nt = 0; nt < NW; nt++)
 #pragma unroll
       for (int e = 0; e < 2; e++) {
         d[nt][e] = in0 ? fmaf(d[nt][e], kLog2e, -sl[nt][e] * f0) : -INFINITY;
@@ -313,7 +344,7 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
       }
     if (__any_sync(0xffffffffu, grown)) {
 #pragma unroll
-      for (int nt = 0; nt < NTV; nt++)
+      for (int nt = 0; nt < NW; nt++)
 #pragma unroll
         for (int e = 0; e < 2; e++) {
           float mx = fmaxf(d[nt][e], d[nt][e + 2]);
@@ -332,7 +363,7 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
         }
     }
 #pragma unroll
-    for (int nt = 0; nt < NTV; nt++) {
+    for (int nt = 0; nt < NW; nt++) {
       float p[4];
 #pragma unroll
       for (int e = 0; e < 2; e++) {
@@ -342,7 +373,7 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
         l[nt][e] += p[e] + p[e + 2];
       }
       const uint32_t w[2] = {transpose_8x8(pack_h2(p[0], p[1])), transpose_8x8(pack_h2(p[2], p[3]))};      // keys 0..7, 8..15 of head g4
-      const int tile = part * NTV + nt;
+      const int tile = T0 + nt;
       if (rp >= 8) {
         const uint32_t at = row_at(r8 + (mi >> 1) * 8, min(tile * 8 / rp, a.G - 1));
 #pragma unroll
@@ -369,26 +400,27 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
         }
       }
     }
-    __syncwarp();
-    if (lane == 0 && i + a.nslot < np) issue(i + a.nslot);
+    pair_barrier(pair);                                  // both are done with the page, and with each other's scores
+    if (lane == 0 && hf == 0 && i + a.nslot < np) issue(i + a.nslot, s_pid[i + a.nslot]);
   }
+  __syncthreads();                                      // every page has been read: the ring becomes the partial outputs
   if (tid == 0 && s_abort && a.status) atomicExch(a.status, (int)B200_ERR_TIMEOUT_TMA);
   if (s_abort) drain_after_abort();
-  __syncthreads();                                      // every page has been read: the ring becomes the partial outputs
+  __syncthreads();
 #pragma unroll
-  for (int nt = 0; nt < NTV; nt++)
+  for (int nt = 0; nt < NW; nt++)
 #pragma unroll
     for (int e = 0; e < 2; e++) {
       float v = l[nt][e];
       v += __shfl_xor_sync(0xffffffffu, v, 4);
       v += __shfl_xor_sync(0xffffffffu, v, 8);
       v += __shfl_xor_sync(0xffffffffu, v, 16);
-      const int slot = nt * 8 + 2 * t4 + e;
+      const int slot = (T0 + nt) * 8 + 2 * t4 + e;
       if (g4 == 0) {
-        s_ml[warp][slot][0] = mu[nt][e];
-        s_ml[warp][slot][1] = v;
+        s_ml[pair][slot][0] = mu[nt][e];
+        s_ml[pair][slot][1] = v;
       }
-      float* acc = s_acc + ((size_t)warp * NTV * 8 + slot) * DK;
+      float* acc = s_acc + ((size_t)pair * SLOTS + slot) * DK;
 #pragma unroll
       for (int m = 0; m < DK / 16; m++) {
         acc[m * 16 + g4] = o[nt][m][e];
@@ -396,37 +428,45 @@ __global__ void __launch_bounds__(256) mixed_decode_kernel(const __grid_constant
       }
     }
   __syncthreads();
-  const int n_slots = gridDim.y * NTV * 8, n_out = NTV * 8 * DK;
-  const size_t row = ((size_t)b * a.S + split) * n_slots + part * NTV * 8;
-  auto finish = [&](int slot, int e, float M, float L, float A) {
-    const int h = head_of(part * NTV * 8 + slot);
-    if (h < 0) return;
-    if (a.sinks) {
-      const float sk = a.sinks[h] * kLog2e, M2 = fmaxf(M, sk), c = M == -INFINITY ? 0.f : ex2_approx(M - M2);
-      L = L * c + ex2_approx(sk - M2);
-      A *= c;
-    }
-    const float v = L > 0.f ? A / L : 0.f;
-    const size_t at = ((size_t)b * a.H + h) * DK + e;
-    if (a.out_f32) a.out_f32[at] = v;
-    if (a.out_bf16) a.out_bf16[at] = __float2bfloat16(v);
-  };
-  for (int x = tid; x < n_out; x += blockDim.x) {
-    const int slot = x / DK, e = x % DK;
-    float M = -INFINITY, L = 0.f, A = 0.f;
-    for (int w = 0; w < nw; w++) M = fmaxf(M, s_ml[w][slot][0]);
-    for (int w = 0; w < nw; w++) {
-      const float c = s_ml[w][slot][0] == -INFINITY ? 0.f : ex2_approx(s_ml[w][slot][0] - M);
+  // the pairs' shares: each one's factor per head takes the place of its maximum
+  const size_t row = ((size_t)b * a.S + split) * SLOTS;
+  for (int slot = tid; slot < SLOTS; slot += blockDim.x) {
+    const int h = slot % rp < rep && slot < a.G * rp ? slot / rp * rep + slot % rp : -1;
+    float M = -INFINITY, L = 0.f;
+    for (int w = 0; w < pairs; w++) M = fmaxf(M, s_ml[w][slot][0]);
+    const bool last = a.S == 1;
+    const float sk = last && a.sinks && h >= 0 ? a.sinks[h] * kLog2e : -INFINITY, M2 = fmaxf(M, sk);
+    for (int w = 0; w < pairs; w++) {
+      const float c = s_ml[w][slot][0] == -INFINITY ? 0.f : ex2_approx(s_ml[w][slot][0] - M2);
       L += s_ml[w][slot][1] * c;
-      A += s_acc[((size_t)w * NTV * 8 + slot) * DK + e] * c;
+      s_ml[w][slot][0] = c;
     }
-    if (a.S == 1) {
-      finish(slot, e, M, L, A);
+    if (last) {
+      if (sk != -INFINITY) L += ex2_approx(sk - M2);
+      const float inv = L > 0.f ? 1.f / L : 0.f;
+      for (int w = 0; w < pairs; w++) s_ml[w][slot][0] *= inv;
     } else {
-      a.part_acc[(row + slot) * DK + e] = A;
-      if (e == 0) {
-        a.part_ml[(row + slot) * 2] = M;
-        a.part_ml[(row + slot) * 2 + 1] = L;
+      a.part_ml[(row + slot) * 2] = M;
+      a.part_ml[(row + slot) * 2 + 1] = L;
+    }
+  }
+  __syncthreads();
+  for (int x = tid; x < SLOTS * (DK / 4); x += blockDim.x) {
+    const int slot = x / (DK / 4), e = x % (DK / 4) * 4;
+    float4 A = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int w = 0; w < pairs; w++) {
+      const float4 v = *(const float4*)(s_acc + ((size_t)w * SLOTS + slot) * DK + e);
+      const float c = s_ml[w][slot][0];
+      A.x = fmaf(v.x, c, A.x); A.y = fmaf(v.y, c, A.y); A.z = fmaf(v.z, c, A.z); A.w = fmaf(v.w, c, A.w);
+    }
+    if (a.S > 1) {
+      *(float4*)(a.part_acc + (row + slot) * DK + e) = A;
+    } else if (slot < a.G * rp && slot % rp < rep) {
+      const size_t at = ((size_t)b * a.H + slot / rp * rep + slot % rp) * DK + e;
+      if (a.out_f32) *(float4*)(a.out_f32 + at) = A;
+      if (a.out_bf16) {
+        const __nv_bfloat162 p0 = __floats2bfloat162_rn(A.x, A.y), p1 = __floats2bfloat162_rn(A.z, A.w);
+        *(uint2*)(a.out_bf16 + at) = make_uint2(*(const uint32_t*)&p0, *(const uint32_t*)&p1);
       }
     }
   }
@@ -471,50 +511,56 @@ __global__ void __launch_bounds__(DK) mixed_merge_kernel(const float* __restrict
   if (out_bf16) out_bf16[at] = __float2bfloat16(v);
 }
 
-// Padded group size, tiles of eight padded heads (even), and tiles a CTA keeps the outputs of; false: sizes the kernel does not take.
-static bool mixed_decode_plan(int H, int G, int DK, int& rp, int& nt, int& ntv) {
+// Padded group size and tiles of eight padded heads (2, 4 or 8); false: sizes the kernel does not take.
+static bool mixed_decode_plan(int H, int G, int DK, int& rp, int& nt) {
   if (G < 1 || H < 1 || H % G || (DK != 64 && DK != 128)) return false;
   const int rep = H / G;
   rp = rep <= 1 ? 1 : rep <= 2 ? 2 : rep <= 4 ? 4 : (rep + 7) / 8 * 8;
   const int tiles = (G * rp + 7) / 8;
   nt = tiles <= 2 ? 2 : tiles <= 4 ? 4 : 8;
-  ntv = DK == 128 && nt == 8 ? 4 : nt;
   return tiles <= 8 && G * DK <= 1536;
 }
 B200_API int b200_mixed_decode_ok(int H, int G, int DK) {
-  int rp, nt, ntv;
-  return mixed_decode_plan(H, G, DK, rp, nt, ntv) ? 1 : 0;
+  int rp, nt;
+  return mixed_decode_plan(H, G, DK, rp, nt) ? 1 : 0;
 }
 B200_API size_t b200_mixed_decode_scratch_floats(int B, int H, int G, int DK, int S) {
-  int rp, nt, ntv;
-  if (!mixed_decode_plan(H, G, DK, rp, nt, ntv)) return 0;
-  return (size_t)B * S * nt * 8 * (DK + 2);
+  int rp, nt;
+  return mixed_decode_plan(H, G, DK, rp, nt) ? (size_t)B * S * nt * 8 * (DK + 2) : 0;
 }
-template <int DK, int NT, int NTV>
+// 32-bit words of what b200_mixed_decode_prepare writes.
+B200_API size_t b200_mixed_decode_prepared_words(int H, int G, int DK) {
+  int rp, nt;
+  return mixed_decode_plan(H, G, DK, rp, nt) ? (size_t)nt * nt * 32 + 8 * nt : 0;
+}
+// mix fp32 [H][H] (bf16 values), slopes [H] of the mixed scores (or null) -> the form the decode kernel reads.
+B200_API int b200_mixed_decode_prepare(const float* mix, const float* slopes, int H, int G, int DK, void* out, cudaStream_t st) {
+  int rp, nt;
+  if (!mix || !out || ((uintptr_t)out & 15) || !mixed_decode_plan(H, G, DK, rp, nt)) return B200_ERR_BAD_ARG;
+  mixed_prepare_kernel<<<1, 256, 0, st>>>(mix, slopes, H, G, rp, nt, (uint2*)out);
+  return (int)cudaGetLastError();
+}
+template <int DK, int NT, int THREADS>
 static int launch_mixed_decode(MixedDecArgs a, const void* kc, int n_pages, int B, float* scratch, cudaStream_t st) {
-  const int W = a.G * DK, page = 32 * W, parts = NT / NTV;
-  constexpr int kOut = NTV * 8 * DK * 4;
-  // two CTAs of four warps to an SM where half its shared memory holds enough pages, else one of up to eight
-  const size_t fixed = 1024 + 34 * 8 + (8 * NT + 2) * (DK + 8) * 2 + 16 + NT / 2 * NTV * 256 + ((size_t)a.max_pages + 1) * 4;
+  const int W = a.G * DK, page = 32 * W;
+  const size_t out = (size_t)NT * 8 * DK * 4;
+  const size_t fixed = 1024 + 20 * 8 + NT * NT * 128 + (8 * NT + 1) * (DK + 8) * 2 + ((size_t)a.max_pages + 4) * 4;
   if (fixed > 100 * 1024) return B200_ERR_BAD_ARG;
-  int nw = 0;
-  if (fixed + 8 * (size_t)page <= 106 * 1024 && fixed + 4 * (size_t)kOut <= 106 * 1024) {
-    nw = 4;
-    a.nslot = (106 * 1024 - fixed) / page >= 16 ? 16 : (int)((106 * 1024 - fixed) / page) / 4 * 4;
-  } else {
-    const size_t room = 220 * 1024 - fixed;
-    const int cap = (int)(room / page < 16 ? room / page : 16);
-    for (int w = 8; w >= 2; w--)
-      if (cap >= w && (size_t)w * kOut <= room && (!nw || cap / w * w > a.nslot)) {
-        nw = w;
-        a.nslot = cap / w * w;
-      }
-    if (!nw) return B200_ERR_BAD_ARG;
+  const size_t room = 222 * 1024 - fixed;               // (the rest of an SM's: this kernel's static part)
+  int pairs = 0;
+  for (int p = THREADS / 64; p >= 1 && (!pairs || p > THREADS / 128); p--) {      // the most pages in flight, of many warps
+    const size_t left = room - (size_t)p * NT * 512;
+    const int cap = (int)(left / page < 18 ? left / page : 18);
+    if (cap >= p && p * out <= left && (!pairs || cap / p * p > a.nslot)) {
+      pairs = p;
+      a.nslot = cap / p * p;
+    }
   }
+  if (!pairs) return B200_ERR_BAD_ARG;
   a.part_acc = scratch;
   a.part_ml = scratch ? scratch + (size_t)B * a.S * NT * 8 * DK : nullptr;
-  const size_t ring = (size_t)a.nslot * page > (size_t)nw * kOut ? (size_t)a.nslot * page : (size_t)nw * kOut, smem = fixed + ring;
-  auto kern = mixed_decode_kernel<DK, NT, NTV>;
+  const size_t ring = (size_t)a.nslot * page > pairs * out ? (size_t)a.nslot * page : pairs * out, smem = fixed + (size_t)pairs * NT * 512 + ring;
+  auto kern = mixed_decode_kernel<DK, NT, THREADS>;
   static size_t configured = 0;
   if (smem > configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -524,31 +570,31 @@ static int launch_mixed_decode(MixedDecArgs a, const void* kc, int n_pages, int 
   CUtensorMap tm;
   const int rc = make_tmap_rows8(&tm, kc, (uint64_t)n_pages * 16, W, W / 64);
   if (rc) return rc;
-  const int err = launch_pdl(kern, dim3(a.S, parts, B), dim3(32 * nw), smem, st, tm, a);
+  const int err = launch_pdl(kern, dim3(a.S, B), dim3(64 * pairs), smem, st, tm, a);
   if (err || a.S == 1) return err;
   return launch_pdl(mixed_merge_kernel<DK>, dim3(a.H, B), dim3(DK), 0, st, (const float*)a.part_acc, (const float*)a.part_ml, a.sinks, a.H, a.H / a.G, a.rp, NT * 8,
                     a.S, a.out_f32, a.out_bf16);
 }
-// q fp32 [B][H][DK], scaled; mix fp32 [H][H] (bf16 values); kc fp16 [n_pages][16][G * DK]; sizes as b200_mixed_decode_ok has them.  S: shares of the
-// keys, at most 64 (scratch where there are several).
-B200_API int b200_mixed_decode(const float* q, const void* kc, const float* mix, const float* slopes, const float* sinks, const int* page_table,
-                               int max_pages, int n_pages, const int* seq_lens, int B, int H, int G, int DK, int window, int S, float* out_f32,
-                               void* out_bf16, float* scratch, int* status, cudaStream_t st) {
+// q fp32 [B][H][DK], scaled; mix: prepared (above); kc fp16 [n_pages][16][G * DK]; sizes as b200_mixed_decode_ok has them.  S: shares of the keys, at
+// most 64 (scratch where there are several).
+B200_API int b200_mixed_decode(const float* q, const void* kc, const void* mix, const float* sinks, const int* page_table, int max_pages, int n_pages,
+                               const int* seq_lens, int B, int H, int G, int DK, int window, int S, float* out_f32, void* out_bf16, float* scratch,
+                               int* status, cudaStream_t st) {
   MixedDecArgs a = {};
-  int nt, ntv;
+  int nt;
   if (B < 1 || S < 1 || S > 64 || window < 0 || max_pages < 1 || !q || !kc || !mix || (!out_f32 && !out_bf16) || (S > 1 && !scratch) ||
-      !mixed_decode_plan(H, G, DK, a.rp, nt, ntv) || ((uintptr_t)q & 7))
+      !mixed_decode_plan(H, G, DK, a.rp, nt) || (((uintptr_t)q | (uintptr_t)mix) & 15))
     return B200_ERR_BAD_ARG;
-  a.q = q; a.mix = mix; a.slopes = slopes; a.sinks = sinks; a.page_table = page_table; a.seq_lens = seq_lens; a.max_pages = max_pages; a.H = H; a.G = G;
+  a.q = q; a.mix = (const uint2*)mix; a.sinks = sinks; a.page_table = page_table; a.seq_lens = seq_lens; a.max_pages = max_pages; a.H = H; a.G = G;
   a.window = window; a.S = S; a.out_f32 = out_f32; a.out_bf16 = (__nv_bfloat16*)out_bf16; a.status = status;
   if (DK == 64) {
-    if (nt == 2) return launch_mixed_decode<64, 2, 2>(a, kc, n_pages, B, scratch, st);
-    if (nt == 4) return launch_mixed_decode<64, 4, 4>(a, kc, n_pages, B, scratch, st);
-    return launch_mixed_decode<64, 8, 8>(a, kc, n_pages, B, scratch, st);
+    if (nt == 2) return launch_mixed_decode<64, 2, 384>(a, kc, n_pages, B, scratch, st);
+    if (nt == 4) return launch_mixed_decode<64, 4, 384>(a, kc, n_pages, B, scratch, st);
+    return launch_mixed_decode<64, 8, 384>(a, kc, n_pages, B, scratch, st);
   }
-  if (nt == 2) return launch_mixed_decode<128, 2, 2>(a, kc, n_pages, B, scratch, st);
-  if (nt == 4) return launch_mixed_decode<128, 4, 4>(a, kc, n_pages, B, scratch, st);
-  return launch_mixed_decode<128, 8, 4>(a, kc, n_pages, B, scratch, st);
+  if (nt == 2) return launch_mixed_decode<128, 2, 384>(a, kc, n_pages, B, scratch, st);
+  if (nt == 4) return launch_mixed_decode<128, 4, 384>(a, kc, n_pages, B, scratch, st);
+  return launch_mixed_decode<128, 8, 256>(a, kc, n_pages, B, scratch, st);
 }
 
 // ------------------------------------------------------------------ prompts: wide queries on the 5th-generation tensor cores

@@ -114,6 +114,7 @@ class _Block:
     act: torch.Tensor | None = None              # PolyNorm's four numbers
     moe: _Experts | None = None
     mix: torch.Tensor | None = None              # fp32 [heads][heads]
+    mix_dec: torch.Tensor | None = None          # mixture and slopes as the decode kernel reads them
     slopes: torch.Tensor | None = None           # what a step of distance takes off a score, per head (behind the mixture)
     silent: torch.Tensor | None = None           # zeros: the scores of the silent sinks
     out_bias: torch.Tensor | None = None         # times the layer scale: joins the residual ahead of the layer
@@ -315,6 +316,8 @@ class HybridEngine(PagedEngine):
         if m.distance_bias:
             slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / m.heads) for h in range(m.heads)], dtype=torch.float64, device=self.device)
             b.slopes = (slopes if b.mix is None else b.mix.double() @ slopes).float()
+        if b.dec:
+            b.mix_dec = ops.mixed_decode_prepare(b.mix, b.slopes, m.heads, m.kv_heads, b.DK)
         if m.silent_sink:
             b.silent = torch.zeros(m.heads, dtype=torch.float32, device=self.device)
         return b
@@ -550,7 +553,7 @@ class HybridEngine(PagedEngine):
             ops.qkv_finish(proj, 0, k_off, -1, self.pos, self.slot, None, 1.0, H, 1, m.dim, m.vdim, b.DK, b.DV, 0, 1, False, 0.0, m.scale, PAGE, q32=q, kc=kc,
                            maps=G, bias=b.bias)
             S = self._mixed_splits(T, min(pages, m.window // PAGE + 2) if m.window else pages)
-            ops.mixed_decode(q, kc, b.mix, b.slopes, self.page_table, self.seq_lens, T, H, G, b.DK, window=m.window, S=S, sinks=b.silent, out_f32=o32, out_bf16=o16,
+            ops.mixed_decode(q, kc, b.mix_dec, self.page_table, self.seq_lens, T, H, G, b.DK, window=m.window, S=S, sinks=b.silent, out_f32=o32, out_bf16=o16,
                              scratch=self.mixed_scratch, status=self.status)
             return 2 + (S > 1)
         tc = b.tc and not decode

@@ -54,7 +54,8 @@ _SIGS = {
     "b200_depth_norm": [_P, c_size_t, _P, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_float, _P, _P, _P, _P, _P, c_long, _P],
     "b200_poly_norm": [_P, c_int, c_int, c_int, _P, c_float, _P, _P, c_int, _P],
     "b200_mixed_finish": [_P] + [c_int] * 3 + [_P, _P, c_float, _P] + [c_int] * 5 + [_P, _P, _P, c_int, _P],
-    "b200_mixed_decode": [_P] * 6 + [c_int, c_int, _P] + [c_int] * 6 + [_P] * 5,
+    "b200_mixed_decode": [_P] * 5 + [c_int, c_int, _P] + [c_int] * 6 + [_P] * 5,
+    "b200_mixed_decode_prepare": [_P, _P, c_int, c_int, c_int, _P, _P],
     "b200_mixed_decode_ok": [c_int] * 3,
     "b200_mixed_prefill": [_P] * 5 + [c_int, _P, _P, _P] + [c_int] * 7 + [_P] * 4,
     "b200_mixed_prefill_ok": [c_int] * 2,
@@ -107,6 +108,8 @@ def lib():
         L.b200_latent_decode_scratch_floats.restype = c_size_t
         L.b200_mixed_decode_scratch_floats.argtypes = [c_int] * 5
         L.b200_mixed_decode_scratch_floats.restype = c_size_t
+        L.b200_mixed_decode_prepared_words.argtypes = [c_int] * 3
+        L.b200_mixed_decode_prepared_words.restype = c_size_t
         L.b200_gla_chunk_bytes.argtypes = [c_int] * 6
         L.b200_gla_chunk_bytes.restype = c_size_t
         _lib = L
@@ -489,10 +492,17 @@ def mixed_decode_scratch_floats(B, H, G, DK, S):
     return lib().b200_mixed_decode_scratch_floats(B, H, G, DK, S)
 
 
-def mixed_decode(q, kc, mix, slopes, page_table, seq_lens, B, H, G, DK, window=0, S=1, sinks=None, out_f32=None, out_bf16=None, scratch=None, status=None):
+def mixed_decode_prepare(mix, slopes, H, G, DK):
+    """The mixture (fp32 [H, H] of bf16 values) and the mixed scores' ``slopes`` [H] in the form :func:`mixed_decode` reads: once per layer, at load."""
+    out = torch.empty(lib().b200_mixed_decode_prepared_words(H, G, DK), dtype=torch.int32, device=mix.device)
+    _check(lib().b200_mixed_decode_prepare(_p(mix), _p(slopes), H, G, DK, _p(out), _st()), "mixed_decode_prepare")
+    return out
+
+
+def mixed_decode(q, kc, mix, page_table, seq_lens, B, H, G, DK, window=0, S=1, sinks=None, out_f32=None, out_bf16=None, scratch=None, status=None):
     """One query token per sequence, heads mixed on the scores (see ``mixed_attn.cu``): ``q`` fp32 [B, H, DK], scaled and not mixed; ``kc`` fp16 [pages, 1, 16,
-    G * DK], keys and values; ``slopes`` [H]: of the mixed scores.  ``S``: shares of the keys, at most 64."""
-    _check(lib().b200_mixed_decode(_p(q), _p(kc), _p(mix), _p(slopes), _p(sinks), _p(page_table), page_table.shape[1], kc.shape[0], _p(seq_lens), B, H, G, DK,
+    G * DK], keys and values; ``mix`` from :func:`mixed_decode_prepare`.  ``S``: shares of the keys, at most 64."""
+    _check(lib().b200_mixed_decode(_p(q), _p(kc), _p(mix), _p(sinks), _p(page_table), page_table.shape[1], kc.shape[0], _p(seq_lens), B, H, G, DK,
                                    window, S, _p(out_f32), _p(out_bf16), _p(scratch), _p(status), _st()), "mixed_decode")
 
 

@@ -223,7 +223,7 @@ def mixed(kernel, qs, ks, mix, scale, window, bias=None):
             q32, before = torch.full((T, H * DK), 7.0, device=DEV), kc.clone()
             ops.qkv_finish(row, 0, nq, -1, slot, slot, None, 1.0, H, 1, dim, dim, DK, DK, 0, 1, False, 0.0, scale, 16, q32=q32, kc=kc, maps=G, bias=bias.to(DEV))
             assert torch.equal(kc, before)               # the very rows the other finish writes
-            ops.mixed_decode(q32, kc, mix.to(DEV), slopes, tab, ctx, B, H, G, DK, S=S, out_f32=out, status=st, window=window, sinks=args["sinks"],
+            ops.mixed_decode(q32, kc, ops.mixed_decode_prepare(mix.to(DEV), slopes, H, G, DK), tab, ctx, B, H, G, DK, S=S, out_f32=out, status=st, window=window, sinks=args["sinks"],
                              scratch=torch.full((ops.mixed_decode_scratch_floats(B, H, G, DK, S),), float("nan"), device=DEV))
             assert S == 1 or (out.cpu() - first).abs().max() <= 2e-3 * first.abs().max()
             first = out.clone().cpu()
@@ -262,7 +262,7 @@ def test_attention_with_mixed_heads(kernel, tol, H, G, dim, window):
         tol = 1.2e-2                                    # every row sees one key: the same rounding everywhere
     shapes = [(1, 1), (1, 77), (1, 300), (1, 51), (1, 128), (1, 129)] if kernel == "decode" else [(1, 1), (3, 20), (64, 64), (130, 141), (1, 33), (200, 260)]
     qs, ks = [f(t, H, dim) for t, _ in shapes], [f(n, G, dim) for _, n in shapes]
-    mix = f(H, H) * 0.6 * H ** -0.5 + torch.eye(H)
+    mix = (f(H, H) * 0.6 * H ** -0.5 + torch.eye(H)).bfloat16().float()          # what a checkpoint holds
     scale = 1.3 * dim ** -0.5
     got = mixed(kernel, qs, ks, mix, scale, window, f(H * dim + G * dim))
     assert rel(got, want_mixed(qs, ks, mix, scale, window)) < tol
@@ -275,7 +275,7 @@ def test_a_window_starts_with_its_first_key(kernel, window):
     H, G, D = 4, 2, 64
     g = torch.Generator().manual_seed(3)
     qs, ks, inside = [], [], []
-    mix = torch.eye(H) + 0.1 * torch.randn(H, H, generator=g)
+    mix = (torch.eye(H) + 0.1 * torch.randn(H, H, generator=g)).bfloat16().float()
     for at in (0, 1, 15, 16, 63, 64, 127, 128, 130):
         for far in (window - 1, window):                # the query's distance from the key
             n = at + far + 1
