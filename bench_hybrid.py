@@ -309,11 +309,12 @@ def time_kazolorn_kernels(cfg, dev, reps: int = 12) -> list[dict]:
         bench(f"gemm output, residual [{n}]", lambda: ops.gemm_bf16(ao, wo, n, d, nq, out_f32=x, resid_f32=x, status=st), wo.numel() * 2 + n * (nq * 2 + d * 8), 2.0 * n * d * nq)
         if dense:
             F = dense.ffn
-            up, dn, gu, z, act, coef = bf(F, d), bf(d, F), bf(2 * F, d), rnd(n, F), bf(n, F), rnd(4)
-            bench(f"gemm up [{n}]", lambda: ops.gemm_bf16(a, up, n, F, d, out_f32=z, status=st), (F * d + n * d) * 2 + n * F * 4, 2.0 * n * F * d, like=f"gemm swiglu gate/up [{n}]")
+            zb = 4 if n <= 64 else 2                        # bytes of an activation on its way to PolyNorm
+            up, dn, gu, z, act, coef = bf(F, d), bf(d, F), bf(2 * F, d), rnd(n, F) if zb == 4 else bf(n, F), bf(n, F), rnd(4)
+            bench(f"gemm up [{n}]", lambda: ops.gemm_bf16(a, up, n, F, d, out_f32=z if zb == 4 else None, out_bf16=z if zb == 2 else None, status=st), (F * d + n * d) * 2 + n * F * zb, 2.0 * n * F * d, like=f"gemm swiglu gate/up [{n}]")
             bench(f"gemm swiglu gate/up [{n}]", lambda: ops.gemm_bf16(a, gu, n, 2 * F, d, out_bf16=act, ldc=F, act=ops.ACT_SWIGLU_PAIR, status=st), (2 * F * d + n * (d + F)) * 2,
                   4.0 * n * F * d)
-            bench(f"poly_norm [{n}]", lambda: ops.poly_norm(z, F, coef, 1e-6, act), n * F * 6, like=f"rmsnorm [{n}]")
+            bench(f"poly_norm [{n}]", lambda: ops.poly_norm(z, F, coef, 1e-6, act), n * F * (zb + 2), like=f"rmsnorm [{n}]")
             bench(f"gemm down, layer scale [{n}]", lambda: ops.gemm_bf16(act, dn, n, d, F, out_f32=x, accumulate=True, col_scale=ls, status=st), (F * d + n * F) * 2 + n * d * 8,
                   2.0 * n * F * d, like=f"gemm down, residual [{n}]")
             bench(f"gemm down, residual [{n}]", lambda: ops.gemm_bf16(act, dn, n, d, F, out_f32=x, resid_f32=x, status=st), (F * d + n * F) * 2 + n * d * 8, 2.0 * n * F * d)

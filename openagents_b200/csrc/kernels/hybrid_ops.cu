@@ -260,6 +260,8 @@ B200_API int b200_norm_dyt(float* x, int T, int D, const int* ids, const void* e
 // Per row:  x = sum over j < n of w[j] * X_j   (X_j: row t of xs + j * stride; the embedding output and every layer's result so far)
 //           out = x + add                     (the next layer adds its results to this row: `add` is a bias they carry, or null)
 //           h1 = x / rms(x) * g1, h2 = x / rms(x) * g2   (two norms of the same x; each given or not; bf16 or fp32)
+//           part_k = sum over j < n of pw[k][j] * X_j    (k < parts: what later layers will want of the same X_j, read once for all of them)
+// base (or null): a row added to x as it is, such a partial sum from an earlier call.
 // Rows are ld floats apart in xs, out and h, D of them live; the others are written as zeros.  zero: a buffer cleared on the side.
 struct DepthArgs {
   const float* xs;
@@ -277,7 +279,12 @@ struct DepthArgs {
   float* hf2;
   float4* zero;
   int nz4;
+  const float* base;       // [T][ld] or null
+  float* part;             // parts slabs of `stride` floats
+  const float* pw;         // [parts][ldw]
+  int parts, ldw;
 };
+constexpr int kDepthParts = 3;
 __global__ void __launch_bounds__(256) depth_norm_kernel(const DepthArgs a) {
   extern __shared__ float depth_row[];               // [D]
   __shared__ float red[32];
@@ -289,14 +296,25 @@ __global__ void __launch_bounds__(256) depth_norm_kernel(const DepthArgs a) {
   float ss = 0.f;
   for (int i = tid; i < a.ld; i += nt) {
     float v = 0.f;
+    float p[kDepthParts] = {};
     if (i < a.D) {
       const float* x = a.xs + at + i;
-      if (!a.w) v = *x;
+      if (a.base) v = a.base[at + i];
+      if (!a.w) v += *x;
       else
-        for (int j = 0; j < a.n; j++) v = fmaf(a.w[j], x[j * a.stride], v);
+        for (int j = 0; j < a.n; j++) {
+          const float e = x[j * a.stride];
+          v = fmaf(a.w[j], e, v);
+#pragma unroll
+          for (int k = 0; k < kDepthParts; k++)
+            if (k < a.parts) p[k] = fmaf(a.pw[k * a.ldw + j], e, p[k]);
+        }
       depth_row[i] = v;
       ss += v * v;
     }
+#pragma unroll
+    for (int k = 0; k < kDepthParts; k++)
+      if (k < a.parts) a.part[k * a.stride + at + i] = p[k];
     if (a.out) a.out[at + i] = i < a.D && a.add ? v + a.add[i] : v;
   }
   if (!a.g1 && !a.g2) return;
@@ -315,8 +333,14 @@ __global__ void __launch_bounds__(256) depth_norm_kernel(const DepthArgs a) {
     }
   }
 }
-// The same on 16-byte accesses with the row in registers (widths that are multiples of 4).
-template <int R>
+// The same on 16-byte accesses with the row in registers (widths that are multiples of 4).  PARTS: whether there are partial sums to make.
+__device__ __forceinline__ void fma4(float4& v, float w, const float4& e) {
+  v.x = fmaf(w, e.x, v.x);
+  v.y = fmaf(w, e.y, v.y);
+  v.z = fmaf(w, e.z, v.z);
+  v.w = fmaf(w, e.w, v.w);
+}
+template <int R, bool PARTS>
 __global__ void __launch_bounds__(256) depth_norm_vec_kernel(const DepthArgs a) {
   __shared__ float red[32];
   const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x, D4 = a.D >> 2, l4 = a.ld >> 2;
@@ -325,23 +349,33 @@ __global__ void __launch_bounds__(256) depth_norm_vec_kernel(const DepthArgs a) 
   pdl_wait();
   for (int i = blockIdx.x * nt + tid; i < a.nz4; i += gridDim.x * nt) a.zero[i] = z;
   const size_t at = (size_t)t * l4;
-  float4 v[R];
+  float4 v[R], p[PARTS ? kDepthParts : 1][R];
 #pragma unroll
-  for (int k = 0; k < R; k++) v[k] = z;
+  for (int k = 0; k < R; k++) v[k] = a.base && tid + k * nt < D4 ? ((const float4*)a.base)[at + tid + k * nt] : z;
+  if constexpr (PARTS) {
+#pragma unroll
+    for (int m = 0; m < kDepthParts; m++)
+#pragma unroll
+      for (int k = 0; k < R; k++) p[m][k] = z;
+  }
   const float4* x = (const float4*)a.xs + at;
   const size_t s4 = a.stride >> 2;
   if (!a.w) {
 #pragma unroll
     for (int k = 0; k < R; k++)
-      if (tid + k * nt < D4) v[k] = x[tid + k * nt];
+      if (tid + k * nt < D4) fma4(v[k], 1.f, x[tid + k * nt]);
   } else {
-    constexpr int U = R >= 4 ? 2 : 8 / R;             // layers in flight
+    constexpr int U = R >= 8 ? 1 : R >= 4 ? 2 : 8 / R;            // layers in flight
     for (int j0 = 0; j0 < a.n; j0 += U) {
       float4 e[U][R];
-      float w[U];
+      float w[U], pw[PARTS ? kDepthParts : 1][U];
 #pragma unroll
       for (int u = 0; u < U; u++) {
         w[u] = j0 + u < a.n ? a.w[j0 + u] : 0.f;
+        if constexpr (PARTS) {
+#pragma unroll
+          for (int m = 0; m < kDepthParts; m++) pw[m][u] = m < a.parts && j0 + u < a.n ? a.pw[m * a.ldw + j0 + u] : 0.f;
+        }
 #pragma unroll
         for (int k = 0; k < R; k++) e[u][k] = j0 + u < a.n && tid + k * nt < D4 ? x[(j0 + u) * s4 + tid + k * nt] : z;
       }
@@ -349,12 +383,20 @@ __global__ void __launch_bounds__(256) depth_norm_vec_kernel(const DepthArgs a) 
       for (int u = 0; u < U; u++)
 #pragma unroll
         for (int k = 0; k < R; k++) {
-          v[k].x = fmaf(w[u], e[u][k].x, v[k].x);
-          v[k].y = fmaf(w[u], e[u][k].y, v[k].y);
-          v[k].z = fmaf(w[u], e[u][k].z, v[k].z);
-          v[k].w = fmaf(w[u], e[u][k].w, v[k].w);
+          fma4(v[k], w[u], e[u][k]);
+          if constexpr (PARTS) {
+#pragma unroll
+            for (int m = 0; m < kDepthParts; m++) fma4(p[m][k], pw[m][u], e[u][k]);
+          }
         }
     }
+  }
+  if constexpr (PARTS) {
+#pragma unroll
+    for (int m = 0; m < kDepthParts; m++)
+#pragma unroll
+      for (int k = 0; k < R; k++)
+        if (m < a.parts && tid + k * nt < l4) ((float4*)a.part)[m * s4 + at + tid + k * nt] = p[m][k];
   }
   float ss = 0.f;
 #pragma unroll
@@ -385,20 +427,24 @@ __global__ void __launch_bounds__(256) depth_norm_vec_kernel(const DepthArgs a) 
   if (a.g1) put(a.g1, a.hb1, a.hf1);
   if (a.g2) put(a.g2, a.hb2, a.hf2);
 }
-// xs fp32: n slabs `stride` floats apart, rows ld apart.  Outputs share ld.
+// xs fp32: n slabs `stride` floats apart, rows ld apart.  Outputs share ld; part: `parts` (at most 3) slabs as far apart.
 B200_API int b200_depth_norm(const float* xs, size_t stride, const float* w, int n, int T, int D, int ld, float* out, const float* add,
                              const float* g1, const float* g2, float eps, void* hb1, void* hb2, float* hf1, float* hf2, float* zero,
-                             long zero_n, cudaStream_t st) {
+                             long zero_n, const float* base, float* part, const float* pw, int parts, int ldw, cudaStream_t st) {
+  if (parts < 0 || parts > kDepthParts || (parts && (!part || !pw || !w || ldw < n))) return B200_ERR_BAD_ARG;
   if (T < 1 || D < 1 || ld < D || n < 1 || !xs || (!w && n != 1) || (g1 && !hb1 && !hf1) || (g2 && !hb2 && !hf2)) return B200_ERR_BAD_ARG;
   if (zero && (zero_n % 4 || (uintptr_t)zero % 16)) return B200_ERR_BAD_ARG;
   DepthArgs a;
   a.xs = xs; a.stride = stride; a.w = w; a.n = n; a.D = D; a.ld = ld; a.out = out; a.add = add; a.g1 = g1; a.g2 = g2; a.eps = eps;
   a.hb1 = (__nv_bfloat16*)hb1; a.hb2 = (__nv_bfloat16*)hb2; a.hf1 = hf1; a.hf2 = hf2; a.zero = (float4*)zero; a.nz4 = zero ? (int)(zero_n / 4) : 0;
+  a.base = base; a.part = part; a.pw = pw; a.parts = parts; a.ldw = ldw;
   const uintptr_t align = (uintptr_t)xs | (uintptr_t)out | (uintptr_t)add | (uintptr_t)g1 | (uintptr_t)g2 | (uintptr_t)hb1 | (uintptr_t)hb2 |
-                          (uintptr_t)hf1 | (uintptr_t)hf2;
+                          (uintptr_t)hf1 | (uintptr_t)hf2 | (uintptr_t)base | (uintptr_t)part;
   if (align % 16 == 0 && D % 4 == 0 && ld % 4 == 0 && stride % 4 == 0 && ld <= 256 * 4 * 8) {
     const int n4 = ld / 4, nt = n4 > 128 ? 256 : n4 > 64 ? 128 : 64, R = (n4 + nt - 1) / nt;
-    auto kern = R <= 1 ? depth_norm_vec_kernel<1> : R <= 2 ? depth_norm_vec_kernel<2> : R <= 4 ? depth_norm_vec_kernel<4> : depth_norm_vec_kernel<8>;
+    auto kern = R <= 1 ? depth_norm_vec_kernel<1, false> : R <= 2 ? depth_norm_vec_kernel<2, false> : R <= 4 ? depth_norm_vec_kernel<4, false> : depth_norm_vec_kernel<8, false>;
+    if (parts)
+      kern = R <= 1 ? depth_norm_vec_kernel<1, true> : R <= 2 ? depth_norm_vec_kernel<2, true> : R <= 4 ? depth_norm_vec_kernel<4, true> : depth_norm_vec_kernel<8, true>;
     return launch_pdl(kern, dim3(T), dim3(nt), 0, st, a);
   }
   const size_t smem = (size_t)D * 4;
@@ -415,16 +461,26 @@ B200_API int b200_depth_norm(const float* xs, size_t stride, const float* w, int
 // ------------------------------------------------------------------ PolyNorm
 
 // Per row of F values z:  a N(z) + b N(z^2) + c N(z^3) + e, N dividing a row by its root mean square (powers element by element), with
-// coef = (a, b, c, e).  in fp32 [T][ldi]; out bf16 or fp32 [T][ldo], columns F..ldo zero.
+// coef = (a, b, c, e).  in fp32 or bf16 [T][ldi]; out bf16 or fp32 [T][ldo], columns F..ldo zero.
 constexpr int kPolyRegs = 8;
-__global__ void __launch_bounds__(512) poly_norm_kernel(const float* __restrict__ in, int ldi, int F, const float* __restrict__ coef, float eps,
+__device__ __forceinline__ float4 get4(const float* p, int i) { return ((const float4*)p)[i]; }
+__device__ __forceinline__ float4 get4(const __nv_bfloat16* p, int i) {
+  const uint2 v = ((const uint2*)p)[i];
+  const float2 x = __bfloat1622float2(*(const __nv_bfloat162*)&v.x), y = __bfloat1622float2(*(const __nv_bfloat162*)&v.y);
+  return make_float4(x.x, x.y, y.x, y.y);
+}
+__device__ __forceinline__ float get1(const float* p, int i) { return p[i]; }
+__device__ __forceinline__ float get1(const __nv_bfloat16* p, int i) { return __bfloat162float(p[i]); }
+
+template <typename IT>
+__global__ void __launch_bounds__(512) poly_norm_kernel(const IT* __restrict__ in, int ldi, int F, const float* __restrict__ coef, float eps,
                                                         __nv_bfloat16* __restrict__ ob, float* __restrict__ of, int ldo, int vec) {
   __shared__ float red[3][32];
   const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
   const float ca = coef[0], cb = coef[1], cc = coef[2], ce = coef[3];
   pdl_trigger();
   pdl_wait();
-  const float* zr = in + (size_t)t * ldi;
+  const IT* zr = in + (size_t)t * ldi;
   const int F4 = F >> 2;
   float s2 = 0.f, s4 = 0.f, s6 = 0.f;
   auto stat = [&](float z) {
@@ -438,16 +494,16 @@ __global__ void __launch_bounds__(512) poly_norm_kernel(const float* __restrict_
 #pragma unroll
     for (int k = 0; k < kPolyRegs; k++) {
       const int i = tid + k * nt;
-      v[k] = i < F4 ? ((const float4*)zr)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+      v[k] = i < F4 ? get4(zr, i) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
 #pragma unroll
     for (int k = 0; k < kPolyRegs; k++) { stat(v[k].x); stat(v[k].y); stat(v[k].z); stat(v[k].w); }
     for (int i = tid + kPolyRegs * nt; i < F4; i += nt) {
-      const float4 e = ((const float4*)zr)[i];
+      const float4 e = get4(zr, i);
       stat(e.x); stat(e.y); stat(e.z); stat(e.w);
     }
   } else {
-    for (int i = tid; i < F; i += nt) stat(zr[i]);
+    for (int i = tid; i < F; i += nt) stat(get1(zr, i));
   }
   const int lane = tid & 31, w = tid >> 5, nw = nt >> 5;
   s2 = warp_sum(s2); s4 = warp_sum(s4); s6 = warp_sum(s6);
@@ -470,19 +526,22 @@ __global__ void __launch_bounds__(512) poly_norm_kernel(const float* __restrict_
 #pragma unroll
     for (int k = 0; k < kPolyRegs; k++)
       if (tid + k * nt < F4) store(tid + k * nt, v[k]);
-    for (int i = tid + kPolyRegs * nt; i < F4; i += nt) store(i, ((const float4*)zr)[i]);
+    for (int i = tid + kPolyRegs * nt; i < F4; i += nt) store(i, get4(zr, i));
   }
   for (int i = (vec ? F : 0) + tid; i < ldo; i += nt) {
-    const float o = i < F ? f(zr[i]) : 0.f;
+    const float o = i < F ? f(get1(zr, i)) : 0.f;
     if (ob) ob[(size_t)t * ldo + i] = __float2bfloat16(o);
     if (of) of[(size_t)t * ldo + i] = o;
   }
 }
-B200_API int b200_poly_norm(const float* in, int ldi, int T, int F, const float* coef, float eps, void* ob, float* of, int ldo, cudaStream_t st) {
-  if (T < 1 || F < 1 || ldi < F || ldo < F || !in || !coef || (!ob && !of) || of == in) return B200_ERR_BAD_ARG;
+B200_API int b200_poly_norm(const void* in, int in_bf16, int ldi, int T, int F, const float* coef, float eps, void* ob, float* of, int ldo,
+                            cudaStream_t st) {
+  if (T < 1 || F < 1 || ldi < F || ldo < F || !in || !coef || (!ob && !of) || of == in || ob == in) return B200_ERR_BAD_ARG;
   const int vec = F % 4 == 0 && ldi % 4 == 0 && ldo % 4 == 0 && (((uintptr_t)in | (uintptr_t)ob | (uintptr_t)of) & 15) == 0;
   const int threads = F >= 4096 ? 512 : F >= 1024 ? 256 : 128;
-  return launch_pdl(poly_norm_kernel, dim3(T), dim3(threads), 0, st, in, ldi, F, coef, eps, (__nv_bfloat16*)ob, of, ldo, vec);
+  if (in_bf16)
+    return launch_pdl(poly_norm_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, st, (const __nv_bfloat16*)in, ldi, F, coef, eps, (__nv_bfloat16*)ob, of, ldo, vec);
+  return launch_pdl(poly_norm_kernel<float>, dim3(T), dim3(threads), 0, st, (const float*)in, ldi, F, coef, eps, (__nv_bfloat16*)ob, of, ldo, vec);
 }
 
 // ------------------------------------------------------------------ attention: finish of the projections

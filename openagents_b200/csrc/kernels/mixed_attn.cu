@@ -49,33 +49,56 @@ __device__ __forceinline__ void put8(__half* p, const float (&v)[8]) {
   *(uint4*)p = o;
 }
 // One block per token.  A thread keeps eight columns of one group's queries (REP of them; REP = 0: any number, read again for every head) and
-// walks the heads: REP multiply-adds per result, results leave as whole rows.
-template <int REP, typename CT>
+// walks the heads: REP multiply-adds per result, results leave as whole rows.  VEC: rows, heads and bias come in 16-byte pieces.
+template <int REP, bool VEC, typename CT>
 __global__ void __launch_bounds__(256) mixed_finish_kernel(const MixedArgs a, CT* __restrict__ kc) {
   extern __shared__ __align__(16) float sT[];       // [H][H]
-  pdl_trigger();
-  pdl_wait();
   const int t = blockIdx.x, tid = threadIdx.x, rep = REP ? REP : a.H / a.G;
   for (int i = tid; i < a.H * a.H; i += 256) sT[i] = a.mix[i];
-  __syncthreads();
+  pdl_trigger();
+  pdl_wait();
   const float* row = a.in + (size_t)t * a.ld;
   const int n8 = a.G * a.DK >> 3, d8 = a.DK >> 3;   // pieces of eight columns of a cache row, of one head
   const int shares = max(1, 256 / n8), per = (a.H + shares - 1) / shares;
   auto fetch = [&](int col, int d, float (&v)[8]) {
+    if constexpr (VEC) {
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
+      if (d < a.dim) {
+        x = *(const float4*)(row + col + d);
+        y = *(const float4*)(row + col + d + 4);
+        if (a.bias) {
+          const float4 p = *(const float4*)(a.bias + col + d), q = *(const float4*)(a.bias + col + d + 4);
+          x.x += p.x; x.y += p.y; x.z += p.z; x.w += p.w;
+          y.x += q.x; y.y += q.y; y.z += q.z; y.w += q.w;
+        }
+      }
+      v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+    } else {
 #pragma unroll
-    for (int i = 0; i < 8; i++) v[i] = d + i < a.dim ? row[col + d + i] + (a.bias ? a.bias[col + d + i] : 0.f) : 0.f;
+      for (int i = 0; i < 8; i++) v[i] = d + i < a.dim ? row[col + d + i] + (a.bias ? a.bias[col + d + i] : 0.f) : 0.f;
+    }
   };
-  for (int it = tid; it < n8 * shares; it += 256) {
-    const int p = it % n8, c = p / d8, d = (p % d8) << 3, h0 = it / n8 * per, h1 = min(a.H, h0 + per);
+  const int s = a.slot[t];
+  if (s >= 0)
+    for (int p = tid; p < n8; p += 256) {
+      float v[8];
+      fetch(a.k_off + p / d8 * a.dim, (p % d8) << 3, v);
+      put8(kc + ((size_t)(s / a.page_size) * a.page_size + s % a.page_size) * n8 * 8 + p * 8, v);
+    }
+  for (int it = tid; it < n8 * shares || it == tid; it += 256) {
+    const bool live = it < n8 * shares;
+    const int p = it % n8, c = p / d8, d = (p % d8) << 3, h0 = it / n8 * per, h1 = live ? min(a.H, h0 + per) : 0;
     float q[REP ? REP : 1][8];
     if constexpr (REP > 0) {
+      if (live)
 #pragma unroll
-      for (int r = 0; r < REP; r++) {
-        fetch((c * REP + r) * a.dim, d, q[r]);
+        for (int r = 0; r < REP; r++) {
+          fetch((c * REP + r) * a.dim, d, q[r]);
 #pragma unroll
-        for (int i = 0; i < 8; i++) q[r][i] *= a.q_scale;
-      }
+          for (int i = 0; i < 8; i++) q[r][i] *= a.q_scale;
+        }
     }
+    if (it == tid) __syncthreads();                 // sT; every thread comes here once, its first queries on their way
     for (int h = h0; h < h1; h++) {
       const float* m = sT + h * a.H + c * rep;
       float o[8];
@@ -98,23 +121,16 @@ __global__ void __launch_bounds__(256) mixed_finish_kernel(const MixedArgs a, CT
       if (a.q16) put8(a.q16 + at, o);
     }
   }
-  const int s = a.slot[t];
-  if (s < 0) return;
-  for (int p = tid; p < n8; p += 256) {
-    float v[8];
-    fetch(a.k_off + p / d8 * a.dim, (p % d8) << 3, v);
-    put8(kc + ((size_t)(s / a.page_size) * a.page_size + s % a.page_size) * n8 * 8 + p * 8, v);
-  }
 }
-template <typename CT>
+template <bool VEC, typename CT>
 static int launch_mixed_finish(int T, const MixedArgs& a, CT* kc, cudaStream_t st) {
   const size_t smem = (size_t)a.H * a.H * 4;
-  auto kern = mixed_finish_kernel<0, CT>;
+  auto kern = mixed_finish_kernel<0, VEC, CT>;
   switch (a.H / a.G) {
-    case 1: kern = mixed_finish_kernel<1, CT>; break;
-    case 2: kern = mixed_finish_kernel<2, CT>; break;
-    case 4: kern = mixed_finish_kernel<4, CT>; break;
-    case 8: kern = mixed_finish_kernel<8, CT>; break;
+    case 1: kern = mixed_finish_kernel<1, VEC, CT>; break;
+    case 2: kern = mixed_finish_kernel<2, VEC, CT>; break;
+    case 4: kern = mixed_finish_kernel<4, VEC, CT>; break;
+    case 8: kern = mixed_finish_kernel<8, VEC, CT>; break;
   }
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -131,7 +147,9 @@ B200_API int b200_mixed_finish(const float* in, int ld, int T, int k_off, const 
   MixedArgs a;
   a.in = in; a.ld = ld; a.k_off = k_off; a.bias = bias; a.mix = mix; a.q_scale = q_scale; a.slot = slot; a.H = H; a.G = G; a.dim = dim; a.DK = DK;
   a.page_size = page_size; a.q32 = q32; a.q16 = (__half*)q16;
-  return cache_f32 ? launch_mixed_finish(T, a, (float*)kc, st) : launch_mixed_finish(T, a, (__half*)kc, st);
+  const bool vec = ((ld | k_off | dim) & 7) == 0 && (((uintptr_t)in | (uintptr_t)bias) & 15) == 0;
+  if (vec) return cache_f32 ? launch_mixed_finish<true>(T, a, (float*)kc, st) : launch_mixed_finish<true>(T, a, (__half*)kc, st);
+  return cache_f32 ? launch_mixed_finish<false>(T, a, (float*)kc, st) : launch_mixed_finish<false>(T, a, (__half*)kc, st);
 }
 
 // ------------------------------------------------------------------ decoding: one query token per sequence
@@ -867,13 +885,14 @@ __global__ void __launch_bounds__(384, 1) mixed_prefill_kernel(const __grid_cons
       tc_fence_after();
       float sv[HK];
       {
-        uint32_t r[32];
+        uint32_t r0[32], r1[32];
+        tmem_ld32(S_T + b * KEYS + lane_addr + hsel * HK, r0);
+        tmem_ld32(S_T + b * KEYS + lane_addr + hsel * HK + 32, r1);
+        tmem_ld_wait();
 #pragma unroll
-        for (int c = 0; c < HK / 32; c++) {
-          tmem_ld32(S_T + b * KEYS + lane_addr + hsel * HK + c * 32, r);
-          tmem_ld_wait();
-#pragma unroll
-          for (int i = 0; i < 32; i++) sv[c * 32 + i] = fmaf(slope, (float)(c * 32 + i), __uint_as_float(r[i]));
+        for (int i = 0; i < 32; i++) {
+          sv[i] = fmaf(slope, (float)i, __uint_as_float(r0[i]));
+          sv[32 + i] = fmaf(slope, (float)(32 + i), __uint_as_float(r1[i]));
         }
       }
       tc_fence_before();

@@ -30,6 +30,7 @@ from .qweight import WeightSource
 
 MIXED_CTAS = 592             # most CTAs of a mixed-head decode launch that splits the keys
 LATENT_CTAS = 592            # most CTAs of a latent decode launch that splits the keys
+DEPTH_GROUP = 4              # depth averages that share one reading of the results so far
 MOE_EXPERTS, MOE_TOP = 256, 32   # most experts of a layer, and of a token
 SHORT_TOKENS = 16            # latent attention: entries of up to this many new tokens work in the latent space
 ALONE = ("polynorm", "swiglu")   # activations that are no epilogue of the up projection
@@ -459,6 +460,12 @@ class HybridEngine(PagedEngine):
         if self.cfg.depth_average:
             # the embedding output, every layer's result (the row a layer adds into becomes one), and what goes on to the head
             self.hist = ws("hist", (len(self.runs) + 1, T, d), f32, zero=True)
+            self.parts = ws("parts", (DEPTH_GROUP - 1, T, d), f32)
+            # row i: the weights of what layer run i reads (the first reads the embedding output itself), as many as there can be
+            self.averages = torch.zeros((len(self.runs) + 1, len(self.runs) + 1), dtype=f32, device=dev)
+            self.averages[0, 0] = 1.0
+            for i, r in enumerate(self.runs):
+                self.averages[i + 1, : i + 2] = r.block.average
             self.hf2, self.hb2 = ws("hf2", (small * d,), f32), ws("hb2", (big * d,), bf)
             self.z = ws("z", (T * n_ffn,), f32, zero=True)
         moe = [(b.spec.moe, b.moe) for b in self.blocks if b.moe is not None]
@@ -739,32 +746,41 @@ class HybridEngine(PagedEngine):
 
     def _walk_parallel(self, T: int, decode: bool, f32: bool, step) -> int:
         """Mixer and feed-forward of a layer read the same residual row and add into a copy of it, which then is the layer's result; the depth average over
-        the results so far makes the next layer's row, and its two norms, in one pass."""
+        the results so far makes the next layer's row, and its two norms, in one pass.  Every DEPTH_GROUP-th average reads all results, and sums up what the
+        averages behind it want of them; those then read that sum and the results since."""
         eps, D = self.cfg.norm_eps, self.d
         h, _, views = self._buffers(T, f32)
         h2 = (self.hf2 if f32 else self.hb2)[: T * self.dp].view(T, self.dp)
         add = not f32 and T <= QGEMM_MAX_TOKENS
-        n, weights = 0, None
+        n = 0
+
+        def average(i: int, **kw):
+            """The row that layer run ``i`` reads (behind the last one: the head)."""
+            lead = i - i % DEPTH_GROUP
+            if i > lead:
+                ops.depth_norm(self.hist[lead + 1: i + 1, :T], D, eps, weights=self.averages[i, lead + 1:], base=self.parts[i - lead - 1, :T], **kw)
+                return
+            ahead = min(DEPTH_GROUP - 1, len(self.runs) - i)
+            ops.depth_norm(self.hist[: i + 1, :T], D, eps, weights=self.averages[i], parts=self.parts[:ahead, :T] if ahead else None,
+                           part_weights=self.averages[i + 1: i + 1 + ahead] if ahead else None, **kw)
         for i, r in enumerate(self.runs):
             b = r.block
             proj, mix, act = views(b)
             out = self.hist[i + 1, :T]
             ff = b.norm2 is not None
-            ops.depth_norm(self.hist[: i + 1, :T], D, eps, weights=weights, out=out, add=b.out_bias, g1=b.norm1.w, h1=h, g2=b.norm2.w if ff else None,
-                           h2=h2 if ff else None, zero=proj if add else None)
+            average(i, out=out, add=b.out_bias, g1=b.norm1.w, h1=h, g2=b.norm2.w if ff else None, h2=h2 if ff else None, zero=proj if add else None)
             self._mm(h, b.proj, proj, add=add)
             n += self._mix(r, proj, mix, T, f32, step) + 3
             self._mm(mix, b.out, out, into=1.0, scale=b.ls1)
             if b.moe is not None:
                 n += self._experts(b, h2, out, i)
             elif ff:
-                z = self.z[: T * b.up.N].view(T, -1)
+                z = self.z[: T * b.up.N].view(T, -1) if f32 or add else self.z.view(torch.bfloat16)[: T * b.up.N].view(T, -1)
                 self._mm(h2, b.up, z)
                 ops.poly_norm(z, b.spec.ffn, b.act, eps, act)
                 self._mm(act, b.down, out, into=1.0, scale=b.ls2)
                 n += 3
-            weights = b.average
-        ops.depth_norm(self.hist[: len(self.runs) + 1, :T], D, weights=weights, out=self.x[:T])
+        average(len(self.runs), out=self.x[:T])
         self._tail = None
         return n + 1
 

@@ -51,8 +51,8 @@ _SIGS = {
                                 _P, _P, c_int, _P, _P, _P],
     "b200_expert_gate_up": [_P, c_int, c_int, _P, c_int, _P, _P, c_int, _P, _P],
     "b200_expert_down": [_P, c_int, c_int, _P, c_int, _P, c_int, _P, _P, c_int, _P],
-    "b200_depth_norm": [_P, c_size_t, _P, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_float, _P, _P, _P, _P, _P, c_long, _P],
-    "b200_poly_norm": [_P, c_int, c_int, c_int, _P, c_float, _P, _P, c_int, _P],
+    "b200_depth_norm": [_P, c_size_t, _P, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_float, _P, _P, _P, _P, _P, c_long, _P, _P, _P, c_int, c_int, _P],
+    "b200_poly_norm": [_P, c_int, c_int, c_int, c_int, _P, c_float, _P, _P, c_int, _P],
     "b200_mixed_finish": [_P] + [c_int] * 3 + [_P, _P, c_float, _P] + [c_int] * 5 + [_P, _P, _P, c_int, _P],
     "b200_mixed_decode": [_P] * 5 + [c_int, c_int, _P] + [c_int] * 6 + [_P] * 5,
     "b200_mixed_decode_prepare": [_P, _P, c_int, c_int, c_int, _P, _P],
@@ -453,21 +453,26 @@ def head_matvec(A, W, out, heads, head_k, head_ldc, alpha=1.0, gate=None):
                                   _p(gate), 0 if gate is None else gate.stride(0), head_k, head_ldc, _st()), "head_matvec")
 
 
-def depth_norm(xs, D, eps=0.0, weights=None, out=None, add=None, g1=None, g2=None, h1=None, h2=None, zero=None):
+def depth_norm(xs, D, eps=0.0, weights=None, out=None, add=None, g1=None, g2=None, h1=None, h2=None, zero=None, base=None, parts=None,
+               part_weights=None):
     """``x = sum_j weights[j] * xs[j]`` over the slabs of ``xs`` (fp32 [n, >= T, ld], D columns live; a slice along the rows is fine; ``weights`` None: one
-    slab as it is); ``out`` [T, ld] = x + ``add``; ``h1`` / ``h2`` (both bf16 or fp32, [T, ld]) = x over its root mean square, times ``g1`` / ``g2``."""
+    slab as it is); ``out`` [T, ld] = x + ``add``; ``h1`` / ``h2`` (both bf16 or fp32, [T, ld]) = x over its root mean square, times ``g1`` / ``g2``.
+    ``base`` [T, ld] is added to x; ``parts`` [k, T, ld] (at most 3, slabs as far apart as those of ``xs``) take other weighted sums of the same slabs,
+    ``part_weights`` [k, >= n]."""
     n, T, ld = xs.shape
     f32 = next((h.dtype == torch.float32 for h in (h1, h2) if h is not None), False)
     b, f = (lambda h: None if f32 else _p(h)), (lambda h: _p(h) if f32 else None)                   # noqa: E731
     _check(lib().b200_depth_norm(_p(xs), xs.stride(0), _p(weights), n, T, D, ld, _p(out), _p(add), _p(g1), _p(g2), eps, b(h1), b(h2), f(h1), f(h2),
-                                 _p(zero), 0 if zero is None else zero.numel(), _st()), "depth_norm")
+                                 _p(zero), 0 if zero is None else zero.numel(), _p(base), _p(parts), _p(part_weights), 0 if parts is None else parts.shape[0],
+                                 0 if parts is None else part_weights.stride(0), _st()), "depth_norm")
+    assert parts is None or parts.stride(0) == xs.stride(0)
 
 
 def poly_norm(z, F, coef, eps, out):
-    """``a N(z) + b N(z^2) + c N(z^3) + e`` per row of ``z`` (fp32 [T, >= F]), N dividing by the root mean square, ``coef`` = (a, b, c, e); ``out`` bf16 or fp32,
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` per row of ``z`` (fp32 or bf16 [T, >= F]), N dividing by the root mean square, ``coef`` = (a, b, c, e); ``out`` bf16 or fp32,
     columns beyond F zero."""
     f32 = out.dtype == torch.float32
-    _check(lib().b200_poly_norm(_p(z), z.stride(0), z.shape[0], F, _p(coef), eps, None if f32 else _p(out), _p(out) if f32 else None, out.stride(0), _st()),
+    _check(lib().b200_poly_norm(_p(z), int(z.dtype == torch.bfloat16), z.stride(0), z.shape[0], F, _p(coef), eps, None if f32 else _p(out), _p(out) if f32 else None, out.stride(0), _st()),
            "poly_norm")
 
 

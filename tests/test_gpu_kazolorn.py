@@ -54,6 +54,17 @@ def test_depth_average_and_the_norms_behind_it(T, D, ld, n):
         for h, gain in ((h1, g1), (h2, g2)):
             assert rel(h[:, :D].float(), R.rms_norm(x, gain[:D].double(), 1e-4)) < tol and not h[:, D:].any()
         assert torch.equal(d[:n].cpu(), xs[:n])
+    for k in (1, 2, 3):                                # sums that later averages start from, and an average that does
+        slabs, pw = torch.full((n + 4, T, ld), 7.0, device=DEV), torch.randn(k, n + 2, generator=g)
+        slabs[:n] = xs[:n, :T].to(DEV)
+        out = torch.empty(T, ld, device=DEV)
+        ops.depth_norm(slabs[:n], D, weights=w.to(DEV), out=out, parts=slabs[n: n + k], part_weights=pw.to(DEV))
+        assert rel(out[:, :D], x) < 2e-6 and (slabs[n + k:] == 7.0).all()
+        for m in range(k):
+            want = R.depth_average([s[:T, :D].double() for s in xs[:n]], pw[m, :n].double())
+            assert rel(slabs[n + m, :, :D], want) < 2e-6 and not slabs[n + m, :, D:].any()
+        ops.depth_norm(slabs[:n], D, weights=w.to(DEV), out=out, base=slabs[n])
+        assert rel(out[:, :D], x + R.depth_average([s[:T, :D].double() for s in xs[:n]], pw[0, :n].double())) < 2e-6
     out, h = torch.empty(T, ld, device=DEV), torch.empty(T, ld, device=DEV)
     ops.depth_norm(d[:1, :T], D, 1e-4, out=out, g2=g2.to(DEV), h2=h)                # one slab as it is, one norm
     assert torch.equal(out[:, :D].cpu(), xs[0, :T, :D]) and rel(h[:, :D], R.rms_norm(xs[0, :T, :D].double(), g2[:D].double(), 1e-4)) < 2e-6
@@ -71,6 +82,9 @@ def test_poly_norm(T, F, ld):
         out = torch.full((T, ld), 7.0, dtype=dt, device=DEV)
         ops.poly_norm(z.to(DEV), F, coef.to(DEV), 1e-4, out)
         assert rel(out[:, :F].float(), want) < tol and not out[:, F:].any()
+        zb = z.bfloat16()
+        ops.poly_norm(zb.to(DEV), F, coef.to(DEV), 1e-4, out.fill_(7.0))
+        assert rel(out[:, :F].float(), R.poly_norm(zb[:, :F].double(), coef.double(), 1e-4)) < tol and not out[:, F:].any()
     for k in range(4):                                # each of the four numbers on its own
         one = torch.zeros(4)
         one[k] = 1.5
@@ -319,6 +333,10 @@ CONFIGS = {
     "few": R.config([L(64, 1, 1, 64, ff=96), L(32, 16, 1, 1, ff=64, experts=1), L(128, 4, 2, 100, ff=48, experts=9, top=4)], width=64, vocab=300, eps=1e-3),
     # heads and windows of a usual kind
     "usual": R.config([L(64, 12, 3, 80, ff=136), L(64, 12, 3, 48, ff=72, experts=10, top=1), L(128, 8, 4, 130, ff=64, experts=6, top=2), L(64, 16, 2, 96, ff=136)], width=128, vocab=260),
+    # nothing is a multiple of anything
+    "ragged": R.config([L(20, 7, 7, 50, ff=37), L(52, 9, 3, 31, ff=21, experts=7, top=5), L(101, 10, 2, 18, ff=75, scale=0.05)], width=93, vocab=127, eps=1e-2),
+    # the head layouts of large models: slices of the queries on both sides of tensor memory, one and two score accumulators
+    "heads": R.config([L(128, 32, 8, 150, ff=64), L(128, 20, 5, 60, ff=40, experts=4, top=2), L(64, 64, 8, 90), L(128, 14, 7, 130)], width=80, vocab=144),
     # more key heads than the tensor-core kernels take, head sizes beyond them
     "wide": R.config([L(136, 4, 2, 40, ff=72), L(72, 18, 18, 70, ff=40, experts=4, top=2), L(200, 2, 1, 96, ff=64)], width=96, vocab=264),
 }
@@ -396,7 +414,7 @@ def test_residual_after_every_layer(tmp_path, name, dtype):
         e.end(n)
 
 
-@pytest.mark.parametrize("name", ["odd", "usual"])
+@pytest.mark.parametrize("name", ["odd", "usual", "heads"])
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_batches_of_unequal_requests_reuse_pages(tmp_path, name, dtype):
     """Portions beside single tokens in any order, sequences left out of steps, and a pool so tight that pages come round again; each request's logits are those
@@ -577,7 +595,7 @@ def test_generate_and_device_side_decode_loop(tmp_path, dtype):
     assert [first] + hist[:, 0].tolist() == out
 
 
-@pytest.mark.parametrize("name", ["odd", "usual", "wide"])
+@pytest.mark.parametrize("name", ["odd", "usual", "wide", "heads", "ragged"])
 def test_workspace_canaries(tmp_path, name):
     for dtype in ("float32", "bfloat16"):
         cfg, W = model(name, dtype, 13)
