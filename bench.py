@@ -103,7 +103,7 @@ def main():
     ap.add_argument("--extras", default="train,moe", help="side benchmarks reported under extra: comma list of train, moe, or none")
     ap.add_argument("--no-baseline", action="store_true", help="skip the PyTorch baseline arm (vs_baseline stays null)")
     ap.add_argument("--workload", default="decode", choices=["decode", "hybrid"], help="hybrid: prefill and decode of the hybrid engine at "
-                    "--model's layer sizes beside the Llama engine at equal size, and its kernels one by one (bench_hybrid.py)")
+                    "--model's layer sizes beside the closest other engine at equal size, and its kernels one by one (bench_hybrid.py)")
     ap.add_argument("--tp", type=int, default=0, help="ranks per tensor-parallel replica (0: all ranks up to 4; 8 GPUs then run "
                     "two replicas of 4, each serving half of the batch)")
     args = ap.parse_args()

@@ -254,9 +254,12 @@ def time_kazolorn_kernels(cfg, dev, reps: int = 12) -> list[dict]:
         xs, w, g, h1, h2 = rnd(slabs + 1, n, d), rnd(slabs), rnd(d), bf(n, d), bf(n, d)
         bench(f"depth_norm of {slabs} [{n}]", lambda: ops.depth_norm(xs[:slabs], d, 1e-6, weights=w, out=xs[slabs], add=g, g1=g, g2=g, h1=h1, h2=h2), n * d * (4 * slabs + 8),
               like=f"rmsnorm [{n}]")
+        more, pw = rnd(slabs + 3, n, d), rnd(3, slabs)
+        bench(f"depth_norm of {slabs}, three sums more [{n}]", lambda: ops.depth_norm(more[:slabs], d, 1e-6, weights=w, out=xs[slabs], add=g, g1=g, g2=g, h1=h1, h2=h2,
+                                                                                     parts=more[slabs:], part_weights=pw), n * d * (4 * slabs + 20), like=f"rmsnorm [{n}]")
         x = rnd(n, d)
         bench(f"rmsnorm [{n}]", lambda: ops.rmsnorm(x, g, 1e-6, hb=h1), n * d * 6)
-        del xs
+        del xs, more
     # ---- attention
     nq, nk = H * D, G * D
     for n, seqs in ((T, 1), (B, B), (1, 1)):

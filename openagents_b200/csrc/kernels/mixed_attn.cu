@@ -562,7 +562,8 @@ template <int DK, int NT, int THREADS>
 static int launch_mixed_decode(MixedDecArgs a, const void* kc, int n_pages, int B, float* scratch, cudaStream_t st) {
   const int W = a.G * DK, page = 32 * W;
   const size_t out = (size_t)NT * 8 * DK * 4;
-  const size_t fixed = 1024 + 20 * 8 + NT * NT * 128 + (8 * NT + 1) * (DK + 8) * 2 + ((size_t)a.max_pages + 4) * 4;
+  const int listed = a.window > 0 ? min(a.max_pages, a.window / 16 + 2) : a.max_pages;      // pages a share can have
+  const size_t fixed = 1024 + 20 * 8 + NT * NT * 128 + (8 * NT + 1) * (DK + 8) * 2 + ((size_t)listed + 4) * 4;
   if (fixed > 100 * 1024) return B200_ERR_BAD_ARG;
   const size_t room = 222 * 1024 - fixed;               // (the rest of an SM's: this kernel's static part)
   int pairs = 0;

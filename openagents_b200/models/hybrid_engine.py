@@ -1,15 +1,18 @@
-"""Engine for hybrid stacks: softmax attention over the paged cache (plain, chunked, differential, or in a latent space) and gated linear
-attention with a state slot per sequence, layer by layer in the order the configuration gives.
+"""Engine for hybrid stacks: softmax attention over the paged cache (plain, windowed, chunked, differential, with mixed heads, or in a latent space) and
+gated linear attention with a state slot per sequence, layer by layer in the order the configuration gives.
 
-Batching, pages, state slots, CUDA graphs and the public operations are ``PagedEngine``'s.  Two kinds of residual step: with a norm on both
+Batching, pages, state slots, CUDA graphs and the public operations are ``PagedEngine``'s.  Three kinds of residual step: with a norm on both
 sides of every sublayer, ``norm_residual`` (the previous sublayer's norm, the residual sum, this one's norm, in one pass) takes the fp32 row an
 output projection left; with a norm ahead only (Dynamic Tanh), the output projection adds its scaled product into the residual itself and
-``norm_dyt`` reads it.  Per sublayer one fused projection (queries, keys, values, gates, latents in one matrix), the mixer, and the output
+``norm_dyt`` reads it; with parallel sublayers and a depth average, both output projections add their products, scaled per channel, into the layer's
+row of a history, and ``depth_norm`` makes the next layer's row and its two norms out of that history.  Per sublayer one fused projection (queries, keys, values, gates, latents in one matrix), the mixer, and the output
 projection.  A looped span of layers runs several times with the same weights; every run has a cache (or state) of its own.  The residual
 stream, norms, rotations, scores, decays and states are fp32 in both modes.
 
 Latent attention: a step's short entries (single decoded tokens, portions of a few) come first in the batch and work in the latent space,
 straight on the cache; the others expand the latents of their context into keys and values and take the prompt kernel.
+
+Mixed heads: prompts take the mixture on the queries (wide ones, on a cache row of all heads' keys), decoding takes it on the scores.
 
 ``dtype`` "bfloat16": projections and activations in bf16 on the tensor cores (up to ``small_path_tokens`` decoded tokens: the
 bf16 mat-vec on fp32 activations), fp16 keys, values and latents.  "float32": fp32 activations and caches throughout, products on

@@ -160,7 +160,7 @@ class CpuBackend(Backend):
 
 class CudaBackend(Backend):
     """A sm_100a engine (the registry's pick: dense ``LlamaEngine``, tensor-parallel when given a communicator, the
-    expert-parallel ``MoEEngine`` for models with experts, ``HybridEngine`` for stacks of recurrent, latent and differential attention layers).  Sampling happens on the device: greedy rows take the engine's fused
+    expert-parallel ``MoEEngine`` for models with experts, ``HybridEngine`` for stacks of recurrent, latent, differential and mixed-head attention layers).  Sampling happens on the device: greedy rows take the engine's fused
     arg-max (merged across vocabulary shards under tensor parallelism), the others the top-k / top-p kernel; a step
     copies back four bytes per sequence."""
     name = "cuda"
@@ -307,7 +307,7 @@ class CudaBackend(Backend):
 
 def open_backend(path: str, backend: str = "cuda", device="cuda:0", **engine_args) -> Backend:
     """The backend for a model (GGUF file or checkpoint folder) by its architecture: the paged engines (or the fp32 oracle) for the
-    llama and gpt-oss families, the paged hybrid engine for folirax and pesorax, the recompute backends for GPT-2-shape checkpoints."""
+    llama and gpt-oss families, the paged hybrid engine for folirax, pesorax and kazolorn, the recompute backends for GPT-2-shape checkpoints."""
     from ..models.config import HYBRID_ARCHS
     from ..models.registry import peek_architecture
     arch = peek_architecture(path)

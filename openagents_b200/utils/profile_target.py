@@ -13,7 +13,8 @@ pair (norm + all-gather push -> GEMM, GEMM -> reduce-scatter); ``zero_adamw``: t
 ``attn_train_fwd`` / ``attn_train_bwd``: training attention at GPT-2-small's shape (16 x 1024 tokens, 12 heads of 64);
 ``gemm_mn``: the weight-gradient GEMM (both operands read token-major); ``norm_slots``: the RMSNorm that is the tensor-parallel
 all-reduce, 64 rows of 4096 on a one-rank heap; ``gla_chunked`` / ``gla_decode``: gated linear attention of an 8B-size hybrid layer, a
-2048-token prompt / a decode step of 64 sequences.
+2048-token prompt / a decode step of 64 sequences; ``mixed_finish`` / ``mixed_prefill`` / ``mixed_decode``: attention with mixed heads at
+the same sizes (32 heads, 8 key heads of 128).
 """
 from __future__ import annotations
 
@@ -79,6 +80,22 @@ def main():
             fn = lambda: ops.attn_prefill(q, kc, vc, table, pages, z, tl, tl, 1, T, Hq, Hkv, hd, out_bf16=out)
         else:
             fn = lambda: ops.attn_prefill_tc05(q, kc, vc, table, z, tl, tl, 1, T, Hq, Hkv, out_bf16=out, status=status)
+    elif case in ("mixed_finish", "mixed_prefill", "mixed_decode"):
+        T, H, G, D = 2048, 32, 8, 128
+        B = 64 if case == "mixed_decode" else 1
+        pages = T // 16
+        kc = torch.randn((B * pages + 1, 1, 16, G * D), device=DEV).half()
+        table, lens = torch.arange(B * pages, dtype=torch.int32, device=DEV).view(B, pages) + 1, torch.full((B,), T, dtype=torch.int32, device=DEV)
+        mix, slopes, silent = torch.randn(H, H, device=DEV).bfloat16().float() * H ** -0.5, torch.rand(H, device=DEV) * 0.01, torch.zeros(H, device=DEV)
+        if case == "mixed_decode":
+            S, q, out = 2, torch.randn(B, H * D, device=DEV) / math.sqrt(D), torch.empty((B, H * D), dtype=torch.bfloat16, device=DEV)
+            prep, scratch = ops.mixed_decode_prepare(mix, slopes, H, G, D), torch.empty(ops.mixed_decode_scratch_floats(B, H, G, D, S), device=DEV)
+            fn = lambda: ops.mixed_decode(q, kc, prep, table, lens, B, H, G, D, S=S, sinks=silent, out_bf16=out, scratch=scratch, status=status)
+        else:
+            q, out = torch.randn(T, H * G * D, device=DEV).half() / math.sqrt(D), torch.empty((T, H * D), dtype=torch.bfloat16, device=DEV)
+            row, slot, z = torch.randn(T, (H + G) * D, device=DEV), torch.arange(16, 16 + T, dtype=torch.int32, device=DEV), torch.zeros(1, dtype=torch.int32, device=DEV)
+            fn = ((lambda: ops.mixed_finish(row, H * D, None, mix, D ** -0.5, slot, H, G, D, D, q, kc)) if case == "mixed_finish" else
+                  (lambda: ops.mixed_prefill(q, kc, slopes, table, z, lens, lens, 1, T, H, G, D, sinks=silent, out_bf16=out, status=status)))
     elif case in ("step64", "step1"):
         from ..models.config import LLAMA3_8B
         from ..models.engine import LlamaEngine
