@@ -688,7 +688,7 @@ def test_a_window_of_the_plain_kernels(tmp_path):
     any-size one (the mixer as another design would configure it)."""
     from openagents_b200.ops import cuda_ops as ops
     g = torch.Generator().manual_seed(9)
-    H, G, D, window = 8, 2, 64, 40
+    H, G, D, window = 12, 4, 64, 40
     lens, ctx = [1, 30, 70, 1], [77, 30, 141, 33]
     table, n_pages = pages_of(ctx)
     kc = torch.zeros(n_pages, G, 16, D, dtype=torch.float16, device=DEV)
