@@ -28,14 +28,16 @@ CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fopenmp", "-Wall", "-Wno-unused-fun
 
 
 # Kernels whose results are specified in IEEE 32-bit arithmetic (accurate division, roots, exponentials): no fast math.
-PRECISE = ("kernels/hybrid_ops.cu", "kernels/latent_attn.cu", "kernels/linear_attn.cu", "kernels/mixed_attn.cu", "kernels/moe.cu")
+PRECISE = ("kernels/delta_rule.cu", "kernels/hybrid_ops.cu", "kernels/latent_attn.cu", "kernels/linear_attn.cu", "kernels/mixed_attn.cu", "kernels/moe.cu",
+           "kernels/ssd.cu")
 
 # Parts of the libraries that stand on their own, for a process that serves one model family from a tree without built files.
 SUBSETS = {
     "hybrid": {"host": ("kv/kv_alloc.cpp",),
-               "cuda": ("kernels/attn_decode.cu", "kernels/attn_prefill_tc05.cu", "kernels/decode_ops.cu", "kernels/gemm_tc05.cu",
+               "cuda": ("kernels/attn_decode.cu", "kernels/attn_prefill_tc05.cu", "kernels/decode_ops.cu", "kernels/delta_rule.cu",
+                        "kernels/gemm_tc05.cu",
                         "kernels/hybrid_ops.cu", "kernels/latent_attn.cu", "kernels/linear_attn.cu", "kernels/matvec.cu", "kernels/mixed_attn.cu",
-                        "kernels/moe.cu")},
+                        "kernels/moe.cu", "kernels/ssd.cu")},
 }
 
 

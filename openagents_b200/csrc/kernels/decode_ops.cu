@@ -28,12 +28,12 @@ B200_API int b200_set_prefetch(int on) {
 // Weight types of the embedding table.
 enum { EMB_F32 = 0, EMB_BF16 = 1, EMB_Q8R = 2, EMB_Q6KR = 3 };
 
-// ids [T]; out fp32 [T][D].  `w` is the main plane, `w2` the scale plane (fp16) where one exists.
+// ids [T]; out fp32 [T][D], times `scale`.  `w` is the main plane, `w2` the scale plane (fp16) where one exists.
 // vocab_lo / vocab_n select a vocabulary shard: rows outside it produce zeros (tensor-parallel
 // embedding; the all-reduce that follows adds the one non-zero shard).
 __global__ void embedding_kernel(const int* __restrict__ ids, float* __restrict__ out, int D, int type,
                                  const uint8_t* __restrict__ w, const __half* __restrict__ w2,
-                                 int vocab_lo, int vocab_n) {
+                                 int vocab_lo, int vocab_n, float scale) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
@@ -45,16 +45,16 @@ __global__ void embedding_kernel(const int* __restrict__ ids, float* __restrict_
   }
   if (type == EMB_F32) {
     const float* r = (const float*)w + (size_t)id * D;
-    for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = r[i];
+    for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = r[i] * scale;
   } else if (type == EMB_BF16) {
     const __nv_bfloat16* r = (const __nv_bfloat16*)w + (size_t)id * D;
-    for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = __bfloat162float(r[i]);
+    for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = __bfloat162float(r[i]) * scale;
   } else if (type == EMB_Q8R) {
     const int8_t* r = (const int8_t*)w + (size_t)id * D;
     const __half* d = w2 + (size_t)id * (D / 32);
     for (int i = threadIdx.x; i < D; i += blockDim.x) {
       int slot = (i & ~7) | x8_slot(i & 7);
-      o[i] = __half2float(d[i >> 5]) * (float)r[slot];
+      o[i] = __half2float(d[i >> 5]) * (float)r[slot] * scale;
     }
   } else {  // EMB_Q6KR: 208-byte superblocks [lo words 128][T words 64][scales 16] + d plane
     const int nsb = D / 256;
@@ -72,15 +72,15 @@ __global__ void embedding_kernel(const int* __restrict__ ids, float* __restrict_
       const int hi = (tw >> (8 * (slot & 3) + 2 * (slot >> 2) + 4 * (word & 1))) & 3;
       const int q = (nib | (hi << 4)) - 32;
       const float sc = (float)((const int8_t*)(blk + 192))[e >> 4];
-      o[i] = __half2float(dp[sb]) * sc * (float)q;
+      o[i] = __half2float(dp[sb]) * sc * (float)q * scale;
     }
   }
 }
 
 B200_API int b200_embedding(const int* ids, float* out, int T, int D, int type, const void* w,
-                            const void* w2, int vocab_lo, int vocab_n, cudaStream_t st) {
+                            const void* w2, int vocab_lo, int vocab_n, float scale, cudaStream_t st) {
   return launch_pdl(embedding_kernel, dim3(T), dim3(256), 0, st, ids, out, D, type, (const uint8_t*)w,
-                    (const __half*)w2, vocab_lo, vocab_n);
+                    (const __half*)w2, vocab_lo, vocab_n, scale);
 }
 
 // ------------------------------------------------------------------ RMSNorm (+ quantize)
@@ -360,22 +360,23 @@ __global__ void rope_kv_kernel(const float* __restrict__ qkv, const int* __restr
   }
 }
 
-__global__ void rope_table_kernel(float2* __restrict__ tab, int n_pos, int hd, float theta) {
+// freq [half] (or null: theta^(-2j/hd)): the frequencies, where they are not a plain power series.
+__global__ void rope_table_kernel(float2* __restrict__ tab, int n_pos, int hd, float theta, const double* __restrict__ freq) {
   const int half = hd >> 1;
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n_pos * half) return;
   const int p = i / half, j = i % half;
-  const double inv = exp2(-2.0 * (double)j / (double)hd * log2((double)theta));
+  const double inv = freq ? freq[j] : exp2(-2.0 * (double)j / (double)hd * log2((double)theta));
   double sn, cs;
   sincos((double)p * inv, &sn, &cs);
   tab[i] = make_float2((float)cs, (float)sn);
 }
 
 // (cos, sin) table [n_pos][hd/2] for b200_rope_kv; built once per engine.
-B200_API int b200_rope_table(void* tab, int n_pos, int hd, float theta, cudaStream_t st) {
+B200_API int b200_rope_table(void* tab, int n_pos, int hd, float theta, const double* freq, cudaStream_t st) {
   if (hd % 2 || n_pos < 1) return B200_ERR_BAD_ARG;
   const int n = n_pos * (hd / 2);
-  rope_table_kernel<<<(n + 255) / 256, 256, 0, st>>>((float2*)tab, n_pos, hd, theta);
+  rope_table_kernel<<<(n + 255) / 256, 256, 0, st>>>((float2*)tab, n_pos, hd, theta, freq);
   return (int)cudaGetLastError();
 }
 

@@ -858,6 +858,7 @@ B200_API int b200_gemm_heads(const void* A, const void* B, int M, int heads, int
 //   mode 1: B rows are interleaved (gate_0, up_0, gate_1, ...), N = 2 * ffn; out_bf16 [rows][ldc] gets
 //           silu(gate) * up, N / 2 columns per row; with gate_w, row m's weight multiplies the expert's INPUT
 //           (gate and up ahead of the activation).
+//   mode 3: experts without a gate: out_bf16 [rows][ldc] gets the square of relu(product), N columns per row.
 //   mode 2: N = d_model; row m is added, scaled by gate_w[m], into token meta[2m+1] of rank meta[2m]:
 //           fp32 [tokens][ldc] at byte offset sym_off of that rank's symmetric heap.  The kernel ends
 //           with the cross-rank barrier, so afterwards every rank's residual stream is complete.  gate_w null:
@@ -869,7 +870,7 @@ B200_API int b200_moe_gemm(const void* A, const void* B, int groups, int group_r
                            const SymTable* sym, size_t sym_off, const float* col_scale, long live_rows, int* status, cudaStream_t st) {
   if (groups <= 0 || group_rows <= 0 || group_rows % BM || N <= 0 || K <= 0 || (lda % 8) || (ldb % 8) || (K % 8) || (N % 4))
     return B200_ERR_BAD_ARG;
-  if (mode == 1 ? (!out_bf16 || (ldc % 8) || (N % 32)) : (mode != 2 || !meta || (ldc % 4) || (sym_off % 16)))
+  if (mode == 1 || mode == 3 ? (!out_bf16 || (ldc % 8) || (mode == 1 && N % 32)) : (mode != 2 || !meta || (ldc % 4) || (sym_off % 16)))
     return B200_ERR_BAD_ARG;
   const int M = groups * group_rows;
   if (mode == 2 && !sym && !sym_off) return B200_ERR_BAD_ARG;
@@ -882,10 +883,11 @@ B200_API int b200_moe_gemm(const void* A, const void* B, int groups, int group_r
   if (rc) return rc;
   GemmEpi e = {};
   e.out_bf16 = (__nv_bfloat16*)out_bf16; e.ldc = ldc;
-  e.group_rows = group_rows; e.group_n = N; e.group_counts = counts; e.moe_mode = mode; e.meta = meta; e.gate_w = gate_w;
+  e.group_rows = group_rows; e.group_n = N; e.group_counts = counts; e.moe_mode = mode == 3 ? 0 : mode; e.meta = meta; e.gate_w = gate_w;
   e.rows_per_rank = 1;
   e.alpha = 1.f;
   e.col_scale = mode == 2 ? col_scale : nullptr;
+  if (mode == 3) e.act = ACT_RELU2;
   if (mode == 2 && !sym) {            // the rows' own memory: the offset is an address
     e.sym_off = sym_off;
   } else if (mode == 2) {

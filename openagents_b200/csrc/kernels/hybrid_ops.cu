@@ -12,7 +12,7 @@ using namespace b200;
 // ------------------------------------------------------------------ residual step
 
 // Per row:  x += y / rms(y) * gy   (when y is given; rms over D, eps inside the root)
-//           h  = x / rms(x) * gh   (when gh is given) -> bf16 and/or fp32, columns D..ldh written as zeros
+//           h  = x / rms(x) * gh   (gh null: h = x) -> bf16 and/or fp32 (when either is given), columns D..ldh written as zeros
 // i.e. the norm behind one sublayer, the residual sum and the norm ahead of the next in one pass over the row.
 // zero_a / zero_b: buffers cleared on the side; y_clear: the row of y is left zeroed.  Both serve the K-split projections,
 // which add into their outputs.
@@ -58,23 +58,26 @@ __global__ void __launch_bounds__(1024) norm_residual_kernel(float* __restrict__
     if (y_clear)
       for (int i = threadIdx.x; i < ldy; i += nt) y[(size_t)t * ldy + i] = 0.f;
   }
-  if (!gh) return;
-  float ss = 0.f;
+  if (!hb && !hf) return;
+  float r = 1.f;
+  if (gh) {
+    float ss = 0.f;
 #pragma unroll
-  for (int k = 0; k < kNormRegs; k++) ss += v[k] * v[k];
-  for (int i = threadIdx.x + kNormRegs * nt; i < D; i += nt) ss += xr[i] * xr[i];
-  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)D + eps);
+    for (int k = 0; k < kNormRegs; k++) ss += v[k] * v[k];
+    for (int i = threadIdx.x + kNormRegs * nt; i < D; i += nt) ss += xr[i] * xr[i];
+    r = 1.f / sqrtf(block_sum(ss, red) / (float)D + eps);
+  }
 #pragma unroll
   for (int k = 0; k < kNormRegs; k++) {
     const int i = threadIdx.x + k * nt;
     if (i < ldh) {
-      const float o = i < D ? v[k] * r * gh[i] : 0.f;
+      const float o = i < D ? (gh ? v[k] * r * gh[i] : v[k]) : 0.f;
       if (hb) hb[(size_t)t * ldh + i] = __float2bfloat16(o);
       if (hf) hf[(size_t)t * ldh + i] = o;
     }
   }
   for (int i = threadIdx.x + kNormRegs * nt; i < ldh; i += nt) {
-    const float o = i < D ? xr[i] * r * gh[i] : 0.f;
+    const float o = i < D ? (gh ? xr[i] * r * gh[i] : xr[i]) : 0.f;
     if (hb) hb[(size_t)t * ldh + i] = __float2bfloat16(o);
     if (hf) hf[(size_t)t * ldh + i] = o;
   }
@@ -123,17 +126,23 @@ __global__ void __launch_bounds__(256) norm_residual_vec_kernel(float4* __restri
       if (y_clear) yr[i] = z;
     }
   }
-  if (!gh) return;
-  float ss = 0.f;
+  if (!hb && !hf) return;
+  float r = 1.f;
+  if (gh) {
+    float ss = 0.f;
 #pragma unroll
-  for (int k = 0; k < R; k++) ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
-  const float r = 1.f / sqrtf(block_sum(ss, red) * inv_d + eps);
+    for (int k = 0; k < R; k++) ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    r = 1.f / sqrtf(block_sum(ss, red) * inv_d + eps);
+  }
 #pragma unroll
   for (int k = 0; k < R; k++) {
     const int i = tid + k * nt;
     if (i >= ldh4) continue;           // ldh4 > D4: padding columns are zeros
-    const float4 g = i < D4 ? gh[i] : z;
-    const float4 o = make_float4(v[k].x * r * g.x, v[k].y * r * g.y, v[k].z * r * g.z, v[k].w * r * g.w);
+    float4 o = v[k];
+    if (gh) {
+      const float4 g = i < D4 ? gh[i] : z;
+      o = make_float4(v[k].x * r * g.x, v[k].y * r * g.y, v[k].z * r * g.z, v[k].w * r * g.w);
+    }
     if (hb) {
       const __nv_bfloat162 p0 = __floats2bfloat162_rn(o.x, o.y), p1 = __floats2bfloat162_rn(o.z, o.w);
       *(uint2*)(hb + ((size_t)t * ldh4 + i) * 4) = make_uint2(*(const uint32_t*)&p0, *(const uint32_t*)&p1);
@@ -146,7 +155,7 @@ __global__ void __launch_bounds__(256) norm_residual_vec_kernel(float4* __restri
 B200_API int b200_norm_residual(float* y, int ldy, const float* gy, float* x, int T, int D, const float* gh, float eps, void* hb,
                                 float* hf, int ldh, int y_clear, float* zero_a, long zero_a_n, float* zero_b, long zero_b_n,
                                 cudaStream_t st) {
-  if (T < 1 || D < 1 || !x || (y && (!gy || ldy < D)) || (gh && (ldh < D || (!hb && !hf)))) return B200_ERR_BAD_ARG;
+  if (T < 1 || D < 1 || !x || (y && (!gy || ldy < D)) || (gh && !hb && !hf) || ((hb || hf) && ldh < D)) return B200_ERR_BAD_ARG;
   if ((zero_a && (zero_a_n % 4 || (uintptr_t)zero_a % 16)) || (zero_b && (zero_b_n % 4 || (uintptr_t)zero_b % 16)))
     return B200_ERR_BAD_ARG;
   const uintptr_t align = (uintptr_t)x | (uintptr_t)y | (uintptr_t)gy | (uintptr_t)gh | (uintptr_t)hb | (uintptr_t)hf;
@@ -749,6 +758,271 @@ B200_API int b200_qkv_finish(const float* in, int ld, int T, int q_off, int k_of
   const dim3 grid(T, (n_heads + 3) / 4);
   if (cache_f32) return launch_pdl(qkv_finish_kernel<float>, grid, dim3(128), 0, st, a, (float*)kc, (float*)vc);
   return launch_pdl(qkv_finish_kernel<__half>, grid, dim3(128), 0, st, a, (__half*)kc, (__half*)vc);
+}
+
+// ------------------------------------------------------------------ attention: finish of projections that are normed as whole rows
+
+// One CTA per token: q and k are each divided by the root mean square of the WHOLE projection row (all heads together) and multiplied by a weight per column
+// (q_w / k_w; null: left alone), then rotated on the first `rot` dimensions of every head with the (cos, sin) table (style as in qkv_finish); queries
+// are scaled.  Values (v_norm) are divided by their root mean square per head, then (lam) mixed with the first mixing layer's values of the same token:
+// v <- (1 - lam) v + lam v_first; without lam but with v_first they are written there.  Keys and values go to the paged cache, padding zero.
+struct RowQkvArgs {
+  const float* in;         // [T][ld]
+  int ld, q_off, k_off, v_off;
+  const float* q_w;        // [H * dim] or null
+  const float* k_w;        // [G * dim] or null
+  const int* pos;
+  const int* slot;
+  const float2* tab;       // [tab_len][rot / 2]
+  int tab_len;
+  int H, G, dim, vdim, DK, DV, rot, style, page_size, v_norm;
+  float eps, q_scale;
+  const float* lam;        // one number or null
+  float* v_first;          // [T][G * vdim] or null
+  float* q32;              // [T][H][DK] or null
+  __half* q16;             // [T][H][DK] or null
+};
+template <typename CT, bool VEC>
+__global__ void __launch_bounds__(256) row_qkv_finish_kernel(const RowQkvArgs a, CT* __restrict__ kc, CT* __restrict__ vc) {
+  extern __shared__ __align__(16) float row_s[];           // q row | k row
+  __shared__ float red[2][8];
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const float* row = a.in + (size_t)t * a.ld;
+  const int nq = a.H * a.dim, nk = a.G * a.dim, s = a.slot[t], p = a.pos[t];
+  const int page = s >= 0 ? s / a.page_size : 0, off = s >= 0 ? s % a.page_size : 0;
+  float sq = 0.f, sk = 0.f;
+  if constexpr (VEC) {
+    auto sum = [](float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; };
+#pragma unroll 4
+    for (int i = tid; i < nq / 4; i += 256) {
+      const float4 v = *(const float4*)(row + a.q_off + 4 * i);
+      *(float4*)(row_s + 4 * i) = v;
+      sq += sum(v);
+    }
+    for (int i = tid; i < nk / 4; i += 256) {
+      const float4 v = *(const float4*)(row + a.k_off + 4 * i);
+      *(float4*)(row_s + nq + 4 * i) = v;
+      sk += sum(v);
+    }
+  } else {
+    for (int i = tid; i < nq; i += 256) {
+      const float v = row[a.q_off + i];
+      row_s[i] = v;
+      sq += v * v;
+    }
+    for (int i = tid; i < nk; i += 256) {
+      const float v = row[a.k_off + i];
+      row_s[nq + i] = v;
+      sk += v * v;
+    }
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; i++) { sq += red[0][i]; sk += red[1][i]; }
+  const float rq = a.q_w ? 1.f / sqrtf(sq / (float)nq + a.eps) : 1.f, rk = a.k_w ? 1.f / sqrtf(sk / (float)nk + a.eps) : 1.f;
+  const int half = a.rot >> 1;
+  const float2* cs = a.tab + (size_t)min(max(p, 0), a.tab_len - 1) * half;
+  if constexpr (VEC) {                                     // four columns of a head, and the four they turn with
+    const int skip = a.style == 1 ? half : 0, units = (a.DK - skip) >> 2;
+    for (int i = tid; i < (a.H + a.G) * units; i += 256) {
+      const int hh = i / units, u = i - hh * units;
+      const bool is_q = hh < a.H;
+      if (!is_q && s < 0) continue;
+      const int c = 4 * u < half || a.style == 0 ? 4 * u : 4 * u + skip;
+      const float* src = row_s + hh * a.dim;               // the k row follows the q row
+      const float* w = is_q ? a.q_w ? a.q_w + hh * a.dim : nullptr : a.k_w ? a.k_w + (hh - a.H) * a.dim : nullptr;
+      const float r = is_q ? rq : rk, m = is_q ? a.q_scale : 1.f;
+      auto get = [&](int at) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (at < a.dim) {
+          v = *(const float4*)(src + at);
+          if (w) {
+            const float4 g = __ldg((const float4*)(w + at));
+            v = make_float4(v.x * r * g.x, v.y * r * g.y, v.z * r * g.z, v.w * r * g.w);
+          }
+        }
+        return v;
+      };
+      auto store = [&](int at, float4 v) {
+        v.x *= m; v.y *= m; v.z *= m; v.w *= m;
+        if (is_q) {
+          const size_t o = ((size_t)t * a.H + hh) * a.DK + at;
+          if (a.q32) put4(a.q32 + o, v);
+          if (a.q16) put4(a.q16 + o, v);
+        } else {
+          put4(kc + (((size_t)page * a.G + hh - a.H) * a.page_size + off) * a.DK + at, v);
+        }
+      };
+      float4 x = get(c);
+      if (a.style == 1 && c < half) {
+        float4 y = get(c + half);
+        const float4 e0 = __ldg((const float4*)(cs + c)), e1 = __ldg((const float4*)(cs + c + 2));
+        const float4 x1 = make_float4(x.x * e0.x - y.x * e0.y, x.y * e0.z - y.y * e0.w, x.z * e1.x - y.z * e1.y, x.w * e1.z - y.w * e1.w);
+        y = make_float4(y.x * e0.x + x.x * e0.y, y.y * e0.z + x.y * e0.w, y.z * e1.x + x.z * e1.y, y.w * e1.z + x.w * e1.w);
+        store(c, x1);
+        store(c + half, y);
+        continue;
+      }
+      if (a.style == 0 && c < a.rot) {
+        const float4 e = __ldg((const float4*)(cs + c / 2));
+        x = make_float4(x.x * e.x - x.y * e.y, x.y * e.x + x.x * e.y, x.z * e.z - x.w * e.w, x.w * e.z + x.z * e.w);
+      }
+      store(c, x);
+    }
+  } else {
+    const int pairs = (a.DK + 1) >> 1;
+    for (int i = tid; i < (a.H + a.G) * pairs; i += 256) {
+      const int hh = i / pairs, j = i - hh * pairs;
+      const bool is_q = hh < a.H;
+      if (!is_q && s < 0) continue;
+      const int i0 = j < half && a.style == 1 ? j : 2 * j, i1 = j < half && a.style == 1 ? j + half : 2 * j + 1;
+      const float* src = row_s + hh * a.dim;
+      const float* w = is_q ? a.q_w ? a.q_w + hh * a.dim : nullptr : a.k_w ? a.k_w + (hh - a.H) * a.dim : nullptr;
+      const float r = is_q ? rq : rk, m = is_q ? a.q_scale : 1.f;
+      float x = i0 < a.dim ? (w ? src[i0] * r * w[i0] : src[i0]) : 0.f, y = i1 < a.dim ? (w ? src[i1] * r * w[i1] : src[i1]) : 0.f;
+      if (j < half) {
+        const float2 e = cs[j];
+        const float x1 = x * e.x - y * e.y;
+        y = y * e.x + x * e.y;
+        x = x1;
+      }
+      if (is_q) {
+        const size_t o = ((size_t)t * a.H + hh) * a.DK;
+        if (a.q32) { a.q32[o + i0] = x * m; if (i1 < a.DK) a.q32[o + i1] = y * m; }
+        if (a.q16) { a.q16[o + i0] = __float2half(x * m); if (i1 < a.DK) a.q16[o + i1] = __float2half(y * m); }
+      } else {
+        CT* kd = kc + (((size_t)page * a.G + hh - a.H) * a.page_size + off) * a.DK;
+        put(kd + i0, x);
+        if (i1 < a.DK) put(kd + i1, y);
+      }
+    }
+  }
+  const float lam = a.lam ? *a.lam : 0.f;
+  for (int g = warp; g < a.G; g += 8) {                    // a warp per value head
+    const float* v = row + a.v_off + g * a.vdim;
+    float ss = 0.f;
+    if (a.v_norm)
+      for (int e = lane; e < a.vdim; e += 32) ss += v[e] * v[e];
+    const float r = a.v_norm ? 1.f / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps) : 1.f;
+    float* first = a.v_first ? a.v_first + ((size_t)t * a.G + g) * a.vdim : nullptr;
+    CT* dst = vc + (((size_t)page * a.G + g) * a.page_size + off) * a.DV;
+    for (int e = lane; e < a.DV; e += 32) {
+      float x = 0.f;
+      if (e < a.vdim) {
+        x = v[e] * r;
+        if (a.lam) x = (1.f - lam) * x + lam * first[e];
+        else if (first) first[e] = x;
+      }
+      if (s >= 0) put(dst + e, x);
+    }
+  }
+}
+// cache_f32: kc / vc hold fp32 instead of fp16; layout [page][G][page_size][DK or DV].
+B200_API int b200_row_qkv_finish(const float* in, int ld, int T, int q_off, int k_off, int v_off, const float* q_w, const float* k_w, const int* pos,
+                                 const int* slot, const void* tab, int tab_len, int H, int G, int dim, int vdim, int DK, int DV, int rot, int style,
+                                 int v_norm, float eps, float q_scale, int page_size, const float* lam, float* v_first, float* q32, void* q16, void* kc,
+                                 void* vc, int cache_f32, cudaStream_t st) {
+  if (T < 1 || H < 1 || G < 1 || H % G || dim < 1 || vdim < 1 || dim > DK || vdim > DV || (rot & 1) || rot > dim || rot < 0 || page_size < 1 || !kc || !vc ||
+      (!q32 && !q16) || (rot && (!tab || tab_len < 1)) || (lam && !v_first))
+    return B200_ERR_BAD_ARG;
+  const size_t smem = (size_t)(H + G) * dim * 4;
+  if (smem > 200 * 1024) return B200_ERR_BAD_ARG;
+  RowQkvArgs a;
+  a.in = in; a.ld = ld; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off; a.q_w = q_w; a.k_w = k_w; a.pos = pos; a.slot = slot; a.tab = (const float2*)tab;
+  a.tab_len = tab_len; a.H = H; a.G = G; a.dim = dim; a.vdim = vdim; a.DK = DK; a.DV = DV; a.rot = rot; a.style = style; a.page_size = page_size;
+  a.v_norm = v_norm; a.eps = eps; a.q_scale = q_scale; a.lam = lam; a.v_first = v_first; a.q32 = q32; a.q16 = (__half*)q16;
+  const bool vec = ((ld | q_off | k_off | dim | DK) & 3) == 0 && rot % 8 == 0 &&
+                   (((uintptr_t)in | (uintptr_t)q_w | (uintptr_t)k_w | (uintptr_t)tab | (uintptr_t)q32 | (uintptr_t)q16 | (uintptr_t)kc) & 15) == 0;
+  auto run = [&](auto kern, auto* k, auto* v) {
+    if (smem > 48 * 1024) {
+      cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      if (e != cudaSuccess) return (int)e;
+    }
+    return launch_pdl(kern, dim3(T), dim3(256), smem, st, a, k, v);
+  };
+  if (cache_f32)
+    return vec ? run(row_qkv_finish_kernel<float, true>, (float*)kc, (float*)vc) : run(row_qkv_finish_kernel<float, false>, (float*)kc, (float*)vc);
+  return vec ? run(row_qkv_finish_kernel<__half, true>, (__half*)kc, (__half*)vc) : run(row_qkv_finish_kernel<__half, false>, (__half*)kc, (__half*)vc);
+}
+
+// ------------------------------------------------------------------ gated norm in equal parts
+
+// Per row of D values y:  v = y * silu(z)   (z null: v = y), each of NG equal parts of v divided by its own root mean square, times w [D].
+// y fp32 [T][ldy], z fp32 [T][ldz]; out bf16 and/or fp32 [T][ldo], columns D..ldo zero.  One CTA per (row, part).
+__global__ void __launch_bounds__(256) group_norm_kernel(const float* __restrict__ y, int ldy, const float* __restrict__ z, int ldz, int D, int NG,
+                                                         const float* __restrict__ w, float eps, __nv_bfloat16* __restrict__ ob, float* __restrict__ of,
+                                                         int ldo, int vec) {
+  extern __shared__ __align__(16) float part_s[];          // [D / NG]
+  __shared__ float red[32];
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, g = blockIdx.y, n = D / NG, tid = threadIdx.x, nt = blockDim.x;
+  const float* yr = y + (size_t)t * ldy + g * n;
+  const float* zr = z ? z + (size_t)t * ldz + g * n : nullptr;
+  const size_t at = (size_t)t * ldo + g * n;
+  auto gate = [](float a, float b) { return a * (b / (1.f + expf(-b))); };
+  float ss = 0.f;
+  if (vec) {
+#pragma unroll 4
+    for (int i = tid; i < n / 4; i += nt) {
+      float4 v = *(const float4*)(yr + 4 * i);
+      if (zr) {
+        const float4 q = *(const float4*)(zr + 4 * i);
+        v = make_float4(gate(v.x, q.x), gate(v.y, q.y), gate(v.z, q.z), gate(v.w, q.w));
+      }
+      *(float4*)(part_s + 4 * i) = v;
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int i = tid; i < n; i += nt) {
+      const float v = zr ? gate(yr[i], zr[i]) : yr[i];
+      part_s[i] = v;
+      ss += v * v;
+    }
+  }
+  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+  if (vec) {
+    for (int i = tid; i < n / 4; i += nt) {                // every thread meets the elements it wrote
+      const float4 v = *(const float4*)(part_s + 4 * i), q = *(const float4*)(w + g * n + 4 * i);
+      const float4 o = make_float4(v.x * r * q.x, v.y * r * q.y, v.z * r * q.z, v.w * r * q.w);
+      if (ob) {
+        const __nv_bfloat162 p0 = __floats2bfloat162_rn(o.x, o.y), p1 = __floats2bfloat162_rn(o.z, o.w);
+        *(uint2*)(ob + at + 4 * i) = make_uint2(*(const uint32_t*)&p0, *(const uint32_t*)&p1);
+      }
+      if (of) *(float4*)(of + at + 4 * i) = o;
+    }
+  } else {
+    for (int i = tid; i < n; i += nt) {
+      const float o = part_s[i] * r * w[g * n + i];
+      if (ob) ob[at + i] = __float2bfloat16(o);
+      if (of) of[at + i] = o;
+    }
+  }
+  if (g == NG - 1)
+    for (int i = D + tid; i < ldo; i += nt) {
+      if (ob) ob[(size_t)t * ldo + i] = __float2bfloat16(0.f);
+      if (of) of[(size_t)t * ldo + i] = 0.f;
+    }
+}
+B200_API int b200_group_norm(const float* y, int ldy, const float* z, int ldz, int T, int D, int NG, const float* w, float eps, void* ob, float* of, int ldo,
+                             cudaStream_t st) {
+  if (T < 1 || D < 1 || NG < 1 || D % NG || ldy < D || (z && ldz < D) || ldo < D || !y || !w || (!ob && !of)) return B200_ERR_BAD_ARG;
+  const int n = D / NG;
+  const size_t smem = (size_t)n * 4;
+  if (smem > 200 * 1024) return B200_ERR_BAD_ARG;
+  const int vec = ((n | ldy | ldz | ldo) & 3) == 0 && (((uintptr_t)y | (uintptr_t)z | (uintptr_t)w | (uintptr_t)ob | (uintptr_t)of) & 15) == 0;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(group_norm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return (int)e;
+  }
+  const int threads = n >= 1024 ? 256 : n >= 256 ? 128 : 64;
+  return launch_pdl(group_norm_kernel, dim3(T, NG), dim3(threads), smem, st, y, ldy, z, z ? ldz : 0, D, NG, w, eps, (__nv_bfloat16*)ob, of, ldo, vec);
 }
 
 // ------------------------------------------------------------------ attention in 32-bit arithmetic, any head size

@@ -8,7 +8,7 @@
 // This file is compiled without fast math; decays, their logarithms and exponentials, the state and the norms are fp32.
 #include <cooperative_groups.h>
 
-#include "common.cuh"
+#include "chunk_mma.cuh"
 
 namespace cg = cooperative_groups;
 using namespace b200;
@@ -219,23 +219,8 @@ B200_API int b200_gla_recurrent(const float* in, int ld, int q_off, int k_off, i
 // rounded to bf16 once.  A as a product of q e^{b} and k e^{-b} is exact in relative terms but the second factor grows with the
 // decay; a chunk whose decay passes e^-60 in some channel takes the direct sum, whose exponents are never positive.
 
-constexpr int GC = 64;                 // tokens per chunk
 constexpr float kFactorLimit = 60.f;
 constexpr int kMaxRank = 64;
-
-// Walks (row, column) of a row-major grid in steps of a block, without a division per step.
-struct GridWalk {
-  int r, c, dr, dc, cols;
-  __device__ __forceinline__ GridWalk(int start, int step, int n_cols) : r(start / n_cols), c(start % n_cols), dr(step / n_cols), dc(step % n_cols), cols(n_cols) {}
-  __device__ __forceinline__ void next() {
-    r += dr;
-    c += dc;
-    if (c >= cols) {
-      c -= cols;
-      r++;
-    }
-  }
-};
 
 struct GlaChunkWs {
   __nv_bfloat16 *qh, *ql, *kh, *kl;    // [T][H][DP] decayed queries / keys, value and remainder
@@ -246,40 +231,6 @@ struct GlaChunkWs {
                                        // operand registers (value columns as rows), four of values, four of remainders
   int nvt;                             // value tiles, a multiple of 4
 };
-
-// Chunk c of a sequence whose tokens start at row q_start owns slot q_start / 64 + seq + c: no two chunks of a batch share one.
-__device__ __forceinline__ size_t chunk_slot(int q_start, int seq, int c) { return (size_t)(q_start / GC) + seq + c; }
-
-__device__ __forceinline__ void split_bf16(float x, __nv_bfloat16& hi, __nv_bfloat16& lo) {
-  hi = __float2bfloat16(x);
-  lo = __float2bfloat16(x - __bfloat162float(hi));
-}
-__device__ __forceinline__ uint32_t pack_bf2(__nv_bfloat16 a, __nv_bfloat16 b) {
-  __nv_bfloat162 p = __halves2bfloat162(a, b);
-  return *(uint32_t*)&p;
-}
-__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  __nv_bfloat16 xh, xl, yh, yl;
-  split_bf16(x, xh, xl);
-  split_bf16(y, yh, yl);
-  hi = pack_bf2(xh, yh);
-  lo = pack_bf2(xl, yl);
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t s32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
 
 constexpr int prep_threads(int dp) { return dp >= 64 ? 512 : 256; }
 
@@ -787,7 +738,6 @@ __global__ void __launch_bounds__(256, NV <= 2 ? 2 : 1) gla_output_kernel(const 
 }
 
 static int chunk_dp(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : dim <= 256 ? 256 : 0; }
-static size_t align256(size_t n) { return (n + 255) & ~(size_t)255; }
 static int value_tiles(int VP) { return (VP + 63) / 64 * 4; }
 
 // Bytes of workspace for b200_gla_chunked; 0: sizes it does not take (the caller then uses b200_gla_recurrent).

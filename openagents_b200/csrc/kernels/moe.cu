@@ -31,6 +31,7 @@ struct MoeDispatchArgs {
   size_t recv_w_off;          // fp32 [E_local][C] gate weight
   size_t counts_off;          // int32 [E_local] rows claimed so far (zero before the layer starts)
   int score;                  // weights of the chosen: 0 the softmax over them, 1 the sigmoid of each one's own logit
+  float scale;                // multiplies the weights
   int dispatch;               // 0: the choice only (topk_ids, topk_w), nothing moves
   int local;                  // one rank without a symmetric heap: the offsets are addresses, no barrier at the end
   int* topk_ids;              // optional [T][top_k] (this rank), for tests and telemetry
@@ -98,7 +99,7 @@ __global__ void __launch_bounds__(256) moe_route_dispatch_kernel(const MoeDispat
       }
       if (bi == 0x7fffffff) bi = 0;              // a row without a finite logit
       if (k == 0) mx = best;
-      const float ex = a.score == 1 ? 1.f / (1.f + expf(-best)) : __expf(best - mx);
+      const float ex = a.score == 1 ? 1.f / (1.f + expf(-best)) : expf(best - mx);
       sum += ex;
       if (lane == k) { my_val = ex; my_sel = bi; }
 #pragma unroll
@@ -107,7 +108,7 @@ __global__ void __launch_bounds__(256) moe_route_dispatch_kernel(const MoeDispat
     }
     if (lane < a.top_k) {
       const int k = lane;
-      const float wgt = a.score == 1 ? my_val : my_val / sum;
+      const float wgt = (a.score == 1 ? my_val : my_val / sum) * a.scale;
       s_sel[k] = my_sel;
       s_w[k] = wgt;
       if (a.topk_ids) a.topk_ids[(size_t)t * a.top_k + k] = my_sel;
@@ -159,7 +160,7 @@ __global__ void moe_zero_kernel(int* p, int n) {
 // score: see MoeDispatchArgs.  sym null: one rank; the offsets are then addresses, and counts_off = 0 asks for the choice alone.
 B200_API int b200_moe_route_dispatch(const void* h, const float* hf, const float* wr, const float* br, int T, int d, int E, int top_k,
                                      int E_local, int C, size_t recv_x_off, size_t recv_meta_off, size_t recv_w_off,
-                                     size_t counts_off, int* topk_ids, float* topk_w, int score, const SymTable* sym, int* status,
+                                     size_t counts_off, int* topk_ids, float* topk_w, int score, float scale, const SymTable* sym, int* status,
                                      cudaStream_t st) {
   const int dispatch = sym || counts_off;
   if (T < 1 || E < 1 || E > kMoeMaxExperts || top_k < 1 || top_k > kMoeMaxTopK || top_k > E || (d % 8) || (!h && (dispatch || !hf)) ||
@@ -169,7 +170,7 @@ B200_API int b200_moe_route_dispatch(const void* h, const float* hf, const float
   MoeDispatchArgs a;
   a.h = (const __nv_bfloat16*)h; a.hf = hf; a.wr = wr; a.br = br; a.T = T; a.d = d; a.E = E; a.top_k = top_k;
   a.E_local = E_local; a.C = C; a.recv_x_off = recv_x_off; a.recv_meta_off = recv_meta_off; a.recv_w_off = recv_w_off;
-  a.counts_off = counts_off; a.topk_ids = topk_ids; a.topk_w = topk_w; a.status = status; a.score = score; a.dispatch = dispatch;
+  a.counts_off = counts_off; a.topk_ids = topk_ids; a.topk_w = topk_w; a.status = status; a.score = score; a.scale = scale; a.dispatch = dispatch;
   a.local = !sym;
   if (sym) a.sym = *sym;
   else a.sym = SymTable{};
@@ -220,6 +221,36 @@ __global__ void __launch_bounds__(256) expert_gate_up_kernel(const float* __rest
     if (lane == 0 && j0 + r < F) mid[(size_t)ts * F + j0 + r] = a / (1.f + expf(-a)) * b;
   }
 }
+// mid[t][s][j] = w * relu(u_j)^2, u the up product of token t's s-th expert with its fp32 row and w the expert's weight (null: one): experts without a
+// gate, whose weight multiplies their output (the down product is linear, so it may as well be taken here).  Weights [E][F][K] bf16.
+__global__ void __launch_bounds__(256) expert_up_kernel(const float* __restrict__ x, int K, const __nv_bfloat16* __restrict__ w1, int F, const int* __restrict__ ids,
+                                                        const float* __restrict__ wts, int top, float* __restrict__ mid) {
+  constexpr int RW = 2 * kExpertRows;
+  pdl_trigger();
+  pdl_wait();
+  const int ts = blockIdx.x, lane = threadIdx.x & 31, j0 = (blockIdx.y * 8 + (threadIdx.x >> 5)) * RW;
+  if (j0 >= F) return;
+  const float* xr = x + (size_t)(ts / top) * K;
+  const __nv_bfloat16* w = w1 + (size_t)ids[ts] * F * K;
+  float u[RW];
+#pragma unroll
+  for (int r = 0; r < RW; r++) u[r] = 0.f;
+#pragma unroll 2
+  for (int k = lane * 8; k < K; k += 256) {
+    uint4 q[RW];
+#pragma unroll
+    for (int r = 0; r < RW; r++) q[r] = ldg_stream(w + (size_t)min(j0 + r, F - 1) * K + k);
+    const float4 x0 = *(const float4*)(xr + k), x1 = *(const float4*)(xr + k + 4);
+#pragma unroll
+    for (int r = 0; r < RW; r++) u[r] += dot8(q[r], x0, x1);
+  }
+  const float wt = wts ? wts[ts] : 1.f;
+#pragma unroll
+  for (int r = 0; r < RW; r++) {
+    const float v = fmaxf(warp_sum(u[r]), 0.f);
+    if (lane == 0 && j0 + r < F) mid[(size_t)ts * F + j0 + r] = wt * v * v;
+  }
+}
 // out[t][n] += scale[n] * sum over s of (W_down of token t's s-th expert) mid[t][s].  w2 [E][N][F] bf16; scale [N] or null.
 __global__ void __launch_bounds__(256) expert_down_kernel(const float* __restrict__ mid, int F, const __nv_bfloat16* __restrict__ w2, int N,
                                                           const int* __restrict__ ids, int top, const float* __restrict__ scale, float* __restrict__ out,
@@ -256,6 +287,12 @@ B200_API int b200_expert_gate_up(const float* x, int T, int K, const void* w13, 
   if (T < 1 || top < 1 || K < 8 || K % 8 || F < 8 || F % 8 || !ids || (((uintptr_t)x | (uintptr_t)w13) & 15)) return B200_ERR_BAD_ARG;
   const int per = 8 * kExpertRows;
   return launch_pdl(expert_gate_up_kernel, dim3(T * top, (F + per - 1) / per), dim3(256), 0, st, x, K, (const __nv_bfloat16*)w13, F, ids, wts, top, mid);
+}
+// As b200_expert_gate_up for experts without a gate: w1 [E][F][K], the square of relu, the weight on the result.
+B200_API int b200_expert_up(const float* x, int T, int K, const void* w1, int F, const int* ids, const float* wts, int top, float* mid, cudaStream_t st) {
+  if (T < 1 || top < 1 || K < 8 || K % 8 || F < 8 || F % 8 || !ids || (((uintptr_t)x | (uintptr_t)w1) & 15)) return B200_ERR_BAD_ARG;
+  const int per = 16 * kExpertRows;
+  return launch_pdl(expert_up_kernel, dim3(T * top, (F + per - 1) / per), dim3(256), 0, st, x, K, (const __nv_bfloat16*)w1, F, ids, wts, top, mid);
 }
 B200_API int b200_expert_down(const float* mid, int T, int F, const void* w2, int N, const int* ids, int top, const float* scale, float* out, int ldo,
                               cudaStream_t st) {

@@ -69,7 +69,7 @@ class CheckpointDirSource(WeightSource):
         self.device = device
         ranks = {}
         for name, (_, shape, _, _) in self.file.entries.items():      # sizes only a tensor's shape gives
-            if name.startswith("l") and name.endswith((".mix.a1", ".mix.dq")) and len(shape) == 2 and name[1:-7].isdigit():
+            if name.startswith("l") and name.endswith((".mix.a1", ".mix.dq", ".mix.w1")) and len(shape) == 2 and name[1:-7].isdigit():
                 ranks[int(name[1:-7])] = shape[0]
         self.cfg = config_from_json(self.json, ranks, name=os.path.basename(os.path.normpath(path)))
         self.metadata: dict = {}

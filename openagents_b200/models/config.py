@@ -7,6 +7,7 @@ The presets are the shapes the benchmark configurations name; the server detects
 from __future__ import annotations
 
 import json
+import math
 from dataclasses import asdict, dataclass, replace
 
 
@@ -14,7 +15,8 @@ from dataclasses import asdict, dataclass, replace
 class MixerSpec:
     """What mixes tokens in one layer of a hybrid stack.  ``kind`` "attention": softmax attention over the paged cache;
     "latent": softmax attention whose keys and values are projections of one cached latent per token; "gla": gated linear
-    attention with a decay per key channel and a state slot per sequence."""
+    attention with a decay per key channel; "delta": the generalized delta rule; "ssd": Mamba-2's state-space duality (the last three with a state slot per
+    sequence)."""
     kind: str
     heads: int
     dim: int                       # per-head query / key size
@@ -44,12 +46,22 @@ class MixerSpec:
     q_rank: int = 0                # size of the queries' latent
     sink: bool = False             # a learned term per head in the softmax's denominator
     out_gate: bool = False         # a sigmoid gate per output element
-    # gla
+    # attention whose projections are normed as whole rows
+    row_norm: bool = False         # all of q, and all of k, divided by its root mean square and weighted, ahead of the rotation
+    v_norm: bool = False           # values divided by their root mean square per head
+    v_mix: bool = False            # a learned mixture with the values of the first such layer
+    rope_scaling: tuple[float, float, float, float] | None = None      # (factor, low, high, original): long wavelengths stretched, as in Llama 3.1
+    # ssd (``dim``: the state size)
+    groups: int = 1                # heads / groups heads share an input and an output vector
+    norm_groups: int = 1           # equal parts of the gated output that are normed on their own
+    conv: int = 4                  # taps of the causal filter
+    # gla, delta
     tau: float = 1.0               # decay = sigmoid(z)^(1/tau)
+    log_decay: float = 0.0         # delta: decay = exp(-log_decay * sigmoid(z))
     rank: int = 16                 # rank of the decay's projection
 
     def __post_init__(self):
-        if self.kind not in ("attention", "latent", "gla"):
+        if self.kind not in ("attention", "latent", "gla", "delta", "ssd"):
             raise ValueError(f"unknown mixer {self.kind!r}")
         if min(self.heads, self.dim, self.vdim) < 1:
             raise ValueError("a mixer's heads and sizes must be positive")
@@ -71,20 +83,68 @@ class MixerSpec:
                 raise ValueError("the key/value heads must divide the query heads")
             if not 0 <= self.rope_dims <= self.dim or self.rope_dims % 2:
                 raise ValueError("the rotated dimensions must be even and within the head")
+            if self.rows_normed and (self.qk_norm or self.head_gate or self.kv_from is not None or self.bias or self.tied_kv or self.maps > 1):
+                raise ValueError("norms of whole projections and mixed values go with plain attention")
+            if self.rope_scaling is not None:
+                factor, low, high, original = self.rope_scaling
+                if not self.rows_normed or min(factor, low, original) <= 0 or high <= low:
+                    raise ValueError("bad frequency scaling, or one without norms of whole projections")
+        elif self.kind == "ssd":
+            if self.groups < 1 or self.heads % self.groups or self.norm_groups < 1 or self.heads * self.vdim % self.norm_groups or self.conv < 1:
+                raise ValueError("the groups must divide the heads, the norm's parts the row, and the filter needs a tap")
+        elif self.kind == "delta":
+            if self.log_decay <= 0:
+                raise ValueError("the decay's exponent must be positive")
         elif self.tau == 0:
             raise ValueError("tau must not be zero")
 
 
+    @property
+    def rows_normed(self) -> bool:
+        """Attention whose projections are finished row by row."""
+        return self.row_norm or self.v_norm or self.v_mix
+
+    @property
+    def stateful(self) -> bool:
+        return self.kind in ("gla", "delta", "ssd")
+
+    @property
+    def channels(self) -> int:
+        """ssd: what passes the filter."""
+        return self.heads * self.vdim + 2 * self.groups * self.dim
+
+    def rope_frequencies(self) -> list[float]:
+        """Angle per position of every rotated pair: base^(-2i/dims); with ``rope_scaling``, wavelengths longer than original / low are divided by the factor,
+        shorter than original / high kept, and those between mixed."""
+        out = []
+        for i in range(self.rope_dims // 2):
+            f = self.rope_base ** (-2.0 * i / self.rope_dims)
+            if self.rope_scaling is not None:
+                factor, low, high, original = self.rope_scaling
+                turns = original * f / (2.0 * math.pi)               # original over the wavelength
+                keep = min(1.0, max(0.0, (turns - low) / (high - low)))
+                f = (1.0 - keep) * f / factor + keep * f
+            out.append(f)
+        return out
+
+
 @dataclass(frozen=True)
 class ExpertSpec:
-    """A mixture of gated feed-forwards (silu) in place of one: each token uses the ``top`` experts with the largest scores, weighted by the sigmoid of
-    their router logits, not renormalised; the weight multiplies what goes into an expert."""
+    """A mixture of feed-forwards in place of one: each token uses the ``top`` experts with the largest scores.  ``score`` "sigmoid": weights are the sigmoids
+    of the chosen router logits, as they are; "softmax": the softmax of all logits, renormalised over the chosen; times ``scale``.  ``weigh`` "input": the weight
+    multiplies what goes into an expert; "output": what comes out.  ``shared``: width of one more feed-forward that every token uses (0: none)."""
     experts: int
     top: int
+    score: str = "sigmoid"
+    scale: float = 1.0
+    weigh: str = "input"
+    shared: int = 0
 
     def __post_init__(self):
         if not 1 <= self.top <= self.experts:
             raise ValueError("a token's experts must be at least one and no more than there are")
+        if self.score not in ("sigmoid", "softmax") or self.weigh not in ("input", "output") or self.shared < 0:
+            raise ValueError("bad router score, place of the weight or shared width")
 
 
 @dataclass(frozen=True)
@@ -99,7 +159,7 @@ class LayerSpec:
 
 @dataclass(frozen=True)
 class ModelConfig:
-    arch: str = "llama"            # llama | gpt2 | gpt-oss | folirax | pesorax | kazolorn
+    arch: str = "llama"            # llama | gpt2 | gpt-oss | folirax | pesorax | kazolorn | tekosun
     n_layers: int = 2
     d_model: int = 256
     n_heads: int = 4
@@ -125,7 +185,9 @@ class ModelConfig:
     walk: str = "serial"           # "parallel": mixer and feed-forward of a layer read the same residual (a norm each) and are added together
     layer_scale: bool = False      # a learned factor per channel on what either adds
     depth_average: bool = False    # what a layer hands on is a learned mixture of the embedding output and every layer's result so far
-    post_norm: bool = True         # a norm behind every sublayer as well
+    pre_norm: bool = True          # a norm ahead of every sublayer
+    post_norm: bool = True         # a norm behind every sublayer
+    embed_scale: float = 1.0       # multiplies the embedding
     residual_mult: float = 1.0     # multiplies what a sublayer adds to the residual (stacks without post_norm)
     loop: tuple[int, int, int] | None = None     # (start, stop, times): these layers run ``times`` times in a row, the embedding added ahead of every pass but the first
     logit_scale: float = 1.0
@@ -155,7 +217,7 @@ class ModelConfig:
     @property
     def has_state(self) -> bool:
         """Whether some layer carries a recurrent state from token to token."""
-        return any(l.mixer.kind == "gla" for l in self.layers)
+        return any(l.mixer.stateful for l in self.layers)
 
     def n_params(self) -> int:
         d, f, v = self.d_model, self.ffn, self.vocab
@@ -407,8 +469,93 @@ def _kazolorn_to_json(cfg: ModelConfig) -> dict:
     return {"architecture": "Kazolorn", "layers": layers, "width": cfg.d_model, "vocab": cfg.vocab, "norm": {"eps": cfg.norm_eps}}
 
 
+DELTA_LOG_DECAY = math.exp(-0.5)   # Tekosun: log decays lie between this, negated, and 0
+
+
+def _tekosun(c: dict, ranks: dict[int, int], name: str, context: int) -> ModelConfig:
+    """Tekosun: generalized delta rule, Mamba-2 and windowed attention (whole-row query and key norms, normed and mixed values, scaled rotation) in any order; a norm
+    behind every sublayer only; mixtures of squared-relu experts with a shared one; a scaled embedding."""
+    layers = []
+    for i, e in enumerate(_need(c, "layers", list, "")):
+        w = f"layers[{i}]."
+        mx, kind = _need(e, "mixer", dict, w), _need(e, "type", str, w)
+        w2 = w + "mixer."
+        heads = _need(mx, "heads", int, w2)
+        if kind == "general_delta":
+            dim = _need(mx, "dim", int, w2)
+            m = MixerSpec("delta", heads, dim, dim, log_decay=DELTA_LOG_DECAY, rank=ranks.get(i, MixerSpec.rank))
+        elif kind == "mamba2":
+            m = MixerSpec("ssd", heads, _need(mx, "state", int, w2), _need(mx, "vdim", int, w2), groups=_need(mx, "groups", int, w2),
+                          norm_groups=_need(mx, "norm_groups", int, w2), conv=_need(mx, "conv", int, w2))
+        elif kind == "attention":
+            window = 0 if mx.get("mask") is None else _need(_need(mx, "mask", dict, w2), "size", int, w2 + "mask.")
+            if mx.get("mask") is not None and window < 1:
+                raise ValueError(f"config: {w2}mask.size must be positive")
+            rot = {"base": 1.0, "dims": 0} if "rot" in mx and mx["rot"] is None else _need(mx, "rot", dict, w2)      # null: no rotation
+            scaling = None
+            if rot.get("scaling") is not None:
+                sc = _need(rot, "scaling", dict, w2 + "rot.")
+                scaling = tuple(_need(sc, k, float, w2 + "rot.scaling.") for k in ("factor", "low", "high", "original"))
+            if not isinstance(mx.get("v_mix", False), bool):
+                raise ValueError(f"config: {w2}v_mix must be true or false")
+            dim = _need(mx, "dim", int, w2)
+            m = MixerSpec("attention", heads, dim, dim if mx.get("vdim") is None else _need(mx, "vdim", int, w2), kv_heads=_need(mx, "kv_heads", int, w2),
+                          scale=_need(mx, "scale", float, w2), rope_base=_need(rot, "base", float, w2 + "rot."), rope_dims=_need(rot, "dims", int, w2 + "rot."),
+                          rope_style="half", rope_scaling=scaling, row_norm=True, v_norm=True, v_mix=mx.get("v_mix", False), window=window)
+            first = next((l.mixer for l in layers if l.mixer.v_mix), m)
+            if m.v_mix and (m.kv_heads, m.vdim) != (first.kv_heads, first.vdim):
+                raise ValueError(f"config: {w2}v_mix: the values have another size than the first such layer's")
+        else:
+            raise ValueError(f"config: {w}type {kind!r} is not a mixer of this design")
+        mlp, ff, moe = e.get("mlp"), 0, None
+        if mlp is not None:
+            if _need(mlp, "kind", str, w + "mlp.") != "moe":
+                raise ValueError(f"config: {w}mlp.kind {mlp['kind']!r} is not known")
+            ff = _need(_need(mlp, "expert", dict, w + "mlp."), "ff", int, w + "mlp.expert.")
+            router = _need(mlp, "router", dict, w + "mlp.")
+            shared = 0 if mlp.get("shared") is None else _need(_need(mlp, "shared", dict, w + "mlp."), "ff", int, w + "mlp.shared.")
+            if ff < 1 or (mlp.get("shared") is not None and shared < 1):
+                raise ValueError(f"config: {w}mlp: the widths must be positive")
+            w3 = w + "mlp.router."
+            moe = ExpertSpec(_need(router, "experts", int, w3), _need(router, "top", int, w3), "softmax",
+                             1.0 if router.get("scale") is None else _need(router, "scale", float, w3), "output", shared)
+        layers.append(LayerSpec(m, ff, "relu2", moe))
+    if not layers:
+        raise ValueError("config: layers is empty")
+    mx = [l.mixer for l in layers]
+    scale = 1.0 if c.get("embedding") is None or c["embedding"].get("scale") is None else _need(c["embedding"], "scale", float, "embedding.")
+    return ModelConfig(arch="tekosun", n_layers=len(layers), d_model=_need(c, "width", int, ""), vocab=_need(c, "vocab", int, ""),
+                       n_heads=max(m.heads for m in mx), n_kv_heads=max(1, *(m.kv_heads for m in mx)), head_dim=max(m.dim for m in mx),
+                       ffn=max(l.ffn for l in layers), context=context, norm_eps=_need(_need(c, "norm", dict, ""), "eps", float, "norm."),
+                       layers=tuple(layers), norm="rms1", pre_norm=False, embed_scale=scale, name=name)
+
+
+def _tekosun_to_json(cfg: ModelConfig) -> dict:
+    layers = []
+    for l in cfg.layers:
+        m, mlp = l.mixer, None
+        if m.kind == "delta":
+            kind, mx = "general_delta", {"heads": m.heads, "dim": m.dim}
+        elif m.kind == "ssd":
+            kind, mx = "mamba2", {"heads": m.heads, "vdim": m.vdim, "state": m.dim, "groups": m.groups, "norm_groups": m.norm_groups, "conv": m.conv}
+        else:
+            rot = {"base": m.rope_base, "dims": m.rope_dims}
+            if m.rope_scaling is not None:
+                rot["scaling"] = dict(zip(("factor", "low", "high", "original"), m.rope_scaling))
+            kind, mx = "attention", {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale, "rot": rot, "v_mix": m.v_mix,
+                                     "mask": {"size": m.window} if m.window else None}
+        if l.moe:
+            mlp = {"kind": "moe", "expert": {"ff": l.ffn}, "router": {"experts": l.moe.experts, "top": l.moe.top, "scale": l.moe.scale},
+                   "shared": {"ff": l.moe.shared} if l.moe.shared else None}
+        layers.append({"type": kind, "mixer": mx, "mlp": mlp})
+    return {"architecture": "Tekosun", "layers": layers, "width": cfg.d_model, "vocab": cfg.vocab, "norm": {"eps": cfg.norm_eps},
+            "embedding": {"scale": cfg.embed_scale}, "ranks": {str(i): l.mixer.rank for i, l in enumerate(cfg.layers) if l.mixer.kind == "delta"}}
+
+
 def hybrid_to_json(cfg: ModelConfig) -> dict:
     """The inverse of ``config_from_json``."""
+    if cfg.arch == "tekosun":
+        return _tekosun_to_json(cfg)
     if cfg.arch == "pesorax":
         return _pesorax_to_json(cfg)
     if cfg.arch == "kazolorn":
@@ -429,7 +576,7 @@ def hybrid_to_json(cfg: ModelConfig) -> dict:
             "ranks": {str(i): l.mixer.rank for i, l in enumerate(cfg.layers) if l.mixer.kind == "gla"}}
 
 
-JSON_ARCHITECTURES = {"Folirax": _folirax, "Pesorax": _pesorax, "Kazolorn": _kazolorn}
+JSON_ARCHITECTURES = {"Folirax": _folirax, "Pesorax": _pesorax, "Kazolorn": _kazolorn, "Tekosun": _tekosun}
 HYBRID_ARCHS = tuple(a.lower() for a in JSON_ARCHITECTURES)
 
 
@@ -515,5 +662,23 @@ def kazolorn_stack(width: int, ffn: int, vocab: int, layers: int, heads: int, kv
 KAZOLORN_8B = kazolorn_stack(4096, 14336, 128256, 32, 32, 8, 128, 4096, "kazolorn-8b-shape")
 KAZOLORN_MOE = kazolorn_stack(2048, 8192, 32000, 16, 16, 4, 128, 1024, "kazolorn-moe-shape", experts=32, top=4, expert_ffn=2048)
 
+def tekosun_stack(width: int, vocab: int, groups: int, heads: int, kv_heads: int, dim: int, window: int, delta_heads: int, delta_dim: int, rank: int, ssd_heads: int,
+                  ssd_vdim: int, state: int, experts: int, top: int, expert_ffn: int, shared: int, name: str) -> ModelConfig:
+    """A regular stack: ``groups`` times (delta rule, attention, delta rule, state-space duality), a mixture of experts behind each."""
+    moe = ExpertSpec(experts, top, "softmax", 1.5, "output", shared)
+    delta = LayerSpec(MixerSpec("delta", delta_heads, delta_dim, delta_dim, log_decay=DELTA_LOG_DECAY, rank=rank), expert_ffn, "relu2", moe)
+    attn = LayerSpec(MixerSpec("attention", heads, dim, dim, kv_heads=kv_heads, scale=dim ** -0.5, rope_base=500000.0, rope_dims=dim, rope_style="half",
+                               rope_scaling=(8.0, 1.0, 4.0, 8192.0), row_norm=True, v_norm=True, v_mix=True, window=window), expert_ffn, "relu2", moe)
+    ssd = LayerSpec(MixerSpec("ssd", ssd_heads, state, ssd_vdim, groups=1, norm_groups=1, conv=4), expert_ffn, "relu2", moe)
+    layers = (delta, attn, delta, ssd) * groups
+    return ModelConfig(arch="tekosun", n_layers=len(layers), d_model=width, n_heads=max(heads, delta_heads, ssd_heads), n_kv_heads=kv_heads,
+                       head_dim=max(dim, delta_dim, state), ffn=expert_ffn, vocab=vocab, context=HYBRID_CONTEXT, norm_eps=1e-6, layers=layers, norm="rms1",
+                       pre_norm=False, embed_scale=4.0, name=name)
+
+
+# layers of the 8B preset's width, and a smaller stack; 32 experts of which a token uses four, and a shared one of the size of two
+TEKOSUN_8B = tekosun_stack(4096, 128256, 8, 32, 8, 128, 4096, 64, 64, 128, 128, 64, 128, 32, 4, 2048, 4096, "tekosun-8b-shape")
+TEKOSUN_1B = tekosun_stack(2048, 32000, 4, 16, 4, 128, 1024, 32, 64, 96, 64, 64, 128, 32, 4, 1024, 2048, "tekosun-1b-shape")
+
 PRESETS = {c.name: c for c in (TINY_LLAMA, LLAMA3_8B, LLAMA3_70B, GPT2_SMALL, GPT_OSS_20B, FOLIRAX_8B, FOLIRAX_1B, PESORAX_8B, PESORAX_1B, KAZOLORN_8B,
-                               KAZOLORN_MOE)}
+                               KAZOLORN_MOE, TEKOSUN_8B, TEKOSUN_1B)}

@@ -1,8 +1,9 @@
 """Engine for hybrid stacks: softmax attention over the paged cache (plain, windowed, chunked, differential, with mixed heads, or in a latent space) and
-gated linear attention with a state slot per sequence, layer by layer in the order the configuration gives.
+recurrent layers with a state slot per sequence (gated linear attention, the generalized delta rule, Mamba-2's state-space duality), layer by layer in
+the order the configuration gives.
 
-Batching, pages, state slots, CUDA graphs and the public operations are ``PagedEngine``'s.  Three kinds of residual step: with a norm on both
-sides of every sublayer, ``norm_residual`` (the previous sublayer's norm, the residual sum, this one's norm, in one pass) takes the fp32 row an
+Batching, pages, state slots, CUDA graphs and the public operations are ``PagedEngine``'s.  Three kinds of residual step: with a norm behind
+every sublayer, and possibly one ahead, ``norm_residual`` (the previous sublayer's norm, the residual sum, this one's norm, in one pass) takes the fp32 row an
 output projection left; with a norm ahead only (Dynamic Tanh), the output projection adds its scaled product into the residual itself and
 ``norm_dyt`` reads it; with parallel sublayers and a depth average, both output projections add their products, scaled per channel, into the layer's
 row of a history, and ``depth_norm`` makes the next layer's row and its two norms out of that history.  Per sublayer one fused projection (queries, keys, values, gates, latents in one matrix), the mixer, and the output
@@ -35,6 +36,8 @@ MIXED_CTAS = 592             # most CTAs of a mixed-head decode launch that spli
 LATENT_CTAS = 592            # most CTAs of a latent decode launch that splits the keys
 DEPTH_GROUP = 4              # depth averages that share one reading of the results so far
 MOE_EXPERTS, MOE_TOP = 256, 32   # most experts of a layer, and of a token
+DELTA_DIM, DELTA_RANK = 256, 1024    # largest heads of the delta rule, and rank of its decay
+SSD_DIM = 256                # largest state and value sizes of a state-space head
 SHORT_TOKENS = 16            # latent attention: entries of up to this many new tokens work in the latent space
 ALONE = ("polynorm", "swiglu")   # activations that are no epilogue of the up projection
 ACTS = {None: (ops.EPI_STORE, ops.ACT_NONE, 0), "relu2": (ops.EPI_RELU2, ops.ACT_RELU2, 1), "gelu": (ops.EPI_GELU_ERF, ops.ACT_GELU_ERF, 2)}
@@ -42,6 +45,11 @@ ACTS = {None: (ops.EPI_STORE, ops.ACT_NONE, 0), "relu2": (ops.EPI_RELU2, ops.ACT
 
 def _up(n: int, m: int) -> int:
     return (n + m - 1) // m * m
+
+
+def _state_pad(vdim: int) -> int:
+    """Columns of a state row: multiples of 8; wide ones divide among the CTAs of a cluster."""
+    return _up(vdim, 8 if vdim <= 128 else 32)
 
 
 @dataclass
@@ -88,14 +96,33 @@ class _Experts:
     """A mixture's weights; F: the experts' width, padded."""
     F: int
     router: torch.Tensor         # fp32 [E][dp]
-    w13: torch.Tensor            # bf16 [E * 2 F][dp], rows interleaved (gate, up)
+    w13: torch.Tensor            # bf16 [E * 2 F][dp], rows interleaved (gate, up); experts without a gate: [E * F][dp]
     w2: torch.Tensor             # bf16 [E * dp][F]
+
+
+@dataclass
+class _Delta:
+    """A delta-rule mixer's own weights; offs: columns of r, k, v, the output gate, the removal rate and the low-rank decay input."""
+    offs: tuple[int, ...]
+    w2: torch.Tensor             # bf16 [heads * dim][rank padded to 8]
+    w0: torch.Tensor
+    rate: torch.Tensor
+
+
+@dataclass
+class _Ssd:
+    """A Mamba-2 mixer's own weights."""
+    conv: torch.Tensor           # fp32 [channels][taps]
+    conv_b: torch.Tensor
+    dt_bias: torch.Tensor
+    A_log: torch.Tensor
+    D: torch.Tensor
 
 
 @dataclass
 class _Block:
     spec: LayerSpec
-    norm1: _Norm
+    norm1: _Norm | None
     norm1b: _Norm | None
     proj: _Lin
     out: _Lin
@@ -107,6 +134,11 @@ class _Block:
     lam: torch.Tensor | None = None
     sink: torch.Tensor | None = None
     lat: _Latent | None = None
+    delta: _Delta | None = None
+    ssd: _Ssd | None = None
+    q_norm: torch.Tensor | None = None           # norms of whole projections
+    k_norm: torch.Tensor | None = None
+    v_mix: torch.Tensor | None = None            # the share of the first mixing layer's values (that layer itself: None)
     table: torch.Tensor | None = None
     a2: torch.Tensor | None = None
     b2: torch.Tensor | None = None
@@ -134,6 +166,7 @@ class _Run:
     joins: bool
     kv: int = -1                 # index among the key / value caches (latent mixers: among the latent caches)
     state: torch.Tensor | None = None
+    ring: torch.Tensor | None = None             # ssd: the latest inputs of the filter, by position
 
 
 @dataclass
@@ -166,7 +199,7 @@ def plan_latent_batch(q_len: list[int], ctx: list[int], short_rows: int, ctx_row
 
 
 class HybridEngine(PagedEngine):
-    ARCHS = ("folirax", "pesorax", "kazolorn")
+    ARCHS = ("folirax", "pesorax", "kazolorn", "tekosun")
     world = 1                    # one GPU; the serving layer asks
     vocab_sharded = False
 
@@ -181,14 +214,16 @@ class HybridEngine(PagedEngine):
         slots = 0 if not cfg.has_state else (state_slots if state_slots is not None else max_batch + max(4, max_batch // 4))
         self._init_paged(device, max_batch, max_ctx, n_pages, max_tokens, canaries, state_slots=slots)
         self.dp = _up(self.d, 8)
-        # Dynamic Tanh has no statistics of a row, so the residual itself can carry the padding (zeros stay zeros)
-        self.dx = self.dp if cfg.norm != "rms" else self.d
+        # Dynamic Tanh and the depth average read whole rows element by element, so the residual itself can carry the padding (zeros stay zeros)
+        self.dx = self.dp if not cfg.post_norm else self.d
         self.parallel = cfg.walk == "parallel"
-        if self.parallel != cfg.depth_average or cfg.layer_scale != cfg.depth_average or (cfg.norm == "rms1") != self.parallel or \
+        if self.parallel != cfg.depth_average or cfg.layer_scale != cfg.depth_average or (self.parallel and cfg.norm != "rms1") or \
                 (self.parallel and cfg.loop is not None) or any(l.act in ALONE or l.mixer.out_bias for l in cfg.layers) and not self.parallel:
             raise ValueError("a depth average goes with parallel sublayers, layer scales and norms stored as they are, without a loop")
-        if cfg.post_norm != (cfg.norm == "rms") or (cfg.post_norm and cfg.loop is not None):
-            raise ValueError("norms on both sides go with RMS norms and without a loop, Dynamic Tanh with a norm ahead only")
+        if cfg.post_norm != (cfg.norm != "dyt" and not self.parallel) or (cfg.post_norm and cfg.loop is not None) or not (cfg.pre_norm or cfg.post_norm):
+            raise ValueError("a norm behind every sublayer goes with RMS norms and without a loop, Dynamic Tanh with a norm ahead only")
+        if any(l.moe is not None for l in cfg.layers) and not (self.parallel or cfg.post_norm):
+            raise ValueError("mixtures of experts go with parallel sublayers or a norm behind them")
         # Decode batches up to this size take the mat-vec kernels.  Measured (ms per step, one token, mat-vec / GEMM): width 2048
         # 1.04 / 1.30, width 4096 4.41 / 4.19; the GEMM costs the same at eight tokens, the mat-vec grows with each.
         self.small_path_tokens = min(MATVEC_MAX_TOKENS, int(os.environ.get("B200_SMALL_PATH_TOKENS", 1)))
@@ -216,6 +251,13 @@ class HybridEngine(PagedEngine):
             return _Norm(self._wide(w))
         return _Norm(self._wide(w), self._wide(self._vector(src, name + ".b")), self._vector(src, name + ".alpha"))
 
+    def _norms(self, src: WeightSource, name: str) -> tuple[_Norm | None, _Norm | None]:
+        """The norms ahead of a sublayer and behind it; where there are both, the second one's name ends with a b."""
+        if self.cfg.pre_norm and self.cfg.post_norm:
+            return self._norm(src, name), self._norm(src, name + "b")
+        n = self._norm(src, name)
+        return (n, None) if self.cfg.pre_norm else (None, n)
+
     def _wide(self, v: torch.Tensor) -> torch.Tensor:
         return torch.nn.functional.pad(v, (0, self.dp - self.d))
 
@@ -228,9 +270,9 @@ class HybridEngine(PagedEngine):
         """(cos, sin) of every position of the cache, shared by the layers with the same rotation."""
         if not m.rope_dims:
             return None
-        key = (m.rope_base, m.rope_dims)
+        key = (m.rope_base, m.rope_dims, m.rope_scaling, m.rows_normed)
         if key not in self._tables:
-            self._tables[key] = ops.rope_table(self.max_pages * PAGE, m.rope_dims, m.rope_base, self.device)
+            self._tables[key] = ops.rope_table(self.max_pages * PAGE, m.rope_dims, m.rope_base, self.device, m.rope_frequencies() if m.rows_normed else None)
         return self._tables[key]
 
     def _load(self, src: WeightSource):
@@ -241,16 +283,15 @@ class HybridEngine(PagedEngine):
         self._tables: dict[tuple, torch.Tensor] = {}
         for i, spec in enumerate(cfg.layers):
             p = f"l{i}."
-            b = {"gla": self._load_gla, "attention": self._load_attention, "latent": self._load_latent}[spec.mixer.kind](src, p + "mix.", spec)
-            b.norm1 = self._norm(src, p + "norm1")
-            if cfg.post_norm:
-                b.norm1b = self._norm(src, p + "norm1b")
+            load = {"gla": self._load_gla, "delta": self._load_delta, "ssd": self._load_ssd, "attention": self._load_attention, "latent": self._load_latent}
+            b = load[spec.mixer.kind](src, p + "mix.", spec)
+            b.norm1, b.norm1b = self._norms(src, p + "norm1")
             if spec.ffn:
-                b.norm2 = self._norm(src, p + "norm2")
-                if cfg.post_norm:
-                    b.norm2b = self._norm(src, p + "norm2b")
+                b.norm2, b.norm2b = self._norms(src, p + "norm2")
                 if spec.moe:
                     b.moe = self._load_experts(src, p + "mlp.", spec)
+                    if spec.moe.shared:
+                        b.up, b.down = (self._lin(self._matrix(src, f"{p}mlp.shared.{n}")) for n in ("up", "down"))
                 else:
                     b.up, b.down = self._lin(self._matrix(src, p + "mlp.up")), self._lin(self._matrix(src, p + "mlp.down"))
                 if spec.act == "polynorm":
@@ -271,8 +312,10 @@ class HybridEngine(PagedEngine):
         for i, joins in cfg.layer_runs():
             b, m = self.blocks[i], cfg.layers[i].mixer
             run = _Run(b, joins)
-            if m.kind == "gla":
+            if m.stateful:
                 run.state = torch.zeros((self.state_slots, m.heads, m.dim, b.DV), dtype=torch.float32, device=self.device)
+                if m.kind == "ssd":
+                    run.ring = torch.zeros((self.state_slots, m.conv, m.channels), dtype=torch.float32, device=self.device)
             else:
                 own = self.latent_specs if m.kind == "latent" else self.kv_specs
                 if m.kind == "attention" and m.kv_from is not None:
@@ -291,6 +334,27 @@ class HybridEngine(PagedEngine):
         b.a2 = src.get(p + "a2").to_float().to(self.device).t().contiguous()
         b.b2, b.o_norm = self._vector(src, p + "a2.b"), self._vector(src, p + "norm")
         b.out = self._out_proj(src, p + "o", m.heads, m.vdim, b.DV)
+        return b
+
+    def _load_delta(self, src: WeightSource, p: str, spec: LayerSpec) -> _Block:
+        m = spec.mixer
+        if max(m.dim, m.vdim) > DELTA_DIM or m.rank > DELTA_RANK:
+            raise ValueError(f"delta rule: heads of at most {DELTA_DIM} channels, ranks up to {DELTA_RANK}")
+        hd = m.heads * m.dim
+        b = _Block(spec, None, None, self._lin(torch.cat([self._matrix(src, p + n) for n in ("r", "k", "v", "g", "a", "w1")])), None, DV=_state_pad(m.vdim))
+        w2 = torch.nn.functional.pad(self._matrix(src, p + "w2"), (0, _up(m.rank, 8) - m.rank)).to(self.device).contiguous()
+        b.delta = _Delta(tuple(i * hd for i in range(6)), w2, self._vector(src, p + "w0"), self._vector(src, p + "a.b"))
+        b.o_norm = self._vector(src, p + "norm")
+        b.out = self._out_proj(src, p + "o", m.heads, m.vdim, b.DV)
+        return b
+
+    def _load_ssd(self, src: WeightSource, p: str, spec: LayerSpec) -> _Block:
+        m = spec.mixer
+        if max(m.dim, m.vdim) > SSD_DIM:
+            raise ValueError(f"state-space layers: at most {SSD_DIM} state dimensions and value columns to a head")
+        b = _Block(spec, None, None, self._lin(self._matrix(src, p + "in")), self._lin(self._matrix(src, p + "o")), DV=_state_pad(m.vdim))
+        b.ssd = _Ssd(self._vector(src, p + "conv").view(m.channels, m.conv), *(self._vector(src, p + n) for n in ("conv.b", "dt_bias", "A_log", "D")))
+        b.o_norm = self._vector(src, p + "norm")
         return b
 
     def _load_attention(self, src: WeightSource, p: str, spec: LayerSpec) -> _Block:
@@ -322,6 +386,10 @@ class HybridEngine(PagedEngine):
             b.slopes = (slopes if b.mix is None else b.mix.double() @ slopes).float()
         if b.dec:
             b.mix_dec = ops.mixed_decode_prepare(b.mix, b.slopes, m.heads, m.kv_heads, b.DK)
+        if m.row_norm:
+            b.q_norm, b.k_norm = self._vector(src, p + "q.norm"), self._vector(src, p + "k.norm")
+        if m.v_mix and any(o.spec.mixer.v_mix for o in self.blocks):
+            b.v_mix = self._vector(src, p + "vmix")
         if m.silent_sink:
             b.silent = torch.zeros(m.heads, dtype=torch.float32, device=self.device)
         return b
@@ -330,11 +398,14 @@ class HybridEngine(PagedEngine):
         E, F, d, pad = spec.moe.experts, _up(spec.ffn, 16), self.d, torch.nn.functional.pad
         if E > MOE_EXPERTS or spec.moe.top > MOE_TOP:
             raise ValueError(f"at most {MOE_EXPERTS} experts, {MOE_TOP} of them per token")
-        w13 = torch.zeros((E, F, 2, self.dp), dtype=torch.bfloat16, device=self.device)
+        if (spec.act, spec.moe.weigh) not in (("swiglu", "input"), ("relu2", "output")):
+            raise ValueError(f"experts: {spec.act} with the weight on the {spec.moe.weigh} has no kernel")
+        parts = ["gate", "up"] if spec.act == "swiglu" else ["up"]
+        w13 = torch.zeros((E, F, len(parts), self.dp), dtype=torch.bfloat16, device=self.device)
         w2 = torch.zeros((E, self.dp, F), dtype=torch.bfloat16, device=self.device)
         for e in range(E):
-            w13[e, : spec.ffn, 0, :d] = self._matrix(src, f"{p}e{e}.gate").to(self.device)
-            w13[e, : spec.ffn, 1, :d] = self._matrix(src, f"{p}e{e}.up").to(self.device)
+            for i, n in enumerate(parts):
+                w13[e, : spec.ffn, i, :d] = self._matrix(src, f"{p}e{e}.{n}").to(self.device)
             w2[e, :d, : spec.ffn] = self._matrix(src, f"{p}e{e}.down").to(self.device)
         router = pad(self._vector(src, p + "router").view(E, d), (0, self.dp - d)).contiguous()
         return _Experts(F, router, w13.view(-1, self.dp), w2.view(-1, F))
@@ -428,6 +499,13 @@ class HybridEngine(PagedEngine):
         gla = [b for b in self.blocks if b.spec.mixer.kind == "gla"]
         self.gla_ws = ws("gla_ws", (max((ops.gla_chunk_bytes(T, self.max_batch, m.heads, m.dim, dv, m.rank)
                                          for m, dv in ((b.spec.mixer, b.DV) for b in gla)), default=0) if not self.exact else 0,), torch.uint8)
+        delta = [(b.spec.mixer, b.DV) for b in self.blocks if b.delta is not None]
+        self.delta_ws = ws("delta_ws", (max((ops.delta_chunk_bytes(T, self.max_batch, m.heads, m.dim, dv, m.log_decay) for m, dv in delta), default=0)
+                                        if not self.exact else 0,), torch.uint8)
+        ssd = [(b.spec.mixer, b.DV) for b in self.blocks if b.ssd is not None]
+        self.ssd_ws = ws("ssd_ws", (max((ops.ssd_prefill_bytes(T, self.max_batch, m.heads, dv, m.dim, m.groups, self.exact) for m, dv in ssd), default=0),), torch.uint8)
+        self.ssd_y = ws("ssd_y", (T * max((m.heads * m.vdim for m, _ in ssd), default=0),), f32)
+        self.v_first = ws("v_first", (T * max((m.kv_heads * m.vdim for _, m, _ in attn if m.v_mix), default=0),), f32)
         # latent attention: rows in the latent space (all of a step's where the any-size kernel runs), and the expanded context of the others
         self.short_rows = min(T, max(self.max_batch, 256))
         rows = lambda b: self.short_rows if b.tc else T                                      # noqa: E731
@@ -591,9 +669,15 @@ class HybridEngine(PagedEngine):
         vc = kc if m.tied_kv else self.vc[r.kv]
         tc_prompt, wide = b.tc and not decode, b.tc and decode and m.maps > 1
         q = (self.q16 if tc_prompt else self.q32)[: T * HQ * b.DK * (m.maps if wide else 1)].view(T, -1)
-        ops.qkv_finish(proj, 0, k_off, v_off, self.pos, self.slot, b.table, m.rope_base, HQ, m.kv_heads, m.dim, m.vdim, b.DK, b.DV,
-                       m.rope_dims, 0 if m.rope_style == "pairs" else 1, m.qk_norm, cfg.norm_eps, m.scale, PAGE, q32=None if tc_prompt else q,
-                       q16=q if tc_prompt else None, kc=kc, vc=vc, maps=m.maps, q_wide=wide, bias=b.bias)
+        if m.rows_normed:
+            first = self.v_first[: T * m.kv_heads * m.vdim] if m.v_mix else None
+            ops.row_qkv_finish(proj, 0, k_off, v_off, b.q_norm, b.k_norm, self.pos, self.slot, b.table, HQ, m.kv_heads, m.dim, m.vdim, b.DK, b.DV, m.rope_dims,
+                               0 if m.rope_style == "pairs" else 1, m.v_norm, cfg.norm_eps, m.scale, PAGE, kc, vc, q32=None if tc_prompt else q,
+                               q16=q if tc_prompt else None, lam=b.v_mix, v_first=first)
+        else:
+            ops.qkv_finish(proj, 0, k_off, v_off, self.pos, self.slot, b.table, m.rope_base, HQ, m.kv_heads, m.dim, m.vdim, b.DK, b.DV,
+                           m.rope_dims, 0 if m.rope_style == "pairs" else 1, m.qk_norm, cfg.norm_eps, m.scale, PAGE, q32=None if tc_prompt else q,
+                           q16=q if tc_prompt else None, kc=kc, vc=vc, maps=m.maps, q_wide=wide, bias=b.bias)
         gate = proj[:, g_off:] if m.head_gate else None
         out32, out16 = o32, o16
         if m.maps > 1:
@@ -682,6 +766,31 @@ class HybridEngine(PagedEngine):
         ops.gla_chunked(*args, max_q, self.gla_ws, out_f32=o32, out_bf16=o16)
         return 3
 
+    def _delta(self, r: _Run, proj, T: int, decode: bool, n_seqs: int, max_q: int, pages: int, o32, o16) -> int:
+        b, m, w = r.block, r.block.spec.mixer, r.block.delta
+        qs, ql = (self.iota, self.ones) if decode else (self.q_start, self.q_len)
+        args = (proj, w.offs, m.rank, w.w2, w.w0, w.rate, b.o_norm, r.state, qs, ql, self.seq_lens, self.state_slot, n_seqs, m.heads, m.dim, m.vdim, b.DV,
+                m.log_decay, self.cfg.norm_eps, o32 if o32 is not None else o16)
+        if decode or self.exact or not ops.delta_chunk_bytes(T, n_seqs, m.heads, m.dim, b.DV, m.log_decay):
+            ops.delta_recurrent(*args)
+            return 1
+        ops.delta_chunked(*args, max_q=max_q, ws=self.delta_ws)
+        return 3
+
+    def _ssd(self, r: _Run, proj, T: int, decode: bool, n_seqs: int, max_q: int, pages: int, o32, o16) -> int:
+        b, m, w = r.block, r.block.spec.mixer, r.block.ssd
+        inner = m.heads * m.vdim
+        y = self.ssd_y[: T * inner].view(T, inner)
+        qs, ql = (self.iota, self.ones) if decode else (self.q_start, self.q_len)
+        args = (proj, inner, inner + m.channels, w.conv, w.conv_b, w.dt_bias, w.A_log, w.D, r.state, r.ring, qs, ql, self.seq_lens, self.state_slot, n_seqs,
+                m.heads, m.vdim, m.dim, m.groups, b.DV, y)
+        if decode:
+            ops.ssd_decode(*args)
+        else:
+            ops.ssd_prefill(*args, max_q=max_q, ws=self.ssd_ws, exact=self.exact)
+        ops.group_norm(y, inner, m.norm_groups, b.o_norm, self.cfg.norm_eps, o32 if o32 is not None else o16, gate=proj[:, :inner])
+        return 2 if decode else 3 if self.exact else 4
+
     def _run_layers(self, T: int, decode: bool, n_seqs: int, max_q: int, pages: int) -> int:
         f32 = self.exact or (decode and T <= min(self.small_path_tokens, self.matvec_rows))
         walk = self._walk_parallel if self.parallel else self._walk_sandwich if self.cfg.post_norm else self._walk_prenorm
@@ -695,29 +804,34 @@ class HybridEngine(PagedEngine):
         return h, dict(hf=h) if f32 else dict(hb=h), views
 
     def _mix(self, r: _Run, proj, mix, T: int, f32: bool, step) -> int:
-        fn = {"gla": self._gla, "attention": self._attention, "latent": self._latent}[r.block.spec.mixer.kind]
+        fn = {"gla": self._gla, "delta": self._delta, "ssd": self._ssd, "attention": self._attention, "latent": self._latent}[r.block.spec.mixer.kind]
         return fn(r, proj, T, *step, mix if f32 else None, None if f32 else mix)
 
     def _walk_sandwich(self, T: int, decode: bool, f32: bool, step) -> int:
-        """A norm on both sides of every sublayer: each residual step waits for the next norm."""
+        """A norm behind every sublayer, and possibly one ahead (else the next sublayer reads the residual itself): each residual step waits for what comes next."""
         eps, x, y = self.cfg.norm_eps, self.x[:T], self.y[:T]
         h, hk, views = self._buffers(T, f32)
         add = not f32 and T <= QGEMM_MAX_TOKENS          # one row tile: the projections may split K and add into zeroed outputs
         gy, n = None, 0
-        for r in self.runs:
+        gain = lambda norm: None if norm is None else norm.w                                 # noqa: E731
+        for i, r in enumerate(self.runs):
             b = r.block
             proj, mix, act = views(b)
-            ops.norm_residual(x, eps, y=y if gy is not None else None, gy=gy, gh=b.norm1.w, y_clear=add, zero=proj if add else None,
+            ops.norm_residual(x, eps, y=y if gy is not None else None, gy=gy, gh=gain(b.norm1), y_clear=add, zero=proj if add else None,
                               zero2=y if add and gy is None else None, **hk)
             self._mm(h, b.proj, proj, add=add)
             n += self._mix(r, proj, mix, T, f32, step)
             self._mm(mix, b.out, y, add=add)
             gy, n = b.norm1b.w, n + 3
-            if act is not None:
-                ops.norm_residual(x, eps, y=y, gy=gy, gh=b.norm2.w, y_clear=add, **hk)
-                self._mm(h, b.up, act, act=b.spec.act)
-                self._mm(act, b.down, y, add=add)
-                gy, n = b.norm2b.w, n + 3
+            if b.norm2b is not None:
+                ops.norm_residual(x, eps, y=y, gy=gy, gh=gain(b.norm2), y_clear=add or act is None, **hk)
+                if act is not None:                      # one feed-forward, or the shared one of a mixture
+                    self._mm(h, b.up, act, act=b.spec.act)
+                    self._mm(act, b.down, y, add=add)
+                    n += 2
+                if b.moe is not None:                    # the chosen experts add to it
+                    n += self._experts(b, h, y, i)
+                gy, n = b.norm2b.w, n + 1
         if decode:
             self._tail = gy                              # the last residual step is folded into the final norm
         else:
@@ -788,22 +902,25 @@ class HybridEngine(PagedEngine):
         return n + 1
 
     def _experts(self, b: _Block, h, out, run: int) -> int:
-        """The chosen experts' sum, scaled per channel, into ``out``: fp32 rows by mat-vecs, bf16 rows gathered by expert and by grouped GEMMs."""
-        T, top, x = h.shape[0], b.spec.moe.top, b.moe
+        """The chosen experts' sum, scaled per channel where the layer has that, added to ``out``: fp32 rows by mat-vecs, bf16 rows gathered by expert and by grouped GEMMs."""
+        T, m, x = h.shape[0], b.spec.moe, b.moe
+        top, gated = m.top, b.spec.act == "swiglu"
+        how = dict(score=ops.SCORE_SIGMOID if m.score == "sigmoid" else ops.SCORE_SOFTMAX, scale=m.scale)
         ids, w = self.topk_ids[: T * top].view(T, top), self.topk_w[: T * top].view(T, top)
         if h.dtype == torch.float32:
             mid = self.mid[: T * top * x.F]
-            ops.moe_choose(h, x.router, top, ids, w, score=ops.SCORE_SIGMOID)
-            ops.expert_gate_up(h, x.w13, x.F, ids, w, mid)
+            ops.moe_choose(h, x.router, top, ids, w, **how)
+            (ops.expert_gate_up if gated else ops.expert_up)(h, x.w13, x.F, ids, w, mid)
             ops.expert_down(mid, x.w2, self.dp, ids, out, scale=b.ls2)
             return 3
         E, counts = b.spec.moe.experts, self.expert_counts[run]
         ops.moe_route_dispatch(h, None, x.router, None, top, E, self.cap, self.recv_x.data_ptr(), self.recv_meta.data_ptr(), self.recv_w.data_ptr(),
-                               counts.data_ptr(), None, topk_ids=ids, topk_w=w, status=self.status, score=ops.SCORE_SIGMOID)
-        ops.moe_gemm(self.recv_x, x.w13, E, self.cap, 2 * x.F, self.dp, counts, 1, out_bf16=self.recv_mid, ldc=x.F, gate_w=self.recv_w, status=self.status,
-                     live_rows=T * top)
+                               counts.data_ptr(), None, topk_ids=ids, topk_w=w, status=self.status, **how)
+        on = m.weigh == "input"                          # where the weights of the choice go
+        ops.moe_gemm(self.recv_x, x.w13, E, self.cap, (2 if gated else 1) * x.F, self.dp, counts, 1 if gated else 3, out_bf16=self.recv_mid, ldc=x.F,
+                     gate_w=self.recv_w if on else None, status=self.status, live_rows=T * top)
         ops.moe_gemm(self.recv_mid, x.w2, E, self.cap, self.dp, x.F, counts, 2, ldc=self.dp, meta=self.recv_meta, sym_off=out.data_ptr(), col_scale=b.ls2,
-                     status=self.status, live_rows=T * top)
+                     gate_w=None if on else self.recv_w, status=self.status, live_rows=T * top)
         return 3
 
     def _dyt(self, x, norm: _Norm, emb=None, **kw):
@@ -817,7 +934,7 @@ class HybridEngine(PagedEngine):
         hk = dict(hf=h) if f32 else dict(hb=h)
         if self.cfg.norm == "dyt":
             self._dyt(rows, self.final_norm, **hk)
-        elif self.cfg.norm == "rms1":
+        elif self.parallel:
             ops.depth_norm(rows[None], self.d, eps, g1=self.final_norm.w, h1=h)
         else:
             ops.norm_residual(rows, eps, y=self.y[:nb] if gy is not None else None, gy=gy, gh=self.final_norm.w, **hk)
@@ -836,6 +953,7 @@ class HybridEngine(PagedEngine):
         return n
 
     def _embed(self, T: int):
-        if self.parallel and any(b.moe is not None for b in self.blocks) and not self.exact:
+        if any(b.moe is not None for b in self.blocks) and not self.exact:
             ops.moe_zero(self.expert_counts)
-        ops.embedding(self.ids, self.hist[0, :T] if self.parallel else self.x[:T], ops.EMB_BF16, self.emb, vocab_n=self.V)
+        ops.embedding(self.ids, self.hist[0, :T] if self.parallel else self.x[:T], ops.EMB_BF16, self.emb, vocab_n=self.V,
+                      scale=self.cfg.embed_scale)

@@ -440,7 +440,7 @@ class PagedEngine:
             B, P = self.max_batch, self.max_pages
             pin = lambda *shape, dt=torch.int32: torch.zeros(shape, dtype=dt).pin_memory() if torch.cuda.is_available() else torch.zeros(shape, dtype=dt)
             self._stg = {"seq": pin(B, dt=torch.int64), "ids": pin(B), "pos": pin(B), "slot": pin(B), "ctx": pin(B), "table": pin(B, P),
-                         "out": pin(B), "last_batch": None}
+                         "out": pin(B), "last_batch": None, "copied": torch.cuda.Event() if torch.cuda.is_available() else None}
         return self._stg
 
     @torch.no_grad()
@@ -453,6 +453,8 @@ class PagedEngine:
         if B > self.max_batch:
             raise ValueError("batch exceeds the engine's workspace")
         st = self._decode_staging()
+        if st["copied"] is not None:              # the arrays are rewritten only once the previous step's copies have left them
+            st["copied"].synchronize()
         batch = tuple(seq_ids)
         same = st["last_batch"] == batch
         if not same:
@@ -483,6 +485,8 @@ class PagedEngine:
             upload()
             self._graphs[key] = self._capture(B, bucket)
         upload()
+        if st["copied"] is not None:
+            st["copied"].record()
         g, n = self._graphs[key]
         g.replay()
         self.launches_per_decode = n

@@ -79,7 +79,7 @@ def hybrid_tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
     for i, l in enumerate(cfg.layers):
         p, m = f"l{i}.", l.mixer
         for n in ("norm1", "norm2") if l.ffn else ("norm1",):
-            s += norm(p + n) + (norm(p + n + "b") if cfg.post_norm else [])
+            s += norm(p + n) + (norm(p + n + "b") if cfg.post_norm and cfg.pre_norm else [])
         p += "mix."
         if m.kind == "latent":
             qk = m.dim + m.rot_dim
@@ -91,6 +91,16 @@ def hybrid_tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
                 s.append(TensorSpec(p + "sink", (m.heads,), "bias"))
             if m.out_gate:
                 s.append(TensorSpec(p + "g", (m.heads * m.vdim, d), "matrix"))
+        elif m.kind == "delta":
+            hd = m.heads * m.dim
+            s += [TensorSpec(p + n, (hd, d), "matrix") for n in ("r", "k", "v", "g", "a")]
+            s += [TensorSpec(p + "a.b", (hd,), "bias"), TensorSpec(p + "w1", (m.rank, d), "matrix"), TensorSpec(p + "w2", (hd, m.rank), "matrix"),
+                  TensorSpec(p + "w0", (hd,), "bias"), TensorSpec(p + "norm", (hd,), "norm")]
+        elif m.kind == "ssd":
+            inner = m.heads * m.vdim
+            s += [TensorSpec(p + "in", (inner + m.channels + m.heads, d), "matrix"), TensorSpec(p + "conv", (m.channels, m.conv), "sink"),
+                  TensorSpec(p + "conv.b", (m.channels,), "bias"), TensorSpec(p + "dt_bias", (m.heads,), "bias"), TensorSpec(p + "A_log", (m.heads,), "bias"),
+                  TensorSpec(p + "D", (m.heads,), "norm"), TensorSpec(p + "norm", (inner,), "norm")]
         else:
             s.append(TensorSpec(p + "q", (m.maps * m.heads * m.dim, d), "matrix"))
         if m.kind == "gla":
@@ -106,6 +116,10 @@ def hybrid_tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
                     s += [TensorSpec(p + n, (rows, d), "matrix")] + ([TensorSpec(f"{p}{n}.b", (rows,), "bias")] if m.bias else [])
             if m.head_gate:
                 s.append(TensorSpec(p + "g", (m.heads, d), "matrix"))
+            if m.row_norm:
+                s += [TensorSpec(p + "q.norm", (m.heads * m.dim,), "norm"), TensorSpec(p + "k.norm", (m.kv_heads * m.dim,), "norm")]
+            if m.v_mix:
+                s.append(TensorSpec(p + "vmix", (1,), "sink"))
             if m.maps == 2:
                 s += [TensorSpec(p + n, (m.dim,), "bias") for n in ("lq1", "lk1", "lq2", "lk2")]
             if m.mix_heads:
@@ -115,8 +129,9 @@ def hybrid_tensor_specs(cfg: ModelConfig) -> list[TensorSpec]:
             s.append(TensorSpec(p + "o.b", (d,), "bias"))
         p = f"l{i}.mlp."
         if l.moe:
-            for e in range(l.moe.experts):
-                s += [TensorSpec(f"{p}e{e}.{n}", shape, "matrix") for n, shape in (("gate", (l.ffn, d)), ("up", (l.ffn, d)), ("down", (d, l.ffn)))]
+            parts = (["gate"] if l.act == "swiglu" else []) + ["up", "down"]
+            for e, f in [(f"e{e}", l.ffn) for e in range(l.moe.experts)] + ([("shared", l.moe.shared)] if l.moe.shared else []):
+                s += [TensorSpec(f"{p}{e}.{n}", (d, f) if n == "down" else (f, d), "matrix") for n in parts]
             s.append(TensorSpec(p + "router", (l.moe.experts, d), "router"))
         elif l.ffn:
             s += [TensorSpec(p + "up", (l.ffn, d), "matrix"), TensorSpec(p + "down", (d, l.ffn), "matrix")]

@@ -21,13 +21,15 @@ SCORE_SOFTMAX, SCORE_SIGMOID = 0, 1
 ACT_NONE, ACT_GELU, ACT_SWIGLU_PAIR, ACT_RELU2, ACT_GELU_ERF = 0, 1, 2, 3, 4
 
 _P = c_void_p
+_DELTA = [_P, c_int, _P, c_int, _P, c_int] + [_P] * 8 + [c_int] * 5 + [c_float, c_float, _P, _P, c_int]
+_SSD = [_P, c_int, c_int, c_int] + [_P] * 11 + [c_int] * 7 + [_P, c_int]
 _SIGS = {
-    "b200_embedding": [_P, _P, c_int, c_int, c_int, _P, _P, c_int, c_int, _P],
+    "b200_embedding": [_P, _P, c_int, c_int, c_int, _P, _P, c_int, c_int, c_float, _P],
     "b200_rmsnorm": [_P, _P, c_float, c_int, c_int, _P, _P, _P, _P, _P, _P, c_int, _P, c_long, c_size_t, c_int, _P, _P],
     "b200_rmsnorm_allgather": [_P, _P, c_float, c_int, c_int, c_int, c_size_t, _P, _P],
     "b200_quantize_x": [_P, c_int, c_int, _P, _P, _P, _P],
     "b200_rope_kv": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, _P, c_int, _P],
-    "b200_rope_table": [_P, c_int, c_int, c_float, _P],
+    "b200_rope_table": [_P, c_int, c_int, c_float, _P, _P],
     "b200_swiglu": [_P, c_int, c_int, _P, _P, c_int, _P],
     "b200_add_inplace": [_P, _P, c_size_t, _P],
     "b200_argmax": [_P, c_int, c_int, _P, _P, c_int, _P, _P],
@@ -48,8 +50,9 @@ _SIGS = {
     "b200_gemm_heads": [_P, _P] + [c_int] * 7 + [_P, _P, c_int, c_int, c_float, _P, c_int, c_int, _P, _P],
     "b200_moe_gemm": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, _P, _P, _P, c_size_t, _P, c_long, _P, _P],
     "b200_moe_route_dispatch": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_size_t, c_size_t, c_size_t, c_size_t,
-                                _P, _P, c_int, _P, _P, _P],
+                                _P, _P, c_int, c_float, _P, _P, _P],
     "b200_expert_gate_up": [_P, c_int, c_int, _P, c_int, _P, _P, c_int, _P, _P],
+    "b200_expert_up": [_P, c_int, c_int, _P, c_int, _P, _P, c_int, _P, _P],
     "b200_expert_down": [_P, c_int, c_int, _P, c_int, _P, c_int, _P, _P, c_int, _P],
     "b200_depth_norm": [_P, c_size_t, _P, c_int, c_int, c_int, c_int, _P, _P, _P, _P, c_float, _P, _P, _P, _P, _P, c_long, _P, _P, _P, c_int, c_int, _P],
     "b200_poly_norm": [_P, c_int, c_int, c_int, c_int, _P, c_float, _P, _P, c_int, _P],
@@ -85,6 +88,12 @@ _SIGS = {
     "b200_latent_decode": [_P, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, _P, _P],
     "b200_latent_decode_ok": [c_int, c_int, c_int],
     "b200_logits_finish": [_P, c_size_t, c_float, c_float, _P],
+    "b200_row_qkv_finish": [_P] + [c_int] * 5 + [_P] * 5 + [c_int] * 10 + [c_float, c_float, c_int] + [_P] * 6 + [c_int, _P],
+    "b200_group_norm": [_P, c_int, _P, c_int, c_int, c_int, c_int, _P, c_float, _P, _P, c_int, _P],
+    "b200_delta_recurrent": _DELTA + [_P],
+    "b200_delta_chunked": _DELTA + [c_int, c_int, _P, c_size_t, _P],
+    "b200_ssd_decode": _SSD + [_P],
+    "b200_ssd_prefill": _SSD + [c_int, c_int, c_int, _P, c_size_t, _P],
     "b200_gla_chunked": [_P] + [c_int] * 7 + [_P] * 8 + [c_int] * 5 + [c_float] * 3 + [_P, _P, c_int, c_int, c_int, _P, c_size_t, _P],
     "b200_gla_recurrent": [_P] + [c_int] * 7 + [_P] * 8 + [c_int] * 5 + [c_float] * 3 + [_P, _P, c_int, _P],
 }
@@ -110,6 +119,10 @@ def lib():
         L.b200_mixed_decode_scratch_floats.restype = c_size_t
         L.b200_mixed_decode_prepared_words.argtypes = [c_int] * 3
         L.b200_mixed_decode_prepared_words.restype = c_size_t
+        L.b200_delta_chunk_bytes.argtypes = [c_int] * 5 + [c_float]
+        L.b200_delta_chunk_bytes.restype = c_size_t
+        L.b200_ssd_prefill_bytes.argtypes = [c_int] * 7
+        L.b200_ssd_prefill_bytes.restype = c_size_t
         L.b200_gla_chunk_bytes.argtypes = [c_int] * 6
         L.b200_gla_chunk_bytes.restype = c_size_t
         _lib = L
@@ -138,10 +151,10 @@ def _check(rc: int, what: str):
         raise RuntimeError(f"{what} failed with code {rc}")
 
 
-def embedding(ids, out, emb_type, w, w2=None, vocab_lo=0, vocab_n=None):
+def embedding(ids, out, emb_type, w, w2=None, vocab_lo=0, vocab_n=None, scale=1.0):
     T, D = out.shape
     _check(lib().b200_embedding(_p(ids), _p(out), T, D, emb_type, _p(w), _p(w2), vocab_lo,
-                                vocab_n if vocab_n is not None else 2 ** 31 - 1, _st()), "embedding")
+                                vocab_n if vocab_n is not None else 2 ** 31 - 1, scale, _st()), "embedding")
 
 
 def rmsnorm(x, g, eps, xq=None, xd=None, xs16=None, hb=None, hf=None, signal_sym=None, zero=None, slots=None):
@@ -183,10 +196,12 @@ def rope_kv(qkv, pos, slot, q_out, q_out_h, kc, vc, Hq, Hkv, hd, page_size, thet
            "rope_kv")
 
 
-def rope_table(n_pos, hd, theta, device):
-    """fp32 [n_pos][hd/2][2] table of (cos, sin), computed in double precision on the device."""
+def rope_table(n_pos, hd, theta, device, freq=None):
+    """fp32 [n_pos][hd/2][2] table of (cos, sin), computed in double precision on the device; ``freq``: hd/2 frequencies (numbers) in place of the
+    powers of ``theta``."""
     tab = torch.empty((n_pos, hd // 2, 2), dtype=torch.float32, device=device)
-    _check(lib().b200_rope_table(_p(tab), n_pos, hd, theta, _st()), "rope_table")
+    f = None if freq is None else torch.tensor(freq, dtype=torch.float64, device=device)
+    _check(lib().b200_rope_table(_p(tab), n_pos, hd, theta, _p(f), _st()), "rope_table")
     return tab
 
 
@@ -341,19 +356,20 @@ def qgemm(w, x_bf16, T, out_f32=None, out_bf16=None, ldo=None, bias=None, epi=QE
 
 # ---------------------------------------------------------------- mixture of experts
 def moe_route_dispatch(h_bf16, h_f32, router_w, router_b, top_k, E_local, C, recv_x_off, recv_meta_off, recv_w_off, counts_off,
-                       sym, topk_ids=None, topk_w=None, status=None, score=SCORE_SOFTMAX):
-    """Router + top-k + weights (``score``: softmax over the chosen, or each one's sigmoid) + expert-parallel dispatch of ``h_bf16`` [T][d] (see
+                       sym, topk_ids=None, topk_w=None, status=None, score=SCORE_SOFTMAX, scale=1.0):
+    """Router + top-k + weights (``score``: softmax over the chosen, which is also the softmax over all of them renormalised, or each one's sigmoid; times
+    ``scale``) + expert-parallel dispatch of ``h_bf16`` [T][d] (see
     ``moe.cu``); the router (fp32 weights) reads ``h_f32`` when given.  ``sym`` None: one rank, the offsets are addresses."""
     T, d = (h_bf16 if h_bf16 is not None else h_f32).shape
     E = router_w.shape[0]
     _check(lib().b200_moe_route_dispatch(_p(h_bf16), _p(h_f32), _p(router_w), _p(router_b), T, d, E, top_k, E_local, C, recv_x_off,
-                                         recv_meta_off, recv_w_off, counts_off, _p(topk_ids), _p(topk_w), score, _sym(sym),
+                                         recv_meta_off, recv_w_off, counts_off, _p(topk_ids), _p(topk_w), score, scale, _sym(sym),
                                          _p(status), _st()), "moe_route_dispatch")
 
 
 def moe_gemm(A, B, groups, group_rows, N, K, counts, mode, out_bf16=None, ldc=0, meta=None, gate_w=None, sym=None,
              sym_off=0, status=None, lda=None, ldb=None, col_scale=None, live_rows=0):
-    """Grouped expert GEMM (see ``gemm_tc05.cu``): mode 1 = gate/up with fused SwiGLU, mode 2 = down
+    """Grouped expert GEMM (see ``gemm_tc05.cu``): mode 1 = gate/up with fused SwiGLU, mode 3 = up with the square of relu, mode 2 = down
     projection fused with the weighted combine into the source ranks' residual streams.  Mode 1 with ``gate_w``: the weight multiplies
     the expert's input.  Mode 2 without ``sym``: ``sym_off`` is the address of the fp32 [tokens, ldc] destination; ``col_scale`` [N] multiplies
     what is added.  ``live_rows``: the most rows all groups hold together."""
@@ -361,16 +377,22 @@ def moe_gemm(A, B, groups, group_rows, N, K, counts, mode, out_bf16=None, ldc=0,
                                ldc, _p(meta), _p(gate_w), _sym(sym), sym_off, _p(col_scale), live_rows, _p(status), _st()), "moe_gemm")
 
 
-def moe_choose(h, router_w, top_k, ids, w, score=SCORE_SOFTMAX):
+def moe_choose(h, router_w, top_k, ids, w, score=SCORE_SOFTMAX, scale=1.0):
     """The choice alone: expert ids (int32) and weights (fp32), [T, top_k], of the rows ``h`` (bf16 or fp32)."""
     f32, E = h.dtype == torch.float32, router_w.shape[0]
-    moe_route_dispatch(None if f32 else h, h if f32 else None, router_w, None, top_k, E, 0, 0, 0, 0, 0, None, topk_ids=ids, topk_w=w, score=score)
+    moe_route_dispatch(None if f32 else h, h if f32 else None, router_w, None, top_k, E, 0, 0, 0, 0, 0, None, topk_ids=ids, topk_w=w, score=score,
+                       scale=scale)
 
 
 def expert_gate_up(x, w13, F, ids, weights, mid):
     """``mid[t, s] = silu(w g) * (w u)`` for the chosen experts of fp32 rows ``x`` [T, K]; ``w13`` bf16 [E * 2 F, K], rows interleaved (gate, up); ``ids`` /
     ``weights`` [T, top] (None: weights of one)."""
     _check(lib().b200_expert_gate_up(_p(x), x.shape[0], x.shape[1], _p(w13), F, _p(ids), _p(weights), ids.shape[1], _p(mid), _st()), "expert_gate_up")
+
+
+def expert_up(x, w1, F, ids, weights, mid):
+    """``mid[t, s] = w relu(u)^2`` for the chosen experts (no gate) of fp32 rows ``x`` [T, K]; ``w1`` bf16 [E * F, K]."""
+    _check(lib().b200_expert_up(_p(x), x.shape[0], x.shape[1], _p(w1), F, _p(ids), _p(weights), ids.shape[1], _p(mid), _st()), "expert_up")
 
 
 def expert_down(mid, w2, N, ids, out, scale=None):
@@ -407,7 +429,7 @@ def count_mismatch(a, b) -> torch.Tensor:
 
 # ---------------------------------------------------------------- hybrid stacks (attention and recurrent layers, norms on both sides)
 def norm_residual(x, eps, y=None, gy=None, gh=None, hb=None, hf=None, y_clear=False, zero=None, zero2=None):
-    """``x += y / rms(y) * gy`` (with ``y``), then ``h = x / rms(x) * gh`` (with ``gh``) into ``hb`` (bf16) and/or ``hf`` (fp32), whose
+    """``x += y / rms(y) * gy`` (with ``y``), then ``h = x / rms(x) * gh`` (without ``gh``: ``h = x``) into ``hb`` (bf16) and/or ``hf`` (fp32), whose
     columns beyond x's width are written as zeros.  ``y_clear`` leaves y's rows zeroed; ``zero`` / ``zero2``: contiguous fp32
     tensors cleared on the side."""
     T, D = x.shape
@@ -599,3 +621,69 @@ def gla_chunked(proj, offs, rank, a2, b2, w, state, q_start, q_len, ctx_len, slo
     _check(lib().b200_gla_chunked(_p(proj), proj.stride(0), *offs, rank, _p(a2), _p(b2), _p(w), _p(state), _p(q_start), _p(q_len),
                                   _p(ctx_len), _p(slots), n_seqs, H, dim, vdim, VP, tau, q_scale, eps, _p(out_f32), _p(out_bf16),
                                   o.stride(0), proj.shape[0], max_q, _p(ws), ws.numel(), _st()), "gla_chunked")
+
+
+# ---------------------------------------------------------------- projections normed as whole rows, gated norm in parts
+def row_qkv_finish(proj, q_off, k_off, v_off, q_w, k_w, pos, slot, table, H, G, dim, vdim, DK, DV, rot, style, v_norm, eps, q_scale, page_size, kc, vc,
+                   q32=None, q16=None, lam=None, v_first=None):
+    """Queries and keys of a fused projection row, each normed over all its heads together (``q_w`` / ``k_w``: weights per column, None: not normed), rotated and
+    scaled; values normed per head (``v_norm``) and mixed, ``(1 - lam) v + lam v_first`` (without ``lam``: written to ``v_first``, fp32 [T, G * vdim], where
+    given); keys and values to the paged cache."""
+    _check(lib().b200_row_qkv_finish(_p(proj), proj.stride(0), proj.shape[0], q_off, k_off, v_off, _p(q_w), _p(k_w), _p(pos), _p(slot), _p(table),
+                                     0 if table is None else table.shape[0], H, G, dim, vdim, DK, DV, rot, style, int(v_norm), eps, q_scale, page_size,
+                                     _p(lam), _p(v_first), _p(q32), _p(q16), _p(kc), _p(vc), int(kc.dtype == torch.float32), _st()), "row_qkv_finish")
+
+
+def group_norm(y, D, groups, w, eps, out, gate=None):
+    """``v = y * silu(gate)`` (fp32 [T, >= D] views; ``gate`` None: ``v = y``), each of ``groups`` equal parts divided by its own root mean square, times ``w`` [D];
+    ``out`` bf16 or fp32, columns beyond D zero."""
+    f32 = out.dtype == torch.float32
+    _check(lib().b200_group_norm(_p(y), y.stride(0), _p(gate), 0 if gate is None else gate.stride(0), y.shape[0], D, groups, _p(w), eps,
+                                 None if f32 else _p(out), _p(out) if f32 else None, out.stride(0), _st()), "group_norm")
+
+
+# ---------------------------------------------------------------- generalized delta rule (see ``delta_rule.cu``)
+def _delta_args(proj, offs, rank, w2, w0, ab, norm, state, q_start, q_len, ctx_len, slots, n_seqs, H, dim, vdim, VP, decay, eps, out):
+    f32 = out.dtype == torch.float32
+    return (_p(proj), proj.stride(0), (c_int * 6)(*offs), rank, _p(w2), w2.shape[1], _p(w0), _p(ab), _p(norm), _p(state), _p(q_start), _p(q_len), _p(ctx_len),
+            _p(slots), n_seqs, H, dim, vdim, VP, decay, eps, _p(out) if f32 else None, None if f32 else _p(out), out.stride(0))
+
+
+def delta_recurrent(*args):
+    """Generalized delta rule token by token over every sequence's new tokens.  Arguments: the fused projections; ``offs``: their columns of r, k, v, the output
+    gate, the removal rate and the low-rank decay input; ``rank``; ``w2`` bf16 [H * dim, rank padded to 8]; ``w0`` and ``ab`` [H * dim]; ``norm`` [H * vdim];
+    ``state`` fp32 [slots, H, dim, VP]; q_start, q_len, ctx_len, slots; n_seqs, H, dim, vdim, VP; ``decay`` (log w = -decay * sigmoid); eps; ``out`` (bf16 or
+    fp32 [T, H * VP])."""
+    _check(lib().b200_delta_recurrent(*_delta_args(*args), _st()), "delta_recurrent")
+
+
+def delta_chunk_bytes(T, n_seqs, H, dim, VP, decay):
+    """Workspace of :func:`delta_chunked`; 0 for sizes it does not take."""
+    return lib().b200_delta_chunk_bytes(T, n_seqs, H, dim, VP, decay)
+
+
+def delta_chunked(*args, max_q, ws):
+    """:func:`delta_recurrent` for prompts, in 64-token chunks on the tensor cores; ``ws``: uint8 workspace."""
+    _check(lib().b200_delta_chunked(*_delta_args(*args), args[0].shape[0], max_q, _p(ws), ws.numel(), _st()), "delta_chunked")
+
+
+# ---------------------------------------------------------------- state-space duality (see ``ssd.cu``)
+def _ssd_args(proj, x_off, dt_off, conv, conv_b, dt_bias, A_log, D, state, ring, q_start, q_len, ctx_len, slots, n_seqs, H, P, N, G, PP, y):
+    return (_p(proj), proj.stride(0), x_off, dt_off, _p(conv), _p(conv_b), _p(dt_bias), _p(A_log), _p(D), _p(state), _p(ring), _p(q_start), _p(q_len), _p(ctx_len),
+            _p(slots), n_seqs, H, P, N, G, conv.shape[1], PP, _p(y), y.stride(0))
+
+
+def ssd_decode(*args):
+    """One token per sequence of a Mamba-2 layer: filter, recurrence and skip.  Arguments: the projections (fp32), their columns of [x, B, C] and of dt; ``conv`` fp32
+    [channels, taps] and its bias; dt_bias, A_log, D [H]; ``state`` fp32 [slots, H, N, PP]; ``ring`` fp32 [slots, taps, channels]; q_start, q_len, ctx_len,
+    slots; n_seqs, H, P, N, G, PP; ``y`` fp32 [T, >= H * P]."""
+    _check(lib().b200_ssd_decode(*_ssd_args(*args), _st()), "ssd_decode")
+
+
+def ssd_prefill_bytes(T, n_seqs, H, PP, N, G, exact=False):
+    return lib().b200_ssd_prefill_bytes(T, n_seqs, H, PP, N, G, int(exact))
+
+
+def ssd_prefill(*args, max_q, ws, exact=False):
+    """The same for prompts: 64-token chunks on the tensor cores, or (``exact``) token by token in fp32; ``ws``: uint8 workspace."""
+    _check(lib().b200_ssd_prefill(*_ssd_args(*args), args[0].shape[0], max_q, int(exact), _p(ws), ws.numel(), _st()), "ssd_prefill")
