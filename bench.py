@@ -112,7 +112,7 @@ def main():
         return
     if args.workload == "hybrid":
         import bench_hybrid
-        args.model = args.model if args.model.startswith(("folirax", "pesorax", "kazolorn")) else "folirax-8b-shape"
+        args.model = args.model if args.model.startswith(("folirax", "pesorax", "kazolorn", "tekosun")) else "folirax-8b-shape"
         print(json.dumps(bench_hybrid.run(args)))
         return
     if args.impl not in ("b200", "baseline"):

@@ -1,7 +1,7 @@
-"""Prefill and decode throughput of the hybrid engine (Folirax, Pesorax, Kazolorn) at a real model's layer sizes, beside the closest other engine at equal size:
+"""Prefill and decode throughput of the hybrid engine (Folirax, Pesorax, Kazolorn, Tekosun) at a real model's layer sizes, beside the closest other engine at equal size:
 the Llama engine, or, for a stack with experts, the mixture-of-experts engine.
 
-    python bench.py --workload hybrid [--model folirax-8b-shape | pesorax-8b-shape | kazolorn-8b-shape | kazolorn-moe-shape | ...] [--steps K] [--warmup W]
+    python bench.py --workload hybrid [--model folirax-8b-shape | pesorax-8b-shape | kazolorn-8b-shape | kazolorn-moe-shape | tekosun-8b-shape | ...] [--steps K] [--warmup W]
 
 Both engines hold bf16 random weights of the same width, feed-forward, head layout, depth and vocabulary, run the same prompts
 and batches, and are timed with CUDA events: a 2048-token prompt, four of them in one call, and decode steps (replayed graphs
@@ -353,6 +353,122 @@ def time_kazolorn_kernels(cfg, dev, reps: int = 12) -> list[dict]:
     return bench.rows
 
 
+def time_tekosun_kernels(cfg, dev, reps: int = 12) -> list[dict]:
+    """Every kernel that a Tekosun layer has and another engine's layer has not, at 2048 prompt tokens and at decode steps, and its counterpart: gated linear attention
+    of the same width (heads of 128 x 256) for the recurrences, the mixture-of-experts engine's kernels for the rest.  A recurrence's bytes are its projection
+    rows and outputs, and for decoding its state, read and written."""
+    from openagents_b200.ops import cuda_ops as ops
+    bench = _Timer(dev, reps)
+    dl, sd, at = (next(l.mixer for l in cfg.layers if l.mixer.kind == k) for k in ("delta", "ssd", "attention"))
+    mix = next(l for l in cfg.layers if l.moe)
+    d, T, B, ctx, eps = cfg.d_model, PROMPT, 64, PROMPT, 1e-6
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    rnd = lambda *s: torch.randn(*s, device=dev)                       # noqa: E731
+    bf = lambda *s: torch.randn(*s, device=dev).bfloat16()             # noqa: E731
+    hf = lambda *s: torch.randn(*s, device=dev).half()                 # noqa: E731
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)     # noqa: E731
+    for n in (T, B, 1):
+        x, y, hb, gn = rnd(n, d), rnd(n, d), bf(n, d), rnd(d)
+        bench(f"norm_residual behind only [{n}]", lambda: ops.norm_residual(x, eps, y=y, gy=gn, hb=hb), n * d * 14, like=f"rmsnorm [{n}]")
+        bench(f"rmsnorm [{n}]", lambda: ops.rmsnorm(x, gn, eps, hb=hb), n * d * 6)
+    # ---- recurrences
+    H, D, r = dl.heads, dl.dim, dl.rank
+    hd, ld = H * D, (5 * H * D + r + 7) // 8 * 8
+    w2, w0, ab, gain = bf(hd, (r + 7) // 8 * 8), rnd(hd) - 3, rnd(hd), rnd(hd)
+    Hg, dk, dv, rg = d // 256, 128, 256, 16
+    qk, vv = Hg * dk, Hg * dv
+    lg = (2 * qk + 2 * vv + rg + 7) // 8 * 8
+    go = (0, qk, 2 * qk, 2 * qk + vv, 2 * qk + 2 * vv)
+    a2, b2, wg = rnd(rg, qk), rnd(qk), rnd(dv)
+    Hs, P, N, G = sd.heads, sd.vdim, sd.dim, sd.groups
+    inner, ls = Hs * P, (sd.heads * sd.vdim + sd.channels + sd.heads + 7) // 8 * 8
+    conv, cb, dtb, A, skip, sn = rnd(sd.channels, sd.conv), rnd(sd.channels), rnd(Hs) - 3, rnd(Hs), rnd(Hs), rnd(inner)
+    offs = tuple(i * hd for i in range(6))
+    s1, s2, s3, ring = rnd(B, H, D, D), rnd(B, Hs, N, P), rnd(B, Hg, dk, dv), rnd(B, sd.conv, sd.channels)
+    for seqs in (1, 4):
+        n = seqs * T
+        qs, ql, sl = i32([T * b for b in range(seqs)]), i32([T] * seqs), i32(list(range(seqs)))
+        row, out = rnd(n, ld), bf(n, hd)
+        ws = torch.empty(ops.delta_chunk_bytes(n, seqs, H, D, D, dl.log_decay), dtype=torch.uint8, device=dev)
+        bench(f"delta_chunked [{seqs} x {T}] (3 kernels)", lambda: ops.delta_chunked(row, offs, r, w2, w0, ab, gain, s1, qs, ql, ql, sl, seqs, H, D, D, D, dl.log_decay, eps, out,
+                                                                                     max_q=T, ws=ws), n * (ld * 4 + hd * 2), like=f"gla_chunked [{seqs} x {T}] (3 kernels)")
+        row, y = rnd(n, ls), rnd(n, inner)
+        ws = torch.empty(ops.ssd_prefill_bytes(n, seqs, Hs, P, N, G), dtype=torch.uint8, device=dev)
+        bench(f"ssd_prefill [{seqs} x {T}] (3 kernels)", lambda: ops.ssd_prefill(row, inner, inner + sd.channels, conv, cb, dtb, A, skip, s2, ring, qs, ql, ql, sl, seqs, Hs, P, N, G, P, y,
+                                                                                 max_q=T, ws=ws), n * ((sd.channels + Hs) * 4 + inner * 4), like=f"gla_chunked [{seqs} x {T}] (3 kernels)")
+        row, out = rnd(n, lg), bf(n, vv)
+        ws = torch.empty(ops.gla_chunk_bytes(n, seqs, Hg, dk, dv, rg), dtype=torch.uint8, device=dev)
+        bench(f"gla_chunked [{seqs} x {T}] (3 kernels)", lambda: ops.gla_chunked(row, go, rg, a2, b2, wg, s3, qs, ql, ql, sl, seqs, Hg, dk, dv, dv, 16.0, dk ** -0.5, eps, T, ws, out_bf16=out),
+              n * (lg * 4 + vv * 2))
+    for n in (B, 1):
+        sl, one, held = i32(list(range(n))), i32([1] * n), i32([ctx] * n)
+        row, out = rnd(n, ld), bf(n, hd)
+        bench(f"delta_recurrent [{n}]", lambda: ops.delta_recurrent(row, offs, r, w2, w0, ab, gain, s1, sl, one, held, sl, n, H, D, D, D, dl.log_decay, eps, out),
+              n * (8 * H * D * D + ld * 4 + hd * 2) + w2.numel() * 2, like=f"gla_recurrent [{n}]")
+        row2, y = rnd(n, ls), rnd(n, inner)
+        bench(f"ssd_decode [{n}]", lambda: ops.ssd_decode(row2, inner, inner + sd.channels, conv, cb, dtb, A, skip, s2, ring, sl, one, held, sl, n, Hs, P, N, G, P, y),
+              n * (8 * Hs * N * P + (1 + sd.conv) * sd.channels * 4 + inner * 4), like=f"gla_recurrent [{n}]")
+        row3, out3 = rnd(n, lg), bf(n, vv)
+        bench(f"gla_recurrent [{n}]", lambda: ops.gla_recurrent(row3, go, rg, a2, b2, wg, s3, sl, one, held, sl, n, Hg, dk, dv, dv, 16.0, dk ** -0.5, eps, out_bf16=out3),
+              n * (8 * Hg * dk * dv + lg * 4))
+    for n in (T, B, 1):
+        y, z, o = rnd(n, inner), rnd(n, ls), bf(n, inner)
+        bench(f"group_norm gated [{n} x {inner}]", lambda: ops.group_norm(y, inner, sd.norm_groups, sn, eps, o, gate=z[:, :inner]), n * inner * 10, like=f"rmsnorm [{n}]")
+    # ---- attention's projections
+    Hq, G, D = at.heads, at.kv_heads, at.dim
+    nq, nk, pages = Hq * D, G * D, (ctx + 15) // 16
+    wq, wk, lam = rnd(nq), rnd(nk), torch.full((1,), 0.3, device=dev)
+    for n, seqs in ((T, 1), (B, B), (1, 1)):
+        row, first = rnd(n, nq + 2 * nk), rnd(n, nk)
+        pos, slot = i32([ctx - 1] * n if n != T else list(range(n))), i32(list(range(n)))
+        kc, vc = hf(seqs * pages + 1, G, 16, D), hf(seqs * pages + 1, G, 16, D)
+        q16, q32, tab = hf(n, nq), rnd(n, nq), ops.rope_table(ctx, at.rope_dims, at.rope_base, dev, at.rope_frequencies())
+        tabf = ops.rope_table(ctx, D, at.rope_base, dev)
+        q = dict(q16=q16) if n == T else dict(q32=q32)
+        nb = n * ((nq + 2 * nk) * 4 + nq * (2 if n == T else 4) + 2 * nk * 2)
+        bench(f"row_qkv_finish mixing [{n}]", lambda: ops.row_qkv_finish(row, 0, nq, nq + nk, wq, wk, pos, slot, tab, Hq, G, D, D, D, D, at.rope_dims, 1, True, eps, at.scale, 16, kc, vc,
+                                                                         lam=lam, v_first=first, **q), nb + n * nk * 4, like=f"rope_kv [{n}]")
+        bench(f"rope_kv [{n}]", lambda: ops.rope_kv(row, pos, slot, None if n == T else q32, q16 if n == T else None, kc, vc, Hq, G, D, 16, at.rope_base, 0, at.scale, table=tabf), nb)
+        del kc, vc
+    # ---- products
+    for n in (T, B):
+        a = bf(n, d)
+        for nm, cols in (("gemm delta projection", ld), ("gemm mamba projection", ls), ("gemm qkv", nq + 2 * nk)):
+            wt, o3 = bf(cols, d), torch.zeros(n, cols, device=dev)
+            bench(f"{nm} [{n}]", lambda: ops.gemm_bf16(a, wt, n, cols, d, out_f32=o3, accumulate=n <= 64, status=st), cols * d * 2 + n * (d * 2 + cols * 4), 2.0 * n * cols * d,
+                  like=None if nm == "gemm qkv" else f"gemm qkv [{n}]")
+    # ---- experts
+    E, top, F, scale = mix.moe.experts, mix.moe.top, mix.ffn, mix.moe.scale
+    w13, w1, w2e, router = bf(E * 2 * F, d) * 0.02, bf(E * F, d) * 0.02, bf(E * d, F) * 0.02, rnd(E, d) * 0.02
+    for n in (T, B):
+        cap = (n + 127) // 128 * 128
+        rx, mid, meta, rw = bf(E * cap, d), bf(E * cap, F), torch.zeros(E * cap, 2, dtype=torch.int32, device=dev), rnd(E * cap)
+        h, x, ids, w = bf(n, d), rnd(n, d), torch.zeros(n, top, dtype=torch.int32, device=dev), rnd(n, top)
+        cnt = torch.zeros(64, E, dtype=torch.int32, device=dev)
+        used = min(E, n * top)
+        for nm, sc, like in (("route and dispatch, scaled", scale, "route and dispatch"), ("route and dispatch", 1.0, None)):
+            cnt.zero_()
+            turn = iter(range(64))
+            bench(f"{nm} [{n}]", lambda: ops.moe_route_dispatch(h, None, router, None, top, E, cap, rx.data_ptr(), meta.data_ptr(), rw.data_ptr(), cnt[next(turn)].data_ptr(), None,
+                                                                topk_ids=ids, topk_w=w, status=st, scale=sc), n * d * 2 * (1 + top) + E * d * 4, like=like and f"{like} [{n}]")
+        bench(f"experts up, relu2 [{n}]", lambda: ops.moe_gemm(rx, w1, E, cap, F, d, cnt[0], 3, out_bf16=mid, ldc=F, status=st, live_rows=n * top),
+              used * F * d * 2 + n * top * (d + F) * 2, 2.0 * n * top * F * d, like=f"experts gate/up [{n}]")
+        bench(f"experts gate/up [{n}]", lambda: ops.moe_gemm(rx, w13, E, cap, 2 * F, d, cnt[0], 1, out_bf16=mid, ldc=F, status=st, live_rows=n * top),
+              used * 2 * F * d * 2 + n * top * (d + F) * 2, 4.0 * n * top * F * d)
+        bench(f"experts down [{n}]", lambda: ops.moe_gemm(mid, w2e, E, cap, d, F, cnt[0], 2, ldc=d, meta=meta, gate_w=rw, sym_off=x.data_ptr(), status=st, live_rows=n * top),
+              used * F * d * 2 + n * top * (F * 2 + d * 4), 2.0 * n * top * F * d)
+        Fs = mix.moe.shared
+        if Fs:
+            up, dn, act, y = bf(Fs, d), bf(d, Fs), bf(n, Fs), torch.zeros(n, d, device=dev)
+            bench(f"gemm shared up [{n}]", lambda: ops.gemm_bf16(h, up, n, Fs, d, out_bf16=act, act=ops.ACT_RELU2, status=st), (Fs * d + n * (d + Fs)) * 2, 2.0 * n * Fs * d, like=f"gemm qkv [{n}]")
+            bench(f"gemm shared down [{n}]", lambda: ops.gemm_bf16(act, dn, n, d, Fs, out_f32=y, accumulate=n <= 64, status=st), (Fs * d + n * Fs) * 2 + n * d * 4, 2.0 * n * Fs * d, like=f"gemm qkv [{n}]")
+    h, x, ids, w, mid = rnd(1, d), rnd(1, d), i32([list(range(top))]), rnd(1, top), rnd(1, top, F)
+    bench("expert_up [1]", lambda: ops.expert_up(h, w1, F, ids, w, mid), top * F * d * 2, like="expert_gate_up [1]")
+    bench("expert_gate_up [1]", lambda: ops.expert_gate_up(h, w13, F, ids, w, mid), top * 2 * F * d * 2)
+    bench("expert_down [1]", lambda: ops.expert_down(mid, w2e, d, ids, x), top * F * d * 2)
+    return bench.rows
+
+
 def time_kernels(cfg, dev, reps: int = 12) -> list[dict]:
     """Every kernel of one hybrid layer pair at 2048 prompt tokens and at a 64-sequence decode step, and its Llama counterpart."""
     from openagents_b200.ops import cuda_ops as ops
@@ -443,4 +559,4 @@ def run(args) -> dict:
     ours, llama = time_engine(cfg, dev, args.steps, max(3, args.warmup)), time_engine(llama_cfg, dev, args.steps, max(3, args.warmup))
     return {"workload": "hybrid", "model": cfg.name, "dtype": "bf16", "data": "synthetic", "prompt": PROMPT, "peaks": peaks()[2], "hybrid": ours,
             "moe_equal_size" if llama_cfg.n_experts else "llama_equal_size": llama,
-            "kernels": {"pesorax": time_pesorax_kernels, "kazolorn": time_kazolorn_kernels}.get(cfg.arch, time_kernels)(cfg, dev)}
+            "kernels": {"pesorax": time_pesorax_kernels, "kazolorn": time_kazolorn_kernels, "tekosun": time_tekosun_kernels}.get(cfg.arch, time_kernels)(cfg, dev)}

@@ -235,3 +235,83 @@ def generate(cfg, W, prompt, n):
         rows.append(row)
         row = forward(cfg, W, [ids[-1]], seq)[-1]
     return ids, torch.stack(rows)
+
+
+# ---------------------------------------------------------------- small random models
+def moe(ff, experts, top, scale=1.0, shared=24):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "scale": scale}, "shared": {"ff": shared} if shared else None}
+
+
+def layer_delta(dim, heads, mlp=None):
+    return {"type": "general_delta", "mixer": {"dim": dim, "heads": heads}, "mlp": mlp}
+
+
+def layer_mamba(heads, vdim, state, groups=1, norm_groups=1, conv=4, mlp=None):
+    return {"type": "mamba2", "mixer": {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "norm_groups": norm_groups, "conv": conv}, "mlp": mlp}
+
+
+def layer_attention(dim, vdim, heads, kv_heads, rot_dims, window=0, base=10000.0, scaling=None, scale=None, v_mix=True, mlp=None):
+    """``scaling``: (factor, low, high, original)."""
+    rot = {"base": base, "dims": rot_dims}
+    if scaling is not None:
+        rot["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    return {"type": "attention", "mlp": mlp, "mixer": {"dim": dim, "vdim": vdim, "heads": heads, "kv_heads": kv_heads, "rot": rot, "v_mix": v_mix,
+                                                       "scale": dim ** -0.5 if scale is None else scale, "mask": {"size": window} if window else None}}
+
+
+def config(layers, width, vocab, eps=1e-5, scale=1.0):
+    return {"architecture": "Tekosun", "layers": layers, "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": scale}}
+
+
+def random_weights(cfg, seed=0, rank=8):
+    """Seeded weights, rounded to bf16 (what a checkpoint holds), returned in float64."""
+    g = torch.Generator().manual_seed(seed)
+    W = {}
+
+    def put(name, *shape, std=None, mean=0.0):
+        s = shape[-1] ** -0.5 if std is None else std
+        W[name] = (torch.randn(shape, generator=g, dtype=torch.float64) * s + mean).to(torch.bfloat16).double()
+    d = cfg["width"]
+    put("embed", cfg["vocab"], d, std=1.0 / cfg["embedding"]["scale"])
+    for i, L in enumerate(cfg["layers"]):
+        p, mx, mlp = f"l{i}.", L["mixer"], L.get("mlp")
+        put(p + "norm1", d, std=0.2, mean=0.8)
+        if L["type"] == "general_delta":
+            hd = mx["heads"] * mx["dim"]
+            for n in ("r", "k", "v", "g", "a"):
+                put(f"{p}mix.{n}", hd, d)
+            put(p + "mix.a.b", hd, std=1.0, mean=0.5)
+            put(p + "mix.w1", rank, d)
+            put(p + "mix.w2", hd, rank, std=1.5 * rank ** -0.5)
+            put(p + "mix.w0", hd, std=2.0, mean=-3.0)
+            put(p + "mix.norm", hd, std=0.2, mean=1.0)
+            put(p + "mix.o", d, hd)
+        elif L["type"] == "mamba2":
+            H, inner = mx["heads"], mx["heads"] * mx["vdim"]
+            channels = inner + 2 * mx["groups"] * mx["state"]
+            put(p + "mix.in", inner + channels + H, d, std=1.3 * d ** -0.5)
+            put(p + "mix.conv", channels, mx["conv"], std=0.7)
+            put(p + "mix.conv.b", channels, std=0.3)
+            put(p + "mix.dt_bias", H, std=1.0, mean=-2.0)
+            put(p + "mix.A_log", H, std=1.0)
+            put(p + "mix.D", H, std=0.5, mean=0.5)
+            put(p + "mix.norm", inner, std=0.2, mean=1.0)
+            put(p + "mix.o", d, inner)
+        else:
+            H, G = mx["heads"], mx["kv_heads"]
+            for n, rows in (("q", H * mx["dim"]), ("k", G * mx["dim"]), ("v", G * mx["vdim"])):
+                put(f"{p}mix.{n}", rows, d)
+            put(p + "mix.q.norm", H * mx["dim"], std=0.5, mean=1.5)
+            put(p + "mix.k.norm", G * mx["dim"], std=0.5, mean=1.5)
+            if mx["v_mix"]:
+                W[p + "mix.vmix"] = torch.tensor(0.15 + 0.4 * torch.rand(1, generator=g).item(), dtype=torch.float64).to(torch.bfloat16).double()
+            put(p + "mix.o", d, H * mx["vdim"])
+        if mlp is not None:
+            put(p + "norm2", d, std=0.2, mean=0.8)
+            for e, ff in [(f"e{e}", mlp["expert"]["ff"]) for e in range(mlp["router"]["experts"])] + ([("shared", mlp["shared"]["ff"])] if mlp["shared"] else []):
+                put(f"{p}mlp.{e}.up", ff, d)
+                put(f"{p}mlp.{e}.down", d, ff)
+            put(p + "mlp.router", mlp["router"]["experts"], d, std=2.0 * d ** -0.5)
+    put("final.norm", d, std=0.3, mean=1.0)
+    put("head", cfg["vocab"], d, std=4.0 * d ** -0.5)
+    return W
