@@ -405,8 +405,8 @@ def time_tekosun_kernels(cfg, dev, reps: int = 12) -> list[dict]:
         row, out = rnd(n, ld), bf(n, hd)
         bench(f"delta_recurrent [{n}]", lambda: ops.delta_recurrent(row, offs, r, w2, w0, ab, gain, s1, sl, one, held, sl, n, H, D, D, D, dl.log_decay, eps, out),
               n * (8 * H * D * D + ld * 4 + hd * 2) + w2.numel() * 2, like=f"gla_recurrent [{n}]")
-        row2, y = rnd(n, ls), rnd(n, inner)
-        bench(f"ssd_decode [{n}]", lambda: ops.ssd_decode(row2, inner, inner + sd.channels, conv, cb, dtb, A, skip, s2, ring, sl, one, held, sl, n, Hs, P, N, G, P, y),
+        row2, y, ws = rnd(n, ls), rnd(n, inner), torch.empty(ops.ssd_decode_bytes(n, Hs, P, N, G), dtype=torch.uint8, device=dev)
+        bench(f"ssd_decode [{n}]", lambda: ops.ssd_decode(row2, inner, inner + sd.channels, conv, cb, dtb, A, skip, s2, ring, sl, one, held, sl, n, Hs, P, N, G, P, y, ws=ws),
               n * (8 * Hs * N * P + (1 + sd.conv) * sd.channels * 4 + inner * 4), like=f"gla_recurrent [{n}]")
         row3, out3 = rnd(n, lg), bf(n, vv)
         bench(f"gla_recurrent [{n}]", lambda: ops.gla_recurrent(row3, go, rg, a2, b2, wg, s3, sl, one, held, sl, n, Hg, dk, dv, dv, 16.0, dk ** -0.5, eps, out_bf16=out3),

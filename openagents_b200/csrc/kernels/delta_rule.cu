@@ -41,26 +41,46 @@ __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-
 
 // ------------------------------------------------------------------ token by token
 
-// Decoding, and the prompts of the 32-bit mode.  One cluster per (head, sequence), whose CTAs share the value columns.  A thread keeps R rows of one
-// float4 column of the state in registers over all tokens.  One pass over the old state gives both what the removal reads, u^T S, and the output's part
+// Decoding, and the prompts of the 32-bit mode.  One cluster per head and share of the sequences, whose CTAs share the value columns.  A CTA walks the tokens
+// of its sequences one by one; while it works on one, the projections of the next, and with a new sequence its state, are on their way into the other half of
+// a double buffer.  The state is updated in shared memory.  One pass over the old state gives both what the removal reads, u^T S, and the output's part
 // (r w)^T S; the rest of the output is two numbers per token:  o = (r w)^T S - (r . c) (u^T S) + (r . k) v.
-template <int R>
-__global__ void __launch_bounds__(256, R <= 8 ? 2 : 1) delta_recurrent_kernel(const DeltaArgs a) {
+__device__ __forceinline__ void cp_async4(void* dst, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(s32(dst)), "l"(src) : "memory");
+}
+struct DeltaLayout {                       // floats of shared memory
+  int state, row, ch, ur, x, read, red, total;      // offsets; state and row: of the first of two buffers
+  int state_n, row_n;                      // sizes of one buffer
+};
+__host__ __device__ inline DeltaLayout delta_layout(int dim, int W, int rank8) {
+  DeltaLayout l;
+  const int groups = 256 / (W / 4);
+  auto up4 = [](int n) { return (n + 3) & ~3; };
+  l.state_n = dim * W;
+  l.row_n = up4(3 * dim) + 2 * W + rank8;  // r k a | v g | x
+  l.state = 0;
+  l.row = 2 * l.state_n;
+  l.ch = l.row + 2 * l.row_n;
+  l.ur = l.ch + 4 * dim;
+  l.x = l.ur + up4(2 * dim);
+  l.read = l.x + rank8;
+  l.red = l.read + W;
+  l.total = l.red + groups * 2 * W;
+  return l;
+}
+__global__ void __launch_bounds__(256, 4) delta_recurrent_kernel(const DeltaArgs a, int n_seqs, const DeltaLayout l) {
   extern __shared__ __align__(16) float sm[];
   cg::cluster_group cluster = cg::this_cluster();
   const int CL = cluster.num_blocks(), part = cluster.block_rank();
   const int nv_all = a.VP >> 2, nv = nv_all / CL, W = nv * 4, e0 = part * W;     // this CTA's columns [e0, e0 + W)
   const int groups = 256 / nv;
-  float4* s_ch = (float4*)sm;              // [dim] (w, c, k, -)
-  float2* s_ur = (float2*)(s_ch + a.dim);  // [dim] (u, r w)
-  float* s_x = (float*)(s_ur + a.dim);     // [rank8]
-  float* s_v = s_x + a.rank8 + ((4 - ((2 * a.dim + a.rank8) & 3)) & 3);      // [W], 16-byte aligned
-  float* s_read = s_v + W;                 // [W]
-  float* s_red = s_read + W;               // [groups][2][W]
+  float4* s_ch = (float4*)(sm + l.ch);     // [dim] (w, c, k, -)
+  float2* s_ur = (float2*)(sm + l.ur);     // [dim] (u, r w)
+  float *s_x = sm + l.x, *s_read = sm + l.read, *s_red = sm + l.red;
   __shared__ float red[3][8], red1[32];
   __shared__ float s_part[2];              // this CTA's sum of squares, by token parity
   pdl_trigger();
-  const int h = blockIdx.x / CL, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int h = blockIdx.x / CL, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   // TPC threads share a channel's low-rank product; its weights are read while the projection still runs
   int TPC = 1;
   while (TPC < 8 && a.dim * TPC * 2 <= 256) TPC *= 2;
@@ -72,40 +92,97 @@ __global__ void __launch_bounds__(256, R <= 8 ? 2 : 1) delta_recurrent_kernel(co
   for (int i = 0; i < 4; i++) held[i] = mine && (sub + i * TPC) * 8 < a.rank8 ? ((const uint4*)wrow)[sub + i * TPC] : make_uint4(0u, 0u, 0u, 0u);
   const float w0 = mine ? a.w0[h * a.dim + ch] : 0.f, ab = mine ? a.ab[h * a.dim + ch] : 0.f;
   const float wo = (tid < W && e0 + tid < a.vdim) ? a.norm[h * a.vdim + e0 + tid] : 0.f;
-  pdl_wait();
-  const int n = a.q_len[b], t0 = a.q_start[b], slot = a.slot[b];
-  const bool fresh = a.ctx_len[b] - n == 0 || slot < 0;
-  const int grp = tid / nv, col = tid % nv;
+  const int grp = tid / nv, col = tid % nv, rka = (3 * a.dim + 3) & ~3;
   const bool active = grp < groups;
-  float4* S = (float4*)(a.state + ((size_t)max(slot, 0) * a.H + h) * a.dim * a.VP) + part * nv + col;
-  float4 st[R];
-#pragma unroll
-  for (int k = 0; k < R; k++) {
-    const int d = grp + k * groups;
-    st[k] = (active && !fresh && d < a.dim) ? S[(size_t)d * nv_all] : make_float4(0.f, 0.f, 0.f, 0.f);
+  pdl_wait();
+  struct Seq { int n, t0, slot; bool fresh; };
+  auto meta = [&](int b) {
+    Seq q = {0, 0, -1, true};
+    if (b < n_seqs) {
+      q.n = a.q_len[b];
+      q.t0 = a.q_start[b];
+      q.slot = a.slot[b];
+      q.fresh = a.ctx_len[b] - q.n == 0 || q.slot < 0;
+    }
+    return q;
+  };
+  auto state_of = [&](int slot) { return (float4*)(a.state + ((size_t)max(slot, 0) * a.H + h) * a.dim * a.VP) + part * nv; };
+  auto fetch_row = [&](int t, int buf) {
+    const float* src = a.in + (size_t)t * a.ld;
+    float* dst = sm + l.row + buf * l.row_n;
+    for (int d = tid; d < a.dim; d += 256) {
+      const int c = h * a.dim + d;
+      cp_async4(dst + d, src + a.r_off + c);
+      cp_async4(dst + a.dim + d, src + a.k_off + c);
+      cp_async4(dst + 2 * a.dim + d, src + a.a_off + c);
+    }
+    for (int e = tid; e < W; e += 256) {
+      const bool live = e0 + e < a.vdim;
+      const int c = h * a.vdim + e0 + e;
+      if (live) {
+        cp_async4(dst + rka + e, src + a.v_off + c);
+        cp_async4(dst + rka + W + e, src + a.g_off + c);
+      } else {
+        dst[rka + e] = dst[rka + W + e] = 0.f;
+      }
+    }
+    for (int r = tid; r < a.rank8; r += 256) {
+      if (r < a.rank) cp_async4(dst + rka + 2 * W + r, src + a.x_off + r);
+      else dst[rka + 2 * W + r] = 0.f;
+    }
+  };
+  auto fetch_state = [&](const Seq& q, int buf) {
+    float4* dst = (float4*)(sm + l.state + buf * l.state_n);
+    const float4* src = state_of(q.slot);
+    if (!active) return;
+    for (int d = grp; d < a.dim; d += groups) {          // the thread that will work on it: no barrier between this and its use but the copy's own
+      if (!q.fresh) cp_async16(s32(dst + d * nv + col), src + (size_t)d * nv_all + col);
+      else dst[d * nv + col] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  int b = blockIdx.y, i = 0, sbuf = 0, rbuf = 0, step = 0;
+  Seq cur = meta(b), nxt = meta(b + gridDim.y);
+  while (b < n_seqs && cur.n < 1) {         // an entry without tokens
+    b += gridDim.y;
+    cur = nxt;
+    nxt = meta(b + gridDim.y);
   }
-  for (int i = 0; i < n; i++) {
-    const float* row = a.in + (size_t)(t0 + i) * a.ld;
+  if (b < n_seqs) {
+    fetch_state(cur, 0);
+    fetch_row(cur.t0, 0);
+    cp_async_commit();
+  }
+  while (b < n_seqs) {
+    cp_async_wait_all();
+    __syncthreads();                       // this token's data has landed, and everyone is done with the other buffers
+    const bool last = i + 1 == cur.n;
+    if (!last) {
+      fetch_row(cur.t0 + i + 1, rbuf ^ 1);
+    } else if (b + gridDim.y < n_seqs && nxt.n > 0) {
+      fetch_state(nxt, sbuf ^ 1);
+      fetch_row(nxt.t0, rbuf ^ 1);
+    }
+    cp_async_commit();
+    const float* row = sm + l.row + rbuf * l.row_n;
+    const float *s_v = row + rka, *s_g = s_v + W;
+    float4* S = (float4*)(sm + l.state + sbuf * l.state_n) + col;
+    for (int r = tid; r < a.rank8; r += 256) s_x[r] = tanhf(row[rka + 2 * W + r]);
     float kk = 0.f, rr = 0.f, ar = 0.f;
     if (mine && sub == 0) {
-      const int c = h * a.dim + ch;
-      kk = row[a.k_off + c];
-      rr = row[a.r_off + c];
-      ar = row[a.a_off + c];
+      rr = row[ch];
+      kk = row[a.dim + ch];
+      ar = row[2 * a.dim + ch];
     }
-    const float gate = (tid < W && e0 + tid < a.vdim) ? row[a.g_off + h * a.vdim + e0 + tid] : 0.f;      // used at the end
-    for (int r = tid; r < a.rank8; r += 256) s_x[r] = r < a.rank ? tanhf(row[a.x_off + r]) : 0.f;
-    for (int e = tid; e < W; e += 256) s_v[e] = e0 + e < a.vdim ? row[a.v_off + h * a.vdim + e0 + e] : 0.f;
     __syncthreads();
     float z = 0.f;
     auto dot = [&](uint4 q, int at) {
       const __nv_bfloat162* p = (const __nv_bfloat162*)&q;
-#pragma unroll
-      for (int j = 0; j < 4; j++) {
-        const float2 f = __bfloat1622float2(p[j]);
-        z = fmaf(f.x, s_x[at + 2 * j], z);
-        z = fmaf(f.y, s_x[at + 2 * j + 1], z);
-      }
+      const float4 x0 = *(const float4*)(s_x + at), x1 = *(const float4*)(s_x + at + 4);
+      float2 f;
+      f = __bfloat1622float2(p[0]); z = fmaf(f.x, x0.x, z); z = fmaf(f.y, x0.y, z);
+      f = __bfloat1622float2(p[1]); z = fmaf(f.x, x0.z, z); z = fmaf(f.y, x0.w, z);
+      f = __bfloat1622float2(p[2]); z = fmaf(f.x, x1.x, z); z = fmaf(f.y, x1.y, z);
+      f = __bfloat1622float2(p[3]); z = fmaf(f.x, x1.z, z); z = fmaf(f.y, x1.w, z);
     };
 #pragma unroll
     for (int j = 0; j < 4; j++)
@@ -127,64 +204,79 @@ __global__ void __launch_bounds__(256, R <= 8 ? 2 : 1) delta_recurrent_kernel(co
     __syncthreads();
     if (active) {
       float4 rd = make_float4(0.f, 0.f, 0.f, 0.f), p = rd;
-#pragma unroll
-      for (int k = 0; k < R; k++) {
-        const int d = grp + k * groups;
-        if (d >= a.dim) break;
+#pragma unroll 4
+      for (int d = grp; d < a.dim; d += groups) {
         const float2 ur = s_ur[d];
-        rd.x = fmaf(ur.x, st[k].x, rd.x); rd.y = fmaf(ur.x, st[k].y, rd.y); rd.z = fmaf(ur.x, st[k].z, rd.z); rd.w = fmaf(ur.x, st[k].w, rd.w);
-        p.x = fmaf(ur.y, st[k].x, p.x); p.y = fmaf(ur.y, st[k].y, p.y); p.z = fmaf(ur.y, st[k].z, p.z); p.w = fmaf(ur.y, st[k].w, p.w);
+        const float4 x = S[d * nv];
+        rd.x = fmaf(ur.x, x.x, rd.x); rd.y = fmaf(ur.x, x.y, rd.y); rd.z = fmaf(ur.x, x.z, rd.z); rd.w = fmaf(ur.x, x.w, rd.w);
+        p.x = fmaf(ur.y, x.x, p.x); p.y = fmaf(ur.y, x.y, p.y); p.z = fmaf(ur.y, x.z, p.z); p.w = fmaf(ur.y, x.w, p.w);
       }
       *(float4*)(s_red + (size_t)(grp * 2) * W + 4 * col) = rd;
       *(float4*)(s_red + (size_t)(grp * 2 + 1) * W + 4 * col) = p;
     }
     __syncthreads();
     float ss = 0.f;
-    for (int e = tid; e < W; e += 256) {   // W <= 256: once
+    if (tid < W) {                         // W <= 256
       float rd = 0.f, p = 0.f;
+#pragma unroll 4
       for (int g = 0; g < groups; g++) {
-        rd += s_red[(size_t)(g * 2) * W + e];
-        p += s_red[(size_t)(g * 2 + 1) * W + e];
+        rd += s_red[(size_t)(g * 2) * W + tid];
+        p += s_red[(size_t)(g * 2 + 1) * W + tid];
       }
-      s_read[e] = rd;
-      const float o = p - rc * rd + rk * s_v[e];
-      s_red[e] = o;                        // this column's first partial sum has been read
-      ss += o * o;                         // padding columns are zero
+      s_read[tid] = rd;
+      const float o = p - rc * rd + rk * s_v[tid];
+      s_red[tid] = o;                      // this column's first partial sum has been read
+      ss = o * o;                          // padding columns are zero
     }
     ss = block_sum(ss, red1);              // its barriers also publish s_read
     if (active) {
       const float4 v = *(const float4*)(s_v + 4 * col), rd = *(const float4*)(s_read + 4 * col);
-#pragma unroll
-      for (int k = 0; k < R; k++) {
-        const int d = grp + k * groups;
-        if (d >= a.dim) break;
+      float4* dst = state_of(cur.slot) + col;
+      const bool keep = last && cur.slot >= 0;
+#pragma unroll 4
+      for (int d = grp; d < a.dim; d += groups) {
         const float4 c = s_ch[d];
-        st[k].x = fmaf(c.x, st[k].x, fmaf(c.z, v.x, -c.y * rd.x));
-        st[k].y = fmaf(c.x, st[k].y, fmaf(c.z, v.y, -c.y * rd.y));
-        st[k].z = fmaf(c.x, st[k].z, fmaf(c.z, v.z, -c.y * rd.z));
-        st[k].w = fmaf(c.x, st[k].w, fmaf(c.z, v.w, -c.y * rd.w));
+        float4 x = S[d * nv];
+        x.x = fmaf(c.x, x.x, fmaf(c.z, v.x, -c.y * rd.x));
+        x.y = fmaf(c.x, x.y, fmaf(c.z, v.y, -c.y * rd.y));
+        x.z = fmaf(c.x, x.z, fmaf(c.z, v.z, -c.y * rd.z));
+        x.w = fmaf(c.x, x.w, fmaf(c.z, v.w, -c.y * rd.w));
+        if (!last) S[d * nv] = x;
+        else if (keep) dst[(size_t)d * nv_all] = x;
       }
     }
     if (CL > 1) {
-      if (tid == 0) s_part[i & 1] = ss;
+      if (tid == 0) s_part[step & 1] = ss;
       cluster.sync();
       ss = 0.f;
-      for (int p = 0; p < CL; p++) ss += *cluster.map_shared_rank(&s_part[i & 1], p);
+      for (int p = 0; p < CL; p++) ss += *cluster.map_shared_rank(&s_part[step & 1], p);
     }
     const float r = 1.f / sqrtf(ss / (float)a.vdim + a.eps);
     if (tid < W) {
-      const float o = e0 + tid < a.vdim ? s_red[tid] * r * wo * sigmoid_f(gate) : 0.f;
-      const size_t at = (size_t)(t0 + i) * a.ldo + (size_t)h * a.VP + e0 + tid;
+      const float o = e0 + tid < a.vdim ? s_red[tid] * r * wo * sigmoid_f(s_g[tid]) : 0.f;
+      const size_t at = (size_t)(cur.t0 + i) * a.ldo + (size_t)h * a.VP + e0 + tid;
       if (a.out_f32) a.out_f32[at] = o;
       if (a.out_bf16) a.out_bf16[at] = __float2bfloat16(o);
     }
-    __syncthreads();
-  }
-  if (slot >= 0 && active) {
-#pragma unroll
-    for (int k = 0; k < R; k++) {
-      const int d = grp + k * groups;
-      if (d < a.dim) S[(size_t)d * nv_all] = st[k];
+    step++;
+    rbuf ^= 1;
+    i++;
+    if (last) {
+      i = 0;
+      sbuf ^= 1;
+      bool skipped = false;
+      do {                                 // past entries without tokens, whose successors were not fetched ahead
+        b += gridDim.y;
+        cur = nxt;
+        nxt = meta(b + gridDim.y);
+        if (b < n_seqs && cur.n < 1) skipped = true;
+      } while (b < n_seqs && cur.n < 1);
+      if (skipped && b < n_seqs) {
+        __syncthreads();
+        fetch_state(cur, sbuf);
+        fetch_row(cur.t0, rbuf);
+        cp_async_commit();
+      }
     }
   }
   if (CL > 1) cluster.sync();              // peers may still be reading this CTA's sum
@@ -203,13 +295,33 @@ static int delta_fill(DeltaArgs& a, const float* in, int ld, const int* offs, in
   return 0;
 }
 
-template <int R>
-static int launch_delta_recurrent(const DeltaArgs& a, int CL, int n_seqs, cudaStream_t st) {
-  const int nv = a.VP / 4 / CL, groups = 256 / nv;
+// offs: columns of r, k, v, the output gate, the removal rate and the low-rank decay input in a row of `in`.
+B200_API int b200_delta_recurrent(const float* in, int ld, const int* offs, int rank, const void* w2, int rank8, const float* w0, const float* ab,
+                                  const float* norm, float* state, const int* q_start, const int* q_len, const int* ctx_len, const int* slot, int n_seqs,
+                                  int H, int dim, int vdim, int VP, float decay, float eps, float* out_f32, void* out_bf16, int ldo, cudaStream_t st) {
+  DeltaArgs a;
+  int rc = delta_fill(a, in, ld, offs, rank, w2, rank8, w0, ab, norm, state, q_start, q_len, ctx_len, slot, n_seqs, H, dim, vdim, VP, decay, eps, out_f32,
+                      out_bf16, ldo);
+  if (rc) return rc;
+  // CTAs per head: until a state share is 32 KB at most and the SMs are covered, eight float4 columns each at least
+  int CL = 1;
+  while (CL < 8 && (VP / 4) % (2 * CL) == 0 && VP / 4 / (2 * CL) >= 8 && (dim * VP / CL > 8192 || (long)H * n_seqs * CL < 148)) CL *= 2;
+  const DeltaLayout l = delta_layout(dim, VP / CL, rank8);
+  const size_t smem = 4 * (size_t)l.total;
+  if (smem > 200 * 1024) return B200_ERR_BAD_ARG;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(delta_recurrent_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  // shares of the sequences: no more CTAs than run at a time, all with about the same number of sequences
+  const int fit = (int)(227 * 1024 / (smem + 1024)), resident = 148 * (fit < 1 ? 1 : fit > 4 ? 4 : fit);
+  const int most = resident / (H * CL) > 1 ? resident / (H * CL) : 1, rounds = (n_seqs + most - 1) / most, shares = (n_seqs + rounds - 1) / rounds;
   cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(a.H * CL, n_seqs);
+  cfg.gridDim = dim3(H * CL, shares);
   cfg.blockDim = dim3(256);
-  cfg.dynamicSmemBytes = 4 * ((size_t)6 * a.dim + a.rank8 + 4 + 8 * nv + (size_t)groups * 8 * nv);      // at most 6 + 4 + 2 + 8 KB
+  cfg.dynamicSmemBytes = smem;
   cfg.stream = st;
   cudaLaunchAttribute attr[2];
   attr[0].id = cudaLaunchAttributeClusterDimension;
@@ -219,26 +331,7 @@ static int launch_delta_recurrent(const DeltaArgs& a, int CL, int n_seqs, cudaSt
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = b200_pdl_enabled() ? 2 : 1;
-  return (int)cudaLaunchKernelEx(&cfg, delta_recurrent_kernel<R>, a);
-}
-
-// offs: columns of r, k, v, the output gate, the removal rate and the low-rank decay input in a row of `in`.
-B200_API int b200_delta_recurrent(const float* in, int ld, const int* offs, int rank, const void* w2, int rank8, const float* w0, const float* ab,
-                                  const float* norm, float* state, const int* q_start, const int* q_len, const int* ctx_len, const int* slot, int n_seqs,
-                                  int H, int dim, int vdim, int VP, float decay, float eps, float* out_f32, void* out_bf16, int ldo, cudaStream_t st) {
-  DeltaArgs a;
-  int rc = delta_fill(a, in, ld, offs, rank, w2, rank8, w0, ab, norm, state, q_start, q_len, ctx_len, slot, n_seqs, H, dim, vdim, VP, decay, eps, out_f32,
-                      out_bf16, ldo);
-  if (rc) return rc;
-  auto rows = [&](int cl) { const int groups = 256 / (VP / 4 / cl); return (dim + groups - 1) / groups; };
-  int CL = 1;                            // CTAs per head: until the rows fit the registers and the SMs are covered, eight float4 columns each at least
-  while (CL < 8 && (VP / 4) % (2 * CL) == 0 && (rows(CL) > 16 || ((long)H * n_seqs * CL < 148 && VP / 4 / (2 * CL) >= 8))) CL *= 2;
-  const int R = rows(CL);
-  if (R <= 2) return launch_delta_recurrent<2>(a, CL, n_seqs, st);
-  if (R <= 4) return launch_delta_recurrent<4>(a, CL, n_seqs, st);
-  if (R <= 8) return launch_delta_recurrent<8>(a, CL, n_seqs, st);
-  if (R <= 16) return launch_delta_recurrent<16>(a, CL, n_seqs, st);
-  return B200_ERR_BAD_ARG;
+  return (int)cudaLaunchKernelEx(&cfg, delta_recurrent_kernel, a, n_seqs, l);
 }
 
 // ------------------------------------------------------------------ prompts: 64-token chunks on the tensor cores
@@ -260,7 +353,8 @@ B200_API int b200_delta_recurrent(const float* in, int ld, const int* offs, int 
 // once.  The factors e^b and e^-b stay within e^(64 decay).
 
 constexpr float kDeltaSpan = 60.f;       // most of GC * decay
-constexpr int kBlk = 16 * 24;            // a 16 x 16 block of bf16, rows 48 bytes apart (conflict-free for ldmatrix)
+constexpr int kBlk = 16 * 16;            // a 16 x 16 block of bf16; the halves of rows 4-7 and 12-15 change places (conflict-free for ldmatrix)
+__device__ __forceinline__ int in_block(int t, int s) { return t * 16 + ((((s >> 3) ^ (t >> 2)) & 1) << 3) + (s & 7); }
 constexpr int kRankSlice = 64;
 
 struct DeltaWs {                         // per (chunk slot, head); fragments of 32 lanes
@@ -272,18 +366,20 @@ struct DeltaWs {                         // per (chunk slot, head); fragments of
   int nvt;                               // value tiles of 16
 };
 
+// Shared memory: scratch | k, c, r | u, whose place the matrices take once it is in registers | v.  Each operand in two parts (values, remainders).
 template <int DP>
 struct DeltaSmem {
-  static constexpr int LQ = DP + 8, ROWS = GC * LQ;
+  static constexpr int LQ = DP + 8, ROWS = GC * LQ, OP = 2 * ROWS * 2;      // OP: bytes of an operand
   static constexpr int LW = kRankSlice + 8;
-  static constexpr int kOperands = 8 * ROWS * 2;                 // r u k c, values and remainders
-  static constexpr int kBlocks = 8 * 10 * kBlk * 2;              // -M (diagonal: its inverse), N, A, -B
-  static constexpr int kScratch = (4 * 16 * 17 + 256 + GC + DP) * 4;      // fp32 diagonal blocks of M; column sums; unit-key factors; e^{b_C}
+  static constexpr int kScratch = (4 * 16 * 17 + 256 + GC + DP) * 4;         // fp32 diagonal blocks of M; column sums; unit-key factors; e^{b_C}
+  static constexpr int kBlocks = 8 * 10 * kBlk * 2;                          // -M (diagonal: its inverse), N, A, -B
+  static constexpr int kTail = OP > kBlocks ? OP : kBlocks;
+  // only until the decays are known: tanh(x) in two parts and a slice of w2 over k, c, r; their product behind u
+  static constexpr int kProduct = GC * (DP + 1) * 4;
+  static_assert(2 * GC * LW * 2 + DP * LW * 2 <= 3 * OP, "the decay's operands fit the space of k, c and r");
   static int bytes(int nvt) {
-    const int fixed = kOperands + kBlocks + kScratch, v = GC * (nvt * 16 + 8) * 2;
-    // the decay's product uses the space of the blocks and of v: tanh(x) in two parts, a slice of w2, and its result
-    const int decay = 2 * GC * LW * 2 + DP * LW * 2 + GC * (DP + 1) * 4;
-    return fixed + (kBlocks + v > decay ? v : decay - kBlocks + 16);
+    const int with_v = kTail + GC * (nvt * 16 + 8) * 2, with_product = OP + kProduct;
+    return kScratch + 3 * OP + (with_v > with_product ? with_v : with_product);
   }
 };
 
@@ -291,21 +387,21 @@ struct DeltaSmem {
 __device__ __forceinline__ int tri(int i, int j) { return i * (i + 1) / 2 + j; }
 
 template <int DP>
-__global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, const DeltaWs ws) {
+__global__ void __launch_bounds__(256, DP <= 64 ? 2 : 1) delta_prepare_kernel(const DeltaArgs a, const DeltaWs ws) {
   using L = DeltaSmem<DP>;
   constexpr int LQ = L::LQ, LW = L::LW, NG = 256 / DP, TPT = GC / NG, KD = DP / 16;
   extern __shared__ __align__(16) uint8_t smem[];
-  __nv_bfloat16* sr = (__nv_bfloat16*)smem;                      // values, then remainders, of each
-  __nv_bfloat16 *su = sr + 2 * L::ROWS, *sk = su + 2 * L::ROWS, *sc = sk + 2 * L::ROWS;
-  float* sd = (float*)(smem + L::kOperands);                     // [4][16][17]
+  float* sd = (float*)smem;                                      // [4][16][17]
   float* stot = sd + 4 * 16 * 17;                                // [NG][DP]
   float* sinv = stot + 256;                                      // [GC]
   float* sdec = sinv + GC;                                       // [DP]
-  __nv_bfloat16* sb = (__nv_bfloat16*)(smem + L::kOperands + L::kScratch);      // blocks: [4 matrices][value, remainder][10][16][24]
-  __nv_bfloat16* sv = sb + 8 * 10 * kBlk;                        // [GC][LV]
-  __nv_bfloat16* sx = sb;                                        // [2][GC][LW]   } only until the decays are known
+  __nv_bfloat16* sk = (__nv_bfloat16*)(smem + L::kScratch);      // values, then remainders, of each
+  __nv_bfloat16 *sc = sk + 2 * L::ROWS, *sr = sc + 2 * L::ROWS, *su = sr + 2 * L::ROWS;
+  __nv_bfloat16* sb = su;                                        // blocks: [4 matrices][value, remainder][10][kBlk]
+  __nv_bfloat16* sv = su + L::kTail / 2;                         // [GC][LV]
+  __nv_bfloat16* sx = sk;                                        // [2][GC][LW]   } only until the decays are known
   __nv_bfloat16* sw = sx + 2 * GC * LW;                          // [DP][LW]      }
-  float* sz = (float*)(sw + DP * LW);                            // [GC][DP + 1]  }
+  float* sz = (float*)(su + 2 * L::ROWS);                        // [GC][DP + 1]  }
   const int LV = ws.nvt * 16 + 8;
   pdl_trigger();
   const int c = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
@@ -314,6 +410,11 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
   if (c * GC >= len) return;
   const int n = min(GC, len - c * GC), t0 = qs + c * GC;
   const float* in = a.in + (size_t)t0 * a.ld;
+  if (((a.vdim | a.dim | a.v_off | a.r_off | a.k_off | a.a_off | a.ld) & 3) == 0 && tid % GC < n) {      // rows read later, into L2 now
+    const int what = tid / GC;
+    const float* p = in + (size_t)(tid % GC) * a.ld + (what == 0 ? a.k_off + h * a.dim : what == 1 ? a.r_off + h * a.dim : what == 2 ? a.a_off + h * a.dim : a.v_off + h * a.vdim);
+    prefetch_l2(p, (what == 3 ? a.vdim : a.dim) * 4);
+  }
   // ---- z = W2 tanh(x): 64 tokens x DP channels, 64 ranks at a time; warp = 16 tokens x half of the channels
   {
     constexpr int NT = DP / 16;                                  // n8 tiles per warp
@@ -321,10 +422,16 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
     const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * (DP / 2);
     for (int r0 = 0; r0 < a.rank; r0 += kRankSlice) {
       if (r0) __syncthreads();
-      for (int i = tid; i < GC * kRankSlice; i += 256) {
-        const int t = i / kRankSlice, r = i % kRankSlice;
-        const float x = t < n && r0 + r < a.rank ? tanhf(in[(size_t)t * a.ld + a.x_off + r0 + r]) : 0.f;
-        split_bf16(x, sx[t * LW + r], sx[GC * LW + t * LW + r]);
+      {
+        const int r = tid % kRankSlice, q = tid / kRankSlice;    // a thread: one rank of every fourth token
+        float x[GC / 4];
+#pragma unroll
+        for (int i = 0; i < GC / 4; i++) x[i] = q + 4 * i < n && r0 + r < a.rank ? in[(size_t)(q + 4 * i) * a.ld + a.x_off + r0 + r] : 0.f;
+#pragma unroll
+        for (int i = 0; i < GC / 4; i++) {
+          const float e = expf(-2.f * fabsf(x[i])), y = copysignf((1.f - e) / (1.f + e), x[i]);      // tanh
+          split_bf16(y, sx[(q + 4 * i) * LW + r], sx[GC * LW + (q + 4 * i) * LW + r]);
+        }
       }
       for (int i = tid; i < DP * (kRankSlice / 8); i += 256) {
         const int d = i / (kRankSlice / 8), r = i % (kRankSlice / 8) * 8;
@@ -353,15 +460,20 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
 #pragma unroll
       for (int e = 0; e < 4; e++) sz[(m0 + g4 + 8 * (e >> 1)) * (DP + 1) + n0 + 8 * j + 2 * t4 + (e & 1)] = acc[j][e];
   }
-  for (int t = warp; t < GC; t += 8) {                           // unit keys
-    float ss = 0.f;
-    if (t < n)
-      for (int d = lane; d < a.dim; d += 32) {
-        const float k = in[(size_t)t * a.ld + a.k_off + h * a.dim + d];
-        ss += k * k;
-      }
-    ss = warp_sum(ss);
-    if (lane == 0) sinv[t] = 1.f / sqrtf(ss + kUnitEps);
+  {                                                              // unit keys: a warp takes eight tokens
+    float ss[8] = {};
+    for (int d = lane; d < a.dim; d += 32) {
+      float k[8];
+#pragma unroll
+      for (int i = 0; i < 8; i++) k[i] = warp * 8 + i < n ? in[(size_t)(warp * 8 + i) * a.ld + a.k_off + h * a.dim + d] : 0.f;
+#pragma unroll
+      for (int i = 0; i < 8; i++) ss[i] = fmaf(k[i], k[i], ss[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+      ss[i] = warp_sum(ss[i]);
+      if (lane == i) sinv[warp * 8 + i] = 1.f / sqrtf(ss[i] + kUnitEps);
+    }
   }
   __syncthreads();
   // ---- running sums of the log decays, and the decayed operands: a thread owns one channel of TPT consecutive tokens
@@ -428,11 +540,15 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
     }
   }
   // ---- the four triangular matrices, 40 blocks of 16 x 16, five per warp: (u, r) x (c, k)
+  float blocks[5][2][4];
+#pragma unroll
   for (int q = 0; q < 5; q++) {
     const int unit = warp * 5 + q, mat = unit / 10, blk = unit % 10;        // mat 0: u c (-M), 1: u k (N), 2: r k (A), 3: r c (-B)
     const int i = blk >= 6 ? 3 : blk >= 3 ? 2 : blk >= 1 ? 1 : 0, j = blk - i * (i + 1) / 2;
     const __nv_bfloat16 *X = mat < 2 ? su : sr, *Y = (mat == 0 || mat == 3) ? sc : sk;
-    float acc[2][4] = {};
+    float (&acc)[2][4] = blocks[q];
+#pragma unroll
+    for (int m = 0; m < 2; m++) acc[m][0] = acc[m][1] = acc[m][2] = acc[m][3] = 0.f;
 #pragma unroll
     for (int k0 = 0; k0 < DP; k0 += 16) {
       uint32_t xh[4], xl[4], yh[4], yl[4];
@@ -449,6 +565,31 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
       mma_bf16(acc[0], xl, yh[0], yh[1]);
       mma_bf16(acc[1], xl, yh[2], yh[3]);
     }
+  }
+  // rows d0..d0 + 16 (as MMA rows) of the tokens of tile i, from a [token][channel] operand kept in two parts
+  auto columns = [&](const __nv_bfloat16* p, int d0, int i, float (&z)[2][4]) {
+    uint32_t hi[4], lo[4];
+    const int at = (i * 16 + (lane >> 4) * 8 + (lane & 7)) * LQ + d0 + ((lane >> 3) & 1) * 8;
+    ldsm4t(s32(p + at), hi);
+    ldsm4t(s32(p + L::ROWS + at), lo);
+#pragma unroll
+    for (int m = 0; m < 4; m++) {
+      const float2 x = __bfloat1622float2(*(const __nv_bfloat162*)&hi[m]), y = __bfloat1622float2(*(const __nv_bfloat162*)&lo[m]);
+      z[m >> 1][(m & 1) * 2] = x.x + y.x;
+      z[m >> 1][(m & 1) * 2 + 1] = x.y + y.y;
+    }
+  };
+  float u[4][2][4];                                              // this warp's columns of u: the matrices take its place
+  if (warp < KD) {
+#pragma unroll
+    for (int i = 0; i < 4; i++) columns(su, warp * 16, i, u[i]);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int q = 0; q < 5; q++) {
+    const int unit = warp * 5 + q, mat = unit / 10, blk = unit % 10;
+    const int i = blk >= 6 ? 3 : blk >= 3 ? 2 : blk >= 1 ? 1 : 0, j = blk - i * (i + 1) / 2;
+    float (&acc)[2][4] = blocks[q];
     __nv_bfloat16* hi = sb + (mat * 2) * 10 * kBlk + blk * kBlk;
     __nv_bfloat16* lo = hi + 10 * kBlk;
 #pragma unroll
@@ -468,8 +609,8 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
         } else {
           uint32_t p, r;
           split2(x, y, p, r);
-          *(uint32_t*)(hi + t * 24 + s) = p;
-          *(uint32_t*)(lo + t * 24 + s) = r;
+          *(uint32_t*)(hi + in_block(t, s)) = p;
+          *(uint32_t*)(lo + in_block(t, s)) = r;
         }
       }
   }
@@ -484,15 +625,16 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
     for (int k = 0; k < 16; k++)
 #pragma unroll
       for (int t = k + 1; t < 16; t++) x[t] = fmaf(m[t * 17 + k], x[k], x[t]);
-    __nv_bfloat16* hi = sb + tri(i, i) * kBlk + s;
+    __nv_bfloat16* hi = sb + tri(i, i) * kBlk;
 #pragma unroll
-    for (int t = 0; t < 16; t++) split_bf16(x[t], hi[t * 24], hi[10 * kBlk + t * 24]);
+    for (int t = 0; t < 16; t++) split_bf16(x[t], hi[in_block(t, s)], hi[10 * kBlk + in_block(t, s)]);
   }
   __syncthreads();
 
   // block (i, j) of matrix `mat` as the B operand (token columns, earlier tokens contracted)
+  const int blk_at = in_block((lane >> 4) * 8 + (lane & 7), ((lane >> 3) & 1) * 8);
   auto block = [&](int mat, int i, int j, uint32_t (&hi)[4], uint32_t (&lo)[4]) {
-    const __nv_bfloat16* p = sb + (mat * 2) * 10 * kBlk + tri(i, j) * kBlk + ((lane >> 4) * 8 + (lane & 7)) * 24 + ((lane >> 3) & 1) * 8;
+    const __nv_bfloat16* p = sb + (mat * 2) * 10 * kBlk + tri(i, j) * kBlk + blk_at;
     ldsm4(s32(p), hi);
     ldsm4(s32(p + 10 * kBlk), lo);
   };
@@ -516,19 +658,6 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
     split2(z[1][0], z[1][1], hi[2], lo[2]);
     split2(z[1][2], z[1][3], hi[3], lo[3]);
   };
-  // rows d0..d0 + 16 (as MMA rows) of the tokens of tile i, from a [token][channel] operand kept in two parts
-  auto columns = [&](const __nv_bfloat16* p, int d0, int i, float (&z)[2][4]) {
-    uint32_t hi[4], lo[4];
-    const int at = (i * 16 + (lane >> 4) * 8 + (lane & 7)) * LQ + d0 + ((lane >> 3) & 1) * 8;
-    ldsm4t(s32(p + at), hi);
-    ldsm4t(s32(p + L::ROWS + at), lo);
-#pragma unroll
-    for (int m = 0; m < 4; m++) {
-      const float2 x = __bfloat1622float2(*(const __nv_bfloat162*)&hi[m]), y = __bfloat1622float2(*(const __nv_bfloat162*)&lo[m]);
-      z[m >> 1][(m & 1) * 2] = x.x + y.x;
-      z[m >> 1][(m & 1) * 2 + 1] = x.y + y.y;
-    }
-  };
   // (I + M) X = Z, tile by tile: z holds tile i of Z and of what the earlier tiles of X (xh, xl) take off it
   auto solve = [&](int i, float (&z)[2][4], uint32_t (&xh)[4][4], uint32_t (&xl)[4][4]) {
     uint32_t bh[4], bl[4], zh[4], zl[4];
@@ -551,9 +680,7 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
       const int d0 = cb * 16;
 #pragma unroll
       for (int i = 0; i < 4; i++) {
-        float z[2][4];
-        columns(su, d0, i, z);
-        solve(i, z, xh, xl);
+        solve(i, u[i], xh, xl);
       }
       uint4* dst = ws.r + (slot * KD + cb) * 4 * 64 + lane * 2;
 #pragma unroll
@@ -646,7 +773,8 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a, c
   }
 }
 
-constexpr int state_stages(int dp) { return dp >= 128 ? 3 : 4; }
+constexpr int state_stages(int dp) { return dp >= 128 ? 2 : 4; }
+constexpr int state_bytes(int dp, int warps) { return state_stages(dp) * (dp * dp + warps * 16 * dp) * 4; }
 
 // One CTA = some value tiles of one head of one sequence, a warp 16 value columns (as MMA rows) x all key channels: S'^T = S^T G^T + F^T.  The accumulators,
 // split into values and remainders, are the A operand of the next chunk's product as they lie, and that is the form a chunk's starting state is stored in.
@@ -657,7 +785,8 @@ __global__ void __launch_bounds__(128) delta_state_kernel(const DeltaArgs a, con
   pdl_trigger();
   pdl_wait();
   const int h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3, NT = blockDim.x;
-  const int vb = blockIdx.x * (NT >> 5) + warp, vt = min(vb, ws.nvt - 1);
+  const int vb0 = blockIdx.x * (NT >> 5), vb = vb0 + warp, vt = min(vb, ws.nvt - 1);
+  const int FN = min(NT >> 5, ws.nvt - vb0) * (DP / 8) * 32, SN = GN + (NT >> 5) * (DP / 8) * 32;      // float4 of F; of a stage
   const bool mine = vb < ws.nvt;
   const int len = a.q_len[seq], qs = a.q_start[seq], slot = a.slot[seq];
   const bool fresh = a.ctx_len[seq] - len == 0 || slot < 0;
@@ -666,9 +795,16 @@ __global__ void __launch_bounds__(128) delta_state_kernel(const DeltaArgs a, con
   const size_t base = chunk_slot(qs, seq, 0) * a.H + h;
   const uint4* gsrc = ws.g + base * GN;
   const size_t gstep = (size_t)a.H * GN;
+  const float4* fsrc = ws.f + (base * ws.nvt + vb0) * (DP / 8) * 32;
+  const size_t fstep = (size_t)a.H * ws.nvt * (DP / 8) * 32;
   auto load = [&](int c) {
-    if (c < nc)
-      for (int i = tid; i < GN; i += NT) cp_async16(s32(sg + (c % ST) * GN + i), gsrc + c * gstep + i);
+    if (c < nc) {
+      uint4* dst = sg + (c % ST) * SN;
+#pragma unroll 4
+      for (int i = tid; i < GN; i += NT) cp_async16(s32(dst + i), gsrc + c * gstep + i);
+#pragma unroll 4
+      for (int i = tid; i < FN; i += NT) cp_async16(s32(dst + GN + i), fsrc + c * fstep + i);
+    }
     cp_async_commit();                  // empty past the end: keeps the count of groups in flight
   };
 #pragma unroll
@@ -682,7 +818,6 @@ __global__ void __launch_bounds__(128) delta_state_kernel(const DeltaArgs a, con
       acc[j][e] = (!fresh && v < a.VP && d < a.dim) ? S[(size_t)d * a.VP + v] : 0.f;
     }
   for (int c = 0; c < nc; c++) {
-    const float4* f = ws.f + ((base + (size_t)c * a.H) * ws.nvt + vt) * (DP / 8) * 32 + lane;
     uint32_t sh[KD][4], sl[KD][4];
     uint4* frag = ws.s + ((base + (size_t)c * a.H) * ws.nvt + vt) * KD * 64 + lane * 2;
 #pragma unroll
@@ -696,15 +831,16 @@ __global__ void __launch_bounds__(128) delta_state_kernel(const DeltaArgs a, con
         frag[kd * 64 + 1] = make_uint4(sl[kd][0], sl[kd][1], sl[kd][2], sl[kd][3]);
       }
     }
-#pragma unroll
-    for (int j = 0; j < DP / 8; j++) {
-      const float4 x = __ldg(f + j * 32);
-      acc[j][0] = x.x; acc[j][1] = x.y; acc[j][2] = x.z; acc[j][3] = x.w;
-    }
     cp_async_wait<ST - 2>();
     __syncthreads();                    // chunk c has landed, and everyone is done with the stage that is refilled now
     load(c + ST - 1);
-    const uint4* g = sg + (c % ST) * GN + lane * 2;
+    const uint4* g = sg + (c % ST) * SN + lane * 2;
+    const float4* f = (const float4*)(sg + (c % ST) * SN + GN) + (vt - vb0) * (DP / 8) * 32 + lane;
+#pragma unroll
+    for (int j = 0; j < DP / 8; j++) {
+      const float4 x = f[j * 32];
+      acc[j][0] = x.x; acc[j][1] = x.y; acc[j][2] = x.z; acc[j][3] = x.w;
+    }
 #pragma unroll
     for (int kd = 0; kd < KD; kd++)
 #pragma unroll
@@ -848,11 +984,11 @@ B200_API size_t b200_delta_chunk_bytes(int T, int n_seqs, int H, int dim, int VP
 
 template <int DP>
 static int launch_delta_chunked(const DeltaArgs& a, const DeltaWs& w, int n_seqs, int max_q, cudaStream_t st) {
-  const int s1 = DeltaSmem<DP>::bytes(w.nvt), s2 = state_stages(DP) * DP * DP * 4, s3 = GC * (w.nvt * 16 + 4) * 4;
+  const int s1 = DeltaSmem<DP>::bytes(w.nvt), s3 = GC * (w.nvt * 16 + 4) * 4;
   static int configured = 0;
   if (s1 > configured) {
     cudaError_t e = cudaFuncSetAttribute(delta_prepare_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, s1);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_state_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, s2);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_state_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, state_bytes(DP, 4));
     if (e != cudaSuccess) return (int)e;
     configured = s1;
   }
@@ -861,7 +997,7 @@ static int launch_delta_chunked(const DeltaArgs& a, const DeltaWs& w, int n_seqs
   if (rc) return rc;
   int warps = min(4, w.nvt);                 // fewer value tiles to a CTA until the SMs are covered
   while (warps > 1 && (long)a.H * n_seqs * ((w.nvt + warps - 1) / warps) < 148) warps >>= 1;
-  rc = launch_pdl(delta_state_kernel<DP>, dim3((w.nvt + warps - 1) / warps, a.H, n_seqs), dim3(32 * warps), s2, st, a, w);
+  rc = launch_pdl(delta_state_kernel<DP>, dim3((w.nvt + warps - 1) / warps, a.H, n_seqs), dim3(32 * warps), state_bytes(DP, warps), st, a, w);
   if (rc) return rc;
   auto out = w.nvt <= 4 ? delta_output_kernel<DP, 1> : delta_output_kernel<DP, 2>;
   return launch_pdl(out, dim3(nc, a.H, n_seqs), dim3(256), s3, st, a, w);

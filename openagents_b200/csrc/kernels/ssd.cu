@@ -125,111 +125,187 @@ __global__ void __launch_bounds__(256) ssd_conv_kernel(const SsdArgs a, const Ss
 
 // ------------------------------------------------------------------ token by token
 
-// One cluster of CTAs per (head, sequence), sharing the value columns; a thread keeps R state rows of one float4 column in registers over all tokens.
-// FUSED: one token per sequence (decoding): the filter is applied here, and its input written to the ring: the row of the current position, which no CTA
+// The CTAs of a head share its value columns and the sequences.  A CTA walks the tokens of its sequences one by one; while it works on one, the filtered inputs
+// of the next, and with a new sequence its state, are on their way into the other half of a double buffer.  The state is updated in shared memory.
+// FUSED (a few sequences with one token each): the filter is applied here, and its input written to the ring: the row of the current position, which no CTA
 // reads.  Otherwise the filter has run (fp32), and the ring takes the portion's last inputs.
-template <int R, bool FUSED>
-__global__ void __launch_bounds__(256, R <= 8 ? 2 : 1) ssd_recurrent_kernel(const SsdArgs a, const SsdConv<float> o) {
+__device__ __forceinline__ void cp_async4(void* dst, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(s32(dst)), "l"(src) : "memory");
+}
+struct SsdLayout {                         // floats of shared memory: two states, two rows, the partial outputs
+  int state_n, row_n, row, y, total;
+};
+static SsdLayout ssd_layout(int N, int W) {
+  SsdLayout l;
+  l.state_n = N * W;
+  l.row_n = W + 2 * N + 4;                 // x | B | C | dt, log decay
+  l.row_n = (l.row_n + 3) & ~3;
+  l.row = 2 * l.state_n;
+  l.y = l.row + 2 * l.row_n;
+  l.total = l.y + 256 / (W / 4) * W;
+  return l;
+}
+template <bool FUSED>
+__global__ void __launch_bounds__(256, 4) ssd_recurrent_kernel(const SsdArgs a, const SsdConv<float> o, int n_seqs, const SsdLayout l) {
   extern __shared__ __align__(16) float sm[];
-  const int CL = gridDim.x / a.H, part = blockIdx.x % CL, h = blockIdx.x / CL, b = blockIdx.y, tid = threadIdx.x;
+  const int CL = gridDim.x / a.H, part = blockIdx.x % CL, h = blockIdx.x / CL, tid = threadIdx.x;
   const int nv_all = a.PP >> 2, nv = nv_all / CL, W = nv * 4, e0 = part * W;     // this CTA's columns [e0, e0 + W)
   const int groups = 256 / nv, g = h / (a.H / a.G);
-  float* s_b = sm;                         // [N], times dt
-  float* s_c = s_b + a.N;                  // [N]
-  float* s_x = s_c + a.N + ((4 - ((2 * a.N) & 3)) & 3);      // [W], 16-byte aligned
-  float* s_y = s_x + W;                    // [groups][W]
+  float* s_y = sm + l.y;                   // [groups][W]
   pdl_trigger();
   const float A = -expf(a.A_log[h]), Dh = a.D[h], dtb = a.dt_bias[h];
   const int xc = a.H * a.P;
-  // this thread's first channel of the filter: x columns, then B, then C of the group
+  // the filter's channels that this CTA needs: x columns, then B, then C of the group; `own`: those it keeps the ring of
   const int n_ch = W + 2 * a.N;
   auto channel = [&](int i) {
     if (i < W) return e0 + i < a.P ? h * a.P + e0 + i : -1;
     const int j = i - W, which = j / a.N;
     return xc + (which * a.G + g) * a.N + j - which * a.N;
   };
-  pdl_wait();
-  const int n = a.q_len[b], t0 = a.q_start[b], slot = a.slot[b], p0 = a.ctx_len[b] - n;
-  const bool fresh = p0 == 0 || slot < 0;
+  const bool first_head = part == 0 && h % (a.H / a.G) == 0;
+  auto own = [&](int i) { return i < W || first_head; };
   const int grp = tid / nv, col = tid % nv;
   const bool active = grp < groups;
-  float4* S = (float4*)(a.state + ((size_t)max(slot, 0) * a.H + h) * a.N * a.PP) + part * nv + col;
-  float4 st[R];
-#pragma unroll
-  for (int k = 0; k < R; k++) {
-    const int d = grp + k * groups;
-    st[k] = (active && !fresh && d < a.N) ? S[(size_t)d * nv_all] : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
-  for (int i = 0; i < n; i++) {
-    const size_t t = t0 + i;
-    float dt;
-    if constexpr (FUSED) {
-      const float* row = a.in + t * a.ld;
-      dt = softplus_f(row[a.dt_off + h] + dtb);
-      for (int q = tid; q < n_ch; q += 256) {
-        const int ch = channel(q);
-        float s = 0.f;
-        if (ch >= 0) {
-          const float cur = row[a.x_off + ch], *w = a.cw + (size_t)ch * a.taps;
-          if (!fresh)
-            for (int j = 0; j < a.taps - 1; j++) s = fmaf(w[j], ring_at(a, slot, p0 - a.taps + 1 + j, ch), s);
-          s = silu_f(fmaf(w[a.taps - 1], cur, s) + a.cb[ch]);
-          if (slot >= 0 && (q < W || (part == 0 && h % (a.H / a.G) == 0))) a.ring[((size_t)slot * a.taps + p0 % a.taps) * a.CC + ch] = cur;
-        }
-        if (q < W) s_x[q] = s;
-        else if (q < W + a.N) s_b[q - W] = s * dt;
-        else s_c[q - W - a.N] = s;
-      }
-    } else {
-      dt = o.dt[t * a.H + h];
-      for (int q = tid; q < n_ch; q += 256) {
-        if (q < W) s_x[q] = o.x[(t * a.H + h) * a.PP + e0 + q];
-        else if (q < W + a.N) s_b[q - W] = o.B[(t * a.G + g) * a.NP + q - W] * dt;
-        else s_c[q - W - a.N] = o.C[(t * a.G + g) * a.NP + q - W - a.N];
-      }
+  pdl_wait();
+  struct Seq { int n, t0, slot, p0; bool fresh; };
+  auto meta = [&](int b) {
+    Seq q = {0, 0, -1, 0, true};
+    if (b < n_seqs) {
+      q.n = a.q_len[b];
+      q.t0 = a.q_start[b];
+      q.slot = a.slot[b];
+      q.p0 = a.ctx_len[b] - q.n;
+      q.fresh = q.p0 == 0 || q.slot < 0;
     }
-    const float al = expf(A * dt);
-    __syncthreads();
+    return q;
+  };
+  auto state_of = [&](int slot) { return (float4*)(a.state + ((size_t)max(slot, 0) * a.H + h) * a.N * a.PP) + part * nv; };
+  auto fetch_state = [&](const Seq& q, int buf) {
+    float4* dst = (float4*)(sm + buf * l.state_n);
+    const float4* src = state_of(q.slot);
+    if (!active) return;
+    for (int d = grp; d < a.N; d += groups) {
+      if (!q.fresh) cp_async16(s32(dst + d * nv + col), src + (size_t)d * nv_all + col);
+      else dst[d * nv + col] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  auto fetch_row = [&](size_t t, int buf) {
+    float* dst = sm + l.row + buf * l.row_n;
+    for (int q = tid; q < n_ch + 2; q += 256) {
+      const float* src;
+      if (q < W) src = o.x + (t * a.H + h) * a.PP + e0 + q;
+      else if (q < W + a.N) src = o.B + (t * a.G + g) * a.NP + q - W;
+      else if (q < n_ch) src = o.C + (t * a.G + g) * a.NP + q - W - a.N;
+      else src = (q == n_ch ? o.dt : o.la) + t * a.H + h;
+      cp_async4(dst + q, src);
+    }
+  };
+  auto filter_row = [&](const Seq& q, int buf) {          // FUSED
+    float* dst = sm + l.row + buf * l.row_n;
+    const float* row = a.in + (size_t)q.t0 * a.ld;
+    for (int i = tid; i < n_ch; i += 256) {
+      const int ch = channel(i);
+      float s = 0.f;
+      if (ch >= 0) {
+        const float cur = row[a.x_off + ch], *w = a.cw + (size_t)ch * a.taps;
+        if (!q.fresh)
+          for (int j = 0; j < a.taps - 1; j++) s = fmaf(w[j], ring_at(a, q.slot, q.p0 - a.taps + 1 + j, ch), s);
+        s = silu_f(fmaf(w[a.taps - 1], cur, s) + a.cb[ch]);
+        if (q.slot >= 0 && own(i)) a.ring[((size_t)q.slot * a.taps + q.p0 % a.taps) * a.CC + ch] = cur;
+      }
+      dst[i] = s;
+    }
+    if (tid == 0) {
+      dst[n_ch] = softplus_f(row[a.dt_off + h] + dtb);
+      dst[n_ch + 1] = A * dst[n_ch];
+    }
+  };
+  int b = blockIdx.y, i = 0, sbuf = 0, rbuf = 0;
+  Seq cur = meta(b), nxt = meta(b + gridDim.y);
+  while (b < n_seqs && cur.n < 1) {         // an entry without tokens
+    b += gridDim.y;
+    cur = nxt;
+    nxt = meta(b + gridDim.y);
+  }
+  auto begin = [&]() {
+    fetch_state(cur, sbuf);
+    if (FUSED) filter_row(cur, rbuf);
+    else fetch_row(cur.t0, rbuf);
+    cp_async_commit();
+  };
+  if (b < n_seqs) begin();
+  while (b < n_seqs) {
+    cp_async_wait_all();
+    __syncthreads();                       // this token's data has landed, and everyone is done with the other buffers
+    const bool last = i + 1 == cur.n;
+    if (!FUSED) {
+      if (!last) {
+        fetch_row(cur.t0 + i + 1, rbuf ^ 1);
+      } else if (b + gridDim.y < n_seqs && nxt.n > 0) {
+        fetch_state(nxt, sbuf ^ 1);
+        fetch_row(nxt.t0, rbuf ^ 1);
+      }
+      cp_async_commit();
+    }
+    const float* row = sm + l.row + rbuf * l.row_n;
+    const float *s_b = row + W, *s_c = s_b + a.N;
+    const float dt = row[n_ch], al = expf(row[n_ch + 1]);
     if (active) {
-      const float4 x = *(const float4*)(s_x + 4 * col);
+      const bool keep = last && cur.slot >= 0;
+      float4* S = (float4*)(sm + sbuf * l.state_n) + col;
+      float4* dst = state_of(cur.slot) + col;
+      float4 x = *(const float4*)(row + 4 * col);
+      x.x *= dt; x.y *= dt; x.z *= dt; x.w *= dt;
       float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-      for (int k = 0; k < R; k++) {
-        const int d = grp + k * groups;
-        if (d >= a.N) break;
+#pragma unroll 4
+      for (int d = grp; d < a.N; d += groups) {
         const float bb = s_b[d], cc = s_c[d];
-        st[k].x = fmaf(al, st[k].x, bb * x.x);
-        st[k].y = fmaf(al, st[k].y, bb * x.y);
-        st[k].z = fmaf(al, st[k].z, bb * x.z);
-        st[k].w = fmaf(al, st[k].w, bb * x.w);
-        y.x = fmaf(cc, st[k].x, y.x);
-        y.y = fmaf(cc, st[k].y, y.y);
-        y.z = fmaf(cc, st[k].z, y.z);
-        y.w = fmaf(cc, st[k].w, y.w);
+        float4 v = S[d * nv];
+        v.x = fmaf(al, v.x, bb * x.x);
+        v.y = fmaf(al, v.y, bb * x.y);
+        v.z = fmaf(al, v.z, bb * x.z);
+        v.w = fmaf(al, v.w, bb * x.w);
+        if (!last) S[d * nv] = v;
+        else if (keep) dst[(size_t)d * nv_all] = v;
+        y.x = fmaf(cc, v.x, y.x);
+        y.y = fmaf(cc, v.y, y.y);
+        y.z = fmaf(cc, v.z, y.z);
+        y.w = fmaf(cc, v.w, y.w);
       }
       *(float4*)(s_y + grp * W + 4 * col) = y;
     }
     __syncthreads();
-    for (int e = tid; e < W; e += 256) {
-      float y = Dh * s_x[e];
-      for (int q = 0; q < groups; q++) y += s_y[q * W + e];
-      if (e0 + e < a.P) a.y[t * a.ldy + h * a.P + e0 + e] = y;
+    if (tid < W && e0 + tid < a.P) {       // W <= 256
+      float y = Dh * row[tid];
+#pragma unroll 4
+      for (int q = 0; q < groups; q++) y += s_y[q * W + tid];
+      a.y[(size_t)(cur.t0 + i) * a.ldy + h * a.P + e0 + tid] = y;
     }
-    __syncthreads();
+    rbuf ^= 1;
+    i++;
+    if (last) {
+      if (!FUSED && cur.slot >= 0)
+        for (int q = tid; q < n_ch; q += 256) {
+          const int ch = channel(q);
+          if (ch < 0 || !own(q)) continue;
+          for (int j = max(0, cur.n - a.taps + 1); j < cur.n; j++)
+            a.ring[((size_t)cur.slot * a.taps + (cur.p0 + j) % a.taps) * a.CC + ch] = a.in[(size_t)(cur.t0 + j) * a.ld + a.x_off + ch];
+        }
+      i = 0;
+      sbuf ^= 1;
+      bool skipped = false;
+      do {                                 // past entries without tokens, whose successors were not fetched ahead
+        b += gridDim.y;
+        cur = nxt;
+        nxt = meta(b + gridDim.y);
+        if (b < n_seqs && cur.n < 1) skipped = true;
+      } while (b < n_seqs && cur.n < 1);
+      if ((FUSED || skipped) && b < n_seqs) {
+        __syncthreads();
+        begin();
+      }
+    }
   }
-  if (slot >= 0 && active) {
-#pragma unroll
-    for (int k = 0; k < R; k++) {
-      const int d = grp + k * groups;
-      if (d < a.N) S[(size_t)d * nv_all] = st[k];
-    }
-  }
-  if (!FUSED && slot >= 0)
-    for (int q = tid; q < n_ch; q += 256) {
-      const int ch = channel(q);
-      if (ch < 0 || !(q < W || (part == 0 && h % (a.H / a.G) == 0))) continue;
-      for (int i = max(0, n - a.taps + 1); i < n; i++) a.ring[((size_t)slot * a.taps + (p0 + i) % a.taps) * a.CC + ch] = a.in[(size_t)(t0 + i) * a.ld + a.x_off + ch];
-    }
 }
 
 static int ssd_fill(SsdArgs& a, const float* in, int ld, int x_off, int dt_off, const float* cw, const float* cb, const float* dt_bias, const float* A_log,
@@ -246,14 +322,22 @@ static int ssd_fill(SsdArgs& a, const float* in, int ld, int x_off, int dt_off, 
 
 template <bool FUSED>
 static int launch_ssd_recurrent(const SsdArgs& a, const SsdConv<float>& o, int n_seqs, cudaStream_t st) {
-  auto rows = [&](int cl) { const int groups = 256 / (a.PP / 4 / cl); return (a.N + groups - 1) / groups; };
-  int CL = 1;                            // CTAs per head: until the rows fit the registers and the SMs are covered, eight float4 columns each at least
-  while (CL < 8 && (a.PP / 4) % (2 * CL) == 0 && (rows(CL) > 16 || ((long)a.H * n_seqs * CL < 148 && a.PP / 4 / (2 * CL) >= 8))) CL *= 2;
-  const int R = rows(CL), nv = a.PP / 4 / CL;
-  if (R > 16) return B200_ERR_BAD_ARG;
-  const size_t smem = 4 * ((size_t)2 * a.N + 4 + 4 * nv + (size_t)(256 / nv) * 4 * nv);
-  auto kern = R <= 2 ? ssd_recurrent_kernel<2, FUSED> : R <= 4 ? ssd_recurrent_kernel<4, FUSED> : R <= 8 ? ssd_recurrent_kernel<8, FUSED> : ssd_recurrent_kernel<16, FUSED>;
-  return launch_pdl(kern, dim3(a.H * CL, n_seqs), dim3(256), smem, st, a, o);
+  // CTAs per head: until a state share is 32 KB at most and the SMs are covered, eight float4 columns each at least
+  int CL = 1;
+  while (CL < 8 && (a.PP / 4) % (2 * CL) == 0 && a.PP / 4 / (2 * CL) >= 8 && (a.N * a.PP / CL > 8192 || (long)a.H * n_seqs * CL < 148)) CL *= 2;
+  const SsdLayout l = ssd_layout(a.N, a.PP / CL);
+  const size_t smem = 4 * (size_t)l.total;
+  if (smem > 200 * 1024) return B200_ERR_BAD_ARG;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(ssd_recurrent_kernel<FUSED>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  // shares of the sequences: no more CTAs than run at a time, all with about the same number of sequences
+  const int fit = (int)(227 * 1024 / (smem + 1024)), resident = 148 * (fit < 1 ? 1 : fit > 4 ? 4 : fit);
+  const int most = resident / (a.H * CL) > 1 ? resident / (a.H * CL) : 1, rounds = (n_seqs + most - 1) / most;
+  return launch_pdl(ssd_recurrent_kernel<FUSED>, dim3(a.H * CL, (n_seqs + rounds - 1) / rounds), dim3(256), smem, st, a, o, n_seqs, l);
 }
 
 template <typename OT>
@@ -284,11 +368,22 @@ static int launch_ssd_conv(const SsdArgs& a, const SsdConv<OT>& o, int n_seqs, i
 #define SSD_FILL                                                                                                                                       \
   ssd_fill(a, in, ld, x_off, dt_off, cw, cb, dt_bias, A_log, D, state, ring, q_start, q_len, ctx_len, slot, n_seqs, H, P, N, G, taps, PP, y, ldy)
 
-// One token per sequence.
-B200_API int b200_ssd_decode(SSD_PARAMS, cudaStream_t st) {
+constexpr int kFusedSeqs = 4;           // decode steps of up to this many sequences apply the filter in the recurrence's kernel
+
+// One token per sequence.  ws: b200_ssd_decode_bytes bytes, 256-byte aligned.
+B200_API size_t b200_ssd_decode_bytes(int n_seqs, int H, int PP, int N, int G) {
+  return n_seqs <= kFusedSeqs ? 0 : ssd_conv_bytes(n_seqs, H, PP, G, (N + 15) / 16 * 16, 4);
+}
+B200_API int b200_ssd_decode(SSD_PARAMS, void* ws, size_t ws_bytes, cudaStream_t st) {
   SsdArgs a;
   int rc = SSD_FILL;
-  return rc ? rc : launch_ssd_recurrent<true>(a, SsdConv<float>{}, n_seqs, st);
+  if (rc) return rc;
+  if (n_seqs <= kFusedSeqs) return launch_ssd_recurrent<true>(a, SsdConv<float>{}, n_seqs, st);
+  if (ws_bytes < b200_ssd_decode_bytes(n_seqs, H, PP, N, G) || ((uintptr_t)ws % 256)) return B200_ERR_BAD_ARG;
+  char* p = (char*)ws;
+  const SsdConv<float> o = ssd_conv_ws<float>(a, p, n_seqs);
+  rc = launch_ssd_conv(a, o, n_seqs, 1, st);
+  return rc ? rc : launch_ssd_recurrent<false>(a, o, n_seqs, st);
 }
 
 // ------------------------------------------------------------------ prompts: 64-token chunks on the tensor cores
@@ -311,12 +406,21 @@ struct ChunkDecay {
   float2 dt, b;
   float total;
 };
-__device__ __forceinline__ ChunkDecay chunk_decay(const SsdArgs& a, const SsdConv<__nv_bfloat16>& o, int t0, int n, int h, int lane) {
-  ChunkDecay r;
+struct RawDecay {
+  float2 dt, la;
+};
+__device__ __forceinline__ RawDecay load_decay(const SsdArgs& a, const SsdConv<__nv_bfloat16>& o, int t0, int n, int h, int lane) {
   const size_t at = (size_t)(t0 + 2 * lane) * a.H + h;
   const bool v0 = 2 * lane < n, v1 = 2 * lane + 1 < n;
+  RawDecay r;
   r.dt = make_float2(v0 ? o.dt[at] : 0.f, v1 ? o.dt[at + a.H] : 0.f);
-  const float l0 = v0 ? o.la[at] : 0.f, l1 = v1 ? o.la[at + a.H] : 0.f;
+  r.la = make_float2(v0 ? o.la[at] : 0.f, v1 ? o.la[at + a.H] : 0.f);
+  return r;
+}
+__device__ __forceinline__ ChunkDecay chunk_decay(const RawDecay& raw, int lane) {
+  ChunkDecay r;
+  r.dt = raw.dt;
+  const float l0 = raw.la.x, l1 = raw.la.y;
   float s = l0 + l1;
 #pragma unroll
   for (int d = 1; d < 32; d <<= 1) {
@@ -376,11 +480,16 @@ __global__ void __launch_bounds__(256) ssd_state_kernel(const SsdArgs a, const S
       acc[j][e] = (!fresh && v < a.PP && d < a.N) ? S[(size_t)d * a.PP + v] : 0.f;
     }
   const int pt = ps * 4 + warp;
-  ChunkDecay next = chunk_decay(a, ws.c, qs, min(GC, len), h, lane);
+  float f0, f1, dec;
+  auto factors = [&](const RawDecay& raw) {
+    const ChunkDecay dc = chunk_decay(raw, lane);
+    f0 = dc.dt.x * expf(dc.total - dc.b.x);
+    f1 = dc.dt.y * expf(dc.total - dc.b.y);
+    dec = expf(dc.total);
+  };
+  factors(load_decay(a, ws.c, qs, min(GC, len), h, lane));
   for (int c = 0; c < nc; c++) {
-    const ChunkDecay dc = next;
-    if (c + 1 < nc) next = chunk_decay(a, ws.c, qs + (c + 1) * GC, min(GC, len - (c + 1) * GC), h, lane);      // in flight
-    const float f0 = dc.dt.x * expf(dc.total - dc.b.x), f1 = dc.dt.y * expf(dc.total - dc.b.y), dec = expf(dc.total);
+    const RawDecay next = load_decay(a, ws.c, qs + (c + 1) * GC, len - (c + 1) * GC, h, lane);      // in flight until the products are done
     cp_async_wait<kSsdStages - 2>();
     __syncthreads();                    // chunk c has landed, and everyone is done with the stage that is refilled now
     load(c + kSsdStages - 1);
@@ -427,6 +536,7 @@ __global__ void __launch_bounds__(256) ssd_state_kernel(const SsdArgs a, const S
         mma_bf16(acc[j + 1], xl, bb[2], bb[3]);
       }
     }
+    factors(next);
   }
   cp_async_wait_all();
   if (slot < 0) return;
@@ -450,165 +560,177 @@ __global__ void __launch_bounds__(256) ssd_state_kernel(const SsdArgs a, const S
     }
 }
 
-// Outputs of one chunk and head over all its value columns; a warp takes half of the tokens of NV value tiles.
+// Outputs of one chunk and HB heads of a group over all their value columns: B and C, and the product C B^T, serve all of them.  A warp takes half of the
+// tokens of NV value tiles.  While a head's outputs are formed, the next one's x is on its way.
 template <int NV>
-__global__ void __launch_bounds__(256, NV <= 2 ? 2 : 1) ssd_output_kernel(const SsdArgs a, const SsdWs ws) {
+__global__ void __launch_bounds__(256, NV <= 2 ? 2 : 1) ssd_output_kernel(const SsdArgs a, const SsdWs ws, int HB) {
   constexpr int LA = GC + 8;
   extern __shared__ __align__(16) __nv_bfloat16 o16[];
   const int LN = a.NP + 8, LX = ws.npt * 16 + 8, LO = ws.npt * 16 + 4;
-  __nv_bfloat16 *sC = o16, *sX = sC + GC * LN, *sB = sX + GC * LX;
-  __nv_bfloat16 *sAh = sB + GC * LN, *sAl = sAh + GC * LA;
-  float* so = (float*)sB;                                      // [GC][LO], over B and A once they are used
+  __nv_bfloat16 *sC = o16, *sX0 = sC + GC * LN, *sAh = sX0 + 2 * GC * LX, *sAl = sAh + GC * LA, *sB = sAl + GC * LA;
+  float* so = (float*)sB;                                      // [GC][LO], over B once it is used
   __shared__ float s_b[GC], s_dt[GC];
   pdl_trigger();
   pdl_wait();
-  const int c = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, g = h / (a.H / a.G);
+  const int c = blockIdx.x, h0 = blockIdx.y * HB, seq = blockIdx.z, tid = threadIdx.x, g = h0 / (a.H / a.G);
   const int warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
   const int len = a.q_len[seq], qs = a.q_start[seq];
   if (c * GC >= len) return;
   const bool with_state = c > 0 || !(a.ctx_len[seq] - len == 0 || a.slot[seq] < 0);
   const int n = min(GC, len - c * GC), t0 = qs + c * GC;
   const int n8 = a.NP / 8, p8 = ws.npt * 2;
-  for (int i = tid; i < 2 * GC * n8; i += 256) {
-    const int which = i / (GC * n8), t = (i / n8) % GC, x = i % n8 * 8;
+  for (GridWalk w(tid, 256, n8); w.r < 2 * GC; w.next()) {
+    const int which = w.r >= GC, t = w.r - which * GC, x = w.c * 8;
     __nv_bfloat16* dst = (which ? sB : sC) + t * LN + x;
     if (t < n) cp_async16(s32(dst), (which ? ws.c.B : ws.c.C) + ((size_t)(t0 + t) * a.G + g) * a.NP + x);
     else *(uint4*)dst = make_uint4(0u, 0u, 0u, 0u);
   }
+  auto load_x = [&](int k) {
+    for (GridWalk w(tid, 256, p8); w.r < GC; w.next()) {
+      const int t = w.r, x = w.c * 8;
+      __nv_bfloat16* dst = sX0 + (k & 1) * GC * LX + t * LX + x;
+      if (t < n && x < a.PP) cp_async16(s32(dst), ws.c.x + ((size_t)(t0 + t) * a.H + h0 + k) * a.PP + x);
+      else *(uint4*)dst = make_uint4(0u, 0u, 0u, 0u);
+    }
+  };
+  load_x(0);
   cp_async_commit();
-  for (int i = tid; i < GC * p8; i += 256) {
-    const int t = i / p8, x = i % p8 * 8;
-    __nv_bfloat16* dst = sX + t * LX + x;
-    if (t < n && x < a.PP) cp_async16(s32(dst), ws.c.x + ((size_t)(t0 + t) * a.H + h) * a.PP + x);
-    else *(uint4*)dst = make_uint4(0u, 0u, 0u, 0u);
-  }
-  cp_async_commit();
-  if (warp == 0) {
-    const ChunkDecay dc = chunk_decay(a, ws.c, t0, n, h, lane);
-    *(float2*)(s_b + 2 * lane) = dc.b;
-    *(float2*)(s_dt + 2 * lane) = dc.dt;
-  }
-  cp_async_wait<1>();
+  RawDecay raw = {};                                            // warp 0's
+  if (warp == 0) raw = load_decay(a, ws.c, t0, n, h0, lane);
+  cp_async_wait<0>();
   __syncthreads();
-  {                                                            // C B^T with its decays: warp = 16 tokens x 32 earlier ones
-    const int m0 = (warp >> 1) * 16, n0 = (warp & 1) * 32;
-    float acc[4][4] = {};
-    if (n0 <= m0 + 15) {
-      for (int k0 = 0; k0 < a.NP; k0 += 16) {
-        uint32_t ca[4];
-        ldsm4(s32(sC + (m0 + (lane & 15)) * LN + k0 + (lane >> 4) * 8), ca);
+  // C B^T: warp = 16 tokens x 32 earlier ones
+  const int m0 = (warp >> 1) * 16, n0 = (warp & 1) * 32;
+  float cb[4][4] = {};
+  if (n0 <= m0 + 15) {
+    for (int k0 = 0; k0 < a.NP; k0 += 16) {
+      uint32_t ca[4];
+      ldsm4(s32(sC + (m0 + (lane & 15)) * LN + k0 + (lane >> 4) * 8), ca);
 #pragma unroll
-        for (int j = 0; j < 4; j += 2) {
-          uint32_t bb[4];
-          ldsm4(s32(sB + (n0 + (j + (lane >> 4)) * 8 + (lane & 7)) * LN + k0 + ((lane >> 3) & 1) * 8), bb);
-          mma_bf16(acc[j], ca, bb[0], bb[1]);
-          mma_bf16(acc[j + 1], ca, bb[2], bb[3]);
-        }
+      for (int j = 0; j < 4; j += 2) {
+        uint32_t bb[4];
+        ldsm4(s32(sB + (n0 + (j + (lane >> 4)) * 8 + (lane & 7)) * LN + k0 + ((lane >> 3) & 1) * 8), bb);
+        mma_bf16(cb[j], ca, bb[0], bb[1]);
+        mma_bf16(cb[j + 1], ca, bb[2], bb[3]);
       }
     }
+  }
+  const int vq = warp & 3, th = warp >> 2;
+  const bool vec = ((a.P | a.ldy) & 3) == 0 && ((uintptr_t)a.y & 15) == 0;
+  for (int k = 0; k < HB; k++) {
+    const int h = h0 + k;
+    const __nv_bfloat16* sX = sX0 + (k & 1) * GC * LX;
+    if (warp == 0) {
+      const ChunkDecay dc = chunk_decay(raw, lane);
+      *(float2*)(s_b + 2 * lane) = dc.b;
+      *(float2*)(s_dt + 2 * lane) = dc.dt;
+    }
+    cp_async_wait<0>();
+    __syncthreads();                                           // x and the decays of this head; the last one's outputs have been read
+    if (k + 1 < HB) {
+      load_x(k + 1);
+      if (warp == 0) raw = load_decay(a, ws.c, t0, n, h + 1, lane);
+    }
+    cp_async_commit();
 #pragma unroll
     for (int j = 0; j < 4; j++)
 #pragma unroll
       for (int hf = 0; hf < 2; hf++) {
         const int t = m0 + g4 + 8 * hf, s = n0 + 8 * j + 2 * t4;
-        const float x = s <= t ? acc[j][2 * hf] * expf(s_b[t] - s_b[s]) * s_dt[s] : 0.f;
-        const float y = s + 1 <= t ? acc[j][2 * hf + 1] * expf(s_b[t] - s_b[s + 1]) * s_dt[s + 1] : 0.f;
+        const float x = s <= t ? cb[j][2 * hf] * expf(s_b[t] - s_b[s]) * s_dt[s] : 0.f;
+        const float y = s + 1 <= t ? cb[j][2 * hf + 1] * expf(s_b[t] - s_b[s + 1]) * s_dt[s + 1] : 0.f;
         uint32_t hi, lo;
         split2(x, y, hi, lo);
         *(uint32_t*)(sAh + t * LA + s) = hi;
         *(uint32_t*)(sAl + t * LA + s) = lo;
       }
-  }
-  cp_async_wait<0>();
-  __syncthreads();
-  const int vq = warp & 3, th = warp >> 2;
-  float acc[NV][4][4];                                         // value tile vq + 4 i; columns = tokens 32 th + 8 j + 2 t4 (+ 1)
+    float acc[NV][4][4];                                       // value tile vq + 4 i; columns = tokens 32 th + 8 j + 2 t4 (+ 1)
 #pragma unroll
-  for (int i = 0; i < NV; i++)
+    for (int i = 0; i < NV; i++)
 #pragma unroll
-    for (int j = 0; j < 4; j++) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
-  if (with_state) {
-    const uint4* frag = ws.s + (chunk_slot(qs, seq, c) * a.H + h) * ws.npt * ws.kn * 64 + lane * 2;
-#pragma unroll 2
-    for (int kd = 0; kd < ws.kn; kd++) {
-      uint32_t cc[2][4];
+      for (int j = 0; j < 4; j++) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
+    if (with_state) {
+      const uint4* frag = ws.s + (chunk_slot(qs, seq, c) * a.H + h) * ws.npt * ws.kn * 64 + lane * 2;
+#pragma unroll 4
+      for (int kd = 0; kd < ws.kn; kd++) {
+        uint32_t cc[2][4];
 #pragma unroll
-      for (int m = 0; m < 2; m++) ldsm4(s32(sC + (32 * th + 16 * m + (lane >> 4) * 8 + (lane & 7)) * LN + kd * 16 + ((lane >> 3) & 1) * 8), cc[m]);
+        for (int m = 0; m < 2; m++) ldsm4(s32(sC + (32 * th + 16 * m + (lane >> 4) * 8 + (lane & 7)) * LN + kd * 16 + ((lane >> 3) & 1) * 8), cc[m]);
 #pragma unroll
-      for (int i = 0; i < NV; i++) {
-        const uint4* p = frag + ((size_t)min(vq + 4 * i, ws.npt - 1) * ws.kn + kd) * 64;
-        const uint4 xh = __ldg(p), xl = __ldg(p + 1);
-        const uint32_t sh[4] = {xh.x, xh.y, xh.z, xh.w}, sl[4] = {xl.x, xl.y, xl.z, xl.w};
+        for (int i = 0; i < NV; i++) {
+          const uint4* p = frag + ((size_t)min(vq + 4 * i, ws.npt - 1) * ws.kn + kd) * 64;
+          const uint4 xh = __ldg(p), xl = __ldg(p + 1);
+          const uint32_t sh[4] = {xh.x, xh.y, xh.z, xh.w}, sl[4] = {xl.x, xl.y, xl.z, xl.w};
 #pragma unroll
-        for (int m = 0; m < 2; m++) {
-          mma_bf16(acc[i][2 * m], sh, cc[m][0], cc[m][1]);
-          mma_bf16(acc[i][2 * m + 1], sh, cc[m][2], cc[m][3]);
-          mma_bf16(acc[i][2 * m], sl, cc[m][0], cc[m][1]);
-          mma_bf16(acc[i][2 * m + 1], sl, cc[m][2], cc[m][3]);
+          for (int m = 0; m < 2; m++) {
+            mma_bf16(acc[i][2 * m], sh, cc[m][0], cc[m][1]);
+            mma_bf16(acc[i][2 * m + 1], sh, cc[m][2], cc[m][3]);
+            mma_bf16(acc[i][2 * m], sl, cc[m][0], cc[m][1]);
+            mma_bf16(acc[i][2 * m + 1], sl, cc[m][2], cc[m][3]);
+          }
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 4; j++) {
+        const float2 b = *(const float2*)(s_b + 32 * th + 8 * j + 2 * t4);
+        const float e0 = expf(b.x), e1 = expf(b.y);
+#pragma unroll
+        for (int i = 0; i < NV; i++) {
+          acc[i][j][0] *= e0;
+          acc[i][j][1] *= e1;
+          acc[i][j][2] *= e0;
+          acc[i][j][3] *= e1;
+        }
+      }
+    }
+    __syncthreads();                                           // the decayed products of all warps
+#pragma unroll
+    for (int kt = 0; kt < GC / 16; kt++) {
+      if (kt * 16 >= 32 * th + 32) break;                      // later tokens than any of this warp's
+      uint32_t xa[NV][4];
+#pragma unroll
+      for (int i = 0; i < NV; i++)
+        ldsm4t(s32(sX + (kt * 16 + (lane >> 4) * 8 + (lane & 7)) * LX + min(vq + 4 * i, ws.npt - 1) * 16 + ((lane >> 3) & 1) * 8), xa[i]);
+#pragma unroll
+      for (int m = 0; m < 2; m++) {
+        const int at = (32 * th + 16 * m + (lane >> 4) * 8 + (lane & 7)) * LA + kt * 16 + ((lane >> 3) & 1) * 8;
+        uint32_t bh[4], bl[4];
+        ldsm4(s32(sAh + at), bh);
+        ldsm4(s32(sAl + at), bl);
+#pragma unroll
+        for (int i = 0; i < NV; i++) {
+          mma_bf16(acc[i][2 * m], xa[i], bh[0], bh[1]);
+          mma_bf16(acc[i][2 * m + 1], xa[i], bh[2], bh[3]);
+          mma_bf16(acc[i][2 * m], xa[i], bl[0], bl[1]);
+          mma_bf16(acc[i][2 * m + 1], xa[i], bl[2], bl[3]);
         }
       }
     }
 #pragma unroll
-    for (int j = 0; j < 4; j++) {
-      const float2 b = *(const float2*)(s_b + 32 * th + 8 * j + 2 * t4);
-      const float e0 = expf(b.x), e1 = expf(b.y);
-#pragma unroll
-      for (int i = 0; i < NV; i++) {
-        acc[i][j][0] *= e0;
-        acc[i][j][1] *= e1;
-        acc[i][j][2] *= e0;
-        acc[i][j][3] *= e1;
-      }
-    }
-  }
-#pragma unroll
-  for (int kt = 0; kt < GC / 16; kt++) {
-    if (kt * 16 >= 32 * th + 32) break;                        // later tokens than any of this warp's
-    uint32_t xa[NV][4];
-#pragma unroll
     for (int i = 0; i < NV; i++)
-      ldsm4t(s32(sX + (kt * 16 + (lane >> 4) * 8 + (lane & 7)) * LX + min(vq + 4 * i, ws.npt - 1) * 16 + ((lane >> 3) & 1) * 8), xa[i]);
+      if (vq + 4 * i < ws.npt) {
 #pragma unroll
-    for (int m = 0; m < 2; m++) {
-      const int at = (32 * th + 16 * m + (lane >> 4) * 8 + (lane & 7)) * LA + kt * 16 + ((lane >> 3) & 1) * 8;
-      uint32_t bh[4], bl[4];
-      ldsm4(s32(sAh + at), bh);
-      ldsm4(s32(sAl + at), bl);
+        for (int j = 0; j < 4; j++)
 #pragma unroll
-      for (int i = 0; i < NV; i++) {
-        mma_bf16(acc[i][2 * m], xa[i], bh[0], bh[1]);
-        mma_bf16(acc[i][2 * m + 1], xa[i], bh[2], bh[3]);
-        mma_bf16(acc[i][2 * m], xa[i], bl[0], bl[1]);
-        mma_bf16(acc[i][2 * m + 1], xa[i], bl[2], bl[3]);
+          for (int e = 0; e < 4; e++) so[(32 * th + 8 * j + 2 * t4 + (e & 1)) * LO + (vq + 4 * i) * 16 + g4 + 8 * (e >> 1)] = acc[i][j][e];
       }
-    }
-  }
-  __syncthreads();                                             // B and A have been read: the outputs take their place
-#pragma unroll
-  for (int i = 0; i < NV; i++)
-    if (vq + 4 * i < ws.npt) {
-#pragma unroll
-      for (int j = 0; j < 4; j++)
-#pragma unroll
-        for (int e = 0; e < 4; e++) so[(32 * th + 8 * j + 2 * t4 + (e & 1)) * LO + (vq + 4 * i) * 16 + g4 + 8 * (e >> 1)] = acc[i][j][e];
-    }
-  __syncthreads();
-  const float D = a.D[h];
-  const bool vec = ((a.P | a.ldy) & 3) == 0 && ((uintptr_t)a.y & 15) == 0;
-  GridWalk w(tid, 256, vec ? a.P / 4 : a.P);
+    __syncthreads();
+    const float D = a.D[h];
+    GridWalk w(tid, 256, vec ? a.P / 4 : a.P);
 #pragma unroll 4
-  for (; w.r < n; w.next()) {
-    const int t = w.r;
-    float* dst = a.y + (size_t)(t0 + t) * a.ldy + h * a.P;
-    if (vec) {
-      const int e = w.c * 4;
-      float4 o = *(const float4*)(so + t * LO + e);
-      const uint2 x = *(const uint2*)(sX + t * LX + e);
-      const float2 x0 = __bfloat1622float2(*(const __nv_bfloat162*)&x.x), x1 = __bfloat1622float2(*(const __nv_bfloat162*)&x.y);
-      o.x = fmaf(D, x0.x, o.x); o.y = fmaf(D, x0.y, o.y); o.z = fmaf(D, x1.x, o.z); o.w = fmaf(D, x1.y, o.w);
-      *(float4*)(dst + e) = o;
-    } else {
-      dst[w.c] = fmaf(D, __bfloat162float(sX[t * LX + w.c]), so[t * LO + w.c]);
+    for (; w.r < n; w.next()) {
+      const int t = w.r;
+      float* dst = a.y + (size_t)(t0 + t) * a.ldy + h * a.P;
+      if (vec) {
+        const int e = w.c * 4;
+        float4 o = *(const float4*)(so + t * LO + e);
+        const uint2 x = *(const uint2*)(sX + t * LX + e);
+        const float2 x0 = __bfloat1622float2(*(const __nv_bfloat162*)&x.x), x1 = __bfloat1622float2(*(const __nv_bfloat162*)&x.y);
+        o.x = fmaf(D, x0.x, o.x); o.y = fmaf(D, x0.y, o.y); o.z = fmaf(D, x1.x, o.z); o.w = fmaf(D, x1.y, o.w);
+        *(float4*)(dst + e) = o;
+      } else {
+        dst[w.c] = fmaf(D, __bfloat162float(sX[t * LX + w.c]), so[t * LO + w.c]);
+      }
     }
   }
 }
@@ -622,15 +744,19 @@ B200_API size_t b200_ssd_prefill_bytes(int T, int n_seqs, int H, int PP, int N, 
 
 template <int NV>
 static int launch_ssd_output(const SsdArgs& a, const SsdWs& w, int n_seqs, int max_q, cudaStream_t st) {
-  const size_t ba = (size_t)GC * 2 * (a.NP + 8 + 2 * (GC + 8)), tile = (size_t)GC * 4 * (w.npt * 16 + 4);
-  const size_t smem = (size_t)GC * 2 * (a.NP + 8 + w.npt * 16 + 8) + (ba > tile ? ba : tile);
+  const size_t b = (size_t)GC * 2 * (a.NP + 8), tile = (size_t)GC * 4 * (w.npt * 16 + 4);
+  const size_t smem = (size_t)GC * 2 * (a.NP + 8 + 2 * (w.npt * 16 + 8) + 2 * (GC + 8)) + (b > tile ? b : tile);
+  if (smem > 225 * 1024) return B200_ERR_BAD_ARG;
   static size_t configured = 0;
   if (smem > configured) {
     cudaError_t e = cudaFuncSetAttribute(ssd_output_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = smem;
   }
-  return launch_pdl(ssd_output_kernel<NV>, dim3((max_q + GC - 1) / GC, a.H, n_seqs), dim3(256), smem, st, a, w);
+  const int chunks = (max_q + GC - 1) / GC, rep = a.H / a.G;
+  int HB = 1;                                // heads to a CTA: more, as long as there are some CTAs to every SM
+  while (HB < 8 && rep % (2 * HB) == 0 && (long)chunks * n_seqs * a.H / (2 * HB) >= 4 * 148) HB *= 2;
+  return launch_pdl(ssd_output_kernel<NV>, dim3(chunks, a.H / HB, n_seqs), dim3(256), smem, st, a, w, HB);
 }
 
 // Prompts: T rows in all, max_q = longest portion of a sequence; ws: b200_ssd_prefill_bytes bytes, 256-byte aligned.  exact: token by token in fp32.

@@ -503,7 +503,8 @@ class HybridEngine(PagedEngine):
         self.delta_ws = ws("delta_ws", (max((ops.delta_chunk_bytes(T, self.max_batch, m.heads, m.dim, dv, m.log_decay) for m, dv in delta), default=0)
                                         if not self.exact else 0,), torch.uint8)
         ssd = [(b.spec.mixer, b.DV) for b in self.blocks if b.ssd is not None]
-        self.ssd_ws = ws("ssd_ws", (max((ops.ssd_prefill_bytes(T, self.max_batch, m.heads, dv, m.dim, m.groups, self.exact) for m, dv in ssd), default=0),), torch.uint8)
+        self.ssd_ws = ws("ssd_ws", (max((max(ops.ssd_prefill_bytes(T, self.max_batch, m.heads, dv, m.dim, m.groups, self.exact),
+                                               ops.ssd_decode_bytes(self.max_batch, m.heads, dv, m.dim, m.groups)) for m, dv in ssd), default=0),), torch.uint8)
         self.ssd_y = ws("ssd_y", (T * max((m.heads * m.vdim for m, _ in ssd), default=0),), f32)
         self.v_first = ws("v_first", (T * max((m.kv_heads * m.vdim for _, m, _ in attn if m.v_mix), default=0),), f32)
         # latent attention: rows in the latent space (all of a step's where the any-size kernel runs), and the expanded context of the others
@@ -785,11 +786,11 @@ class HybridEngine(PagedEngine):
         args = (proj, inner, inner + m.channels, w.conv, w.conv_b, w.dt_bias, w.A_log, w.D, r.state, r.ring, qs, ql, self.seq_lens, self.state_slot, n_seqs,
                 m.heads, m.vdim, m.dim, m.groups, b.DV, y)
         if decode:
-            ops.ssd_decode(*args)
+            ops.ssd_decode(*args, ws=self.ssd_ws)
         else:
             ops.ssd_prefill(*args, max_q=max_q, ws=self.ssd_ws, exact=self.exact)
         ops.group_norm(y, inner, m.norm_groups, b.o_norm, self.cfg.norm_eps, o32 if o32 is not None else o16, gate=proj[:, :inner])
-        return 2 if decode else 3 if self.exact else 4
+        return (2 if not ops.ssd_decode_bytes(n_seqs, m.heads, b.DV, m.dim, m.groups) else 3) if decode else 3 if self.exact else 4
 
     def _run_layers(self, T: int, decode: bool, n_seqs: int, max_q: int, pages: int) -> int:
         f32 = self.exact or (decode and T <= min(self.small_path_tokens, self.matvec_rows))

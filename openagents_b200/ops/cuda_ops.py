@@ -92,7 +92,7 @@ _SIGS = {
     "b200_group_norm": [_P, c_int, _P, c_int, c_int, c_int, c_int, _P, c_float, _P, _P, c_int, _P],
     "b200_delta_recurrent": _DELTA + [_P],
     "b200_delta_chunked": _DELTA + [c_int, c_int, _P, c_size_t, _P],
-    "b200_ssd_decode": _SSD + [_P],
+    "b200_ssd_decode": _SSD + [_P, c_size_t, _P],
     "b200_ssd_prefill": _SSD + [c_int, c_int, c_int, _P, c_size_t, _P],
     "b200_gla_chunked": [_P] + [c_int] * 7 + [_P] * 8 + [c_int] * 5 + [c_float] * 3 + [_P, _P, c_int, c_int, c_int, _P, c_size_t, _P],
     "b200_gla_recurrent": [_P] + [c_int] * 7 + [_P] * 8 + [c_int] * 5 + [c_float] * 3 + [_P, _P, c_int, _P],
@@ -121,6 +121,8 @@ def lib():
         L.b200_mixed_decode_prepared_words.restype = c_size_t
         L.b200_delta_chunk_bytes.argtypes = [c_int] * 5 + [c_float]
         L.b200_delta_chunk_bytes.restype = c_size_t
+        L.b200_ssd_decode_bytes.argtypes = [c_int] * 5
+        L.b200_ssd_decode_bytes.restype = c_size_t
         L.b200_ssd_prefill_bytes.argtypes = [c_int] * 7
         L.b200_ssd_prefill_bytes.restype = c_size_t
         L.b200_gla_chunk_bytes.argtypes = [c_int] * 6
@@ -673,11 +675,16 @@ def _ssd_args(proj, x_off, dt_off, conv, conv_b, dt_bias, A_log, D, state, ring,
             _p(slots), n_seqs, H, P, N, G, conv.shape[1], PP, _p(y), y.stride(0))
 
 
-def ssd_decode(*args):
+def ssd_decode_bytes(n_seqs, H, PP, N, G):
+    """Workspace of :func:`ssd_decode`."""
+    return lib().b200_ssd_decode_bytes(n_seqs, H, PP, N, G)
+
+
+def ssd_decode(*args, ws):
     """One token per sequence of a Mamba-2 layer: filter, recurrence and skip.  Arguments: the projections (fp32), their columns of [x, B, C] and of dt; ``conv`` fp32
     [channels, taps] and its bias; dt_bias, A_log, D [H]; ``state`` fp32 [slots, H, N, PP]; ``ring`` fp32 [slots, taps, channels]; q_start, q_len, ctx_len,
-    slots; n_seqs, H, P, N, G, PP; ``y`` fp32 [T, >= H * P]."""
-    _check(lib().b200_ssd_decode(*_ssd_args(*args), _st()), "ssd_decode")
+    slots; n_seqs, H, P, N, G, PP; ``y`` fp32 [T, >= H * P]; ``ws``: uint8 workspace."""
+    _check(lib().b200_ssd_decode(*_ssd_args(*args), _p(ws), ws.numel(), _st()), "ssd_decode")
 
 
 def ssd_prefill_bytes(T, n_seqs, H, PP, N, G, exact=False):

@@ -268,7 +268,8 @@ class Ssd:
         args = (rows, self.inner, self.inner + self.CC, self.conv.to(DEV), self.cb.to(DEV), self.dtb.to(DEV), self.A.to(DEV), self.D.to(DEV), state, ring, qs, ql, ctx, i32(*slots),
                 len(lens), self.H, self.P, self.N, self.G, self.PP, y)
         if kernel == "decode":
-            ops.ssd_decode(*args)
+            n = ops.ssd_decode_bytes(len(lens), self.H, self.PP, self.N, self.G)
+            ops.ssd_decode(*args, ws=torch.full((n,), 255, dtype=torch.uint8, device=DEV))
         else:
             exact = kernel == "exact"
             n = ops.ssd_prefill_bytes(rows.shape[0], len(lens), self.H, self.PP, self.N, self.G, exact)
