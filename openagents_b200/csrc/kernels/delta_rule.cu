@@ -38,21 +38,24 @@ constexpr int kDeltaRank = 1024;      // most ranks of the decay's projection
 constexpr float kUnitEps = 1e-6f;
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+// The same on the hardware's exponential and reciprocal (some 1e-7 relative), for operands that are rounded to two bf16 numbers.
+__device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 
 // ------------------------------------------------------------------ token by token
 
 // Decoding, and the prompts of the 32-bit mode.  One cluster per head and share of the sequences, whose CTAs share the value columns.  A CTA walks the tokens
 // of its sequences one by one; while it works on one, the projections of the next, and with a new sequence its state, are on their way into the other half of
-// a double buffer.  The state is updated in shared memory.  One pass over the old state gives both what the removal reads, u^T S, and the output's part
-// (r w)^T S; the rest of the output is two numbers per token:  o = (r w)^T S - (r . c) (u^T S) + (r . k) v.
+// a double buffer.  The state is updated in shared memory.  With n = 1 / (sum k^2 + 1e-6), R = k^T S and p = (r w)^T S, from one pass over the old state,
+//   o = p - n (r . a k) R + (r . k) v        S' = diag(w) S - a k (n R) + k v^T
+// so a token needs three sums over the channels and one reduction over the state's rows.
 __device__ __forceinline__ void cp_async4(void* dst, const float* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(s32(dst)), "l"(src) : "memory");
 }
 struct DeltaLayout {                       // floats of shared memory
-  int state, row, ch, ur, x, read, red, total;      // offsets; state and row: of the first of two buffers
+  int state, row, ch, kr, x, z, read, red, total;      // offsets; state and row: of the first of two buffers
   int state_n, row_n;                      // sizes of one buffer
 };
-__host__ __device__ inline DeltaLayout delta_layout(int dim, int W, int rank8) {
+static DeltaLayout delta_layout(int dim, int W, int rank8) {
   DeltaLayout l;
   const int groups = 256 / (W / 4);
   auto up4 = [](int n) { return (n + 3) & ~3; };
@@ -61,39 +64,64 @@ __host__ __device__ inline DeltaLayout delta_layout(int dim, int W, int rank8) {
   l.state = 0;
   l.row = 2 * l.state_n;
   l.ch = l.row + 2 * l.row_n;
-  l.ur = l.ch + 4 * dim;
-  l.x = l.ur + up4(2 * dim);
-  l.read = l.x + rank8;
+  l.kr = l.ch + 4 * dim;
+  l.x = l.kr + up4(2 * dim);
+  l.z = l.x + rank8;
+  l.read = l.z + up4(dim);
   l.red = l.read + W;
   l.total = l.red + groups * 2 * W;
   return l;
 }
+constexpr int kRowPieces = 3;              // elements of a projection row that a thread fetches without working out their places again
+
+// DIM, NV: channels and float4 columns of a CTA's share of a head, where they are known (0: not).
+template <int DIM, int NV>
 __global__ void __launch_bounds__(256, 4) delta_recurrent_kernel(const DeltaArgs a, int n_seqs, const DeltaLayout l) {
   extern __shared__ __align__(16) float sm[];
   cg::cluster_group cluster = cg::this_cluster();
-  const int CL = cluster.num_blocks(), part = cluster.block_rank();
-  const int nv_all = a.VP >> 2, nv = nv_all / CL, W = nv * 4, e0 = part * W;     // this CTA's columns [e0, e0 + W)
+  const int CL = cluster.num_blocks(), part = cluster.block_rank(), dim = DIM ? DIM : a.dim;
+  const int nv_all = a.VP >> 2, nv = NV ? NV : nv_all / CL, W = nv * 4, e0 = part * W;     // this CTA's columns [e0, e0 + W)
   const int groups = 256 / nv;
-  float4* s_ch = (float4*)(sm + l.ch);     // [dim] (w, c, k, -)
-  float2* s_ur = (float2*)(sm + l.ur);     // [dim] (u, r w)
-  float *s_x = sm + l.x, *s_read = sm + l.read, *s_red = sm + l.red;
-  __shared__ float red[3][8], red1[32];
+  float4* s_ch = (float4*)(sm + l.ch);     // [dim] (w, a k, k, -)
+  float2* s_kr = (float2*)(sm + l.kr);     // [dim] (k, r w)
+  float *s_x = sm + l.x, *s_z = sm + l.z, *s_read = sm + l.read, *s_red = sm + l.red;
+  __shared__ float red[3][8], red1[8];
   __shared__ float s_part[2];              // this CTA's sum of squares, by token parity
   pdl_trigger();
   const int h = blockIdx.x / CL, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   // TPC threads share a channel's low-rank product; its weights are read while the projection still runs
   int TPC = 1;
-  while (TPC < 8 && a.dim * TPC * 2 <= 256) TPC *= 2;
+  while (TPC < 8 && dim * TPC * 2 <= 256) TPC *= 2;
   const int ch = tid / TPC, sub = tid % TPC;
-  const bool mine = ch < a.dim;
-  const __nv_bfloat16* wrow = a.w2 + (size_t)(h * a.dim + (mine ? ch : 0)) * a.rank8;
+  const __nv_bfloat16* wrow = a.w2 + (size_t)(h * dim + (ch < dim ? ch : 0)) * a.rank8;
   uint4 held[4];
 #pragma unroll
-  for (int i = 0; i < 4; i++) held[i] = mine && (sub + i * TPC) * 8 < a.rank8 ? ((const uint4*)wrow)[sub + i * TPC] : make_uint4(0u, 0u, 0u, 0u);
-  const float w0 = mine ? a.w0[h * a.dim + ch] : 0.f, ab = mine ? a.ab[h * a.dim + ch] : 0.f;
+  for (int i = 0; i < 4; i++) held[i] = ch < dim && (sub + i * TPC) * 8 < a.rank8 ? ((const uint4*)wrow)[sub + i * TPC] : make_uint4(0u, 0u, 0u, 0u);
+  const float w0 = tid < dim ? a.w0[h * dim + tid] : 0.f, ab = tid < dim ? a.ab[h * dim + tid] : 0.f;
   const float wo = (tid < W && e0 + tid < a.vdim) ? a.norm[h * a.vdim + e0 + tid] : 0.f;
-  const int grp = tid / nv, col = tid % nv, rka = (3 * a.dim + 3) & ~3;
+  const int grp = tid / nv, col = tid % nv, rka = (3 * dim + 3) & ~3;
   const bool active = grp < groups;
+  // element i of a row as kept in shared memory: its column in the projections (< 0: zero)
+  const int row_n = rka + 2 * W + a.rank8;
+  auto column = [&](int i) {
+    if (i < 3 * dim) {
+      const int which = i / dim;
+      return (which == 0 ? a.r_off : which == 1 ? a.k_off : a.a_off) + h * dim + i - which * dim;
+    }
+    i -= rka;
+    if (i < 0) return -1;
+    if (i < 2 * W) {
+      const int e = i < W ? i : i - W;
+      return e0 + e < a.vdim ? (i < W ? a.v_off : a.g_off) + h * a.vdim + e0 + e : -1;
+    }
+    return i - 2 * W < a.rank ? a.x_off + i - 2 * W : -1;
+  };
+  const uint32_t with = __ballot_sync(0xffffffffu, ch < dim);      // whole groups of TPC threads
+  int piece[kRowPieces];
+#pragma unroll
+  for (int k = 0; k < kRowPieces; k++) piece[k] = tid + 256 * k < row_n ? column(tid + 256 * k) : -1;
+  for (int i = tid; i < 2 * row_n; i += 256)
+    if (column(i % row_n) < 0) sm[l.row + i / row_n * l.row_n + i % row_n] = 0.f;       // stays zero
   pdl_wait();
   struct Seq { int n, t0, slot; bool fresh; };
   auto meta = [&](int b) {
@@ -106,38 +134,28 @@ __global__ void __launch_bounds__(256, 4) delta_recurrent_kernel(const DeltaArgs
     }
     return q;
   };
-  auto state_of = [&](int slot) { return (float4*)(a.state + ((size_t)max(slot, 0) * a.H + h) * a.dim * a.VP) + part * nv; };
+  auto state_of = [&](int slot) { return (float4*)(a.state + ((size_t)max(slot, 0) * a.H + h) * dim * a.VP) + part * nv + (size_t)grp * nv_all + col; };
+  const int ds = groups * nv;              // from one of a thread's state rows to the next, in shared memory
+  const size_t dg = (size_t)groups * nv_all;
   auto fetch_row = [&](int t, int buf) {
     const float* src = a.in + (size_t)t * a.ld;
     float* dst = sm + l.row + buf * l.row_n;
-    for (int d = tid; d < a.dim; d += 256) {
-      const int c = h * a.dim + d;
-      cp_async4(dst + d, src + a.r_off + c);
-      cp_async4(dst + a.dim + d, src + a.k_off + c);
-      cp_async4(dst + 2 * a.dim + d, src + a.a_off + c);
-    }
-    for (int e = tid; e < W; e += 256) {
-      const bool live = e0 + e < a.vdim;
-      const int c = h * a.vdim + e0 + e;
-      if (live) {
-        cp_async4(dst + rka + e, src + a.v_off + c);
-        cp_async4(dst + rka + W + e, src + a.g_off + c);
-      } else {
-        dst[rka + e] = dst[rka + W + e] = 0.f;
-      }
-    }
-    for (int r = tid; r < a.rank8; r += 256) {
-      if (r < a.rank) cp_async4(dst + rka + 2 * W + r, src + a.x_off + r);
-      else dst[rka + 2 * W + r] = 0.f;
+#pragma unroll
+    for (int k = 0; k < kRowPieces; k++)
+      if (piece[k] >= 0) cp_async4(dst + tid + 256 * k, src + piece[k]);
+    for (int i = tid + 256 * kRowPieces; i < row_n; i += 256) {
+      const int c = column(i);
+      if (c >= 0) cp_async4(dst + i, src + c);
     }
   };
   auto fetch_state = [&](const Seq& q, int buf) {
-    float4* dst = (float4*)(sm + l.state + buf * l.state_n);
-    const float4* src = state_of(q.slot);
     if (!active) return;
-    for (int d = grp; d < a.dim; d += groups) {          // the thread that will work on it: no barrier between this and its use but the copy's own
-      if (!q.fresh) cp_async16(s32(dst + d * nv + col), src + (size_t)d * nv_all + col);
-      else dst[d * nv + col] = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4* dst = (float4*)(sm + l.state + buf * l.state_n) + grp * nv + col;
+    const float4* src = state_of(q.slot);
+#pragma unroll 4
+    for (int d = grp; d < dim; d += groups, dst += ds, src += dg) {
+      if (!q.fresh) cp_async16(s32(dst), src);
+      else *dst = make_float4(0.f, 0.f, 0.f, 0.f);
     }
   };
   int b = blockIdx.y, i = 0, sbuf = 0, rbuf = 0, step = 0;
@@ -165,95 +183,107 @@ __global__ void __launch_bounds__(256, 4) delta_recurrent_kernel(const DeltaArgs
     cp_async_commit();
     const float* row = sm + l.row + rbuf * l.row_n;
     const float *s_v = row + rka, *s_g = s_v + W;
-    float4* S = (float4*)(sm + l.state + sbuf * l.state_n) + col;
+    float4* S = (float4*)(sm + l.state + sbuf * l.state_n) + grp * nv + col;
     for (int r = tid; r < a.rank8; r += 256) s_x[r] = tanhf(row[rka + 2 * W + r]);
-    float kk = 0.f, rr = 0.f, ar = 0.f;
-    if (mine && sub == 0) {
-      rr = row[ch];
-      kk = row[a.dim + ch];
-      ar = row[2 * a.dim + ch];
+    __syncthreads();
+    if (ch < dim) {
+      float z = 0.f;
+      auto dot = [&](uint4 q, int at) {
+        const __nv_bfloat162* p = (const __nv_bfloat162*)&q;
+        const float4 x0 = *(const float4*)(s_x + at), x1 = *(const float4*)(s_x + at + 4);
+        float2 f;
+        f = __bfloat1622float2(p[0]); z = fmaf(f.x, x0.x, z); z = fmaf(f.y, x0.y, z);
+        f = __bfloat1622float2(p[1]); z = fmaf(f.x, x0.z, z); z = fmaf(f.y, x0.w, z);
+        f = __bfloat1622float2(p[2]); z = fmaf(f.x, x1.x, z); z = fmaf(f.y, x1.y, z);
+        f = __bfloat1622float2(p[3]); z = fmaf(f.x, x1.z, z); z = fmaf(f.y, x1.w, z);
+      };
+#pragma unroll
+      for (int j = 0; j < 4; j++)
+        if ((sub + j * TPC) * 8 < a.rank8) dot(held[j], (sub + j * TPC) * 8);
+      for (int j = sub + 4 * TPC; j * 8 < a.rank8; j += TPC) dot(((const uint4*)wrow)[j], j * 8);
+      for (int o = 1; o < TPC; o <<= 1) z += __shfl_xor_sync(with, z, o);
+      if (sub == 0) s_z[ch] = z;
     }
     __syncthreads();
-    float z = 0.f;
-    auto dot = [&](uint4 q, int at) {
-      const __nv_bfloat162* p = (const __nv_bfloat162*)&q;
-      const float4 x0 = *(const float4*)(s_x + at), x1 = *(const float4*)(s_x + at + 4);
-      float2 f;
-      f = __bfloat1622float2(p[0]); z = fmaf(f.x, x0.x, z); z = fmaf(f.y, x0.y, z);
-      f = __bfloat1622float2(p[1]); z = fmaf(f.x, x0.z, z); z = fmaf(f.y, x0.w, z);
-      f = __bfloat1622float2(p[2]); z = fmaf(f.x, x1.x, z); z = fmaf(f.y, x1.y, z);
-      f = __bfloat1622float2(p[3]); z = fmaf(f.x, x1.z, z); z = fmaf(f.y, x1.w, z);
-    };
-#pragma unroll
-    for (int j = 0; j < 4; j++)
-      if ((sub + j * TPC) * 8 < a.rank8) dot(held[j], (sub + j * TPC) * 8);
-    for (int j = sub + 4 * TPC; j * 8 < a.rank8; j += TPC) dot(((const uint4*)wrow)[j], j * 8);
-    for (int o = 1; o < TPC; o <<= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
-    const float rate = sigmoid_f(ar + ab), w = expf(-a.decay * sigmoid_f(z + w0));
-    float q0 = warp_sum(kk * kk), q1 = warp_sum(rr * rate * kk), q2 = warp_sum(rr * kk);       // other lanes hold zeros
-    if (lane == 0) { red[0][warp] = q0; red[1][warp] = q1; red[2][warp] = q2; }
-    __syncthreads();
-    q0 = q1 = q2 = 0.f;
-#pragma unroll
-    for (int j = 0; j < 8; j++) { q0 += red[0][j]; q1 += red[1][j]; q2 += red[2][j]; }
-    const float inv = 1.f / sqrtf(q0 + kUnitEps), rc = q1 * inv, rk = q2;
-    if (mine && sub == 0) {
-      s_ch[ch] = make_float4(w, rate * kk * inv, kk, 0.f);
-      s_ur[ch] = make_float2(kk * inv, rr * w);
+    if (warp * 32 < dim) {                 // one channel per lane
+      float q0 = 0.f, q1 = 0.f, q2 = 0.f;
+      if (tid < dim) {
+        const float rr = row[tid], kk = row[dim + tid], rate = sigmoid_f(row[2 * dim + tid] + ab), w = expf(-a.decay * sigmoid_f(s_z[tid] + w0));
+        s_ch[tid] = make_float4(w, rate * kk, kk, 0.f);
+        s_kr[tid] = make_float2(kk, rr * w);
+        q0 = kk * kk;
+        q1 = rr * rate * kk;
+        q2 = rr * kk;
+      }
+      q0 = warp_sum(q0);
+      q1 = warp_sum(q1);
+      q2 = warp_sum(q2);
+      if (lane == 0) { red[0][warp] = q0; red[1][warp] = q1; red[2][warp] = q2; }
     }
     __syncthreads();
     if (active) {
       float4 rd = make_float4(0.f, 0.f, 0.f, 0.f), p = rd;
+      const float4* x4 = S;
 #pragma unroll 4
-      for (int d = grp; d < a.dim; d += groups) {
-        const float2 ur = s_ur[d];
-        const float4 x = S[d * nv];
-        rd.x = fmaf(ur.x, x.x, rd.x); rd.y = fmaf(ur.x, x.y, rd.y); rd.z = fmaf(ur.x, x.z, rd.z); rd.w = fmaf(ur.x, x.w, rd.w);
-        p.x = fmaf(ur.y, x.x, p.x); p.y = fmaf(ur.y, x.y, p.y); p.z = fmaf(ur.y, x.z, p.z); p.w = fmaf(ur.y, x.w, p.w);
+      for (int d = grp; d < dim; d += groups, x4 += ds) {
+        const float2 kr = s_kr[d];
+        const float4 x = *x4;
+        rd.x = fmaf(kr.x, x.x, rd.x); rd.y = fmaf(kr.x, x.y, rd.y); rd.z = fmaf(kr.x, x.z, rd.z); rd.w = fmaf(kr.x, x.w, rd.w);
+        p.x = fmaf(kr.y, x.x, p.x); p.y = fmaf(kr.y, x.y, p.y); p.z = fmaf(kr.y, x.z, p.z); p.w = fmaf(kr.y, x.w, p.w);
       }
       *(float4*)(s_red + (size_t)(grp * 2) * W + 4 * col) = rd;
       *(float4*)(s_red + (size_t)(grp * 2 + 1) * W + 4 * col) = p;
     }
     __syncthreads();
-    float ss = 0.f;
-    if (tid < W) {                         // W <= 256
-      float rd = 0.f, p = 0.f;
-#pragma unroll 4
-      for (int g = 0; g < groups; g++) {
-        rd += s_red[(size_t)(g * 2) * W + tid];
-        p += s_red[(size_t)(g * 2 + 1) * W + tid];
+    float o = 0.f;
+    if (warp * 32 < W) {                   // one column per lane; W <= 256
+      float q0 = 0.f, q1 = 0.f, q2 = 0.f;
+      for (int j = 0; j * 32 < dim; j++) { q0 += red[0][j]; q1 += red[1][j]; q2 += red[2][j]; }
+      const float inv = 1.f / (q0 + kUnitEps);
+      if (tid < W) {
+        float rd = 0.f, p = 0.f;
+#pragma unroll 8
+        for (int g = 0; g < groups; g++) {
+          rd += s_red[(size_t)(g * 2) * W + tid];
+          p += s_red[(size_t)(g * 2 + 1) * W + tid];
+        }
+        rd *= inv;
+        s_read[tid] = rd;
+        o = p - q1 * rd + q2 * s_v[tid];   // padding columns are zero
       }
-      s_read[tid] = rd;
-      const float o = p - rc * rd + rk * s_v[tid];
-      s_red[tid] = o;                      // this column's first partial sum has been read
-      ss = o * o;                          // padding columns are zero
+      const float ss = warp_sum(o * o);
+      if (lane == 0) red1[warp] = ss;
     }
-    ss = block_sum(ss, red1);              // its barriers also publish s_read
+    __syncthreads();
     if (active) {
       const float4 v = *(const float4*)(s_v + 4 * col), rd = *(const float4*)(s_read + 4 * col);
-      float4* dst = state_of(cur.slot) + col;
+      float4* dst = state_of(cur.slot);
       const bool keep = last && cur.slot >= 0;
+      float4* x4 = S;
 #pragma unroll 4
-      for (int d = grp; d < a.dim; d += groups) {
+      for (int d = grp; d < dim; d += groups, x4 += ds, dst += dg) {
         const float4 c = s_ch[d];
-        float4 x = S[d * nv];
+        float4 x = *x4;
         x.x = fmaf(c.x, x.x, fmaf(c.z, v.x, -c.y * rd.x));
         x.y = fmaf(c.x, x.y, fmaf(c.z, v.y, -c.y * rd.y));
         x.z = fmaf(c.x, x.z, fmaf(c.z, v.z, -c.y * rd.z));
         x.w = fmaf(c.x, x.w, fmaf(c.z, v.w, -c.y * rd.w));
-        if (!last) S[d * nv] = x;
-        else if (keep) dst[(size_t)d * nv_all] = x;
+        if (!last) *x4 = x;
+        else if (keep) *dst = x;
       }
     }
+    float ss = 0.f;
+    if (CL > 1 || warp * 32 < W)
+      for (int j = 0; j * 32 < W; j++) ss += red1[j];
     if (CL > 1) {
       if (tid == 0) s_part[step & 1] = ss;
       cluster.sync();
       ss = 0.f;
       for (int p = 0; p < CL; p++) ss += *cluster.map_shared_rank(&s_part[step & 1], p);
     }
-    const float r = 1.f / sqrtf(ss / (float)a.vdim + a.eps);
     if (tid < W) {
-      const float o = e0 + tid < a.vdim ? s_red[tid] * r * wo * sigmoid_f(s_g[tid]) : 0.f;
+      if (e0 + tid < a.vdim) o *= wo * sigmoid_f(s_g[tid]) / sqrtf(ss / (float)a.vdim + a.eps);
+      else o = 0.f;
       const size_t at = (size_t)(cur.t0 + i) * a.ldo + (size_t)h * a.VP + e0 + tid;
       if (a.out_f32) a.out_f32[at] = o;
       if (a.out_bf16) a.out_bf16[at] = __float2bfloat16(o);
@@ -309,12 +339,10 @@ B200_API int b200_delta_recurrent(const float* in, int ld, const int* offs, int 
   const DeltaLayout l = delta_layout(dim, VP / CL, rank8);
   const size_t smem = 4 * (size_t)l.total;
   if (smem > 200 * 1024) return B200_ERR_BAD_ARG;
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(delta_recurrent_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-    if (e != cudaSuccess) return (int)e;
-    configured = true;
-  }
+  const bool w64 = VP / CL == 64;
+  auto kern = w64 && dim == 64 ? delta_recurrent_kernel<64, 16> : w64 && dim == 128 ? delta_recurrent_kernel<128, 16> : delta_recurrent_kernel<0, 0>;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+  if (e != cudaSuccess) return (int)e;
   // shares of the sequences: no more CTAs than run at a time, all with about the same number of sequences
   const int fit = (int)(227 * 1024 / (smem + 1024)), resident = 148 * (fit < 1 ? 1 : fit > 4 ? 4 : fit);
   const int most = resident / (H * CL) > 1 ? resident / (H * CL) : 1, rounds = (n_seqs + most - 1) / most, shares = (n_seqs + rounds - 1) / rounds;
@@ -331,7 +359,7 @@ B200_API int b200_delta_recurrent(const float* in, int ld, const int* offs, int 
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = b200_pdl_enabled() ? 2 : 1;
-  return (int)cudaLaunchKernelEx(&cfg, delta_recurrent_kernel, a, n_seqs, l);
+  return (int)cudaLaunchKernelEx(&cfg, kern, a, n_seqs, l);
 }
 
 // ------------------------------------------------------------------ prompts: 64-token chunks on the tensor cores
@@ -358,11 +386,11 @@ __device__ __forceinline__ int in_block(int t, int s) { return t * 16 + ((((s >>
 constexpr int kRankSlice = 64;
 
 struct DeltaWs {                         // per (chunk slot, head); fragments of 32 lanes
-  uint4* r;                              // [DP / 16][4 token tiles of 16][lane][2]: R as the B operand of R S, values and remainders
-  uint4* g;                              // [DP / 16][DP / 16][lane][2]: G likewise
+  uint4* r;                              // [DP / 16][4 token tiles of 16][2][lane]: R as the B operand of R S, values and remainders
+  uint4* g;                              // [DP / 16][DP / 16][2][lane]: G likewise
   float4* q;                             // [value tiles][8 token tiles of 8][lane]: Q as accumulators
   float4* f;                             // [value tiles][DP / 8][lane]: F as accumulators
-  uint4* s;                              // [value tiles][DP / 16][lane][2]: the state at the chunk's start as the A operand
+  uint4* s;                              // [value tiles][DP / 16][2][lane]: the state at the chunk's start as the A operand
   int nvt;                               // value tiles of 16
 };
 
@@ -370,8 +398,8 @@ struct DeltaWs {                         // per (chunk slot, head); fragments of
 template <int DP>
 struct DeltaSmem {
   static constexpr int LQ = DP + 8, ROWS = GC * LQ, OP = 2 * ROWS * 2;      // OP: bytes of an operand
-  static constexpr int LW = kRankSlice + 8;
-  static constexpr int kScratch = (4 * 16 * 17 + 256 + GC + DP) * 4;         // fp32 diagonal blocks of M; column sums; unit-key factors; e^{b_C}
+  static constexpr int LW = kRankSlice + 8, THREADS = DP >= 128 ? 512 : 256;
+  static constexpr int kScratch = (4 * 16 * 17 + 2 * THREADS + GC + DP) * 4;         // fp32 diagonal blocks of M; column sums; unit-key factors; e^{b_C}
   static constexpr int kBlocks = 8 * 10 * kBlk * 2;                          // -M (diagonal: its inverse), N, A, -B
   static constexpr int kTail = OP > kBlocks ? OP : kBlocks;
   // only until the decays are known: tanh(x) in two parts and a slice of w2 over k, c, r; their product behind u
@@ -387,13 +415,13 @@ struct DeltaSmem {
 __device__ __forceinline__ int tri(int i, int j) { return i * (i + 1) / 2 + j; }
 
 template <int DP>
-__global__ void __launch_bounds__(256, DP <= 64 ? 2 : 1) delta_prepare_kernel(const DeltaArgs a, const DeltaWs ws) {
+__global__ void __launch_bounds__(DeltaSmem<DP>::THREADS, DP <= 64 ? 2 : 1) delta_prepare_kernel(const DeltaArgs a, const DeltaWs ws) {
   using L = DeltaSmem<DP>;
-  constexpr int LQ = L::LQ, LW = L::LW, NG = 256 / DP, TPT = GC / NG, KD = DP / 16;
+  constexpr int LQ = L::LQ, LW = L::LW, THREADS = L::THREADS, NW = THREADS / 32, NG = THREADS / (DP / 2), TPT = GC / NG, KD = DP / 16;
   extern __shared__ __align__(16) uint8_t smem[];
   float* sd = (float*)smem;                                      // [4][16][17]
   float* stot = sd + 4 * 16 * 17;                                // [NG][DP]
-  float* sinv = stot + 256;                                      // [GC]
+  float* sinv = stot + 2 * THREADS;                              // [GC]
   float* sdec = sinv + GC;                                       // [DP]
   __nv_bfloat16* sk = (__nv_bfloat16*)(smem + L::kScratch);      // values, then remainders, of each
   __nv_bfloat16 *sc = sk + 2 * L::ROWS, *sr = sc + 2 * L::ROWS, *su = sr + 2 * L::ROWS;
@@ -403,37 +431,40 @@ __global__ void __launch_bounds__(256, DP <= 64 ? 2 : 1) delta_prepare_kernel(co
   __nv_bfloat16* sw = sx + 2 * GC * LW;                          // [DP][LW]      }
   float* sz = (float*)(su + 2 * L::ROWS);                        // [GC][DP + 1]  }
   const int LV = ws.nvt * 16 + 8;
-  pdl_trigger();
   const int c = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
   pdl_wait();
   const int len = a.q_len[seq], qs = a.q_start[seq];
-  if (c * GC >= len) return;
+  if (c * GC >= len) {
+    pdl_trigger();
+    return;
+  }
   const int n = min(GC, len - c * GC), t0 = qs + c * GC;
   const float* in = a.in + (size_t)t0 * a.ld;
-  if (((a.vdim | a.dim | a.v_off | a.r_off | a.k_off | a.a_off | a.ld) & 3) == 0 && tid % GC < n) {      // rows read later, into L2 now
+  if (((a.vdim | a.dim | a.v_off | a.r_off | a.k_off | a.a_off | a.ld) & 3) == 0 && tid < 4 * GC && tid % GC < n) {      // rows read later, into L2 now
     const int what = tid / GC;
     const float* p = in + (size_t)(tid % GC) * a.ld + (what == 0 ? a.k_off + h * a.dim : what == 1 ? a.r_off + h * a.dim : what == 2 ? a.a_off + h * a.dim : a.v_off + h * a.vdim);
     prefetch_l2(p, (what == 3 ? a.vdim : a.dim) * 4);
   }
-  // ---- z = W2 tanh(x): 64 tokens x DP channels, 64 ranks at a time; warp = 16 tokens x half of the channels
+  // ---- z = W2 tanh(x): 64 tokens x DP channels, 64 ranks at a time; warp = 16 tokens x a share of the channels
   {
-    constexpr int NT = DP / 16;                                  // n8 tiles per warp
+    constexpr int NT = DP / 2 / NW;                              // n8 tiles per warp
     float acc[NT][4] = {};
-    const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * (DP / 2);
+    const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * NT * 8;
     for (int r0 = 0; r0 < a.rank; r0 += kRankSlice) {
       if (r0) __syncthreads();
       {
-        const int r = tid % kRankSlice, q = tid / kRankSlice;    // a thread: one rank of every fourth token
-        float x[GC / 4];
+        constexpr int TS = THREADS / kRankSlice;                 // a thread: one rank of every TS-th token
+        const int r = tid % kRankSlice, q = tid / kRankSlice;
+        float x[GC / TS];
 #pragma unroll
-        for (int i = 0; i < GC / 4; i++) x[i] = q + 4 * i < n && r0 + r < a.rank ? in[(size_t)(q + 4 * i) * a.ld + a.x_off + r0 + r] : 0.f;
+        for (int i = 0; i < GC / TS; i++) x[i] = q + TS * i < n && r0 + r < a.rank ? in[(size_t)(q + TS * i) * a.ld + a.x_off + r0 + r] : 0.f;
 #pragma unroll
-        for (int i = 0; i < GC / 4; i++) {
-          const float e = expf(-2.f * fabsf(x[i])), y = copysignf((1.f - e) / (1.f + e), x[i]);      // tanh
-          split_bf16(y, sx[(q + 4 * i) * LW + r], sx[GC * LW + (q + 4 * i) * LW + r]);
+        for (int i = 0; i < GC / TS; i++) {
+          const float e = __expf(-2.f * fabsf(x[i])), y = copysignf(__fdividef(1.f - e, 1.f + e), x[i]);      // tanh
+          split_bf16(y, sx[(q + TS * i) * LW + r], sx[GC * LW + (q + TS * i) * LW + r]);
         }
       }
-      for (int i = tid; i < DP * (kRankSlice / 8); i += 256) {
+      for (int i = tid; i < DP * (kRankSlice / 8); i += THREADS) {
         const int d = i / (kRankSlice / 8), r = i % (kRankSlice / 8) * 8;
         *(uint4*)(sw + d * LW + r) = d < a.dim && r0 + r < a.rank8 ? *(const uint4*)(a.w2 + (size_t)(h * a.dim + d) * a.rank8 + r0 + r) : make_uint4(0u, 0u, 0u, 0u);
       }
@@ -460,90 +491,109 @@ __global__ void __launch_bounds__(256, DP <= 64 ? 2 : 1) delta_prepare_kernel(co
 #pragma unroll
       for (int e = 0; e < 4; e++) sz[(m0 + g4 + 8 * (e >> 1)) * (DP + 1) + n0 + 8 * j + 2 * t4 + (e & 1)] = acc[j][e];
   }
-  {                                                              // unit keys: a warp takes eight tokens
-    float ss[8] = {};
+  {                                                              // unit keys: a warp takes KT tokens
+    constexpr int KT = GC / NW;
+    float ss[KT] = {};
     for (int d = lane; d < a.dim; d += 32) {
-      float k[8];
+      float x[KT];
 #pragma unroll
-      for (int i = 0; i < 8; i++) k[i] = warp * 8 + i < n ? in[(size_t)(warp * 8 + i) * a.ld + a.k_off + h * a.dim + d] : 0.f;
+      for (int i = 0; i < KT; i++) x[i] = warp * KT + i < n ? in[(size_t)(warp * KT + i) * a.ld + a.k_off + h * a.dim + d] : 0.f;
 #pragma unroll
-      for (int i = 0; i < 8; i++) ss[i] = fmaf(k[i], k[i], ss[i]);
+      for (int i = 0; i < KT; i++) ss[i] = fmaf(x[i], x[i], ss[i]);
     }
 #pragma unroll
-    for (int i = 0; i < 8; i++) {
+    for (int i = 0; i < KT; i++) {
       ss[i] = warp_sum(ss[i]);
-      if (lane == i) sinv[warp * 8 + i] = 1.f / sqrtf(ss[i] + kUnitEps);
+      if (lane == i) sinv[warp * KT + i] = 1.f / sqrtf(ss[i] + kUnitEps);
     }
   }
   __syncthreads();
-  // ---- running sums of the log decays, and the decayed operands: a thread owns one channel of TPT consecutive tokens
+  // ---- running sums of the log decays, and the decayed operands: a thread owns two channels of TPT consecutive tokens
   {
-    const int d = tid % DP, grp = tid / DP, ch = h * a.dim + d;
-    const bool live = d < a.dim;
-    const float w0 = live ? a.w0[ch] : 0.f, ab = live ? a.ab[ch] : 0.f;
-    float b[TPT], sum = 0.f;
+    const int d = tid % (DP / 2) * 2, grp = tid / (DP / 2), c0 = h * a.dim + d;
+    const bool l0 = d < a.dim, l1 = d + 1 < a.dim, even = ((a.dim | a.r_off | a.k_off | a.a_off | a.ld) & 1) == 0;
+    const float2 w0 = make_float2(l0 ? a.w0[c0] : 0.f, l1 ? a.w0[c0 + 1] : 0.f), ab = make_float2(l0 ? a.ab[c0] : 0.f, l1 ? a.ab[c0 + 1] : 0.f);
+    float2 b[TPT], sum = make_float2(0.f, 0.f);
 #pragma unroll
     for (int i = 0; i < TPT; i++) {
       const int t = grp * TPT + i;
-      if (live && t < n) sum -= a.decay * sigmoid_f(sz[t * (DP + 1) + d] + w0);
+      if (t < n) {
+        if (l0) sum.x -= a.decay * sigmoid_fast(sz[t * (DP + 1) + d] + w0.x);
+        if (l1) sum.y -= a.decay * sigmoid_fast(sz[t * (DP + 1) + d + 1] + w0.y);
+      }
       b[i] = sum;
     }
-    stot[grp * DP + d] = sum;
+    *(float2*)(stot + grp * DP + d) = sum;
     __syncthreads();
-    float before = 0.f, total = 0.f;
+    float2 before = make_float2(0.f, 0.f), total = before;
 #pragma unroll
     for (int g = 0; g < NG; g++) {
-      const float x = stot[g * DP + d];
-      if (g < grp) before += x;
-      total += x;
+      const float2 x = *(const float2*)(stot + g * DP + d);
+      if (g < grp) {
+        before.x += x.x;
+        before.y += x.y;
+      }
+      total.x += x.x;
+      total.y += x.y;
     }
-    if (grp == 0) sdec[d] = expf(total);
-    float eb = expf(before);                                     // e^{b_(t-1)}
-    constexpr int LB = TPT < 8 ? TPT : 8;
+    if (grp == 0) *(float2*)(sdec + d) = make_float2(expf(total.x), expf(total.y));
+    float2 eb = make_float2(__expf(before.x), __expf(before.y));      // e^{b_(t-1)}
+    auto pair = [&](const float* p, bool row) -> float2 {
+      if (!row || !l0) return make_float2(0.f, 0.f);
+      if (even) return __ldg((const float2*)p);                  // an even head size: both channels exist
+      return make_float2(__ldg(p), l1 ? __ldg(p + 1) : 0.f);
+    };
+    constexpr int LB = TPT < 4 ? TPT : 4;
 #pragma unroll
     for (int i0 = 0; i0 < TPT; i0 += LB) {
-      float r[LB], k[LB], x[LB];
+      float2 r[LB], k[LB], x[LB];
 #pragma unroll
       for (int i = 0; i < LB; i++) {
         const int t = grp * TPT + i0 + i;
-        const float* row = in + (size_t)t * a.ld + ch;
-        const bool ok = live && t < n;
-        r[i] = ok ? __ldg(row + a.r_off) : 0.f;
-        k[i] = ok ? __ldg(row + a.k_off) : 0.f;
-        x[i] = ok ? __ldg(row + a.a_off) : 0.f;
+        const float* row = in + (size_t)t * a.ld + c0;
+        r[i] = pair(row + a.r_off, t < n);
+        k[i] = pair(row + a.k_off, t < n);
+        x[i] = pair(row + a.a_off, t < n);
       }
 #pragma unroll
       for (int i = 0; i < LB; i++) {
         const int t = grp * TPT + i0 + i, at = t * LQ + d;
-        const float e = expf(before + b[i0 + i]), ie = 1.f / e, u = k[i] * sinv[t];
-        auto put = [&](__nv_bfloat16* p, float v) { split_bf16(v, p[at], p[L::ROWS + at]); };
-        put(sr, r[i] * e);
-        put(su, u * eb);
-        put(sk, k[i] * ie);
-        put(sc, -sigmoid_f(x[i] + ab) * u * ie);                 // stored negated: every product with it is taken off
-        eb = e;
+        const float ex = __expf(before.x + b[i0 + i].x), ey = __expf(before.y + b[i0 + i].y), inv = sinv[t];
+        const float ix = __fdividef(1.f, ex), iy = __fdividef(1.f, ey), ux = k[i].x * inv, uy = k[i].y * inv;
+        auto put = [&](__nv_bfloat16* p, float vx, float vy) {
+          uint32_t hi, lo;
+          split2(vx, vy, hi, lo);
+          *(uint32_t*)(p + at) = hi;
+          *(uint32_t*)(p + L::ROWS + at) = lo;
+        };
+        put(sr, r[i].x * ex, r[i].y * ey);
+        put(su, ux * eb.x, uy * eb.y);
+        put(sk, k[i].x * ix, k[i].y * iy);
+        put(sc, -sigmoid_fast(x[i].x + ab.x) * ux * ix, -sigmoid_fast(x[i].y + ab.y) * uy * iy);      // negated: every product with it is taken off
+        eb = make_float2(ex, ey);
       }
     }
   }
   __syncthreads();                                               // sz is no longer needed: blocks and v take its place
   if (((a.vdim | a.v_off | a.ld) & 3) == 0) {
-    for (int i = tid; i < GC * ws.nvt * 4; i += 256) {
+    for (int i = tid; i < GC * ws.nvt * 4; i += THREADS) {
       const int t = i / (ws.nvt * 4), e = i % (ws.nvt * 4) * 4;
       float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
       if (t < n && e < a.vdim) x = __ldg((const float4*)(in + (size_t)t * a.ld + a.v_off + h * a.vdim + e));
       *(uint2*)(sv + t * LV + e) = make_uint2(pack_bf2(__float2bfloat16(x.x), __float2bfloat16(x.y)), pack_bf2(__float2bfloat16(x.z), __float2bfloat16(x.w)));
     }
   } else {
-    for (int i = tid; i < GC * ws.nvt * 16; i += 256) {
+    for (int i = tid; i < GC * ws.nvt * 16; i += THREADS) {
       const int t = i / (ws.nvt * 16), e = i % (ws.nvt * 16);
       sv[t * LV + e] = __float2bfloat16(t < n && e < a.vdim ? in[(size_t)t * a.ld + a.v_off + h * a.vdim + e] : 0.f);
     }
   }
-  // ---- the four triangular matrices, 40 blocks of 16 x 16, five per warp: (u, r) x (c, k)
-  float blocks[5][2][4];
+  // ---- the four triangular matrices, 40 blocks of 16 x 16, BPW per warp: (u, r) x (c, k)
+  constexpr int BPW = (40 + NW - 1) / NW;
+  float blocks[BPW][2][4];
 #pragma unroll
-  for (int q = 0; q < 5; q++) {
-    const int unit = warp * 5 + q, mat = unit / 10, blk = unit % 10;        // mat 0: u c (-M), 1: u k (N), 2: r k (A), 3: r c (-B)
+  for (int q = 0; q < BPW; q++) {
+    const int unit = min(warp * BPW + q, 39), mat = unit / 10, blk = unit % 10;        // mat 0: u c (-M), 1: u k (N), 2: r k (A), 3: r c (-B)
     const int i = blk >= 6 ? 3 : blk >= 3 ? 2 : blk >= 1 ? 1 : 0, j = blk - i * (i + 1) / 2;
     const __nv_bfloat16 *X = mat < 2 ? su : sr, *Y = (mat == 0 || mat == 3) ? sc : sk;
     float (&acc)[2][4] = blocks[q];
@@ -586,8 +636,9 @@ __global__ void __launch_bounds__(256, DP <= 64 ? 2 : 1) delta_prepare_kernel(co
   }
   __syncthreads();
 #pragma unroll
-  for (int q = 0; q < 5; q++) {
-    const int unit = warp * 5 + q, mat = unit / 10, blk = unit % 10;
+  for (int q = 0; q < BPW; q++) {
+    if (warp * BPW + q >= 40) break;
+    const int unit = warp * BPW + q, mat = unit / 10, blk = unit % 10;
     const int i = blk >= 6 ? 3 : blk >= 3 ? 2 : blk >= 1 ? 1 : 0, j = blk - i * (i + 1) / 2;
     float (&acc)[2][4] = blocks[q];
     __nv_bfloat16* hi = sb + (mat * 2) * 10 * kBlk + blk * kBlk;
@@ -674,7 +725,7 @@ __global__ void __launch_bounds__(256, DP <= 64 ? 2 : 1) delta_prepare_kernel(co
     as_operand(x, xh[i], xl[i]);
   };
   const size_t slot = chunk_slot(qs, seq, c) * a.H + h;
-  for (int cb = warp; cb < KD + ws.nvt; cb += 8) {
+  for (int cb = warp; cb < KD + ws.nvt; cb += NW) {
     uint32_t xh[4][4], xl[4][4], bh[4], bl[4];
     if (cb < KD) {                                               // 16 key channels: R and G
       const int d0 = cb * 16;
@@ -682,7 +733,7 @@ __global__ void __launch_bounds__(256, DP <= 64 ? 2 : 1) delta_prepare_kernel(co
       for (int i = 0; i < 4; i++) {
         solve(i, u[i], xh, xl);
       }
-      uint4* dst = ws.r + (slot * KD + cb) * 4 * 64 + lane * 2;
+      uint4* dst = ws.r + (slot * KD + cb) * 4 * 64 + lane;
 #pragma unroll
       for (int i = 0; i < 4; i++) {
         float z[2][4];
@@ -695,9 +746,9 @@ __global__ void __launch_bounds__(256, DP <= 64 ? 2 : 1) delta_prepare_kernel(co
         uint32_t hi[4], lo[4];
         as_operand(z, hi, lo);                                   // tiles (d 0-7, t 0-7), (d 8-15, t 0-7), (d 0-7, t 8-15), (d 8-15, t 8-15)
         dst[i * 64] = make_uint4(transpose_8x8(hi[0]), transpose_8x8(hi[1]), transpose_8x8(hi[2]), transpose_8x8(hi[3]));
-        dst[i * 64 + 1] = make_uint4(transpose_8x8(lo[0]), transpose_8x8(lo[1]), transpose_8x8(lo[2]), transpose_8x8(lo[3]));
+        dst[i * 64 + 32] = make_uint4(transpose_8x8(lo[0]), transpose_8x8(lo[1]), transpose_8x8(lo[2]), transpose_8x8(lo[3]));
       }
-      uint4* gd = ws.g + (slot * KD + cb) * KD * 64 + lane * 2;
+      uint4* gd = ws.g + (slot * KD + cb) * KD * 64 + lane;
 #pragma unroll
       for (int jn = 0; jn < KD; jn++) {
         float z[2][4] = {};
@@ -718,7 +769,7 @@ __global__ void __launch_bounds__(256, DP <= 64 ? 2 : 1) delta_prepare_kernel(co
         uint32_t hi[4], lo[4];
         as_operand(z, hi, lo);
         gd[jn * 64] = make_uint4(transpose_8x8(hi[0]), transpose_8x8(hi[1]), transpose_8x8(hi[2]), transpose_8x8(hi[3]));
-        gd[jn * 64 + 1] = make_uint4(transpose_8x8(lo[0]), transpose_8x8(lo[1]), transpose_8x8(lo[2]), transpose_8x8(lo[3]));
+        gd[jn * 64 + 32] = make_uint4(transpose_8x8(lo[0]), transpose_8x8(lo[1]), transpose_8x8(lo[2]), transpose_8x8(lo[3]));
       }
     } else {                                                     // 16 value columns: Q and F
       const int vb = cb - KD;
@@ -771,6 +822,7 @@ __global__ void __launch_bounds__(256, DP <= 64 ? 2 : 1) delta_prepare_kernel(co
       }
     }
   }
+  pdl_trigger();                                                 // late: the sequential kernel behind this one wants its CTAs spread over idle SMs
 }
 
 constexpr int state_stages(int dp) { return dp >= 128 ? 2 : 4; }
@@ -819,7 +871,7 @@ __global__ void __launch_bounds__(128) delta_state_kernel(const DeltaArgs a, con
     }
   for (int c = 0; c < nc; c++) {
     uint32_t sh[KD][4], sl[KD][4];
-    uint4* frag = ws.s + ((base + (size_t)c * a.H) * ws.nvt + vt) * KD * 64 + lane * 2;
+    uint4* frag = ws.s + ((base + (size_t)c * a.H) * ws.nvt + vt) * KD * 64 + lane;
 #pragma unroll
     for (int kd = 0; kd < KD; kd++) {
       split2(acc[2 * kd][0], acc[2 * kd][1], sh[kd][0], sl[kd][0]);
@@ -828,13 +880,13 @@ __global__ void __launch_bounds__(128) delta_state_kernel(const DeltaArgs a, con
       split2(acc[2 * kd + 1][2], acc[2 * kd + 1][3], sh[kd][3], sl[kd][3]);
       if (mine) {
         frag[kd * 64] = make_uint4(sh[kd][0], sh[kd][1], sh[kd][2], sh[kd][3]);
-        frag[kd * 64 + 1] = make_uint4(sl[kd][0], sl[kd][1], sl[kd][2], sl[kd][3]);
+        frag[kd * 64 + 32] = make_uint4(sl[kd][0], sl[kd][1], sl[kd][2], sl[kd][3]);
       }
     }
     cp_async_wait<ST - 2>();
     __syncthreads();                    // chunk c has landed, and everyone is done with the stage that is refilled now
     load(c + ST - 1);
-    const uint4* g = sg + (c % ST) * SN + lane * 2;
+    const uint4* g = sg + (c % ST) * SN + lane;
     const float4* f = (const float4*)(sg + (c % ST) * SN + GN) + (vt - vb0) * (DP / 8) * 32 + lane;
 #pragma unroll
     for (int j = 0; j < DP / 8; j++) {
@@ -845,7 +897,7 @@ __global__ void __launch_bounds__(128) delta_state_kernel(const DeltaArgs a, con
     for (int kd = 0; kd < KD; kd++)
 #pragma unroll
       for (int jn = 0; jn < KD; jn++) {
-        const uint4 bh = g[(kd * KD + jn) * 64], bl = g[(kd * KD + jn) * 64 + 1];
+        const uint4 bh = g[(kd * KD + jn) * 64], bl = g[(kd * KD + jn) * 64 + 32];
         mma_bf16(acc[2 * jn], sh[kd], bh.x, bh.y);
         mma_bf16(acc[2 * jn + 1], sh[kd], bh.z, bh.w);
         mma_bf16(acc[2 * jn], sh[kd], bl.x, bl.y);
@@ -898,14 +950,14 @@ __global__ void __launch_bounds__(256) delta_output_kernel(const DeltaArgs a, co
       uint4 rh[2], rl[2];
 #pragma unroll
       for (int m = 0; m < 2; m++) {
-        const uint4* p = ws.r + ((slot * KD + kd) * 4 + 2 * th + m) * 64 + lane * 2;
+        const uint4* p = ws.r + ((slot * KD + kd) * 4 + 2 * th + m) * 64 + lane;
         rh[m] = __ldg(p);
-        rl[m] = __ldg(p + 1);
+        rl[m] = __ldg(p + 32);
       }
 #pragma unroll
       for (int i = 0; i < NV; i++) {
-        const uint4* p = ws.s + ((slot * ws.nvt + min(vq + 4 * i, ws.nvt - 1)) * KD + kd) * 64 + lane * 2;
-        const uint4 xh = __ldg(p), xl = __ldg(p + 1);
+        const uint4* p = ws.s + ((slot * ws.nvt + min(vq + 4 * i, ws.nvt - 1)) * KD + kd) * 64 + lane;
+        const uint4 xh = __ldg(p), xl = __ldg(p + 32);
         const uint32_t sh[4] = {xh.x, xh.y, xh.z, xh.w}, sl[4] = {xl.x, xl.y, xl.z, xl.w};
 #pragma unroll
         for (int m = 0; m < 2; m++) {
@@ -993,10 +1045,10 @@ static int launch_delta_chunked(const DeltaArgs& a, const DeltaWs& w, int n_seqs
     configured = s1;
   }
   const int nc = (max_q + GC - 1) / GC;
-  int rc = launch_pdl(delta_prepare_kernel<DP>, dim3(nc, a.H, n_seqs), dim3(256), s1, st, a, w);
+  int rc = launch_pdl(delta_prepare_kernel<DP>, dim3(nc, a.H, n_seqs), dim3(DeltaSmem<DP>::THREADS), s1, st, a, w);
   if (rc) return rc;
   int warps = min(4, w.nvt);                 // fewer value tiles to a CTA until the SMs are covered
-  while (warps > 1 && (long)a.H * n_seqs * ((w.nvt + warps - 1) / warps) < 148) warps >>= 1;
+  while (warps > 1 && (long)a.H * n_seqs * ((w.nvt + warps / 2 - 1) / (warps / 2)) <= 148) warps >>= 1;
   rc = launch_pdl(delta_state_kernel<DP>, dim3((w.nvt + warps - 1) / warps, a.H, n_seqs), dim3(32 * warps), state_bytes(DP, warps), st, a, w);
   if (rc) return rc;
   auto out = w.nvt <= 4 ? delta_output_kernel<DP, 1> : delta_output_kernel<DP, 2>;

@@ -57,7 +57,7 @@ __device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bf
 constexpr int kConvTokens = 16;
 template <typename OT, int TAPS>
 __global__ void __launch_bounds__(256) ssd_conv_kernel(const SsdArgs a, const SsdConv<OT> o) {
-  pdl_trigger();
+  // triggers by ending: the sequential kernel behind this one wants its CTAs spread over idle SMs
   pdl_wait();
   const int seq = blockIdx.z, i0 = blockIdx.x * kConvTokens, len = a.q_len[seq];
   if (i0 >= len) return;
@@ -397,7 +397,7 @@ B200_API int b200_ssd_decode(SSD_PARAMS, void* ws, size_t ws_bytes, cudaStream_t
 
 struct SsdWs {
   SsdConv<__nv_bfloat16> c;
-  uint4* s;                     // [chunk slots][H][P tiles of 16][NP / 16][lane][2]: the state at the chunk's start (value columns as rows)
+  uint4* s;                     // [chunk slots][H][P tiles of 16][NP / 16][2][lane]: the state at the chunk's start (value columns as rows)
   int npt, kn;                  // tiles of 16 value columns / state dimensions
 };
 
@@ -436,34 +436,40 @@ __device__ __forceinline__ ChunkDecay chunk_decay(const RawDecay& raw, int lane)
 
 constexpr int kSsdStages = 3;
 
-// One CTA = 64 value columns x 64 state dimensions of one head of one sequence; a warp owns 16 value columns and half of the dimensions.  The state is kept
+// One CTA = 64 value columns x 2 DW state dimensions of one head of one sequence; a warp owns 16 value columns and half of the dimensions.  The state is kept
 // transposed (value columns as the rows of the MMA), so that its accumulators, split in two, are operands of the output product as they lie.
+template <int DW>
 __global__ void __launch_bounds__(256) ssd_state_kernel(const SsdArgs a, const SsdWs ws) {
-  constexpr int LN = 72, STAGE = 2 * GC * LN;                  // B slice | x
+  constexpr int DS = 2 * DW, LN = DS + 8, LX = 72, STAGE = GC * (LN + LX), NJ = DW / 8;      // B slice | x
   extern __shared__ __align__(16) __nv_bfloat16 sb16[];
   pdl_trigger();
   pdl_wait();
-  const int nslices = (ws.kn + 3) / 4;
-  const int ps = blockIdx.x / nslices, n0 = blockIdx.x % nslices * 64, v0 = ps * 64, h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
-  const int warp = (tid >> 5) & 3, dw = (tid >> 7) * 32, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3, g = h / (a.H / a.G);
+  const int nslices = (a.NP + DS - 1) / DS;
+  const int ps = blockIdx.x / nslices, n0 = blockIdx.x % nslices * DS, v0 = ps * 64, h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
+  const int warp = (tid >> 5) & 3, dw = (tid >> 7) * DW, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3, g = h / (a.H / a.G);
   const int len = a.q_len[seq], qs = a.q_start[seq], slot = a.slot[seq], p0 = a.ctx_len[seq] - len;
   const bool fresh = p0 == 0 || slot < 0;
   const int nc = (len + GC - 1) / GC;
   float* S = a.state + ((size_t)max(slot, 0) * a.H + h) * a.N * a.PP;
-  // this thread's 16-byte pieces of a chunk: two of B, two of x
-  const int pt0 = tid / 8, px = (tid % 8) * 8;
-  const bool blive = n0 + px < a.NP, xlive = v0 + px < a.PP;
+  // this thread's 16-byte pieces of a chunk: two of x, and as many of B as its rows are long
+  constexpr int BQ = DS / 8, BT = 256 / BQ;
+  const int pt0 = tid / 8, px = (tid % 8) * 8, bt0 = tid / BQ, bx = (tid % BQ) * 8;
+  const bool blive = n0 + bx < a.NP, xlive = v0 + px < a.PP;
   auto load = [&](int c) {
     if (c < nc) {
       __nv_bfloat16* st = sb16 + (c % kSsdStages) * STAGE;
 #pragma unroll
+      for (int m = 0; m < GC / BT; m++) {
+        const int i = c * GC + bt0 + BT * m;
+        __nv_bfloat16* db = st + (bt0 + BT * m) * LN + bx;
+        if (blive && i < len) cp_async16(s32(db), ws.c.B + ((size_t)(qs + i) * a.G + g) * a.NP + n0 + bx);
+        else *(uint4*)db = make_uint4(0u, 0u, 0u, 0u);
+      }
+#pragma unroll
       for (int m = 0; m < 2; m++) {
         const int i = c * GC + pt0 + 32 * m;
-        const size_t t = qs + i;
-        __nv_bfloat16 *db = st + (pt0 + 32 * m) * LN + px, *dx = db + GC * LN;
-        if (blive && i < len) cp_async16(s32(db), ws.c.B + (t * a.G + g) * a.NP + n0 + px);
-        else *(uint4*)db = make_uint4(0u, 0u, 0u, 0u);
-        if (xlive && i < len) cp_async16(s32(dx), ws.c.x + (t * a.H + h) * a.PP + v0 + px);
+        __nv_bfloat16* dx = st + GC * LN + (pt0 + 32 * m) * LX + px;
+        if (xlive && i < len) cp_async16(s32(dx), ws.c.x + ((size_t)(qs + i) * a.H + h) * a.PP + v0 + px);
         else *(uint4*)dx = make_uint4(0u, 0u, 0u, 0u);
       }
     }
@@ -471,9 +477,9 @@ __global__ void __launch_bounds__(256) ssd_state_kernel(const SsdArgs a, const S
   };
 #pragma unroll
   for (int c = 0; c < kSsdStages - 1; c++) load(c);
-  float acc[4][4];                      // rows v0 + 16 warp + g4 (+ 8), columns n0 + dw + 8 j + 2 t4 (+ 1)
+  float acc[NJ][4];                      // rows v0 + 16 warp + g4 (+ 8), columns n0 + dw + 8 j + 2 t4 (+ 1)
 #pragma unroll
-  for (int j = 0; j < 4; j++)
+  for (int j = 0; j < NJ; j++)
 #pragma unroll
     for (int e = 0; e < 4; e++) {
       const int v = v0 + warp * 16 + g4 + 8 * (e >> 1), d = n0 + dw + 8 * j + 2 * t4 + (e & 1);
@@ -496,7 +502,7 @@ __global__ void __launch_bounds__(256) ssd_state_kernel(const SsdArgs a, const S
     const __nv_bfloat16 *sB = sb16 + (c % kSsdStages) * STAGE, *sX = sB + GC * LN;
     if (c > 0 || !fresh) {
 #pragma unroll
-      for (int kd = 0; kd < 2; kd++) {
+      for (int kd = 0; kd < DW / 16; kd++) {
         const int kt = (n0 + dw) / 16 + kd;
         uint4 hi, lo;
         split2(acc[2 * kd][0], acc[2 * kd][1], hi.x, lo.x);
@@ -504,20 +510,20 @@ __global__ void __launch_bounds__(256) ssd_state_kernel(const SsdArgs a, const S
         split2(acc[2 * kd + 1][0], acc[2 * kd + 1][1], hi.z, lo.z);
         split2(acc[2 * kd + 1][2], acc[2 * kd + 1][3], hi.w, lo.w);
         if (pt < ws.npt && kt < ws.kn) {
-          uint4* frag = ws.s + (((chunk_slot(qs, seq, c) * a.H + h) * ws.npt + pt) * ws.kn + kt) * 64 + lane * 2;
+          uint4* frag = ws.s + (((chunk_slot(qs, seq, c) * a.H + h) * ws.npt + pt) * ws.kn + kt) * 64 + lane;
           frag[0] = hi;
-          frag[1] = lo;
+          frag[32] = lo;
         }
       }
 #pragma unroll
-      for (int j = 0; j < 4; j++)
+      for (int j = 0; j < NJ; j++)
 #pragma unroll
         for (int e = 0; e < 4; e++) acc[j][e] *= dec;
     }
 #pragma unroll
     for (int kt = 0; kt < GC / 16; kt++) {
       uint32_t xa[4], xh[4], xl[4];     // X^T: 16 value columns x 16 tokens, times the tokens' factors
-      ldsm4t(s32(sX + (kt * 16 + (lane >> 4) * 8 + (lane & 7)) * LN + warp * 16 + ((lane >> 3) & 1) * 8), xa);
+      ldsm4t(s32(sX + (kt * 16 + (lane >> 4) * 8 + (lane & 7)) * LX + warp * 16 + ((lane >> 3) & 1) * 8), xa);
       const float fa = __shfl_sync(0xffffffffu, f0, kt * 8 + t4), fb = __shfl_sync(0xffffffffu, f1, kt * 8 + t4);
       const float fc = __shfl_sync(0xffffffffu, f0, kt * 8 + 4 + t4), fd = __shfl_sync(0xffffffffu, f1, kt * 8 + 4 + t4);
 #pragma unroll
@@ -527,7 +533,7 @@ __global__ void __launch_bounds__(256) ssd_state_kernel(const SsdArgs a, const S
       }
       const int r = kt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
 #pragma unroll
-      for (int j = 0; j < 4; j += 2) {
+      for (int j = 0; j < NJ; j += 2) {
         uint32_t bb[4];
         ldsm4t(s32(sB + r * LN + dw + (j + (lane >> 4)) * 8), bb);
         mma_bf16(acc[j], xh, bb[0], bb[1]);
@@ -541,7 +547,7 @@ __global__ void __launch_bounds__(256) ssd_state_kernel(const SsdArgs a, const S
   cp_async_wait_all();
   if (slot < 0) return;
 #pragma unroll
-  for (int j = 0; j < 4; j++)
+  for (int j = 0; j < NJ; j++)
 #pragma unroll
     for (int e = 0; e < 4; e++) {
       const int v = v0 + warp * 16 + g4 + 8 * (e >> 1), d = n0 + dw + 8 * j + 2 * t4 + (e & 1);
@@ -554,8 +560,8 @@ __global__ void __launch_bounds__(256) ssd_state_kernel(const SsdArgs a, const S
       if (e < a.P && i >= 0) a.ring[((size_t)slot * a.taps + (p0 + i) % a.taps) * a.CC + h * a.P + e] = a.in[(size_t)(qs + i) * a.ld + a.x_off + h * a.P + e];
     }
   if (ps == 0 && h % (a.H / a.G) == 0)
-    for (int q = tid; q < 128 * (a.taps - 1); q += 256) {
-      const int d = n0 + q % 64, which = (q >> 6) & 1, i = len - 1 - q / 128, ch = a.H * a.P + (which * a.G + g) * a.N + d;
+    for (int q = tid; q < 2 * DS * (a.taps - 1); q += 256) {
+      const int d = n0 + q % DS, which = q / DS % 2, i = len - 1 - q / (2 * DS), ch = a.H * a.P + (which * a.G + g) * a.N + d;
       if (d < a.N && i >= 0) a.ring[((size_t)slot * a.taps + (p0 + i) % a.taps) * a.CC + ch] = a.in[(size_t)(qs + i) * a.ld + a.x_off + ch];
     }
 }
@@ -632,13 +638,17 @@ __global__ void __launch_bounds__(256, NV <= 2 ? 2 : 1) ssd_output_kernel(const 
       if (warp == 0) raw = load_decay(a, ws.c, t0, n, h + 1, lane);
     }
     cp_async_commit();
+    const float bt[2] = {s_b[m0 + g4], s_b[m0 + g4 + 8]};
+    // the decays on the hardware's exponential: these products become two bf16 numbers each.  Blocks above the diagonal stay as they are, zero.
 #pragma unroll
     for (int j = 0; j < 4; j++)
 #pragma unroll
       for (int hf = 0; hf < 2; hf++) {
+        if (n0 > m0 + 15 && k) continue;
         const int t = m0 + g4 + 8 * hf, s = n0 + 8 * j + 2 * t4;
-        const float x = s <= t ? cb[j][2 * hf] * expf(s_b[t] - s_b[s]) * s_dt[s] : 0.f;
-        const float y = s + 1 <= t ? cb[j][2 * hf + 1] * expf(s_b[t] - s_b[s + 1]) * s_dt[s + 1] : 0.f;
+        const float2 bs = *(const float2*)(s_b + s), ds = *(const float2*)(s_dt + s);
+        const float x = s <= t ? cb[j][2 * hf] * __expf(bt[hf] - bs.x) * ds.x : 0.f;
+        const float y = s + 1 <= t ? cb[j][2 * hf + 1] * __expf(bt[hf] - bs.y) * ds.y : 0.f;
         uint32_t hi, lo;
         split2(x, y, hi, lo);
         *(uint32_t*)(sAh + t * LA + s) = hi;
@@ -650,7 +660,7 @@ __global__ void __launch_bounds__(256, NV <= 2 ? 2 : 1) ssd_output_kernel(const 
 #pragma unroll
       for (int j = 0; j < 4; j++) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
     if (with_state) {
-      const uint4* frag = ws.s + (chunk_slot(qs, seq, c) * a.H + h) * ws.npt * ws.kn * 64 + lane * 2;
+      const uint4* frag = ws.s + (chunk_slot(qs, seq, c) * a.H + h) * ws.npt * ws.kn * 64 + lane;
 #pragma unroll 4
       for (int kd = 0; kd < ws.kn; kd++) {
         uint32_t cc[2][4];
@@ -659,7 +669,7 @@ __global__ void __launch_bounds__(256, NV <= 2 ? 2 : 1) ssd_output_kernel(const 
 #pragma unroll
         for (int i = 0; i < NV; i++) {
           const uint4* p = frag + ((size_t)min(vq + 4 * i, ws.npt - 1) * ws.kn + kd) * 64;
-          const uint4 xh = __ldg(p), xl = __ldg(p + 1);
+          const uint4 xh = __ldg(p), xl = __ldg(p + 32);
           const uint32_t sh[4] = {xh.x, xh.y, xh.z, xh.w}, sl[4] = {xl.x, xl.y, xl.z, xl.w};
 #pragma unroll
           for (int m = 0; m < 2; m++) {
@@ -778,14 +788,11 @@ B200_API int b200_ssd_prefill(SSD_PARAMS, int T, int max_q, int exact, void* ws,
   w.kn = a.NP / 16;
   rc = launch_ssd_conv(a, w.c, n_seqs, max_q, st);
   if (rc) return rc;
-  constexpr int s2 = kSsdStages * 2 * GC * 72 * 2;
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(ssd_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, s2);
-    if (e != cudaSuccess) return (int)e;
-    configured = true;
-  }
-  rc = launch_pdl(ssd_state_kernel, dim3((w.npt + 3) / 4 * ((w.kn + 3) / 4), H, n_seqs), dim3(256), (size_t)s2, st, a, w);
+  const int slices = a.NP <= 64 ? 1 : (a.NP + 127) / 128, s2 = kSsdStages * GC * ((a.NP <= 64 ? 64 : 128) + 8 + 72) * 2;
+  auto walk = a.NP <= 64 ? ssd_state_kernel<32> : ssd_state_kernel<64>;
+  cudaError_t e = cudaFuncSetAttribute(walk, cudaFuncAttributeMaxDynamicSharedMemorySize, s2);
+  if (e != cudaSuccess) return (int)e;
+  rc = launch_pdl(walk, dim3((w.npt + 3) / 4 * slices, H, n_seqs), dim3(256), (size_t)s2, st, a, w);
   if (rc) return rc;
   if (w.npt <= 4) return launch_ssd_output<1>(a, w, n_seqs, max_q, st);
   if (w.npt <= 8) return launch_ssd_output<2>(a, w, n_seqs, max_q, st);
