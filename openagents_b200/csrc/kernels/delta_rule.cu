@@ -37,75 +37,90 @@ constexpr int kDeltaDim = 256;        // most key channels of a head
 constexpr int kDeltaRank = 1024;      // most ranks of the decay's projection
 constexpr float kUnitEps = 1e-6f;
 
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float sigmoid_f(float x) { return __fdividef(1.f, 1.f + expf(-x)); }
 // The same on the hardware's exponential and reciprocal (some 1e-7 relative), for operands that are rounded to two bf16 numbers.
 __device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 
 // ------------------------------------------------------------------ token by token
 
 // Decoding, and the prompts of the 32-bit mode.  One cluster per head and share of the sequences, whose CTAs share the value columns.  A CTA walks the tokens
-// of its sequences one by one; while it works on one, the projections of the next, and with a new sequence its state, are on their way into the other half of
-// a double buffer.  The state is updated in shared memory.  With n = 1 / (sum k^2 + 1e-6), R = k^T S and p = (r w)^T S, from one pass over the old state,
+// of its sequences one by one.  While the state meets one token, what the next one does to it (decays, rates) is computed from its projections, and the
+// projections of the one after, and with a new sequence its state, are on their way.  The state is updated in shared memory.  With n = 1 / (sum k^2 + 1e-6), R = k^T S and p = (r w)^T S, from one pass over the old state,
 //   o = p - n (r . a k) R + (r . k) v        S' = diag(w) S - a k (n R) + k v^T
 // so a token needs three sums over the channels and one reduction over the state's rows.
 __device__ __forceinline__ void cp_async4(void* dst, const float* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(s32(dst)), "l"(src) : "memory");
 }
 struct DeltaLayout {                       // floats of shared memory
-  int state, row, ch, kr, x, z, read, red, total;      // offsets; state and row: of the first of two buffers
+  int state, row, ch, kr, x, z, read, red, total;      // offsets; of the first buffer (two of state, ch and kr, three of row)
   int state_n, row_n;                      // sizes of one buffer
 };
-static DeltaLayout delta_layout(int dim, int W, int rank8) {
+static DeltaLayout delta_layout(int dim, int W, int rank8, int threads) {
   DeltaLayout l;
-  const int groups = 256 / (W / 4);
+  const int groups = threads / (W / 4);
   auto up4 = [](int n) { return (n + 3) & ~3; };
   l.state_n = dim * W;
   l.row_n = up4(3 * dim) + 2 * W + rank8;  // r k a | v g | x
   l.state = 0;
   l.row = 2 * l.state_n;
-  l.ch = l.row + 2 * l.row_n;
-  l.kr = l.ch + 4 * dim;
-  l.x = l.kr + up4(2 * dim);
+  l.ch = l.row + 3 * l.row_n;
+  l.kr = l.ch + 8 * dim;
+  l.x = l.kr + up4(4 * dim);
   l.z = l.x + rank8;
   l.read = l.z + up4(dim);
   l.red = l.read + W;
   l.total = l.red + groups * 2 * W;
   return l;
 }
-constexpr int kRowPieces = 3;              // elements of a projection row that a thread fetches without working out their places again
+constexpr int kRowPieces = 4;              // elements of a projection row that a thread fetches without working out their places again
 
 // DIM, NV: channels and float4 columns of a CTA's share of a head, where they are known (0: not).
-template <int DIM, int NV>
-__global__ void __launch_bounds__(256, 4) delta_recurrent_kernel(const DeltaArgs a, int n_seqs, const DeltaLayout l) {
+// The fewer threads share a token, the less each spends on anything but the state.
+template <int DIM, int NV, int NT>
+__global__ void __launch_bounds__(NT, NT == 128 ? 3 : 2) delta_recurrent_kernel(const DeltaArgs a, int n_seqs, const DeltaLayout l) {
   extern __shared__ __align__(16) float sm[];
   cg::cluster_group cluster = cg::this_cluster();
   const int CL = cluster.num_blocks(), part = cluster.block_rank(), dim = DIM ? DIM : a.dim;
   const int nv_all = a.VP >> 2, nv = NV ? NV : nv_all / CL, W = nv * 4, e0 = part * W;     // this CTA's columns [e0, e0 + W)
-  const int groups = 256 / nv;
-  float4* s_ch = (float4*)(sm + l.ch);     // [dim] (w, a k, k, -)
-  float2* s_kr = (float2*)(sm + l.kr);     // [dim] (k, r w)
+  const int groups = NT / nv;
+  float4* s_ch = (float4*)(sm + l.ch);     // [2][dim] (w, a k, k, -)
+  float2* s_kr = (float2*)(sm + l.kr);     // [2][dim] (k, r w)
   float *s_x = sm + l.x, *s_z = sm + l.z, *s_read = sm + l.read, *s_red = sm + l.red;
-  __shared__ float red[3][8], red1[8];
+  __shared__ float red[2][3][8], red1[8];
   __shared__ float s_part[2];              // this CTA's sum of squares, by token parity
   pdl_trigger();
   const int h = blockIdx.x / CL, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   // TPC threads share a channel's low-rank product; its weights are read while the projection still runs
   int TPC = 1;
-  while (TPC < 8 && dim * TPC * 2 <= 256) TPC *= 2;
+  while (TPC < 8 && dim * TPC * 2 <= NT) TPC *= 2;
   const int ch = tid / TPC, sub = tid % TPC;
   const __nv_bfloat16* wrow = a.w2 + (size_t)(h * dim + (ch < dim ? ch : 0)) * a.rank8;
-  uint4 held[4];
+  constexpr int HELD = 1024 / NT;
+  uint4 held[HELD];
 #pragma unroll
-  for (int i = 0; i < 4; i++) held[i] = ch < dim && (sub + i * TPC) * 8 < a.rank8 ? ((const uint4*)wrow)[sub + i * TPC] : make_uint4(0u, 0u, 0u, 0u);
-  const float w0 = tid < dim ? a.w0[h * dim + tid] : 0.f, ab = tid < dim ? a.ab[h * dim + tid] : 0.f;
+  for (int i = 0; i < HELD; i++) held[i] = ch < dim && (sub + i * TPC) * 8 < a.rank8 ? ((const uint4*)wrow)[sub + i * TPC] : make_uint4(0u, 0u, 0u, 0u);
+  const int cc = NT - 1 - tid;                // the last warps take a channel each, the first ones an output column
+  const float w0 = cc < dim ? a.w0[h * dim + cc] : 0.f, ab = cc < dim ? a.ab[h * dim + cc] : 0.f;
   const float wo = (tid < W && e0 + tid < a.vdim) ? a.norm[h * a.vdim + e0 + tid] : 0.f;
   const int grp = tid / nv, col = tid % nv, rka = (3 * dim + 3) & ~3;
-  const bool active = grp < groups;
+  constexpr int ROWS = DIM ? DIM * NV / NT : 0;                // a thread's state rows, where they are known and all threads have as many
+  static_assert(DIM == 0 || (NT % NV == 0 && DIM % (NT / NV) == 0), "whole rows for every thread");
+  const bool active = DIM || grp < groups;
+  auto rows = [&](auto body) {
+    if constexpr (ROWS > 0) {
+#pragma unroll
+      for (int k = 0; k < ROWS; k++) body(grp + k * groups, k);
+    } else {
+      int k = 0;
+#pragma unroll 4
+      for (int d = grp; d < dim; d += groups) body(d, k++);
+    }
+  };
   // element i of a row as kept in shared memory: its column in the projections (< 0: zero)
   const int row_n = rka + 2 * W + a.rank8;
   auto column = [&](int i) {
     if (i < 3 * dim) {
-      const int which = i / dim;
+      const int which = (i >= dim) + (i >= 2 * dim);
       return (which == 0 ? a.r_off : which == 1 ? a.k_off : a.a_off) + h * dim + i - which * dim;
     }
     i -= rka;
@@ -119,13 +134,14 @@ __global__ void __launch_bounds__(256, 4) delta_recurrent_kernel(const DeltaArgs
   const uint32_t with = __ballot_sync(0xffffffffu, ch < dim);      // whole groups of TPC threads
   int piece[kRowPieces];
 #pragma unroll
-  for (int k = 0; k < kRowPieces; k++) piece[k] = tid + 256 * k < row_n ? column(tid + 256 * k) : -1;
-  for (int i = tid; i < 2 * row_n; i += 256)
-    if (column(i % row_n) < 0) sm[l.row + i / row_n * l.row_n + i % row_n] = 0.f;       // stays zero
+  for (int k = 0; k < kRowPieces; k++) piece[k] = tid + NT * k < row_n ? column(tid + NT * k) : -1;
+  for (int i = tid; i < 3 * l.row_n / 4; i += NT) ((float4*)(sm + l.row))[i] = make_float4(0.f, 0.f, 0.f, 0.f);      // what no copy writes stays zero
+  __syncthreads();
   pdl_wait();
-  struct Seq { int n, t0, slot; bool fresh; };
-  auto meta = [&](int b) {
-    Seq q = {0, 0, -1, true};
+  // a token: row t0 + i of entry b, whose n tokens start at row t0 (n = 0: nothing to do)
+  struct Item { int b, i, n, t0, slot; bool fresh; };
+  auto first = [&](int b) {
+    Item q = {b, 0, 0, 0, -1, true};
     if (b < n_seqs) {
       q.n = a.q_len[b];
       q.t0 = a.q_start[b];
@@ -134,111 +150,122 @@ __global__ void __launch_bounds__(256, 4) delta_recurrent_kernel(const DeltaArgs
     }
     return q;
   };
+  auto next = [&](const Item& q) {
+    if (q.i + 1 >= q.n) return first(q.b + gridDim.y);
+    Item r = q;
+    r.i++;
+    return r;
+  };
   auto state_of = [&](int slot) { return (float4*)(a.state + ((size_t)max(slot, 0) * a.H + h) * dim * a.VP) + part * nv + (size_t)grp * nv_all + col; };
   const int ds = groups * nv;              // from one of a thread's state rows to the next, in shared memory
   const size_t dg = (size_t)groups * nv_all;
-  auto fetch_row = [&](int t, int buf) {
-    const float* src = a.in + (size_t)t * a.ld;
+  auto fetch_row = [&](const Item& q, int buf) {
+    if (q.n < 1) return;
+    const float* src = a.in + (size_t)(q.t0 + q.i) * a.ld;
     float* dst = sm + l.row + buf * l.row_n;
 #pragma unroll
     for (int k = 0; k < kRowPieces; k++)
-      if (piece[k] >= 0) cp_async4(dst + tid + 256 * k, src + piece[k]);
-    for (int i = tid + 256 * kRowPieces; i < row_n; i += 256) {
+      if (piece[k] >= 0) cp_async4(dst + tid + NT * k, src + piece[k]);
+    for (int i = tid + NT * kRowPieces; i < row_n; i += NT) {
       const int c = column(i);
       if (c >= 0) cp_async4(dst + i, src + c);
     }
   };
-  auto fetch_state = [&](const Seq& q, int buf) {
-    if (!active) return;
+  auto fetch_state = [&](const Item& q, int buf) {
+    if (!active || q.n < 1) return;
     float4* dst = (float4*)(sm + l.state + buf * l.state_n) + grp * nv + col;
     const float4* src = state_of(q.slot);
-#pragma unroll 4
-    for (int d = grp; d < dim; d += groups, dst += ds, src += dg) {
-      if (!q.fresh) cp_async16(s32(dst), src);
-      else *dst = make_float4(0.f, 0.f, 0.f, 0.f);
+    const uint32_t to = s32(dst);
+    if (!q.fresh) rows([&](int, int k) { cp_async16(to + k * ds * 16, src + k * dg); });
+    else rows([&](int, int k) { dst[k * ds] = make_float4(0.f, 0.f, 0.f, 0.f); });
+  };
+  // what a token does to the state, in three steps with a barrier between them
+  auto low_rank = [&](const float* row) {
+    for (int r = tid; r < a.rank8; r += NT) {
+      const float x = row[rka + 2 * W + r], e = expf(-2.f * fabsf(x));
+      s_x[r] = copysignf(__fdividef(1.f - e, 1.f + e), x);      // tanh
     }
   };
-  int b = blockIdx.y, i = 0, sbuf = 0, rbuf = 0, step = 0;
-  Seq cur = meta(b), nxt = meta(b + gridDim.y);
-  while (b < n_seqs && cur.n < 1) {         // an entry without tokens
-    b += gridDim.y;
-    cur = nxt;
-    nxt = meta(b + gridDim.y);
-  }
-  if (b < n_seqs) {
-    fetch_state(cur, 0);
-    fetch_row(cur.t0, 0);
-    cp_async_commit();
-  }
-  while (b < n_seqs) {
-    cp_async_wait_all();
-    __syncthreads();                       // this token's data has landed, and everyone is done with the other buffers
-    const bool last = i + 1 == cur.n;
-    if (!last) {
-      fetch_row(cur.t0 + i + 1, rbuf ^ 1);
-    } else if (b + gridDim.y < n_seqs && nxt.n > 0) {
-      fetch_state(nxt, sbuf ^ 1);
-      fetch_row(nxt.t0, rbuf ^ 1);
+  auto decay_logits = [&]() {
+    if (ch >= dim) return;
+    float z = 0.f;
+    auto dot = [&](uint4 q, int at) {
+      const __nv_bfloat162* p = (const __nv_bfloat162*)&q;
+      const float4 x0 = *(const float4*)(s_x + at), x1 = *(const float4*)(s_x + at + 4);
+      float2 f;
+      f = __bfloat1622float2(p[0]); z = fmaf(f.x, x0.x, z); z = fmaf(f.y, x0.y, z);
+      f = __bfloat1622float2(p[1]); z = fmaf(f.x, x0.z, z); z = fmaf(f.y, x0.w, z);
+      f = __bfloat1622float2(p[2]); z = fmaf(f.x, x1.x, z); z = fmaf(f.y, x1.y, z);
+      f = __bfloat1622float2(p[3]); z = fmaf(f.x, x1.z, z); z = fmaf(f.y, x1.w, z);
+    };
+#pragma unroll
+    for (int j = 0; j < HELD; j++)
+      if ((sub + j * TPC) * 8 < a.rank8) dot(held[j], (sub + j * TPC) * 8);
+    for (int j = sub + HELD * TPC; j * 8 < a.rank8; j += TPC) dot(((const uint4*)wrow)[j], j * 8);
+    for (int o = 1; o < TPC; o <<= 1) z += __shfl_xor_sync(with, z, o);
+    if (sub == 0) s_z[ch] = z;
+  };
+  auto channels = [&](const float* row, int buf) {
+    if (NT - 1 - (warp * 32 + 31) >= dim) return;                  // no channel in this warp
+    float q0 = 0.f, q1 = 0.f, q2 = 0.f;
+    if (cc < dim) {
+      const float rr = row[cc], kk = row[dim + cc], rate = sigmoid_f(row[2 * dim + cc] + ab), w = expf(-a.decay * sigmoid_f(s_z[cc] + w0));
+      s_ch[buf * dim + cc] = make_float4(w, rate * kk, kk, 0.f);
+      s_kr[buf * dim + cc] = make_float2(kk, rr * w);
+      q0 = kk * kk;
+      q1 = rr * rate * kk;
+      q2 = rr * kk;
     }
+    q0 = warp_sum(q0);
+    q1 = warp_sum(q1);
+    q2 = warp_sum(q2);
+    if (lane == 0) { red[buf][0][NT / 32 - 1 - warp] = q0; red[buf][1][NT / 32 - 1 - warp] = q1; red[buf][2][NT / 32 - 1 - warp] = q2; }
+  };
+  Item cur = first(blockIdx.y), nxt = next(cur), aft = next(nxt);
+  fetch_state(cur, 0);
+  fetch_row(cur, 0);
+  fetch_row(nxt, 1);
+  cp_async_commit();
+  cp_async_wait_all();
+  __syncthreads();
+  low_rank(sm + l.row);
+  __syncthreads();
+  decay_logits();
+  __syncthreads();
+  channels(sm + l.row, 0);
+  int sbuf = 0, rbuf = 0, step = 0;
+  while (cur.b < n_seqs) {
+    cp_async_wait_all();
+    __syncthreads();                       // the state and the next token's projections have landed; this token's channels are ready
+    const int r1 = rbuf == 2 ? 0 : rbuf + 1, r2 = r1 == 2 ? 0 : r1 + 1, kb = step & 1;
+    if (nxt.i == 0) fetch_state(nxt, sbuf ^ 1);
+    fetch_row(aft, r2);
     cp_async_commit();
+    const Item later = next(aft);          // looked up ahead of its use
     const float* row = sm + l.row + rbuf * l.row_n;
+    const float* row1 = sm + l.row + r1 * l.row_n;
     const float *s_v = row + rka, *s_g = s_v + W;
     float4* S = (float4*)(sm + l.state + sbuf * l.state_n) + grp * nv + col;
-    for (int r = tid; r < a.rank8; r += 256) s_x[r] = tanhf(row[rka + 2 * W + r]);
-    __syncthreads();
-    if (ch < dim) {
-      float z = 0.f;
-      auto dot = [&](uint4 q, int at) {
-        const __nv_bfloat162* p = (const __nv_bfloat162*)&q;
-        const float4 x0 = *(const float4*)(s_x + at), x1 = *(const float4*)(s_x + at + 4);
-        float2 f;
-        f = __bfloat1622float2(p[0]); z = fmaf(f.x, x0.x, z); z = fmaf(f.y, x0.y, z);
-        f = __bfloat1622float2(p[1]); z = fmaf(f.x, x0.z, z); z = fmaf(f.y, x0.w, z);
-        f = __bfloat1622float2(p[2]); z = fmaf(f.x, x1.x, z); z = fmaf(f.y, x1.y, z);
-        f = __bfloat1622float2(p[3]); z = fmaf(f.x, x1.z, z); z = fmaf(f.y, x1.w, z);
-      };
-#pragma unroll
-      for (int j = 0; j < 4; j++)
-        if ((sub + j * TPC) * 8 < a.rank8) dot(held[j], (sub + j * TPC) * 8);
-      for (int j = sub + 4 * TPC; j * 8 < a.rank8; j += TPC) dot(((const uint4*)wrow)[j], j * 8);
-      for (int o = 1; o < TPC; o <<= 1) z += __shfl_xor_sync(with, z, o);
-      if (sub == 0) s_z[ch] = z;
-    }
-    __syncthreads();
-    if (warp * 32 < dim) {                 // one channel per lane
-      float q0 = 0.f, q1 = 0.f, q2 = 0.f;
-      if (tid < dim) {
-        const float rr = row[tid], kk = row[dim + tid], rate = sigmoid_f(row[2 * dim + tid] + ab), w = expf(-a.decay * sigmoid_f(s_z[tid] + w0));
-        s_ch[tid] = make_float4(w, rate * kk, kk, 0.f);
-        s_kr[tid] = make_float2(kk, rr * w);
-        q0 = kk * kk;
-        q1 = rr * rate * kk;
-        q2 = rr * kk;
-      }
-      q0 = warp_sum(q0);
-      q1 = warp_sum(q1);
-      q2 = warp_sum(q2);
-      if (lane == 0) { red[0][warp] = q0; red[1][warp] = q1; red[2][warp] = q2; }
-    }
-    __syncthreads();
+    const bool live = cur.n > 0, last = cur.i + 1 >= cur.n;
+    low_rank(row1);
     if (active) {
       float4 rd = make_float4(0.f, 0.f, 0.f, 0.f), p = rd;
-      const float4* x4 = S;
-#pragma unroll 4
-      for (int d = grp; d < dim; d += groups, x4 += ds) {
-        const float2 kr = s_kr[d];
-        const float4 x = *x4;
+      const float2* kr_at = s_kr + kb * dim;
+      rows([&](int d, int k) {
+        const float2 kr = kr_at[d];
+        const float4 x = S[k * ds];
         rd.x = fmaf(kr.x, x.x, rd.x); rd.y = fmaf(kr.x, x.y, rd.y); rd.z = fmaf(kr.x, x.z, rd.z); rd.w = fmaf(kr.x, x.w, rd.w);
         p.x = fmaf(kr.y, x.x, p.x); p.y = fmaf(kr.y, x.y, p.y); p.z = fmaf(kr.y, x.z, p.z); p.w = fmaf(kr.y, x.w, p.w);
-      }
+      });
       *(float4*)(s_red + (size_t)(grp * 2) * W + 4 * col) = rd;
       *(float4*)(s_red + (size_t)(grp * 2 + 1) * W + 4 * col) = p;
     }
     __syncthreads();
+    decay_logits();
     float o = 0.f;
     if (warp * 32 < W) {                   // one column per lane; W <= 256
       float q0 = 0.f, q1 = 0.f, q2 = 0.f;
-      for (int j = 0; j * 32 < dim; j++) { q0 += red[0][j]; q1 += red[1][j]; q2 += red[2][j]; }
+      for (int j = 0; j * 32 < dim; j++) { q0 += red[kb][0][j]; q1 += red[kb][1][j]; q2 += red[kb][2][j]; }
       const float inv = 1.f / (q0 + kUnitEps);
       if (tid < W) {
         float rd = 0.f, p = 0.f;
@@ -255,22 +282,18 @@ __global__ void __launch_bounds__(256, 4) delta_recurrent_kernel(const DeltaArgs
       if (lane == 0) red1[warp] = ss;
     }
     __syncthreads();
+    channels(row1, kb ^ 1);
     if (active) {
       const float4 v = *(const float4*)(s_v + 4 * col), rd = *(const float4*)(s_read + 4 * col);
+      const float4* c_at = s_ch + kb * dim;
+      auto updated = [&](int d, int k) {
+        const float4 c = c_at[d], x = S[k * ds];
+        return make_float4(fmaf(c.x, x.x, fmaf(c.z, v.x, -c.y * rd.x)), fmaf(c.x, x.y, fmaf(c.z, v.y, -c.y * rd.y)), fmaf(c.x, x.z, fmaf(c.z, v.z, -c.y * rd.z)),
+                           fmaf(c.x, x.w, fmaf(c.z, v.w, -c.y * rd.w)));
+      };
       float4* dst = state_of(cur.slot);
-      const bool keep = last && cur.slot >= 0;
-      float4* x4 = S;
-#pragma unroll 4
-      for (int d = grp; d < dim; d += groups, x4 += ds, dst += dg) {
-        const float4 c = s_ch[d];
-        float4 x = *x4;
-        x.x = fmaf(c.x, x.x, fmaf(c.z, v.x, -c.y * rd.x));
-        x.y = fmaf(c.x, x.y, fmaf(c.z, v.y, -c.y * rd.y));
-        x.z = fmaf(c.x, x.z, fmaf(c.z, v.z, -c.y * rd.z));
-        x.w = fmaf(c.x, x.w, fmaf(c.z, v.w, -c.y * rd.w));
-        if (!last) *x4 = x;
-        else if (keep) *dst = x;
-      }
+      if (!last) rows([&](int d, int k) { S[k * ds] = updated(d, k); });
+      else if (live && cur.slot >= 0) rows([&](int d, int k) { dst[k * dg] = updated(d, k); });
     }
     float ss = 0.f;
     if (CL > 1 || warp * 32 < W)
@@ -281,33 +304,19 @@ __global__ void __launch_bounds__(256, 4) delta_recurrent_kernel(const DeltaArgs
       ss = 0.f;
       for (int p = 0; p < CL; p++) ss += *cluster.map_shared_rank(&s_part[step & 1], p);
     }
-    if (tid < W) {
+    if (tid < W && live) {
       if (e0 + tid < a.vdim) o *= wo * sigmoid_f(s_g[tid]) / sqrtf(ss / (float)a.vdim + a.eps);
       else o = 0.f;
-      const size_t at = (size_t)(cur.t0 + i) * a.ldo + (size_t)h * a.VP + e0 + tid;
+      const size_t at = (size_t)(cur.t0 + cur.i) * a.ldo + (size_t)h * a.VP + e0 + tid;
       if (a.out_f32) a.out_f32[at] = o;
       if (a.out_bf16) a.out_bf16[at] = __float2bfloat16(o);
     }
     step++;
-    rbuf ^= 1;
-    i++;
-    if (last) {
-      i = 0;
-      sbuf ^= 1;
-      bool skipped = false;
-      do {                                 // past entries without tokens, whose successors were not fetched ahead
-        b += gridDim.y;
-        cur = nxt;
-        nxt = meta(b + gridDim.y);
-        if (b < n_seqs && cur.n < 1) skipped = true;
-      } while (b < n_seqs && cur.n < 1);
-      if (skipped && b < n_seqs) {
-        __syncthreads();
-        fetch_state(cur, sbuf);
-        fetch_row(cur.t0, rbuf);
-        cp_async_commit();
-      }
-    }
+    rbuf = r1;
+    if (nxt.i == 0) sbuf ^= 1;
+    cur = nxt;
+    nxt = aft;
+    aft = later;
   }
   if (CL > 1) cluster.sync();              // peers may still be reading this CTA's sum
 }
@@ -333,22 +342,23 @@ B200_API int b200_delta_recurrent(const float* in, int ld, const int* offs, int 
   int rc = delta_fill(a, in, ld, offs, rank, w2, rank8, w0, ab, norm, state, q_start, q_len, ctx_len, slot, n_seqs, H, dim, vdim, VP, decay, eps, out_f32,
                       out_bf16, ldo);
   if (rc) return rc;
-  // CTAs per head: until a state share is 32 KB at most and the SMs are covered, eight float4 columns each at least
+  // CTAs per head: until a state share is 32 KB at most and the SMs are covered, eight (for the SMs' sake: sixteen) float4 columns each at least
   int CL = 1;
-  while (CL < 8 && (VP / 4) % (2 * CL) == 0 && VP / 4 / (2 * CL) >= 8 && (dim * VP / CL > 8192 || (long)H * n_seqs * CL < 148)) CL *= 2;
-  const DeltaLayout l = delta_layout(dim, VP / CL, rank8);
+  while (CL < 8 && (VP / 4) % (2 * CL) == 0 && VP / 4 / (2 * CL) >= 8 && (dim * VP / CL > 8192 || (VP / CL > 64 && (long)H * n_seqs * CL < 148))) CL *= 2;
+  const bool w64 = VP / CL == 64 && (dim == 64 || dim == 128);
+  const int threads = w64 ? 128 : 256;
+  const DeltaLayout l = delta_layout(dim, VP / CL, rank8, threads);
   const size_t smem = 4 * (size_t)l.total;
   if (smem > 200 * 1024) return B200_ERR_BAD_ARG;
-  const bool w64 = VP / CL == 64;
-  auto kern = w64 && dim == 64 ? delta_recurrent_kernel<64, 16> : w64 && dim == 128 ? delta_recurrent_kernel<128, 16> : delta_recurrent_kernel<0, 0>;
+  auto kern = !w64 ? delta_recurrent_kernel<0, 0, 256> : dim == 64 ? delta_recurrent_kernel<64, 16, 128> : delta_recurrent_kernel<128, 16, 128>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
   if (e != cudaSuccess) return (int)e;
   // shares of the sequences: no more CTAs than run at a time, all with about the same number of sequences
-  const int fit = (int)(227 * 1024 / (smem + 1024)), resident = 148 * (fit < 1 ? 1 : fit > 4 ? 4 : fit);
+  const int fit = (int)(227 * 1024 / (smem + 1024)), most_fit = threads == 128 ? 3 : 2, resident = 148 * (fit < 1 ? 1 : fit > most_fit ? most_fit : fit);
   const int most = resident / (H * CL) > 1 ? resident / (H * CL) : 1, rounds = (n_seqs + most - 1) / most, shares = (n_seqs + rounds - 1) / rounds;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(H * CL, shares);
-  cfg.blockDim = dim3(256);
+  cfg.blockDim = dim3(threads);
   cfg.dynamicSmemBytes = smem;
   cfg.stream = st;
   cudaLaunchAttribute attr[2];
