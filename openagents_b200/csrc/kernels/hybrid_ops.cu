@@ -783,12 +783,12 @@ struct RowQkvArgs {
   __half* q16;             // [T][H][DK] or null
 };
 template <typename CT, bool VEC>
-__global__ void __launch_bounds__(256) row_qkv_finish_kernel(const RowQkvArgs a, CT* __restrict__ kc, CT* __restrict__ vc) {
+__global__ void __launch_bounds__(512) row_qkv_finish_kernel(const RowQkvArgs a, CT* __restrict__ kc, CT* __restrict__ vc) {
   extern __shared__ __align__(16) float row_s[];           // q row | k row
-  __shared__ float red[2][8];
+  __shared__ float red[2][16];
   pdl_trigger();
   pdl_wait();
-  const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nt = blockDim.x, nw = nt >> 5;
   const float* row = a.in + (size_t)t * a.ld;
   const int nq = a.H * a.dim, nk = a.G * a.dim, s = a.slot[t], p = a.pos[t];
   const int page = s >= 0 ? s / a.page_size : 0, off = s >= 0 ? s % a.page_size : 0;
@@ -796,23 +796,23 @@ __global__ void __launch_bounds__(256) row_qkv_finish_kernel(const RowQkvArgs a,
   if constexpr (VEC) {
     auto sum = [](float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; };
 #pragma unroll 4
-    for (int i = tid; i < nq / 4; i += 256) {
+    for (int i = tid; i < nq / 4; i += nt) {
       const float4 v = *(const float4*)(row + a.q_off + 4 * i);
       *(float4*)(row_s + 4 * i) = v;
       sq += sum(v);
     }
-    for (int i = tid; i < nk / 4; i += 256) {
+    for (int i = tid; i < nk / 4; i += nt) {
       const float4 v = *(const float4*)(row + a.k_off + 4 * i);
       *(float4*)(row_s + nq + 4 * i) = v;
       sk += sum(v);
     }
   } else {
-    for (int i = tid; i < nq; i += 256) {
+    for (int i = tid; i < nq; i += nt) {
       const float v = row[a.q_off + i];
       row_s[i] = v;
       sq += v * v;
     }
-    for (int i = tid; i < nk; i += 256) {
+    for (int i = tid; i < nk; i += nt) {
       const float v = row[a.k_off + i];
       row_s[nq + i] = v;
       sk += v * v;
@@ -821,16 +821,34 @@ __global__ void __launch_bounds__(256) row_qkv_finish_kernel(const RowQkvArgs a,
   sq = warp_sum(sq);
   sk = warp_sum(sk);
   if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+  const float lam = a.lam ? *a.lam : 0.f;
+  for (int g = warp; g < a.G; g += nw) {                    // a warp per value head
+    const float* v = row + a.v_off + g * a.vdim;
+    float ss = 0.f;
+    if (a.v_norm)
+      for (int e = lane; e < a.vdim; e += 32) ss += v[e] * v[e];
+    const float r = a.v_norm ? 1.f / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps) : 1.f;
+    float* first = a.v_first ? a.v_first + ((size_t)t * a.G + g) * a.vdim : nullptr;
+    CT* dst = vc + (((size_t)page * a.G + g) * a.page_size + off) * a.DV;
+    for (int e = lane; e < a.DV; e += 32) {
+      float x = 0.f;
+      if (e < a.vdim) {
+        x = v[e] * r;
+        if (a.lam) x = (1.f - lam) * x + lam * first[e];
+        else if (first) first[e] = x;
+      }
+      if (s >= 0) put(dst + e, x);
+    }
+  }
   __syncthreads();
   sq = sk = 0.f;
-#pragma unroll
-  for (int i = 0; i < 8; i++) { sq += red[0][i]; sk += red[1][i]; }
+  for (int i = 0; i < nw; i++) { sq += red[0][i]; sk += red[1][i]; }
   const float rq = a.q_w ? 1.f / sqrtf(sq / (float)nq + a.eps) : 1.f, rk = a.k_w ? 1.f / sqrtf(sk / (float)nk + a.eps) : 1.f;
   const int half = a.rot >> 1;
   const float2* cs = a.tab + (size_t)min(max(p, 0), a.tab_len - 1) * half;
   if constexpr (VEC) {                                     // four columns of a head, and the four they turn with
     const int skip = a.style == 1 ? half : 0, units = (a.DK - skip) >> 2;
-    for (int i = tid; i < (a.H + a.G) * units; i += 256) {
+    for (int i = tid; i < (a.H + a.G) * units; i += nt) {
       const int hh = i / units, u = i - hh * units;
       const bool is_q = hh < a.H;
       if (!is_q && s < 0) continue;
@@ -877,7 +895,7 @@ __global__ void __launch_bounds__(256) row_qkv_finish_kernel(const RowQkvArgs a,
     }
   } else {
     const int pairs = (a.DK + 1) >> 1;
-    for (int i = tid; i < (a.H + a.G) * pairs; i += 256) {
+    for (int i = tid; i < (a.H + a.G) * pairs; i += nt) {
       const int hh = i / pairs, j = i - hh * pairs;
       const bool is_q = hh < a.H;
       if (!is_q && s < 0) continue;
@@ -903,25 +921,6 @@ __global__ void __launch_bounds__(256) row_qkv_finish_kernel(const RowQkvArgs a,
       }
     }
   }
-  const float lam = a.lam ? *a.lam : 0.f;
-  for (int g = warp; g < a.G; g += 8) {                    // a warp per value head
-    const float* v = row + a.v_off + g * a.vdim;
-    float ss = 0.f;
-    if (a.v_norm)
-      for (int e = lane; e < a.vdim; e += 32) ss += v[e] * v[e];
-    const float r = a.v_norm ? 1.f / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps) : 1.f;
-    float* first = a.v_first ? a.v_first + ((size_t)t * a.G + g) * a.vdim : nullptr;
-    CT* dst = vc + (((size_t)page * a.G + g) * a.page_size + off) * a.DV;
-    for (int e = lane; e < a.DV; e += 32) {
-      float x = 0.f;
-      if (e < a.vdim) {
-        x = v[e] * r;
-        if (a.lam) x = (1.f - lam) * x + lam * first[e];
-        else if (first) first[e] = x;
-      }
-      if (s >= 0) put(dst + e, x);
-    }
-  }
 }
 // cache_f32: kc / vc hold fp32 instead of fp16; layout [page][G][page_size][DK or DV].
 B200_API int b200_row_qkv_finish(const float* in, int ld, int T, int q_off, int k_off, int v_off, const float* q_w, const float* k_w, const int* pos,
@@ -944,7 +943,7 @@ B200_API int b200_row_qkv_finish(const float* in, int ld, int T, int q_off, int 
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
       if (e != cudaSuccess) return (int)e;
     }
-    return launch_pdl(kern, dim3(T), dim3(256), smem, st, a, k, v);
+    return launch_pdl(kern, dim3(T), dim3(T <= 2 * 148 && (H + G) * dim >= 2048 ? 512 : 256), smem, st, a, k, v);
   };
   if (cache_f32)
     return vec ? run(row_qkv_finish_kernel<float, true>, (float*)kc, (float*)vc) : run(row_qkv_finish_kernel<float, false>, (float*)kc, (float*)vc);
