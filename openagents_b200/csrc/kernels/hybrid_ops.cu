@@ -787,6 +787,10 @@ __global__ void __launch_bounds__(512) row_qkv_finish_kernel(const RowQkvArgs a,
   extern __shared__ __align__(16) float row_s[];           // q row | k row
   __shared__ float red[2][16];
   pdl_trigger();
+  if (VEC && blockIdx.x < 8 && threadIdx.x < 2) {          // the weights, needed behind the sums, into L2 now
+    const float* w = threadIdx.x ? a.k_w : a.q_w;
+    if (w) prefetch_l2(w, (threadIdx.x ? a.G : a.H) * a.dim * 4);
+  }
   pdl_wait();
   const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nt = blockDim.x, nw = nt >> 5;
   const float* row = a.in + (size_t)t * a.ld;

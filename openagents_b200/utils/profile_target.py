@@ -14,7 +14,8 @@ pair (norm + all-gather push -> GEMM, GEMM -> reduce-scatter); ``zero_adamw``: t
 ``gemm_mn``: the weight-gradient GEMM (both operands read token-major); ``norm_slots``: the RMSNorm that is the tensor-parallel
 all-reduce, 64 rows of 4096 on a one-rank heap; ``gla_chunked`` / ``gla_decode``: gated linear attention of an 8B-size hybrid layer, a
 2048-token prompt / a decode step of 64 sequences; ``mixed_finish`` / ``mixed_prefill`` / ``mixed_decode``: attention with mixed heads at
-the same sizes (32 heads, 8 key heads of 128).
+the same sizes (32 heads, 8 key heads of 128); ``delta_chunked`` / ``delta_decode`` and ``ssd_chunked`` / ``ssd_decode``: the generalized delta rule (64 heads
+of 64 x 64) and state-space duality (128 heads of 64, state 128) of an 8B-size Tekosun layer, likewise.
 """
 from __future__ import annotations
 
@@ -240,6 +241,25 @@ def main():
                 dk ** -0.5, 1e-6)
         ws = torch.empty(ops.gla_chunk_bytes(T, B, H, dk, dv, r), dtype=torch.uint8, device=DEV)
         fn = (lambda: ops.gla_chunked(*args, per, ws, out_bf16=out)) if case == "gla_chunked" else (lambda: ops.gla_recurrent(*args, out_bf16=out))
+    elif case in ("delta_chunked", "delta_decode", "ssd_chunked", "ssd_decode"):
+        B, T = (1, 2048) if case.endswith("chunked") else (64, 64)
+        per = T // B
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=DEV)
+        rnd = lambda *s: torch.randn(*s, device=DEV)
+        seqs = (i32([per * b for b in range(B)]), i32([per] * B), i32([per + 1] * B), i32(list(range(B))), B)
+        if case.startswith("delta"):
+            H, D, r, decay = 64, 64, 128, math.exp(-0.5)
+            hd = H * D
+            args = (rnd(T, 5 * hd + r), tuple(i * hd for i in range(6)), r, rnd(hd, r).bfloat16(), rnd(hd) - 3, rnd(hd), rnd(hd), rnd(B, H, D, D), *seqs, H, D, D, D, decay, 1e-6,
+                    torch.empty((T, hd), dtype=torch.bfloat16, device=DEV))
+            ws = torch.empty(ops.delta_chunk_bytes(T, B, H, D, D, decay), dtype=torch.uint8, device=DEV)
+            fn = (lambda: ops.delta_chunked(*args, max_q=T, ws=ws)) if case == "delta_chunked" else (lambda: ops.delta_recurrent(*args))
+        else:
+            H, P, N, G, taps = 128, 64, 128, 1, 4
+            inner, CC = H * P, H * P + 2 * G * N
+            args = (rnd(T, inner + CC + H), inner, inner + CC, rnd(CC, taps), rnd(CC), rnd(H) - 3, rnd(H), rnd(H), rnd(B, H, N, P), rnd(B, taps, CC), *seqs, H, P, N, G, P, rnd(T, inner))
+            ws = torch.empty(max(ops.ssd_prefill_bytes(T, B, H, P, N, G), ops.ssd_decode_bytes(B, H, P, N, G)), dtype=torch.uint8, device=DEV)
+            fn = (lambda: ops.ssd_prefill(*args, max_q=T, ws=ws)) if case == "ssd_chunked" else (lambda: ops.ssd_decode(*args, ws=ws))
     else:
         raise SystemExit(f"unknown case {case}")
     fn()                                  # warm-up outside the profiled range
