@@ -307,7 +307,7 @@ class CudaBackend(Backend):
 
 def open_backend(path: str, backend: str = "cuda", device="cuda:0", **engine_args) -> Backend:
     """The backend for a model (GGUF file or checkpoint folder) by its architecture: the paged engines (or the fp32 oracle) for the
-    llama and gpt-oss families, the paged hybrid engine for folirax, pesorax and kazolorn, the recompute backends for GPT-2-shape checkpoints."""
+    llama and gpt-oss families, the paged hybrid engine for folirax, pesorax, kazolorn and tekosun, the recompute backends for GPT-2-shape checkpoints."""
     from ..models.config import HYBRID_ARCHS
     from ..models.registry import peek_architecture
     arch = peek_architecture(path)
