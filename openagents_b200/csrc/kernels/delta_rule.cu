@@ -37,7 +37,7 @@ constexpr int kDeltaDim = 256;        // most key channels of a head
 constexpr int kDeltaRank = 1024;      // most ranks of the decay's projection
 constexpr float kUnitEps = 1e-6f;
 
-__device__ __forceinline__ float sigmoid_f(float x) { return __fdividef(1.f, 1.f + expf(-x)); }
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 // The same on the hardware's exponential and reciprocal (some 1e-7 relative), for operands that are rounded to two bf16 numbers.
 __device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 
@@ -181,10 +181,7 @@ __global__ void __launch_bounds__(NT, NT == 128 ? 3 : 2) delta_recurrent_kernel(
   };
   // what a token does to the state, in three steps with a barrier between them
   auto low_rank = [&](const float* row) {
-    for (int r = tid; r < a.rank8; r += NT) {
-      const float x = row[rka + 2 * W + r], e = expf(-2.f * fabsf(x));
-      s_x[r] = copysignf(__fdividef(1.f - e, 1.f + e), x);      // tanh
-    }
+    for (int r = tid; r < a.rank8; r += NT) s_x[r] = tanhf(row[rka + 2 * W + r]);
   };
   auto decay_logits = [&]() {
     if (ch >= dim) return;
